@@ -46,6 +46,10 @@ extern "C" {
 #define MK_TYPE_Q3_K 11
 #define MK_TYPE_Q5_K 13
 #define MK_TYPE_BF16 30
+/* mk_load_config.compute_dtype */
+#define MK_COMPUTE_DEFAULT 0 /* what the checkpoint's format is served with */
+#define MK_COMPUTE_BF16 1    /* 16-bit matrix operands, 32-bit accumulation */
+#define MK_COMPUTE_F32 2     /* everything in 32-bit */
 
 /* Matmul path selection for mk_k_qmatmul. */
 #define MK_PATH_AUTO 0
@@ -91,6 +95,11 @@ typedef struct mk_load_config {
      * schedules its own sequences (data-parallel lanes) and each MoE layer sends the routed token rows to the rank that
      * holds the expert and the outputs back (dispatch / combine all-to-all over NVLink peer memory). */
     int32_t ep_mode;
+    /* Models with recurrent layers keep one state slot per live sequence: how many (0 = max_batch_lanes). */
+    int32_t state_slots;
+    /* Safetensors checkpoints: MK_COMPUTE_DEFAULT or MK_COMPUTE_BF16 = bfloat16 matrix operands with 32-bit accumulation;
+     * MK_COMPUTE_F32 = everything in 32-bit, K/V pages included (no tensor cores). */
+    int32_t compute_dtype;
 } mk_load_config;
 
 /* CausalLm::runtime_spec (src/architecture.rs:312-316,1039). */
@@ -154,7 +163,11 @@ typedef struct mk_gguf_summary {
 } mk_gguf_summary;
 int32_t mk_gguf_inspect(const char* path, mk_gguf_summary* out);
 
-/* LoadedRuntime::load (src/runtime.rs:104-145) for a GGUF file. */
+/* LoadedRuntime::load (src/runtime.rs:104-145): loads a checkpoint with the registered format that recognises it - a GGUF file
+ * (first shard of a family), or a folder with config.json and model.safetensors whose config names a registered
+ * architecture. */
+int32_t mk_model_load(const char* path, const mk_load_config* cfg, mk_model** out);
+/* The same under its older name. */
 int32_t mk_model_load_gguf(const char* path, const mk_load_config* cfg, mk_model** out);
 /* A host-only model with deterministic one-hot logits (next token after feeding token t at position p
  * is (31 t + 7 p + 3) mod vocab): drives the scheduler, the KV pool and the prefix cache without a GPU,
@@ -239,6 +252,20 @@ typedef struct mk_lane_sampling {
     float u;
 } mk_lane_sampling;
 int32_t mk_forward_set_sampling(mk_model* m, const mk_lane_sampling* lanes, int32_t n_lanes);
+
+/* Which rows of the NEXT forward with MK_FWD_WANT_LOGITS are projected to logits: counts[i] row numbers of lane i (0 = its
+ * first token of this forward; a count may be 0), concatenated in `rows`.  mk_read_output then returns one row per number,
+ * lanes in order.  Default: every lane's last row.  Forgotten after one forward. */
+int32_t mk_forward_set_logit_rows(mk_model* m, const int32_t* counts, const int32_t* rows, int32_t n_lanes);
+
+/* Keep the residual stream after every layer (f32) of the following forwards on the device / copy those of the last forward:
+ * [layers][tokens][hidden], `capacity` floats of room, *n_tokens receives the tokens of that forward.  Safetensors
+ * checkpoints only. */
+int32_t mk_model_capture_residuals(mk_model* m, int32_t on);
+int32_t mk_model_read_residuals(mk_model* m, float* out, int64_t capacity, int32_t* n_tokens);
+
+/* Recurrent-state slots of the model (0 when it keeps no recurrent state) and how many are held by sessions. */
+int32_t mk_state_slots_query(mk_model* m, int32_t* total, int32_t* in_use);
 
 #define MK_FWD_WANT_LOGITS 1u  /* copy [lanes, vocab] f32 logits to the host at the barrier */
 #define MK_FWD_WANT_TOKENS 2u  /* on-device greedy selection, one u32 per lane */

@@ -16,6 +16,7 @@ MK_OK, MK_KV_EXHAUSTED = 0, 1
 TYPE_F32, TYPE_F16, TYPE_Q8_0, TYPE_Q4_K, TYPE_Q6_K = 0, 1, 8, 12, 14
 TYPE_Q4_0, TYPE_Q5_0, TYPE_Q5_1, TYPE_Q2_K, TYPE_Q3_K, TYPE_Q5_K, TYPE_BF16 = 2, 6, 7, 10, 11, 13, 30
 PATH_AUTO, PATH_GEMV, PATH_TENSOR, PATH_HALF, PATH_STREAM = 0, 1, 2, 3, 4
+COMPUTE_DEFAULT, COMPUTE_BF16, COMPUTE_F32 = 0, 1, 2
 FWD_WANT_LOGITS, FWD_WANT_TOKENS = 1, 2
 
 
@@ -31,7 +32,8 @@ class LoadConfig(C.Structure):
     _fields_ = [("device_ordinal", C.c_int32), ("block_tokens", C.c_int32), ("slab_blocks", C.c_int32),
                 ("kv_capacity_tokens", C.c_int64), ("prefix_capacity_tokens", C.c_int64), ("kv_dtype", C.c_int32),
                 ("max_batch_tokens", C.c_int32), ("max_batch_lanes", C.c_int32), ("matmul_path", C.c_int32),
-                ("ep_rank", C.c_int32), ("ep_size", C.c_int32), ("ep_mode", C.c_int32)]
+                ("ep_rank", C.c_int32), ("ep_size", C.c_int32), ("ep_mode", C.c_int32), ("state_slots", C.c_int32),
+                ("compute_dtype", C.c_int32)]
 
 
 class GgufSummary(C.Structure):
@@ -144,6 +146,7 @@ SIGNATURES = {
     "mk_last_error": (C.c_char_p, []),
     "mk_version": (C.c_char_p, []),
     "mk_device_count": (_i32, []),
+    "mk_model_load": (_i32, [C.c_char_p, C.POINTER(LoadConfig), C.POINTER(P)]),
     "mk_model_load_gguf": (_i32, [C.c_char_p, C.POINTER(LoadConfig), C.POINTER(P)]),
     "mk_model_new_fake": (_i32, [_i32, _i32, C.POINTER(LoadConfig), _i64, C.POINTER(P)]),
     "mk_model_fake_inject": (_i32, [P, _i32, _i64]),
@@ -249,6 +252,10 @@ SIGNATURES = {
     "mk_k_sample": (_i32, [P, _i32, _i32, P, _i32, P]),
     "mk_k_penalties": (_i32, [P, _i32, P, _i32, C.c_float, P, _i32, C.c_float, C.c_float]),
     "mk_forward_set_sampling": (_i32, [P, P, _i32]),
+    "mk_forward_set_logit_rows": (_i32, [P, P, P, _i32]),
+    "mk_model_capture_residuals": (_i32, [P, _i32]),
+    "mk_model_read_residuals": (_i32, [P, P, _i64, C.POINTER(_i32)]),
+    "mk_state_slots_query": (_i32, [P, C.POINTER(_i32), C.POINTER(_i32)]),
     "mk_k_moe_route": (_i32, [P, _i32, _i32, _i32, P, P]),
 }
 

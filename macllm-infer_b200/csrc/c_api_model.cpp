@@ -3,7 +3,7 @@
 #include "../../include/macllm_b200.h"
 #include "c_api_util.h"
 #include "engine.h"
-#include "model.h"
+#include "model_registry.h"
 #include "prefix_cache.h"
 #include <cstring>
 
@@ -12,6 +12,7 @@ using namespace mk;
 struct mk_model {
     std::unique_ptr<PagedLm> lm;
     std::vector<mk_lane_sampling> sampling;  // settings of the next forward (mk_forward_set_sampling)
+    std::vector<int32_t> row_counts, rows;   // logit rows of the next forward (mk_forward_set_logit_rows)
 };
 struct mk_session { std::unique_ptr<LmSession> s; };
 struct mk_reservation { std::unique_ptr<LmReservation> r; };
@@ -81,6 +82,10 @@ ModelConfig to_model_config(const mk_load_config* cfg) {
         c.ep_mode = cfg->ep_mode;
         if (c.ep_mode != 0 && c.ep_mode != 1) throw std::runtime_error("ep_mode must be 0 or 1");
     }
+    if (cfg->state_slots < 0) throw std::runtime_error("state_slots must not be negative");
+    c.state_slots = cfg->state_slots;
+    if (cfg->compute_dtype < MK_COMPUTE_DEFAULT || cfg->compute_dtype > MK_COMPUTE_F32) throw std::runtime_error("compute_dtype is none of MK_COMPUTE_*");
+    c.compute_f32 = cfg->compute_dtype == MK_COMPUTE_F32;
     return c;
 }
 
@@ -90,53 +95,23 @@ extern "C" {
 
 // ------------------------------------------------------------------------------------------ model
 
-int32_t mk_gguf_inspect(const char* path, mk_gguf_summary* out) {
+int32_t mk_model_load(const char* path, const mk_load_config* cfg, mk_model** out) {
     return guarded([&] {
-        if (path == nullptr || out == nullptr) throw std::runtime_error("mk_gguf_inspect: null argument");
-        GgufFile f(path);
-        ModelSpec s = model_spec_from_gguf(f);
-        GgufAudit a = validate_decoder_tensors(f, s);
-        memset(out, 0, sizeof *out);
-        strncpy(out->architecture, s.arch.c_str(), sizeof out->architecture - 1);
-        out->n_layers = s.layers;
-        out->hidden_size = s.hidden;
-        out->q_heads = s.q_heads;
-        out->kv_heads = s.kv_heads;
-        out->head_dim = s.head_dim;
-        out->rotary_dim = s.rotary_dim;
-        out->ffn_size = s.ffn;
-        out->vocab_size = s.vocab;
-        out->max_context = s.max_context;
-        out->experts = s.experts;
-        out->experts_used = s.experts_used;
-        out->expert_ffn_size = s.expert_ffn;
-        out->tied_embeddings = s.tied ? 1 : 0;
-        for (const LayerSpec& l : s.layer) {
-            out->sliding_layers += l.sliding ? 1 : 0;
-            out->nope_layers += l.rope ? 0 : 1;
-            out->qk_norm |= l.qk_norm ? 1 : 0;
-        }
-        out->tensors_in_file = a.tensors_in_file;
-        out->matrices = a.matrices;
-        out->vectors = a.vectors;
-        out->matrix_bytes = a.matrix_bytes;
-    });
-}
-
-int32_t mk_model_load_gguf(const char* path, const mk_load_config* cfg, mk_model** out) {
-    return guarded([&] {
+        if (path == nullptr || out == nullptr) throw std::runtime_error("mk_model_load: null argument");
         require_device();
         auto m = std::make_unique<mk_model>();
-        m->lm = std::make_unique<Model>(path, to_model_config(cfg));
+        m->lm = load_model(path, to_model_config(cfg));
         *out = m.release();
     });
 }
+
+int32_t mk_model_load_gguf(const char* path, const mk_load_config* cfg, mk_model** out) { return mk_model_load(path, cfg, out); }
 
 int32_t mk_model_new_fake(int32_t vocab, int32_t max_context, const mk_load_config* cfg, int64_t fail_forward_at, mk_model** out) {
     return guarded([&] {
         ModelConfig c = to_model_config(cfg);
         auto fake = std::make_unique<FakeLm>(vocab, max_context, c.block_tokens, c.slab_blocks, c.kv_capacity_tokens,
-                                             c.prefix_capacity_tokens);
+                                             c.prefix_capacity_tokens, c.state_slots);
         if (fail_forward_at >= 0) fake->fail_forward_at(fail_forward_at);
         auto m = std::make_unique<mk_model>();
         m->lm = std::move(fake);
@@ -164,26 +139,27 @@ int32_t mk_model_free(mk_model* m) {
     return guarded([&] { delete m; });
 }
 
-int32_t mk_ep_unique_id(uint8_t* id_out) {
-    return guarded([&] {
-        require_device();
-        EpComm::unique_id(id_out);
-    });
-}
-
 int32_t mk_model_ep_init(mk_model* m, const uint8_t* id) {
-    return guarded([&] {
-        Model* model = dynamic_cast<Model*>(m->lm.get());
-        if (model == nullptr) throw std::runtime_error("mk_model_ep_init needs a GGUF model");
-        model->ep_init(id);
-    });
+    return guarded([&] { m->lm->ep_init(id); });
 }
 
 int32_t mk_model_ep_idle_tick(mk_model* m) {
+    return guarded([&] { m->lm->ep_idle_tick(); });
+}
+
+int32_t mk_model_capture_residuals(mk_model* m, int32_t on) {
+    return guarded([&] { m->lm->capture_residuals(on != 0); });
+}
+
+int32_t mk_model_read_residuals(mk_model* m, float* out, int64_t capacity, int32_t* n_tokens) {
+    return guarded([&] { *n_tokens = m->lm->read_residuals(out, capacity); });
+}
+
+int32_t mk_state_slots_query(mk_model* m, int32_t* total, int32_t* in_use) {
     return guarded([&] {
-        Model* model = dynamic_cast<Model*>(m->lm.get());
-        if (model == nullptr) throw std::runtime_error("mk_model_ep_idle_tick needs a GGUF model");
-        model->ep_idle_tick();
+        const StateSlots* s = m->lm->state_slots();
+        *total = s ? s->capacity() : 0;
+        *in_use = s ? s->in_use() : 0;
     });
 }
 
@@ -307,6 +283,21 @@ int32_t mk_forward_set_sampling(mk_model* m, const mk_lane_sampling* lanes, int3
     });
 }
 
+int32_t mk_forward_set_logit_rows(mk_model* m, const int32_t* counts, const int32_t* rows, int32_t n_lanes) {
+    return guarded([&] {
+        if (n_lanes < 0 || (n_lanes > 0 && counts == nullptr)) throw std::runtime_error("mk_forward_set_logit_rows: bad arguments");
+        int64_t total = 0;
+        for (int32_t i = 0; i < n_lanes; ++i) {
+            if (counts[i] < 0) throw std::runtime_error("mk_forward_set_logit_rows: a negative row count");
+            total += counts[i];
+        }
+        if (total > 0 && rows == nullptr) throw std::runtime_error("mk_forward_set_logit_rows: bad arguments");
+        m->row_counts.assign(counts, counts + n_lanes);
+        m->rows.assign(rows, rows + total);
+        m->rows.push_back(0);  // so that the address of an empty list is not null
+    });
+}
+
 int32_t mk_forward_batch_reserved(mk_model* m, const mk_lane* lanes, int32_t n_lanes, mk_reservation* r, uint32_t flags) {
     return guarded([&] {
         if (r == nullptr) throw std::runtime_error("forward needs a KV reservation");
@@ -315,6 +306,18 @@ int32_t mk_forward_batch_reserved(mk_model* m, const mk_lane* lanes, int32_t n_l
         std::vector<LmLane> ll = to_lanes(lanes, n_lanes);
         std::vector<mk_lane_sampling> sampling = std::move(m->sampling);  // one forward only
         m->sampling.clear();
+        std::vector<int32_t> row_counts = std::move(m->row_counts), rows = std::move(m->rows);
+        m->row_counts.clear();
+        m->rows.clear();
+        if (!row_counts.empty()) {
+            if ((int32_t)row_counts.size() != n_lanes) throw std::runtime_error("logit rows cover another number of lanes than the forward");
+            const int32_t* at = rows.data();
+            for (int32_t i = 0; i < n_lanes; ++i) {
+                ll[(size_t)i].logit_rows = at;
+                ll[(size_t)i].n_logit_rows = row_counts[(size_t)i];
+                at += row_counts[(size_t)i];
+            }
+        }
         if (!sampling.empty()) {
             if ((int32_t)sampling.size() != n_lanes) throw std::runtime_error("sampling settings cover another number of lanes than the forward");
             for (int32_t i = 0; i < n_lanes; ++i) {

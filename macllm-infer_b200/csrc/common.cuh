@@ -26,6 +26,7 @@ enum ActKind : int { ACT_Q8K = 0, ACT_Q80 = 1 };
 //         p2 = scales [rows*nb][16] (int8), p3 = d [rows*nb] (f16)
 //  Q8_0 : p0 = qs [rows][cols] (int8), p1 = d [rows][cols/32] (f16)
 //  F32  : p0 = values
+//  BF16 : p0 = values (read in place by the embedding gather only)
 struct QWeight {
     int type = QT_F32;
     int64_t rows = 0, cols = 0;

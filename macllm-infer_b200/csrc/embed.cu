@@ -28,6 +28,8 @@ __global__ void embed_kernel(QWeight W, const uint32_t* ids, float scale, float*
         float v;
         if (W.type == QT_F32) {
             v = ((const float*)W.p0)[row * cols + k];
+        } else if (W.type == QT_BF16) {
+            v = __uint_as_float((uint32_t)((const uint16_t*)W.p0)[row * cols + k] << 16);
         } else if (W.type == QT_Q8_0) {
             int nb = cols / 32;
             v = __half2float(((const __half*)W.p1)[row * nb + k / 32]) * (float)((const int8_t*)W.p0)[row * cols + k];

@@ -1,0 +1,135 @@
+// See mixer_spec.h.
+#include "mixer_spec.h"
+#include <cmath>
+#include <map>
+#include <stdexcept>
+
+namespace mk {
+
+namespace {
+
+std::map<std::string, MixerSpecReader>& readers() {
+    static std::map<std::string, MixerSpecReader> all;
+    return all;
+}
+
+int size_of(const Json& v, int lo = 1, int hi = 1 << 24) {
+    const int64_t n = v.integer();
+    if (n < lo || n > hi) throw std::runtime_error(v.where() + " is out of range");
+    return (int)n;
+}
+
+RotarySpec read_rotary(const Json& mixer, int head_dim) {
+    RotarySpec r;
+    const Json* rot = mixer.find("rot");
+    if (rot == nullptr || rot->is_null()) return r;
+    r.dims = size_of(rot->at("dims"), 0, head_dim);
+    if (r.dims % 2 != 0) throw std::runtime_error(rot->where() + ".dims must be even");
+    r.base = rot->at("base").number();
+    if (!(r.base > 0)) throw std::runtime_error(rot->where() + ".base must be positive");
+    const Json* s = rot->find("scaling");
+    if (s != nullptr && !s->is_null()) {
+        r.scaled = true;
+        r.factor = s->at("factor").number();
+        r.low = s->at("low").number();
+        r.high = s->at("high").number();
+        r.original = s->at("original").number();
+        if (!(r.factor > 0 && r.original > 0)) throw std::runtime_error(s->where() + " needs a positive factor and original context");
+    }
+    return r;
+}
+
+void check_groups(const Json& where, int heads, int kv_heads) {
+    if (heads % kv_heads != 0) throw std::runtime_error(where.where() + ": heads must be a multiple of kv_heads");
+}
+
+// Sizilorn: WKV time-mixing layers and layers that run gated attention beside the gated delta rule, Dynamic Tanh norms, and
+// a token input of its own for every layer.
+MixerSpec read_sizilorn(const Json& c, const SafetensorsFile& f) {
+    MixerSpec s;
+    s.arch = "Sizilorn";
+    s.vocab = size_of(c.at("vocab"));
+    s.width = size_of(c.at("width"));
+    s.norm = NormKind::DynTanh;
+    s.eps = (float)c.at("norm").at("eps").number();
+    if (!(s.eps >= 0.f)) throw std::runtime_error("config norm.eps must not be negative");
+    const Json* side = c.find("token_side");
+    if (side != nullptr && !side->is_null()) s.side_dim = size_of(side->at("dim"));
+    const auto& layers = c.at("layers").items();
+    if (layers.empty()) throw std::runtime_error("config lists no layers");
+    for (size_t i = 0; i < layers.size(); ++i) {
+        const Json& j = layers[i];
+        const Json& m = j.at("mixer");
+        const std::string type = j.at("type").str();
+        MixerLayerSpec l;
+        if (type == "wkv") {
+            l.kind = MixerKind::Wkv;
+            l.wkv.heads = size_of(m.at("heads"));
+            l.wkv.dim = size_of(m.at("dim"));
+            const std::string w1 = "l" + std::to_string(i) + ".mix.w1";
+            const StTensor* t = f.find(w1);
+            if (t == nullptr || t->shape.size() != 2) throw std::runtime_error("tensor `" + w1 + "` must be a matrix");
+            l.wkv.rank = (int)t->shape[0];
+        } else if (type == "parallel") {
+            l.kind = MixerKind::Parallel;
+            const Json& a = m.at("left");
+            l.attn.heads = size_of(a.at("heads"));
+            l.attn.kv_heads = size_of(a.at("kv_heads"));
+            l.attn.dim = size_of(a.at("dim"));
+            l.attn.vdim = size_of(a.at("vdim"));
+            l.attn.scale = (float)a.at("scale").number();
+            l.attn.rot = read_rotary(a, l.attn.dim);
+            check_groups(a, l.attn.heads, l.attn.kv_heads);
+            const Json& d = m.at("right");
+            l.delta.heads = size_of(d.at("heads"));
+            l.delta.kv_heads = size_of(d.at("kv_heads"));
+            l.delta.dim = size_of(d.at("dim"));
+            l.delta.vdim = size_of(d.at("vdim"));
+            l.delta.taps = size_of(d.at("conv"));
+            check_groups(d, l.delta.heads, l.delta.kv_heads);
+        } else {
+            throw std::runtime_error(j.where() + ".type `" + type + "` is not a known mixer");
+        }
+        const Json* mlp = j.find("mlp");
+        if (mlp != nullptr && !mlp->is_null()) {
+            if (mlp->at("kind").str() != "dense") throw std::runtime_error(mlp->where() + ".kind `" + mlp->at("kind").str() + "` is not supported");
+            l.ff = size_of(mlp->at("ff"));
+        }
+        s.layers.push_back(l);
+    }
+    return s;
+}
+
+const RegisterMixerArchitecture register_sizilorn("Sizilorn", read_sizilorn);
+
+}  // namespace
+
+RegisterMixerArchitecture::RegisterMixerArchitecture(const std::string& name, MixerSpecReader reader) { readers()[name] = std::move(reader); }
+
+MixerSpec read_mixer_spec(const Json& config, const SafetensorsFile& f) {
+    const std::string arch = config.at("architecture").str();
+    auto it = readers().find(arch);
+    if (it == readers().end()) throw std::runtime_error("architecture `" + arch + "` is not supported");
+    return it->second(config, f);
+}
+
+std::vector<double> rotary_frequencies(const RotarySpec& r) {
+    std::vector<double> f((size_t)(r.dims / 2));
+    const double two_pi = 2.0 * std::acos(-1.0);
+    for (int i = 0; i < r.dims / 2; ++i) {
+        double v = std::pow(r.base, -2.0 * i / r.dims);
+        if (r.scaled) {
+            const double wavelength = two_pi / v;
+            if (wavelength > r.original / r.low) {
+                v /= r.factor;
+            } else if (!(wavelength < r.original / r.high)) {
+                const double s = (r.original / wavelength - r.low) / (r.high - r.low);
+                v = (1.0 - s) * v / r.factor + s * v;
+            }
+        }
+        f[(size_t)i] = v;
+    }
+    return f;
+}
+
+}  // namespace mk

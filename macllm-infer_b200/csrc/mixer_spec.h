@@ -1,0 +1,74 @@
+// Decoders described layer by layer by a config.json: every layer names its sequence mixer, that mixer's sizes and its
+// feed-forward.  The reader of one architecture turns its config.json into this description; the executor (mixer_lm.h) and
+// the kernels see nothing else of it.
+#pragma once
+#include "json.h"
+#include "safetensors_file.h"
+#include <functional>
+#include <string>
+#include <vector>
+
+namespace mk {
+
+enum class NormKind { None, DynTanh };
+
+// Rotary positions on the first `dims` dimensions of a head; dims = 0: none.
+struct RotarySpec {
+    int dims = 0;
+    double base = 10000.0;
+    bool interleaved = true;  // pairs (2i, 2i + 1); false: (i, i + dims / 2)
+    // stretch of the long wavelengths: below `low` turns over the original context by `factor`, above `high` not at all
+    bool scaled = false;
+    double factor = 1.0, low = 1.0, high = 1.0, original = 1.0;
+    bool operator==(const RotarySpec& o) const {
+        return dims == o.dims && base == o.base && interleaved == o.interleaved && scaled == o.scaled &&
+               (!scaled || (factor == o.factor && low == o.low && high == o.high && original == o.original));
+    }
+};
+// The frequency of every pair, in radians per position.
+std::vector<double> rotary_frequencies(const RotarySpec& r);
+
+// Grouped-query attention; per-head query / key RMS norm before the rotation, a sigmoid gate per head on the output.
+struct AttentionSpec {
+    int heads = 0, kv_heads = 0, dim = 0, vdim = 0;
+    float scale = 1.f;
+    RotarySpec rot;
+};
+
+// Gated delta rule behind a short causal convolution; head h reads query / key head h / (heads / kv_heads).
+struct DeltaSpec {
+    int heads = 0, kv_heads = 0, dim = 0, vdim = 0, taps = 1;
+};
+
+// Time mixing with a data-dependent decay per key channel and a bonus for the current token.
+struct WkvSpec {
+    int heads = 0, dim = 0, rank = 0;  // rank of the decay's low-rank projection
+};
+
+enum class MixerKind { Wkv, Parallel };  // Parallel: attention and the gated delta rule side by side
+
+struct MixerLayerSpec {
+    MixerKind kind = MixerKind::Wkv;
+    WkvSpec wkv;
+    AttentionSpec attn;
+    DeltaSpec delta;
+    int ff = 0;  // width of the gated feed-forward, 0: the layer has none
+};
+
+struct MixerSpec {
+    std::string arch;
+    int vocab = 0, width = 0, side_dim = 0;
+    float eps = 1e-6f;
+    NormKind norm = NormKind::DynTanh;
+    std::vector<MixerLayerSpec> layers;
+};
+
+// Reads `config` (and sizes that only the tensors know) for the architecture it names.
+MixerSpec read_mixer_spec(const Json& config, const SafetensorsFile& f);
+
+using MixerSpecReader = std::function<MixerSpec(const Json& config, const SafetensorsFile& f)>;
+struct RegisterMixerArchitecture {
+    RegisterMixerArchitecture(const std::string& name, MixerSpecReader reader);
+};
+
+}  // namespace mk

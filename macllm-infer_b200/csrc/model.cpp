@@ -90,14 +90,11 @@ ModelSpec model_spec_from_gguf(const GgufFile& f) {
 
 // ---------------------------------------------------------------------------- load
 
-Model::Model(const std::string& gguf_path, const ModelConfig& cfg) : cfg_(cfg) {
-    int ndev = 0;
-    if (cudaGetDeviceCount(&ndev) != cudaSuccess || ndev <= 0) {
-        cudaGetLastError();
-        throw std::runtime_error("no usable CUDA device: this library has no CPU fallback");
-    }
-    if (cfg.device < 0 || cfg.device >= ndev) throw std::runtime_error("device ordinal out of range");
-    MK_CUDA(cudaSetDevice(cfg.device));
+static const std::vector<const char*> kclass_names = {"qgemm_tc", "hgemm_tc", "qstream_tc", "qgemv", "paged_attention", "add_norm_quant", "rope_kv_scatter",
+                                                      "actmul_quant", "embed", "build_batch", "argmax", "moe", "hgemm_tc_splitk", "ep_exchange"};
+
+Model::Model(const std::string& gguf_path, const ModelConfig& cfg) : DeviceLm(cfg, kclass_names) {
+    open_device();
     GgufFile f(gguf_path);
     ms_ = model_spec_from_gguf(f);
     validate_decoder_tensors(f, ms_);  // before any device memory is touched
@@ -114,11 +111,9 @@ Model::Model(const std::string& gguf_path, const ModelConfig& cfg) : cfg_(cfg) {
     if (f.has("tokenizer.ggml.eos_token_id")) spec_.stop_ids.push_back((uint32_t)f.get_int("tokenizer.ggml.eos_token_id"));
     bool any_sliding = false;
     for (const LayerSpec& l : ms_.layer) any_sliding |= l.sliding;
-    init_pool(cfg.block_tokens, cfg.slab_blocks, cfg.kv_capacity_tokens, cfg.prefix_capacity_tokens, !any_sliding);
+    init_pool(cfg.block_tokens, cfg.slab_blocks, cfg.kv_capacity_tokens, cfg.prefix_capacity_tokens,
+              any_sliding ? "sliding-window layers" : nullptr);
 
-    MK_CUDA(cudaStreamCreateWithFlags(&stream_, cudaStreamNonBlocking));
-    MK_CUDA(cudaEventCreate(&ev_start_));
-    MK_CUDA(cudaEventCreate(&ev_stop_));
     load_weights(f);
 
     const int64_t esz = cfg.kv_f16 ? 2 : 4;
@@ -137,16 +132,6 @@ Model::Model(const std::string& gguf_path, const ModelConfig& cfg) : cfg_(cfg) {
     const int64_t P = moe ? (int64_t)T * ms_.experts_used : 0;
     const int fw = moe ? ms_.expert_ffn : ms_.ffn;
     const int64_t frows = moe ? P : T;
-    cu_.alloc((size_t)(B + 1) * 4);
-    pos_.alloc((size_t)T * 4);
-    tok_lane_.alloc((size_t)T * 4);
-    slots_.alloc((size_t)T * 8);
-    last_.alloc((size_t)B * 4);
-    tile_lane_.alloc((size_t)(T + B) * 4);
-    tile_row_.alloc((size_t)(T + B) * 4);
-    ntiles_.alloc(4);
-    err_.alloc(4);
-    err_.zero(stream_);
     h_.alloc((size_t)T * ms_.hidden * 4);
     qkv_.alloc((size_t)T * (AW + 2 * KW) * 4);
     attn_.alloc((size_t)T * AW * 4);
@@ -173,10 +158,6 @@ Model::Model(const std::string& gguf_path, const ModelConfig& cfg) : cfg_(cfg) {
             ep_gather_.alloc((size_t)cfg_.ep_size * T * ms_.hidden * 4);
         }
     }
-    logits_.alloc((size_t)B * ms_.vocab * 4);
-    tokens_.alloc((size_t)B * 4);
-    argmax_scratch_.alloc(argmax_scratch_bytes(B));
-    argmax_scratch_.zero(stream_);
     a_qs_.alloc((size_t)T * aw);
     a_d_.alloc((size_t)T * (aw / 32 + 1) * 4);
     a_bs_.alloc((size_t)T * (aw / 16 + 1) * 2);
@@ -189,8 +170,6 @@ Model::Model(const std::string& gguf_path, const ModelConfig& cfg) : cfg_(cfg) {
     l_d_.alloc((size_t)B * (ms_.hidden / 32 + 1) * 4);
     l_bs_.alloc((size_t)B * (ms_.hidden / 16 + 1) * 2);
     l_xh_.alloc((size_t)B * ms_.hidden * 2);
-    tc_ws_.status.alloc(4);
-    tc_ws_.status.zero(stream_);
     // the largest split-K scratch any matmul of this model can ask for
     size_t partial = 0;
     auto consider = [&](const QWeight& w, int rows_t) {
@@ -203,8 +182,7 @@ Model::Model(const std::string& gguf_path, const ModelConfig& cfg) : cfg_(cfg) {
     }
     consider(ms_.tied ? token_embd_.w : output_.w, B);
     tc_ws_.partial.alloc(std::max<size_t>(partial, 1) * 4);
-    size_t stage_bytes = (size_t)B * sizeof(LaneHeader) + (size_t)(pool_->max_blocks() + B) * 4 + (size_t)T * 4 + 64 +
-                         (size_t)B * sizeof(LaneSampling) + 16;
+    size_t extra_stage = 0;
     attn_tc_ = attention_tc_supported(ms_.q_heads, ms_.kv_heads, ms_.head_dim, cfg_.block_tokens, cfg_.kv_f16);
     if (attn_tc_) {
         attn_max_entries_ = attention_tc_max_entries(B, ms_.kv_heads);
@@ -213,11 +191,9 @@ Model::Model(const std::string& gguf_path, const ModelConfig& cfg) : cfg_(cfg) {
         attn_counters_.alloc((size_t)B * ms_.kv_heads * 4);
         attn_counters_.zero(stream_);
         // work lists: key-share entries (8 ints), prefill tiles (2 ints), split one-token lanes (3 ints)
-        stage_bytes += ((size_t)(T + B) * 2 + (size_t)attn_max_entries_ * 8 + (size_t)B * 3) * 4 + 16;
+        extra_stage = ((size_t)(T + B) * 2 + (size_t)attn_max_entries_ * 8 + (size_t)B * 3) * 4 + 64;
     }
-    stage_host_.ensure(stage_bytes);
-    stage_dev_.alloc(stage_bytes);
-    out_host_.ensure((size_t)B * ms_.vocab * 4 + (size_t)B * 4 + 16);
+    alloc_tick(extra_stage);
     MK_CUDA(cudaStreamSynchronize(stream_));
     build_half_cache();
     build_qstream();
@@ -225,9 +201,6 @@ Model::Model(const std::string& gguf_path, const ModelConfig& cfg) : cfg_(cfg) {
 
 Model::~Model() {
     if (stream_) cudaStreamSynchronize(stream_);
-    if (ev_start_) cudaEventDestroy(ev_start_);
-    if (ev_stop_) cudaEventDestroy(ev_stop_);
-    if (stream_) cudaStreamDestroy(stream_);
 }
 
 void Model::upload_f32(const GgufFile& f, const std::string& name, int64_t n, DevBuf& out) {
@@ -319,7 +292,7 @@ const float* Model::ep_exchange_layer(LayerWeights& w, const LayerSpec& ls, cons
     const int EL = ep_local_experts(), H = ms_.hidden, F = ms_.expert_ffn;
     const int capacity = (int)std::min<int64_t>((int64_t)D.ranks * D.cap_rows, INT32_MAX);
     const uint32_t epoch = ep_->next_epoch();
-    int32_t* status = tc_ws_.status.as<int32_t>();
+    int32_t* status = status_.as<int32_t>();
     // the other ranks' row counts are not known on the host (a peer may run a prefill chunk while this rank decodes), and
     // a narrow chunk under many rows costs a pass over the expert's weights per chunk: always the full width
     (void)T;
@@ -428,63 +401,6 @@ void Model::rope_tables_for(double theta, const float*& cos_t, const float*& sin
     rope_.push_back(std::move(t));
 }
 
-// ---------------------------------------------------------------------------- profiling
-
-static const char* kclass_names[] = {"qgemm_tc", "hgemm_tc", "qstream_tc", "qgemv", "paged_attention", "add_norm_quant", "rope_kv_scatter", "actmul_quant",
-                                     "embed", "build_batch", "argmax", "moe", "hgemm_tc_splitk", "ep_exchange"};
-
-void Model::profile_enable(bool on) {
-    profiling_ = on;
-    if (on) for (int i = 0; i < KC_COUNT; ++i) { prof_[i] = KernelProfile{}; prof_[i].name = kclass_names[i]; }
-}
-
-void Model::prof_begin(int cls, double bytes, double flops) {
-    if (!profiling_) return;
-    ProfSpan sp;
-    sp.cls = cls;
-    sp.bytes = bytes;
-    sp.flops = flops;
-    for (cudaEvent_t* e : {&sp.a, &sp.b}) {
-        if (event_pool_.empty()) {
-            MK_CUDA(cudaEventCreate(e));
-        } else {
-            *e = event_pool_.back();
-            event_pool_.pop_back();
-        }
-    }
-    MK_CUDA(cudaEventRecord(sp.a, stream_));
-    spans_.push_back(sp);
-}
-
-void Model::prof_end() {
-    if (!profiling_ || spans_.empty()) return;
-    MK_CUDA(cudaEventRecord(spans_.back().b, stream_));
-}
-
-void Model::prof_resolve() {
-    for (ProfSpan& sp : spans_) {
-        float ms = 0.f;
-        if (cudaEventElapsedTime(&ms, sp.a, sp.b) == cudaSuccess) {
-            KernelProfile& k = prof_[sp.cls];
-            ++k.launches;
-            k.ms += ms;
-            k.bytes += sp.bytes;
-            k.flops += sp.flops;
-        } else {
-            cudaGetLastError();
-        }
-        event_pool_.push_back(sp.a);
-        event_pool_.push_back(sp.b);
-    }
-    spans_.clear();
-}
-
-std::vector<PagedLm::KernelProfile> Model::profile_query() {
-    std::vector<KernelProfile> out;
-    for (int i = 0; i < KC_COUNT; ++i) if (prof_[i].launches > 0) out.push_back(prof_[i]);
-    return out;
-}
-
 // ---------------------------------------------------------------------------- forward
 
 bool Model::tensor_path(const QWeight& W, int T) const {
@@ -507,7 +423,7 @@ HgemmScratch Model::hgemm_scratch() const {
     HgemmScratch ws;
     ws.partial = tc_ws_.partial.as<float>();
     ws.partial_floats = tc_ws_.partial.size() / 4;
-    ws.status = tc_ws_.status.as<int32_t>();
+    ws.status = status_.as<int32_t>();
     return ws;
 }
 
@@ -542,7 +458,7 @@ void Model::matmul(const DeviceWeight& DW, const ActQ& x, int T, float* y, int l
     if (tc) {
         size_t need = qgemm_tc_partial_floats(W, T);
         tc_ws_.partial.ensure(need * 4);
-        launch_qgemm_tc_scratch(W, x, T, y, ldy, scale, softcap, tc_ws_.partial.as<float>(), tc_ws_.status.as<int32_t>(), stream_);
+        launch_qgemm_tc_scratch(W, x, T, y, ldy, scale, softcap, tc_ws_.partial.as<float>(), status_.as<int32_t>(), stream_);
         launches_ += need > 0 ? 2 : 1;
     } else {
         launch_qgemv(W, x, T, y, ldy, scale, softcap, stream_);
@@ -692,7 +608,7 @@ int Model::matmul_stream(const QStreamWeight& W, const ActQ& x, int T, float* y,
                           (W2 ? (double)W2->rows * (double)(W2->cols / 256) * (W2->fmt ? 210.0 : 144.0) : 0.0);
     prof_begin(KC_QSTREAM, wbytes + 2.0 * T * W.cols + 4.0 * T * rows, 2.0 * T * rows * (double)W.cols);
     int splits = launch_qstream_tc(W, x.xh, T, y, ldy, tc_ws_.partial.as<float>(), tc_ws_.partial.size() / 4,
-                                   tc_ws_.status.as<int32_t>(), stream_, max_splits, W2);
+                                   status_.as<int32_t>(), stream_, max_splits, W2);
     prof_end();
     ++launches_;
     return splits;
@@ -701,55 +617,14 @@ int Model::matmul_stream(const QStreamWeight& W, const ActQ& x, int T, float* y,
 static int act_kind_of(const QWeight& w) { return w.type == QT_Q8_0 ? ACT_Q80 : ACT_Q8K; }
 
 void Model::run_forward(const std::vector<LmLane>& lanes, KvReservation& r, uint32_t flags) {
-    MK_CUDA(cudaSetDevice(cfg_.device));
-    const int B = (int)lanes.size();
-    int T = 0;
-    for (const LmLane& l : lanes) T += l.n_tokens;
-    if (B > cfg_.max_batch_lanes) throw std::runtime_error("batch has more lanes than max_batch_lanes");
-    if (T > cfg_.max_batch_tokens) throw std::runtime_error("batch has more tokens than max_batch_tokens");
+    Tick tick = stage_tick(lanes, r, flags);
+    const int B = tick.B, T = tick.T, R = tick.R;
+    if (R > cfg_.max_batch_lanes) throw std::runtime_error("more logit rows than max_batch_lanes");
     const int H = ms_.hidden, AW = ms_.q_heads * ms_.head_dim, KW = ms_.kv_heads * ms_.head_dim, d = ms_.head_dim;
     const int QKVW = AW + 2 * KW;
     const int bt = pool_->block_tokens();
     const int q_tile = attention_q_tile(ms_.q_heads, ms_.kv_heads);
 
-    // ---- stage the per-lane headers, block tables and token ids in one pinned buffer, one copy
-    uint8_t* hp = stage_host_.as<uint8_t>();
-    LaneHeader* hdr = reinterpret_cast<LaneHeader*>(hp);
-    size_t off_tables = (size_t)B * sizeof(LaneHeader);
-    uint32_t* tab = reinterpret_cast<uint32_t*>(hp + off_tables);
-    int n_tab = 0, tiles = 0;
-    for (int i = 0; i < B; ++i) {
-        const std::vector<KvBlockId>& blocks = r.lane_blocks((size_t)i);
-        hdr[i].start_pos = lanes[(size_t)i].start_pos;
-        hdr[i].n_tokens = lanes[(size_t)i].n_tokens;
-        hdr[i].table_off = n_tab;
-        hdr[i].n_blocks = (int32_t)blocks.size();
-        for (const KvBlockId& b : blocks) tab[n_tab++] = b.slot;
-        tiles += (lanes[(size_t)i].n_tokens + q_tile - 1) / q_tile;
-    }
-    size_t off_ids = off_tables + (size_t)n_tab * 4;
-    uint32_t* ids = reinterpret_cast<uint32_t*>(hp + off_ids);
-    int tpos = 0;
-    for (const LmLane& l : lanes) {
-        memcpy(ids + tpos, l.ids, (size_t)l.n_tokens * 4);
-        tpos += l.n_tokens;
-    }
-    size_t stage_bytes = off_ids + (size_t)T * 4;
-    // per-lane sampling settings, only when some lane does not take the plain argmax
-    bool any_stochastic = false;
-    for (const LmLane& l : lanes) any_stochastic |= l.temperature > 0.f;
-    size_t off_sampling = 0;
-    if (any_stochastic && (flags & FWD_WANT_TOKENS)) {
-        off_sampling = (stage_bytes + 15) / 16 * 16;
-        LaneSampling* sp = reinterpret_cast<LaneSampling*>(hp + off_sampling);
-        for (int i = 0; i < B; ++i) {
-            const LmLane& l = lanes[(size_t)i];
-            if (!mk::device_sampling_covers(l.temperature, l.top_k, ms_.vocab))
-                throw std::runtime_error("the device sampler covers greedy selection and 1 <= top_k <= 1024");
-            sp[i] = LaneSampling{l.temperature, l.top_k, l.top_p, l.u};
-        }
-        stage_bytes = off_sampling + (size_t)B * sizeof(LaneSampling);
-    }
     // work lists of the tensor-core attention (the same for every layer of the tick)
     size_t off_tiles = 0, off_entries = 0, off_dec = 0;
     int n_attn_tiles = 0, n_attn_entries = 0, n_attn_dec = 0;
@@ -760,48 +635,21 @@ void Model::run_forward(const std::vector<LmLane>& lanes, KvReservation& r, uint
         for (int i = 0; i < B; ++i) {
             plan_sp_[(size_t)i] = lanes[(size_t)i].start_pos;
             plan_nt_[(size_t)i] = lanes[(size_t)i].n_tokens;
-            plan_nb_[(size_t)i] = hdr[i].n_blocks;
+            plan_nb_[(size_t)i] = tick.hdr[i].n_blocks;
         }
         plan_attention_tc(plan_sp_.data(), plan_nt_.data(), plan_nb_.data(), B, ms_.q_heads, ms_.kv_heads, attn_plan_);
         n_attn_tiles = attn_plan_.n_tiles();
         n_attn_entries = attn_plan_.n_entries();
         n_attn_dec = attn_plan_.n_dec_lanes();
         if (n_attn_entries > attn_max_entries_) throw std::runtime_error("attention work list exceeds its scratch");
-        off_entries = (stage_bytes + 15) / 16 * 16;  // 32-byte records read as two 16-byte loads
-        off_tiles = off_entries + attn_plan_.entries.size() * 4;
-        off_dec = off_tiles + attn_plan_.tiles.size() * 4;
-        stage_bytes = off_dec + attn_plan_.dec_lanes.size() * 4;
-        if (stage_bytes > stage_host_.size()) throw std::runtime_error("tick staging buffer is too small");
-        if (n_attn_tiles) memcpy(hp + off_tiles, attn_plan_.tiles.data(), attn_plan_.tiles.size() * 4);
-        if (n_attn_entries) memcpy(hp + off_entries, attn_plan_.entries.data(), attn_plan_.entries.size() * 4);
-        if (n_attn_dec) memcpy(hp + off_dec, attn_plan_.dec_lanes.data(), attn_plan_.dec_lanes.size() * 4);
+        off_entries = stage_bytes(tick, attn_plan_.entries.data(), attn_plan_.entries.size() * 4);  // 32-byte records read as two 16-byte loads
+        off_tiles = stage_bytes(tick, attn_plan_.tiles.data(), attn_plan_.tiles.size() * 4);
+        off_dec = stage_bytes(tick, attn_plan_.dec_lanes.data(), attn_plan_.dec_lanes.size() * 4);
     }
-    if (stage_bytes > stage_dev_.size()) throw std::runtime_error("tick staging buffer is too small");
-    MK_CUDA(cudaEventRecord(ev_start_, stream_));
-    MK_CUDA(cudaMemcpyAsync(stage_dev_.ptr(), hp, stage_bytes, cudaMemcpyHostToDevice, stream_));
-    h2d_bytes_ += (int64_t)stage_bytes;
-    uint8_t* dp = stage_dev_.as<uint8_t>();
-
-    BatchDesc bd;
-    bd.lanes = B;
-    bd.T = T;
-    bd.max_tiles = tiles;
-    bd.hdr = reinterpret_cast<const LaneHeader*>(dp);
-    bd.tables = reinterpret_cast<const uint32_t*>(dp + off_tables);
-    bd.cu_seqlens = cu_.as<int32_t>();
-    bd.positions = pos_.as<int32_t>();
-    bd.token_lane = tok_lane_.as<int32_t>();
-    bd.slots = slots_.as<int64_t>();
-    bd.last_index = last_.as<int32_t>();
-    bd.tile_lane = tile_lane_.as<int32_t>();
-    bd.tile_row0 = tile_row_.as<int32_t>();
-    bd.n_tiles = ntiles_.as<int32_t>();
-    bd.error_flag = err_.as<int32_t>();
-    prof_begin(KC_BATCH, 0, 0);
-        launch_build_batch(bd, bt, q_tile, stream_);
-        prof_end();
-    ++launches_;
-    const uint32_t* ids_dev = reinterpret_cast<const uint32_t*>(dp + off_ids);
+    upload_tick(tick, q_tile, KC_BATCH);
+    const uint8_t* dp = tick.dp;
+    const BatchDesc& bd = tick.bd;
+    const uint32_t* ids_dev = tick.ids;
 
     // ---- copy-on-write page copies of shared partial tails (cache.rs:3042-3089)
     for (const KvCowCopy& c : r.cow_copies()) {
@@ -1087,7 +935,7 @@ void Model::run_forward(const std::vector<LmLane>& lanes, KvReservation& r, uint
                 const QStreamWeight& W = w.qs_gu;
                 prof_begin(KC_QSTREAM, (double)W.rows * (double)(W.cols / 256) * 144.0 + 2.0 * T * W.cols + 2.0 * T * ms_.ffn,
                            2.0 * T * (double)W.rows * (double)W.cols);
-                launch_qstream_tc(W, xf.xh, T, nullptr, 0, nullptr, 0, tc_ws_.status.as<int32_t>(), stream_, 1, nullptr, ls.act,
+                launch_qstream_tc(W, xf.xh, T, nullptr, 0, nullptr, 0, status_.as<int32_t>(), stream_, 1, nullptr, ls.act,
                                   f_xh_.as<__half>(), ms_.ffn);
                 prof_end();
                 ++launches_;
@@ -1134,7 +982,7 @@ void Model::run_forward(const std::vector<LmLane>& lanes, KvReservation& r, uint
             launch_f32_gemv(w.router.as<float>(), E, H, normed_.as<float>(), T, router_logits_.as<float>(), stream_);
             prof_end();
             prof_begin(KC_MOE, 4.0 * T * E + 8.0 * P, 0);
-            launch_moe_route(router_logits_.as<float>(), T, E, K, sel_e_.as<int32_t>(), sel_w_.as<float>(), tc_ws_.status.as<int32_t>(), stream_);
+            launch_moe_route(router_logits_.as<float>(), T, E, K, sel_e_.as<int32_t>(), sel_w_.as<float>(), status_.as<int32_t>(), stream_);
             prof_end();
             prof_begin(KC_MOE, 12.0 * P, 0);
             launch_moe_group(sel_e_.as<int32_t>(), T, K, E, grp_off_.as<int32_t>(), pos_of_pair_.as<int32_t>(), tok_of_pos_.as<int32_t>(),
@@ -1166,13 +1014,13 @@ void Model::run_forward(const std::vector<LmLane>& lanes, KvReservation& r, uint
                 prof_end();
                 const double gu_bytes = (double)w.qs_gu.rows * (double)(w.qs_gu.cols / 256) * 144.0;
                 prof_begin(KC_QSTREAM, gu_bytes + 2.0 * P * H + 2.0 * P * F, 2.0 * P * 2.0 * F * H);
-                launch_qstream_tc_grouped(w.qs_gu, EL, off, e_xh_.as<__half>(), P, moe_chunk_rows(T, K, E), nullptr, 0, tc_ws_.status.as<int32_t>(), stream_,
+                launch_qstream_tc_grouped(w.qs_gu, EL, off, e_xh_.as<__half>(), P, moe_chunk_rows(T, K, E), nullptr, 0, status_.as<int32_t>(), stream_,
                                           ls.act, f_xh_.as<__half>(), F);
                 prof_end();
                 const double dn_bytes = (double)w.qs_down.rows * (double)(w.qs_down.cols / 256) * (w.qs_down.fmt ? 210.0 : 144.0);
                 prof_begin(KC_QSTREAM, dn_bytes + 2.0 * P * F + 4.0 * P * H, 2.0 * P * (double)F * H);
                 launch_qstream_tc_grouped(w.qs_down, EL, off, f_xh_.as<__half>(), P, moe_chunk_rows(T, K, E), e_down_.as<float>(), H,
-                                          tc_ws_.status.as<int32_t>(), stream_);
+                                          status_.as<int32_t>(), stream_);
                 prof_end();
             } else {
                 launch_qgemv_grouped(w.gate.w, EL, off, tok_of_pos_.as<int32_t>(), xq, e_gate_.as<float>(), F, stream_);
@@ -1188,7 +1036,7 @@ void Model::run_forward(const std::vector<LmLane>& lanes, KvReservation& r, uint
             } else if (ep && ep_->has_exchange()) {
                 launch_moe_combine_exchange(e_down_.as<float>(), sel_e_.as<int32_t>(), sel_w_.as<float>(), pos_of_pair_.as<int32_t>(), T, K,
                                             H, e0, e0 + EL, ep_->peers(), ep_->next_epoch(), down_.as<float>(),
-                                            tc_ws_.status.as<int32_t>(), stream_);
+                                            status_.as<int32_t>(), stream_);
             } else {
                 prof_begin(KC_MOE, 4.0 * P * H + 4.0 * T * H, 2.0 * P * H);
                 launch_moe_combine(e_down_.as<float>(), sel_e_.as<int32_t>(), sel_w_.as<float>(), pos_of_pair_.as<int32_t>(), T, K, H,
@@ -1225,90 +1073,35 @@ void Model::run_forward(const std::vector<LmLane>& lanes, KvReservation& r, uint
     // logits tail (src/decoder.rs:3333-3356): last rows -> final norm -> output projection -> scale -> softcap
     const DeviceWeight& head_dw = ms_.tied ? token_embd_ : output_;
     const QWeight& head = head_dw.w;
-    {
-        const bool f16_B = dense_matrices_ || (cfg_.matmul_path != 1 && (cfg_.matmul_path == 2 || B > 8));
+    if (R > 0) {
+        const bool f16_B = dense_matrices_ || (cfg_.matmul_path != 1 && (cfg_.matmul_path == 2 || R > 8));
         int kind = act_kind_of(head);
-        ActQ xl = act_view(l_qs_, l_d_, l_bs_, l_xh_, B, H, kind, f16_B);
+        ActQ xl = act_view(l_qs_, l_d_, l_bs_, l_xh_, R, H, kind, f16_B);
         NormQuantArgs ng;
         ng.h = h_.as<float>();
         ng.norm_w = output_norm_.as<float>();
         ng.eps = ms_.eps;
-        ng.rows = B;
+        ng.rows = R;
         ng.dim = H;
-        ng.row_index = bd.last_index;
+        ng.row_index = tick.out_rows;
         ng.act_kind = kind;
         ng.out = xl;
-        prof_begin(KC_NORM_QUANT, 5.0 * B * H, 0);
+        prof_begin(KC_NORM_QUANT, 5.0 * R * H, 0);
         launch_add_norm_quant(ng, stream_);
         prof_end();
         ++launches_;
-        if (qs_head_.ready && f16_B && B >= qstream_min_rows_ && B <= kQStreamMaxRows && xl.xh != nullptr)
-            matmul_stream(qs_head_, xl, B, logits_.as<float>(), ms_.vocab, 1);
+        if (qs_head_.ready && f16_B && R >= qstream_min_rows_ && R <= kQStreamMaxRows && xl.xh != nullptr)
+            matmul_stream(qs_head_, xl, R, logits_.as<float>(), ms_.vocab, 1);
         else
-            matmul(head_dw, xl, B, logits_.as<float>(), ms_.vocab, ms_.final_logit_scale, ms_.final_softcap);
+            matmul(head_dw, xl, R, logits_.as<float>(), ms_.vocab, ms_.final_logit_scale, ms_.final_softcap);
     }
-    if (flags & FWD_WANT_TOKENS) {
-        prof_begin(KC_SAMPLE, 4.0 * B * ms_.vocab, 0);
-        if (off_sampling != 0)
-            launch_sample(logits_.as<float>(), B, ms_.vocab, reinterpret_cast<const LaneSampling*>(dp + off_sampling), tokens_.as<uint32_t>(),
-                          tc_ws_.status.as<int32_t>(), stream_);
-        else
-            launch_argmax(logits_.as<float>(), B, ms_.vocab, tokens_.as<uint32_t>(), argmax_scratch_.ptr(), stream_);
-        prof_end();
-        ++launches_;
-    }
-    // results travel to pinned host memory on the same stream; the barrier is in fetch_output
-    uint8_t* oh = out_host_.as<uint8_t>();
-    size_t tok_off = (size_t)B * ms_.vocab * 4;
-    if (flags & FWD_WANT_LOGITS) MK_CUDA(cudaMemcpyAsync(oh, logits_.ptr(), tok_off, cudaMemcpyDeviceToHost, stream_));
-    if (flags & FWD_WANT_TOKENS) MK_CUDA(cudaMemcpyAsync(oh + tok_off, tokens_.ptr(), (size_t)B * 4, cudaMemcpyDeviceToHost, stream_));
-    MK_CUDA(cudaMemcpyAsync(oh + tok_off + (size_t)B * 4, err_.ptr(), 4, cudaMemcpyDeviceToHost, stream_));
-    MK_CUDA(cudaMemcpyAsync(oh + tok_off + (size_t)B * 4 + 4, tc_ws_.status.ptr(), 4, cudaMemcpyDeviceToHost, stream_));
-    d2h_bytes_ += 8 + ((flags & FWD_WANT_LOGITS) ? (int64_t)tok_off : 0) + ((flags & FWD_WANT_TOKENS) ? (int64_t)B * 4 : 0);
-    MK_CUDA(cudaEventRecord(ev_stop_, stream_));
-    timed_ = true;
-    out_lanes_ = B;
-    out_flags_ = flags;
+    finish_tick(tick, KC_SAMPLE);
 }
 
-void Model::fetch_output(float* logits, uint32_t* tokens) {
-    MK_CUDA(cudaStreamSynchronize(stream_));
-    if (profiling_) prof_resolve();
-    const int B = out_lanes_;
-    uint8_t* oh = out_host_.as<uint8_t>();
-    size_t tok_off = (size_t)B * ms_.vocab * 4;
-    int32_t flags[2];
-    memcpy(flags, oh + tok_off + (size_t)B * 4, 8);
-    if (flags[0] != 0) throw std::runtime_error("batch descriptor index out of range on the device (flag " + std::to_string(flags[0]) + ")");
-    if (flags[1] != 0) {
-        // the status word is sticky on the device: clear it so that the next forward starts clean
-        cudaMemsetAsync(tc_ws_.status.ptr(), 0, 4, stream_);
-        if ((flags[1] & 0xFFFF0000) == kSampleEmptyStatus)
-            throw std::runtime_error("sampling distribution is empty (lane " + std::to_string(flags[1] & 0xFFFF) + ")");  // src/sampling.rs:352-355
-        if ((flags[1] & 0xFFFF0000) == kMoeRouteStatus)
-            throw std::runtime_error("router produced non-finite logits for token row " + std::to_string(flags[1] & 0xFFFF));  // src/decoder.rs:474-483
-        throw std::runtime_error("a bounded wait inside a kernel gave up (tensor-core matmul pipeline or expert exchange; status " + std::to_string(flags[1]) + ")");
-    }
-    if (logits) {
-        if (!(out_flags_ & FWD_WANT_LOGITS)) throw std::runtime_error("logits were not requested for this forward");
-        memcpy(logits, oh, tok_off);
-    }
-    if (tokens) {
-        if (!(out_flags_ & FWD_WANT_TOKENS)) throw std::runtime_error("tokens were not requested for this forward");
-        memcpy(tokens, oh + tok_off, (size_t)B * 4);
-    }
-}
-
-void Model::device_synchronize() { MK_CUDA(cudaStreamSynchronize(stream_)); }
-
-float Model::last_forward_ms() const {
-    if (!timed_) return 0.f;
-    float ms = 0.f;
-    if (cudaEventElapsedTime(&ms, ev_start_, ev_stop_) != cudaSuccess) {
-        cudaGetLastError();
-        return 0.f;
-    }
-    return ms;
+std::string Model::status_message(int32_t status) const {
+    if ((status & 0xFFFF0000) == kMoeRouteStatus)
+        return "router produced non-finite logits for token row " + std::to_string(status & 0xFFFF);  // src/decoder.rs:474-483
+    return DeviceLm::status_message(status);
 }
 
 }  // namespace mk

@@ -3,10 +3,10 @@
 // Mirrors DecoderModel of the reference (src/decoder.rs: load :2980-3105, forward_inner_batch
 // :3146-3358) for the attention-only families llama, smollm3, qwen3, qwen3moe and gemma2.
 #pragma once
+#include "device_lm.h"
 #include "device_util.h"
 #include "gguf_file.h"
 #include "kernels.h"
-#include "paged_lm.h"
 #include "qgemm_tc.h"
 #include "hgemm_tc.h"
 #include "qstream_tc.h"
@@ -49,47 +49,20 @@ struct GgufAudit {
 // (src/gguf_model.rs:3388-3776); throws with the reference's wording on the first violation.  Host only.
 GgufAudit validate_decoder_tensors(const GgufFile& f, const ModelSpec& s);
 
-struct ModelConfig {
-    int device = 0;
-    int block_tokens = 16, slab_blocks = 8;
-    int64_t kv_capacity_tokens = 4096, prefix_capacity_tokens = 0;
-    bool kv_f16 = true;
-    int max_batch_tokens = 2048, max_batch_lanes = 64;
-    // 0 auto (integer GEMV for a few rows, in-kernel dequant GEMM for tens of rows, f16-image GEMM for wide
-    // ticks when the image fits), 1 integer GEMV only, 2 in-kernel dequant GEMM whenever the shape allows,
-    // 3 f16-image GEMM whenever more than 8 rows share a matrix, 4 like 0 but nothing falls back to the in-kernel
-    // dequant GEMM (f16 images for wide ticks, streamed Q4_K / Q6_K blocks for 1..64 rows)
-    int matmul_path = 0;
-    // expert parallelism of a sparse-MoE model: this process holds experts [ep_rank, ep_rank + 1) * experts / ep_size
-    // and exchanges per-layer partial sums with the other ranks; ep_size <= 1 keeps every expert here
-    int ep_rank = 0, ep_size = 1;
-    // 0: all ranks run the same ticks on the same tokens (partial sums exchanged); 1: every rank schedules its own
-    // sequences and each MoE layer sends the routed rows to the experts' ranks and the outputs back (ep_dispatch.cu)
-    int ep_mode = 0;
-};
-
-class Model : public PagedLm {
+class Model : public DeviceLm {
 public:
     Model(const std::string& gguf_path, const ModelConfig& cfg);
     ~Model() override;
 
     const ModelSpec& model_spec() const { return ms_; }
     // Joins the expert-parallel group (collective over all ep_size ranks; `id` is EpComm::unique_id from rank 0).
-    void ep_init(const uint8_t* id);
+    void ep_init(const uint8_t* id) override;
     // ep_mode 1: the exchanges of one tick for a rank that has no lane to run (it serves the other ranks' rows).
-    void ep_idle_tick();
-    bool device_sampling_covers(float temperature, int top_k) const override { return mk::device_sampling_covers(temperature, top_k, ms_.vocab); }
-    float last_forward_ms() const override;
-    int64_t launch_count() const override { return launches_; }
-    int64_t h2d_bytes() const override { return h2d_bytes_; }
-    int64_t d2h_bytes() const override { return d2h_bytes_; }
-    void profile_enable(bool on) override;
-    std::vector<KernelProfile> profile_query() override;
+    void ep_idle_tick() override;
 
 protected:
     void run_forward(const std::vector<LmLane>& lanes, KvReservation& r, uint32_t flags) override;
-    void fetch_output(float* logits, uint32_t* tokens) override;
-    void device_synchronize() override;
+    std::string status_message(int32_t status) const override;
 
 private:
     struct LayerWeights {
@@ -113,21 +86,7 @@ private:
     void rope_tables_for(double theta, const float*& cos_t, const float*& sin_t);
 
     ModelSpec ms_;
-    ModelConfig cfg_;
-    cudaStream_t stream_ = nullptr;
-    cudaEvent_t ev_start_ = nullptr, ev_stop_ = nullptr;
-    bool timed_ = false;
-    int64_t launches_ = 0, h2d_bytes_ = 0, d2h_bytes_ = 0;
-    // profiling: one event pair per launch group, resolved after the tick's barrier
     enum KClass { KC_GEMM_TC = 0, KC_HGEMM, KC_QSTREAM, KC_GEMV, KC_ATTN, KC_NORM_QUANT, KC_ROPE_KV, KC_ACTMUL, KC_EMBED, KC_BATCH, KC_SAMPLE, KC_MOE, KC_HGEMM_NARROW, KC_EP, KC_COUNT };
-    struct ProfSpan { int cls; double bytes, flops; cudaEvent_t a, b; };
-    bool profiling_ = false;
-    std::vector<ProfSpan> spans_;
-    std::vector<cudaEvent_t> event_pool_;
-    KernelProfile prof_[KC_COUNT];
-    void prof_begin(int cls, double bytes, double flops);
-    void prof_end();
-    void prof_resolve();
 
     std::vector<LayerWeights> lw_;
     DeviceWeight token_embd_, output_;
@@ -136,15 +95,10 @@ private:
     std::vector<std::unique_ptr<RopeTable>> rope_;
 
     DevBuf k_pool_, v_pool_;
-    // per-tick staging
-    PinnedBuf stage_host_;
-    DevBuf stage_dev_;
-    DevBuf cu_, pos_, tok_lane_, slots_, last_, tile_lane_, tile_row_, ntiles_, err_;
     // tensor-core attention: split-KV partials of one-token lanes
     DevBuf attn_part_o_, attn_part_ml_, attn_counters_;
     bool attn_tc_ = false;
     // f16 weight images for wide ticks
-    DevBuf argmax_scratch_;
     bool half_cache_ = false;
     int hgemm_min_rows_ = 33;
     int64_t half_cache_bytes_ = 0;
@@ -171,7 +125,7 @@ private:
     std::vector<int32_t> plan_sp_, plan_nt_, plan_nb_;
     // activations
     // qkv_: [T][AW + 2 KW] (q | k | v per row); gu_: [T][2 ffn] (gate | up per row)
-    DevBuf h_, qkv_, attn_, proj_, gu_, down_, normed_, logits_, tokens_;
+    DevBuf h_, qkv_, attn_, proj_, gu_, down_, normed_;
     DevBuf a_qs_, a_d_, a_bs_, a_xh_;   // quantised activations of width hidden / attention width
     DevBuf f_qs_, f_d_, f_bs_, f_xh_;   // quantised activations of width ffn
     DevBuf l_qs_, l_d_, l_bs_, l_xh_;   // last-token rows for the output projection
@@ -187,9 +141,6 @@ private:
     uint64_t ep_wait_ns_ = kEpWaitNs;
     const float* ep_exchange_layer(LayerWeights& w, const LayerSpec& ls, const __half* grouped_rows, const int32_t* offsets, int T);
     QgemmWorkspace tc_ws_;
-    PinnedBuf out_host_;
-    int out_lanes_ = 0;
-    uint32_t out_flags_ = 0;
 };
 
 }  // namespace mk

@@ -5,14 +5,14 @@
 namespace mk {
 
 void PagedLm::init_pool(int block_tokens, int slab_blocks, int64_t capacity_tokens, int64_t prefix_capacity_tokens,
-                        bool allow_prefix_cache) {
+                        const char* no_prefix_reason) {
     if (block_tokens <= 0 || slab_blocks <= 0 || capacity_tokens <= 0)
         throw std::runtime_error("KV pool configuration must be positive");
     int64_t max_blocks = (capacity_tokens + block_tokens - 1) / block_tokens;  // src/runtime.rs:194
     pool_ = std::make_shared<KvPool>(block_tokens, slab_blocks, max_blocks);
     if (prefix_capacity_tokens > 0) {
-        if (!allow_prefix_cache)  // :4352-4372: rejected for models with a sliding-window layer
-            throw std::runtime_error("the automatic prefix cache is not supported for models with sliding-window layers");
+        if (no_prefix_reason != nullptr)  // :4352-4372: rejected for models with a sliding-window layer
+            throw std::runtime_error(std::string("the automatic prefix cache is not supported for models with ") + no_prefix_reason);
         int64_t budget = std::min((prefix_capacity_tokens + block_tokens - 1) / block_tokens, max_blocks);  // :3403-3412
         prefix_cache_ = std::make_unique<TokenPrefixCache<Snapshot>>((size_t)block_tokens, (size_t)budget);
     }
@@ -30,6 +30,13 @@ std::unique_ptr<LmSession> PagedLm::fork_session_prefix(LmSession& s, int64_t lo
     if (s.table->logical_len() != s.logical_len) throw std::runtime_error("decoder session block table disagrees with its sequence length");
     auto f = std::make_unique<LmSession>();
     f->owner = this;
+    if (state_slots_ && logical_len > 0) {
+        // a recurrent state exists for the sequence's end only
+        if (logical_len != s.logical_len)
+            throw std::runtime_error("a session with recurrent state can be forked at its current length only");
+        f->state = acquire_state();
+        copy_state(s.state->current(), f->state->current());
+    }
     f->table = s.table->fork_prefix(logical_len);
     f->logical_len = logical_len;
     return f;
@@ -44,7 +51,15 @@ void PagedLm::clear_session(LmSession& s) {  // :3804-3818
     int64_t old_len = s.table->logical_len();
     s.table->clear();
     if (old_len != 0 && s.table->logical_len() != 0) return;  // a reservation keeps the table locked
+    s.state.reset();
     s.logical_len = 0;
+}
+
+std::unique_ptr<StateLease> PagedLm::acquire_state() {
+    const int slot = state_slots_->acquire();
+    if (slot < 0)
+        throw KvPoolExhausted(1, 0, 0, "every recurrent-state slot is in use (" + std::to_string(state_slots_->capacity()) + " slots)");
+    return std::make_unique<StateLease>(state_slots_, slot);
 }
 
 int64_t PagedLm::reset_session_for_prompt(LmSession& s, const uint32_t* tokens, size_t n) {  // :3494-3532
@@ -112,6 +127,7 @@ std::unique_ptr<LmReservation> PagedLm::reserve_batch(const std::vector<LmLane>&
         r->sessions.push_back(l.session);
         r->start_pos.push_back(l.start_pos);
         r->n_tokens.push_back(l.n_tokens);
+        r->new_state.push_back(state_slots_ && !l.session->state ? acquire_state() : nullptr);
     }
     for (;;) {
         try {
@@ -156,13 +172,34 @@ void PagedLm::forward_batch_reserved(const std::vector<LmLane>& lanes, std::uniq
             reservation->n_tokens[i] != l.n_tokens)
             throw std::runtime_error("paged KV reservation lane " + std::to_string(i) +
                                      " does not match session, order, start or token count");  // src/decoder.rs:4076-4090
+        if (l.logit_rows != nullptr) {
+            if (flags & FWD_WANT_TOKENS) throw std::runtime_error("token selection reads each lane's last row: it cannot be combined with chosen logit rows");
+            for (int r = 0; r < l.n_logit_rows; ++r)
+                if (l.logit_rows[r] < 0 || l.logit_rows[r] >= l.n_tokens) throw std::runtime_error("a chosen logit row lies outside its lane's tokens");
+        }
+    }
+    std::vector<LmLane> placed;
+    if (state_slots_) {
+        placed = lanes;
+        for (size_t i = 0; i < placed.size(); ++i) {
+            const StateLease* own = placed[i].session->state.get();
+            const StateLease* use = own ? own : reservation->new_state[i].get();
+            if (use == nullptr) throw std::runtime_error("a lane's recurrent-state slot was given back before its forward");
+            placed[i].state_in = own ? own->current() : -1;
+            placed[i].state_out = own ? own->next() : use->current();
+        }
     }
     KvReservation& paged = *reservation->paged;
     paged.mark_all_used();
-    run_forward(lanes, paged, flags);  // a throw leaves every session untouched; the reservation rolls back
+    run_forward(state_slots_ ? placed : lanes, paged, flags);  // a throw leaves every session untouched; the reservation rolls back
     forward_unread_ = true;
     paged.commit();
-    for (const LmLane& l : lanes) l.session->logical_len = (int64_t)l.start_pos + l.n_tokens;
+    for (size_t i = 0; i < lanes.size(); ++i) {
+        LmSession& s = *lanes[i].session;
+        s.logical_len = (int64_t)lanes[i].start_pos + lanes[i].n_tokens;
+        if (s.state) s.state->flip();
+        else if (state_slots_) s.state = std::move(reservation->new_state[i]);
+    }
     last_lanes_ = (int)lanes.size();
     last_flags_ = flags;
 }
@@ -183,12 +220,13 @@ void PagedLm::synchronize() {  // :3785-3788
 // ---------------------------------------------------------------------------- FakeLm
 
 FakeLm::FakeLm(int vocab, int max_context, int block_tokens, int slab_blocks, int64_t capacity_tokens,
-               int64_t prefix_capacity_tokens) {
+               int64_t prefix_capacity_tokens, int state_slots) {
     spec_.vocab = vocab;
     spec_.max_context = max_context;
     spec_.layers = 1;
     spec_.hidden = 1;
-    init_pool(block_tokens, slab_blocks, capacity_tokens, prefix_capacity_tokens, true);
+    init_pool(block_tokens, slab_blocks, capacity_tokens, prefix_capacity_tokens, state_slots > 0 ? "recurrent layers" : nullptr);
+    if (state_slots > 0) init_state_slots(state_slots);
 }
 
 void FakeLm::run_forward(const std::vector<LmLane>& lanes, KvReservation&, uint32_t) {

@@ -6,6 +6,7 @@
 #pragma once
 #include "kv_pool.h"
 #include "prefix_cache.h"
+#include "state_slots.h"
 #include <memory>
 #include <optional>
 #include <string>
@@ -18,6 +19,7 @@ class PagedLm;
 struct LmSession {
     PagedLm* owner = nullptr;
     std::unique_ptr<KvTable> table;
+    std::unique_ptr<StateLease> state;  // models with recurrent layers: the sequence's slot, from its first forward on
     int64_t logical_len = 0;
 };
 
@@ -32,6 +34,13 @@ struct LmLane {
     int32_t top_k = 0;
     float top_p = 1.f;
     float u = 0.f;
+    // which of this lane's rows the forward projects to logits: null = its last row; otherwise n_logit_rows row numbers
+    // within the lane's tokens (possibly none), whose logits come out in this order
+    const int32_t* logit_rows = nullptr;
+    int32_t n_logit_rows = 0;
+    // recurrent state, filled in by forward_batch_reserved: the slot half to read (-1: the sequence starts here) and to write
+    int32_t state_in = -1, state_out = -1;
+    int rows_out() const { return logit_rows == nullptr ? 1 : n_logit_rows; }
 };
 
 struct LmReservation {
@@ -39,6 +48,7 @@ struct LmReservation {
     std::vector<LmSession*> sessions;
     std::vector<int32_t> start_pos, n_tokens;
     std::unique_ptr<KvReservation> paged;
+    std::vector<std::unique_ptr<StateLease>> new_state;  // slots of the lanes that had none yet (null for the others)
 };
 
 struct LmRuntimeSpec {
@@ -78,7 +88,8 @@ public:
     // CausalLm::forward_batch_tokens_reserved: validates every lane before any mutation, consumes the
     // reservation, enqueues the tick and commits the block tables.
     void forward_batch_reserved(const std::vector<LmLane>& lanes, std::unique_ptr<LmReservation> reservation, uint32_t flags);
-    // CausalLm::read_output_to_cpu: completion barrier; retired pages become free.
+    // CausalLm::read_output_to_cpu: completion barrier; retired pages become free.  `logits` takes one row per row asked
+    // for (see LmLane::logit_rows), lanes in order.
     void read_output(float* logits, uint32_t* tokens);
     // CausalLm::synchronize
     void synchronize();
@@ -100,11 +111,25 @@ public:
         double ms = 0, bytes = 0, flops = 0;
     };
     virtual void profile_enable(bool) {}
+    // Keep the residual stream after every layer of the next forwards; read_residuals copies those of the last one,
+    // [layers][tokens][hidden] in f32, and returns the token count.
+    virtual void capture_residuals(bool) { throw std::runtime_error("this model does not expose its residual stream"); }
+    virtual int read_residuals(float*, int64_t) { throw std::runtime_error("this model does not expose its residual stream"); }
+    // Expert parallelism (sparse-MoE models): see mk_model_ep_init / mk_model_ep_idle_tick.
+    virtual void ep_init(const uint8_t*) { throw std::runtime_error("expert parallelism needs a GGUF model"); }
+    virtual void ep_idle_tick() { throw std::runtime_error("expert parallelism needs a GGUF model"); }
+    // Recurrent-state slots, or null when the model keeps none.
+    const StateSlots* state_slots() const { return state_slots_.get(); }
     virtual std::vector<KernelProfile> profile_query() { return {}; }
     void validate_session(const LmSession& s) const;
 
 protected:
-    void init_pool(int block_tokens, int slab_blocks, int64_t capacity_tokens, int64_t prefix_capacity_tokens, bool allow_prefix_cache);
+    // `no_prefix_reason` (null = allowed): why this model cannot share prompt prefixes.
+    void init_pool(int block_tokens, int slab_blocks, int64_t capacity_tokens, int64_t prefix_capacity_tokens, const char* no_prefix_reason);
+    // Models with recurrent layers: one slot per sequence that may be live at a time.
+    void init_state_slots(int slots) { state_slots_ = std::make_shared<StateSlots>(slots); }
+    // Copy the state of slot half `from` to `to` in every layer (session forks).
+    virtual void copy_state(int from, int to) { (void)from; (void)to; }
     // Enqueue the device work of one tick.  `r` holds the provisional block tables of every lane.
     virtual void run_forward(const std::vector<LmLane>& lanes, KvReservation& r, uint32_t flags) = 0;
     // Wait for the tick and copy the requested outputs to the host.
@@ -117,6 +142,8 @@ protected:
     std::shared_ptr<KvPool> pool_;
     using Snapshot = std::unique_ptr<KvTable>;
     std::unique_ptr<TokenPrefixCache<Snapshot>> prefix_cache_;
+    std::shared_ptr<StateSlots> state_slots_;
+    std::unique_ptr<StateLease> acquire_state();
     int last_lanes_ = 0;
     uint32_t last_flags_ = 0;
     bool forward_unread_ = false;  // a forward was enqueued and neither read_output nor synchronize has run since
@@ -128,7 +155,8 @@ protected:
 // (31 * t + 7 * p + 3) mod vocab.
 class FakeLm : public PagedLm {
 public:
-    FakeLm(int vocab, int max_context, int block_tokens, int slab_blocks, int64_t capacity_tokens, int64_t prefix_capacity_tokens);
+    FakeLm(int vocab, int max_context, int block_tokens, int slab_blocks, int64_t capacity_tokens, int64_t prefix_capacity_tokens,
+           int state_slots = 0);
     // Fail the forward numbered `index` (0-based) with an exception, to test rollback.
     void fail_forward_at(int64_t index) { fail_at_ = index; }
     // The same for the completion barrier (site 1), prompt admission (site 2), the cleanup drain (site 3) and the clearing

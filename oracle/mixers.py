@@ -1,0 +1,290 @@
+"""Plain NumPy statement of the mixer-built decoders (the Sizilorn design and its parts), test infrastructure only.
+
+One function per mechanism, whole sequences at once, float64 unless the caller passes other arrays; recurrences are written
+token by token.  Nothing here is shared with the CUDA path.  Shapes: x, h [T, width]; a head-wise array [T, heads, dim].
+"""
+from __future__ import annotations
+
+import numpy as np
+
+
+# ------------------------------------------------------------------------------------------------ elementwise
+
+def sigmoid(z):
+    return 0.5 * (1.0 + np.tanh(0.5 * z))
+
+
+def silu(z):
+    return z * sigmoid(z)
+
+
+def gelu_tanh(z):
+    return 0.5 * z * (1.0 + np.tanh(np.sqrt(2.0 / np.pi) * (z + 0.044715 * z ** 3)))
+
+
+def softplus(z):
+    return np.maximum(z, 0.0) + np.log1p(np.exp(-np.abs(z)))
+
+
+# ------------------------------------------------------------------------------------------------ norms
+
+def rms(x, eps):
+    """Division by the root mean square over the last axis, eps inside the root."""
+    return x / np.sqrt(np.mean(x * x, axis=-1, keepdims=True) + eps)
+
+
+def dyn_tanh(x, alpha, w, b):
+    return np.tanh(alpha * x) * w + b
+
+
+# ------------------------------------------------------------------------------------------------ rotation
+
+def rope_frequencies(dims, base, scaling=None):
+    """One frequency per pair; `scaling` = dict(factor, low, high, original) stretches the long wavelengths."""
+    f = base ** (-2.0 * np.arange(dims // 2) / dims)
+    if not scaling:
+        return f
+    out = []
+    for fi in f:
+        wavelength = 2.0 * np.pi / fi
+        turns = scaling["original"] / wavelength
+        if turns > scaling["high"]:
+            out.append(fi)
+        elif turns < scaling["low"]:
+            out.append(fi / scaling["factor"])
+        else:
+            s = (turns - scaling["low"]) / (scaling["high"] - scaling["low"])
+            out.append((1.0 - s) * fi / scaling["factor"] + s * fi)
+    return np.array(out)
+
+
+def rotate_interleaved(x, positions, dims, freqs):
+    """x [T, heads, dim]: the pairs (2i, 2i + 1) of the first `dims` dimensions turn by position * freqs[i]."""
+    a = np.asarray(positions, np.float64)[:, None] * freqs[None, :]
+    c, s = np.cos(a)[:, None, :], np.sin(a)[:, None, :]
+    out = x.copy()
+    u, v = x[..., 0:dims:2], x[..., 1:dims:2]
+    out[..., 0:dims:2] = u * c - v * s
+    out[..., 1:dims:2] = v * c + u * s
+    return out
+
+
+# ------------------------------------------------------------------------------------------------ attention
+
+def causal_attention(q, k, v, scale):
+    """q [T, H, d], k [T, G, d], v [T, G, e]; query head h reads key/value head h // (H // G)."""
+    T, H, _ = q.shape
+    group = H // k.shape[1]
+    out = np.empty((T, H, v.shape[2]), q.dtype)
+    mask = np.tril(np.ones((T, T), bool))
+    for h in range(H):
+        s = (q[:, h] @ k[:, h // group].T) * scale
+        s = np.where(mask, s, -np.inf)
+        p = np.exp(s - s.max(axis=1, keepdims=True))
+        out[:, h] = (p / p.sum(axis=1, keepdims=True)) @ v[:, h // group]
+    return out
+
+
+def gated_attention(h, W, cfg, eps):
+    """Grouped-query attention with per-head query/key norms, interleaved rotation and a per-head output gate."""
+    T = h.shape[0]
+    H, G, d, e = cfg["heads"], cfg["kv_heads"], cfg["dim"], cfg["vdim"]
+    q = rms((h @ W["q"].T).reshape(T, H, d), eps) * W["q.norm"]
+    k = rms((h @ W["k"].T).reshape(T, G, d), eps) * W["k.norm"]
+    v = (h @ W["v"].T).reshape(T, G, e)
+    rot = cfg.get("rot")
+    if rot:
+        f = rope_frequencies(rot["dims"], rot["base"], rot.get("scaling"))
+        pos = np.arange(T)
+        q, k = rotate_interleaved(q, pos, rot["dims"], f), rotate_interleaved(k, pos, rot["dims"], f)
+    o = causal_attention(q, k, v, cfg["scale"])
+    o = o * sigmoid(h @ W["g"].T)[:, :, None]
+    return o.reshape(T, H * e) @ W["o"].T
+
+
+# ------------------------------------------------------------------------------------------------ gated delta rule
+
+def causal_conv(x, taps):
+    """Depthwise convolution over time, x [T, C], taps [C, K], last tap = the current token, zeros before the start."""
+    T, K = x.shape[0], taps.shape[1]
+    padded = np.concatenate([np.zeros((K - 1, x.shape[1]), x.dtype), x])
+    return sum(padded[j:j + T] * taps[:, j] for j in range(K))
+
+
+def unit(x):
+    return x / np.sqrt(np.sum(x * x, axis=-1, keepdims=True) + 1e-6)
+
+
+def delta_decay(alpha, a_log, dt_bias):
+    return np.exp(-np.exp(a_log) * softplus(alpha + dt_bias))
+
+
+def delta_rule(q, k, v, g, beta, state=None):
+    """q, k [T, G, d], v [T, H, e], g, beta [T, H]; head h reads q/k head h // (H // G).  Returns (o [T, H, e], state)."""
+    T, H, e = v.shape
+    group = H // q.shape[1]
+    S = np.zeros((H, q.shape[2], e), v.dtype) if state is None else state.copy()
+    o = np.empty_like(v)
+    for t in range(T):
+        qt, kt = np.repeat(q[t], group, axis=0), np.repeat(k[t], group, axis=0)
+        S *= g[t][:, None, None]
+        u = beta[t][:, None] * (v[t] - np.einsum("hde,hd->he", S, kt))
+        S += kt[:, :, None] * u[:, None, :]
+        o[t] = np.einsum("hde,hd->he", S, qt)
+    return o, S
+
+
+def gated_delta(h, W, cfg, eps):
+    T = h.shape[0]
+    H, G, d, e = cfg["heads"], cfg["kv_heads"], cfg["dim"], cfg["vdim"]
+    q = silu(causal_conv(h @ W["q"].T, W["q.conv"])).reshape(T, G, d)
+    k = silu(causal_conv(h @ W["k"].T, W["k.conv"])).reshape(T, G, d)
+    v = silu(causal_conv(h @ W["v"].T, W["v.conv"])).reshape(T, H, e)
+    q, k = unit(q) / np.sqrt(d), unit(k)
+    beta = sigmoid(h @ W["b"].T)
+    g = delta_decay(h @ W["a"].T, W["A_log"], W["dt_bias"])
+    o, _ = delta_rule(q, k, v, g, beta)
+    o = rms(o, eps) * W["norm"] * silu(h @ W["g"].T).reshape(T, H, e)
+    return o.reshape(T, H * e) @ W["o"].T
+
+
+def parallel_mixer(h, W, cfg, eps):
+    """Half the sum of the two branches' RMS-normed outputs."""
+    sub = lambda p: {k[len(p):]: v for k, v in W.items() if k.startswith(p)}
+    left = gated_attention(h, sub("left."), cfg["left"], eps)
+    right = gated_delta(h, sub("right."), cfg["right"], eps)
+    return 0.5 * (rms(left, eps) * W["left.out"] + rms(right, eps) * W["right.out"])
+
+
+# ------------------------------------------------------------------------------------------------ WKV time mixing
+
+def token_shift(h, mu):
+    prev = np.concatenate([np.zeros((1, h.shape[1]), h.dtype), h[:-1]])
+    return h + (prev - h) * mu
+
+
+def wkv_decay(mix_w, w1, w2, w0):
+    return np.exp(-np.exp(np.tanh(mix_w @ w1.T) @ w2.T + w0))
+
+
+def wkv_rule(r, k, v, w, u, state=None):
+    """r, k, v, w [T, H, d], u [H, d].  Returns (o [T, H, d], state)."""
+    T, H, d = r.shape
+    S = np.zeros((H, d, d), r.dtype) if state is None else state.copy()
+    o = np.empty_like(r)
+    for t in range(T):
+        kv = k[t][:, :, None] * v[t][:, None, :]
+        o[t] = np.einsum("hkv,hk->hv", S + u[:, :, None] * kv, r[t])
+        S = w[t][:, :, None] * S + kv
+    return o, S
+
+
+def wkv_mixer(h, W, cfg, eps):
+    T = h.shape[0]
+    H, d = cfg["heads"], cfg["dim"]
+    mix = {s: token_shift(h, W["mu." + s]) for s in "rkvgw"}
+    r, k, v = ((mix[s] @ W[s].T).reshape(T, H, d) for s in "rkv")
+    w = wkv_decay(mix["w"], W["w1"], W["w2"], W["w0"]).reshape(T, H, d)
+    o, _ = wkv_rule(r, k, v, w, W["u"])
+    return (rms(o, eps).reshape(T, H * d) * W["norm"] * silu(mix["g"] @ W["g"].T)) @ W["o"].T
+
+
+# ------------------------------------------------------------------------------------------------ feed-forward, token input
+
+def gated_mlp(h, W):
+    return (silu(h @ W["gate"].T) * (h @ W["up"].T)) @ W["down"].T
+
+
+def token_side(x, e, W, eps):
+    """The per-layer token input: e [T, dim] is the layer's slice of the side embedding."""
+    y = (gelu_tanh(x @ W["gate"].T) * e) @ W["proj"].T
+    return x + rms(y, eps) * W["norm"]
+
+
+# ------------------------------------------------------------------------------------------------ the decoder
+
+class MixerDecoder:
+    """config: the parsed config.json; tensors: name -> array."""
+
+    def __init__(self, config, tensors, dtype=np.float64):
+        self.cfg = config
+        self.w = {k: np.asarray(v, dtype) for k, v in tensors.items()}
+
+    def _sub(self, prefix):
+        return {k[len(prefix):]: v for k, v in self.w.items() if k.startswith(prefix)}
+
+    def _norm(self, name, x):
+        return dyn_tanh(x, self.w[name + ".alpha"], self.w[name], self.w[name + ".b"])
+
+    def residuals(self, tokens):
+        """The residual stream after every layer: [layers, T, width]."""
+        tokens = np.asarray(tokens)
+        eps = self.cfg["norm"]["eps"]
+        side = self.cfg.get("token_side")
+        x = self.w["embed"][tokens]
+        out = []
+        for i, layer in enumerate(self.cfg["layers"]):
+            p = f"l{i}."
+            mixer = {"wkv": wkv_mixer, "parallel": parallel_mixer}[layer["type"]]
+            x = x + mixer(self._norm(p + "norm1", x), self._sub(p + "mix."), layer["mixer"], eps)
+            if layer.get("mlp"):
+                x = x + gated_mlp(self._norm(p + "norm2", x), self._sub(p + "mlp."))
+            if side:
+                e = self.w["side.embed"][tokens][:, i * side["dim"]:(i + 1) * side["dim"]]
+                x = token_side(x, e, self._sub(p + "side."), eps)
+            out.append(x)
+        return np.stack(out)
+
+    def logits(self, tokens):
+        return self._norm("final.norm", self.residuals(tokens)[-1]) @ self.w["head"].T
+
+
+def read_safetensors(path):
+    """name -> float32 / int32 array (bfloat16 widened)."""
+    import json
+    import struct
+    raw = open(path, "rb").read()
+    (n,) = struct.unpack("<Q", raw[:8])
+    head = json.loads(raw[8:8 + n])
+    out = {}
+    for name, t in head.items():
+        if name == "__metadata__":
+            continue
+        lo, hi = t["data_offsets"]
+        b = raw[8 + n + lo:8 + n + hi]
+        if t["dtype"] == "BF16":
+            a = (np.frombuffer(b, np.uint16).astype(np.uint32) << 16).view(np.float32)
+        else:
+            a = np.frombuffer(b, {"F32": np.float32, "F16": np.float16, "I32": np.int32}[t["dtype"]])
+        out[name] = a.reshape(t["shape"])
+    return out
+
+
+def write_safetensors(path, tensors):
+    """Writes float arrays as bfloat16 (rounded to nearest even) and int32 arrays as they are."""
+    import json
+    import struct
+    head, blobs, at = {}, [], 0
+    for name, a in tensors.items():
+        a = np.asarray(a)
+        if a.dtype == np.int32:
+            b, kind = a.tobytes(), "I32"
+        else:
+            b, kind = to_bf16_bits(a).tobytes(), "BF16"
+        head[name] = {"dtype": kind, "shape": list(a.shape), "data_offsets": [at, at + len(b)]}
+        blobs.append(b)
+        at += len(b)
+    j = json.dumps(head).encode()
+    j += b" " * (-len(j) % 8)
+    with open(path, "wb") as f:
+        f.write(struct.pack("<Q", len(j)) + j + b"".join(blobs))
+
+
+def to_bf16_bits(a):
+    u = np.ascontiguousarray(a, np.float32).view(np.uint32)
+    return ((u + 0x7FFF + ((u >> 16) & 1)) >> 16).astype(np.uint16)
+
+
+def bf16(a):
+    """The nearest bfloat16 values, as float32."""
+    return (to_bf16_bits(a).astype(np.uint32) << 16).view(np.float32).reshape(np.shape(a))
