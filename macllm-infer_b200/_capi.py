@@ -11,6 +11,7 @@ from pathlib import Path
 
 HERE = Path(__file__).resolve().parent
 LIB_PATH = HERE / "libmacllm_b200.so"
+SERVING_LIB_PATH = HERE / "libmacllm_b200_serving.so"  # the part behind safetensors checkpoints (see build.build_for_serving)
 
 MK_OK, MK_KV_EXHAUSTED = 0, 1
 TYPE_F32, TYPE_F16, TYPE_Q8_0, TYPE_Q4_K, TYPE_Q6_K = 0, 1, 8, 12, 14
@@ -259,6 +260,9 @@ SIGNATURES = {
     "mk_k_moe_route": (_i32, [P, _i32, _i32, _i32, P, P]),
 }
 
+# entry points that only the full library carries
+FULL_LIBRARY_ONLY = ("mk_k_", "mk_gguf_", "mk_ep_unique_id")
+
 _lib = None
 
 
@@ -266,14 +270,19 @@ def lib() -> C.CDLL:
     """Load the shared library (once) and attach signatures.  Raises when it has not been built."""
     global _lib
     if _lib is None:
-        if not LIB_PATH.exists():
+        path = LIB_PATH if LIB_PATH.exists() else SERVING_LIB_PATH
+        if not path.exists():
             raise MkError(f"{LIB_PATH} is missing: run `python macllm-infer_b200/build.py` (there is no CPU fallback)")
-        handle = C.CDLL(str(LIB_PATH))
+        handle = C.CDLL(str(path))
         missing = [name for name in SIGNATURES if not hasattr(handle, name)]
+        if path == SERVING_LIB_PATH:
+            missing = [name for name in missing if not name.startswith(FULL_LIBRARY_ONLY)]
         if missing:
-            raise MkError(f"{LIB_PATH} does not export {missing}: rebuild it")
+            raise MkError(f"{path} does not export {missing}: rebuild it")
         for name, (res, args) in SIGNATURES.items():
-            fn = getattr(handle, name)
+            fn = getattr(handle, name, None)
+            if fn is None:
+                continue
             fn.restype = res
             fn.argtypes = args
         _lib = handle

@@ -2,6 +2,9 @@
 
 Usage: python macllm-infer_b200/build.py [--force]
 Objects are cached under macllm-infer_b200/build/ and rebuilt when a source or header is newer.
+
+build_for_serving() is what a fresh checkout needs to serve a safetensors checkpoint: the same library without the GGUF
+formats, their quantised matmuls and the kernel-level entry points.  It compiles nothing when a current library is there.
 """
 from __future__ import annotations
 
@@ -15,6 +18,11 @@ HERE = Path(__file__).resolve().parent
 CSRC = HERE / "csrc"
 BUILD = HERE / "build"
 LIB = HERE / "libmacllm_b200.so"
+SERVING_LIB = HERE / "libmacllm_b200_serving.so"
+# the translation units behind a safetensors checkpoint; the rest serves GGUF files and kernel-level callers
+SERVING = ["attention.cu", "attention_tc.cu", "batch.cu", "c_api_core.cpp", "c_api_model.cpp", "device_lm.cpp", "embed.cu", "engine.cpp", "hgemm_tc.cu",
+           "json.cpp", "kv_pool.cpp", "linear_state.cu", "mixer_lm.cpp", "mixer_ops.cu", "mixer_spec.cpp", "model_registry.cpp", "paged_lm.cpp",
+           "rope_kv.cu", "safetensors_file.cpp", "sample.cu", "seed_model.cpp", "device_info.cpp", "weights.cpp"]
 
 NVCC = os.environ.get("NVCC", "/usr/local/cuda/bin/nvcc")
 COMMON = [
@@ -30,9 +38,16 @@ def _newest_header() -> float:
     return max(p.stat().st_mtime for p in hs)
 
 
-def build(force: bool = False, verbose: bool = False) -> Path:
+def _stale(lib: Path, srcs) -> bool:
+    return not lib.exists() or lib.stat().st_mtime < max(_newest_header(), max(p.stat().st_mtime for p in srcs))
+
+
+def _all_sources():
+    return sorted(list(CSRC.glob("*.cu")) + list(CSRC.glob("*.cpp")))
+
+
+def _build(lib: Path, srcs, force: bool, verbose: bool) -> Path:
     BUILD.mkdir(exist_ok=True)
-    srcs = sorted(list(CSRC.glob("*.cu")) + list(CSRC.glob("*.cpp")))
     hdr_time = _newest_header()
     jobs = []
     objs = []
@@ -52,15 +67,25 @@ def build(force: bool = False, verbose: bool = False) -> Path:
         return r.stderr
 
     if jobs:
-        with ThreadPoolExecutor(max_workers=min(8, len(jobs))) as ex:
+        with ThreadPoolExecutor(max_workers=min(os.cpu_count() or 8, len(jobs))) as ex:
             for out in ex.map(run, jobs):
                 if verbose and out:
                     print(out)
-    if jobs or not LIB.exists():
-        link = [NVCC, "-shared", "-o", str(LIB), *map(str, objs), "-Xcompiler", "-fopenmp", "-lgomp", "-lcudart_static",
+    if jobs or _stale(lib, objs):
+        link = [NVCC, "-shared", "-o", str(lib), *map(str, objs), "-Xcompiler", "-fopenmp", "-lgomp", "-lcudart_static",
                 "-gencode", "arch=compute_100a,code=sm_100a"]
         run(link)
-    return LIB
+    return lib
+
+
+def build(force: bool = False, verbose: bool = False) -> Path:
+    return _build(LIB, _all_sources(), force, verbose)
+
+
+def build_for_serving() -> Path:
+    if LIB.exists():
+        return build()
+    return _build(SERVING_LIB, [CSRC / n for n in SERVING], False, False)
 
 
 if __name__ == "__main__":

@@ -61,11 +61,19 @@ private:
     size_t n_ = 0;
 };
 
-// The f16 image of one weight matrix [rows][cols] plus the TMA descriptor of its 128-row x 64-column
-// boxes (see hgemm_tc.h).  Built once at load time from the device copy of the quantised matrix.
+constexpr int kMaxRowGroups = 8;
+
+// The 16-bit image of one weight matrix [rows][cols] plus the TMA descriptor of its 128-row x 64-column
+// boxes (see hgemm_tc.h).  Built once at load time: f16 from the device copy of a quantised matrix, bf16 from a dense
+// checkpoint.
 struct HalfWeight {
-    DevBuf values;               // rows * cols halves, row-major
+    DevBuf values;               // rows * cols 16-bit values, row-major
     int64_t rows = 0, cols = 0;
+    bool bf16 = false;           // bfloat16 values (the activations then are too), else f16
+    // Stacked projections that do not share their input: row tiles [group_end[g - 1], group_end[g]) multiply the rows of
+    // input g.  The inputs lie one after the other, T rows each.  One group: the usual case.
+    int n_groups = 1;
+    int group_end[kMaxRowGroups] = {};
     alignas(64) unsigned char tmap[128] = {};  // CUtensorMap (opaque here, 64-byte aligned)
     bool ready = false;
 };

@@ -21,6 +21,7 @@
 #include "hgemm_tc.h"
 #include "kernels.h"
 #include <cuda.h>
+#include <cuda_bf16.h>
 #include <mutex>
 
 namespace mk {
@@ -183,7 +184,18 @@ struct HgParams {
     int gated;
     __half* yh;
     int ldyh;
+    int bf16;  // both operands (and yh) are bfloat16
+    // stacked projections with inputs of their own: the first row of input g in the activation matrix is g * T
+    int n_groups;
+    int group_end[kMaxRowGroups];
 };
+
+__device__ __forceinline__ int group_row0(const HgParams& p, int m_tile) {
+    if (p.n_groups == 1) return 0;
+    int g = 0;
+    while (g < p.n_groups - 1 && m_tile >= p.group_end[g]) ++g;
+    return g * p.T;
+}
 
 template <int BN, int STAGES>
 struct HgSmem {
@@ -271,6 +283,7 @@ hgemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant_
             for (int item = blockIdx.x; item < total_items && ok; item += gridDim.x) {
                 int m_tile, n_tile, kb0, kb1;
                 decode(item, m_tile, n_tile, kb0, kb1);
+                const int x_row = group_row0(p, m_tile) + n_tile * BN;
                 for (int kb = kb0; kb < kb1; ++kb, ++it) {
                     const uint32_t st = it % STAGES, ph = (it / STAGES) & 1;
                     if (it == STAGES && !waited) {  // the ring is full of weights: now the activations
@@ -289,10 +302,10 @@ hgemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant_
                     mbar_expect_tx(&full[st], (uint32_t)L::STAGE_BYTES);
                     tma_load_2d(a_dst, &tm_w, kb * HG_BK, m_tile * HG_BM, &full[st]);
                     if (waited) {
-                        tma_load_2d(b_dst, &tm_x, kb * HG_BK, n_tile * BN, &full[st]);
+                        tma_load_2d(b_dst, &tm_x, kb * HG_BK, x_row, &full[st]);
                     } else {
                         held_x[st] = kb * HG_BK;
-                        held_y[st] = n_tile * BN;
+                        held_y[st] = x_row;
                     }
                 }
             }
@@ -305,7 +318,7 @@ hgemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant_
     } else if (warp == 1) {
         // ---- MMA issuer
         if (lane == 0) {
-            const uint32_t idesc = (1u << 4) | ((uint32_t)(BN >> 3) << 17) | ((uint32_t)(HG_BM >> 4) << 24);
+            const uint32_t idesc = (1u << 4) | (p.bf16 ? (1u << 7) | (1u << 10) : 0u) | ((uint32_t)(BN >> 3) << 17) | ((uint32_t)(HG_BM >> 4) << 24);
             uint32_t it = 0, tile_it = 0;
             bool ok = true;
             for (int item = blockIdx.x; item < total_items && ok; item += gridDim.x, ++tile_it) {
@@ -390,7 +403,8 @@ hgemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant_
                         int tok = tok0 + cb + i + (odd ? 1 : 0);
                         if (row < p.rows && tok < p.T) {
                             float a = p.gated == 1 ? hg_silu(g) : hg_gelu_tanh(g);
-                            p.yh[(int64_t)tok * p.ldyh + feature] = __float2half_rn(a * u);
+                            if (p.bf16) reinterpret_cast<__nv_bfloat16*>(p.yh)[(int64_t)tok * p.ldyh + feature] = __float2bfloat16_rn(a * u);
+                            else p.yh[(int64_t)tok * p.ldyh + feature] = __float2half_rn(a * u);
                         }
                     }
                 } else if (row < p.rows) {
@@ -437,15 +451,15 @@ EncodeTiledFn encode_fn() {
     return fn;
 }
 
-// f16 matrix [n_rows][cols] row-major, boxes of box_rows x 64 columns, 128-byte swizzle, zero fill.
-void encode_half_matrix(CUtensorMap* out, const void* base, int64_t n_rows, int64_t cols, int box_rows) {
+// 16-bit matrix [n_rows][cols] row-major, boxes of box_rows x 64 columns, 128-byte swizzle, zero fill.
+void encode_half_matrix(CUtensorMap* out, const void* base, int64_t n_rows, int64_t cols, int box_rows, bool bf16 = false) {
     if ((reinterpret_cast<uintptr_t>(base) & 15) != 0) throw std::runtime_error("hgemm: matrix base must be 16-byte aligned");
     cuuint64_t dims[2] = {(cuuint64_t)cols, (cuuint64_t)n_rows};
     cuuint64_t strides[1] = {(cuuint64_t)cols * 2};
     cuuint32_t box[2] = {(cuuint32_t)HG_BK, (cuuint32_t)box_rows};
     cuuint32_t elem[2] = {1, 1};
-    CUresult r = encode_fn()(out, CU_TENSOR_MAP_DATA_TYPE_FLOAT16, 2, const_cast<void*>(base), dims, strides, box, elem,
-                             CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
+    CUresult r = encode_fn()(out, bf16 ? CU_TENSOR_MAP_DATA_TYPE_BFLOAT16 : CU_TENSOR_MAP_DATA_TYPE_FLOAT16, 2, const_cast<void*>(base), dims, strides,
+                             box, elem, CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
                              CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
     if (r != CUDA_SUCCESS) throw std::runtime_error("cuTensorMapEncodeTiled failed with code " + std::to_string((int)r));
 }
@@ -528,6 +542,32 @@ void build_half_weight_interleaved(const QWeight& gate, const QWeight& up, HalfW
     out.ready = true;
 }
 
+void build_bf16_weight(const float* values, int64_t rows, int64_t cols, HalfWeight& out, cudaStream_t s, const std::vector<int64_t>& group_rows) {
+    if (rows <= 0 || cols <= 0 || cols % HG_BK != 0) throw std::runtime_error("build_bf16_weight: columns must be padded to a multiple of 64");
+    if (group_rows.size() > (size_t)kMaxRowGroups) throw std::runtime_error("build_bf16_weight: too many stacked projections");
+    std::vector<__nv_bfloat16> bits((size_t)(rows * cols));
+#pragma omp parallel for
+    for (int64_t i = 0; i < rows * cols; ++i) bits[(size_t)i] = __float2bfloat16_rn(values[i]);
+    out.rows = rows;
+    out.cols = cols;
+    out.bf16 = true;
+    out.n_groups = 1;
+    if (group_rows.size() > 1) {
+        out.n_groups = (int)group_rows.size();
+        int64_t end = 0;
+        for (size_t g = 0; g < group_rows.size(); ++g) {
+            if (group_rows[g] % HG_BM != 0) throw std::runtime_error("build_bf16_weight: a stacked projection must be a multiple of 128 rows");
+            end += group_rows[g];
+            out.group_end[g] = (int)(end / HG_BM);
+        }
+        if (end != rows) throw std::runtime_error("build_bf16_weight: stacked projections do not add up");
+    }
+    out.values.upload(bits.data(), bits.size() * 2, s);
+    MK_CUDA(cudaStreamSynchronize(s));
+    encode_half_matrix(reinterpret_cast<CUtensorMap*>(out.tmap), out.values.ptr(), rows, cols, HG_BM, true);
+    out.ready = true;
+}
+
 void build_half_weight(const QWeight& W, HalfWeight& out, cudaStream_t s) {
     const QWeight* one = &W;
     build_half_weight_stacked(&one, 1, out, s);
@@ -596,7 +636,7 @@ int launch_hgemm_any(const HalfWeight& W, const __half* xh, int T, float* y, int
         pl.kb_per_split = (int)(W.cols / HG_BK);
     }
     alignas(64) CUtensorMap tx;
-    encode_half_matrix(&tx, xh, T, W.cols, pl.bn);
+    encode_half_matrix(&tx, xh, (int64_t)T * W.n_groups, W.cols, pl.bn, W.bf16);
     HgParams p;
     p.T = T;
     p.K = (int)W.cols;
@@ -614,6 +654,9 @@ int launch_hgemm_any(const HalfWeight& W, const __half* xh, int T, float* y, int
     p.gated = gated;
     p.yh = yh;
     p.ldyh = ldyh;
+    p.bf16 = W.bf16 ? 1 : 0;
+    p.n_groups = W.n_groups;
+    for (int g = 0; g < kMaxRowGroups; ++g) p.group_end[g] = W.group_end[g];
     const int grid = std::min(device_sm_count(), p.row_tiles * p.n_tiles * p.splits);
     const CUtensorMap& tw = *reinterpret_cast<const CUtensorMap*>(W.tmap);
     if (pl.bn == 256) launch_hg<256, 4>(tw, tx, p, grid, s);

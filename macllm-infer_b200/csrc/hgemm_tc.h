@@ -28,6 +28,11 @@ void build_half_weight_stacked(const QWeight* const* parts, int n_parts, HalfWei
 // row 2j+1 = up row j), for launch_hgemm_tc_gated.
 void build_half_weight_interleaved(const QWeight& gate, const QWeight& up, HalfWeight& out, cudaStream_t s);
 
+// A dense matrix given as f32 host values [rows][cols], cols a multiple of 64 (zero-padded by the caller), rounded to bf16.
+// `group_rows` (optional): rows of each stacked projection with an input of its own, multiples of 128 (see HalfWeight).
+void build_bf16_weight(const float* values, int64_t rows, int64_t cols, HalfWeight& out, cudaStream_t s,
+                       const std::vector<int64_t>& group_rows = {});
+
 // How a call is cut into work items (see hgemm_tc.cu); partial_floats is the scratch a split call needs.
 struct HgemmPlan {
     int bn = 0, row_tiles = 0, n_tiles = 0, splits = 1, kb_per_split = 0;
@@ -44,7 +49,8 @@ struct HgemmScratch {
 };
 
 // y[t][n] = scale * sum_k xh[t][k] * Wh[n][k] (then the optional soft cap), t < T, n < rows.
-// xh is [T][cols] f16, 16-byte aligned.  Returns the number of K shares S the call was cut into.  S = 1: y holds
+// xh is [T][cols] in the image's own 16-bit format, 16-byte aligned; an image of n_groups stacked projections takes
+// [n_groups][T][cols].  Returns the number of K shares S the call was cut into.  S = 1: y holds
 // the result.  S > 1 (only when max_splits > 1, scale = 1 and no soft cap): y is NOT written; share s left its
 // partial sums at ws.partial[(s * T + t) * rows + n] and the consumer adds them for s = 0 .. S-1 in that order.
 int launch_hgemm_tc(const HalfWeight& W, const __half* xh, int T, float* y, int ldy, float out_scale, float softcap,
@@ -53,7 +59,8 @@ int launch_hgemm_tc(const HalfWeight& W, const __half* xh, int T, float* y, int 
 // Gated feed-forward front half in one kernel: with W an interleaved gate/up image (2F rows),
 // yh[t][j] = f16(act(sum_k xh[t][k] gate[j][k]) * sum_k xh[t][k] up[j][k]), j < F; act 0 = SiLU, otherwise tanh GELU.
 // The two sums are the f32 accumulators of the plain GEMM and the activation is evaluated like the separate SwiGLU
-// kernel does, so the halves written equal the ones that kernel derives from the plain GEMM's output.
+// kernel does, so the halves written equal the ones that kernel derives from the plain GEMM's output.  (bf16 for a bf16
+// image.)
 void launch_hgemm_tc_gated(const HalfWeight& W, const __half* xh, int T, int act, __half* yh, int ldyh, const HgemmScratch& ws,
                            cudaStream_t s);
 

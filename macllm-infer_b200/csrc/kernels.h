@@ -105,6 +105,9 @@ struct RopeKvArgs {
     int kv_f16 = 1;
     int T = 0, q_heads = 0, kv_heads = 0, d = 0, block_tokens = 16, layers = 0, layer = 0;
     int64_t pool_blocks = 0;  // see kv_page_index
+    int dv = 0;          // width of a value head (0 = d)
+    int d_row = 0;       // width of a head in q_out and in the pools (0 = d): the rest of the row is written as zeros
+    int interleaved = 0; // rotate the pairs (2i, 2i + 1) instead of (i, i + rotary_dim / 2)
 };
 void launch_rope_kv(const RopeKvArgs& a, cudaStream_t s);
 

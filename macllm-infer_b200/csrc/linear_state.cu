@@ -1,0 +1,338 @@
+// See linear_state.h.
+//
+// A warp holds eight value columns of one (lane, head): four groups of eight threads, two columns per group, the column's keys
+// shared out over the group's threads in runs of four.  The state stays in registers while the lane's rows go by.  Rows arrive
+// in shared memory in chunks, fetched with cp.async while the chunk before is being worked on; the sums over the keys of four
+// rows are folded together (each exchange halves what is left), so a row costs under two shuffles per column pair - except the
+// delta rule's S^T k, which the row itself depends on.  Wide prompts cut a head's columns over CTAs of four warps and leave the
+// head norm to a second kernel; ticks of short lanes give a whole head to one CTA, which then finishes the output row itself.
+#include "linear_state.h"
+#include <algorithm>
+
+namespace mk {
+
+namespace {
+
+constexpr int LS_COLS = 8;        // value columns of a warp
+constexpr int LS_WIDE_WARPS = 4;  // warps of a CTA that owns part of a head
+constexpr int LS_MAX_FINISH_V = 128;
+
+__device__ __forceinline__ void ls_cp_async16(void* dst, const void* src) {
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
+}
+__device__ __forceinline__ void ls_cp_async4(void* dst, const void* src) {
+    asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
+}
+__device__ __forceinline__ void ls_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+template <int N>
+__device__ __forceinline__ void ls_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
+
+// `n` rows of `width` floats, row i from src(i), into dst rows `pitch` floats apart; `vec`: everything is 16-byte aligned.
+template <typename Src>
+__device__ __forceinline__ void fetch_rows(float* dst, int pitch, int n, int width, bool vec, Src src) {
+    if (vec) {
+        const int per = width >> 2;
+        for (int i = threadIdx.x; i < n * per; i += blockDim.x) {
+            const int r = i / per, c = (i - r * per) * 4;
+            ls_cp_async16(dst + r * pitch + c, src(r) + c);
+        }
+    } else {
+        for (int i = threadIdx.x; i < n * width; i += blockDim.x) {
+            const int r = i / width, c = i - r * width;
+            ls_cp_async4(dst + r * pitch + c, src(r) + c);
+        }
+    }
+}
+// The same rows of a matmul output that is still in shares.
+__device__ __forceinline__ void sum_rows(float* dst, int pitch, int n, int width, const Shares& y, int64_t row0, int col) {
+    for (int i = threadIdx.x; i < n * width; i += blockDim.x) {
+        const int r = i / width, c = i - r * width;
+        dst[r * pitch + c] = y.at(row0 + r, col + c);
+    }
+}
+
+// Eight values per thread, folded over the eight threads of a group: thread t of the group ends with the sum of value t.
+__device__ __forceinline__ float fold8(const float (&v)[8], int t) {
+    float a[4], b[2];
+    const bool h4 = (t & 4) != 0, h2 = (t & 2) != 0, h1 = (t & 1) != 0;
+#pragma unroll
+    for (int i = 0; i < 4; ++i) a[i] = (h4 ? v[i + 4] : v[i]) + __shfl_xor_sync(0xffffffffu, h4 ? v[i] : v[i + 4], 4);
+#pragma unroll
+    for (int i = 0; i < 2; ++i) b[i] = (h2 ? a[i + 2] : a[i]) + __shfl_xor_sync(0xffffffffu, h2 ? a[i] : a[i + 2], 2);
+    return (h1 ? b[1] : b[0]) + __shfl_xor_sync(0xffffffffu, h1 ? b[0] : b[1], 1);
+}
+
+// One head's row o[0 .. vdim) of packed row `row` (in shared or global memory), by one warp.
+__device__ __forceinline__ void finish_head_row(const LinearStateArgs& a, const float* o, int64_t row, int head, int lane) {
+    float ss = 0.f;
+    for (int v = lane; v < a.vdim; v += 32) ss += o[v] * o[v];
+    ss = warp_sum(ss);
+    const float root = sqrtf(ss / (float)a.vdim + a.eps);
+    const float* nw = a.norm_w + (a.norm_per_head ? head * a.vdim : 0);
+    for (int v = lane; v < a.vdim; v += 32) {
+        const float g = a.gate.at(row, a.gate_col + head * a.vdim + v);
+        a.image.put(row, head * a.vdim + v, o[v] / root * nw[v] * silu_f(g));
+    }
+    if (head == a.heads - 1)
+        for (int c = a.heads * a.vdim + lane; c < a.image.ld; c += 32) a.image.put(row, c, 0.f);
+}
+
+template <int KD, int TT, bool WKV>
+struct LsSmem {
+    static constexpr int KROWS = WKV ? 3 : 2;  // r, k, decay  /  q, k
+    static __host__ __device__ constexpr size_t stage_floats(int cols) { return (size_t)TT * (KROWS * KD + cols + (WKV ? 0 : 4)); }
+    static __host__ __device__ constexpr size_t bytes(int cols, bool finish) { return (2 * stage_floats(cols) + (finish ? (size_t)TT * cols : 0)) * 4; }
+};
+
+template <int KD, bool WKV, bool FINISH>
+__global__ void __launch_bounds__(FINISH ? LS_MAX_FINISH_V / LS_COLS * 32 : LS_WIDE_WARPS * 32)
+linear_state_kernel(WkvScanArgs wa, DeltaScanArgs da) {
+    constexpr int TT = FINISH ? 4 : 16;
+    constexpr int KE = KD / 8;   // keys of a thread
+    constexpr int NJ = KE / 4;
+    using L = LsSmem<KD, TT, WKV>;
+    extern __shared__ __align__(16) float ls_smem[];
+    const LinearStateArgs& a = WKV ? wa.common : da.common;
+
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, grp = lane >> 3, ks = lane & 7;
+    const int cols = (int)(blockDim.x >> 5) * LS_COLS;  // columns of this CTA
+    const int col0 = blockIdx.x * cols;
+    const int head = blockIdx.y, seq = blockIdx.z;
+    const int c_loc = warp * LS_COLS + grp * 2;         // first of the thread's two columns, within the CTA
+    const int my_cols = min(cols, a.vdim - col0);
+
+    // The slot halves were staged by the host and the committed state was written by an earlier tick: neither depends on the
+    // predecessor kernel, so the state is on its way before the wait.
+    pdl_trigger();
+    const int2 half = a.lanes.halves[seq];
+    float S[2][KE];
+    const int64_t head_state = (int64_t)a.vdim * KD;
+#pragma unroll
+    for (int c = 0; c < 2; ++c) {
+        const int v = col0 + c_loc + c;
+        const bool live = half.x >= 0 && v < a.vdim;
+        const float4* src = reinterpret_cast<const float4*>(a.state + ((int64_t)half.x * a.heads + head) * head_state + (int64_t)v * KD);
+#pragma unroll
+        for (int j = 0; j < NJ; ++j) {
+            const float4 x = live ? src[j * 8 + ks] : make_float4(0.f, 0.f, 0.f, 0.f);
+            S[c][4 * j] = x.x; S[c][4 * j + 1] = x.y; S[c][4 * j + 2] = x.z; S[c][4 * j + 3] = x.w;
+        }
+    }
+    float U[WKV ? KE : 1];
+    if (WKV) {
+#pragma unroll
+        for (int e = 0; e < KE; ++e) {
+            const int i = (e >> 2) * 32 + ks * 4 + (e & 3);
+            U[WKV ? e : 0] = i < a.dim ? wa.bonus[head * a.dim + i] : 0.f;
+        }
+    }
+    // key columns past the true dimension and value columns past the last stay zero in both stages
+    for (int i = threadIdx.x; i < (int)(2 * L::stage_floats(cols)); i += blockDim.x) ls_smem[i] = 0.f;
+    __syncthreads();
+    pdl_wait();
+
+    const int first = a.lanes.cu[seq], n = a.lanes.cu[seq + 1] - first;
+    const int kv_head = WKV ? head : head / (a.heads / da.kv_heads);
+    const bool vec = (a.dim & 3) == 0 && (a.vdim & 3) == 0;
+    auto stage = [&](int which) { return ls_smem + (size_t)which * L::stage_floats(cols); };
+    auto fetch = [&](int chunk) {
+        float* s = stage(chunk & 1);
+        const int64_t r0 = first + chunk * TT;
+        const int m = min(TT, n - chunk * TT);
+        float* s_v = s + (size_t)TT * L::KROWS * KD;
+        if (WKV) {
+            const Shares& y = wa.rkv;
+            const int h0 = head * a.dim;
+            if (y.n == 1) {
+                const bool yv = vec && (y.ld & 3) == 0;
+                fetch_rows(s, KD, m, a.dim, yv, [&](int r) { return y.p + (r0 + r) * y.ld + wa.r_col + h0; });
+                fetch_rows(s + TT * KD, KD, m, a.dim, yv, [&](int r) { return y.p + (r0 + r) * y.ld + wa.k_col + h0; });
+                fetch_rows(s_v, cols, m, my_cols, yv && (my_cols & 3) == 0, [&](int r) { return y.p + (r0 + r) * y.ld + wa.v_col + h0 + col0; });
+            } else {
+                sum_rows(s, KD, m, a.dim, y, r0, wa.r_col + h0);
+                sum_rows(s + TT * KD, KD, m, a.dim, y, r0, wa.k_col + h0);
+                sum_rows(s_v, cols, m, my_cols, y, r0, wa.v_col + h0 + col0);
+            }
+            fetch_rows(s + 2 * TT * KD, KD, m, a.dim, vec, [&](int r) { return wa.decay + (r0 + r) * a.heads * a.dim + h0; });
+        } else {
+            const int64_t kw = (int64_t)da.kv_heads * a.dim, vw = (int64_t)a.heads * a.vdim;
+            fetch_rows(s, KD, m, a.dim, vec, [&](int r) { return da.q + (r0 + r) * kw + kv_head * a.dim; });
+            fetch_rows(s + TT * KD, KD, m, a.dim, vec, [&](int r) { return da.k + (r0 + r) * kw + kv_head * a.dim; });
+            fetch_rows(s_v, cols, m, my_cols, vec && (my_cols & 3) == 0, [&](int r) { return da.v + (r0 + r) * vw + head * a.vdim + col0; });
+            float* s_c = s_v + (size_t)TT * cols;
+            for (int r = threadIdx.x; r < m; r += blockDim.x) {
+                ls_cp_async4(s_c + 4 * r, da.decay + (r0 + r) * a.heads + head);
+                ls_cp_async4(s_c + 4 * r + 1, da.beta + (r0 + r) * a.heads + head);
+            }
+        }
+        ls_commit();
+    };
+
+    const int chunks = (n + TT - 1) / TT;
+    if (chunks > 0) fetch(0);
+    for (int ch = 0; ch < chunks; ++ch) {
+        if (ch + 1 < chunks) {
+            fetch(ch + 1);
+            ls_wait<1>();
+        } else {
+            ls_wait<0>();
+        }
+        __syncthreads();
+        const float* s = stage(ch & 1);
+        const float* s_v = s + (size_t)TT * L::KROWS * KD;
+        const int m = min(TT, n - ch * TT);
+        float* s_o = ls_smem + 2 * L::stage_floats(cols);  // FINISH: [TT][cols]
+#pragma unroll 1
+        for (int t0 = 0; t0 < m; t0 += 4) {
+            float part[8];
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+                part[2 * i] = part[2 * i + 1] = 0.f;
+                const int t = t0 + i;
+                if (t >= m) continue;  // uniform over the CTA
+                const float2 v = *reinterpret_cast<const float2*>(s_v + t * cols + c_loc);
+                const float4* k4 = reinterpret_cast<const float4*>(s + TT * KD + t * KD) + ks;
+                const float4* q4 = reinterpret_cast<const float4*>(s + t * KD) + ks;  // r / q
+                if constexpr (WKV) {
+                    const float4* w4 = reinterpret_cast<const float4*>(s + 2 * TT * KD + t * KD) + ks;
+                    float o0 = 0.f, o1 = 0.f;
+#pragma unroll
+                    for (int j = 0; j < NJ; ++j) {
+                        const float4 r = q4[j * 8], k = k4[j * 8], w = w4[j * 8];
+                        const float rr[4] = {r.x, r.y, r.z, r.w}, kk[4] = {k.x, k.y, k.z, k.w}, ww[4] = {w.x, w.y, w.z, w.w};
+#pragma unroll
+                        for (int e = 0; e < 4; ++e) {
+                            const float uk = U[4 * j + e] * kk[e];
+                            o0 = fmaf(rr[e], fmaf(uk, v.x, S[0][4 * j + e]), o0);
+                            o1 = fmaf(rr[e], fmaf(uk, v.y, S[1][4 * j + e]), o1);
+                            S[0][4 * j + e] = fmaf(ww[e], S[0][4 * j + e], kk[e] * v.x);
+                            S[1][4 * j + e] = fmaf(ww[e], S[1][4 * j + e], kk[e] * v.y);
+                        }
+                    }
+                    part[2 * i] = o0;
+                    part[2 * i + 1] = o1;
+                } else {
+                    const float2 gb = *reinterpret_cast<const float2*>(s_v + (size_t)TT * cols + 4 * t);
+                    float d0[2] = {0.f, 0.f}, d1[2] = {0.f, 0.f};
+                    float kk[KE];
+#pragma unroll
+                    for (int j = 0; j < NJ; ++j) {
+                        const float4 k = k4[j * 8];
+                        kk[4 * j] = k.x; kk[4 * j + 1] = k.y; kk[4 * j + 2] = k.z; kk[4 * j + 3] = k.w;
+                    }
+#pragma unroll
+                    for (int e = 0; e < KE; ++e) {
+                        d0[e & 1] = fmaf(S[0][e], kk[e], d0[e & 1]);
+                        d1[e & 1] = fmaf(S[1][e], kk[e], d1[e & 1]);
+                    }
+                    float m0 = d0[0] + d0[1], m1 = d1[0] + d1[1];
+#pragma unroll
+                    for (int x = 1; x < 8; x <<= 1) {
+                        m0 += __shfl_xor_sync(0xffffffffu, m0, x);
+                        m1 += __shfl_xor_sync(0xffffffffu, m1, x);
+                    }
+                    const float u0 = gb.y * (v.x - gb.x * m0), u1 = gb.y * (v.y - gb.x * m1);
+                    float o0 = 0.f, o1 = 0.f;
+#pragma unroll
+                    for (int j = 0; j < NJ; ++j) {
+                        const float4 q = q4[j * 8];
+                        const float qq[4] = {q.x, q.y, q.z, q.w};
+#pragma unroll
+                        for (int e = 0; e < 4; ++e) {
+                            S[0][4 * j + e] = fmaf(kk[4 * j + e], u0, gb.x * S[0][4 * j + e]);
+                            S[1][4 * j + e] = fmaf(kk[4 * j + e], u1, gb.x * S[1][4 * j + e]);
+                            o0 = fmaf(S[0][4 * j + e], qq[e], o0);
+                            o1 = fmaf(S[1][4 * j + e], qq[e], o1);
+                        }
+                    }
+                    part[2 * i] = o0;
+                    part[2 * i + 1] = o1;
+                }
+            }
+            const float o = fold8(part, ks);
+            const int t = t0 + (ks >> 1), c = c_loc + (ks & 1);
+            if (t < m && col0 + c < a.vdim) {
+                if (FINISH) s_o[t * cols + c] = o;
+                else a.out[(int64_t)(first + ch * TT + t) * a.heads * a.vdim + head * a.vdim + col0 + c] = o;
+            }
+        }
+        __syncthreads();  // the stage is free for the chunk after next, and the output rows are complete
+        if (FINISH) {
+            for (int t = warp; t < m; t += (int)(blockDim.x >> 5)) finish_head_row(a, s_o + t * cols, first + ch * TT + t, head, lane);
+            __syncthreads();
+        }
+    }
+
+#pragma unroll
+    for (int c = 0; c < 2; ++c) {
+        const int v = col0 + c_loc + c;
+        if (v >= a.vdim) continue;
+        float4* dst = reinterpret_cast<float4*>(a.state + ((int64_t)half.y * a.heads + head) * head_state + (int64_t)v * KD);
+#pragma unroll
+        for (int j = 0; j < NJ; ++j) dst[j * 8 + ks] = make_float4(S[c][4 * j], S[c][4 * j + 1], S[c][4 * j + 2], S[c][4 * j + 3]);
+    }
+}
+
+__global__ void __launch_bounds__(128) head_norm_gate_kernel(LinearStateArgs a, int rows) {
+    pdl_trigger();
+    pdl_wait();
+    const int64_t i = (int64_t)blockIdx.x * 4 + (threadIdx.x >> 5);
+    if (i >= (int64_t)rows * a.heads) return;
+    const int64_t row = i / a.heads;
+    const int head = (int)(i % a.heads);
+    finish_head_row(a, a.out + row * a.heads * a.vdim + head * a.vdim, row, head, threadIdx.x & 31);
+}
+
+template <int KD, bool WKV, bool FINISH>
+void launch_variant(const WkvScanArgs& wa, const DeltaScanArgs& da, cudaStream_t s) {
+    const LinearStateArgs& a = WKV ? wa.common : da.common;
+    const int warps = FINISH ? (a.vdim + LS_COLS - 1) / LS_COLS : LS_WIDE_WARPS;
+    const int cols = warps * LS_COLS;
+    const size_t smem = LsSmem<KD, FINISH ? 4 : 16, WKV>::bytes(cols, FINISH);
+    auto* kernel = linear_state_kernel<KD, WKV, FINISH>;
+    ensure_dynamic_smem(reinterpret_cast<const void*>(kernel), smem);
+    const dim3 grid((unsigned)((a.vdim + cols - 1) / cols), (unsigned)a.heads, (unsigned)a.lanes.lanes);
+    launch_pdl(kernel, grid, dim3((unsigned)warps * 32), smem, s, wa, da);
+    MK_LAUNCH_CHECK();
+}
+
+template <bool WKV>
+void launch_scan(const WkvScanArgs& wa, const DeltaScanArgs& da, cudaStream_t s) {
+    const LinearStateArgs& a = WKV ? wa.common : da.common;
+    if (a.lanes.lanes <= 0) return;
+    if (a.heads > 65535 || a.lanes.lanes > 65535) throw std::runtime_error("linear-attention scan: at most 65535 heads and lanes");
+    const bool finish = a.image.h != nullptr || a.image.f != nullptr;
+    if (finish && !linear_state_can_finish(a.dim, a.vdim)) throw std::runtime_error("linear-attention scan: the finishing form takes dimensions up to 128");
+    switch (linear_state_key_pad(a.dim)) {
+        case 32: finish ? launch_variant<32, WKV, true>(wa, da, s) : launch_variant<32, WKV, false>(wa, da, s); break;
+        case 64: finish ? launch_variant<64, WKV, true>(wa, da, s) : launch_variant<64, WKV, false>(wa, da, s); break;
+        case 128: finish ? launch_variant<128, WKV, true>(wa, da, s) : launch_variant<128, WKV, false>(wa, da, s); break;
+        default: launch_variant<256, WKV, false>(wa, da, s); break;
+    }
+}
+
+}  // namespace
+
+int linear_state_key_pad(int dim) {
+    for (int p : {32, 64, 128, 256})
+        if (dim <= p) return p;
+    throw std::runtime_error("a recurrent head dimension above 256 is not supported");
+}
+
+bool linear_state_can_finish(int dim, int vdim) { return dim <= 128 && vdim <= LS_MAX_FINISH_V; }
+
+void launch_wkv_scan(const WkvScanArgs& a, cudaStream_t s) { launch_scan<true>(a, DeltaScanArgs{}, s); }
+
+void launch_delta_scan(const DeltaScanArgs& a, cudaStream_t s) {
+    if (a.kv_heads <= 0 || a.common.heads % a.kv_heads != 0) throw std::runtime_error("delta-rule scan: heads must be a multiple of kv_heads");
+    launch_scan<false>(WkvScanArgs{}, a, s);
+}
+
+void launch_head_norm_gate(const LinearStateArgs& a, int rows, cudaStream_t s) {
+    if (rows <= 0) return;
+    const int64_t items = (int64_t)rows * a.heads;
+    launch_pdl(head_norm_gate_kernel, dim3((unsigned)((items + 3) / 4)), dim3(128), 0, s, a, rows);
+    MK_LAUNCH_CHECK();
+}
+
+}  // namespace mk

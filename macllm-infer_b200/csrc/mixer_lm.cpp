@@ -1,0 +1,839 @@
+// See mixer_lm.h.
+#include "mixer_lm.h"
+#include "model_registry.h"
+#include "qstream_tc.h"
+#include <algorithm>
+#include <cmath>
+#include <cstring>
+#include <fstream>
+#include <sstream>
+#include <sys/stat.h>
+
+namespace mk {
+
+namespace {
+
+const std::vector<const char*> class_names = {"hgemm_tc", "hgemm_tc_splitk", "f32_matmul", "wkv_scan", "delta_scan", "paged_attention", "rope_kv_scatter",
+                                              "row_update", "delta_prep", "wkv_decay", "gates", "embed", "build_batch", "argmax"};
+
+int pad_to(int64_t n, int m) { return (int)((n + m - 1) / m * m); }
+
+bool is_mixer_checkpoint(const std::string& dir) {
+    struct stat st;
+    return stat((dir + "/config.json").c_str(), &st) == 0 && S_ISREG(st.st_mode);
+}
+
+const RegisterModelFormat register_mixer_format(ModelFormat{
+    "folder with config.json and model.safetensors", is_mixer_checkpoint,
+    [](const std::string& path, const ModelConfig& cfg) -> std::unique_ptr<PagedLm> { return std::make_unique<MixerLm>(path, cfg); }});
+
+MixerSpec read_spec(const std::string& dir, const SafetensorsFile& f) {
+    std::ifstream in(dir + "/config.json", std::ios::binary);
+    std::stringstream text;
+    text << in.rdbuf();
+    const std::string s = text.str();
+    return read_mixer_spec(Json::parse(s.data(), s.size(), "config"), f);
+}
+
+constexpr int kShortLane = 4;  // lanes up to this many tokens: the recurrence kernels finish the head rows themselves
+
+}  // namespace
+
+struct MixerLm::Pending {
+    int n = 0;
+    Shares y[2];
+    const float* w[2] = {nullptr, nullptr};
+    float coef = 1.f;
+};
+
+MixerLm::MixerLm(const std::string& dir, const ModelConfig& cfg) : DeviceLm(cfg, class_names) {
+    const SafetensorsFile f(dir + "/model.safetensors");
+    ms_ = read_spec(dir, f);
+    f32_ = cfg.compute_f32;
+    esz_ = f32_ ? 4 : 2;
+    if (f32_) cfg_.kv_f16 = false;
+    if (cfg.ep_size > 1) throw std::runtime_error("expert parallelism asked for a model without experts");
+    open_device();
+    spec_.vocab = ms_.vocab;
+    spec_.layers = (int)ms_.layers.size();
+    spec_.hidden = ms_.width;
+    // every layer kind of these decoders carries a recurrent state, of which a prompt prefix keeps no copy
+    init_pool(cfg_.block_tokens, cfg_.slab_blocks, cfg_.kv_capacity_tokens, cfg_.prefix_capacity_tokens, "recurrent layers");
+    init_state_slots(cfg_.state_slots > 0 ? cfg_.state_slots : cfg_.max_batch_lanes);
+    spec_.max_context = (int)std::min<int64_t>(pool_->max_blocks() * pool_->block_tokens(), 1 << 30);
+    lw_.resize(ms_.layers.size());
+    load(f);
+    alloc_activations();
+    MK_CUDA(cudaStreamSynchronize(stream_));
+}
+
+MixerLm::~MixerLm() {
+    if (stream_) cudaStreamSynchronize(stream_);
+}
+
+// ---------------------------------------------------------------------------- load
+
+void MixerLm::upload_f32(const std::vector<float>& v, DevBuf& out) {
+    out.upload(v.data(), v.size() * 4, stream_);
+    MK_CUDA(cudaStreamSynchronize(stream_));
+}
+
+void MixerLm::upload_norm(const SafetensorsFile& f, const std::string& name, Norm& out) {
+    upload_f32(f.values(name, {ms_.width}), out.w);
+    upload_f32(f.values(name + ".b", {ms_.width}), out.b);
+    out.alpha = f.values(name + ".alpha", {}).at(0);
+}
+
+void MixerLm::upload_dense(const SafetensorsFile& f, const std::vector<Part>& parts, int64_t rows, int cols, Dense& out,
+                           const std::vector<int64_t>& group_rows) {
+    const int ld = pad_to(cols, 64);
+    std::vector<float> m((size_t)(rows * ld), 0.f);
+    out.bytes = 0;
+    for (const Part& p : parts) {
+        const std::vector<float> v = f.values(p.name, {p.rows, cols});
+#pragma omp parallel for
+        for (int r = 0; r < p.rows; ++r) memcpy(&m[(size_t)(p.at + (int64_t)r * p.step) * ld], &v[(size_t)r * cols], (size_t)cols * 4);
+        out.bytes += (int64_t)p.rows * cols * esz_;
+    }
+    out.rows = rows;
+    out.ld = ld;
+    out.n_groups = 1;
+    if (group_rows.size() > 1) {
+        out.n_groups = (int)group_rows.size();
+        int64_t end = 0;
+        for (size_t g = 0; g < group_rows.size(); ++g) out.group_end[g] = (int)((end += group_rows[g]) / 128);
+    }
+    if (f32_) upload_f32(m, out.f32);
+    else build_bf16_weight(m.data(), rows, ld, out.half, stream_, group_rows);
+    spec_.weight_bytes += out.bytes;
+    spec_.weight_bytes_per_token += out.bytes;
+}
+
+int MixerLm::rope_table(const RotarySpec& r) {
+    for (size_t i = 0; i < rope_.size(); ++i)
+        if (rope_[i]->spec == r) return (int)i;
+    auto t = std::make_unique<RopeTable>();
+    t->spec = r;
+    if (r.dims > 0) {
+        // angles in f64, so that a far position is as exact as a near one
+        const std::vector<double> freq = rotary_frequencies(r);
+        const int64_t positions = pool_->max_blocks() * pool_->block_tokens(), half = r.dims / 2;
+        std::vector<float> c((size_t)(positions * half)), s((size_t)(positions * half));
+#pragma omp parallel for
+        for (int64_t p = 0; p < positions; ++p)
+            for (int64_t i = 0; i < half; ++i) {
+                const double a = (double)p * freq[(size_t)i];
+                c[(size_t)(p * half + i)] = (float)std::cos(a);
+                s[(size_t)(p * half + i)] = (float)std::sin(a);
+            }
+        upload_f32(c, t->cos_t);
+        upload_f32(s, t->sin_t);
+    }
+    rope_.push_back(std::move(t));
+    return (int)rope_.size() - 1;
+}
+
+int MixerLm::geometry_of(const AttentionSpec& a) {
+    const int need = std::max(a.dim, a.vdim);
+    Geometry g;
+    g.heads = a.heads;
+    g.kv_heads = a.kv_heads;
+    // the tensor-core kernels take rows of 64, 128 or 256; narrower heads are padded with zeros in the pools
+    for (int d : {64, 128, 256})
+        if (need <= d && !g.tc && attention_tc_supported(a.heads, a.kv_heads, d, cfg_.block_tokens, cfg_.kv_f16)) {
+            g.tc = true;
+            g.row_width = d;
+        }
+    if (!g.tc) g.row_width = pad_to(need, 4);
+    if (g.row_width > 256) throw std::runtime_error("attention head dimensions above 256 are not supported");
+    if (a.heads / a.kv_heads > 64) throw std::runtime_error("more than 64 query heads per key/value head are not supported");
+    for (size_t i = 0; i < geo_.size(); ++i)
+        if (geo_[i].heads == g.heads && geo_[i].kv_heads == g.kv_heads && geo_[i].row_width == g.row_width) return (int)i;
+    geo_.push_back(std::move(g));
+    return (int)geo_.size() - 1;
+}
+
+void MixerLm::load(const SafetensorsFile& f) {
+    const int C = ms_.width;
+    // token tables stay as rows to gather
+    auto table = [&](const std::string& name, int64_t cols, DevBuf& out) {
+        if (f32_) upload_f32(f.values(name, {ms_.vocab, cols}), out);
+        else {
+            const std::vector<uint16_t> bits = f.bf16_values(name, {ms_.vocab, cols});
+            out.upload(bits.data(), bits.size() * 2, stream_);
+            MK_CUDA(cudaStreamSynchronize(stream_));
+        }
+        spec_.weight_bytes += ms_.vocab * cols * esz_;
+    };
+    table("embed", C, embed_);
+    if (ms_.side_dim > 0) table("side.embed", (int64_t)ms_.layers.size() * ms_.side_dim, side_embed_);
+    for (int l = 0; l < (int)ms_.layers.size(); ++l) load_layer(f, l);
+    upload_norm(f, "final.norm", final_norm_);
+    upload_dense(f, {{"head", ms_.vocab, 0}}, ms_.vocab, C, head_);
+}
+
+void MixerLm::load_layer(const SafetensorsFile& f, int l) {
+    const MixerLayerSpec& s = ms_.layers[(size_t)l];
+    Layer& w = lw_[(size_t)l];
+    const int C = ms_.width;
+    const int64_t halves = (int64_t)state_slots_->capacity() * 2;
+    const std::string p = "l" + std::to_string(l) + ".", m = p + "mix.";
+    upload_norm(f, p + "norm1", w.norm1);
+    if (s.kind == MixerKind::Wkv) {
+        const int HD = s.wkv.heads * s.wkv.dim, R = s.wkv.rank;
+        // r, k, v, g and the decay's low-rank input, each over its own mix of the token and its predecessor
+        const int big = pad_to(HD, 128), low = pad_to(R, 128);
+        w.c_q = 0; w.c_k = big; w.c_v = 2 * big; w.c_g = 3 * big; w.c_low = 4 * big;
+        upload_dense(f, {{m + "r", HD, w.c_q}, {m + "k", HD, w.c_k}, {m + "v", HD, w.c_v}, {m + "g", HD, w.c_g}, {m + "w1", R, w.c_low}}, 4 * (int64_t)big + low, C,
+                     w.in, {big, big, big, big, low});
+        std::vector<float> mu;
+        for (const char* name : {"r", "k", "v", "g", "w"}) {
+            const std::vector<float> v = f.values(m + "mu." + name, {C});
+            mu.insert(mu.end(), v.begin(), v.end());
+        }
+        upload_f32(mu, w.mu);
+        const std::vector<float> w2 = f.values(m + "w2", {HD, R});
+        std::vector<float> w2t((size_t)HD * R);
+        for (int c = 0; c < HD; ++c)
+            for (int j = 0; j < R; ++j) w2t[(size_t)j * HD + c] = w2[(size_t)c * R + j];
+        upload_f32(w2t, w.w2t);
+        spec_.weight_bytes += (int64_t)HD * R * 4;
+        spec_.weight_bytes_per_token += (int64_t)HD * R * 4;
+        upload_f32(f.values(m + "w0", {HD}), w.w0);
+        upload_f32(f.values(m + "u", {s.wkv.heads, s.wkv.dim}), w.bonus);
+        upload_f32(f.values(m + "norm", {HD}), w.head_norm);
+        upload_dense(f, {{m + "o", C, 0}}, C, HD, w.out);
+        w.kept.alloc((size_t)halves * C * 4);
+        w.state.alloc((size_t)halves * HD * linear_state_key_pad(s.wkv.dim) * 4);
+    } else {
+        const AttentionSpec& a = s.attn;
+        const DeltaSpec& d = s.delta;
+        const std::string L = m + "left.", Rt = m + "right.";
+        // every projection of both branches reads the same input: one stacked matrix
+        std::vector<Part> parts;
+        int at = 0;
+        auto part = [&](const std::string& name, int rows) {
+            const int here = at;
+            parts.push_back({name, rows, here});
+            at = pad_to(at + rows, 4);
+            return here;
+        };
+        w.c_q = part(L + "q", a.heads * a.dim);
+        w.c_k = part(L + "k", a.kv_heads * a.dim);
+        w.c_v = part(L + "v", a.kv_heads * a.vdim);
+        w.c_g = part(L + "g", a.heads);
+        w.d_q = part(Rt + "q", d.kv_heads * d.dim);
+        w.d_k = part(Rt + "k", d.kv_heads * d.dim);
+        w.d_v = part(Rt + "v", d.heads * d.vdim);
+        w.d_a = part(Rt + "a", d.heads);
+        w.d_b = part(Rt + "b", d.heads);
+        w.d_g = part(Rt + "g", d.heads * d.vdim);
+        upload_dense(f, parts, at, C, w.in);
+        upload_f32(f.values(L + "q.norm", {a.dim}), w.q_norm);
+        upload_f32(f.values(L + "k.norm", {a.dim}), w.k_norm);
+        upload_dense(f, {{L + "o", C, 0}}, C, a.heads * a.vdim, w.out);
+        upload_dense(f, {{Rt + "o", C, 0}}, C, d.heads * d.vdim, w.out2);
+        upload_f32(f.values(m + "left.out", {C}), w.out_norm);
+        upload_f32(f.values(m + "right.out", {C}), w.out2_norm);
+        w.geometry = geometry_of(a);
+        w.row_width = geo_[(size_t)w.geometry].row_width;
+        w.rope = rope_table(a.rot);
+        const int64_t page_bytes = (int64_t)a.kv_heads * cfg_.block_tokens * w.row_width * (cfg_.kv_f16 ? 2 : 4);
+        for (DevBuf* pool : {&w.k_pool, &w.v_pool}) {
+            pool->alloc((size_t)(pool_->max_blocks() * page_bytes));
+            pool->zero(stream_);
+        }
+        spec_.kv_bytes_per_token += 2 * page_bytes / cfg_.block_tokens;
+        // delta rule
+        const int kw = d.kv_heads * d.dim, vw = d.heads * d.vdim, channels = 2 * kw + vw;
+        if (d.dim > 256 || d.vdim > 256) throw std::runtime_error("delta-rule head dimensions above 256 are not supported");
+        std::vector<float> conv((size_t)channels * d.taps);
+        int ch0 = 0;
+        for (const auto& part_of : {std::make_pair("q", kw), std::make_pair("k", kw), std::make_pair("v", vw)}) {
+            const std::vector<float> t = f.values(Rt + part_of.first + ".conv", {part_of.second, d.taps});
+            for (int c = 0; c < part_of.second; ++c)
+                for (int j = 0; j < d.taps; ++j) conv[(size_t)j * channels + ch0 + c] = t[(size_t)c * d.taps + j];
+            ch0 += part_of.second;
+        }
+        upload_f32(conv, w.conv);
+        upload_f32(f.values(Rt + "dt_bias", {d.heads}), w.dt_bias);
+        std::vector<float> decay = f.values(Rt + "A_log", {d.heads});
+        for (float& v : decay) v = (float)-std::exp((double)v);
+        upload_f32(decay, w.log_decay);
+        upload_f32(f.values(Rt + "norm", {d.vdim}), w.head_norm);
+        w.tail.alloc((size_t)halves * std::max(1, d.taps - 1) * channels * 4);
+        w.state.alloc((size_t)halves * vw * linear_state_key_pad(d.dim) * 4);
+    }
+    if (s.ff > 0) {
+        upload_norm(f, p + "norm2", w.norm2);
+        upload_dense(f, {{p + "mlp.gate", s.ff, 0, 2}, {p + "mlp.up", s.ff, 1, 2}}, 2 * (int64_t)s.ff, C, w.gate_up);
+        upload_dense(f, {{p + "mlp.down", C, 0}}, C, s.ff, w.down);
+    }
+    if (ms_.side_dim > 0) {
+        upload_dense(f, {{p + "side.gate", ms_.side_dim, 0}}, ms_.side_dim, C, w.side_gate);
+        upload_dense(f, {{p + "side.proj", C, 0}}, C, ms_.side_dim, w.side_proj);
+        upload_f32(f.values(p + "side.norm", {C}), w.side_norm);
+    }
+}
+
+void MixerLm::alloc_activations() {
+    const int64_t T = cfg_.max_batch_tokens;
+    const int B = cfg_.max_batch_lanes, C = ms_.width;
+    int64_t in_rows = 0, mix = 0, a_w = 0, b_w = 0, ff = 0, hd = 0, raw = 0, dqk = 0, dv = 0, dh = 0, attn = 0;
+    for (size_t l = 0; l < lw_.size(); ++l) {
+        const MixerLayerSpec& s = ms_.layers[l];
+        const Layer& w = lw_[l];
+        in_rows = std::max(in_rows, w.in.rows);
+        ff = std::max(ff, (int64_t)s.ff);
+        if (s.kind == MixerKind::Wkv) {
+            mix = 5;
+            const int64_t n = (int64_t)s.wkv.heads * s.wkv.dim;
+            hd = std::max(hd, n);
+            raw = std::max(raw, n);
+            b_w = std::max(b_w, n);
+        } else {
+            a_w = std::max(a_w, (int64_t)s.attn.heads * s.attn.vdim);
+            attn = std::max(attn, (int64_t)s.attn.heads * w.row_width);
+            const int64_t n = (int64_t)s.delta.heads * s.delta.vdim;
+            b_w = std::max(b_w, n);
+            raw = std::max(raw, n);
+            dqk = std::max(dqk, (int64_t)s.delta.kv_heads * s.delta.dim);
+            dv = std::max(dv, n);
+            dh = std::max(dh, (int64_t)s.delta.heads);
+        }
+    }
+    const int64_t ldc = pad_to(C, 64);
+    for (DevBuf& x : x_) x.alloc((size_t)(T * C) * 4);
+    mixes_.alloc((size_t)(mix * T * ldc) * esz_);
+    img_h_.alloc((size_t)(T * ldc) * esz_);
+    img_a_.alloc((size_t)(T * pad_to(a_w, 64)) * esz_);
+    img_b_.alloc((size_t)(T * pad_to(b_w, 64)) * esz_);
+    img_ff_.alloc((size_t)(T * pad_to(ff, 64)) * esz_);
+    img_ff_.zero(stream_);  // the gated matmul writes the true columns only
+    img_side_.alloc((size_t)(T * pad_to(std::max(ms_.side_dim, 1), 64)) * esz_);
+    y_in_.alloc((size_t)(T * std::max<int64_t>(in_rows, ms_.side_dim)) * 4);
+    y_a_.alloc((size_t)(T * C) * 4);
+    y_b_.alloc((size_t)(T * C) * 4);
+    if (f32_) y_gu_.alloc((size_t)(T * 2 * ff) * 4);
+    decay_.alloc((size_t)(T * hd) * 4);
+    raw_.alloc((size_t)(T * raw) * 4);
+    q_rot_.alloc((size_t)(T * attn) * 4);
+    attn_.alloc((size_t)(T * attn) * 4);
+    dq_.alloc((size_t)(T * dqk) * 4);
+    dk_.alloc((size_t)(T * dqk) * 4);
+    dv_.alloc((size_t)(T * dv) * 4);
+    dbeta_.alloc((size_t)(T * dh) * 4);
+    ddecay_.alloc((size_t)(T * dh) * 4);
+    if (!f32_)
+        for (DevBuf& p : partial_) p.alloc(kSplitScratchBytes);
+    size_t extra = (size_t)B * sizeof(int2) + 16;
+    size_t part_o = 0, part_ml = 0, counters = 0;
+    for (const Geometry& g : geo_) {
+        if (g.tc) {
+            const int entries = attention_tc_max_entries(B, g.kv_heads);
+            attn_max_entries_ = std::max(attn_max_entries_, entries);
+            part_o = std::max(part_o, (size_t)entries * g.kv_heads * 16 * g.row_width * 4);
+            part_ml = std::max(part_ml, (size_t)entries * g.kv_heads * 16 * 2 * 4);
+            counters = std::max(counters, (size_t)B * g.kv_heads * 4);
+            extra += ((size_t)(T + B) * 2 + (size_t)entries * 8 + (size_t)B * 3) * 4 + 64;
+        } else {
+            extra += (size_t)(T + B) * 8 + 64;
+        }
+    }
+    attn_part_o_.alloc(part_o);
+    attn_part_ml_.alloc(part_ml);
+    attn_counters_.alloc(counters);
+    attn_counters_.zero(stream_);
+    alloc_tick(extra);
+}
+
+// ---------------------------------------------------------------------------- forward
+
+RowImage MixerLm::image(DevBuf& b, int ld) const {
+    RowImage im;
+    im.ld = ld;
+    if (f32_) im.f = b.as<float>();
+    else im.h = b.as<__nv_bfloat16>();
+    return im;
+}
+
+Shares MixerLm::matmul(const Dense& W, const RowImage& x, int T, DevBuf& y, int scratch) {
+    Shares out;
+    out.p = y.as<float>();
+    out.ld = (int)W.rows;
+    const double bytes = (double)W.bytes + (double)esz_ * T * W.ld * W.n_groups + 4.0 * T * W.rows, flops = 2.0 * T * (double)W.rows * W.ld;
+    if (f32_) {
+        prof_begin(KC_F32_MATMUL, bytes, flops);
+        launch_f32_matmul(W.f32.as<float>(), W.rows, W.ld, x.f, T, y.as<float>(), (int)W.rows, W.n_groups, W.group_end, stream_);
+    } else {
+        prof_begin(T <= 64 ? KC_GEMM_NARROW : KC_GEMM, bytes, flops);
+        HgemmScratch ws;
+        ws.partial = partial_[scratch].as<float>();
+        ws.partial_floats = partial_[scratch].size() / 4;
+        ws.status = status_.as<int32_t>();
+        const int splits = launch_hgemm_tc(W.half, reinterpret_cast<const __half*>(x.h), T, y.as<float>(), (int)W.rows, 1.f, 0.f, ws, stream_, 16);
+        if (splits > 1) {
+            out.p = ws.partial;
+            out.n = splits;
+            out.stride = (int64_t)T * W.rows;
+        }
+    }
+    prof_end();
+    ++launches_;
+    return out;
+}
+
+void MixerLm::set_norm(RowUpdateArgs& a, const Norm& n) const {
+    a.norm = ms_.norm;
+    a.alpha = n.alpha;
+    a.norm_w = n.w.as<float>();
+    a.norm_b = n.b.as<float>();
+}
+
+// Fills in the residual part of a row update; what is pending is added on the way.
+void MixerLm::apply_pending(RowUpdateArgs& a, Pending& p, bool other_buffer) {
+    a.x = x_[cur_].as<float>();
+    a.width = ms_.width;
+    a.n_add = p.n;
+    for (int i = 0; i < p.n; ++i) {
+        a.add[i] = p.y[i];
+        a.add_w[i] = p.w[i];
+    }
+    a.add_coef = p.coef;
+    a.add_eps = ms_.eps;
+    if (p.n > 0) {
+        if (other_buffer) cur_ ^= 1;
+        a.x_out = x_[cur_].as<float>();
+    }
+    p = Pending{};
+}
+
+void MixerLm::run_wkv(const Tick& t, int l, Pending& pend) {
+    const WkvSpec& s = ms_.layers[(size_t)l].wkv;
+    Layer& w = lw_[(size_t)l];
+    const int T = t.T, C = ms_.width, HD = s.heads * s.dim;
+    RowUpdateArgs u;
+    u.rows = T;
+    apply_pending(u, pend, true);
+    set_norm(u, w.norm1);
+    u.n_mix = 5;
+    u.mu = w.mu.as<float>();
+    u.mixes = image(mixes_, w.in.ld);
+    u.lanes = state_lanes_;
+    u.token_lane = t.bd.token_lane;
+    u.kept = w.kept.as<float>();
+    prof_begin(KC_ROW_UPDATE, (double)T * C * (8.0 + 4.0 * u.n_add + 5.0 * esz_), 0);
+    launch_row_update(u, stream_);
+    prof_end();
+    const Shares y = matmul(w.in, u.mixes, T, y_in_, 0);
+    prof_begin(KC_WKV_DECAY, (double)T * (HD + s.rank) * 4.0 + (double)HD * s.rank * 4.0, 2.0 * T * (double)HD * s.rank);
+    launch_wkv_decay(y, w.c_low, T, s.rank, HD, w.w2t.as<float>(), w.w0.as<float>(), decay_.as<float>(), stream_);
+    prof_end();
+    WkvScanArgs a;
+    a.common.lanes = state_lanes_;
+    a.common.state = w.state.as<float>();
+    a.common.heads = s.heads;
+    a.common.dim = a.common.vdim = s.dim;
+    a.common.out = raw_.as<float>();
+    a.common.norm_w = w.head_norm.as<float>();
+    a.common.norm_per_head = 1;
+    a.common.eps = ms_.eps;
+    a.common.gate = y;
+    a.common.gate_col = w.c_g;
+    a.rkv = y;
+    a.r_col = w.c_q;
+    a.k_col = w.c_k;
+    a.v_col = w.c_v;
+    a.decay = decay_.as<float>();
+    a.bonus = w.bonus.as<float>();
+    const RowImage img = image(img_b_, w.out.ld);
+    const bool finish = short_lanes_ && linear_state_can_finish(s.dim, s.dim);
+    if (finish) a.common.image = img;
+    prof_begin(KC_WKV_SCAN, (double)T * HD * 20.0 + 8.0 * t.B * HD * s.dim, 8.0 * T * (double)HD * s.dim);
+    launch_wkv_scan(a, stream_);
+    prof_end();
+    launches_ += 3;
+    if (!finish) {
+        a.common.image = img;
+        prof_begin(KC_GATES, (double)T * HD * (8.0 + esz_), 0);
+        launch_head_norm_gate(a.common, T, stream_);
+        prof_end();
+        ++launches_;
+    }
+    pend.n = 1;
+    pend.y[0] = matmul(w.out, img, T, y_a_, 1);
+}
+
+void MixerLm::run_parallel(const Tick& t, int l, Pending& pend, const std::vector<LmLane>& lanes) {
+    const AttentionSpec& s = ms_.layers[(size_t)l].attn;
+    const DeltaSpec& d = ms_.layers[(size_t)l].delta;
+    Layer& w = lw_[(size_t)l];
+    const int T = t.T, C = ms_.width, D = w.row_width, bt = cfg_.block_tokens;
+    RowUpdateArgs u;
+    u.rows = T;
+    apply_pending(u, pend, false);
+    set_norm(u, w.norm1);
+    u.normed = image(img_h_, w.in.ld);
+    prof_begin(KC_ROW_UPDATE, (double)T * C * (8.0 + 4.0 * u.n_add + esz_), 0);
+    launch_row_update(u, stream_);
+    prof_end();
+    const Shares y = matmul(w.in, u.normed, T, y_in_, 0);
+    ++launches_;
+
+    // ---- attention: head norms, rotation, page write, softmax, head gate
+    Geometry& g = geo_[(size_t)w.geometry];
+    RopeKvArgs ra;
+    ra.q = const_cast<float*>(y.p) + w.c_q;
+    ra.k = y.p + w.c_k;
+    ra.v = y.p + w.c_v;
+    ra.ldq = ra.ldk = ra.ldv = y.ld;
+    ra.qk_splits = ra.v_splits = y.n;
+    ra.qk_split_stride = ra.v_split_stride = y.stride;
+    ra.q_out = q_rot_.as<float>();
+    ra.ldq_out = s.heads * D;
+    ra.q_norm_w = w.q_norm.as<float>();
+    ra.k_norm_w = w.k_norm.as<float>();
+    ra.norm_eps = ms_.eps;
+    if (s.rot.dims > 0) {
+        ra.cos_t = rope_[(size_t)w.rope]->cos_t.as<float>();
+        ra.sin_t = rope_[(size_t)w.rope]->sin_t.as<float>();
+        ra.rotary_dim = s.rot.dims;
+        ra.interleaved = s.rot.interleaved ? 1 : 0;
+    }
+    ra.positions = t.bd.positions;
+    ra.slots = t.bd.slots;
+    ra.k_pool = w.k_pool.ptr();
+    ra.v_pool = w.v_pool.ptr();
+    ra.kv_f16 = cfg_.kv_f16 ? 1 : 0;
+    ra.T = T;
+    ra.q_heads = s.heads;
+    ra.kv_heads = s.kv_heads;
+    ra.d = s.dim;
+    ra.dv = s.vdim;
+    ra.d_row = D;
+    ra.block_tokens = bt;
+    ra.layers = 1;
+    ra.layer = 0;
+    ra.pool_blocks = pool_->max_blocks();
+    // ticks of one-token lanes: the attention kernel prepares its own rows
+    const bool fuse_rope = g.tc && g.plan.n_tiles() == 0 && g.plan.n_entries() > 0 && g.plan.n_dec_lanes() == 0;
+    const double kv_esz = cfg_.kv_f16 ? 2.0 : 4.0;
+    if (!fuse_rope) {
+        prof_begin(KC_ROPE_KV, (double)T * s.heads * (s.dim + D) * 4.0 + (double)T * s.kv_heads * (s.dim + s.vdim + 0.5 * kv_esz * D) * 4.0, 0);
+        launch_rope_kv(ra, stream_);
+        prof_end();
+        ++launches_;
+    }
+    double kv_tokens = 0, flops = 0;
+    for (const LmLane& ln : lanes) {
+        kv_tokens += (double)ln.start_pos + ln.n_tokens;
+        flops += 2.0 * s.heads * (s.dim + s.vdim) * ((double)ln.n_tokens * ln.start_pos + 0.5 * ln.n_tokens * ln.n_tokens);
+    }
+    prof_begin(KC_ATTN, kv_tokens * 2 * s.kv_heads * D * kv_esz + 8.0 * T * s.heads * D, flops);
+    if (g.tc) {
+        AttnTcArgs ta;
+        ta.q = q_rot_.as<float>();
+        ta.out = attn_.as<float>();
+        ta.k_pool = w.k_pool.ptr();
+        ta.v_pool = w.v_pool.ptr();
+        ta.hdr = t.bd.hdr;
+        ta.tables = t.bd.tables;
+        ta.cu_seqlens = t.bd.cu_seqlens;
+        ta.tiles = reinterpret_cast<const int32_t*>(t.dp + g.off_tiles);
+        ta.entries = reinterpret_cast<const int32_t*>(t.dp + g.off_entries);
+        ta.dec_lanes = reinterpret_cast<const int32_t*>(t.dp + g.off_dec);
+        ta.n_tiles = g.plan.n_tiles();
+        ta.n_entries = g.plan.n_entries();
+        ta.n_dec_lanes = g.plan.n_dec_lanes();
+        ta.part_o = attn_part_o_.as<float>();
+        ta.part_ml = attn_part_ml_.as<float>();
+        ta.counters = attn_counters_.as<int32_t>();
+        ta.q_heads = s.heads;
+        ta.kv_heads = s.kv_heads;
+        ta.d = D;
+        ta.block_tokens = bt;
+        ta.layers = 1;
+        ta.pool_blocks = ra.pool_blocks;
+        ta.scale = s.scale;
+        if (fuse_rope) {
+            ta.fused_rope = 1;
+            ta.rk = ra;
+        }
+        launches_ += launch_paged_attention_tc(ta, stream_);
+    } else {
+        AttnArgs at;
+        at.q = q_rot_.as<float>();
+        at.out = attn_.as<float>();
+        at.k_pool = w.k_pool.ptr();
+        at.v_pool = w.v_pool.ptr();
+        at.kv_f16 = ra.kv_f16;
+        at.batch = t.bd;
+        at.batch.tile_lane = reinterpret_cast<int32_t*>(t.dp + g.off_tile_lane);
+        at.batch.tile_row0 = reinterpret_cast<int32_t*>(t.dp + g.off_tile_row);
+        at.batch.max_tiles = (int)g.tile_lane.size();
+        at.q_heads = s.heads;
+        at.kv_heads = s.kv_heads;
+        at.d = D;
+        at.block_tokens = bt;
+        at.layers = 1;
+        at.pool_blocks = ra.pool_blocks;
+        at.scale = s.scale;
+        at.q_tile = attention_q_tile(s.heads, s.kv_heads);
+        launch_paged_attention(at, stream_);
+        ++launches_;
+    }
+    prof_end();
+    const RowImage img_a = image(img_a_, w.out.ld);
+    prof_begin(KC_GATES, (double)T * s.heads * (D * 4.0 + s.vdim * (double)esz_), 0);
+    launch_head_gate(attn_.as<float>(), T, s.heads, D, s.vdim, y, w.c_g, img_a, stream_);
+    prof_end();
+
+    // ---- gated delta rule
+    DeltaPrepArgs dp;
+    dp.y = y;
+    dp.q_col = w.d_q;
+    dp.k_col = w.d_k;
+    dp.v_col = w.d_v;
+    dp.a_col = w.d_a;
+    dp.b_col = w.d_b;
+    dp.rows = T;
+    dp.heads = d.heads;
+    dp.kv_heads = d.kv_heads;
+    dp.dim = d.dim;
+    dp.vdim = d.vdim;
+    dp.taps = d.taps;
+    dp.conv = w.conv.as<float>();
+    dp.dt_bias = w.dt_bias.as<float>();
+    dp.log_decay = w.log_decay.as<float>();
+    dp.lanes = state_lanes_;
+    dp.token_lane = t.bd.token_lane;
+    dp.tail = w.tail.as<float>();
+    dp.q = dq_.as<float>();
+    dp.k = dk_.as<float>();
+    dp.v = dv_.as<float>();
+    dp.beta = dbeta_.as<float>();
+    dp.decay = ddecay_.as<float>();
+    const double channels = 2.0 * d.kv_heads * d.dim + (double)d.heads * d.vdim;
+    prof_begin(KC_DELTA_PREP, 8.0 * T * channels, 0);
+    launch_delta_prep(dp, stream_);
+    prof_end();
+    DeltaScanArgs sc;
+    sc.common.lanes = state_lanes_;
+    sc.common.state = w.state.as<float>();
+    sc.common.heads = d.heads;
+    sc.common.dim = d.dim;
+    sc.common.vdim = d.vdim;
+    sc.common.out = raw_.as<float>();
+    sc.common.norm_w = w.head_norm.as<float>();
+    sc.common.eps = ms_.eps;
+    sc.common.gate = y;
+    sc.common.gate_col = w.d_g;
+    sc.kv_heads = d.kv_heads;
+    sc.q = dp.q;
+    sc.k = dp.k;
+    sc.v = dp.v;
+    sc.decay = dp.decay;
+    sc.beta = dp.beta;
+    const RowImage img_b = image(img_b_, w.out2.ld);
+    const bool finish = short_lanes_ && linear_state_can_finish(d.dim, d.vdim);
+    if (finish) sc.common.image = img_b;
+    const double vw = (double)d.heads * d.vdim;
+    prof_begin(KC_DELTA_SCAN, 4.0 * T * (channels + vw) + 8.0 * t.B * vw * d.dim, 8.0 * T * vw * d.dim);
+    launch_delta_scan(sc, stream_);
+    prof_end();
+    launches_ += 3;
+    if (!finish) {
+        sc.common.image = img_b;
+        prof_begin(KC_GATES, T * vw * (8.0 + esz_), 0);
+        launch_head_norm_gate(sc.common, T, stream_);
+        prof_end();
+        ++launches_;
+    }
+    pend.n = 2;
+    pend.y[0] = matmul(w.out, img_a, T, y_a_, 1);
+    pend.y[1] = matmul(w.out2, img_b, T, y_b_, 2);
+    pend.w[0] = w.out_norm.as<float>();
+    pend.w[1] = w.out2_norm.as<float>();
+    pend.coef = 0.5f;
+}
+
+void MixerLm::run_forward(const std::vector<LmLane>& lanes, KvReservation& r, uint32_t flags) {
+    Tick t = stage_tick(lanes, r, flags);
+    const int B = t.B, T = t.T, R = t.R, C = ms_.width;
+    std::vector<int2> halves;
+    int longest = 0;
+    for (const LmLane& l : lanes) {
+        halves.push_back(make_int2(l.state_in, l.state_out));
+        longest = std::max(longest, l.n_tokens);
+    }
+    short_lanes_ = longest <= kShortLane;
+    const size_t off_halves = stage_bytes(t, halves.data(), halves.size() * sizeof(int2));
+    std::vector<int32_t> sp((size_t)B), nt((size_t)B), nb((size_t)B);
+    for (int i = 0; i < B; ++i) {
+        sp[(size_t)i] = lanes[(size_t)i].start_pos;
+        nt[(size_t)i] = lanes[(size_t)i].n_tokens;
+        nb[(size_t)i] = t.hdr[i].n_blocks;
+    }
+    for (Geometry& g : geo_) {
+        if (g.tc) {
+            plan_attention_tc(sp.data(), nt.data(), nb.data(), B, g.heads, g.kv_heads, g.plan);
+            if (g.plan.n_entries() > attn_max_entries_) throw std::runtime_error("attention work list exceeds its scratch");
+            g.off_entries = stage_bytes(t, g.plan.entries.data(), g.plan.entries.size() * 4);
+            g.off_tiles = stage_bytes(t, g.plan.tiles.data(), g.plan.tiles.size() * 4);
+            g.off_dec = stage_bytes(t, g.plan.dec_lanes.data(), g.plan.dec_lanes.size() * 4);
+        } else {
+            const int q_tile = attention_q_tile(g.heads, g.kv_heads);
+            g.tile_lane.clear();
+            g.tile_row.clear();
+            for (int i = 0; i < B; ++i)
+                for (int r0 = 0; r0 < nt[(size_t)i]; r0 += q_tile) {
+                    g.tile_lane.push_back(i);
+                    g.tile_row.push_back(r0);
+                }
+            g.off_tile_lane = stage_bytes(t, g.tile_lane.data(), g.tile_lane.size() * 4);
+            g.off_tile_row = stage_bytes(t, g.tile_row.data(), g.tile_row.size() * 4);
+        }
+    }
+    upload_tick(t, 64, KC_BATCH);
+    state_lanes_.cu = t.bd.cu_seqlens;
+    state_lanes_.halves = reinterpret_cast<const int2*>(t.dp + off_halves);
+    state_lanes_.lanes = B;
+    // copy-on-write page copies of shared partial tails
+    for (const KvCowCopy& c : r.cow_copies())
+        for (size_t l = 0; l < lw_.size(); ++l)
+            if (lw_[l].row_width > 0) {
+                launch_cow_copy(lw_[l].k_pool.ptr(), lw_[l].v_pool.ptr(), cfg_.kv_f16 ? 1 : 0, c.src_slot, c.dst_slot, c.rows, 1, pool_->max_blocks(),
+                                ms_.layers[l].attn.kv_heads, cfg_.block_tokens, lw_[l].row_width, stream_);
+                ++launches_;
+            }
+    cur_ = 0;
+    QWeight table;
+    table.type = f32_ ? QT_F32 : QT_BF16;
+    table.rows = ms_.vocab;
+    table.cols = C;
+    table.p0 = embed_.ptr();
+    prof_begin(KC_EMBED, (4.0 + esz_) * T * C, 0);
+    launch_embed(table, t.ids, T, 1.f, x_[cur_].as<float>(), stream_);
+    prof_end();
+    ++launches_;
+    if (capture_) captured_.ensure((size_t)lw_.size() * T * C * 4);
+    captured_tokens_ = T;
+
+    Pending pend;
+    for (int l = 0; l < (int)lw_.size(); ++l) {
+        const MixerLayerSpec& s = ms_.layers[(size_t)l];
+        Layer& w = lw_[(size_t)l];
+        if (s.kind == MixerKind::Wkv) run_wkv(t, l, pend);
+        else run_parallel(t, l, pend, lanes);
+        if (s.ff > 0) {
+            RowUpdateArgs u;
+            u.rows = T;
+            apply_pending(u, pend, false);
+            set_norm(u, w.norm2);
+            u.normed = image(img_h_, w.gate_up.ld);
+            prof_begin(KC_ROW_UPDATE, (double)T * C * (8.0 + 4.0 * u.n_add + esz_), 0);
+            launch_row_update(u, stream_);
+            prof_end();
+            const RowImage img = image(img_ff_, w.down.ld);
+            if (f32_) {
+                const Shares gu = matmul(w.gate_up, u.normed, T, y_gu_, 0);
+                prof_begin(KC_GATES, 12.0 * T * s.ff, 0);
+                launch_gated_act(gu, T, s.ff, img, stream_);
+                prof_end();
+            } else {
+                // silu(gate) * up in the matmul's epilogue
+                prof_begin(T <= 64 ? KC_GEMM_NARROW : KC_GEMM, (double)w.gate_up.bytes + 2.0 * T * C + 2.0 * T * s.ff, 2.0 * T * (double)w.gate_up.rows * w.gate_up.ld);
+                HgemmScratch ws;
+                ws.status = status_.as<int32_t>();
+                launch_hgemm_tc_gated(w.gate_up.half, reinterpret_cast<const __half*>(u.normed.h), T, 0, reinterpret_cast<__half*>(img.h), img.ld, ws, stream_);
+                prof_end();
+            }
+            launches_ += 2;
+            pend.n = 1;
+            pend.y[0] = matmul(w.down, img, T, y_a_, 1);
+        }
+        if (ms_.side_dim > 0) {
+            RowUpdateArgs u;
+            u.rows = T;
+            apply_pending(u, pend, false);
+            u.raw = image(img_h_, w.side_gate.ld);
+            prof_begin(KC_ROW_UPDATE, (double)T * C * (8.0 + 4.0 * u.n_add + esz_), 0);
+            launch_row_update(u, stream_);
+            prof_end();
+            const Shares z = matmul(w.side_gate, u.raw, T, y_in_, 0);
+            const RowImage img = image(img_side_, w.side_proj.ld);
+            prof_begin(KC_GATES, (double)T * ms_.side_dim * (4.0 + 2.0 * esz_), 0);
+            launch_side_gate(z, T, ms_.side_dim, t.ids, side_embed_.ptr(), f32_ ? 1 : 0, (int64_t)lw_.size() * ms_.side_dim, l * ms_.side_dim, img, stream_);
+            prof_end();
+            launches_ += 2;
+            pend.n = 1;
+            pend.y[0] = matmul(w.side_proj, img, T, y_a_, 1);
+            pend.w[0] = w.side_norm.as<float>();
+        }
+        if (capture_) {
+            RowUpdateArgs u;
+            u.rows = T;
+            apply_pending(u, pend, false);
+            launch_row_update(u, stream_);
+            ++launches_;
+            MK_CUDA(cudaMemcpyAsync(captured_.as<float>() + (size_t)l * T * C, x_[cur_].ptr(), (size_t)T * C * 4, cudaMemcpyDeviceToDevice, stream_));
+        }
+    }
+    if (R > 0 && (flags & (FWD_WANT_LOGITS | FWD_WANT_TOKENS))) {
+        // the rows asked for: last residual add, final norm, output projection
+        img_h_.ensure((size_t)R * head_.ld * esz_);
+        RowUpdateArgs u;
+        u.rows = R;
+        u.row_index = t.out_rows;
+        apply_pending(u, pend, false);
+        u.x_out = nullptr;
+        set_norm(u, final_norm_);
+        u.normed = image(img_h_, head_.ld);
+        prof_begin(KC_ROW_UPDATE, (double)R * C * (4.0 + 4.0 * u.n_add + esz_), 0);
+        launch_row_update(u, stream_);
+        prof_end();
+        ++launches_;
+        // one buffer receives the logits whatever the row count: no K shares here
+        prof_begin(f32_ ? KC_F32_MATMUL : (R <= 64 ? KC_GEMM_NARROW : KC_GEMM), (double)head_.bytes + (double)esz_ * R * C + 4.0 * R * ms_.vocab,
+                   2.0 * R * (double)ms_.vocab * C);
+        if (f32_) {
+            launch_f32_matmul(head_.f32.as<float>(), head_.rows, head_.ld, u.normed.f, R, logits_.as<float>(), ms_.vocab, 1, nullptr, stream_);
+        } else {
+            HgemmScratch ws;
+            ws.status = status_.as<int32_t>();
+            launch_hgemm_tc(head_.half, reinterpret_cast<const __half*>(u.normed.h), R, logits_.as<float>(), ms_.vocab, 1.f, 0.f, ws, stream_, 1);
+        }
+        prof_end();
+        ++launches_;
+    }
+    finish_tick(t, KC_SAMPLE);
+}
+
+// ---------------------------------------------------------------------------- state and taps
+
+void MixerLm::copy_state(int from, int to) {
+    MK_CUDA(cudaSetDevice(cfg_.device));
+    const size_t halves = (size_t)state_slots_->capacity() * 2;
+    for (Layer& w : lw_)
+        for (DevBuf* b : {&w.state, &w.kept, &w.tail}) {
+            if (b->size() == 0) continue;
+            const size_t n = b->size() / halves;
+            MK_CUDA(cudaMemcpyAsync(b->as<uint8_t>() + (size_t)to * n, b->as<uint8_t>() + (size_t)from * n, n, cudaMemcpyDeviceToDevice, stream_));
+        }
+}
+
+void MixerLm::capture_residuals(bool on) {
+    capture_ = on;
+    captured_tokens_ = 0;
+}
+
+int MixerLm::read_residuals(float* out, int64_t capacity) {
+    if (!capture_ || captured_tokens_ == 0) throw std::runtime_error("no forward has left its residual stream");
+    const int64_t n = (int64_t)lw_.size() * captured_tokens_ * ms_.width;
+    if (out == nullptr || capacity < n) throw std::runtime_error("residual buffer needs " + std::to_string(n) + " floats");
+    MK_CUDA(cudaStreamSynchronize(stream_));
+    MK_CUDA(cudaMemcpy(out, captured_.ptr(), (size_t)n * 4, cudaMemcpyDeviceToHost));
+    return captured_tokens_;
+}
+
+}  // namespace mk

@@ -1,0 +1,420 @@
+// See mixer_ops.h.
+#include "mixer_ops.h"
+#include "device_util.h"
+#include "recurrent_core.cuh"
+#include <algorithm>
+
+namespace mk {
+
+namespace {
+
+// ------------------------------------------------------------------------------------------------ residual update
+
+constexpr int RU_THREADS = 256;
+
+template <int VEC>
+struct Pack {
+    float v[VEC];
+};
+template <int VEC>
+__device__ __forceinline__ Pack<VEC> load_pack(const float* p) {
+    Pack<VEC> r;
+    if constexpr (VEC == 4) {
+        const float4 x = *reinterpret_cast<const float4*>(p);
+        r.v[0] = x.x; r.v[1] = x.y; r.v[2] = x.z; r.v[3] = x.w;
+    } else {
+        r.v[0] = *p;
+    }
+    return r;
+}
+template <int VEC>
+__device__ __forceinline__ void store_pack(float* p, const Pack<VEC>& r) {
+    if constexpr (VEC == 4) *reinterpret_cast<float4*>(p) = make_float4(r.v[0], r.v[1], r.v[2], r.v[3]);
+    else *p = r.v[0];
+}
+template <int VEC>
+__device__ __forceinline__ Pack<VEC> share_pack(const Shares& s, int64_t row, int col) {
+    Pack<VEC> r;
+    if constexpr (VEC == 4) {
+        const float4 x = s.at4(row, col);
+        r.v[0] = x.x; r.v[1] = x.y; r.v[2] = x.z; r.v[3] = x.w;
+    } else {
+        r.v[0] = s.at(row, col);
+    }
+    return r;
+}
+template <int VEC>
+__device__ __forceinline__ void put_pack(const RowImage& im, int64_t row, int col, const Pack<VEC>& r) {
+    if constexpr (VEC == 4) im.put4(row, col, make_float4(r.v[0], r.v[1], r.v[2], r.v[3]));
+    else im.put(row, col, r.v[0]);
+}
+
+__device__ __forceinline__ void zero_tail(const RowImage& im, int64_t row, int width) {
+    for (int c = width + threadIdx.x; c < im.ld; c += blockDim.x) im.put(row, c, 0.f);
+}
+
+// The updated row into `dst` (shared memory): x + coef * branches.  Normed branches are staged in `dst` / `other` first.
+template <int VEC>
+__device__ __forceinline__ void updated_row(const RowUpdateArgs& a, int64_t row, float* dst, float* other, float* red) {
+    const float* x = a.x + row * a.width;
+    const int step = RU_THREADS * VEC;
+    float inv[2] = {1.f, 1.f};
+    const bool normed = a.n_add > 0 && a.add_w[0] != nullptr;
+    if (normed) {
+        for (int b = 0; b < a.n_add; ++b) {
+            float* st = b == 0 ? dst : other;
+            float ss = 0.f;
+            for (int c = threadIdx.x * VEC; c < a.width; c += step) {
+                const Pack<VEC> y = share_pack<VEC>(a.add[b], row, c);
+                store_pack<VEC>(st + c, y);
+#pragma unroll
+                for (int i = 0; i < VEC; ++i) ss = fmaf(y.v[i], y.v[i], ss);
+            }
+            ss = block_sum(ss, red);
+            inv[b] = sqrtf(ss / (float)a.width + a.add_eps);
+        }
+    }
+    // a thread reads and writes the same columns of the staging rows throughout, so no barrier is needed in between
+    for (int c = threadIdx.x * VEC; c < a.width; c += step) {
+        Pack<VEC> v = load_pack<VEC>(x + c);
+        if (normed) {
+            Pack<VEC> sum;
+            const Pack<VEC> y0 = load_pack<VEC>(dst + c), w0 = load_pack<VEC>(a.add_w[0] + c);
+#pragma unroll
+            for (int i = 0; i < VEC; ++i) sum.v[i] = y0.v[i] / inv[0] * w0.v[i];
+            if (a.n_add > 1) {
+                const Pack<VEC> y1 = load_pack<VEC>(other + c), w1 = load_pack<VEC>(a.add_w[1] + c);
+#pragma unroll
+                for (int i = 0; i < VEC; ++i) sum.v[i] += y1.v[i] / inv[1] * w1.v[i];
+            }
+#pragma unroll
+            for (int i = 0; i < VEC; ++i) v.v[i] = fmaf(a.add_coef, sum.v[i], v.v[i]);
+        } else if (a.n_add > 0) {
+            const Pack<VEC> y = share_pack<VEC>(a.add[0], row, c);
+#pragma unroll
+            for (int i = 0; i < VEC; ++i) v.v[i] = fmaf(a.add_coef, y.v[i], v.v[i]);
+        }
+        store_pack<VEC>(dst + c, v);
+    }
+}
+
+template <int VEC>
+__device__ __forceinline__ Pack<VEC> norm_pack(const RowUpdateArgs& a, const Pack<VEC>& x, int c) {
+    Pack<VEC> h;
+    const Pack<VEC> w = load_pack<VEC>(a.norm_w + c), b = load_pack<VEC>(a.norm_b + c);
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) h.v[i] = fmaf(tanhf(a.alpha * x.v[i]), w.v[i], b.v[i]);
+    return h;
+}
+
+// Shared memory: the row, its neighbour (n_mix > 0), and a staging row for a second normed branch.
+template <int VEC>
+__global__ void __launch_bounds__(RU_THREADS) row_update_kernel(RowUpdateArgs a) {
+    extern __shared__ __align__(16) float ru_smem[];
+    __shared__ float red[32];
+    float* cur = ru_smem;
+    float* prv = cur + (a.n_mix > 0 ? a.width : 0);
+    float* other = prv + a.width;
+    pdl_trigger();
+    pdl_wait();
+    const int64_t r = blockIdx.x;
+    const int64_t row = a.row_index ? a.row_index[r] : r;
+    const int step = RU_THREADS * VEC;
+    updated_row<VEC>(a, row, cur, other, red);
+    if (a.x_out != nullptr)
+        for (int c = threadIdx.x * VEC; c < a.width; c += step) store_pack<VEC>(a.x_out + row * a.width + c, load_pack<VEC>(cur + c));
+    if (a.raw.any()) {
+        for (int c = threadIdx.x * VEC; c < a.width; c += step) put_pack<VEC>(a.raw, r, c, load_pack<VEC>(cur + c));
+        zero_tail(a.raw, r, a.width);
+    }
+    if (a.norm == NormKind::None) return;
+    if (a.n_mix == 0) {
+        for (int c = threadIdx.x * VEC; c < a.width; c += step) put_pack<VEC>(a.normed, r, c, norm_pack<VEC>(a, load_pack<VEC>(cur + c), c));
+        zero_tail(a.normed, r, a.width);
+        return;
+    }
+    const int lane = a.token_lane[row];
+    const int2 half = a.lanes.halves[lane];
+    const int first = a.lanes.cu[lane], last = a.lanes.cu[lane + 1] - 1;
+    const bool inside = row > first;
+    if (inside) updated_row<VEC>(a, row - 1, prv, other, red);
+    for (int c = threadIdx.x * VEC; c < a.width; c += step) {
+        const Pack<VEC> h = norm_pack<VEC>(a, load_pack<VEC>(cur + c), c);
+        Pack<VEC> p;
+        if (inside) p = norm_pack<VEC>(a, load_pack<VEC>(prv + c), c);
+        else if (half.x >= 0) p = load_pack<VEC>(a.kept + (int64_t)half.x * a.width + c);
+        else
+#pragma unroll
+            for (int i = 0; i < VEC; ++i) p.v[i] = 0.f;
+        for (int m = 0; m < a.n_mix; ++m) {
+            const Pack<VEC> mu = load_pack<VEC>(a.mu + (int64_t)m * a.width + c);
+            Pack<VEC> o;
+#pragma unroll
+            for (int i = 0; i < VEC; ++i) o.v[i] = fmaf(p.v[i] - h.v[i], mu.v[i], h.v[i]);
+            put_pack<VEC>(a.mixes, (int64_t)m * a.rows + r, c, o);
+        }
+        if (row == last) store_pack<VEC>(a.kept + (int64_t)half.y * a.width + c, h);
+    }
+    for (int m = 0; m < a.n_mix; ++m) zero_tail(a.mixes, (int64_t)m * a.rows + r, a.width);
+}
+
+// ------------------------------------------------------------------------------------------------ WKV decay
+
+constexpr int WD_ROWS = 8, WD_THREADS = 128;
+
+__global__ void __launch_bounds__(WD_THREADS) wkv_decay_kernel(Shares low, int low_col, int rows, int rank, int channels,
+                                                               const float* __restrict__ w2t, const float* __restrict__ w0, float* decay) {
+    extern __shared__ float wd_z[];  // [rank][WD_ROWS]
+    pdl_trigger();
+    pdl_wait();
+    const int r0 = blockIdx.y * WD_ROWS;
+    for (int i = threadIdx.x; i < rank * WD_ROWS; i += WD_THREADS) {
+        const int r = i / rank, j = i - r * rank;
+        wd_z[j * WD_ROWS + r] = r0 + r < rows ? tanhf(low.at(r0 + r, low_col + j)) : 0.f;
+    }
+    __syncthreads();
+    const int c = blockIdx.x * WD_THREADS + threadIdx.x;
+    if (c >= channels) return;
+    float acc[WD_ROWS];
+#pragma unroll
+    for (int r = 0; r < WD_ROWS; ++r) acc[r] = 0.f;
+#pragma unroll 4
+    for (int j = 0; j < rank; ++j) {
+        const float w = w2t[(int64_t)j * channels + c];
+#pragma unroll
+        for (int r = 0; r < WD_ROWS; ++r) acc[r] = fmaf(wd_z[j * WD_ROWS + r], w, acc[r]);
+    }
+    const float b = w0[c];
+#pragma unroll
+    for (int r = 0; r < WD_ROWS; ++r)
+        if (r0 + r < rows) decay[(int64_t)(r0 + r) * channels + c] = expf(-expf(acc[r] + b));
+}
+
+// ------------------------------------------------------------------------------------------------ delta-rule inputs
+
+constexpr int DP_WARPS = 8;
+constexpr int DP_MAX_DIM = 256;
+
+// The raw projection of channel ch (of q | k | v) at row i of the lane (negative: before this tick).
+__device__ __forceinline__ float raw_value(const DeltaPrepArgs& a, int first, int i, int half_in, int ch, int y_col, int channels) {
+    if (i >= 0) return a.y.at(first + i, y_col);
+    if (half_in < 0) return 0.f;
+    return a.tail[((int64_t)half_in * (a.taps - 1) + (a.taps - 1 + i)) * channels + ch];
+}
+
+// One CTA per row; a warp takes one head of q, k or v at a time.
+__global__ void __launch_bounds__(DP_WARPS * 32) delta_prep_kernel(DeltaPrepArgs a) {
+    pdl_trigger();
+    pdl_wait();
+    const int64_t row = blockIdx.x;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int seq = a.token_lane[row];
+    const int first = a.lanes.cu[seq], last = a.lanes.cu[seq + 1] - 1, i = (int)row - first;
+    const int2 half = a.lanes.halves[seq];
+    const int kw = a.kv_heads * a.dim, vw = a.heads * a.vdim, channels = 2 * kw + vw;
+    const int units = 2 * a.kv_heads + a.heads;
+    for (int u = warp; u < units; u += DP_WARPS) {
+        const int kind = u < a.kv_heads ? 0 : (u < 2 * a.kv_heads ? 1 : 2);
+        const int head = kind == 0 ? u : (kind == 1 ? u - a.kv_heads : u - 2 * a.kv_heads);
+        const int dim = kind == 2 ? a.vdim : a.dim;
+        const int ch0 = (kind == 0 ? 0 : (kind == 1 ? kw : 2 * kw)) + head * dim;
+        const int y0 = (kind == 0 ? a.q_col : (kind == 1 ? a.k_col : a.v_col)) + head * dim;
+        float* out = kind == 0 ? a.q + row * kw : (kind == 1 ? a.k + row * kw : a.v + row * vw);
+        float val[DP_MAX_DIM / 32];
+        float ss = 0.f;
+#pragma unroll
+        for (int e = 0; e < DP_MAX_DIM / 32; ++e) {
+            const int c = e * 32 + lane;
+            val[e] = 0.f;
+            if (c < dim) {
+                float sum = 0.f;
+                for (int j = 0; j < a.taps; ++j)
+                    sum = fmaf(a.conv[(int64_t)j * channels + ch0 + c],
+                               raw_value(a, first, i - (a.taps - 1) + j, half.x, ch0 + c, y0 + c, channels), sum);
+                val[e] = silu_f(sum);
+                ss = fmaf(val[e], val[e], ss);
+            }
+        }
+        float f = 1.f;
+        if (kind != 2) {
+            ss = warp_sum(ss);
+            f = 1.0f / sqrtf(ss + 1e-6f);
+            if (kind == 0) f *= rsqrtf((float)a.dim);
+        }
+#pragma unroll
+        for (int e = 0; e < DP_MAX_DIM / 32; ++e) {
+            const int c = e * 32 + lane;
+            if (c < dim) out[head * dim + c] = val[e] * f;
+        }
+    }
+    for (int h = threadIdx.x; h < a.heads; h += DP_WARPS * 32) {
+        a.beta[row * a.heads + h] = sigmoid_f(a.y.at(row, a.b_col + h));
+        a.decay[row * a.heads + h] = recurrent::gated_delta_decay(a.y.at(row, a.a_col + h), a.dt_bias[h], a.log_decay[h]);
+    }
+    if (row == last)
+        for (int t = 0; t < a.taps - 1; ++t)
+            for (int ch = threadIdx.x; ch < channels; ch += DP_WARPS * 32) {
+                const int y_col = ch < kw ? a.q_col + ch : (ch < 2 * kw ? a.k_col + ch - kw : a.v_col + ch - 2 * kw);
+                a.tail[((int64_t)half.y * (a.taps - 1) + t) * channels + ch] = raw_value(a, first, i - (a.taps - 2) + t, half.x, ch, y_col, channels);
+            }
+}
+
+// ------------------------------------------------------------------------------------------------ gates
+
+__global__ void __launch_bounds__(256) head_gate_kernel(const float* attn, int heads, int row_width, int vdim, Shares gate, int gate_col, RowImage out) {
+    extern __shared__ float hg_gate[];
+    pdl_trigger();
+    pdl_wait();
+    const int64_t row = blockIdx.x;
+    for (int h = threadIdx.x; h < heads; h += blockDim.x) hg_gate[h] = sigmoid_f(gate.at(row, gate_col + h));
+    __syncthreads();
+    const float* src = attn + row * heads * row_width;
+    for (int c = threadIdx.x; c < out.ld; c += blockDim.x) {
+        const int h = c / vdim;
+        out.put(row, c, h < heads ? src[h * row_width + (c - h * vdim)] * hg_gate[h] : 0.f);
+    }
+}
+
+__global__ void __launch_bounds__(128) side_gate_kernel(Shares z, int dim, const uint32_t* ids, const void* table, int table_f32, int64_t table_ld,
+                                                        int slice, RowImage out) {
+    pdl_trigger();
+    pdl_wait();
+    const int64_t row = blockIdx.x;
+    const int64_t at = (int64_t)ids[row] * table_ld + slice;
+    for (int c = threadIdx.x; c < out.ld; c += blockDim.x) {
+        float v = 0.f;
+        if (c < dim) {
+            const float e = table_f32 ? static_cast<const float*>(table)[at + c] : __bfloat162float(static_cast<const __nv_bfloat16*>(table)[at + c]);
+            v = gelu_tanh_f(z.at(row, c)) * e;
+        }
+        out.put(row, c, v);
+    }
+}
+
+__global__ void __launch_bounds__(256) gated_act_kernel(Shares gu, int ff, RowImage out) {
+    pdl_trigger();
+    pdl_wait();
+    const int64_t row = blockIdx.x;
+    for (int c = threadIdx.x; c < out.ld; c += blockDim.x) out.put(row, c, c < ff ? silu_f(gu.at(row, 2 * c)) * gu.at(row, 2 * c + 1) : 0.f);
+}
+
+// ------------------------------------------------------------------------------------------------ f32 matmul
+
+constexpr int FM_TILE = 64, FM_K = 16;
+
+// 64 x 64 outputs per CTA, 4 x 4 per thread.
+__global__ void __launch_bounds__(256) f32_matmul_kernel(const float* __restrict__ w, int64_t rows, int cols, const float* __restrict__ x, int T, float* y,
+                                                         int ldy, int n_groups, int4 end_lo, int4 end_hi) {
+    __shared__ float ws[FM_K][FM_TILE + 4], xs[FM_K][FM_TILE + 4];
+    pdl_trigger();
+    pdl_wait();
+    const int64_t n0 = (int64_t)blockIdx.x * FM_TILE;
+    const int t0 = blockIdx.y * FM_TILE;
+    const int ends[kMaxRowGroups] = {end_lo.x, end_lo.y, end_lo.z, end_lo.w, end_hi.x, end_hi.y, end_hi.z, end_hi.w};
+    int g = 0;
+    while (g < n_groups - 1 && n0 / 128 >= ends[g]) ++g;
+    const float* xg = x + (int64_t)g * T * cols;
+    const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
+    float acc[4][4] = {};
+    for (int k0 = 0; k0 < cols; k0 += FM_K) {
+        for (int i = threadIdx.x; i < FM_TILE * FM_K; i += 256) {
+            const int r = i / FM_K, k = i % FM_K;
+            ws[k][r] = n0 + r < rows && k0 + k < cols ? w[(n0 + r) * cols + k0 + k] : 0.f;
+            xs[k][r] = t0 + r < T && k0 + k < cols ? xg[(int64_t)(t0 + r) * cols + k0 + k] : 0.f;
+        }
+        __syncthreads();
+#pragma unroll
+        for (int k = 0; k < FM_K; ++k) {
+            float a[4], b[4];
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+                a[i] = xs[k][ty * 4 + i];
+                b[i] = ws[k][tx * 4 + i];
+            }
+#pragma unroll
+            for (int i = 0; i < 4; ++i)
+#pragma unroll
+                for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(a[i], b[j], acc[i][j]);
+        }
+        __syncthreads();
+    }
+#pragma unroll
+    for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+            const int t = t0 + ty * 4 + i;
+            const int64_t n = n0 + tx * 4 + j;
+            if (t < T && n < rows) y[(int64_t)t * ldy + n] = acc[i][j];
+        }
+}
+
+}  // namespace
+
+void launch_row_update(const RowUpdateArgs& a, cudaStream_t s) {
+    if (a.rows <= 0) return;
+    if (a.n_mix > 0 && (a.x == a.x_out || a.row_index != nullptr)) throw std::runtime_error("launch_row_update: a token shift needs its own output buffer and packed rows");
+    if (a.n_add == 2 && (a.add_w[0] == nullptr || a.add_w[1] == nullptr)) throw std::runtime_error("launch_row_update: two branches are both normed");
+    bool vec = a.width % 4 == 0;
+    for (int b = 0; b < a.n_add; ++b)
+        vec = vec && a.add[b].ld % 4 == 0 && a.add[b].stride % 4 == 0 && (reinterpret_cast<uintptr_t>(a.add[b].p) & 15) == 0;
+    const size_t smem = (size_t)a.width * 4 * (1 + (a.n_mix > 0 ? 1 : 0) + (a.n_add == 2 ? 1 : 0));
+    if (smem > (size_t)200 * 1024) throw std::runtime_error("launch_row_update: the model is too wide");
+    if (vec) {
+        ensure_dynamic_smem(reinterpret_cast<const void*>(&row_update_kernel<4>), smem);
+        launch_pdl(row_update_kernel<4>, dim3((unsigned)a.rows), dim3(RU_THREADS), smem, s, a);
+    } else {
+        ensure_dynamic_smem(reinterpret_cast<const void*>(&row_update_kernel<1>), smem);
+        launch_pdl(row_update_kernel<1>, dim3((unsigned)a.rows), dim3(RU_THREADS), smem, s, a);
+    }
+    MK_LAUNCH_CHECK();
+}
+
+void launch_wkv_decay(const Shares& low, int low_col, int rows, int rank, int channels, const float* w2t, const float* w0, float* decay, cudaStream_t s) {
+    if (rows <= 0) return;
+    const size_t smem = (size_t)rank * WD_ROWS * 4;
+    if (smem > (size_t)200 * 1024) throw std::runtime_error("launch_wkv_decay: the low rank is too large");
+    ensure_dynamic_smem(reinterpret_cast<const void*>(&wkv_decay_kernel), smem);
+    const dim3 grid((unsigned)((channels + WD_THREADS - 1) / WD_THREADS), (unsigned)((rows + WD_ROWS - 1) / WD_ROWS));
+    launch_pdl(wkv_decay_kernel, grid, dim3(WD_THREADS), smem, s, low, low_col, rows, rank, channels, w2t, w0, decay);
+    MK_LAUNCH_CHECK();
+}
+
+void launch_delta_prep(const DeltaPrepArgs& a, cudaStream_t s) {
+    if (a.rows <= 0) return;
+    if (a.dim > DP_MAX_DIM || a.vdim > DP_MAX_DIM) throw std::runtime_error("launch_delta_prep: head dimensions above 256 are not supported");
+    launch_pdl(delta_prep_kernel, dim3((unsigned)a.rows), dim3(DP_WARPS * 32), 0, s, a);
+    MK_LAUNCH_CHECK();
+}
+
+void launch_head_gate(const float* attn, int rows, int heads, int row_width, int vdim, const Shares& gate, int gate_col, const RowImage& out,
+                      cudaStream_t s) {
+    if (rows <= 0) return;
+    launch_pdl(head_gate_kernel, dim3((unsigned)rows), dim3(256), (size_t)heads * 4, s, attn, heads, row_width, vdim, gate, gate_col, out);
+    MK_LAUNCH_CHECK();
+}
+
+void launch_side_gate(const Shares& z, int rows, int dim, const uint32_t* ids, const void* table, int table_f32, int64_t table_ld, int slice,
+                      const RowImage& out, cudaStream_t s) {
+    if (rows <= 0) return;
+    launch_pdl(side_gate_kernel, dim3((unsigned)rows), dim3(128), 0, s, z, dim, ids, table, table_f32, table_ld, slice, out);
+    MK_LAUNCH_CHECK();
+}
+
+void launch_gated_act(const Shares& gu, int rows, int ff, const RowImage& out, cudaStream_t s) {
+    if (rows <= 0) return;
+    launch_pdl(gated_act_kernel, dim3((unsigned)rows), dim3(256), 0, s, gu, ff, out);
+    MK_LAUNCH_CHECK();
+}
+
+void launch_f32_matmul(const float* w, int64_t rows, int cols, const float* x, int T, float* y, int ldy, int n_groups, const int* group_end,
+                       cudaStream_t s) {
+    if (T <= 0) return;
+    int e[kMaxRowGroups] = {};
+    for (int g = 0; g < n_groups && n_groups > 1; ++g) e[g] = group_end[g];
+    const dim3 grid((unsigned)((rows + FM_TILE - 1) / FM_TILE), (unsigned)((T + FM_TILE - 1) / FM_TILE));
+    launch_pdl(f32_matmul_kernel, grid, dim3(256), 0, s, w, rows, cols, x, T, y, ldy, n_groups, make_int4(e[0], e[1], e[2], e[3]),
+               make_int4(e[4], e[5], e[6], e[7]));
+    MK_LAUNCH_CHECK();
+}
+
+}  // namespace mk

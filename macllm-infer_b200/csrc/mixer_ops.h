@@ -1,0 +1,78 @@
+// The steps between the matmuls of mixer-built decoders: residual update with norm and token shift, the decay of WKV time
+// mixing, the short convolution and unit norms of the gated delta rule, output gates, the per-layer token input - and the
+// 32-bit matmul for models computed in f32 throughout.
+#pragma once
+#include "mixer_spec.h"
+#include "row_types.cuh"
+
+namespace mk {
+
+// One CTA per row r (x row = row_index ? row_index[r] : r):
+//   x_out = x + coef * sum over branches b of (add_w[b] ? rms(add[b]) * add_w[b] : add[b])      (n_add branches)
+//   raw    <- x_out                        (optional image)
+//   h       = norm(x_out);  normed <- h    (optional image, n_mix = 0)
+//   mixes[i] <- h + (h' - h) * mu[i]       (n_mix images of `rows` rows each, one after the other), h' = h of the sequence's
+//                                          previous token: recomputed from the row before, or the kept one (zeros at the start)
+// The last row of every lane leaves its h as the kept one.  x and x_out are different buffers when n_mix > 0, because a row
+// reads its neighbour's old value.
+struct RowUpdateArgs {
+    const float* x = nullptr;
+    float* x_out = nullptr;  // may be null (nothing kept)
+    int rows = 0, width = 0;
+    const int32_t* row_index = nullptr;
+    int n_add = 0;
+    Shares add[2];
+    const float* add_w[2] = {nullptr, nullptr};
+    float add_coef = 1.f, add_eps = 0.f;
+    RowImage raw;
+    NormKind norm = NormKind::None;
+    float alpha = 1.f;
+    const float* norm_w = nullptr;
+    const float* norm_b = nullptr;
+    RowImage normed;
+    int n_mix = 0;
+    const float* mu = nullptr;  // [n_mix][width]
+    RowImage mixes;
+    StateLanes lanes;
+    const int32_t* token_lane = nullptr;
+    float* kept = nullptr;      // [slot halves][width]
+};
+void launch_row_update(const RowUpdateArgs& a, cudaStream_t s);
+
+// decay[t][c] = exp(-exp(sum_j tanh(low[t][j]) w2[c][j] + w0[c])), everything in f32.  w2t is w2 transposed, [rank][channels].
+void launch_wkv_decay(const Shares& low, int low_col, int rows, int rank, int channels, const float* w2t, const float* w0, float* decay, cudaStream_t s);
+
+// The gated delta rule's inputs from the raw projections y: a causal convolution of `taps` taps per channel over q | k | v and
+// silu, unit norm per head of q and k (q also times dim^-1/2), beta = sigmoid(b), decay = exp(softplus(a + dt_bias) * log_decay).
+// The kept tail is the last taps - 1 raw rows of a sequence, [slot halves][taps - 1][channels] over q | k | v.
+struct DeltaPrepArgs {
+    Shares y;
+    int q_col = 0, k_col = 0, v_col = 0, a_col = 0, b_col = 0;
+    int rows = 0, heads = 0, kv_heads = 0, dim = 0, vdim = 0, taps = 1;
+    const float* conv = nullptr;       // [taps][channels] over q | k | v
+    const float* dt_bias = nullptr;    // [heads]
+    const float* log_decay = nullptr;  // [heads], negative
+    StateLanes lanes;
+    const int32_t* token_lane = nullptr;
+    float* tail = nullptr;
+    float *q = nullptr, *k = nullptr, *v = nullptr, *beta = nullptr, *decay = nullptr;
+};
+void launch_delta_prep(const DeltaPrepArgs& a, cudaStream_t s);
+
+// out[t][h * vdim + i] = attn[t][h * row_width + i] * sigmoid(gate[t][gate_col + h])
+void launch_head_gate(const float* attn, int rows, int heads, int row_width, int vdim, const Shares& gate, int gate_col, const RowImage& out,
+                      cudaStream_t s);
+
+// out[t][j] = gelu_tanh(z[t][j]) * table[ids[t]][slice + j], j < dim; table [vocab][table_ld] as bfloat16 bits (or f32)
+void launch_side_gate(const Shares& z, int rows, int dim, const uint32_t* ids, const void* table, int table_f32, int64_t table_ld, int slice,
+                      const RowImage& out, cudaStream_t s);
+
+// out[t][j] = silu(gu[t][2j]) * gu[t][2j + 1], j < ff: gate and up rows interleaved
+void launch_gated_act(const Shares& gu, int rows, int ff, const RowImage& out, cudaStream_t s);
+
+// y[t][n] = sum_k x[t][k] w[n][k] in f32, k ascending.  x is [n_groups][T][cols]; weight row n reads input g of its group, whose
+// rows end at 128 * group_end[g] (see HalfWeight).
+void launch_f32_matmul(const float* w, int64_t rows, int cols, const float* x, int T, float* y, int ldy, int n_groups, const int* group_end,
+                       cudaStream_t s);
+
+}  // namespace mk

@@ -10,10 +10,13 @@ namespace mk {
 
 constexpr int RK_MAX_D = 256;
 
-// One warp.  kind: 0 = q, 1 = k, 2 = v; hh = head index within its kind; t = packed token row; x = the warp's d floats
-// of shared memory, holding the finished head on return (after a __syncwarp).
+// Width of a head's row in q_out and in the pools.
+__host__ __device__ __forceinline__ int rope_row_width(const RopeKvArgs& a) { return a.d_row > 0 ? a.d_row : a.d; }
+
+// One warp.  kind: 0 = q, 1 = k, 2 = v; hh = head index within its kind; t = packed token row; x = the warp's row
+// of shared memory, holding the finished head (zero-filled to the row width) on return (after a __syncwarp).
 __device__ __forceinline__ void rope_head_prepare(const RopeKvArgs& a, int kind, int hh, int t, int position, float* x, int lane) {
-    const int d = a.d;
+    const int d = kind == 2 && a.dv > 0 ? a.dv : a.d;
     const float* src = kind == 0 ? a.q + (int64_t)t * a.ldq + hh * d : (kind == 1 ? a.k + (int64_t)t * a.ldk + hh * d : a.v + (int64_t)t * a.ldv + hh * d);
     const int n_parts = kind == 2 ? a.v_splits : a.qk_splits;
     const int64_t part_stride = kind == 2 ? a.v_split_stride : a.qk_split_stride;
@@ -34,6 +37,7 @@ __device__ __forceinline__ void rope_head_prepare(const RopeKvArgs& a, int kind,
             x[i] = v;
         }
     }
+    for (int i = d + lane; i < rope_row_width(a); i += 32) x[i] = 0.f;
     __syncwarp();
 
     const float* nw = kind == 0 ? a.q_norm_w : (kind == 1 ? a.k_norm_w : nullptr);
@@ -51,14 +55,15 @@ __device__ __forceinline__ void rope_head_prepare(const RopeKvArgs& a, int kind,
         const float* s = a.sin_t + (int64_t)position * half;
         float r1[RK_MAX_D / 64], r2[RK_MAX_D / 64];
         int cnt = 0;
+        const int step = a.interleaved ? 2 : 1, off = a.interleaved ? 1 : half;
         for (int i = lane; i < half; i += 32, ++cnt) {
-            float x1 = x[i], x2 = x[i + half];
+            float x1 = x[i * step], x2 = x[i * step + off];
             r1[cnt] = __fsub_rn(__fmul_rn(x1, c[i]), __fmul_rn(x2, s[i]));
             r2[cnt] = __fadd_rn(__fmul_rn(x1, s[i]), __fmul_rn(x2, c[i]));
         }
         __syncwarp();
         cnt = 0;
-        for (int i = lane; i < half; i += 32, ++cnt) { x[i] = r1[cnt]; x[i + half] = r2[cnt]; }
+        for (int i = lane; i < half; i += 32, ++cnt) { x[i * step] = r1[cnt]; x[i * step + off] = r2[cnt]; }
         __syncwarp();
     }
 }

@@ -8,6 +8,7 @@
 // One warp per (token, head); the head vector is staged in shared memory so any head_dim works.
 #include "kernels.h"
 #include "rope_head.cuh"
+#include <algorithm>
 
 namespace mk {
 
@@ -32,7 +33,7 @@ __global__ void __launch_bounds__(RK_WARPS * 32) rope_kv_kernel(RopeKvArgs a) {
     int head = blockIdx.y * RK_WARPS + warp;
     int t = blockIdx.x;
     if (head >= heads_total) return;
-    const int d = a.d;
+    const int d = rope_row_width(a);
     float* x = buf[warp];
 
     int kind, hh;  // 0 = q, 1 = k, 2 = v
@@ -69,7 +70,9 @@ __global__ void cow_copy_kernel(KV* k_pool, KV* v_pool, int64_t src_block, int64
 
 void launch_rope_kv(const RopeKvArgs& a, cudaStream_t s) {
     if (a.T <= 0) return;
-    if (a.d > RK_MAX_D) throw std::runtime_error("launch_rope_kv: head_dim above 256 is not supported");
+    if (std::max({a.d, a.dv, a.d_row}) > RK_MAX_D) throw std::runtime_error("launch_rope_kv: head_dim above 256 is not supported");
+    if (a.d_row > 0 && (a.d_row < a.d || a.d_row < a.dv || a.q_out == nullptr))
+        throw std::runtime_error("launch_rope_kv: padded heads need a separate query output at least as wide as the heads");
     int heads_total = a.q_heads + 2 * a.kv_heads;
     dim3 grid((unsigned)a.T, (unsigned)((heads_total + RK_WARPS - 1) / RK_WARPS));
     if (a.kv_f16)

@@ -1,0 +1,70 @@
+// How rows travel between the matmuls and the kernels around them.
+#pragma once
+#include "common.cuh"
+#include <cuda_bf16.h>
+
+namespace mk {
+
+// A matmul's f32 output [rows][ld], possibly still cut into n partial sums (split-K) `stride` floats apart, which the consumer
+// adds in index order.
+struct Shares {
+    const float* p = nullptr;
+    int n = 1;
+    int64_t stride = 0;
+    int ld = 0;
+#ifdef __CUDACC__
+    __device__ __forceinline__ float at(int64_t row, int col) const {
+        const float* q = p + row * ld + col;
+        float v = *q;
+        for (int s = 1; s < n; ++s) v += q[s * stride];
+        return v;
+    }
+    __device__ __forceinline__ float4 at4(int64_t row, int col) const {  // col, ld and stride multiples of 4
+        const float* q = p + row * ld + col;
+        float4 v = *reinterpret_cast<const float4*>(q);
+        for (int s = 1; s < n; ++s) {
+            const float4 w = *reinterpret_cast<const float4*>(q + s * stride);
+            v.x += w.x; v.y += w.y; v.z += w.z; v.w += w.w;
+        }
+        return v;
+    }
+#endif
+};
+
+// A matmul's input rows [rows][ld]: bfloat16 (h) or f32 (f), whichever is set.  Columns from the matrix's true width up to ld are
+// zeros, written by the kernel that makes the rows.
+struct RowImage {
+    __nv_bfloat16* h = nullptr;
+    float* f = nullptr;
+    int ld = 0;
+#ifdef __CUDACC__
+    __device__ __forceinline__ bool any() const { return h != nullptr || f != nullptr; }
+    __device__ __forceinline__ void put(int64_t row, int col, float v) const {
+        if (h != nullptr) h[row * ld + col] = __float2bfloat16_rn(v);
+        else f[row * ld + col] = v;
+    }
+    __device__ __forceinline__ void put4(int64_t row, int col, float4 v) const {  // col and ld multiples of 4
+        if (h != nullptr) {
+            __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
+            *reinterpret_cast<uint2*>(h + row * ld + col) = make_uint2(*reinterpret_cast<uint32_t*>(&a), *reinterpret_cast<uint32_t*>(&b));
+        } else {
+            *reinterpret_cast<float4*>(f + row * ld + col) = v;
+        }
+    }
+#endif
+};
+
+// The recurrent state of a tick's lanes: per lane the slot half to read (-1: zeros) and the slot half to write.
+struct StateLanes {
+    const int32_t* cu = nullptr;   // [lanes + 1] packed row ranges
+    const int2* halves = nullptr;  // [lanes] (read, write)
+    int lanes = 0;
+};
+
+#ifdef __CUDACC__
+__device__ __forceinline__ float sigmoid_f(float z) { return 1.0f / (1.0f + expf(-z)); }
+__device__ __forceinline__ float silu_f(float z) { return z / (1.0f + expf(-z)); }
+__device__ __forceinline__ float gelu_tanh_f(float z) { return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z))); }
+#endif
+
+}  // namespace mk

@@ -85,7 +85,8 @@ class Model:
 
     @staticmethod
     def _config(device=0, block_tokens=16, slab_blocks=8, kv_capacity_tokens=4096, prefix_capacity_tokens=0, kv_dtype="f16",
-                max_batch_tokens=2048, max_batch_lanes=64, matmul_path=capi.PATH_AUTO, ep_rank=0, ep_size=1, ep_mode=0) -> capi.LoadConfig:
+                max_batch_tokens=2048, max_batch_lanes=64, matmul_path=capi.PATH_AUTO, ep_rank=0, ep_size=1, ep_mode=0, state_slots=0,
+                compute="default") -> capi.LoadConfig:
         cfg = capi.LoadConfig()
         cfg.device_ordinal = device
         cfg.block_tokens = block_tokens
@@ -99,6 +100,8 @@ class Model:
         cfg.ep_rank = ep_rank
         cfg.ep_size = ep_size
         cfg.ep_mode = ep_mode
+        cfg.state_slots = state_slots
+        cfg.compute_dtype = {"default": capi.COMPUTE_DEFAULT, "bfloat16": capi.COMPUTE_BF16, "float32": capi.COMPUTE_F32}[compute]
         return cfg
 
     EP_ID_BYTES = 128
@@ -132,11 +135,17 @@ class Model:
         return out
 
     @classmethod
-    def load_gguf(cls, path, **kw) -> "Model":
+    def load(cls, path, **kw) -> "Model":
+        """A checkpoint of any registered format: a GGUF file, or a folder with config.json (whose `architecture` picks the
+        model) and model.safetensors.  `compute` ("bfloat16" | "float32") applies to safetensors checkpoints."""
         cfg = cls._config(**kw)
         h = C.c_void_p()
-        capi.check(capi.lib().mk_model_load_gguf(str(path).encode(), C.byref(cfg), C.byref(h)))
+        capi.check(capi.lib().mk_model_load(str(path).encode(), C.byref(cfg), C.byref(h)))
         return cls(h)
+
+    @classmethod
+    def load_gguf(cls, path, **kw) -> "Model":
+        return cls.load(path, **kw)
 
     @classmethod
     def fake(cls, vocab=32, max_context=4096, fail_forward_at=-1, **kw) -> "Model":
@@ -209,21 +218,51 @@ class Model:
             arr[i].start_pos = start_pos
         return arr, keep
 
-    def forward_batch(self, lanes, want_logits=True, want_tokens=True):
+    def forward_batch(self, lanes, want_logits=True, want_tokens=True, rows=None):
         """reserve_batch_kv + forward_batch_tokens_reserved + read_output_to_cpu for one packed ragged
-        batch.  Returns (logits [lanes, vocab] or None, tokens [lanes] or None)."""
+        batch.  Returns (logits [lanes, vocab] or None, tokens [lanes] or None).  `rows`: per lane, the row numbers
+        within its tokens whose logits are returned instead (concatenated); tokens cannot be asked for then."""
         arr, keep = self._lanes(lanes)
         r = C.c_void_p()
         capi.check(capi.lib().mk_reserve_batch(self._h, arr, len(lanes), C.byref(r)))
         flags = (capi.FWD_WANT_LOGITS if want_logits else 0) | (capi.FWD_WANT_TOKENS if want_tokens else 0)
+        n_rows = len(lanes)
+        if rows is not None:
+            counts = np.array([len(x) for x in rows], np.int32)
+            flat = np.array([i for x in rows for i in x] + [0], np.int32)
+            n_rows = int(counts.sum())
+            status = capi.lib().mk_forward_set_logit_rows(self._h, counts.ctypes.data, flat.ctypes.data, len(rows))
+            if status != capi.MK_OK:
+                capi.lib().mk_reservation_drop(r)
+                capi.check(status)
         capi.check(capi.lib().mk_forward_batch_reserved(self._h, arr, len(lanes), r, flags))
         vocab = self.spec().vocab_size
-        logits = np.empty((len(lanes), vocab), np.float32) if want_logits else None
+        logits = np.empty((n_rows, vocab), np.float32) if want_logits else None
         tokens = np.empty(len(lanes), np.uint32) if want_tokens else None
         capi.check(capi.lib().mk_read_output(self._h, None if logits is None else logits.ctypes.data,
                                              None if tokens is None else tokens.ctypes.data))
         del keep
         return logits, tokens
+
+    def capture_residuals(self, on: bool = True) -> None:
+        """Keep the residual stream after every layer of the following forwards (safetensors checkpoints)."""
+        capi.check(capi.lib().mk_model_capture_residuals(self._h, 1 if on else 0))
+
+    def residuals(self, n_tokens: int) -> np.ndarray:
+        """[layers, tokens, hidden] of the last forward, which ran `n_tokens` tokens."""
+        sp = self.spec()
+        out = np.empty((sp.n_layers, n_tokens, sp.hidden_size), np.float32)
+        n = C.c_int32()
+        capi.check(capi.lib().mk_model_read_residuals(self._h, out.ctypes.data, out.size, C.byref(n)))
+        if n.value != n_tokens:
+            raise ValueError(f"the last forward ran {n.value} tokens, not {n_tokens}")
+        return out
+
+    def state_slots(self) -> tuple[int, int]:
+        """(recurrent-state slots, slots held by sessions); (0, 0) for a model without recurrent layers."""
+        a, b = C.c_int32(), C.c_int32()
+        capi.check(capi.lib().mk_state_slots_query(self._h, C.byref(a), C.byref(b)))
+        return a.value, b.value
 
     def last_forward_ms(self) -> float:
         v = C.c_float()
