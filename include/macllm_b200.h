@@ -163,6 +163,19 @@ typedef struct mk_gguf_summary {
 } mk_gguf_summary;
 int32_t mk_gguf_inspect(const char* path, mk_gguf_summary* out);
 
+/* Host-only audit of a safetensors checkpoint (folder with config.json and model.safetensors): the configuration read and
+ * every tensor it implies present with the expected shape.  A checkpoint mk_model_load would refuse is refused here with the
+ * same message. */
+typedef struct mk_mixer_summary {
+    char architecture[32];
+    int32_t vocab_size, hidden_size, n_layers;
+    int32_t wkv_layers, parallel_layers, ffn_layers, side_dim, reserved_;
+    int64_t tensors_in_file, tensors_read, parameters;
+} mk_mixer_summary;
+int32_t mk_mixer_inspect(const char* dir, mk_mixer_summary* out);
+/* Rotary frequencies [dims / 2] (radians per position); `scaling` = {factor, low, high, original} or NULL. */
+int32_t mk_rotary_frequencies(int32_t dims, double base, const double* scaling, double* out);
+
 /* LoadedRuntime::load (src/runtime.rs:104-145): loads a checkpoint with the registered format that recognises it - a GGUF file
  * (first shard of a family), or a folder with config.json and model.safetensors whose config names a registered
  * architecture. */

@@ -46,6 +46,12 @@ class GgufSummary(C.Structure):
                 ("vectors", C.c_int64), ("matrix_bytes", C.c_int64)]
 
 
+class MixerSummary(C.Structure):
+    _fields_ = [("architecture", C.c_char * 32), ("vocab_size", C.c_int32), ("hidden_size", C.c_int32), ("n_layers", C.c_int32),
+                ("wkv_layers", C.c_int32), ("parallel_layers", C.c_int32), ("ffn_layers", C.c_int32), ("side_dim", C.c_int32),
+                ("reserved_", C.c_int32), ("tensors_in_file", C.c_int64), ("tensors_read", C.c_int64), ("parameters", C.c_int64)]
+
+
 class RuntimeSpec(C.Structure):
     _fields_ = [("vocab_size", C.c_int32), ("max_context", C.c_int32), ("n_layers", C.c_int32), ("hidden_size", C.c_int32),
                 ("n_stop_tokens", C.c_int32), ("stop_token_ids", C.c_uint32 * 8), ("weight_bytes", C.c_int64),
@@ -256,6 +262,8 @@ SIGNATURES = {
     "mk_forward_set_logit_rows": (_i32, [P, P, P, _i32]),
     "mk_model_capture_residuals": (_i32, [P, _i32]),
     "mk_model_read_residuals": (_i32, [P, P, _i64, C.POINTER(_i32)]),
+    "mk_mixer_inspect": (_i32, [C.c_char_p, C.POINTER(MixerSummary)]),
+    "mk_rotary_frequencies": (_i32, [_i32, C.c_double, P, P]),
     "mk_state_slots_query": (_i32, [P, C.POINTER(_i32), C.POINTER(_i32)]),
     "mk_k_moe_route": (_i32, [P, _i32, _i32, _i32, P, P]),
 }

@@ -3,6 +3,7 @@
 #include "../../include/macllm_b200.h"
 #include "c_api_util.h"
 #include "engine.h"
+#include "mixer_spec.h"
 #include "model_registry.h"
 #include "prefix_cache.h"
 #include <cstring>
@@ -94,6 +95,45 @@ ModelConfig to_model_config(const mk_load_config* cfg) {
 extern "C" {
 
 // ------------------------------------------------------------------------------------------ model
+
+int32_t mk_mixer_inspect(const char* dir, mk_mixer_summary* out) {
+    return guarded([&] {
+        if (dir == nullptr || out == nullptr) throw std::runtime_error("mk_mixer_inspect: null argument");
+        const SafetensorsFile f(std::string(dir) + "/model.safetensors");
+        const MixerSpec s = read_mixer_spec_of(dir, f);
+        const MixerAudit a = validate_mixer_tensors(s, f);
+        memset(out, 0, sizeof *out);
+        strncpy(out->architecture, s.arch.c_str(), sizeof out->architecture - 1);
+        out->vocab_size = s.vocab;
+        out->hidden_size = s.width;
+        out->n_layers = (int32_t)s.layers.size();
+        for (const MixerLayerSpec& l : s.layers) {
+            (l.kind == MixerKind::Wkv ? out->wkv_layers : out->parallel_layers)++;
+            out->ffn_layers += l.ff > 0 ? 1 : 0;
+        }
+        out->side_dim = s.side_dim;
+        out->tensors_in_file = a.tensors_in_file;
+        out->tensors_read = a.tensors_read;
+        out->parameters = a.parameters;
+    });
+}
+
+int32_t mk_rotary_frequencies(int32_t dims, double base, const double* scaling, double* out) {
+    return guarded([&] {
+        RotarySpec r;
+        r.dims = dims;
+        r.base = base;
+        if (scaling != nullptr) {
+            r.scaled = true;
+            r.factor = scaling[0];
+            r.low = scaling[1];
+            r.high = scaling[2];
+            r.original = scaling[3];
+        }
+        const std::vector<double> f = rotary_frequencies(r);
+        std::copy(f.begin(), f.end(), out);
+    });
+}
 
 int32_t mk_model_load(const char* path, const mk_load_config* cfg, mk_model** out) {
     return guarded([&] {

@@ -16,6 +16,9 @@ Engine::Engine(PagedLm& model, const EngineConfig& cfg) : model_(model), cfg_(cf
     if (cfg.scheduler_token_budget <= 0) throw std::runtime_error("scheduler token budget must be positive");
     if (cfg.prefill_token_quantum <= 0) throw std::runtime_error("prefill token quantum must be positive");
     if (cfg.prefill_token_quantum > cfg.scheduler_token_budget) throw std::runtime_error("prefill token quantum cannot exceed the scheduler token budget");
+    // a sequence keeps its recurrent state from its first forward to its end
+    if (model_.state_slots() != nullptr && cfg.max_active_sequences > model_.state_slots()->capacity())
+        throw std::runtime_error("max_active_sequences exceeds the model's " + std::to_string(model_.state_slots()->capacity()) + " recurrent-state slots");
     // worker_main creates every reusable session up front (engine.rs:1336-1360)
     for (int i = 0; i < cfg.max_active_sequences; ++i) sessions_.push_back(model_.new_session());
 }

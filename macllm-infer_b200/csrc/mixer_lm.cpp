@@ -5,8 +5,6 @@
 #include <algorithm>
 #include <cmath>
 #include <cstring>
-#include <fstream>
-#include <sstream>
 #include <sys/stat.h>
 
 namespace mk {
@@ -27,14 +25,6 @@ const RegisterModelFormat register_mixer_format(ModelFormat{
     "folder with config.json and model.safetensors", is_mixer_checkpoint,
     [](const std::string& path, const ModelConfig& cfg) -> std::unique_ptr<PagedLm> { return std::make_unique<MixerLm>(path, cfg); }});
 
-MixerSpec read_spec(const std::string& dir, const SafetensorsFile& f) {
-    std::ifstream in(dir + "/config.json", std::ios::binary);
-    std::stringstream text;
-    text << in.rdbuf();
-    const std::string s = text.str();
-    return read_mixer_spec(Json::parse(s.data(), s.size(), "config"), f);
-}
-
 constexpr int kShortLane = 4;  // lanes up to this many tokens: the recurrence kernels finish the head rows themselves
 
 }  // namespace
@@ -48,7 +38,8 @@ struct MixerLm::Pending {
 
 MixerLm::MixerLm(const std::string& dir, const ModelConfig& cfg) : DeviceLm(cfg, class_names) {
     const SafetensorsFile f(dir + "/model.safetensors");
-    ms_ = read_spec(dir, f);
+    ms_ = read_mixer_spec_of(dir, f);
+    validate_mixer_tensors(ms_, f);  // before any device memory is touched
     f32_ = cfg.compute_f32;
     esz_ = f32_ ? 4 : 2;
     if (f32_) cfg_.kv_f16 = false;

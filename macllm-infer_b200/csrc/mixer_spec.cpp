@@ -1,7 +1,9 @@
 // See mixer_spec.h.
 #include "mixer_spec.h"
 #include <cmath>
+#include <fstream>
 #include <map>
+#include <sstream>
 #include <stdexcept>
 
 namespace mk {
@@ -111,6 +113,94 @@ MixerSpec read_mixer_spec(const Json& config, const SafetensorsFile& f) {
     auto it = readers().find(arch);
     if (it == readers().end()) throw std::runtime_error("architecture `" + arch + "` is not supported");
     return it->second(config, f);
+}
+
+MixerSpec read_mixer_spec_of(const std::string& dir, const SafetensorsFile& f) {
+    std::ifstream in(dir + "/config.json", std::ios::binary);
+    std::stringstream text;
+    text << in.rdbuf();
+    const std::string s = text.str();
+    return read_mixer_spec(Json::parse(s.data(), s.size(), "config"), f);
+}
+
+std::vector<std::pair<std::string, std::vector<int64_t>>> mixer_tensors(const MixerSpec& s) {
+    std::vector<std::pair<std::string, std::vector<int64_t>>> out;
+    const int64_t C = s.width, V = s.vocab;
+    auto add = [&](const std::string& name, std::vector<int64_t> shape) { out.emplace_back(name, std::move(shape)); };
+    auto norm = [&](const std::string& name) {
+        add(name, {C});
+        if (s.norm == NormKind::DynTanh) {
+            add(name + ".b", {C});
+            add(name + ".alpha", {});
+        }
+    };
+    add("embed", {V, C});
+    if (s.side_dim > 0) add("side.embed", {V, (int64_t)s.layers.size() * s.side_dim});
+    for (size_t i = 0; i < s.layers.size(); ++i) {
+        const MixerLayerSpec& l = s.layers[i];
+        const std::string p = "l" + std::to_string(i) + ".", m = p + "mix.";
+        norm(p + "norm1");
+        if (l.kind == MixerKind::Wkv) {
+            const int64_t H = l.wkv.heads, D = l.wkv.dim, n = H * D, r = l.wkv.rank;
+            for (const char* x : {"r", "k", "v", "g", "w"}) add(m + "mu." + x, {C});
+            for (const char* x : {"r", "k", "v", "g"}) add(m + x, {n, C});
+            add(m + "w1", {r, C});
+            add(m + "w2", {n, r});
+            add(m + "w0", {n});
+            add(m + "u", {H, D});
+            add(m + "norm", {n});
+            add(m + "o", {C, n});
+        } else {
+            const AttentionSpec& a = l.attn;
+            const DeltaSpec& d = l.delta;
+            const int64_t qw = (int64_t)a.heads * a.dim, kw = (int64_t)a.kv_heads * a.dim, vw = (int64_t)a.kv_heads * a.vdim;
+            add(m + "left.q", {qw, C});
+            add(m + "left.k", {kw, C});
+            add(m + "left.v", {vw, C});
+            add(m + "left.g", {a.heads, C});
+            add(m + "left.q.norm", {a.dim});
+            add(m + "left.k.norm", {a.dim});
+            add(m + "left.o", {C, (int64_t)a.heads * a.vdim});
+            add(m + "left.out", {C});
+            const int64_t dk = (int64_t)d.kv_heads * d.dim, dv = (int64_t)d.heads * d.vdim;
+            add(m + "right.q", {dk, C});
+            add(m + "right.k", {dk, C});
+            add(m + "right.v", {dv, C});
+            add(m + "right.q.conv", {dk, d.taps});
+            add(m + "right.k.conv", {dk, d.taps});
+            add(m + "right.v.conv", {dv, d.taps});
+            for (const char* x : {"a", "b"}) add(m + "right." + x, {d.heads, C});
+            for (const char* x : {"A_log", "dt_bias"}) add(m + "right." + x, {d.heads});
+            add(m + "right.g", {dv, C});
+            add(m + "right.norm", {d.vdim});
+            add(m + "right.o", {C, dv});
+            add(m + "right.out", {C});
+        }
+        if (l.ff > 0) {
+            norm(p + "norm2");
+            add(p + "mlp.gate", {l.ff, C});
+            add(p + "mlp.up", {l.ff, C});
+            add(p + "mlp.down", {C, l.ff});
+        }
+        if (s.side_dim > 0) {
+            add(p + "side.gate", {s.side_dim, C});
+            add(p + "side.proj", {C, s.side_dim});
+            add(p + "side.norm", {C});
+        }
+    }
+    norm("final.norm");
+    add("head", {V, C});
+    return out;
+}
+
+MixerAudit validate_mixer_tensors(const MixerSpec& s, const SafetensorsFile& f) {
+    MixerAudit a;
+    a.tensors_in_file = (int64_t)f.tensors().size();
+    for (const auto& t : mixer_tensors(s)) {
+        a.parameters += f.require(t.first, t.second).elements();
+        ++a.tensors_read;
+    }
+    return a;
 }
 
 std::vector<double> rotary_frequencies(const RotarySpec& r) {

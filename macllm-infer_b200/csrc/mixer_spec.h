@@ -66,6 +66,19 @@ struct MixerSpec {
 // Reads `config` (and sizes that only the tensors know) for the architecture it names.
 MixerSpec read_mixer_spec(const Json& config, const SafetensorsFile& f);
 
+// Every tensor the executor reads, with its shape.
+std::vector<std::pair<std::string, std::vector<int64_t>>> mixer_tensors(const MixerSpec& s);
+
+struct MixerAudit {
+    int64_t tensors_in_file = 0, tensors_read = 0, parameters = 0;
+};
+// Every tensor of the spec present, floating-point and of the expected shape; throws on the first that is not.  Host only, run
+// before any device memory is touched.  Tensors the spec does not know are left unread.
+MixerAudit validate_mixer_tensors(const MixerSpec& s, const SafetensorsFile& f);
+
+// Reads <dir>/config.json for the checkpoint in `dir`.
+MixerSpec read_mixer_spec_of(const std::string& dir, const SafetensorsFile& f);
+
 using MixerSpecReader = std::function<MixerSpec(const Json& config, const SafetensorsFile& f)>;
 struct RegisterMixerArchitecture {
     RegisterMixerArchitecture(const std::string& name, MixerSpecReader reader);

@@ -134,6 +134,15 @@ class Model:
         out["architecture"] = s.architecture.decode()
         return out
 
+    @staticmethod
+    def inspect_mixer(path) -> dict:
+        """Host-only audit of a safetensors checkpoint folder; raises MkError with the loader's message.  Needs no GPU."""
+        s = capi.MixerSummary()
+        capi.check(capi.lib().mk_mixer_inspect(str(path).encode(), C.byref(s)))
+        out = {name: getattr(s, name) for name, _ in capi.MixerSummary._fields_ if name != "reserved_"}
+        out["architecture"] = s.architecture.decode()
+        return out
+
     @classmethod
     def load(cls, path, **kw) -> "Model":
         """A checkpoint of any registered format: a GGUF file, or a folder with config.json (whose `architecture` picks the

@@ -1,0 +1,150 @@
+"""Small random checkpoints of mixer-built decoders, and schedules that cut sequences into forwards, for the tests."""
+import importlib
+import json
+
+import numpy as np
+
+from oracle import mixers
+
+SCALING = dict(factor=8.0, low=1.0, high=4.0, original=64)
+
+
+def wkv(heads, dim, ff=0):
+    return {"type": "wkv", "mixer": {"heads": heads, "dim": dim}, "mlp": {"kind": "dense", "ff": ff} if ff else None}
+
+
+def parallel(left, right, ff=0):
+    """left = (heads, kv_heads, dim, vdim, rot dims, scaled?), right = (heads, kv_heads, dim, vdim, taps)."""
+    h, g, d, e, rd, scaled = left
+    rot = {"dims": rd, "base": 500.0, "scaling": dict(SCALING) if scaled else None} if rd else None
+    rh, rg, rk, rv, taps = right
+    return {"type": "parallel",
+            "mixer": {"left": {"heads": h, "kv_heads": g, "dim": d, "vdim": e, "scale": 0.9 / d ** 0.5, "rot": rot},
+                      "right": {"heads": rh, "kv_heads": rg, "dim": rk, "vdim": rv, "conv": taps}},
+            "mlp": {"kind": "dense", "ff": ff} if ff else None}
+
+
+def config(layers, width=96, vocab=131, side=12, eps=3e-5):
+    return {"architecture": "Sizilorn", "vocab": vocab, "width": width, "norm": {"eps": eps},
+            "token_side": {"dim": side} if side else None, "layers": layers}
+
+
+def weights(cfg, seed=0, rank=5):
+    """name -> float32 array holding bfloat16 values."""
+    rng = np.random.default_rng(seed)
+    C, V, side = cfg["width"], cfg["vocab"], (cfg.get("token_side") or {}).get("dim", 0)
+    w = {}
+
+    def mat(name, rows, cols, gain=1.0):
+        w[name] = rng.standard_normal((rows, cols)) * gain / np.sqrt(cols)
+
+    def around_one(name, n):
+        w[name] = 1.0 + 0.3 * rng.standard_normal(n)
+
+    def norm(name):
+        around_one(name, C)
+        w[name + ".b"] = 0.1 * rng.standard_normal(C)
+        w[name + ".alpha"] = np.array(rng.uniform(0.5, 0.9))
+
+    w["embed"] = rng.standard_normal((V, C))
+    if side:
+        w["side.embed"] = rng.standard_normal((V, side * len(cfg["layers"])))
+    for i, layer in enumerate(cfg["layers"]):
+        p, m = f"l{i}.", layer["mixer"]
+        norm(p + "norm1")
+        if layer["type"] == "wkv":
+            n = m["heads"] * m["dim"]
+            for s in "rkvgw":
+                w[p + "mix.mu." + s] = rng.uniform(0, 1, C)
+            for s in "rkvg":
+                mat(p + "mix." + s, n, C)
+            mat(p + "mix.w1", rank, C)
+            mat(p + "mix.w2", n, rank)
+            w[p + "mix.w0"] = rng.uniform(-6.0, 0.5, n)
+            w[p + "mix.u"] = rng.standard_normal((m["heads"], m["dim"]))
+            around_one(p + "mix.norm", n)
+            mat(p + "mix.o", C, n)
+        else:
+            a, d = m["left"], m["right"]
+            L, R = p + "mix.left.", p + "mix.right."
+            mat(L + "q", a["heads"] * a["dim"], C)
+            mat(L + "k", a["kv_heads"] * a["dim"], C)
+            mat(L + "v", a["kv_heads"] * a["vdim"], C)
+            mat(L + "g", a["heads"], C)
+            w[L + "q.norm"] = 1.5 + 0.3 * rng.standard_normal(a["dim"])
+            w[L + "k.norm"] = 1.5 + 0.3 * rng.standard_normal(a["dim"])
+            mat(L + "o", C, a["heads"] * a["vdim"])
+            around_one(L + "out", C)
+            for s, n in (("q", d["kv_heads"] * d["dim"]), ("k", d["kv_heads"] * d["dim"]), ("v", d["heads"] * d["vdim"])):
+                mat(R + s, n, C, 2.0)
+                w[R + s + ".conv"] = rng.standard_normal((n, d["conv"])) / np.sqrt(d["conv"])
+            mat(R + "a", d["heads"], C)
+            mat(R + "b", d["heads"], C)
+            w[R + "A_log"] = rng.uniform(-1.0, 1.0, d["heads"])
+            w[R + "dt_bias"] = rng.uniform(-5.0, 0.0, d["heads"])
+            mat(R + "g", d["heads"] * d["vdim"], C)
+            around_one(R + "norm", d["vdim"])
+            mat(R + "o", C, d["heads"] * d["vdim"])
+            around_one(R + "out", C)
+        if layer["mlp"]:
+            norm(p + "norm2")
+            ff = layer["mlp"]["ff"]
+            mat(p + "mlp.gate", ff, C)
+            mat(p + "mlp.up", ff, C)
+            mat(p + "mlp.down", C, ff)
+        if side:
+            mat(p + "side.gate", side, C)
+            mat(p + "side.proj", C, side)
+            w[p + "side.norm"] = 0.5 + 0.2 * rng.standard_normal(C)
+    norm("final.norm")
+    mat("head", V, C)
+    return {k: mixers.bf16(np.asarray(v, np.float32)) for k, v in w.items()}
+
+
+def write(folder, cfg, w):
+    folder.mkdir(parents=True, exist_ok=True)
+    (folder / "config.json").write_text(json.dumps(cfg))
+    mixers.write_safetensors(folder / "model.safetensors", w)
+    return folder
+
+
+def load(folder, compute, capacity=1024, lanes=4, slots=4, **kw):
+    eng = importlib.import_module("macllm_infer_b200.engine")
+    return eng.Model.load(folder, compute=compute, kv_dtype="f32" if compute == "float32" else "f16", kv_capacity_tokens=capacity,
+                          max_batch_tokens=capacity, max_batch_lanes=lanes, state_slots=slots, **kw)
+
+
+# Root mean square of the difference over that of the expected rows.
+LIMIT = {"float32": 3e-5, "bfloat16": 4e-2}
+
+
+def row_errors(got, want):
+    return np.sqrt(np.mean((got - want) ** 2, axis=-1) / np.mean(want ** 2))
+
+
+def assert_rows(got, want, compute, what=""):
+    e = row_errors(got, want)
+    assert e.max() <= LIMIT[compute], f"{what}: row {int(e.argmax())} of {len(e)} is off by {e.max():.2e}"
+
+
+def cut(n, sizes):
+    """Portions of the given sizes, over and over, until n tokens are used."""
+    out, at, i = [], 0, 0
+    while at < n:
+        k = min(sizes[i % len(sizes)], n - at)
+        out.append(k)
+        at += k
+        i += 1
+    return out
+
+
+def run_portions(model, tokens, portions):
+    """Logits of every token, the sequence fed in portions."""
+    s = model.new_session()
+    rows, at = [], 0
+    for k in portions:
+        logits, _ = model.forward_batch([(s, tokens[at:at + k], at)], want_tokens=False, rows=[range(k)])
+        rows.append(logits)
+        at += k
+    s.close()
+    return np.concatenate(rows)

@@ -17,6 +17,7 @@ STRUCTS = {
     "mk_prefix_diagnostics": "PrefixDiagnostics", "mk_lane": "Lane", "mk_engine_config": "EngineConfig", "mk_request": "Request",
     "mk_tick_lane": "TickLane", "mk_engine_stats": "EngineStats", "mk_kernel_profile": "KernelProfile", "mk_attn_case": "AttnCase",
     "mk_gguf_summary": "GgufSummary", "mk_lane_sampling": "LaneSampling", "mk_tick_info": "TickInfo", "mk_batch_trace": "BatchTrace", "mk_request_metrics": "RequestMetrics",
+    "mk_mixer_summary": "MixerSummary",
 }
 
 
