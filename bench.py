@@ -26,7 +26,8 @@ N > 1 (torchrun): dense workloads run N independent replicas, one per GPU, each 
 has no exchange step for them); the sparse-MoE workload runs expert parallelism with data-parallel lanes - every rank
 serves its own requests and each MoE layer exchanges the routed rows (`config.ep`; `--ep off` for replicas).  The
 reported time is the max over ranks.  `--http-clients N` adds a step through the `/completion` endpoint (`http` key),
-`--microbench` prints the Q4_K matmul GB/s of the decode shapes instead.
+`--microbench` prints the Q4_K matmul GB/s of the decode shapes instead, `--mixer` the prefill and decode throughput of
+mixer-built decoders (Sizilorn layers at real-model sizes, random weights) beside the closest GGUF family of equal size.
 """
 from __future__ import annotations
 
@@ -640,6 +641,7 @@ def main():
                          "resident; N > 1: expert parallelism over the same ranks)")
     ap.add_argument("--no-profiled-step", action="store_true", help="skip the extra step that times every launch")
     ap.add_argument("--microbench", action="store_true", help="Q4_K matmul GB/s on the decode shapes instead of the workload")
+    ap.add_argument("--mixer", action="store_true", help="prefill / decode throughput of mixer-built decoders beside the closest GGUF family instead of the workload")
     args = ap.parse_args()
 
     rank, local, world, dist = dist_setup(args.gpus)
@@ -668,6 +670,15 @@ def main():
     if args.microbench:
         if rank == 0:
             microbench()
+        return
+
+    if args.mixer:
+        if rank == 0:
+            bench = importlib.import_module("macllm_infer_b200.mixer_bench")
+            sampler = ClockSampler(local)
+            sampler.start()
+            results = bench.run(peaks(), max(3, args.warmup), max(5, args.steps))
+            print(json.dumps(dict(metric="mixer decoders: device tokens/s", unit=UNIT, data="synthetic", dtype="bf16", results=results, clocks=sampler.stop())))
         return
 
     if args.impl == "reference":

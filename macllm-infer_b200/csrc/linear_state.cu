@@ -1,11 +1,13 @@
 // See linear_state.h.
 //
-// A warp holds eight value columns of one (lane, head): four groups of eight threads, two columns per group, the column's keys
-// shared out over the group's threads in runs of four.  The state stays in registers while the lane's rows go by.  Rows arrive
-// in shared memory in chunks, fetched with cp.async while the chunk before is being worked on; the sums over the keys of four
-// rows are folded together (each exchange halves what is left), so a row costs under two shuffles per column pair - except the
-// delta rule's S^T k, which the row itself depends on.  Wide prompts cut a head's columns over CTAs of four warps and leave the
-// head norm to a second kernel; ticks of short lanes give a whole head to one CTA, which then finishes the output row itself.
+// A group of KS threads holds two value columns of one (lane, head), the columns' keys shared out over the group's threads in
+// runs of four; the state stays in registers while the lane's rows go by.  Rows arrive in shared memory in chunks, fetched with
+// cp.async while the chunk before is being worked on, and a thread loads the next row's vectors while it works on the current
+// one.  The sums over the keys of four rows are folded together (each exchange halves what is left), so a row costs under two
+// shuffles per column pair - except the delta rule's S^T k, which the row itself depends on.  Wide prompts cut a head's columns
+// over CTAs of four warps with sixteen threads per column pair (the delta rule's chain of dependent steps sets the pace there)
+// and leave the head norm to a second kernel; ticks of short lanes give a whole head to one CTA, which then finishes the output
+// row itself: there the state's way through the SM is what counts.
 #include "linear_state.h"
 #include <algorithm>
 
@@ -13,7 +15,6 @@ namespace mk {
 
 namespace {
 
-constexpr int LS_COLS = 8;        // value columns of a warp
 constexpr int LS_WIDE_WARPS = 4;  // warps of a CTA that owns part of a head
 constexpr int LS_MAX_FINISH_V = 128;
 
@@ -51,7 +52,8 @@ __device__ __forceinline__ void sum_rows(float* dst, int pitch, int n, int width
     }
 }
 
-// Eight values per thread, folded over the eight threads of a group: thread t of the group ends with the sum of value t.
+// Eight values per thread, folded over the KS threads of a group: thread t ends with the sum of value t % 8.
+template <int KS>
 __device__ __forceinline__ float fold8(const float (&v)[8], int t) {
     float a[4], b[2];
     const bool h4 = (t & 4) != 0, h2 = (t & 2) != 0, h1 = (t & 1) != 0;
@@ -59,62 +61,71 @@ __device__ __forceinline__ float fold8(const float (&v)[8], int t) {
     for (int i = 0; i < 4; ++i) a[i] = (h4 ? v[i + 4] : v[i]) + __shfl_xor_sync(0xffffffffu, h4 ? v[i] : v[i + 4], 4);
 #pragma unroll
     for (int i = 0; i < 2; ++i) b[i] = (h2 ? a[i + 2] : a[i]) + __shfl_xor_sync(0xffffffffu, h2 ? a[i] : a[i + 2], 2);
-    return (h1 ? b[1] : b[0]) + __shfl_xor_sync(0xffffffffu, h1 ? b[0] : b[1], 1);
+    float r = (h1 ? b[1] : b[0]) + __shfl_xor_sync(0xffffffffu, h1 ? b[0] : b[1], 1);
+#pragma unroll
+    for (int x = 8; x < KS; x <<= 1) r += __shfl_xor_sync(0xffffffffu, r, x);
+    return r;
 }
 
-// One head's row o[0 .. vdim) of packed row `row` (in shared or global memory), by one warp.
-__device__ __forceinline__ void finish_head_row(const LinearStateArgs& a, const float* o, int64_t row, int head, int lane) {
+// One head's row o[0 .. vdim) of packed row `row`, by one warp; gate[v] and norm weights nw[v] of the head.
+template <typename Gate>
+__device__ __forceinline__ void finish_head_row(const LinearStateArgs& a, const float* o, Gate gate, const float* nw, int64_t row, int head, int lane) {
     float ss = 0.f;
     for (int v = lane; v < a.vdim; v += 32) ss += o[v] * o[v];
     ss = warp_sum(ss);
     const float root = sqrtf(ss / (float)a.vdim + a.eps);
-    const float* nw = a.norm_w + (a.norm_per_head ? head * a.vdim : 0);
-    for (int v = lane; v < a.vdim; v += 32) {
-        const float g = a.gate.at(row, a.gate_col + head * a.vdim + v);
-        a.image.put(row, head * a.vdim + v, o[v] / root * nw[v] * silu_f(g));
-    }
+    for (int v = lane; v < a.vdim; v += 32) a.image.put(row, head * a.vdim + v, o[v] / root * nw[v] * silu_f(gate(v)));
     if (head == a.heads - 1)
         for (int c = a.heads * a.vdim + lane; c < a.image.ld; c += 32) a.image.put(row, c, 0.f);
 }
 
-template <int KD, int TT, bool WKV>
-struct LsSmem {
-    static constexpr int KROWS = WKV ? 3 : 2;  // r, k, decay  /  q, k
-    static __host__ __device__ constexpr size_t stage_floats(int cols) { return (size_t)TT * (KROWS * KD + cols + (WKV ? 0 : 4)); }
-    static __host__ __device__ constexpr size_t bytes(int cols, bool finish) { return (2 * stage_floats(cols) + (finish ? (size_t)TT * cols : 0)) * 4; }
+template <int KD, bool WKV, bool FINISH>
+struct Ls {
+    static constexpr int KS = !FINISH && KD >= 64 ? 16 : 8;  // threads of a column pair
+    static constexpr int KE = KD / KS;                       // keys of a thread
+    static constexpr int COLS = 32 / KS * 2;                 // value columns of a warp
+    static constexpr int TT = FINISH ? 4 : 16;               // rows of a chunk
+    static constexpr int KROWS = WKV ? 3 : 2;                // r, k, decay  /  q, k
+    static constexpr int MAX_THREADS = FINISH ? LS_MAX_FINISH_V / COLS * 32 : LS_WIDE_WARPS * 32;
+    static constexpr int MIN_CTAS = FINISH ? (KD >= 128 ? 2 : 3) : 1;
+    // stage: KROWS key-wide rows, the value row, the gate row (FINISH), decay and beta (delta rule)
+    static __host__ __device__ constexpr int row_floats(int cols) { return KROWS * KD + cols * (FINISH ? 2 : 1) + (WKV ? 0 : 4); }
+    static __host__ __device__ constexpr int stage_floats(int cols) { return TT * row_floats(cols); }
+    // two stages; FINISH: the output rows and the head's norm weights
+    static __host__ __device__ constexpr size_t bytes(int cols) { return (2 * (size_t)stage_floats(cols) + (FINISH ? (size_t)(TT + 1) * cols : 0)) * 4; }
 };
 
 template <int KD, bool WKV, bool FINISH>
-__global__ void __launch_bounds__(FINISH ? LS_MAX_FINISH_V / LS_COLS * 32 : LS_WIDE_WARPS * 32)
-linear_state_kernel(WkvScanArgs wa, DeltaScanArgs da) {
-    constexpr int TT = FINISH ? 4 : 16;
-    constexpr int KE = KD / 8;   // keys of a thread
-    constexpr int NJ = KE / 4;
-    using L = LsSmem<KD, TT, WKV>;
+__global__ void __launch_bounds__(Ls<KD, WKV, FINISH>::MAX_THREADS, Ls<KD, WKV, FINISH>::MIN_CTAS)
+linear_state_kernel(const __grid_constant__ WkvScanArgs wa, const __grid_constant__ DeltaScanArgs da) {
+    using L = Ls<KD, WKV, FINISH>;
+    constexpr int TT = L::TT, KS = L::KS, KE = L::KE, NJ = KE / 4;
     extern __shared__ __align__(16) float ls_smem[];
     const LinearStateArgs& a = WKV ? wa.common : da.common;
 
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, grp = lane >> 3, ks = lane & 7;
-    const int cols = (int)(blockDim.x >> 5) * LS_COLS;  // columns of this CTA
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, ks = lane & (KS - 1);
+    const int cols = (int)(blockDim.x >> 5) * L::COLS;                 // columns of this CTA
     const int col0 = blockIdx.x * cols;
-    const int head = blockIdx.y, seq = blockIdx.z;
-    const int c_loc = warp * LS_COLS + grp * 2;         // first of the thread's two columns, within the CTA
+    const int head = blockIdx.y;
+    const int c_loc = warp * L::COLS + lane / KS * 2;                  // first of the thread's two columns, within the CTA
     const int my_cols = min(cols, a.vdim - col0);
+    float* s_o = ls_smem + 2 * L::stage_floats(cols);                  // FINISH: [TT][cols]
+    float* s_nw = s_o + TT * cols;                                     // FINISH: [cols]
 
-    // The slot halves were staged by the host and the committed state was written by an earlier tick: neither depends on the
-    // predecessor kernel, so the state is on its way before the wait.
+    // The lane record was staged by the host, weights never change and the committed state was written by an earlier tick: none
+    // of them depends on the predecessor kernel, so all are on their way before the wait.
     pdl_trigger();
-    const int2 half = a.lanes.halves[seq];
+    const StateLane sl = a.lanes.at(blockIdx.z);
     float S[2][KE];
     const int64_t head_state = (int64_t)a.vdim * KD;
 #pragma unroll
     for (int c = 0; c < 2; ++c) {
         const int v = col0 + c_loc + c;
-        const bool live = half.x >= 0 && v < a.vdim;
-        const float4* src = reinterpret_cast<const float4*>(a.state + ((int64_t)half.x * a.heads + head) * head_state + (int64_t)v * KD);
+        const bool live = sl.in >= 0 && v < a.vdim;
+        const float4* src = reinterpret_cast<const float4*>(a.state + ((int64_t)sl.in * a.heads + head) * head_state + (int64_t)v * KD);
 #pragma unroll
         for (int j = 0; j < NJ; ++j) {
-            const float4 x = live ? src[j * 8 + ks] : make_float4(0.f, 0.f, 0.f, 0.f);
+            const float4 x = live ? __ldcs(src + j * KS + ks) : make_float4(0.f, 0.f, 0.f, 0.f);
             S[c][4 * j] = x.x; S[c][4 * j + 1] = x.y; S[c][4 * j + 2] = x.z; S[c][4 * j + 3] = x.w;
         }
     }
@@ -122,24 +133,29 @@ linear_state_kernel(WkvScanArgs wa, DeltaScanArgs da) {
     if (WKV) {
 #pragma unroll
         for (int e = 0; e < KE; ++e) {
-            const int i = (e >> 2) * 32 + ks * 4 + (e & 3);
+            const int i = (e >> 2) * 4 * KS + ks * 4 + (e & 3);
             U[WKV ? e : 0] = i < a.dim ? wa.bonus[head * a.dim + i] : 0.f;
         }
     }
+    if (FINISH)
+        for (int v = threadIdx.x; v < a.vdim; v += blockDim.x) s_nw[v] = a.norm_w[(a.norm_per_head ? head * a.vdim : 0) + v];
     // key columns past the true dimension and value columns past the last stay zero in both stages
-    for (int i = threadIdx.x; i < (int)(2 * L::stage_floats(cols)); i += blockDim.x) ls_smem[i] = 0.f;
-    __syncthreads();
+    if (a.dim < KD || my_cols < cols) {
+        for (int i = threadIdx.x; i < 2 * L::stage_floats(cols); i += blockDim.x) ls_smem[i] = 0.f;
+        __syncthreads();
+    }
     pdl_wait();
 
-    const int first = a.lanes.cu[seq], n = a.lanes.cu[seq + 1] - first;
+    const int first = sl.first, n = sl.n;
     const int kv_head = WKV ? head : head / (a.heads / da.kv_heads);
     const bool vec = (a.dim & 3) == 0 && (a.vdim & 3) == 0;
-    auto stage = [&](int which) { return ls_smem + (size_t)which * L::stage_floats(cols); };
+    auto stage = [&](int which) { return ls_smem + which * L::stage_floats(cols); };
     auto fetch = [&](int chunk) {
         float* s = stage(chunk & 1);
         const int64_t r0 = first + chunk * TT;
         const int m = min(TT, n - chunk * TT);
-        float* s_v = s + (size_t)TT * L::KROWS * KD;
+        float* s_v = s + TT * L::KROWS * KD;
+        float* s_g = s_v + TT * cols;
         if (WKV) {
             const Shares& y = wa.rkv;
             const int h0 = head * a.dim;
@@ -159,12 +175,13 @@ linear_state_kernel(WkvScanArgs wa, DeltaScanArgs da) {
             fetch_rows(s, KD, m, a.dim, vec, [&](int r) { return da.q + (r0 + r) * kw + kv_head * a.dim; });
             fetch_rows(s + TT * KD, KD, m, a.dim, vec, [&](int r) { return da.k + (r0 + r) * kw + kv_head * a.dim; });
             fetch_rows(s_v, cols, m, my_cols, vec && (my_cols & 3) == 0, [&](int r) { return da.v + (r0 + r) * vw + head * a.vdim + col0; });
-            float* s_c = s_v + (size_t)TT * cols;
+            float* s_c = s_v + TT * cols * (FINISH ? 2 : 1);
             for (int r = threadIdx.x; r < m; r += blockDim.x) {
                 ls_cp_async4(s_c + 4 * r, da.decay + (r0 + r) * a.heads + head);
                 ls_cp_async4(s_c + 4 * r + 1, da.beta + (r0 + r) * a.heads + head);
             }
         }
+        if (FINISH) sum_rows(s_g, cols, m, a.vdim, a.gate, r0, a.gate_col + head * a.vdim);
         ls_commit();
     };
 
@@ -177,89 +194,125 @@ linear_state_kernel(WkvScanArgs wa, DeltaScanArgs da) {
         } else {
             ls_wait<0>();
         }
-        __syncthreads();
-        const float* s = stage(ch & 1);
-        const float* s_v = s + (size_t)TT * L::KROWS * KD;
+        float* s = stage(ch & 1);
+        float* s_v = s + TT * L::KROWS * KD;
+        float* s_c = s_v + TT * cols * (FINISH ? 2 : 1);
         const int m = min(TT, n - ch * TT);
-        float* s_o = ls_smem + 2 * L::stage_floats(cols);  // FINISH: [TT][cols]
-#pragma unroll 1
-        for (int t0 = 0; t0 < m; t0 += 4) {
+        if (!FINISH && (m & 3) != 0) {
+            // rows are taken four at a time: those past the last one change nothing (k = 0, no decay)
+            __syncthreads();
+            for (int t = m; t < ((m + 3) & ~3); ++t) {
+                for (int i = threadIdx.x; i < KD; i += blockDim.x) {
+                    s[t * KD + i] = 0.f;
+                    s[TT * KD + t * KD + i] = 0.f;
+                    if (WKV) s[2 * TT * KD + t * KD + i] = 1.f;
+                }
+                for (int i = threadIdx.x; i < cols; i += blockDim.x) s_v[t * cols + i] = 0.f;
+                if (!WKV && threadIdx.x == 0) {
+                    s_c[4 * t] = 1.f;
+                    s_c[4 * t + 1] = 0.f;
+                }
+            }
+        }
+        __syncthreads();
+        // one row's vectors: r | q in x, k in y, decay in w (WKV)
+        struct Row {
+            float x[KE], y[KE], w[WKV ? KE : 1];
+            float2 v, gb;
+        };
+        auto load_row = [&](int t, Row& r) {
+            const float4* x4 = reinterpret_cast<const float4*>(s + t * KD) + ks;
+            const float4* y4 = reinterpret_cast<const float4*>(s + TT * KD + t * KD) + ks;
+#pragma unroll
+            for (int j = 0; j < NJ; ++j) {
+                const float4 y = y4[j * KS], x = x4[j * KS];
+                r.y[4 * j] = y.x; r.y[4 * j + 1] = y.y; r.y[4 * j + 2] = y.z; r.y[4 * j + 3] = y.w;
+                r.x[4 * j] = x.x; r.x[4 * j + 1] = x.y; r.x[4 * j + 2] = x.z; r.x[4 * j + 3] = x.w;
+            }
+            if constexpr (WKV) {
+                const float4* w4 = reinterpret_cast<const float4*>(s + 2 * TT * KD + t * KD) + ks;
+#pragma unroll
+                for (int j = 0; j < NJ; ++j) {
+                    const float4 w = w4[j * KS];
+                    r.w[4 * j] = w.x; r.w[4 * j + 1] = w.y; r.w[4 * j + 2] = w.z; r.w[4 * j + 3] = w.w;
+                }
+            } else {
+                r.gb = *reinterpret_cast<const float2*>(s_c + 4 * t);
+            }
+            r.v = *reinterpret_cast<const float2*>(s_v + t * cols + c_loc);
+        };
+        auto step = [&](const Row& r, float& out0, float& out1) {
+            float o0 = 0.f, o1 = 0.f;
+            if constexpr (WKV) {
+#pragma unroll
+                for (int e = 0; e < KE; ++e) {
+                    const float uk = U[e] * r.y[e];
+                    o0 = fmaf(r.x[e], fmaf(uk, r.v.x, S[0][e]), o0);
+                    o1 = fmaf(r.x[e], fmaf(uk, r.v.y, S[1][e]), o1);
+                    S[0][e] = fmaf(r.w[e], S[0][e], r.y[e] * r.v.x);
+                    S[1][e] = fmaf(r.w[e], S[1][e], r.y[e] * r.v.y);
+                }
+            } else {
+                float d0[2] = {0.f, 0.f}, d1[2] = {0.f, 0.f};
+#pragma unroll
+                for (int e = 0; e < KE; ++e) {
+                    d0[e & 1] = fmaf(S[0][e], r.y[e], d0[e & 1]);
+                    d1[e & 1] = fmaf(S[1][e], r.y[e], d1[e & 1]);
+                }
+                float m0 = d0[0] + d0[1], m1 = d1[0] + d1[1];
+#pragma unroll
+                for (int x = 1; x < KS; x <<= 1) {
+                    m0 += __shfl_xor_sync(0xffffffffu, m0, x);
+                    m1 += __shfl_xor_sync(0xffffffffu, m1, x);
+                }
+                const float u0 = r.gb.y * (r.v.x - r.gb.x * m0), u1 = r.gb.y * (r.v.y - r.gb.x * m1);
+#pragma unroll
+                for (int e = 0; e < KE; ++e) {
+                    S[0][e] = fmaf(r.y[e], u0, r.gb.x * S[0][e]);
+                    S[1][e] = fmaf(r.y[e], u1, r.gb.x * S[1][e]);
+                    o0 = fmaf(S[0][e], r.x[e], o0);
+                    o1 = fmaf(S[1][e], r.x[e], o1);
+                }
+            }
+            out0 = o0;
+            out1 = o1;
+        };
+        if constexpr (FINISH) {
             float part[8];
+            Row r;
 #pragma unroll
             for (int i = 0; i < 4; ++i) {
                 part[2 * i] = part[2 * i + 1] = 0.f;
-                const int t = t0 + i;
-                if (t >= m) continue;  // uniform over the CTA
-                const float2 v = *reinterpret_cast<const float2*>(s_v + t * cols + c_loc);
-                const float4* k4 = reinterpret_cast<const float4*>(s + TT * KD + t * KD) + ks;
-                const float4* q4 = reinterpret_cast<const float4*>(s + t * KD) + ks;  // r / q
-                if constexpr (WKV) {
-                    const float4* w4 = reinterpret_cast<const float4*>(s + 2 * TT * KD + t * KD) + ks;
-                    float o0 = 0.f, o1 = 0.f;
-#pragma unroll
-                    for (int j = 0; j < NJ; ++j) {
-                        const float4 r = q4[j * 8], k = k4[j * 8], w = w4[j * 8];
-                        const float rr[4] = {r.x, r.y, r.z, r.w}, kk[4] = {k.x, k.y, k.z, k.w}, ww[4] = {w.x, w.y, w.z, w.w};
-#pragma unroll
-                        for (int e = 0; e < 4; ++e) {
-                            const float uk = U[4 * j + e] * kk[e];
-                            o0 = fmaf(rr[e], fmaf(uk, v.x, S[0][4 * j + e]), o0);
-                            o1 = fmaf(rr[e], fmaf(uk, v.y, S[1][4 * j + e]), o1);
-                            S[0][4 * j + e] = fmaf(ww[e], S[0][4 * j + e], kk[e] * v.x);
-                            S[1][4 * j + e] = fmaf(ww[e], S[1][4 * j + e], kk[e] * v.y);
-                        }
-                    }
-                    part[2 * i] = o0;
-                    part[2 * i + 1] = o1;
-                } else {
-                    const float2 gb = *reinterpret_cast<const float2*>(s_v + (size_t)TT * cols + 4 * t);
-                    float d0[2] = {0.f, 0.f}, d1[2] = {0.f, 0.f};
-                    float kk[KE];
-#pragma unroll
-                    for (int j = 0; j < NJ; ++j) {
-                        const float4 k = k4[j * 8];
-                        kk[4 * j] = k.x; kk[4 * j + 1] = k.y; kk[4 * j + 2] = k.z; kk[4 * j + 3] = k.w;
-                    }
-#pragma unroll
-                    for (int e = 0; e < KE; ++e) {
-                        d0[e & 1] = fmaf(S[0][e], kk[e], d0[e & 1]);
-                        d1[e & 1] = fmaf(S[1][e], kk[e], d1[e & 1]);
-                    }
-                    float m0 = d0[0] + d0[1], m1 = d1[0] + d1[1];
-#pragma unroll
-                    for (int x = 1; x < 8; x <<= 1) {
-                        m0 += __shfl_xor_sync(0xffffffffu, m0, x);
-                        m1 += __shfl_xor_sync(0xffffffffu, m1, x);
-                    }
-                    const float u0 = gb.y * (v.x - gb.x * m0), u1 = gb.y * (v.y - gb.x * m1);
-                    float o0 = 0.f, o1 = 0.f;
-#pragma unroll
-                    for (int j = 0; j < NJ; ++j) {
-                        const float4 q = q4[j * 8];
-                        const float qq[4] = {q.x, q.y, q.z, q.w};
-#pragma unroll
-                        for (int e = 0; e < 4; ++e) {
-                            S[0][4 * j + e] = fmaf(kk[4 * j + e], u0, gb.x * S[0][4 * j + e]);
-                            S[1][4 * j + e] = fmaf(kk[4 * j + e], u1, gb.x * S[1][4 * j + e]);
-                            o0 = fmaf(S[0][4 * j + e], qq[e], o0);
-                            o1 = fmaf(S[1][4 * j + e], qq[e], o1);
-                        }
-                    }
-                    part[2 * i] = o0;
-                    part[2 * i + 1] = o1;
+                if (i < m) {  // uniform over the CTA
+                    load_row(i, r);
+                    step(r, part[2 * i], part[2 * i + 1]);
                 }
             }
-            const float o = fold8(part, ks);
-            const int t = t0 + (ks >> 1), c = c_loc + (ks & 1);
-            if (t < m && col0 + c < a.vdim) {
-                if (FINISH) s_o[t * cols + c] = o;
-                else a.out[(int64_t)(first + ch * TT + t) * a.heads * a.vdim + head * a.vdim + col0 + c] = o;
-            }
-        }
-        __syncthreads();  // the stage is free for the chunk after next, and the output rows are complete
-        if (FINISH) {
-            for (int t = warp; t < m; t += (int)(blockDim.x >> 5)) finish_head_row(a, s_o + t * cols, first + ch * TT + t, head, lane);
+            const float o = fold8<KS>(part, ks);
+            const int t = ks >> 1, c = c_loc + (ks & 1);
+            if (t < m && c < a.vdim) s_o[t * cols + c] = o;
             __syncthreads();
+            const float* s_g = s_v + TT * cols;
+            for (int t = warp; t < m; t += (int)(blockDim.x >> 5))
+                finish_head_row(a, s_o + t * cols, [&](int v) { return s_g[t * cols + v]; }, s_nw, first + ch * TT + t, head, lane);
+            __syncthreads();  // the stage is free for the chunk after next
+        } else {
+            Row rows[2];
+            load_row(0, rows[0]);
+#pragma unroll 1
+            for (int t0 = 0; t0 < m; t0 += 4) {
+                float part[8];
+#pragma unroll
+                for (int i = 0; i < 4; ++i) {
+                    load_row(min(t0 + i + 1, TT - 1), rows[(i + 1) & 1]);
+                    step(rows[i & 1], part[2 * i], part[2 * i + 1]);
+                }
+                const float o = fold8<KS>(part, ks);
+                const int t = t0 + ((ks & 7) >> 1), c = c_loc + (ks & 1);
+                if (ks < 8 && t < m && col0 + c < a.vdim)
+                    a.out[(int64_t)(first + ch * TT + t) * a.heads * a.vdim + head * a.vdim + col0 + c] = o;
+            }
+            __syncthreads();  // the stage is free for the chunk after next
         }
     }
 
@@ -267,9 +320,9 @@ linear_state_kernel(WkvScanArgs wa, DeltaScanArgs da) {
     for (int c = 0; c < 2; ++c) {
         const int v = col0 + c_loc + c;
         if (v >= a.vdim) continue;
-        float4* dst = reinterpret_cast<float4*>(a.state + ((int64_t)half.y * a.heads + head) * head_state + (int64_t)v * KD);
+        float4* dst = reinterpret_cast<float4*>(a.state + ((int64_t)sl.out * a.heads + head) * head_state + (int64_t)v * KD);
 #pragma unroll
-        for (int j = 0; j < NJ; ++j) dst[j * 8 + ks] = make_float4(S[c][4 * j], S[c][4 * j + 1], S[c][4 * j + 2], S[c][4 * j + 3]);
+        for (int j = 0; j < NJ; ++j) __stcs(dst + j * KS + ks, make_float4(S[c][4 * j], S[c][4 * j + 1], S[c][4 * j + 2], S[c][4 * j + 3]));
     }
 }
 
@@ -280,15 +333,17 @@ __global__ void __launch_bounds__(128) head_norm_gate_kernel(LinearStateArgs a, 
     if (i >= (int64_t)rows * a.heads) return;
     const int64_t row = i / a.heads;
     const int head = (int)(i % a.heads);
-    finish_head_row(a, a.out + row * a.heads * a.vdim + head * a.vdim, row, head, threadIdx.x & 31);
+    finish_head_row(a, a.out + row * a.heads * a.vdim + head * a.vdim, [&](int v) { return a.gate.at(row, a.gate_col + head * a.vdim + v); },
+                    a.norm_w + (a.norm_per_head ? head * a.vdim : 0), row, head, threadIdx.x & 31);
 }
 
 template <int KD, bool WKV, bool FINISH>
 void launch_variant(const WkvScanArgs& wa, const DeltaScanArgs& da, cudaStream_t s) {
     const LinearStateArgs& a = WKV ? wa.common : da.common;
-    const int warps = FINISH ? (a.vdim + LS_COLS - 1) / LS_COLS : LS_WIDE_WARPS;
-    const int cols = warps * LS_COLS;
-    const size_t smem = LsSmem<KD, FINISH ? 4 : 16, WKV>::bytes(cols, FINISH);
+    using L = Ls<KD, WKV, FINISH>;
+    const int warps = FINISH ? (a.vdim + L::COLS - 1) / L::COLS : LS_WIDE_WARPS;
+    const int cols = warps * L::COLS;
+    const size_t smem = L::bytes(cols);
     auto* kernel = linear_state_kernel<KD, WKV, FINISH>;
     ensure_dynamic_smem(reinterpret_cast<const void*>(kernel), smem);
     const dim3 grid((unsigned)((a.vdim + cols - 1) / cols), (unsigned)a.heads, (unsigned)a.lanes.lanes);

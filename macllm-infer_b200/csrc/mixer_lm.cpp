@@ -317,7 +317,7 @@ void MixerLm::alloc_activations() {
     ddecay_.alloc((size_t)(T * dh) * 4);
     if (!f32_)
         for (DevBuf& p : partial_) p.alloc(kSplitScratchBytes);
-    size_t extra = (size_t)B * sizeof(int2) + 16;
+    size_t extra = (size_t)B * sizeof(StateLane) + 16;
     size_t part_o = 0, part_ml = 0, counters = 0;
     for (const Geometry& g : geo_) {
         if (g.tc) {
@@ -651,14 +651,15 @@ void MixerLm::run_parallel(const Tick& t, int l, Pending& pend, const std::vecto
 void MixerLm::run_forward(const std::vector<LmLane>& lanes, KvReservation& r, uint32_t flags) {
     Tick t = stage_tick(lanes, r, flags);
     const int B = t.B, T = t.T, R = t.R, C = ms_.width;
-    std::vector<int2> halves;
-    int longest = 0;
+    std::vector<StateLane> halves;
+    int longest = 0, first_row = 0;
     for (const LmLane& l : lanes) {
-        halves.push_back(make_int2(l.state_in, l.state_out));
+        halves.push_back(StateLane{l.state_in, l.state_out, first_row, l.n_tokens});
+        first_row += l.n_tokens;
         longest = std::max(longest, l.n_tokens);
     }
     short_lanes_ = longest <= kShortLane;
-    const size_t off_halves = stage_bytes(t, halves.data(), halves.size() * sizeof(int2));
+    const size_t off_halves = stage_bytes(t, halves.data(), halves.size() * sizeof(StateLane));
     std::vector<int32_t> sp((size_t)B), nt((size_t)B), nb((size_t)B);
     for (int i = 0; i < B; ++i) {
         sp[(size_t)i] = lanes[(size_t)i].start_pos;
@@ -686,8 +687,7 @@ void MixerLm::run_forward(const std::vector<LmLane>& lanes, KvReservation& r, ui
         }
     }
     upload_tick(t, 64, KC_BATCH);
-    state_lanes_.cu = t.bd.cu_seqlens;
-    state_lanes_.halves = reinterpret_cast<const int2*>(t.dp + off_halves);
+    state_lanes_.lane = reinterpret_cast<const StateLane*>(t.dp + off_halves);
     state_lanes_.lanes = B;
     // copy-on-write page copies of shared partial tails
     for (const KvCowCopy& c : r.cow_copies())

@@ -134,15 +134,15 @@ __global__ void __launch_bounds__(RU_THREADS) row_update_kernel(RowUpdateArgs a)
         return;
     }
     const int lane = a.token_lane[row];
-    const int2 half = a.lanes.halves[lane];
-    const int first = a.lanes.cu[lane], last = a.lanes.cu[lane + 1] - 1;
+    const StateLane sl = a.lanes.at(lane);
+    const int first = sl.first, last = sl.first + sl.n - 1;
     const bool inside = row > first;
     if (inside) updated_row<VEC>(a, row - 1, prv, other, red);
     for (int c = threadIdx.x * VEC; c < a.width; c += step) {
         const Pack<VEC> h = norm_pack<VEC>(a, load_pack<VEC>(cur + c), c);
         Pack<VEC> p;
         if (inside) p = norm_pack<VEC>(a, load_pack<VEC>(prv + c), c);
-        else if (half.x >= 0) p = load_pack<VEC>(a.kept + (int64_t)half.x * a.width + c);
+        else if (sl.in >= 0) p = load_pack<VEC>(a.kept + (int64_t)sl.in * a.width + c);
         else
 #pragma unroll
             for (int i = 0; i < VEC; ++i) p.v[i] = 0.f;
@@ -153,86 +153,140 @@ __global__ void __launch_bounds__(RU_THREADS) row_update_kernel(RowUpdateArgs a)
             for (int i = 0; i < VEC; ++i) o.v[i] = fmaf(p.v[i] - h.v[i], mu.v[i], h.v[i]);
             put_pack<VEC>(a.mixes, (int64_t)m * a.rows + r, c, o);
         }
-        if (row == last) store_pack<VEC>(a.kept + (int64_t)half.y * a.width + c, h);
+        if (row == last) store_pack<VEC>(a.kept + (int64_t)sl.out * a.width + c, h);
     }
     for (int m = 0; m < a.n_mix; ++m) zero_tail(a.mixes, (int64_t)m * a.rows + r, a.width);
 }
 
 // ------------------------------------------------------------------------------------------------ WKV decay
 
-constexpr int WD_ROWS = 8, WD_THREADS = 128;
+constexpr int WD_COLS = 128;       // channels (threads) of a CTA
+constexpr int WD_STAGE_RANK = 256; // up to this rank the CTA's slice of w2 is staged, on its way before the predecessor is done
 
-__global__ void __launch_bounds__(WD_THREADS) wkv_decay_kernel(Shares low, int low_col, int rows, int rank, int channels,
-                                                               const float* __restrict__ w2t, const float* __restrict__ w0, float* decay) {
-    extern __shared__ float wd_z[];  // [rank][WD_ROWS]
+template <int ROWS>
+__global__ void __launch_bounds__(WD_COLS) wkv_decay_kernel(Shares low, int low_col, int rows, int rank, int channels,
+                                                            const float* __restrict__ w2t, const float* __restrict__ w0, float* decay) {
+    extern __shared__ __align__(16) float wd_smem[];
+    float* z = wd_smem;                // [rank][ROWS]
+    float* ws = z + rank * ROWS;       // [rank][WD_COLS]
+    const int r0 = blockIdx.y * ROWS, c = blockIdx.x * WD_COLS + threadIdx.x;
+    const bool staged = rank <= WD_STAGE_RANK, live = c < channels;
     pdl_trigger();
+    if (staged && live)
+        for (int j = 0; j < rank; ++j)
+            asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"((uint32_t)__cvta_generic_to_shared(ws + j * WD_COLS + threadIdx.x)),
+                         "l"(w2t + (int64_t)j * channels + c)
+                         : "memory");
+    asm volatile("cp.async.commit_group;" ::: "memory");
     pdl_wait();
-    const int r0 = blockIdx.y * WD_ROWS;
-    for (int i = threadIdx.x; i < rank * WD_ROWS; i += WD_THREADS) {
+    for (int i = threadIdx.x; i < rank * ROWS; i += WD_COLS) {
         const int r = i / rank, j = i - r * rank;
-        wd_z[j * WD_ROWS + r] = r0 + r < rows ? tanhf(low.at(r0 + r, low_col + j)) : 0.f;
+        z[j * ROWS + r] = r0 + r < rows ? tanhf(low.at(r0 + r, low_col + j)) : 0.f;
     }
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
     __syncthreads();
-    const int c = blockIdx.x * WD_THREADS + threadIdx.x;
-    if (c >= channels) return;
-    float acc[WD_ROWS];
+    if (!live) return;
+    float acc[ROWS];
 #pragma unroll
-    for (int r = 0; r < WD_ROWS; ++r) acc[r] = 0.f;
+    for (int r = 0; r < ROWS; ++r) acc[r] = 0.f;
 #pragma unroll 4
     for (int j = 0; j < rank; ++j) {
-        const float w = w2t[(int64_t)j * channels + c];
+        const float w = staged ? ws[j * WD_COLS + threadIdx.x] : w2t[(int64_t)j * channels + c];
 #pragma unroll
-        for (int r = 0; r < WD_ROWS; ++r) acc[r] = fmaf(wd_z[j * WD_ROWS + r], w, acc[r]);
+        for (int r = 0; r < ROWS; r += 4) {
+            const float4 v = *reinterpret_cast<const float4*>(z + j * ROWS + r);
+            acc[r] = fmaf(v.x, w, acc[r]);
+            acc[r + 1] = fmaf(v.y, w, acc[r + 1]);
+            acc[r + 2] = fmaf(v.z, w, acc[r + 2]);
+            acc[r + 3] = fmaf(v.w, w, acc[r + 3]);
+        }
     }
     const float b = w0[c];
 #pragma unroll
-    for (int r = 0; r < WD_ROWS; ++r)
+    for (int r = 0; r < ROWS; ++r)
         if (r0 + r < rows) decay[(int64_t)(r0 + r) * channels + c] = expf(-expf(acc[r] + b));
+}
+
+template <int ROWS>
+void launch_decay_rows(const Shares& low, int low_col, int rows, int rank, int channels, const float* w2t, const float* w0, float* decay, cudaStream_t s) {
+    const size_t smem = ((size_t)rank * ROWS + (rank <= WD_STAGE_RANK ? (size_t)rank * WD_COLS : 0)) * 4;
+    if (smem > (size_t)220 * 1024) throw std::runtime_error("launch_wkv_decay: the low rank is too large");
+    ensure_dynamic_smem(reinterpret_cast<const void*>(&wkv_decay_kernel<ROWS>), smem);
+    const dim3 grid((unsigned)((channels + WD_COLS - 1) / WD_COLS), (unsigned)((rows + ROWS - 1) / ROWS));
+    launch_pdl(wkv_decay_kernel<ROWS>, grid, dim3(WD_COLS), smem, s, low, low_col, rows, rank, channels, w2t, w0, decay);
+    MK_LAUNCH_CHECK();
 }
 
 // ------------------------------------------------------------------------------------------------ delta-rule inputs
 
-constexpr int DP_WARPS = 8;
+constexpr int DP_WARPS = 4;
 constexpr int DP_MAX_DIM = 256;
+constexpr int DP_ROWS = 4;   // rows a warp walks on wide ticks: their windows overlap and stay in L1
 
-// The raw projection of channel ch (of q | k | v) at row i of the lane (negative: before this tick).
-__device__ __forceinline__ float raw_value(const DeltaPrepArgs& a, int first, int i, int half_in, int ch, int y_col, int channels) {
-    if (i >= 0) return a.y.at(first + i, y_col);
-    if (half_in < 0) return 0.f;
-    return a.tail[((int64_t)half_in * (a.taps - 1) + (a.taps - 1 + i)) * channels + ch];
+// VEC neighbouring channels of the raw projection at row i of the lane (negative: before this tick).
+template <int VEC>
+__device__ __forceinline__ Pack<VEC> raw_pack(const DeltaPrepArgs& a, const StateLane& sl, int i, int ch, int y_col, int channels) {
+    if (i >= 0) return share_pack<VEC>(a.y, sl.first + i, y_col);
+    if (sl.in >= 0) return load_pack<VEC>(a.tail + ((int64_t)sl.in * (a.taps - 1) + (a.taps - 1 + i)) * channels + ch);
+    Pack<VEC> z;
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) z.v[e] = 0.f;
+    return z;
 }
 
-// One CTA per row; a warp takes one head of q, k or v at a time.
-__global__ void __launch_bounds__(DP_WARPS * 32) delta_prep_kernel(DeltaPrepArgs a) {
+// A warp takes one head of q, k or v and a run of consecutive packed rows; a lane takes VEC neighbouring channels of every 32 * VEC.
+template <int VEC>
+__global__ void __launch_bounds__(DP_WARPS * 32) delta_prep_kernel(DeltaPrepArgs a, int run) {
+    constexpr int NE = DP_MAX_DIM / 32 / VEC;
+    const int kw = a.kv_heads * a.dim, vw = a.heads * a.vdim, channels = 2 * kw + vw;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int u = blockIdx.y * DP_WARPS + warp, units = 2 * a.kv_heads + a.heads;
     pdl_trigger();
     pdl_wait();
-    const int64_t row = blockIdx.x;
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int seq = a.token_lane[row];
-    const int first = a.lanes.cu[seq], last = a.lanes.cu[seq + 1] - 1, i = (int)row - first;
-    const int2 half = a.lanes.halves[seq];
-    const int kw = a.kv_heads * a.dim, vw = a.heads * a.vdim, channels = 2 * kw + vw;
-    const int units = 2 * a.kv_heads + a.heads;
-    for (int u = warp; u < units; u += DP_WARPS) {
-        const int kind = u < a.kv_heads ? 0 : (u < 2 * a.kv_heads ? 1 : 2);
-        const int head = kind == 0 ? u : (kind == 1 ? u - a.kv_heads : u - 2 * a.kv_heads);
-        const int dim = kind == 2 ? a.vdim : a.dim;
-        const int ch0 = (kind == 0 ? 0 : (kind == 1 ? kw : 2 * kw)) + head * dim;
-        const int y0 = (kind == 0 ? a.q_col : (kind == 1 ? a.k_col : a.v_col)) + head * dim;
-        float* out = kind == 0 ? a.q + row * kw : (kind == 1 ? a.k + row * kw : a.v + row * vw);
-        float val[DP_MAX_DIM / 32];
+    const int r0 = blockIdx.x * run, r1 = min(a.rows, r0 + run);
+    if (blockIdx.y == 0)
+        for (int i = threadIdx.x; i < (r1 - r0) * a.heads; i += DP_WARPS * 32) {
+            const int row = r0 + i / a.heads, h = i % a.heads;
+            a.beta[(int64_t)row * a.heads + h] = sigmoid_f(a.y.at(row, a.b_col + h));
+            a.decay[(int64_t)row * a.heads + h] = recurrent::gated_delta_decay(a.y.at(row, a.a_col + h), a.dt_bias[h], a.log_decay[h]);
+        }
+    if (u >= units) return;
+    const int kind = u < a.kv_heads ? 0 : (u < 2 * a.kv_heads ? 1 : 2);
+    const int head = kind == 0 ? u : (kind == 1 ? u - a.kv_heads : u - 2 * a.kv_heads);
+    const int dim = kind == 2 ? a.vdim : a.dim;
+    const int ch0 = (kind == 0 ? 0 : (kind == 1 ? kw : 2 * kw)) + head * dim;
+    const int y0 = (kind == 0 ? a.q_col : (kind == 1 ? a.k_col : a.v_col)) + head * dim;
+    float* out = (kind == 0 ? a.q : (kind == 1 ? a.k : a.v)) + head * dim;
+    const int ldo = kind == 2 ? vw : kw;
+    const int hist = a.taps - 1;
+    int seq = -1;
+    StateLane sl{};
+    for (int row = r0; row < r1; ++row) {
+        if (seq < 0 || row >= sl.first + sl.n) {
+            seq = a.token_lane[row];
+            sl = a.lanes.at(seq);
+        }
+        const int i = row - sl.first;
+        Pack<VEC> val[NE];
         float ss = 0.f;
 #pragma unroll
-        for (int e = 0; e < DP_MAX_DIM / 32; ++e) {
-            const int c = e * 32 + lane;
-            val[e] = 0.f;
-            if (c < dim) {
-                float sum = 0.f;
-                for (int j = 0; j < a.taps; ++j)
-                    sum = fmaf(a.conv[(int64_t)j * channels + ch0 + c],
-                               raw_value(a, first, i - (a.taps - 1) + j, half.x, ch0 + c, y0 + c, channels), sum);
-                val[e] = silu_f(sum);
-                ss = fmaf(val[e], val[e], ss);
+        for (int e = 0; e < NE; ++e) {
+            const int c = (e * 32 + lane) * VEC;
+            if (c >= dim) continue;
+            Pack<VEC> sum;
+#pragma unroll
+            for (int x = 0; x < VEC; ++x) sum.v[x] = 0.f;
+#pragma unroll 4
+            for (int j = 0; j < a.taps; ++j) {
+                const Pack<VEC> w = load_pack<VEC>(a.conv + (int64_t)j * channels + ch0 + c);
+                const Pack<VEC> r = raw_pack<VEC>(a, sl, i - hist + j, ch0 + c, y0 + c, channels);
+#pragma unroll
+                for (int x = 0; x < VEC; ++x) sum.v[x] = fmaf(w.v[x], r.v[x], sum.v[x]);
+            }
+#pragma unroll
+            for (int x = 0; x < VEC; ++x) {
+                val[e].v[x] = silu_f(sum.v[x]);
+                ss = fmaf(val[e].v[x], val[e].v[x], ss);
             }
         }
         float f = 1.f;
@@ -242,21 +296,19 @@ __global__ void __launch_bounds__(DP_WARPS * 32) delta_prep_kernel(DeltaPrepArgs
             if (kind == 0) f *= rsqrtf((float)a.dim);
         }
 #pragma unroll
-        for (int e = 0; e < DP_MAX_DIM / 32; ++e) {
-            const int c = e * 32 + lane;
-            if (c < dim) out[head * dim + c] = val[e] * f;
+        for (int e = 0; e < NE; ++e) {
+            const int c = (e * 32 + lane) * VEC;
+            if (c >= dim) continue;
+#pragma unroll
+            for (int x = 0; x < VEC; ++x) val[e].v[x] *= f;
+            store_pack<VEC>(out + (int64_t)row * ldo + c, val[e]);
         }
+        if (i == sl.n - 1)  // the raw rows the next forward starts from
+            for (int t = 0; t < hist; ++t)
+                for (int c = lane * VEC; c < dim; c += 32 * VEC)
+                    store_pack<VEC>(a.tail + ((int64_t)sl.out * hist + t) * channels + ch0 + c,
+                                    raw_pack<VEC>(a, sl, i - hist + 1 + t, ch0 + c, y0 + c, channels));
     }
-    for (int h = threadIdx.x; h < a.heads; h += DP_WARPS * 32) {
-        a.beta[row * a.heads + h] = sigmoid_f(a.y.at(row, a.b_col + h));
-        a.decay[row * a.heads + h] = recurrent::gated_delta_decay(a.y.at(row, a.a_col + h), a.dt_bias[h], a.log_decay[h]);
-    }
-    if (row == last)
-        for (int t = 0; t < a.taps - 1; ++t)
-            for (int ch = threadIdx.x; ch < channels; ch += DP_WARPS * 32) {
-                const int y_col = ch < kw ? a.q_col + ch : (ch < 2 * kw ? a.k_col + ch - kw : a.v_col + ch - 2 * kw);
-                a.tail[((int64_t)half.y * (a.taps - 1) + t) * channels + ch] = raw_value(a, first, i - (a.taps - 2) + t, half.x, ch, y_col, channels);
-            }
 }
 
 // ------------------------------------------------------------------------------------------------ gates
@@ -371,18 +423,19 @@ void launch_row_update(const RowUpdateArgs& a, cudaStream_t s) {
 
 void launch_wkv_decay(const Shares& low, int low_col, int rows, int rank, int channels, const float* w2t, const float* w0, float* decay, cudaStream_t s) {
     if (rows <= 0) return;
-    const size_t smem = (size_t)rank * WD_ROWS * 4;
-    if (smem > (size_t)200 * 1024) throw std::runtime_error("launch_wkv_decay: the low rank is too large");
-    ensure_dynamic_smem(reinterpret_cast<const void*>(&wkv_decay_kernel), smem);
-    const dim3 grid((unsigned)((channels + WD_THREADS - 1) / WD_THREADS), (unsigned)((rows + WD_ROWS - 1) / WD_ROWS));
-    launch_pdl(wkv_decay_kernel, grid, dim3(WD_THREADS), smem, s, low, low_col, rows, rank, channels, w2t, w0, decay);
-    MK_LAUNCH_CHECK();
+    if (rows > 256) launch_decay_rows<32>(low, low_col, rows, rank, channels, w2t, w0, decay, s);
+    else launch_decay_rows<8>(low, low_col, rows, rank, channels, w2t, w0, decay, s);
 }
 
 void launch_delta_prep(const DeltaPrepArgs& a, cudaStream_t s) {
     if (a.rows <= 0) return;
     if (a.dim > DP_MAX_DIM || a.vdim > DP_MAX_DIM) throw std::runtime_error("launch_delta_prep: head dimensions above 256 are not supported");
-    launch_pdl(delta_prep_kernel, dim3((unsigned)a.rows), dim3(DP_WARPS * 32), 0, s, a);
+    bool vec = a.dim % 4 == 0 && a.vdim % 4 == 0 && a.y.ld % 4 == 0 && a.y.stride % 4 == 0 && (reinterpret_cast<uintptr_t>(a.y.p) & 15) == 0;
+    for (int c : {a.q_col, a.k_col, a.v_col}) vec = vec && c % 4 == 0;
+    const int run = a.rows > 256 ? DP_ROWS : 1;
+    const dim3 grid((unsigned)((a.rows + run - 1) / run), (unsigned)((2 * a.kv_heads + a.heads + DP_WARPS - 1) / DP_WARPS));
+    if (vec) launch_pdl(delta_prep_kernel<4>, grid, dim3(DP_WARPS * 32), 0, s, a, run);
+    else launch_pdl(delta_prep_kernel<1>, grid, dim3(DP_WARPS * 32), 0, s, a, run);
     MK_LAUNCH_CHECK();
 }
 

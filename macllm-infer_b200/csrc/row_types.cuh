@@ -16,12 +16,14 @@ struct Shares {
     __device__ __forceinline__ float at(int64_t row, int col) const {
         const float* q = p + row * ld + col;
         float v = *q;
+#pragma unroll 4
         for (int s = 1; s < n; ++s) v += q[s * stride];
         return v;
     }
     __device__ __forceinline__ float4 at4(int64_t row, int col) const {  // col, ld and stride multiples of 4
         const float* q = p + row * ld + col;
         float4 v = *reinterpret_cast<const float4*>(q);
+#pragma unroll 4
         for (int s = 1; s < n; ++s) {
             const float4 w = *reinterpret_cast<const float4*>(q + s * stride);
             v.x += w.x; v.y += w.y; v.z += w.z; v.w += w.w;
@@ -54,11 +56,20 @@ struct RowImage {
 #endif
 };
 
-// The recurrent state of a tick's lanes: per lane the slot half to read (-1: zeros) and the slot half to write.
+// A tick's lanes as the recurrent kernels see them: the slot half to read (-1: zeros), the half to write, and the packed rows.
+// Staged by the host, so a kernel may read it before its predecessor has finished.
+struct StateLane {
+    int32_t in, out, first, n;
+};
 struct StateLanes {
-    const int32_t* cu = nullptr;   // [lanes + 1] packed row ranges
-    const int2* halves = nullptr;  // [lanes] (read, write)
+    const StateLane* lane = nullptr;  // [lanes], 16-byte aligned
     int lanes = 0;
+#ifdef __CUDACC__
+    __device__ __forceinline__ StateLane at(int i) const {
+        const int4 v = reinterpret_cast<const int4*>(lane)[i];
+        return StateLane{v.x, v.y, v.z, v.w};
+    }
+#endif
 };
 
 #ifdef __CUDACC__
