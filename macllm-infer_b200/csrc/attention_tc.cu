@@ -50,12 +50,19 @@ __device__ __forceinline__ uint32_t pack_half2(float x, float y) {
     return *reinterpret_cast<uint32_t*>(&h);
 }
 
+// What f16 rounding left of two attention weights, as f16 numbers themselves.
+__device__ __forceinline__ uint32_t pack_half2_rest(float x, float y, uint32_t rounded) {
+    const float2 r = __half22float2(*reinterpret_cast<const __half2*>(&rounded));
+    return pack_half2(x - r.x, y - r.y);
+}
+
 // One CTA.  D = head_dim, WARPS warps of 16 items each, KT keys per shared-memory tile.
 // SPLIT = false: work item = tiles[blockIdx.x] = (lane, first query row); the CTA walks every visible key
 //                and writes normalised outputs.
 // SPLIT = true : work item = entries[blockIdx.x] = (lane, split, n_splits) of a one-token lane; the CTA walks
 //                its share of the keys and writes an unnormalised partial.
-template <int D, int WARPS, int KT, bool SPLIT>
+// EXACT: the attention weights are split into two f16 operands, so that they reach the product with V in (nearly) f32.
+template <int D, int WARPS, int KT, bool SPLIT, bool EXACT>
 __global__ void __launch_bounds__(WARPS * 32) attn_tc_kernel(AttnTcArgs a) {
     constexpr int DP = D + 8;              // padded row (halves): conflict-free ldmatrix
     constexpr int M = 16 * WARPS;
@@ -241,12 +248,20 @@ __global__ void __launch_bounds__(WARPS * 32) attn_tc_kernel(AttnTcArgs a) {
         for (int kk = 0; kk < KT / 16; ++kk) {
             uint32_t pf[4] = {pack_half2(s[2 * kk][0], s[2 * kk][1]), pack_half2(s[2 * kk][2], s[2 * kk][3]),
                               pack_half2(s[2 * kk + 1][0], s[2 * kk + 1][1]), pack_half2(s[2 * kk + 1][2], s[2 * kk + 1][3])};
+            uint32_t pr[4];
+            if constexpr (EXACT)
+#pragma unroll
+                for (int i = 0; i < 4; ++i) pr[i] = pack_half2_rest(s[2 * kk + (i >> 1)][(i & 1) * 2], s[2 * kk + (i >> 1)][(i & 1) * 2 + 1], pf[i]);
 #pragma unroll
             for (int j = 0; j < NT_O; j += 2) {
                 uint32_t bf[4];
                 ldmatrix_x4_trans(bf, vt + (kk * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * DP + j * 8 + (lane >> 4) * 8);
                 mma16816(o_acc[j], pf, bf[0], bf[1]);
                 mma16816(o_acc[j + 1], pf, bf[2], bf[3]);
+                if constexpr (EXACT) {
+                    mma16816(o_acc[j], pr, bf[0], bf[1]);
+                    mma16816(o_acc[j + 1], pr, bf[2], bf[3]);
+                }
             }
         }
         __syncthreads();
@@ -298,7 +313,7 @@ __global__ void __launch_bounds__(WARPS * 32) attn_tc_kernel(AttnTcArgs a) {
 // partial, and the CTA that arrives last at the lane's counter merges the shares.
 // LOW8: at most eight query heads per KV head, so rows 8-15 of the A operand are zero and everything that concerns
 // them (half of the softmax and of the accumulator rescaling) is skipped.
-template <int D, int STAGES, bool LOW8>
+template <int D, int STAGES, bool LOW8, bool EXACT>
 __global__ void __launch_bounds__(128) attn_decode_kernel(AttnTcArgs a) {
     constexpr int NH = LOW8 ? 1 : 2;  // accumulator row halves that can hold live rows
     constexpr int DP = D + 8;
@@ -506,12 +521,21 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(AttnTcArgs a) {
         }
         uint32_t pf[4] = {pack_half2(sc[0][0], sc[0][1]), LOW8 ? 0u : pack_half2(sc[0][2], sc[0][3]), pack_half2(sc[1][0], sc[1][1]),
                           LOW8 ? 0u : pack_half2(sc[1][2], sc[1][3])};
+        uint32_t pr[4] = {0u, 0u, 0u, 0u};
+        if constexpr (EXACT)
+#pragma unroll
+            for (int i = 0; i < 4; ++i)
+                if (!LOW8 || (i & 1) == 0) pr[i] = pack_half2_rest(sc[i >> 1][(i & 1) * 2], sc[i >> 1][(i & 1) * 2 + 1], pf[i]);
 #pragma unroll
         for (int j = 0; j < NT_O; j += 2) {
             uint32_t bf[4];
             ldmatrix_x4_trans(bf, vt + ((lane & 7) + ((lane >> 3) & 1) * 8) * DP + j * 8 + (lane >> 4) * 8);
             mma16816(o_acc[j], pf, bf[0], bf[1]);
             mma16816(o_acc[j + 1], pf, bf[2], bf[3]);
+            if constexpr (EXACT) {
+                mma16816(o_acc[j], pr, bf[0], bf[1]);
+                mma16816(o_acc[j + 1], pr, bf[2], bf[3]);
+            }
         }
         __syncwarp();  // the stage is refilled by the next iteration's load
     }
@@ -665,29 +689,29 @@ __global__ void attn_combine_kernel(AttnTcArgs a, int D) {
     }
 }
 
-template <int D, int WARPS, int KT, bool SPLIT>
+template <int D, int WARPS, int KT, bool SPLIT, bool EXACT>
 void launch_variant(const AttnTcArgs& a, int n_work, cudaStream_t s) {
     constexpr size_t smem = (size_t)(16 * WARPS + 4 * KT) * (D + 8) * sizeof(__half);
-    ensure_dynamic_smem(reinterpret_cast<const void*>(&attn_tc_kernel<D, WARPS, KT, SPLIT>), smem);
+    ensure_dynamic_smem(reinterpret_cast<const void*>(&attn_tc_kernel<D, WARPS, KT, SPLIT, EXACT>), smem);
     dim3 grid((unsigned)n_work, (unsigned)a.kv_heads);
-    launch_pdl(attn_tc_kernel<D, WARPS, KT, SPLIT>, grid, dim3(WARPS * 32), smem, s, a);
+    launch_pdl(attn_tc_kernel<D, WARPS, KT, SPLIT, EXACT>, grid, dim3(WARPS * 32), smem, s, a);
     MK_LAUNCH_CHECK();
 }
 
-template <int D>
+template <int D, bool EXACT>
 void launch_for_dim(const AttnTcArgs& a, int warps, cudaStream_t s) {
     if (a.n_tiles > 0) {
-        if (warps == 8) launch_variant<D, 8, 64, false>(a, a.n_tiles, s);
-        else launch_variant<D, 4, 32, false>(a, a.n_tiles, s);  // 32-key tiles: half the shared memory, twice the CTAs per SM (measured +0.4 % on the whole benchmark)
+        if (warps == 8) launch_variant<D, 8, 64, false, EXACT>(a, a.n_tiles, s);
+        else launch_variant<D, 4, 32, false, EXACT>(a, a.n_tiles, s);  // 32-key tiles: half the shared memory, twice the CTAs per SM (measured +0.4 % on the whole benchmark)
     }
     if (a.n_entries > 0) {
         constexpr int STAGES = D >= 256 ? 2 : 3;
         constexpr size_t smem = (size_t)(16 + 4 * STAGES * 2 * 16) * (D + 8) * sizeof(__half);
-        ensure_dynamic_smem(reinterpret_cast<const void*>(&attn_decode_kernel<D, STAGES, true>), smem);
-        ensure_dynamic_smem(reinterpret_cast<const void*>(&attn_decode_kernel<D, STAGES, false>), smem);
+        ensure_dynamic_smem(reinterpret_cast<const void*>(&attn_decode_kernel<D, STAGES, true, EXACT>), smem);
+        ensure_dynamic_smem(reinterpret_cast<const void*>(&attn_decode_kernel<D, STAGES, false, EXACT>), smem);
         dim3 grid((unsigned)a.n_entries, (unsigned)a.kv_heads);
-        if (a.q_heads / a.kv_heads <= 8) launch_pdl(attn_decode_kernel<D, STAGES, true>, grid, dim3(128), smem, s, a);
-        else launch_pdl(attn_decode_kernel<D, STAGES, false>, grid, dim3(128), smem, s, a);
+        if (a.q_heads / a.kv_heads <= 8) launch_pdl(attn_decode_kernel<D, STAGES, true, EXACT>, grid, dim3(128), smem, s, a);
+        else launch_pdl(attn_decode_kernel<D, STAGES, false, EXACT>, grid, dim3(128), smem, s, a);
         MK_LAUNCH_CHECK();
     }
     if (a.n_dec_lanes > 0) {  // lanes whose keys were shared out over several CTAs
@@ -770,9 +794,9 @@ int launch_paged_attention_tc(const AttnTcArgs& a_in, cudaStream_t s) {
     while ((1 << a.bt_shift) < a.block_tokens) ++a.bt_shift;
     int warps = attention_tc_warps(a.q_heads, a.kv_heads);
     switch (a.d) {
-        case 64: launch_for_dim<64>(a, warps, s); break;
-        case 128: launch_for_dim<128>(a, warps, s); break;
-        case 256: launch_for_dim<256>(a, warps, s); break;
+        case 64: a.exact_weights ? launch_for_dim<64, true>(a, warps, s) : launch_for_dim<64, false>(a, warps, s); break;
+        case 128: a.exact_weights ? launch_for_dim<128, true>(a, warps, s) : launch_for_dim<128, false>(a, warps, s); break;
+        case 256: a.exact_weights ? launch_for_dim<256, true>(a, warps, s) : launch_for_dim<256, false>(a, warps, s); break;
         default: throw std::runtime_error("launch_paged_attention_tc: unsupported head_dim");
     }
     return (a.n_tiles > 0 ? 1 : 0) + (a.n_entries > 0 ? 1 : 0) + (a.n_dec_lanes > 0 ? 1 : 0);

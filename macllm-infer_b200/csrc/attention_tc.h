@@ -41,6 +41,8 @@ struct AttnTcArgs {
     int bt_shift = 0;         // log2(block_tokens), filled in by the launcher
     float scale = 1.f, softcap = 0.f;
     int window = 0;
+    // attention weights enter the product with V as the sum of two f16 numbers (about 22 bits) instead of one
+    int exact_weights = 0;
 };
 
 // f16 pools, head_dim 64/128/256, 1/2/4/8 query heads per KV head, block_tokens a power of two >= 16.

@@ -546,6 +546,7 @@ void MixerLm::run_parallel(const Tick& t, int l, Pending& pend, const std::vecto
         ta.layers = 1;
         ta.pool_blocks = ra.pool_blocks;
         ta.scale = s.scale;
+        ta.exact_weights = 1;
         if (fuse_rope) {
             ta.fused_rope = 1;
             ta.rk = ra;
