@@ -48,8 +48,9 @@ MK_HD uint64_t rank_key(float value, uint32_t index) {
 }
 MK_HD uint32_t rank_key_index(uint64_t k) { return 0xFFFFFFFFu - (uint32_t)(k & 0xFFFFFFFFull); }
 
-// exp(x) for x <= 0 (softmax numerators): n = round(x log2 e), r = x - n ln 2 in two fused steps, a degree-6 polynomial
-// in r, then scaling by 2^n through the exponent field (in two exact steps when the result is subnormal).  About 1 ulp
+// exp(x) for x <= 0 (softmax numerators): n = round(x log2 e), r = x - n ln 2 in two fused steps (the argument reduction of
+// W. J. Cody and W. Waite, "Software Manual for the Elementary Functions": ln 2 as 45426 / 65536 plus the rest), the Taylor
+// polynomial of degree 6 in r, then scaling by 2^n through the exponent field (in two exact steps when the result is subnormal).  About 1 ulp
 // from exp; the same bits on the host and on the device.  x below -104 (and -inf) gives 0, x > 0 is treated as 0.
 MK_HD float det_expf(float x) {
     if (!(x > -104.0f)) return 0.0f;  // also NaN
