@@ -216,12 +216,14 @@ def run(peaks: dict, warmup: int, steps: int, prompt=2048, lanes=64, context=102
                 if kind == "sizilorn":
                     path = write_checkpoint(Path(tmp) / s.name, s)
                     model = engine.Model.load(path, state_slots=lanes + 1, **kw)
+                    weights = model.spec().weight_bytes_per_token
                 else:
                     path = seed_gguf.write_seed_gguf(Path(tmp) / f"{s.name}.gguf", closest_spec(s), seed=0)
                     model = engine.Model.load(path, **kw)
+                    weights = seed_gguf.weight_bytes(closest_spec(s))["per_token"]
                 r = measure(model, s.vocab, prompt, lanes, context, warmup, steps, peaks)
                 sp = model.spec()
                 results.append(dict(shape=s.name, model="Sizilorn" if kind == "sizilorn" else "qwen3 family, dense BF16 matrices", layers=int(sp.n_layers),
-                                    width=int(sp.hidden_size), weight_gb=round(sp.weight_bytes_per_token / 1e9, 3), **r))
+                                    width=int(sp.hidden_size), weight_gb=round(weights / 1e9, 3), **r))
                 model.close()
     return results
