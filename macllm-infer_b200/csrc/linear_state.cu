@@ -337,6 +337,33 @@ __global__ void __launch_bounds__(128) head_norm_gate_kernel(LinearStateArgs a, 
                     a.norm_w + (a.norm_per_head ? head * a.vdim : 0), row, head, threadIdx.x & 31);
 }
 
+// The same with four values per thread and G threads per head row (vdim a multiple of 4, at most 4 G): narrow heads share a warp.
+template <int G>
+__global__ void __launch_bounds__(128) head_norm_gate_vec_kernel(LinearStateArgs a, int rows) {
+    pdl_trigger();
+    pdl_wait();
+    const int64_t i = (int64_t)blockIdx.x * (128 / G) + threadIdx.x / G;
+    const bool live = i < (int64_t)rows * a.heads;
+    const int64_t row = live ? i / a.heads : 0;
+    const int head = live ? (int)(i % a.heads) : 0, v = (int)(threadIdx.x % G) * 4;
+    const bool mine = live && v < a.vdim;
+    float4 o = make_float4(0.f, 0.f, 0.f, 0.f), g = o, w = o;
+    if (mine) {
+        o = *reinterpret_cast<const float4*>(a.out + row * a.heads * a.vdim + head * a.vdim + v);
+        g = a.gate.at4(row, a.gate_col + head * a.vdim + v);
+        w = *reinterpret_cast<const float4*>(a.norm_w + (a.norm_per_head ? head * a.vdim : 0) + v);
+    }
+    float ss = o.x * o.x + o.y * o.y + o.z * o.z + o.w * o.w;
+#pragma unroll
+    for (int x = 1; x < G; x <<= 1) ss += __shfl_xor_sync(0xffffffffu, ss, x);
+    const float root = sqrtf(ss / (float)a.vdim + a.eps);
+    if (mine)
+        a.image.put4(row, head * a.vdim + v, make_float4(o.x / root * w.x * silu_f(g.x), o.y / root * w.y * silu_f(g.y), o.z / root * w.z * silu_f(g.z),
+                                                         o.w / root * w.w * silu_f(g.w)));
+    if (live && head == a.heads - 1)
+        for (int c = a.heads * a.vdim + (int)(threadIdx.x % G); c < a.image.ld; c += G) a.image.put(row, c, 0.f);
+}
+
 template <int KD, bool WKV, bool FINISH>
 void launch_variant(const WkvScanArgs& wa, const DeltaScanArgs& da, cudaStream_t s) {
     const LinearStateArgs& a = WKV ? wa.common : da.common;
@@ -386,7 +413,11 @@ void launch_delta_scan(const DeltaScanArgs& a, cudaStream_t s) {
 void launch_head_norm_gate(const LinearStateArgs& a, int rows, cudaStream_t s) {
     if (rows <= 0) return;
     const int64_t items = (int64_t)rows * a.heads;
-    launch_pdl(head_norm_gate_kernel, dim3((unsigned)((items + 3) / 4)), dim3(128), 0, s, a, rows);
+    const bool vec = a.vdim % 4 == 0 && a.vdim <= 128 && a.gate_col % 4 == 0 && a.gate.ld % 4 == 0 && a.gate.stride % 4 == 0 &&
+                     (reinterpret_cast<uintptr_t>(a.gate.p) & 15) == 0;
+    if (vec && a.vdim <= 64) launch_pdl(head_norm_gate_vec_kernel<16>, dim3((unsigned)((items + 7) / 8)), dim3(128), 0, s, a, rows);
+    else if (vec) launch_pdl(head_norm_gate_vec_kernel<32>, dim3((unsigned)((items + 3) / 4)), dim3(128), 0, s, a, rows);
+    else launch_pdl(head_norm_gate_kernel, dim3((unsigned)((items + 3) / 4)), dim3(128), 0, s, a, rows);
     MK_LAUNCH_CHECK();
 }
 

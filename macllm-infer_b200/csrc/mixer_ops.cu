@@ -321,6 +321,19 @@ __global__ void __launch_bounds__(256) head_gate_kernel(const float* attn, int h
     for (int h = threadIdx.x; h < heads; h += blockDim.x) hg_gate[h] = sigmoid_f(gate.at(row, gate_col + h));
     __syncthreads();
     const float* src = attn + row * heads * row_width;
+    if ((vdim & 3) == 0) {  // out.ld is a multiple of 64, a head's row of 4
+        for (int c = threadIdx.x * 4; c < out.ld; c += blockDim.x * 4) {
+            const int h = c / vdim;
+            float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (h < heads) {
+                v = *reinterpret_cast<const float4*>(src + h * row_width + (c - h * vdim));
+                const float g = hg_gate[h];
+                v = make_float4(v.x * g, v.y * g, v.z * g, v.w * g);
+            }
+            out.put4(row, c, v);
+        }
+        return;
+    }
     for (int c = threadIdx.x; c < out.ld; c += blockDim.x) {
         const int h = c / vdim;
         out.put(row, c, h < heads ? src[h * row_width + (c - h * vdim)] * hg_gate[h] : 0.f);
