@@ -169,7 +169,9 @@ int32_t mk_gguf_inspect(const char* path, mk_gguf_summary* out);
 typedef struct mk_mixer_summary {
     char architecture[32];
     int32_t vocab_size, hidden_size, n_layers;
-    int32_t wkv_layers, parallel_layers, ffn_layers, side_dim, reserved_;
+    int32_t wkv_layers, parallel_layers, ffn_layers, side_dim;
+    int32_t latent_layers, mingru_layers;
+    int32_t layer_runs; /* executions of a layer per forward: a looped layer counts once per pass */
     int64_t tensors_in_file, tensors_read, parameters;
 } mk_mixer_summary;
 int32_t mk_mixer_inspect(const char* dir, mk_mixer_summary* out);

@@ -49,7 +49,7 @@ class GgufSummary(C.Structure):
 class MixerSummary(C.Structure):
     _fields_ = [("architecture", C.c_char * 32), ("vocab_size", C.c_int32), ("hidden_size", C.c_int32), ("n_layers", C.c_int32),
                 ("wkv_layers", C.c_int32), ("parallel_layers", C.c_int32), ("ffn_layers", C.c_int32), ("side_dim", C.c_int32),
-                ("reserved_", C.c_int32), ("tensors_in_file", C.c_int64), ("tensors_read", C.c_int64), ("parameters", C.c_int64)]
+                ("latent_layers", C.c_int32), ("mingru_layers", C.c_int32), ("layer_runs", C.c_int32), ("tensors_in_file", C.c_int64), ("tensors_read", C.c_int64), ("parameters", C.c_int64)]
 
 
 class RuntimeSpec(C.Structure):

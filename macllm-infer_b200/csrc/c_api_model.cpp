@@ -108,10 +108,16 @@ int32_t mk_mixer_inspect(const char* dir, mk_mixer_summary* out) {
         out->hidden_size = s.width;
         out->n_layers = (int32_t)s.layers.size();
         for (const MixerLayerSpec& l : s.layers) {
-            (l.kind == MixerKind::Wkv ? out->wkv_layers : out->parallel_layers)++;
+            switch (l.kind) {
+                case MixerKind::Wkv: ++out->wkv_layers; break;
+                case MixerKind::Parallel: ++out->parallel_layers; break;
+                case MixerKind::Latent: ++out->latent_layers; break;
+                case MixerKind::MinGru: ++out->mingru_layers; break;
+            }
             out->ffn_layers += l.ff > 0 ? 1 : 0;
         }
         out->side_dim = s.side_dim;
+        out->layer_runs = (int32_t)s.runs().size();
         out->tensors_in_file = a.tensors_in_file;
         out->tensors_read = a.tensors_read;
         out->parameters = a.parameters;

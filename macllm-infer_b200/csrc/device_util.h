@@ -1,6 +1,7 @@
 // Small RAII helpers for device and pinned host memory.
 #pragma once
 #include "common.cuh"
+#include <cuda_bf16.h>
 #include <vector>
 
 namespace mk {
@@ -63,6 +64,35 @@ private:
 
 constexpr int kMaxRowGroups = 8;
 
+// Where a matmul leaves its result when not as rows y[t][n]: the weight rows are cut into parts of `part_rows`, of which the
+// first `part_valid` count; value (t, part p, row i of the part) goes to
+//   out[p * ld_part + (t' >> block_shift) * ld_block + (t' & (2^block_shift - 1)) * ld_row + i],  t' = row_map ? row_map[t] : t.
+struct MatmulScatter {
+    enum Type : int { F32 = 0, F16 = 1, BF16 = 2 };
+    void* out = nullptr;
+    int type = F32;
+    int part_rows = 0, part_valid = 0;
+    int64_t ld_part = 0, ld_row = 0, ld_block = 0;
+    int block_shift = 31;
+    const int32_t* row_map = nullptr;
+#ifdef __CUDACC__
+    // Offset of weight row n's values, or -1 when they are not kept.
+    __device__ __forceinline__ int64_t column(int64_t n) const {
+        const int64_t p = n / part_rows, i = n - p * part_rows;
+        return i < part_valid ? p * ld_part + i : -1;
+    }
+    __device__ __forceinline__ int64_t row(int t) const {
+        if (row_map != nullptr) t = row_map[t];
+        return (int64_t)(t >> block_shift) * ld_block + (int64_t)(t & (int)((1u << block_shift) - 1u)) * ld_row;
+    }
+    __device__ __forceinline__ void put(int64_t at, float v) const {
+        if (type == F32) static_cast<float*>(out)[at] = v;
+        else if (type == F16) static_cast<__half*>(out)[at] = __float2half_rn(v);
+        else static_cast<__nv_bfloat16*>(out)[at] = __float2bfloat16_rn(v);
+    }
+#endif
+};
+
 // The 16-bit image of one weight matrix [rows][cols] plus the TMA descriptor of its 128-row x 64-column
 // boxes (see hgemm_tc.h).  Built once at load time: f16 from the device copy of a quantised matrix, bf16 from a dense
 // checkpoint.
@@ -74,6 +104,7 @@ struct HalfWeight {
     // input g.  The inputs lie one after the other, T rows each.  One group: the usual case.
     int n_groups = 1;
     int group_end[kMaxRowGroups] = {};
+    int group_tiles = 0;         // > 0: any number of groups, all of this many row tiles (group_end is not read)
     alignas(64) unsigned char tmap[128] = {};  // CUtensorMap (opaque here, 64-byte aligned)
     bool ready = false;
 };

@@ -188,10 +188,14 @@ struct HgParams {
     // stacked projections with inputs of their own: the first row of input g in the activation matrix is g * T
     int n_groups;
     int group_end[kMaxRowGroups];
+    int group_tiles;
+    int scattered;  // the result goes where `scatter` says (splits == 1)
+    MatmulScatter scatter;
 };
 
 __device__ __forceinline__ int group_row0(const HgParams& p, int m_tile) {
     if (p.n_groups == 1) return 0;
+    if (p.group_tiles > 0) return m_tile / p.group_tiles * p.T;
     int g = 0;
     while (g < p.n_groups - 1 && m_tile >= p.group_end[g]) ++g;
     return g * p.T;
@@ -407,6 +411,15 @@ hgemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant_
                             else p.yh[(int64_t)tok * p.ldyh + feature] = __float2half_rn(a * u);
                         }
                     }
+                } else if (p.scattered != 0) {
+                    const int64_t col = row < p.rows ? p.scatter.column(row) : -1;
+                    if (col >= 0) {
+#pragma unroll
+                        for (int i = 0; i < 32; ++i) {
+                            const int tok = tok0 + cb + i;
+                            if (tok < p.T) p.scatter.put(p.scatter.row(tok) + col, __uint_as_float(r[i]));
+                        }
+                    }
                 } else if (row < p.rows) {
 #pragma unroll
                     for (int i = 0; i < 32; ++i) {
@@ -568,6 +581,14 @@ void build_bf16_weight(const float* values, int64_t rows, int64_t cols, HalfWeig
     out.ready = true;
 }
 
+void build_bf16_weight_groups(const float* values, int64_t rows, int64_t cols, int groups, HalfWeight& out, cudaStream_t s) {
+    if (groups <= 0 || rows % groups != 0 || rows / groups % HG_BM != 0)
+        throw std::runtime_error("build_bf16_weight_groups: every stacked projection must be a multiple of 128 rows");
+    build_bf16_weight(values, rows, cols, out, s);
+    out.n_groups = groups;
+    out.group_tiles = (int)(rows / groups / HG_BM);
+}
+
 void build_half_weight(const QWeight& W, HalfWeight& out, cudaStream_t s) {
     const QWeight* one = &W;
     build_half_weight_stacked(&one, 1, out, s);
@@ -609,12 +630,18 @@ HgemmPlan hgemm_tc_plan(int64_t rows, int64_t cols, int T, int max_splits) {
 
 namespace {
 int launch_hgemm_any(const HalfWeight& W, const __half* xh, int T, float* y, int ldy, float out_scale, float softcap,
-                     const HgemmScratch& ws, cudaStream_t s, int max_splits, int gated, __half* yh, int ldyh);
+                     const HgemmScratch& ws, cudaStream_t s, int max_splits, int gated, __half* yh, int ldyh,
+                     const MatmulScatter* scatter = nullptr);
 }
 
 int launch_hgemm_tc(const HalfWeight& W, const __half* xh, int T, float* y, int ldy, float out_scale, float softcap,
                     const HgemmScratch& ws, cudaStream_t s, int max_splits) {
     return launch_hgemm_any(W, xh, T, y, ldy, out_scale, softcap, ws, s, max_splits, 0, nullptr, 0);
+}
+
+void launch_hgemm_tc_scatter(const HalfWeight& W, const __half* xh, int T, const MatmulScatter& to, const HgemmScratch& ws, cudaStream_t s) {
+    if (to.out == nullptr || to.part_rows <= 0) throw std::runtime_error("launch_hgemm_tc_scatter: no destination");
+    launch_hgemm_any(W, xh, T, nullptr, 0, 1.0f, 0.f, ws, s, 1, 0, nullptr, 0, &to);
 }
 
 void launch_hgemm_tc_gated(const HalfWeight& W, const __half* xh, int T, int act, __half* yh, int ldyh, const HgemmScratch& ws,
@@ -625,7 +652,8 @@ void launch_hgemm_tc_gated(const HalfWeight& W, const __half* xh, int T, int act
 
 namespace {
 int launch_hgemm_any(const HalfWeight& W, const __half* xh, int T, float* y, int ldy, float out_scale, float softcap,
-                     const HgemmScratch& ws, cudaStream_t s, int max_splits, int gated, __half* yh, int ldyh) {
+                     const HgemmScratch& ws, cudaStream_t s, int max_splits, int gated, __half* yh, int ldyh,
+                     const MatmulScatter* scatter) {
     if (T <= 0) return 1;
     if (!W.ready) throw std::runtime_error("launch_hgemm_tc: the f16 image of the matrix was not built");
     if (xh == nullptr) throw std::runtime_error("launch_hgemm_tc: f16 activations missing");
@@ -657,6 +685,9 @@ int launch_hgemm_any(const HalfWeight& W, const __half* xh, int T, float* y, int
     p.bf16 = W.bf16 ? 1 : 0;
     p.n_groups = W.n_groups;
     for (int g = 0; g < kMaxRowGroups; ++g) p.group_end[g] = W.group_end[g];
+    p.group_tiles = W.group_tiles;
+    p.scattered = scatter != nullptr ? 1 : 0;
+    if (scatter != nullptr) p.scatter = *scatter;
     const int grid = std::min(device_sm_count(), p.row_tiles * p.n_tiles * p.splits);
     const CUtensorMap& tw = *reinterpret_cast<const CUtensorMap*>(W.tmap);
     if (pl.bn == 256) launch_hg<256, 4>(tw, tx, p, grid, s);

@@ -32,6 +32,8 @@ void build_half_weight_interleaved(const QWeight& gate, const QWeight& up, HalfW
 // `group_rows` (optional): rows of each stacked projection with an input of its own, multiples of 128 (see HalfWeight).
 void build_bf16_weight(const float* values, int64_t rows, int64_t cols, HalfWeight& out, cudaStream_t s,
                        const std::vector<int64_t>& group_rows = {});
+// The same with `groups` stacked projections of rows / groups rows each (a multiple of 128), every one with an input of its own.
+void build_bf16_weight_groups(const float* values, int64_t rows, int64_t cols, int groups, HalfWeight& out, cudaStream_t s);
 
 // How a call is cut into work items (see hgemm_tc.cu); partial_floats is the scratch a split call needs.
 struct HgemmPlan {
@@ -55,6 +57,9 @@ struct HgemmScratch {
 // partial sums at ws.partial[(s * T + t) * rows + n] and the consumer adds them for s = 0 .. S-1 in that order.
 int launch_hgemm_tc(const HalfWeight& W, const __half* xh, int T, float* y, int ldy, float out_scale, float softcap,
                     const HgemmScratch& ws, cudaStream_t s, int max_splits = 1);
+
+// The same product with the result scattered (see MatmulScatter); never cut into K shares.
+void launch_hgemm_tc_scatter(const HalfWeight& W, const __half* xh, int T, const MatmulScatter& to, const HgemmScratch& ws, cudaStream_t s);
 
 // Gated feed-forward front half in one kernel: with W an interleaved gate/up image (2F rows),
 // yh[t][j] = f16(act(sum_k xh[t][k] gate[j][k]) * sum_k xh[t][k] up[j][k]), j < F; act 0 = SiLU, otherwise tanh GELU.

@@ -76,7 +76,7 @@ __device__ __forceinline__ void finish_head_row(const LinearStateArgs& a, const 
     const float root = sqrtf(ss / (float)a.vdim + a.eps);
     for (int v = lane; v < a.vdim; v += 32) a.image.put(row, head * a.vdim + v, o[v] / root * nw[v] * silu_f(gate(v)));
     if (head == a.heads - 1)
-        for (int c = a.heads * a.vdim + lane; c < a.image.ld; c += 32) a.image.put(row, c, 0.f);
+        for (int c = a.heads * a.vdim + lane; c < a.image.end(); c += 32) a.image.put(row, c, 0.f);
 }
 
 template <int KD, bool WKV, bool FINISH>
@@ -361,7 +361,7 @@ __global__ void __launch_bounds__(128) head_norm_gate_vec_kernel(LinearStateArgs
         a.image.put4(row, head * a.vdim + v, make_float4(o.x / root * w.x * silu_f(g.x), o.y / root * w.y * silu_f(g.y), o.z / root * w.z * silu_f(g.z),
                                                          o.w / root * w.w * silu_f(g.w)));
     if (live && head == a.heads - 1)
-        for (int c = a.heads * a.vdim + (int)(threadIdx.x % G); c < a.image.ld; c += G) a.image.put(row, c, 0.f);
+        for (int c = a.heads * a.vdim + (int)(threadIdx.x % G); c < a.image.end(); c += G) a.image.put(row, c, 0.f);
 }
 
 template <int KD, bool WKV, bool FINISH>

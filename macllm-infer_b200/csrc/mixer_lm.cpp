@@ -12,9 +12,7 @@ namespace mk {
 namespace {
 
 const std::vector<const char*> class_names = {"hgemm_tc", "hgemm_tc_splitk", "f32_matmul", "wkv_scan", "delta_scan", "paged_attention", "rope_kv_scatter",
-                                              "row_update", "delta_prep", "wkv_decay", "gates", "embed", "build_batch", "argmax"};
-
-int pad_to(int64_t n, int m) { return (int)((n + m - 1) / m * m); }
+                                              "row_update", "delta_prep", "wkv_decay", "latent_attention", "mingru_scan", "latent_prep", "latent_rows", "gates", "embed", "build_batch", "argmax"};
 
 bool is_mixer_checkpoint(const std::string& dir) {
     struct stat st;
@@ -29,13 +27,6 @@ constexpr int kShortLane = 4;  // lanes up to this many tokens: the recurrence k
 
 }  // namespace
 
-struct MixerLm::Pending {
-    int n = 0;
-    Shares y[2];
-    const float* w[2] = {nullptr, nullptr};
-    float coef = 1.f;
-};
-
 MixerLm::MixerLm(const std::string& dir, const ModelConfig& cfg) : DeviceLm(cfg, class_names) {
     const SafetensorsFile f(dir + "/model.safetensors");
     ms_ = read_mixer_spec_of(dir, f);
@@ -46,14 +37,17 @@ MixerLm::MixerLm(const std::string& dir, const ModelConfig& cfg) : DeviceLm(cfg,
     if (cfg.ep_size > 1) throw std::runtime_error("expert parallelism asked for a model without experts");
     open_device();
     spec_.vocab = ms_.vocab;
-    spec_.layers = (int)ms_.layers.size();
+    runs_ = ms_.runs();
+    spec_.layers = (int)runs_.size();
     spec_.hidden = ms_.width;
     // every layer kind of these decoders carries a recurrent state, of which a prompt prefix keeps no copy
     init_pool(cfg_.block_tokens, cfg_.slab_blocks, cfg_.kv_capacity_tokens, cfg_.prefix_capacity_tokens, "recurrent layers");
     init_state_slots(cfg_.state_slots > 0 ? cfg_.state_slots : cfg_.max_batch_lanes);
     spec_.max_context = (int)std::min<int64_t>(pool_->max_blocks() * pool_->block_tokens(), 1 << 30);
     lw_.resize(ms_.layers.size());
+    rs_.resize(runs_.size());
     load(f);
+    for (int i = 0; i < (int)runs_.size(); ++i) alloc_run(i);
     alloc_activations();
     MK_CUDA(cudaStreamSynchronize(stream_));
 }
@@ -71,33 +65,52 @@ void MixerLm::upload_f32(const std::vector<float>& v, DevBuf& out) {
 
 void MixerLm::upload_norm(const SafetensorsFile& f, const std::string& name, Norm& out) {
     upload_f32(f.values(name, {ms_.width}), out.w);
+    if (ms_.norm != NormKind::DynTanh) return;
     upload_f32(f.values(name + ".b", {ms_.width}), out.b);
     out.alpha = f.values(name + ".alpha", {}).at(0);
+}
+
+void MixerLm::place(const SafetensorsFile& f, const Part& p, int cols, int ld, std::vector<float>& m) {
+    const int n = p.cols > 0 ? p.cols : cols, block = p.block > 0 ? p.block : p.rows;
+    const std::vector<float> v = f.values(p.name, {p.rows, n});
+#pragma omp parallel for
+    for (int r = 0; r < p.rows; ++r) {
+        const int64_t row = p.at + (int64_t)(r / block) * p.pitch + (int64_t)(r % block) * p.step;
+        memcpy(&m[(size_t)(row * ld + p.col)], &v[(size_t)r * n], (size_t)n * 4);
+    }
+}
+
+void MixerLm::upload_matrix(const std::vector<float>& m, int64_t rows, int ld, int64_t true_bytes, Dense& out, const std::vector<int64_t>& group_rows,
+                            int groups, bool per_token) {
+    out.rows = rows;
+    out.ld = ld;
+    out.bytes = true_bytes;
+    out.n_groups = 1;
+    if (groups > 0) {
+        out.n_groups = groups;
+        out.group_tiles = (int)(rows / groups / 128);
+    } else if (group_rows.size() > 1) {
+        out.n_groups = (int)group_rows.size();
+        int64_t end = 0;
+        for (size_t g = 0; g < group_rows.size(); ++g) out.group_end[g] = (int)((end += group_rows[g]) / 128);
+    }
+    if (f32_) upload_f32(m, out.f32);
+    else if (groups > 0) build_bf16_weight_groups(m.data(), rows, ld, groups, out.half, stream_);
+    else build_bf16_weight(m.data(), rows, ld, out.half, stream_, group_rows);
+    spec_.weight_bytes += out.bytes;
+    if (per_token) spec_.weight_bytes_per_token += out.bytes;
 }
 
 void MixerLm::upload_dense(const SafetensorsFile& f, const std::vector<Part>& parts, int64_t rows, int cols, Dense& out,
                            const std::vector<int64_t>& group_rows) {
     const int ld = pad_to(cols, 64);
     std::vector<float> m((size_t)(rows * ld), 0.f);
-    out.bytes = 0;
+    int64_t bytes = 0;
     for (const Part& p : parts) {
-        const std::vector<float> v = f.values(p.name, {p.rows, cols});
-#pragma omp parallel for
-        for (int r = 0; r < p.rows; ++r) memcpy(&m[(size_t)(p.at + (int64_t)r * p.step) * ld], &v[(size_t)r * cols], (size_t)cols * 4);
-        out.bytes += (int64_t)p.rows * cols * esz_;
+        place(f, p, cols, ld, m);
+        bytes += (int64_t)p.rows * (p.cols > 0 ? p.cols : cols) * esz_;
     }
-    out.rows = rows;
-    out.ld = ld;
-    out.n_groups = 1;
-    if (group_rows.size() > 1) {
-        out.n_groups = (int)group_rows.size();
-        int64_t end = 0;
-        for (size_t g = 0; g < group_rows.size(); ++g) out.group_end[g] = (int)((end += group_rows[g]) / 128);
-    }
-    if (f32_) upload_f32(m, out.f32);
-    else build_bf16_weight(m.data(), rows, ld, out.half, stream_, group_rows);
-    spec_.weight_bytes += out.bytes;
-    spec_.weight_bytes_per_token += out.bytes;
+    upload_matrix(m, rows, ld, bytes, out, group_rows, 0);
 }
 
 int MixerLm::rope_table(const RotarySpec& r) {
@@ -158,6 +171,22 @@ void MixerLm::load(const SafetensorsFile& f) {
     };
     table("embed", C, embed_);
     if (ms_.side_dim > 0) table("side.embed", (int64_t)ms_.layers.size() * ms_.side_dim, side_embed_);
+    if (ms_.sinusoid_positions) {
+        upload_norm(f, "embed.norm", embed_norm_);
+        std::vector<double> freq((size_t)(C + 1) / 2);
+        for (size_t i = 0; i < freq.size(); ++i) freq[i] = std::pow(10000.0, -2.0 * (double)i / C);
+        position_freq_.upload(freq.data(), freq.size() * 8, stream_);
+        MK_CUDA(cudaStreamSynchronize(stream_));
+    }
+    if (ms_.loop.times > 0) {
+        const int second = pad_to(C, 64);  // where the embedding output's columns begin in the input of `loop.in`
+        const std::vector<float> w = f.values("loop.in", {C, 2 * C});
+        std::vector<float> m((size_t)C * 2 * second, 0.f);
+        for (int r = 0; r < C; ++r)
+            for (int h = 0; h < 2; ++h) memcpy(&m[((size_t)r * 2 + h) * second], &w[((size_t)r * 2 + h) * C], (size_t)C * 4);
+        upload_matrix(m, C, 2 * second, (int64_t)2 * C * C * esz_, loop_in_, {}, 0);
+        upload_f32(f.values("loop.step", {ms_.loop.times, C}), loop_step_);
+    }
     for (int l = 0; l < (int)ms_.layers.size(); ++l) load_layer(f, l);
     upload_norm(f, "final.norm", final_norm_);
     upload_dense(f, {{"head", ms_.vocab, 0}}, ms_.vocab, C, head_);
@@ -166,8 +195,8 @@ void MixerLm::load(const SafetensorsFile& f) {
 void MixerLm::load_layer(const SafetensorsFile& f, int l) {
     const MixerLayerSpec& s = ms_.layers[(size_t)l];
     Layer& w = lw_[(size_t)l];
+    if (ms_.side_by_side) return load_side_by_side(f, l);
     const int C = ms_.width;
-    const int64_t halves = (int64_t)state_slots_->capacity() * 2;
     const std::string p = "l" + std::to_string(l) + ".", m = p + "mix.";
     upload_norm(f, p + "norm1", w.norm1);
     if (s.kind == MixerKind::Wkv) {
@@ -194,8 +223,6 @@ void MixerLm::load_layer(const SafetensorsFile& f, int l) {
         upload_f32(f.values(m + "u", {s.wkv.heads, s.wkv.dim}), w.bonus);
         upload_f32(f.values(m + "norm", {HD}), w.head_norm);
         upload_dense(f, {{m + "o", C, 0}}, C, HD, w.out);
-        w.kept.alloc((size_t)halves * C * 4);
-        w.state.alloc((size_t)halves * HD * linear_state_key_pad(s.wkv.dim) * 4);
     } else {
         const AttentionSpec& a = s.attn;
         const DeltaSpec& d = s.delta;
@@ -229,12 +256,6 @@ void MixerLm::load_layer(const SafetensorsFile& f, int l) {
         w.geometry = geometry_of(a);
         w.row_width = geo_[(size_t)w.geometry].row_width;
         w.rope = rope_table(a.rot);
-        const int64_t page_bytes = (int64_t)a.kv_heads * cfg_.block_tokens * w.row_width * (cfg_.kv_f16 ? 2 : 4);
-        for (DevBuf* pool : {&w.k_pool, &w.v_pool}) {
-            pool->alloc((size_t)(pool_->max_blocks() * page_bytes));
-            pool->zero(stream_);
-        }
-        spec_.kv_bytes_per_token += 2 * page_bytes / cfg_.block_tokens;
         // delta rule
         const int kw = d.kv_heads * d.dim, vw = d.heads * d.vdim, channels = 2 * kw + vw;
         if (d.dim > 256 || d.vdim > 256) throw std::runtime_error("delta-rule head dimensions above 256 are not supported");
@@ -252,8 +273,6 @@ void MixerLm::load_layer(const SafetensorsFile& f, int l) {
         for (float& v : decay) v = (float)-std::exp((double)v);
         upload_f32(decay, w.log_decay);
         upload_f32(f.values(Rt + "norm", {d.vdim}), w.head_norm);
-        w.tail.alloc((size_t)halves * std::max(1, d.taps - 1) * channels * 4);
-        w.state.alloc((size_t)halves * vw * linear_state_key_pad(d.dim) * 4);
     }
     if (s.ff > 0) {
         upload_norm(f, p + "norm2", w.norm2);
@@ -267,14 +286,62 @@ void MixerLm::load_layer(const SafetensorsFile& f, int l) {
     }
 }
 
+void MixerLm::alloc_run(int run) {
+    const int l = runs_[(size_t)run].layer;
+    const MixerLayerSpec& s = ms_.layers[(size_t)l];
+    const Layer& w = lw_[(size_t)l];
+    RunState& st = rs_[(size_t)run];
+    const size_t halves = (size_t)state_slots_->capacity() * 2;
+    auto pages = [&](DevBuf& pool, int kv_heads) {
+        const int64_t bytes = (int64_t)kv_heads * cfg_.block_tokens * w.row_width * (cfg_.kv_f16 ? 2 : 4);
+        pool.alloc((size_t)(pool_->max_blocks() * bytes));
+        pool.zero(stream_);
+        spec_.kv_bytes_per_token += bytes / cfg_.block_tokens;
+    };
+    if (s.kind == MixerKind::Wkv || ms_.side_by_side) st.kept.alloc(halves * (size_t)ms_.width * 4);  // the token shift's row
+    switch (s.kind) {
+        case MixerKind::Wkv:
+            st.state.alloc(halves * (size_t)s.wkv.heads * s.wkv.dim * linear_state_key_pad(s.wkv.dim) * 4);
+            break;
+        case MixerKind::Parallel: {
+            pages(st.k_pool, s.attn.kv_heads);
+            pages(st.v_pool, s.attn.kv_heads);
+            const DeltaSpec& d = s.delta;
+            st.tail.alloc(halves * (size_t)std::max(1, d.taps - 1) * (2 * (size_t)d.kv_heads * d.dim + (size_t)d.heads * d.vdim) * 4);
+            st.state.alloc(halves * (size_t)d.heads * d.vdim * linear_state_key_pad(d.dim) * 4);
+            break;
+        }
+        case MixerKind::Latent: pages(st.k_pool, 1); break;
+        case MixerKind::MinGru: st.state.alloc(halves * (size_t)s.gru.width * 4); break;
+    }
+}
+
 void MixerLm::alloc_activations() {
     const int64_t T = cfg_.max_batch_tokens;
     const int B = cfg_.max_batch_lanes, C = ms_.width;
     int64_t in_rows = 0, mix = 0, a_w = 0, b_w = 0, ff = 0, hd = 0, raw = 0, dqk = 0, dv = 0, dh = 0, attn = 0;
+    int64_t q_lat = 0, uq = 0, lat = 0, cat = 0;  // widths of latent attention's rows, and of `out`'s input with both branches
+    int lat_groups = 1;
+    int64_t lat_part = 0;
     for (size_t l = 0; l < lw_.size(); ++l) {
         const MixerLayerSpec& s = ms_.layers[l];
         const Layer& w = lw_[l];
         in_rows = std::max(in_rows, w.in.rows);
+        if (ms_.side_by_side) {
+            mix = 2;
+            cat = std::max(cat, (int64_t)w.out.ld);
+            if (s.kind == MixerKind::Latent) {
+                const LatentSpec& a = s.latent;
+                q_lat = std::max(q_lat, (int64_t)w.uq.ld);
+                uq = std::max(uq, (int64_t)a.heads * w.q_width);
+                lat = std::max(lat, (int64_t)a.heads * w.row_width);
+                const LatentGeometry& g = latent_geo_[(size_t)w.geometry];
+                if (g.wide) attn = std::max(attn, (int64_t)a.heads * w.q_width);
+                lat_groups = std::max(lat_groups, g.groups);
+                if (g.tc) lat_part = std::max(lat_part, (int64_t)latent_max_shared_entries(g.groups) * g.groups * latent_tc_heads(a.heads) * w.row_width);
+            }
+            continue;
+        }
         ff = std::max(ff, (int64_t)s.ff);
         if (s.kind == MixerKind::Wkv) {
             mix = 5;
@@ -282,7 +349,7 @@ void MixerLm::alloc_activations() {
             hd = std::max(hd, n);
             raw = std::max(raw, n);
             b_w = std::max(b_w, n);
-        } else {
+        } else if (s.kind == MixerKind::Parallel) {
             a_w = std::max(a_w, (int64_t)s.attn.heads * s.attn.vdim);
             attn = std::max(attn, (int64_t)s.attn.heads * w.row_width);
             const int64_t n = (int64_t)s.delta.heads * s.delta.vdim;
@@ -309,6 +376,19 @@ void MixerLm::alloc_activations() {
     decay_.alloc((size_t)(T * hd) * 4);
     raw_.alloc((size_t)(T * raw) * 4);
     q_rot_.alloc((size_t)(T * attn) * 4);
+    img_q_.alloc((size_t)(T * q_lat) * esz_);
+    img_uq_.alloc((size_t)(T * uq) * esz_);
+    q_lat_.alloc((size_t)(T * lat) * 4);
+    img_lat_.alloc((size_t)(T * lat) * esz_);
+    img_cat_.alloc((size_t)(T * cat) * esz_);
+    img_cat_.zero(stream_);  // padding between and behind the two parts meets zero weights
+    if (ms_.loop.times > 0) img_loop_.alloc((size_t)(T * loop_in_.ld) * esz_);
+    if (lat_part > 0) {
+        lat_part_o_.alloc((size_t)lat_part * 4);
+        lat_part_ml_.alloc((size_t)lat_part / 64 * 2 * 4);
+        lat_counters_.alloc((size_t)latent_max_shared_entries(1) * lat_groups * 4);
+        lat_counters_.zero(stream_);
+    }
     attn_.alloc((size_t)(T * attn) * 4);
     dq_.alloc((size_t)(T * dqk) * 4);
     dk_.alloc((size_t)(T * dqk) * 4);
@@ -331,6 +411,8 @@ void MixerLm::alloc_activations() {
             extra += (size_t)(T + B) * 8 + 64;
         }
     }
+    for (const LatentGeometry& g : latent_geo_) extra += (size_t)latent_max_entries((int)T, g.groups) * 32 + (size_t)T * 4 + 32;
+    if (!latent_geo_.empty()) extra += (size_t)B * sizeof(LaneHeader) + (size_t)(T + B) * 8 + (size_t)T * 4 + (size_t)(pool_->max_blocks() + B) * 4 + 64;
     attn_part_o_.alloc(part_o);
     attn_part_ml_.alloc(part_ml);
     attn_counters_.alloc(counters);
@@ -355,7 +437,7 @@ Shares MixerLm::matmul(const Dense& W, const RowImage& x, int T, DevBuf& y, int 
     const double bytes = (double)W.bytes + (double)esz_ * T * W.ld * W.n_groups + 4.0 * T * W.rows, flops = 2.0 * T * (double)W.rows * W.ld;
     if (f32_) {
         prof_begin(KC_F32_MATMUL, bytes, flops);
-        launch_f32_matmul(W.f32.as<float>(), W.rows, W.ld, x.f, T, y.as<float>(), (int)W.rows, W.n_groups, W.group_end, stream_);
+        launch_f32_matmul(W.f32.as<float>(), W.rows, W.ld, x.f, T, y.as<float>(), (int)W.rows, W.n_groups, W.group_end, stream_, W.group_tiles);
     } else {
         prof_begin(T <= 64 ? KC_GEMM_NARROW : KC_GEMM, bytes, flops);
         HgemmScratch ws;
@@ -374,8 +456,25 @@ Shares MixerLm::matmul(const Dense& W, const RowImage& x, int T, DevBuf& y, int 
     return out;
 }
 
+void MixerLm::matmul_scatter(const Dense& W, const RowImage& x, int T, const MatmulScatter& to) {
+    const double bytes = (double)W.bytes + (double)esz_ * T * W.ld * W.n_groups + (to.type == MatmulScatter::F32 ? 4.0 : 2.0) * T * W.rows;
+    const double flops = 2.0 * T * (double)W.rows * W.ld;
+    if (f32_) {
+        prof_begin(KC_F32_MATMUL, bytes, flops);
+        launch_f32_matmul(W.f32.as<float>(), W.rows, W.ld, x.f, T, nullptr, 0, W.n_groups, W.group_end, stream_, W.group_tiles, 1.f, &to);
+    } else {
+        prof_begin(T <= 64 ? KC_GEMM_NARROW : KC_GEMM, bytes, flops);
+        HgemmScratch ws;
+        ws.status = status_.as<int32_t>();
+        launch_hgemm_tc_scatter(W.half, reinterpret_cast<const __half*>(x.h), T, to, ws, stream_);
+    }
+    prof_end();
+    ++launches_;
+}
+
 void MixerLm::set_norm(RowUpdateArgs& a, const Norm& n) const {
     a.norm = ms_.norm;
+    a.norm_eps = ms_.eps;
     a.alpha = n.alpha;
     a.norm_w = n.w.as<float>();
     a.norm_b = n.b.as<float>();
@@ -383,13 +482,14 @@ void MixerLm::set_norm(RowUpdateArgs& a, const Norm& n) const {
 
 // Fills in the residual part of a row update; what is pending is added on the way.
 void MixerLm::apply_pending(RowUpdateArgs& a, Pending& p, bool other_buffer) {
-    a.x = x_[cur_].as<float>();
+    a.x = p.replace ? nullptr : x_[cur_].as<float>();
     a.width = ms_.width;
     a.n_add = p.n;
     for (int i = 0; i < p.n; ++i) {
         a.add[i] = p.y[i];
         a.add_w[i] = p.w[i];
     }
+    a.add_bias = p.bias;
     a.add_coef = p.coef;
     a.add_eps = ms_.eps;
     if (p.n > 0) {
@@ -399,7 +499,9 @@ void MixerLm::apply_pending(RowUpdateArgs& a, Pending& p, bool other_buffer) {
     p = Pending{};
 }
 
-void MixerLm::run_wkv(const Tick& t, int l, Pending& pend) {
+void MixerLm::run_wkv(const Tick& t, int run, Pending& pend) {
+    const int l = runs_[(size_t)run].layer;
+    RunState& st = rs_[(size_t)run];
     const WkvSpec& s = ms_.layers[(size_t)l].wkv;
     Layer& w = lw_[(size_t)l];
     const int T = t.T, C = ms_.width, HD = s.heads * s.dim;
@@ -412,7 +514,7 @@ void MixerLm::run_wkv(const Tick& t, int l, Pending& pend) {
     u.mixes = image(mixes_, w.in.ld);
     u.lanes = state_lanes_;
     u.token_lane = t.bd.token_lane;
-    u.kept = w.kept.as<float>();
+    u.kept = st.kept.as<float>();
     prof_begin(KC_ROW_UPDATE, (double)T * C * (8.0 + 4.0 * u.n_add + 5.0 * esz_), 0);
     launch_row_update(u, stream_);
     prof_end();
@@ -422,7 +524,7 @@ void MixerLm::run_wkv(const Tick& t, int l, Pending& pend) {
     prof_end();
     WkvScanArgs a;
     a.common.lanes = state_lanes_;
-    a.common.state = w.state.as<float>();
+    a.common.state = st.state.as<float>();
     a.common.heads = s.heads;
     a.common.dim = a.common.vdim = s.dim;
     a.common.out = raw_.as<float>();
@@ -455,7 +557,9 @@ void MixerLm::run_wkv(const Tick& t, int l, Pending& pend) {
     pend.y[0] = matmul(w.out, img, T, y_a_, 1);
 }
 
-void MixerLm::run_parallel(const Tick& t, int l, Pending& pend, const std::vector<LmLane>& lanes) {
+void MixerLm::run_parallel(const Tick& t, int run, Pending& pend, const std::vector<LmLane>& lanes) {
+    const int l = runs_[(size_t)run].layer;
+    RunState& st = rs_[(size_t)run];
     const AttentionSpec& s = ms_.layers[(size_t)l].attn;
     const DeltaSpec& d = ms_.layers[(size_t)l].delta;
     Layer& w = lw_[(size_t)l];
@@ -493,8 +597,8 @@ void MixerLm::run_parallel(const Tick& t, int l, Pending& pend, const std::vecto
     }
     ra.positions = t.bd.positions;
     ra.slots = t.bd.slots;
-    ra.k_pool = w.k_pool.ptr();
-    ra.v_pool = w.v_pool.ptr();
+    ra.k_pool = st.k_pool.ptr();
+    ra.v_pool = st.v_pool.ptr();
     ra.kv_f16 = cfg_.kv_f16 ? 1 : 0;
     ra.T = T;
     ra.q_heads = s.heads;
@@ -525,8 +629,8 @@ void MixerLm::run_parallel(const Tick& t, int l, Pending& pend, const std::vecto
         AttnTcArgs ta;
         ta.q = q_rot_.as<float>();
         ta.out = attn_.as<float>();
-        ta.k_pool = w.k_pool.ptr();
-        ta.v_pool = w.v_pool.ptr();
+        ta.k_pool = st.k_pool.ptr();
+        ta.v_pool = st.v_pool.ptr();
         ta.hdr = t.bd.hdr;
         ta.tables = t.bd.tables;
         ta.cu_seqlens = t.bd.cu_seqlens;
@@ -556,8 +660,8 @@ void MixerLm::run_parallel(const Tick& t, int l, Pending& pend, const std::vecto
         AttnArgs at;
         at.q = q_rot_.as<float>();
         at.out = attn_.as<float>();
-        at.k_pool = w.k_pool.ptr();
-        at.v_pool = w.v_pool.ptr();
+        at.k_pool = st.k_pool.ptr();
+        at.v_pool = st.v_pool.ptr();
         at.kv_f16 = ra.kv_f16;
         at.batch = t.bd;
         at.batch.tile_lane = reinterpret_cast<int32_t*>(t.dp + g.off_tile_lane);
@@ -599,7 +703,7 @@ void MixerLm::run_parallel(const Tick& t, int l, Pending& pend, const std::vecto
     dp.log_decay = w.log_decay.as<float>();
     dp.lanes = state_lanes_;
     dp.token_lane = t.bd.token_lane;
-    dp.tail = w.tail.as<float>();
+    dp.tail = st.tail.as<float>();
     dp.q = dq_.as<float>();
     dp.k = dk_.as<float>();
     dp.v = dv_.as<float>();
@@ -611,7 +715,7 @@ void MixerLm::run_parallel(const Tick& t, int l, Pending& pend, const std::vecto
     prof_end();
     DeltaScanArgs sc;
     sc.common.lanes = state_lanes_;
-    sc.common.state = w.state.as<float>();
+    sc.common.state = st.state.as<float>();
     sc.common.heads = d.heads;
     sc.common.dim = d.dim;
     sc.common.vdim = d.vdim;
@@ -659,6 +763,7 @@ void MixerLm::run_forward(const std::vector<LmLane>& lanes, KvReservation& r, ui
         first_row += l.n_tokens;
         longest = std::max(longest, l.n_tokens);
     }
+    longest_ = longest;
     short_lanes_ = longest <= kShortLane;
     const size_t off_halves = stage_bytes(t, halves.data(), halves.size() * sizeof(StateLane));
     std::vector<int32_t> sp((size_t)B), nt((size_t)B), nb((size_t)B);
@@ -687,17 +792,21 @@ void MixerLm::run_forward(const std::vector<LmLane>& lanes, KvReservation& r, ui
             g.off_tile_row = stage_bytes(t, g.tile_row.data(), g.tile_row.size() * 4);
         }
     }
+    if (!latent_geo_.empty()) plan_latent(t, sp, nt, nb, r);
     upload_tick(t, 64, KC_BATCH);
     state_lanes_.lane = reinterpret_cast<const StateLane*>(t.dp + off_halves);
     state_lanes_.lanes = B;
     // copy-on-write page copies of shared partial tails
     for (const KvCowCopy& c : r.cow_copies())
-        for (size_t l = 0; l < lw_.size(); ++l)
-            if (lw_[l].row_width > 0) {
-                launch_cow_copy(lw_[l].k_pool.ptr(), lw_[l].v_pool.ptr(), cfg_.kv_f16 ? 1 : 0, c.src_slot, c.dst_slot, c.rows, 1, pool_->max_blocks(),
-                                ms_.layers[l].attn.kv_heads, cfg_.block_tokens, lw_[l].row_width, stream_);
-                ++launches_;
-            }
+        for (size_t i = 0; i < rs_.size(); ++i) {
+            RunState& st = rs_[i];
+            const int l = runs_[i].layer;
+            if (st.k_pool.size() == 0) continue;
+            const bool latent = st.v_pool.size() == 0;  // one pool: both arguments name it
+            launch_cow_copy(st.k_pool.ptr(), latent ? st.k_pool.ptr() : st.v_pool.ptr(), cfg_.kv_f16 ? 1 : 0, c.src_slot, c.dst_slot, c.rows, 1,
+                            pool_->max_blocks(), latent ? 1 : ms_.layers[(size_t)l].attn.kv_heads, cfg_.block_tokens, lw_[(size_t)l].row_width, stream_);
+            ++launches_;
+        }
     cur_ = 0;
     QWeight table;
     table.type = f32_ ? QT_F32 : QT_BF16;
@@ -705,19 +814,38 @@ void MixerLm::run_forward(const std::vector<LmLane>& lanes, KvReservation& r, ui
     table.cols = C;
     table.p0 = embed_.ptr();
     prof_begin(KC_EMBED, (4.0 + esz_) * T * C, 0);
-    launch_embed(table, t.ids, T, 1.f, x_[cur_].as<float>(), stream_);
+    if (ms_.sinusoid_positions) {
+        EmbedNormArgs e;
+        e.ids = t.ids;
+        e.positions = t.bd.positions;
+        e.table = embed_.ptr();
+        e.table_f32 = f32_ ? 1 : 0;
+        e.rows = T;
+        e.width = C;
+        e.freq = position_freq_.as<double>();
+        e.norm_w = embed_norm_.w.as<float>();
+        e.eps = ms_.eps;
+        e.x = x_[cur_].as<float>();
+        if (ms_.loop.times > 0) e.image = image(img_loop_, loop_in_.ld).part(loop_in_.ld / 2, loop_in_.ld / 2);
+        launch_embed_norm(e, stream_);
+    } else {
+        launch_embed(table, t.ids, T, 1.f, x_[cur_].as<float>(), stream_);
+    }
     prof_end();
     ++launches_;
-    if (capture_) captured_.ensure((size_t)lw_.size() * T * C * 4);
+    if (capture_) captured_.ensure(runs_.size() * T * C * 4);
     captured_tokens_ = T;
 
     Pending pend;
-    for (int l = 0; l < (int)lw_.size(); ++l) {
+    for (int run = 0; run < (int)runs_.size(); ++run) {
+        const int l = runs_[(size_t)run].layer;
         const MixerLayerSpec& s = ms_.layers[(size_t)l];
         Layer& w = lw_[(size_t)l];
-        if (s.kind == MixerKind::Wkv) run_wkv(t, l, pend);
-        else run_parallel(t, l, pend, lanes);
-        if (s.ff > 0) {
+        if (runs_[(size_t)run].first) begin_pass(t, runs_[(size_t)run].pass, pend);
+        if (ms_.side_by_side) run_side_by_side(t, run, pend, lanes);
+        else if (s.kind == MixerKind::Wkv) run_wkv(t, run, pend);
+        else run_parallel(t, run, pend, lanes);
+        if (s.ff > 0 && !ms_.side_by_side) {
             RowUpdateArgs u;
             u.rows = T;
             apply_pending(u, pend, false);
@@ -768,7 +896,7 @@ void MixerLm::run_forward(const std::vector<LmLane>& lanes, KvReservation& r, ui
             apply_pending(u, pend, false);
             launch_row_update(u, stream_);
             ++launches_;
-            MK_CUDA(cudaMemcpyAsync(captured_.as<float>() + (size_t)l * T * C, x_[cur_].ptr(), (size_t)T * C * 4, cudaMemcpyDeviceToDevice, stream_));
+            MK_CUDA(cudaMemcpyAsync(captured_.as<float>() + (size_t)run * T * C, x_[cur_].ptr(), (size_t)T * C * 4, cudaMemcpyDeviceToDevice, stream_));
         }
     }
     if (R > 0 && (flags & (FWD_WANT_LOGITS | FWD_WANT_TOKENS))) {
@@ -789,11 +917,11 @@ void MixerLm::run_forward(const std::vector<LmLane>& lanes, KvReservation& r, ui
         prof_begin(f32_ ? KC_F32_MATMUL : (R <= 64 ? KC_GEMM_NARROW : KC_GEMM), (double)head_.bytes + (double)esz_ * R * C + 4.0 * R * ms_.vocab,
                    2.0 * R * (double)ms_.vocab * C);
         if (f32_) {
-            launch_f32_matmul(head_.f32.as<float>(), head_.rows, head_.ld, u.normed.f, R, logits_.as<float>(), ms_.vocab, 1, nullptr, stream_);
+            launch_f32_matmul(head_.f32.as<float>(), head_.rows, head_.ld, u.normed.f, R, logits_.as<float>(), ms_.vocab, 1, nullptr, stream_, 0, ms_.logit_scale);
         } else {
             HgemmScratch ws;
             ws.status = status_.as<int32_t>();
-            launch_hgemm_tc(head_.half, reinterpret_cast<const __half*>(u.normed.h), R, logits_.as<float>(), ms_.vocab, 1.f, 0.f, ws, stream_, 1);
+            launch_hgemm_tc(head_.half, reinterpret_cast<const __half*>(u.normed.h), R, logits_.as<float>(), ms_.vocab, ms_.logit_scale, 0.f, ws, stream_, 1);
         }
         prof_end();
         ++launches_;
@@ -806,8 +934,8 @@ void MixerLm::run_forward(const std::vector<LmLane>& lanes, KvReservation& r, ui
 void MixerLm::copy_state(int from, int to) {
     MK_CUDA(cudaSetDevice(cfg_.device));
     const size_t halves = (size_t)state_slots_->capacity() * 2;
-    for (Layer& w : lw_)
-        for (DevBuf* b : {&w.state, &w.kept, &w.tail}) {
+    for (RunState& st : rs_)
+        for (DevBuf* b : {&st.state, &st.kept, &st.tail}) {
             if (b->size() == 0) continue;
             const size_t n = b->size() / halves;
             MK_CUDA(cudaMemcpyAsync(b->as<uint8_t>() + (size_t)to * n, b->as<uint8_t>() + (size_t)from * n, n, cudaMemcpyDeviceToDevice, stream_));
@@ -821,7 +949,7 @@ void MixerLm::capture_residuals(bool on) {
 
 int MixerLm::read_residuals(float* out, int64_t capacity) {
     if (!capture_ || captured_tokens_ == 0) throw std::runtime_error("no forward has left its residual stream");
-    const int64_t n = (int64_t)lw_.size() * captured_tokens_ * ms_.width;
+    const int64_t n = (int64_t)runs_.size() * captured_tokens_ * ms_.width;
     if (out == nullptr || capacity < n) throw std::runtime_error("residual buffer needs " + std::to_string(n) + " floats");
     MK_CUDA(cudaStreamSynchronize(stream_));
     MK_CUDA(cudaMemcpy(out, captured_.ptr(), (size_t)n * 4, cudaMemcpyDeviceToHost));

@@ -50,13 +50,12 @@ __device__ __forceinline__ void put_pack(const RowImage& im, int64_t row, int co
 }
 
 __device__ __forceinline__ void zero_tail(const RowImage& im, int64_t row, int width) {
-    for (int c = width + threadIdx.x; c < im.ld; c += blockDim.x) im.put(row, c, 0.f);
+    for (int c = width + threadIdx.x; c < im.end(); c += blockDim.x) im.put(row, c, 0.f);
 }
 
-// The updated row into `dst` (shared memory): x + coef * branches.  Normed branches are staged in `dst` / `other` first.
+// The updated row into `dst` (shared memory): x + coef * (branches + bias).  Normed branches are staged in `dst` / `other` first.
 template <int VEC>
 __device__ __forceinline__ void updated_row(const RowUpdateArgs& a, int64_t row, float* dst, float* other, float* red) {
-    const float* x = a.x + row * a.width;
     const int step = RU_THREADS * VEC;
     float inv[2] = {1.f, 1.f};
     const bool normed = a.n_add > 0 && a.add_w[0] != nullptr;
@@ -76,7 +75,11 @@ __device__ __forceinline__ void updated_row(const RowUpdateArgs& a, int64_t row,
     }
     // a thread reads and writes the same columns of the staging rows throughout, so no barrier is needed in between
     for (int c = threadIdx.x * VEC; c < a.width; c += step) {
-        Pack<VEC> v = load_pack<VEC>(x + c);
+        Pack<VEC> v;
+        if (a.x != nullptr) v = load_pack<VEC>(a.x + row * a.width + c);
+        else
+#pragma unroll
+            for (int i = 0; i < VEC; ++i) v.v[i] = 0.f;
         if (normed) {
             Pack<VEC> sum;
             const Pack<VEC> y0 = load_pack<VEC>(dst + c), w0 = load_pack<VEC>(a.add_w[0] + c);
@@ -90,7 +93,12 @@ __device__ __forceinline__ void updated_row(const RowUpdateArgs& a, int64_t row,
 #pragma unroll
             for (int i = 0; i < VEC; ++i) v.v[i] = fmaf(a.add_coef, sum.v[i], v.v[i]);
         } else if (a.n_add > 0) {
-            const Pack<VEC> y = share_pack<VEC>(a.add[0], row, c);
+            Pack<VEC> y = share_pack<VEC>(a.add[0], row, c);
+            if (a.add_bias != nullptr) {
+                const Pack<VEC> b = load_pack<VEC>(a.add_bias + c);
+#pragma unroll
+                for (int i = 0; i < VEC; ++i) y.v[i] += b.v[i];
+            }
 #pragma unroll
             for (int i = 0; i < VEC; ++i) v.v[i] = fmaf(a.add_coef, y.v[i], v.v[i]);
         }
@@ -98,12 +106,43 @@ __device__ __forceinline__ void updated_row(const RowUpdateArgs& a, int64_t row,
     }
 }
 
+// Mean and root of (variance + eps) of a staged row, for the layer norm.
+struct RowStats {
+    float mean = 0.f, root = 1.f;
+};
 template <int VEC>
-__device__ __forceinline__ Pack<VEC> norm_pack(const RowUpdateArgs& a, const Pack<VEC>& x, int c) {
-    Pack<VEC> h;
-    const Pack<VEC> w = load_pack<VEC>(a.norm_w + c), b = load_pack<VEC>(a.norm_b + c);
+__device__ __forceinline__ RowStats row_stats(const float* x, int width, float eps, float* red) {
+    const int step = RU_THREADS * VEC;
+    float s = 0.f;
+    for (int c = threadIdx.x * VEC; c < width; c += step) {
+        const Pack<VEC> v = load_pack<VEC>(x + c);
 #pragma unroll
-    for (int i = 0; i < VEC; ++i) h.v[i] = fmaf(tanhf(a.alpha * x.v[i]), w.v[i], b.v[i]);
+        for (int i = 0; i < VEC; ++i) s += v.v[i];
+    }
+    RowStats r;
+    r.mean = block_sum(s, red) / (float)width;
+    s = 0.f;
+    for (int c = threadIdx.x * VEC; c < width; c += step) {
+        const Pack<VEC> v = load_pack<VEC>(x + c);
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) s = fmaf(v.v[i] - r.mean, v.v[i] - r.mean, s);
+    }
+    r.root = sqrtf(block_sum(s, red) / (float)width + eps);
+    return r;
+}
+
+template <int VEC>
+__device__ __forceinline__ Pack<VEC> norm_pack(const RowUpdateArgs& a, const RowStats& st, const Pack<VEC>& x, int c) {
+    Pack<VEC> h;
+    const Pack<VEC> w = load_pack<VEC>(a.norm_w + c);
+    if (a.norm == NormKind::Layer) {
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) h.v[i] = (x.v[i] - st.mean) / st.root * w.v[i];
+    } else {
+        const Pack<VEC> b = load_pack<VEC>(a.norm_b + c);
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) h.v[i] = fmaf(tanhf(a.alpha * x.v[i]), w.v[i], b.v[i]);
+    }
     return h;
 }
 
@@ -128,8 +167,11 @@ __global__ void __launch_bounds__(RU_THREADS) row_update_kernel(RowUpdateArgs a)
         zero_tail(a.raw, r, a.width);
     }
     if (a.norm == NormKind::None) return;
+    // a thread has written the columns of `cur` that it reads itself; block_sum's barriers are all the sums need
+    RowStats st, st_prev;
+    if (a.norm == NormKind::Layer) st = row_stats<VEC>(cur, a.width, a.norm_eps, red);
     if (a.n_mix == 0) {
-        for (int c = threadIdx.x * VEC; c < a.width; c += step) put_pack<VEC>(a.normed, r, c, norm_pack<VEC>(a, load_pack<VEC>(cur + c), c));
+        for (int c = threadIdx.x * VEC; c < a.width; c += step) put_pack<VEC>(a.normed, r, c, norm_pack<VEC>(a, st, load_pack<VEC>(cur + c), c));
         zero_tail(a.normed, r, a.width);
         return;
     }
@@ -137,11 +179,14 @@ __global__ void __launch_bounds__(RU_THREADS) row_update_kernel(RowUpdateArgs a)
     const StateLane sl = a.lanes.at(lane);
     const int first = sl.first, last = sl.first + sl.n - 1;
     const bool inside = row > first;
-    if (inside) updated_row<VEC>(a, row - 1, prv, other, red);
+    if (inside) {
+        updated_row<VEC>(a, row - 1, prv, other, red);
+        if (a.norm == NormKind::Layer) st_prev = row_stats<VEC>(prv, a.width, a.norm_eps, red);
+    }
     for (int c = threadIdx.x * VEC; c < a.width; c += step) {
-        const Pack<VEC> h = norm_pack<VEC>(a, load_pack<VEC>(cur + c), c);
+        const Pack<VEC> h = norm_pack<VEC>(a, st, load_pack<VEC>(cur + c), c);
         Pack<VEC> p;
-        if (inside) p = norm_pack<VEC>(a, load_pack<VEC>(prv + c), c);
+        if (inside) p = norm_pack<VEC>(a, st_prev, load_pack<VEC>(prv + c), c);
         else if (sl.in >= 0) p = load_pack<VEC>(a.kept + (int64_t)sl.in * a.width + c);
         else
 #pragma unroll
@@ -313,16 +358,17 @@ __global__ void __launch_bounds__(DP_WARPS * 32) delta_prep_kernel(DeltaPrepArgs
 
 // ------------------------------------------------------------------------------------------------ gates
 
-__global__ void __launch_bounds__(256) head_gate_kernel(const float* attn, int heads, int row_width, int vdim, Shares gate, int gate_col, RowImage out) {
+__global__ void __launch_bounds__(256) head_gate_kernel(const float* attn, int heads, int row_width, int vdim, Shares gate, int gate_col, RowImage out,
+                                                        const int32_t* rows) {
     extern __shared__ float hg_gate[];
     pdl_trigger();
     pdl_wait();
-    const int64_t row = blockIdx.x;
+    const int64_t row = rows != nullptr ? rows[blockIdx.x] : blockIdx.x;
     for (int h = threadIdx.x; h < heads; h += blockDim.x) hg_gate[h] = sigmoid_f(gate.at(row, gate_col + h));
     __syncthreads();
     const float* src = attn + row * heads * row_width;
-    if ((vdim & 3) == 0) {  // out.ld is a multiple of 64, a head's row of 4
-        for (int c = threadIdx.x * 4; c < out.ld; c += blockDim.x * 4) {
+    if ((vdim & 3) == 0) {  // out.end() is a multiple of 64, a head's row of 4
+        for (int c = threadIdx.x * 4; c < out.end(); c += blockDim.x * 4) {
             const int h = c / vdim;
             float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
             if (h < heads) {
@@ -334,7 +380,7 @@ __global__ void __launch_bounds__(256) head_gate_kernel(const float* attn, int h
         }
         return;
     }
-    for (int c = threadIdx.x; c < out.ld; c += blockDim.x) {
+    for (int c = threadIdx.x; c < out.end(); c += blockDim.x) {
         const int h = c / vdim;
         out.put(row, c, h < heads ? src[h * row_width + (c - h * vdim)] * hg_gate[h] : 0.f);
     }
@@ -346,7 +392,7 @@ __global__ void __launch_bounds__(128) side_gate_kernel(Shares z, int dim, const
     pdl_wait();
     const int64_t row = blockIdx.x;
     const int64_t at = (int64_t)ids[row] * table_ld + slice;
-    for (int c = threadIdx.x; c < out.ld; c += blockDim.x) {
+    for (int c = threadIdx.x; c < out.end(); c += blockDim.x) {
         float v = 0.f;
         if (c < dim) {
             const float e = table_f32 ? static_cast<const float*>(table)[at + c] : __bfloat162float(static_cast<const __nv_bfloat16*>(table)[at + c]);
@@ -360,7 +406,130 @@ __global__ void __launch_bounds__(256) gated_act_kernel(Shares gu, int ff, RowIm
     pdl_trigger();
     pdl_wait();
     const int64_t row = blockIdx.x;
-    for (int c = threadIdx.x; c < out.ld; c += blockDim.x) out.put(row, c, c < ff ? silu_f(gu.at(row, 2 * c)) * gu.at(row, 2 * c + 1) : 0.f);
+    for (int c = threadIdx.x; c < out.end(); c += blockDim.x) out.put(row, c, c < ff ? silu_f(gu.at(row, 2 * c)) * gu.at(row, 2 * c + 1) : 0.f);
+}
+
+// ------------------------------------------------------------------------------------------------ embedding with positions
+
+// Shared memory: the row.
+__global__ void __launch_bounds__(RU_THREADS) embed_norm_kernel(EmbedNormArgs a) {
+    extern __shared__ __align__(16) float en_row[];
+    __shared__ float red[32];
+    pdl_trigger();
+    pdl_wait();
+    const int64_t row = blockIdx.x, at = (int64_t)a.ids[row] * a.width;
+    const double pos = (double)a.positions[row];
+    constexpr double kTwoPi = 6.283185307179586476925;
+    for (int i = threadIdx.x; 2 * i < a.width; i += RU_THREADS) {
+        double angle = pos * a.freq[i];
+        angle -= rint(angle / kTwoPi) * kTwoPi;
+        float sn, cs;
+        sincosf((float)angle, &sn, &cs);
+        for (int j = 0; j < 2 && 2 * i + j < a.width; ++j) {
+            const int c = 2 * i + j;
+            const float e = a.table_f32 ? static_cast<const float*>(a.table)[at + c] : __bfloat162float(static_cast<const __nv_bfloat16*>(a.table)[at + c]);
+            en_row[c] = e + (j == 0 ? sn : cs);
+        }
+    }
+    __syncthreads();
+    const RowStats st = row_stats<1>(en_row, a.width, a.eps, red);
+    for (int c = threadIdx.x; c < a.width; c += RU_THREADS) {
+        const float v = (en_row[c] - st.mean) / st.root * a.norm_w[c];
+        a.x[row * a.width + c] = v;
+        if (a.image.any()) a.image.put(row, c, v);
+    }
+    if (a.image.any()) zero_tail(a.image, row, a.width);
+}
+
+// ------------------------------------------------------------------------------------------------ latents, polynomial activation
+
+constexpr int LP_THREADS = 256;
+
+// Three block sums behind one barrier.
+__device__ __forceinline__ float3 block_sum3(float3 v, float (*red)[3]) {
+    const int lane = threadIdx.x & 31, w = threadIdx.x >> 5;
+    v.x = warp_sum(v.x);
+    v.y = warp_sum(v.y);
+    v.z = warp_sum(v.z);
+    if (lane == 0) {
+        red[w][0] = v.x;
+        red[w][1] = v.y;
+        red[w][2] = v.z;
+    }
+    __syncthreads();
+    float3 r = make_float3(0.f, 0.f, 0.f);
+#pragma unroll
+    for (int i = 0; i < LP_THREADS / 32; ++i) {
+        r.x += red[i][0];
+        r.y += red[i][1];
+        r.z += red[i][2];
+    }
+    return r;
+}
+
+template <int VEC>
+__device__ __forceinline__ void poly_row(const LatentPrepArgs& a, int64_t row, float* z, float (*red)[3]) {
+    const int step = LP_THREADS * VEC;
+    float3 ss = make_float3(0.f, 0.f, 0.f);
+    for (int c = threadIdx.x * VEC; c < a.ff; c += step) {
+        Pack<VEC> v = share_pack<VEC>(a.y, row, a.ff_col + c);
+        const Pack<VEC> b = load_pack<VEC>(a.ff_bias + c);
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) {
+            v.v[i] += b.v[i];
+            const float z1 = v.v[i], z2 = z1 * z1, z3 = z2 * z1;
+            ss.x = fmaf(z1, z1, ss.x);
+            ss.y = fmaf(z2, z2, ss.y);
+            ss.z = fmaf(z3, z3, ss.z);
+        }
+        store_pack<VEC>(z + c, v);
+    }
+    ss = block_sum3(ss, red);
+    const float n = (float)a.ff;
+    const float k1 = a.poly[0] / sqrtf(ss.x / n + a.eps), k2 = a.poly[1] / sqrtf(ss.y / n + a.eps), k3 = a.poly[2] / sqrtf(ss.z / n + a.eps), k0 = a.poly[3];
+    for (int c = threadIdx.x * VEC; c < a.ff; c += step) {
+        Pack<VEC> v = load_pack<VEC>(z + c);
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) v.v[i] = fmaf(fmaf(fmaf(k3, v.v[i], k2), v.v[i], k1), v.v[i], k0);
+        put_pack<VEC>(a.ff_image, row, c, v);
+    }
+    zero_tail(a.ff_image, row, a.ff);
+}
+
+// Shared memory: max(ff, q_rank + kv_rank) floats.
+template <int VEC>
+__global__ void __launch_bounds__(LP_THREADS) latent_prep_kernel(LatentPrepArgs a) {
+    extern __shared__ __align__(16) float lp_row[];
+    __shared__ float red[LP_THREADS / 32][3];
+    pdl_trigger();
+    pdl_wait();
+    const int64_t row = blockIdx.x;
+    if (a.q_rank == 0 || blockIdx.y == 1) {
+        poly_row<VEC>(a, row, lp_row, red);
+        return;
+    }
+    float* kv = lp_row + a.q_rank;
+    float3 ss = make_float3(0.f, 0.f, 0.f);
+    for (int c = threadIdx.x; c < a.q_rank; c += LP_THREADS) {
+        const float v = a.y.at(row, a.q_col + c);
+        lp_row[c] = v;
+        ss.x = fmaf(v, v, ss.x);
+    }
+    for (int c = threadIdx.x; c < a.kv_rank; c += LP_THREADS) {
+        const float v = a.y.at(row, a.kv_col + c);
+        kv[c] = v;
+        ss.y = fmaf(v, v, ss.y);
+    }
+    ss = block_sum3(ss, red);
+    const float rq = sqrtf(ss.x / (float)a.q_rank + a.eps), rk = sqrtf(ss.y / (float)a.kv_rank + a.eps);
+    for (int c = threadIdx.x; c < a.q_rank; c += LP_THREADS) a.q_image.put(row, c, lp_row[c] / rq * a.q_norm[c]);
+    zero_tail(a.q_image, row, a.q_rank);
+    const int64_t at = a.slots[row] * a.kv_width;
+    for (int c = threadIdx.x; c < a.kv_width; c += LP_THREADS) {
+        const float v = c < a.kv_rank ? kv[c] / rk * a.kv_norm[c] : 0.f;
+        if (a.pool_f16) static_cast<__half*>(a.pool)[at + c] = __float2half_rn(v);
+        else static_cast<float*>(a.pool)[at + c] = v;
+    }
 }
 
 // ------------------------------------------------------------------------------------------------ f32 matmul
@@ -369,7 +538,8 @@ constexpr int FM_TILE = 64, FM_K = 16;
 
 // 64 x 64 outputs per CTA, 4 x 4 per thread.
 __global__ void __launch_bounds__(256) f32_matmul_kernel(const float* __restrict__ w, int64_t rows, int cols, const float* __restrict__ x, int T, float* y,
-                                                         int ldy, int n_groups, int4 end_lo, int4 end_hi) {
+                                                         int ldy, float scale, int n_groups, int group_tiles, int4 end_lo, int4 end_hi,
+                                                         MatmulScatter to) {
     __shared__ float ws[FM_K][FM_TILE + 4], xs[FM_K][FM_TILE + 4];
     pdl_trigger();
     pdl_wait();
@@ -377,7 +547,9 @@ __global__ void __launch_bounds__(256) f32_matmul_kernel(const float* __restrict
     const int t0 = blockIdx.y * FM_TILE;
     const int ends[kMaxRowGroups] = {end_lo.x, end_lo.y, end_lo.z, end_lo.w, end_hi.x, end_hi.y, end_hi.z, end_hi.w};
     int g = 0;
-    while (g < n_groups - 1 && n0 / 128 >= ends[g]) ++g;
+    if (group_tiles > 0) g = (int)(n0 / 128 / group_tiles);
+    else
+        while (g < n_groups - 1 && n0 / 128 >= ends[g]) ++g;
     const float* xg = x + (int64_t)g * T * cols;
     const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
     float acc[4][4] = {};
@@ -409,7 +581,13 @@ __global__ void __launch_bounds__(256) f32_matmul_kernel(const float* __restrict
         for (int j = 0; j < 4; ++j) {
             const int t = t0 + ty * 4 + i;
             const int64_t n = n0 + tx * 4 + j;
-            if (t < T && n < rows) y[(int64_t)t * ldy + n] = acc[i][j];
+            if (t >= T || n >= rows) continue;
+            if (to.out == nullptr) {
+                y[(int64_t)t * ldy + n] = acc[i][j] * scale;
+                continue;
+            }
+            const int64_t col = to.column(n);
+            if (col >= 0) to.put(to.row(t) + col, acc[i][j]);
         }
 }
 
@@ -418,6 +596,7 @@ __global__ void __launch_bounds__(256) f32_matmul_kernel(const float* __restrict
 void launch_row_update(const RowUpdateArgs& a, cudaStream_t s) {
     if (a.rows <= 0) return;
     if (a.n_mix > 0 && (a.x == a.x_out || a.row_index != nullptr)) throw std::runtime_error("launch_row_update: a token shift needs its own output buffer and packed rows");
+    if (a.add_bias != nullptr && (a.n_add != 1 || a.add_w[0] != nullptr)) throw std::runtime_error("launch_row_update: a bias goes with one plain branch");
     if (a.n_add == 2 && (a.add_w[0] == nullptr || a.add_w[1] == nullptr)) throw std::runtime_error("launch_row_update: two branches are both normed");
     bool vec = a.width % 4 == 0;
     for (int b = 0; b < a.n_add; ++b)
@@ -453,9 +632,9 @@ void launch_delta_prep(const DeltaPrepArgs& a, cudaStream_t s) {
 }
 
 void launch_head_gate(const float* attn, int rows, int heads, int row_width, int vdim, const Shares& gate, int gate_col, const RowImage& out,
-                      cudaStream_t s) {
+                      cudaStream_t s, const int32_t* row_list) {
     if (rows <= 0) return;
-    launch_pdl(head_gate_kernel, dim3((unsigned)rows), dim3(256), (size_t)heads * 4, s, attn, heads, row_width, vdim, gate, gate_col, out);
+    launch_pdl(head_gate_kernel, dim3((unsigned)rows), dim3(256), (size_t)heads * 4, s, attn, heads, row_width, vdim, gate, gate_col, out, row_list);
     MK_LAUNCH_CHECK();
 }
 
@@ -472,14 +651,35 @@ void launch_gated_act(const Shares& gu, int rows, int ff, const RowImage& out, c
     MK_LAUNCH_CHECK();
 }
 
+void launch_embed_norm(const EmbedNormArgs& a, cudaStream_t s) {
+    if (a.rows <= 0) return;
+    const size_t smem = (size_t)a.width * 4;
+    if (smem > (size_t)200 * 1024) throw std::runtime_error("launch_embed_norm: the model is too wide");
+    ensure_dynamic_smem(reinterpret_cast<const void*>(&embed_norm_kernel), smem);
+    launch_pdl(embed_norm_kernel, dim3((unsigned)a.rows), dim3(RU_THREADS), smem, s, a);
+    MK_LAUNCH_CHECK();
+}
+
+void launch_latent_prep(const LatentPrepArgs& a, cudaStream_t s) {
+    if (a.rows <= 0 || (a.q_rank == 0 && a.ff == 0)) return;
+    const size_t smem = (size_t)std::max(a.ff, a.q_rank + a.kv_rank) * 4;
+    if (smem > (size_t)220 * 1024) throw std::runtime_error("launch_latent_prep: the feed-forward or the latents are too wide");
+    const bool vec = a.ff % 4 == 0 && a.ff_col % 4 == 0 && a.y.ld % 4 == 0 && a.y.stride % 4 == 0 && (reinterpret_cast<uintptr_t>(a.y.p) & 15) == 0;
+    const dim3 grid((unsigned)a.rows, a.q_rank > 0 && a.ff > 0 ? 2u : 1u);
+    auto* kernel = vec ? latent_prep_kernel<4> : latent_prep_kernel<1>;
+    ensure_dynamic_smem(reinterpret_cast<const void*>(kernel), smem);
+    launch_pdl(kernel, grid, dim3(LP_THREADS), smem, s, a);
+    MK_LAUNCH_CHECK();
+}
+
 void launch_f32_matmul(const float* w, int64_t rows, int cols, const float* x, int T, float* y, int ldy, int n_groups, const int* group_end,
-                       cudaStream_t s) {
+                       cudaStream_t s, int group_tiles, float scale, const MatmulScatter* to) {
     if (T <= 0) return;
     int e[kMaxRowGroups] = {};
-    for (int g = 0; g < n_groups && n_groups > 1; ++g) e[g] = group_end[g];
+    for (int g = 0; g < n_groups && n_groups > 1 && group_tiles == 0; ++g) e[g] = group_end[g];
     const dim3 grid((unsigned)((rows + FM_TILE - 1) / FM_TILE), (unsigned)((T + FM_TILE - 1) / FM_TILE));
-    launch_pdl(f32_matmul_kernel, grid, dim3(256), 0, s, w, rows, cols, x, T, y, ldy, n_groups, make_int4(e[0], e[1], e[2], e[3]),
-               make_int4(e[4], e[5], e[6], e[7]));
+    launch_pdl(f32_matmul_kernel, grid, dim3(256), 0, s, w, rows, cols, x, T, y, ldy, scale, n_groups, group_tiles, make_int4(e[0], e[1], e[2], e[3]),
+               make_int4(e[4], e[5], e[6], e[7]), to != nullptr ? *to : MatmulScatter{});
     MK_LAUNCH_CHECK();
 }
 

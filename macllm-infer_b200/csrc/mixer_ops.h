@@ -3,12 +3,14 @@
 // 32-bit matmul for models computed in f32 throughout.
 #pragma once
 #include "mixer_spec.h"
+#include "device_util.h"
 #include "row_types.cuh"
 
 namespace mk {
 
 // One CTA per row r (x row = row_index ? row_index[r] : r):
-//   x_out = x + coef * sum over branches b of (add_w[b] ? rms(add[b]) * add_w[b] : add[b])      (n_add branches)
+//   x_out = x + coef * sum over branches b of (add_w[b] ? rms(add[b]) * add_w[b] : add[b])      (n_add branches; x = 0 when null)
+//   (a single plain branch may carry a bias [width])
 //   raw    <- x_out                        (optional image)
 //   h       = norm(x_out);  normed <- h    (optional image, n_mix = 0)
 //   mixes[i] <- h + (h' - h) * mu[i]       (n_mix images of `rows` rows each, one after the other), h' = h of the sequence's
@@ -23,12 +25,14 @@ struct RowUpdateArgs {
     int n_add = 0;
     Shares add[2];
     const float* add_w[2] = {nullptr, nullptr};
+    const float* add_bias = nullptr;
     float add_coef = 1.f, add_eps = 0.f;
     RowImage raw;
     NormKind norm = NormKind::None;
-    float alpha = 1.f;
+    float alpha = 1.f;          // DynTanh
+    float norm_eps = 0.f;       // Layer
     const float* norm_w = nullptr;
-    const float* norm_b = nullptr;
+    const float* norm_b = nullptr;  // DynTanh
     RowImage normed;
     int n_mix = 0;
     const float* mu = nullptr;  // [n_mix][width]
@@ -59,9 +63,9 @@ struct DeltaPrepArgs {
 };
 void launch_delta_prep(const DeltaPrepArgs& a, cudaStream_t s);
 
-// out[t][h * vdim + i] = attn[t][h * row_width + i] * sigmoid(gate[t][gate_col + h])
+// out[t][h * vdim + i] = attn[t][h * row_width + i] * sigmoid(gate[t][gate_col + h]), t = row_list[0 .. rows) or 0 .. rows - 1
 void launch_head_gate(const float* attn, int rows, int heads, int row_width, int vdim, const Shares& gate, int gate_col, const RowImage& out,
-                      cudaStream_t s);
+                      cudaStream_t s, const int32_t* row_list = nullptr);
 
 // out[t][j] = gelu_tanh(z[t][j]) * table[ids[t]][slice + j], j < dim; table [vocab][table_ld] as bfloat16 bits (or f32)
 void launch_side_gate(const Shares& z, int rows, int dim, const uint32_t* ids, const void* table, int table_f32, int64_t table_ld, int slice,
@@ -71,8 +75,49 @@ void launch_side_gate(const Shares& z, int rows, int dim, const uint32_t* ids, c
 void launch_gated_act(const Shares& gu, int rows, int ff, const RowImage& out, cudaStream_t s);
 
 // y[t][n] = sum_k x[t][k] w[n][k] in f32, k ascending.  x is [n_groups][T][cols]; weight row n reads input g of its group, whose
-// rows end at 128 * group_end[g] (see HalfWeight).
+// rows end at 128 * group_end[g], or are 128 * group_tiles each (see HalfWeight).  `to` scatters the result instead (see
+// MatmulScatter).
 void launch_f32_matmul(const float* w, int64_t rows, int cols, const float* x, int T, float* y, int ldy, int n_groups, const int* group_end,
-                       cudaStream_t s);
+                       cudaStream_t s, int group_tiles = 0, float scale = 1.f, const MatmulScatter* to = nullptr);
+
+// The embedding output of models with sinusoidal positions:  e = table[ids[t]] + sinusoid(positions[t]);  x = layer norm of e, in
+// f32 to x [rows][width] and as a matmul input to `image` (optional).  freq[i] is the frequency of column pair i in f64: the angle
+// of a far position is as exact as that of a near one.
+struct EmbedNormArgs {
+    const uint32_t* ids = nullptr;
+    const int32_t* positions = nullptr;
+    const void* table = nullptr;  // [vocab][width] bfloat16 bits, or f32
+    int table_f32 = 0;
+    int rows = 0, width = 0;
+    const double* freq = nullptr;  // [ceil(width / 2)]
+    const float* norm_w = nullptr;
+    float eps = 0.f;
+    float* x = nullptr;
+    RowImage image;
+};
+void launch_embed_norm(const EmbedNormArgs& a, cudaStream_t s);
+
+// What a row's projections need before the next matmuls, one CTA per (row, part):
+//   part 1 (q_rank > 0): the query latent RMS-normed into q_image, the key/value latent RMS-normed into its page
+//   part 2 (ff > 0):     poly = a N(z) + b N(z^2) + c N(z^3) + e over z = y[ff_col ..] + ff_bias, N = division by the row's root
+//                        mean square
+struct LatentPrepArgs {
+    Shares y;
+    int rows = 0;
+    float eps = 0.f;
+    int q_col = 0, q_rank = 0;
+    const float* q_norm = nullptr;
+    RowImage q_image;
+    int kv_col = 0, kv_rank = 0, kv_width = 0;  // kv_width: columns of a page row, the rest is zeros
+    const float* kv_norm = nullptr;
+    const int64_t* slots = nullptr;
+    void* pool = nullptr;                       // [blocks * block_tokens][kv_width]
+    int pool_f16 = 1;
+    int ff_col = 0, ff = 0;
+    const float* ff_bias = nullptr;
+    const float* poly = nullptr;                // [4]
+    RowImage ff_image;
+};
+void launch_latent_prep(const LatentPrepArgs& a, cudaStream_t s);
 
 }  // namespace mk

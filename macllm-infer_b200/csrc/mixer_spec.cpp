@@ -45,6 +45,14 @@ void check_groups(const Json& where, int heads, int kv_heads) {
     if (heads % kv_heads != 0) throw std::runtime_error(where.where() + ": heads must be a multiple of kv_heads");
 }
 
+// Width of a layer's feed-forward, 0: none.
+int read_dense_ff(const Json& layer) {
+    const Json* mlp = layer.find("mlp");
+    if (mlp == nullptr || mlp->is_null()) return 0;
+    if (mlp->at("kind").str() != "dense") throw std::runtime_error(mlp->where() + ".kind `" + mlp->at("kind").str() + "` is not supported");
+    return size_of(mlp->at("ff"));
+}
+
 // Sizilorn: WKV time-mixing layers and layers that run gated attention beside the gated delta rule, Dynamic Tanh norms, and
 // a token input of its own for every layer.
 MixerSpec read_sizilorn(const Json& c, const SafetensorsFile& f) {
@@ -92,17 +100,67 @@ MixerSpec read_sizilorn(const Json& c, const SafetensorsFile& f) {
         } else {
             throw std::runtime_error(j.where() + ".type `" + type + "` is not a known mixer");
         }
-        const Json* mlp = j.find("mlp");
-        if (mlp != nullptr && !mlp->is_null()) {
-            if (mlp->at("kind").str() != "dense") throw std::runtime_error(mlp->where() + ".kind `" + mlp->at("kind").str() + "` is not supported");
-            l.ff = size_of(mlp->at("ff"));
-        }
+        l.ff = read_dense_ff(j);
         s.layers.push_back(l);
     }
     return s;
 }
 
 const RegisterMixerArchitecture register_sizilorn("Sizilorn", read_sizilorn);
+
+float number_of(const Json& v) {
+    const double x = v.number();
+    if (!std::isfinite(x)) throw std::runtime_error(v.where() + " must be finite");
+    return (float)x;
+}
+
+// Kunonex: latent attention and minGRU layers, mixer and feed-forward side by side behind one layer norm, token shift in front
+// of every mixer, sinusoidal positions, and a run of layers that is passed through several times.
+MixerSpec read_kunonex(const Json& c, const SafetensorsFile&) {
+    MixerSpec s;
+    s.arch = "Kunonex";
+    s.vocab = size_of(c.at("vocab"));
+    s.width = size_of(c.at("width"));
+    s.norm = NormKind::Layer;
+    s.ff_kind = FfKind::Poly;
+    s.side_by_side = true;
+    s.sinusoid_positions = true;
+    s.eps = number_of(c.at("norm").at("eps"));
+    if (!(s.eps >= 0.f)) throw std::runtime_error("config norm.eps must not be negative");
+    s.logit_scale = number_of(c.at("logit_scale"));
+    const auto& layers = c.at("layers").items();
+    if (layers.empty()) throw std::runtime_error("config lists no layers");
+    for (const Json& j : layers) {
+        const Json& m = j.at("mixer");
+        const std::string type = j.at("type").str();
+        MixerLayerSpec l;
+        if (type == "latent_attention") {
+            l.kind = MixerKind::Latent;
+            l.latent.heads = size_of(m.at("heads"));
+            l.latent.dim = size_of(m.at("dim"));
+            l.latent.vdim = size_of(m.at("vdim"));
+            l.latent.q_rank = size_of(m.at("q_rank"));
+            l.latent.kv_rank = size_of(m.at("kv_rank"));
+            l.latent.scale = number_of(m.at("scale"));
+        } else if (type == "mingru") {
+            l.kind = MixerKind::MinGru;
+            l.gru.width = size_of(m.at("width"));
+        } else {
+            throw std::runtime_error(j.where() + ".type `" + type + "` is not a known mixer");
+        }
+        l.ff = read_dense_ff(j);
+        s.layers.push_back(l);
+    }
+    const Json* loop = c.find("loop");
+    if (loop != nullptr && !loop->is_null()) {
+        s.loop.start = size_of(loop->at("start"), 0, (int)layers.size() - 1);
+        s.loop.stop = size_of(loop->at("stop"), s.loop.start + 1, (int)layers.size());
+        s.loop.times = size_of(loop->at("times"), 1, 4096);
+    }
+    return s;
+}
+
+const RegisterMixerArchitecture register_kunonex("Kunonex", read_kunonex);
 
 }  // namespace
 
@@ -135,6 +193,11 @@ std::vector<std::pair<std::string, std::vector<int64_t>>> mixer_tensors(const Mi
         }
     };
     add("embed", {V, C});
+    if (s.sinusoid_positions) norm("embed.norm");
+    if (s.loop.times > 0) {
+        add("loop.in", {C, 2 * C});
+        add("loop.step", {s.loop.times, C});
+    }
     if (s.side_dim > 0) add("side.embed", {V, (int64_t)s.layers.size() * s.side_dim});
     for (size_t i = 0; i < s.layers.size(); ++i) {
         const MixerLayerSpec& l = s.layers[i];
@@ -149,6 +212,26 @@ std::vector<std::pair<std::string, std::vector<int64_t>>> mixer_tensors(const Mi
             add(m + "w0", {n});
             add(m + "u", {H, D});
             add(m + "norm", {n});
+            add(m + "o", {C, n});
+        } else if (l.kind == MixerKind::Latent) {
+            const LatentSpec& a = l.latent;
+            const int64_t qw = (int64_t)a.heads * a.dim, vw = (int64_t)a.heads * a.vdim;
+            add(m + "dq", {a.q_rank, C});
+            add(m + "dq.norm", {a.q_rank});
+            add(m + "uq", {qw, a.q_rank});
+            add(m + "dkv", {a.kv_rank, C});
+            add(m + "dkv.norm", {a.kv_rank});
+            add(m + "uk", {qw, a.kv_rank});
+            add(m + "uv", {vw, a.kv_rank});
+            add(m + "g", {a.heads, C});
+            add(m + "o", {C, vw});
+        } else if (l.kind == MixerKind::MinGru) {
+            const int64_t n = l.gru.width;
+            for (const char* x : {"z", "x"}) {
+                add(m + x, {n, C});
+                add(m + x + ".b", {n});
+            }
+            add(m + "g", {n, C});
             add(m + "o", {C, n});
         } else {
             const AttentionSpec& a = l.attn;
@@ -176,11 +259,17 @@ std::vector<std::pair<std::string, std::vector<int64_t>>> mixer_tensors(const Mi
             add(m + "right.o", {C, dv});
             add(m + "right.out", {C});
         }
+        if (s.side_by_side) add(p + "shift", {C});
         if (l.ff > 0) {
-            norm(p + "norm2");
-            add(p + "mlp.gate", {l.ff, C});
+            if (!s.side_by_side) norm(p + "norm2");
+            if (s.ff_kind == FfKind::Gated) add(p + "mlp.gate", {l.ff, C});
             add(p + "mlp.up", {l.ff, C});
             add(p + "mlp.down", {C, l.ff});
+            if (s.ff_kind == FfKind::Poly) {
+                add(p + "mlp.up.b", {l.ff});
+                add(p + "mlp.down.b", {C});
+                add(p + "mlp.act", {4});
+            }
         }
         if (s.side_dim > 0) {
             add(p + "side.gate", {s.side_dim, C});
@@ -190,6 +279,21 @@ std::vector<std::pair<std::string, std::vector<int64_t>>> mixer_tensors(const Mi
     }
     norm("final.norm");
     add("head", {V, C});
+    return out;
+}
+
+std::vector<LayerRun> MixerSpec::runs() const {
+    std::vector<LayerRun> out;
+    const int n = (int)layers.size();
+    for (int l = 0; l < n;) {
+        if (loop.times == 0 || l != loop.start) {
+            out.push_back(LayerRun{l++, -1, false});
+            continue;
+        }
+        for (int pass = 0; pass < loop.times; ++pass)
+            for (int i = loop.start; i < loop.stop; ++i) out.push_back(LayerRun{i, pass, i == loop.start});
+        l = loop.stop;
+    }
     return out;
 }
 

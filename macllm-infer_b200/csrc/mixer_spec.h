@@ -10,7 +10,7 @@
 
 namespace mk {
 
-enum class NormKind { None, DynTanh };
+enum class NormKind { None, DynTanh, Layer };
 
 // Rotary positions on the first `dims` dimensions of a head; dims = 0: none.
 struct RotarySpec {
@@ -45,14 +45,42 @@ struct WkvSpec {
     int heads = 0, dim = 0, rank = 0;  // rank of the decay's low-rank projection
 };
 
-enum class MixerKind { Wkv, Parallel };  // Parallel: attention and the gated delta rule side by side
+// Attention whose keys and values are two projections of one cached vector of `kv_rank` values per token; queries come from a
+// latent of `q_rank` values.  No positions; a sigmoid gate per head on the output.
+struct LatentSpec {
+    int heads = 0, dim = 0, vdim = 0, q_rank = 0, kv_rank = 0;
+    float scale = 1.f;
+};
+
+// Element-wise gated recurrence over `width` channels whose gates read the current token only.
+struct MinGruSpec {
+    int width = 0;
+};
+
+enum class MixerKind { Wkv, Parallel, Latent, MinGru };  // Parallel: attention and the gated delta rule side by side
+
+enum class FfKind { Gated, Poly };  // silu(gate) * up; a cubic of up, every power over its own root mean square
 
 struct MixerLayerSpec {
     MixerKind kind = MixerKind::Wkv;
     WkvSpec wkv;
     AttentionSpec attn;
     DeltaSpec delta;
-    int ff = 0;  // width of the gated feed-forward, 0: the layer has none
+    LatentSpec latent;
+    MinGruSpec gru;
+    int ff = 0;  // width of the feed-forward, 0: the layer has none
+};
+
+// Layers start .. stop - 1 run `times` times in a row, every pass with a cache and a state of its own.  A pass begins with
+// x <- W_in [x; x0] + step[pass], x0 being the embedding output.
+struct LoopSpec {
+    int start = 0, stop = 0, times = 0;  // times = 0: no loop
+};
+
+// One execution of a layer: pass < 0 outside of the loop; first: the layer a pass begins with.
+struct LayerRun {
+    int layer = 0, pass = -1;
+    bool first = false;
 };
 
 struct MixerSpec {
@@ -60,7 +88,15 @@ struct MixerSpec {
     int vocab = 0, width = 0, side_dim = 0;
     float eps = 1e-6f;
     NormKind norm = NormKind::DynTanh;
+    FfKind ff_kind = FfKind::Gated;
+    // false: mixer and feed-forward one after the other, a norm in front of each.  true: both read one normed row and their sum
+    // is added; the mixer's input is mixed with the previous token's normed row (token shift).
+    bool side_by_side = false;
+    bool sinusoid_positions = false;  // added to the embedding, which a norm then follows
+    float logit_scale = 1.f;
+    LoopSpec loop;
     std::vector<MixerLayerSpec> layers;
+    std::vector<LayerRun> runs() const;  // in the order of execution
 };
 
 // Reads `config` (and sizes that only the tensors know) for the architecture it names.

@@ -33,12 +33,22 @@ struct Shares {
 #endif
 };
 
-// A matmul's input rows [rows][ld]: bfloat16 (h) or f32 (f), whichever is set.  Columns from the matrix's true width up to ld are
-// zeros, written by the kernel that makes the rows.
+// A matmul's input rows [rows][ld]: bfloat16 (h) or f32 (f), whichever is set.  Columns from the matrix's true width up to end()
+// are zeros, written by the kernel that makes the rows.  A row may be made of parts with an image each (part()), one after the
+// other.
 struct RowImage {
     __nv_bfloat16* h = nullptr;
     float* f = nullptr;
     int ld = 0;
+    int cols = 0;  // columns of this part, 0: the whole row
+    __host__ __device__ int end() const { return cols > 0 ? cols : ld; }
+    RowImage part(int first, int n) const {
+        RowImage r = *this;
+        if (r.h != nullptr) r.h += first;
+        if (r.f != nullptr) r.f += first;
+        r.cols = n;
+        return r;
+    }
 #ifdef __CUDACC__
     __device__ __forceinline__ bool any() const { return h != nullptr || f != nullptr; }
     __device__ __forceinline__ void put(int64_t row, int col, float v) const {

@@ -139,7 +139,7 @@ class Model:
         """Host-only audit of a safetensors checkpoint folder; raises MkError with the loader's message.  Needs no GPU."""
         s = capi.MixerSummary()
         capi.check(capi.lib().mk_mixer_inspect(str(path).encode(), C.byref(s)))
-        out = {name: getattr(s, name) for name, _ in capi.MixerSummary._fields_ if name != "reserved_"}
+        out = {name: getattr(s, name) for name, _ in capi.MixerSummary._fields_}
         out["architecture"] = s.architecture.decode()
         return out
 
@@ -258,7 +258,7 @@ class Model:
         capi.check(capi.lib().mk_model_capture_residuals(self._h, 1 if on else 0))
 
     def residuals(self, n_tokens: int) -> np.ndarray:
-        """[layers, tokens, hidden] of the last forward, which ran `n_tokens` tokens."""
+        """[layer runs, tokens, hidden] of the last forward, which ran `n_tokens` tokens."""
         sp = self.spec()
         out = np.empty((sp.n_layers, n_tokens, sp.hidden_size), np.float32)
         n = C.c_int32()

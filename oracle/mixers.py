@@ -1,4 +1,4 @@
-"""Plain NumPy statement of the mixer-built decoders (the Sizilorn design and its parts), test infrastructure only.
+"""Plain NumPy statement of the mixer-built decoders (the Sizilorn and Kunonex designs and their parts), test infrastructure only.
 
 One function per mechanism, whole sequences at once, float64 unless the caller passes other arrays; recurrences are written
 token by token.  Nothing here is shared with the CUDA path.  Shapes: x, h [T, width]; a head-wise array [T, heads, dim].
@@ -35,6 +35,23 @@ def rms(x, eps):
 
 def dyn_tanh(x, alpha, w, b):
     return np.tanh(alpha * x) * w + b
+
+
+def layer_norm(x, w, eps):
+    """Mean taken off, divided by the standard deviation (eps inside the root), times w."""
+    c = x - np.mean(x, axis=-1, keepdims=True)
+    return c / np.sqrt(np.mean(c * c, axis=-1, keepdims=True) + eps) * w
+
+
+# ------------------------------------------------------------------------------------------------ absolute positions
+
+def sinusoid(positions, width):
+    """[positions, width]: sine in the even columns and cosine in the odd ones, column pair i turning at 10000^(-2i / width)."""
+    out = np.zeros((len(positions), width))
+    for c in range(width):
+        a = np.asarray(positions, np.float64) * 10000.0 ** (-2.0 * (c // 2) / width)
+        out[:, c] = np.cos(a) if c % 2 else np.sin(a)
+    return out
 
 
 # ------------------------------------------------------------------------------------------------ rotation
@@ -100,6 +117,17 @@ def gated_attention(h, W, cfg, eps):
     o = causal_attention(q, k, v, cfg["scale"])
     o = o * sigmoid(h @ W["g"].T)[:, :, None]
     return o.reshape(T, H * e) @ W["o"].T
+
+
+def latent_attention(h, W, cfg, eps):
+    """Attention whose keys and values are projections of one small vector per token; no positions; a gate per head."""
+    T, H = h.shape[0], cfg["heads"]
+    q = (rms(h @ W["dq"].T, eps) * W["dq.norm"]) @ W["uq"].T
+    c = rms(h @ W["dkv"].T, eps) * W["dkv.norm"]
+    k, v = c @ W["uk"].T, c @ W["uv"].T
+    o = causal_attention(q.reshape(T, H, cfg["dim"]), k.reshape(T, H, cfg["dim"]), v.reshape(T, H, cfg["vdim"]), cfg["scale"])
+    o = o * sigmoid(h @ W["g"].T)[:, :, None]
+    return o.reshape(T, H * cfg["vdim"]) @ W["o"].T
 
 
 # ------------------------------------------------------------------------------------------------ gated delta rule
@@ -189,7 +217,35 @@ def wkv_mixer(h, W, cfg, eps):
     return (rms(o, eps).reshape(T, H * d) * W["norm"] * silu(mix["g"] @ W["g"].T)) @ W["o"].T
 
 
+# ------------------------------------------------------------------------------------------------ minGRU
+
+def min_gru(z, u, state=None):
+    """z (gate, in 0..1) and u (candidate before its activation), [T, n].  Returns (S [T, n], last S)."""
+    S = np.zeros(z.shape[1], z.dtype) if state is None else state.copy()
+    out = np.empty_like(z)
+    for t in range(z.shape[0]):
+        cand = np.where(u[t] >= 0, u[t] + 0.5, sigmoid(u[t]))
+        S = (1.0 - z[t]) * S + z[t] * cand
+        out[t] = S
+    return out, S
+
+
+def mingru_mixer(h, W, cfg, eps):
+    S, _ = min_gru(sigmoid(h @ W["z"].T + W["z.b"]), h @ W["x"].T + W["x.b"])
+    return (S * silu(h @ W["g"].T)) @ W["o"].T
+
+
 # ------------------------------------------------------------------------------------------------ feed-forward, token input
+
+def poly_norm(z, act, eps):
+    """A cubic of z whose powers are each divided by their own root mean square first."""
+    a, b, c, e = act
+    return a * rms(z, eps) + b * rms(z ** 2, eps) + c * rms(z ** 3, eps) + e
+
+
+def poly_mlp(h, W, eps):
+    return poly_norm(h @ W["up"].T + W["up.b"], W["act"], eps) @ W["down"].T + W["down.b"]
+
 
 def gated_mlp(h, W):
     return (silu(h @ W["gate"].T) * (h @ W["up"].T)) @ W["down"].T
@@ -237,6 +293,50 @@ class MixerDecoder:
 
     def logits(self, tokens):
         return self._norm("final.norm", self.residuals(tokens)[-1]) @ self.w["head"].T
+
+
+class KunonexDecoder(MixerDecoder):
+    """Sinusoidal positions, layers whose mixer and feed-forward read one layer norm side by side, a token shift in front of
+    every mixer, and a run of layers that is passed through several times."""
+
+    def _norm(self, name, x):
+        return layer_norm(x, self.w[name], self.cfg["norm"]["eps"])
+
+    def schedule(self):
+        """(layer, pass) in the order of execution; pass is None outside of the loop."""
+        n, loop = len(self.cfg["layers"]), self.cfg.get("loop")
+        if not loop:
+            return [(i, None) for i in range(n)]
+        a, b = loop["start"], loop["stop"]
+        return ([(i, None) for i in range(a)] + [(i, t) for t in range(loop["times"]) for i in range(a, b)] + [(i, None) for i in range(b, n)])
+
+    def embedding_output(self, tokens):
+        return self._norm("embed.norm", self.w["embed"][tokens] + sinusoid(np.arange(len(tokens)), self.cfg["width"]))
+
+    def residuals(self, tokens):
+        """The residual stream after every layer run: [layer runs, T, width]."""
+        eps = self.cfg["norm"]["eps"]
+        x0 = x = self.embedding_output(np.asarray(tokens))
+        out = []
+        for i, t in self.schedule():
+            if t is not None and i == self.cfg["loop"]["start"]:
+                x = np.concatenate([x, x0], axis=1) @ self.w["loop.in"].T + self.w["loop.step"][t]
+            p, layer = f"l{i}.", self.cfg["layers"][i]
+            h = self._norm(p + "norm1", x)
+            mixer = {"mingru": mingru_mixer, "latent_attention": latent_attention}[layer["type"]]
+            y = mixer(token_shift(h, self.w[p + "shift"]), self._sub(p + "mix."), layer["mixer"], eps)
+            if layer.get("mlp"):
+                y = y + poly_mlp(h, self._sub(p + "mlp."), eps)
+            x = x + y
+            out.append(x)
+        return np.stack(out)
+
+    def logits(self, tokens):
+        return super().logits(tokens) * self.cfg["logit_scale"]
+
+
+def decoder(config, tensors, dtype=np.float64):
+    return {"Sizilorn": MixerDecoder, "Kunonex": KunonexDecoder}[config["architecture"]](config, tensors, dtype)
 
 
 def read_safetensors(path):
