@@ -27,7 +27,8 @@ has no exchange step for them); the sparse-MoE workload runs expert parallelism 
 serves its own requests and each MoE layer exchanges the routed rows (`config.ep`; `--ep off` for replicas).  The
 reported time is the max over ranks.  `--http-clients N` adds a step through the `/completion` endpoint (`http` key),
 `--microbench` prints the Q4_K matmul GB/s of the decode shapes instead, `--mixer` the prefill and decode throughput of
-mixer-built decoders (Sizilorn layers at real-model sizes, random weights) beside the closest GGUF family of equal size.
+a mixer-built decoder design (`--mixer sizilorn`, the default, or `--mixer kunonex`; layers at real-model sizes, random weights)
+beside the closest GGUF family of equal size.
 """
 from __future__ import annotations
 
@@ -641,7 +642,8 @@ def main():
                          "resident; N > 1: expert parallelism over the same ranks)")
     ap.add_argument("--no-profiled-step", action="store_true", help="skip the extra step that times every launch")
     ap.add_argument("--microbench", action="store_true", help="Q4_K matmul GB/s on the decode shapes instead of the workload")
-    ap.add_argument("--mixer", action="store_true", help="prefill / decode throughput of mixer-built decoders beside the closest GGUF family instead of the workload")
+    ap.add_argument("--mixer", nargs="?", const="sizilorn", choices=["sizilorn", "kunonex"],
+                    help="prefill / decode throughput of a mixer-built decoder design beside the closest GGUF family instead of the workload")
     args = ap.parse_args()
 
     rank, local, world, dist = dist_setup(args.gpus)
@@ -677,7 +679,7 @@ def main():
             bench = importlib.import_module("macllm_infer_b200.mixer_bench")
             sampler = ClockSampler(local)
             sampler.start()
-            results = bench.run(peaks(), max(3, args.warmup), max(5, args.steps))
+            results = bench.run(peaks(), max(3, args.warmup), max(5, args.steps), args.mixer)
             print(json.dumps(dict(metric="mixer decoders: device tokens/s", unit=UNIT, data="synthetic", dtype="bf16", results=results, clocks=sampler.stop())))
         return
 

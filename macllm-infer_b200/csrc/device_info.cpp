@@ -6,7 +6,7 @@
 namespace mk {
 
 void ensure_dynamic_smem(const void* func, size_t bytes) {
-    if (bytes <= 48 * 1024) return;
+    if (bytes <= 32 * 1024) return;  // 48 KB need no opt-in, the kernel's static shared memory included
     static std::mutex mu;
     static std::map<std::pair<const void*, int>, size_t> done;
     int dev = 0;

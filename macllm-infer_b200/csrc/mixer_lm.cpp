@@ -98,7 +98,7 @@ void MixerLm::upload_matrix(const std::vector<float>& m, int64_t rows, int ld, i
     else if (groups > 0) build_bf16_weight_groups(m.data(), rows, ld, groups, out.half, stream_);
     else build_bf16_weight(m.data(), rows, ld, out.half, stream_, group_rows);
     spec_.weight_bytes += out.bytes;
-    if (per_token) spec_.weight_bytes_per_token += out.bytes;
+    if (per_token) spec_.weight_bytes_per_token += out.bytes * passes_;
 }
 
 void MixerLm::upload_dense(const SafetensorsFile& f, const std::vector<Part>& parts, int64_t rows, int cols, Dense& out,
@@ -184,10 +184,15 @@ void MixerLm::load(const SafetensorsFile& f) {
         std::vector<float> m((size_t)C * 2 * second, 0.f);
         for (int r = 0; r < C; ++r)
             for (int h = 0; h < 2; ++h) memcpy(&m[((size_t)r * 2 + h) * second], &w[((size_t)r * 2 + h) * C], (size_t)C * 4);
+        passes_ = ms_.loop.times;
         upload_matrix(m, C, 2 * second, (int64_t)2 * C * C * esz_, loop_in_, {}, 0);
         upload_f32(f.values("loop.step", {ms_.loop.times, C}), loop_step_);
     }
-    for (int l = 0; l < (int)ms_.layers.size(); ++l) load_layer(f, l);
+    for (int l = 0; l < (int)ms_.layers.size(); ++l) {
+        passes_ = (int)std::count_if(runs_.begin(), runs_.end(), [&](const LayerRun& r) { return r.layer == l; });
+        load_layer(f, l);
+    }
+    passes_ = 1;
     upload_norm(f, "final.norm", final_norm_);
     upload_dense(f, {{"head", ms_.vocab, 0}}, ms_.vocab, C, head_);
 }

@@ -128,6 +128,7 @@ private:
     // `groups` > 0: equal parts with an input each.  per_token: counted in the bytes of a token's pass.
     void upload_matrix(const std::vector<float>& m, int64_t rows, int ld, int64_t true_bytes, Dense& out, const std::vector<int64_t>& group_rows, int groups,
                        bool per_token = true);
+    int passes_ = 1;  // how often a token's pass runs what is being loaded
     void place(const SafetensorsFile& f, const Part& p, int cols, int ld, std::vector<float>& m);
     void upload_f32(const std::vector<float>& v, DevBuf& out);
     void upload_norm(const SafetensorsFile& f, const std::string& name, Norm& out);

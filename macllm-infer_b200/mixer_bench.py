@@ -1,5 +1,6 @@
 """Throughput of mixer-built decoders (random weights, layers of real-model sizes) beside the closest GGUF family of the same
-width, heads, feed-forward and layer count with dense BF16 matrices.  Used by `bench.py --mixer`.
+width, heads, feed-forward and layer count (looped layers counted once per pass) with dense BF16 matrices.  Used by
+`bench.py --mixer`.
 
 Every figure is device time (CUDA events around the tick, median over the timed ticks); the weights of a tick are several
 times the L2.  The per-class table comes from separate ticks with an event pair around every launch; `roofline` there is the
@@ -44,7 +45,42 @@ SHAPES = [
 ]
 
 
-def config_of(s: Shape) -> dict:
+@dataclass
+class BesideShape:
+    """Pairs of latent-attention and minGRU layers with the feed-forward beside the mixer; `loop` = (start, stop, times)."""
+    name: str
+    width: int
+    pairs: int
+    loop: tuple
+    heads: int
+    dim: int
+    q_rank: int
+    kv_rank: int
+    gru: int
+    ff: int
+    kv_heads: int        # of the closest model
+    vocab: int = 32000
+
+    @property
+    def runs(self) -> int:
+        a, b, n = self.loop
+        return 2 * self.pairs + (b - a) * (n - 1)
+
+
+BESIDE_SHAPES = [
+    BesideShape("w2048", 2048, 3, (2, 4, 2), 16, 128, 1024, 512, 2048, 8192, 4),
+    BesideShape("w4096", 4096, 1, (0, 2, 2), 32, 128, 1536, 512, 4096, 12288, 8),
+]
+
+
+def config_of(s) -> dict:
+    if isinstance(s, BesideShape):
+        mlp = {"kind": "dense", "ff": s.ff}
+        lat = {"type": "latent_attention", "mlp": mlp, "mixer": {"heads": s.heads, "dim": s.dim, "vdim": s.dim, "q_rank": s.q_rank, "kv_rank": s.kv_rank,
+                                                                 "scale": s.dim ** -0.5}}
+        gru = {"type": "mingru", "mlp": mlp, "mixer": {"width": s.gru}}
+        return {"architecture": "Kunonex", "vocab": s.vocab, "width": s.width, "norm": {"eps": 1e-6}, "logit_scale": 1.0,
+                "loop": dict(zip(("start", "stop", "times"), s.loop)), "layers": [lat, gru] * s.pairs}
     mlp = {"kind": "dense", "ff": s.ff}
     wkv = {"type": "wkv", "mixer": {"heads": s.wkv_heads, "dim": s.wkv_dim}, "mlp": mlp}
     par = {"type": "parallel", "mlp": mlp, "mixer": {
@@ -55,9 +91,10 @@ def config_of(s: Shape) -> dict:
             "layers": [wkv, par] * s.pairs}
 
 
-def tensor_shapes(s: Shape) -> dict[str, tuple]:
+def tensor_shapes(s) -> dict[str, tuple]:
     """name -> (shape, mean, deviation)."""
     C, V, out = s.width, s.vocab, {}
+    beside = isinstance(s, BesideShape)
 
     def mat(name, rows, cols):
         out[name] = ((rows, cols), 0.0, cols ** -0.5)
@@ -67,10 +104,44 @@ def tensor_shapes(s: Shape) -> dict[str, tuple]:
 
     def norm(name):
         vec(name, C)
-        vec(name + ".b", C, mean=0.0)
-        vec(name + ".alpha", mean=0.7, dev=0.0)
+        if not beside:
+            vec(name + ".b", C, mean=0.0)
+            vec(name + ".alpha", mean=0.7, dev=0.0)
 
     out["embed"] = ((V, C), 0.0, 1.0)
+    if beside:
+        norm("embed.norm")
+        mat("loop.in", C, 2 * C)
+        vec("loop.step", s.loop[2], C, mean=0.0)
+        for i in range(2 * s.pairs):
+            p = f"l{i}."
+            norm(p + "norm1")
+            vec(p + "shift", C, mean=0.5)
+            if i % 2 == 0:
+                n = s.heads * s.dim
+                mat(p + "mix.dq", s.q_rank, C)
+                vec(p + "mix.dq.norm", s.q_rank)
+                mat(p + "mix.uq", n, s.q_rank)
+                mat(p + "mix.dkv", s.kv_rank, C)
+                vec(p + "mix.dkv.norm", s.kv_rank)
+                mat(p + "mix.uk", n, s.kv_rank)
+                mat(p + "mix.uv", n, s.kv_rank)
+                mat(p + "mix.g", s.heads, C)
+                mat(p + "mix.o", C, n)
+            else:
+                for x in "zxg":
+                    mat(p + "mix." + x, s.gru, C)
+                vec(p + "mix.z.b", s.gru, mean=-2.0, dev=1.0)
+                vec(p + "mix.x.b", s.gru, mean=0.0)
+                mat(p + "mix.o", C, s.gru)
+            mat(p + "mlp.up", s.ff, C)
+            vec(p + "mlp.up.b", s.ff, mean=0.0)
+            mat(p + "mlp.down", C, s.ff)
+            vec(p + "mlp.down.b", C, mean=0.0)
+            vec(p + "mlp.act", 4, mean=0.5)
+        norm("final.norm")
+        mat("head", V, C)
+        return out
     out["side.embed"] = ((V, 2 * s.pairs * s.side), 0.0, 1.0)
     for i in range(2 * s.pairs):
         p = f"l{i}."
@@ -120,7 +191,7 @@ def tensor_shapes(s: Shape) -> dict[str, tuple]:
     return out
 
 
-def write_checkpoint(folder: Path, s: Shape) -> Path:
+def write_checkpoint(folder: Path, s) -> Path:
     """A random checkpoint; big matrices repeat one block of random numbers."""
     folder.mkdir(parents=True, exist_ok=True)
     (folder / "config.json").write_text(json.dumps(config_of(s)))
@@ -141,8 +212,9 @@ def write_checkpoint(folder: Path, s: Shape) -> Path:
     return folder
 
 
-def closest_spec(s: Shape) -> seed_gguf.SeedSpec:
-    return seed_gguf.SeedSpec("qwen3", 2 * s.pairs, s.width, s.heads, s.kv_heads, s.dim, s.ff, s.vocab, context=16384, theta=1e6, eps=1e-6,
+def closest_spec(s) -> seed_gguf.SeedSpec:
+    layers = s.runs if isinstance(s, BesideShape) else 2 * s.pairs
+    return seed_gguf.SeedSpec("qwen3", layers, s.width, s.heads, s.kv_heads, s.dim, s.ff, s.vocab, context=16384, theta=1e6, eps=1e-6,
                               matrix_type=capi.TYPE_BF16, high_type=capi.TYPE_BF16, name=f"closest-{s.name}")
 
 
@@ -206,14 +278,18 @@ def measure(model, vocab: int, prompt: int, lanes: int, context: int, warmup: in
     return out
 
 
-def run(peaks: dict, warmup: int, steps: int, prompt=2048, lanes=64, context=1024) -> list[dict]:
+DESIGNS = {"sizilorn": ("Sizilorn", SHAPES), "kunonex": ("Kunonex", BESIDE_SHAPES)}
+
+
+def run(peaks: dict, warmup: int, steps: int, design="sizilorn", prompt=2048, lanes=64, context=1024) -> list[dict]:
+    title, shapes = DESIGNS[design]
     results = []
     capacity = lanes * (context + 256)
     with tempfile.TemporaryDirectory() as tmp:
-        for s in SHAPES:
+        for s in shapes:
             kw = dict(kv_capacity_tokens=capacity, max_batch_tokens=max(prompt, 2 * context), max_batch_lanes=lanes)
-            for kind in ("sizilorn", "closest"):
-                if kind == "sizilorn":
+            for kind in (design, "closest"):
+                if kind == design:
                     path = write_checkpoint(Path(tmp) / s.name, s)
                     model = engine.Model.load(path, state_slots=lanes + 1, **kw)
                     weights = model.spec().weight_bytes_per_token
@@ -223,7 +299,7 @@ def run(peaks: dict, warmup: int, steps: int, prompt=2048, lanes=64, context=102
                     weights = seed_gguf.weight_bytes(closest_spec(s))["per_token"]
                 r = measure(model, s.vocab, prompt, lanes, context, warmup, steps, peaks)
                 sp = model.spec()
-                results.append(dict(shape=s.name, model="Sizilorn" if kind == "sizilorn" else "qwen3 family, dense BF16 matrices", layers=int(sp.n_layers),
+                results.append(dict(shape=s.name, model=title if kind == design else "qwen3 family, dense BF16 matrices", layers=int(sp.n_layers),
                                     width=int(sp.hidden_size), weight_gb=round(weights / 1e9, 3), **r))
                 model.close()
     return results

@@ -272,12 +272,15 @@ class MixerDecoder:
     def _norm(self, name, x):
         return dyn_tanh(x, self.w[name + ".alpha"], self.w[name], self.w[name + ".b"])
 
+    def embedding_output(self, tokens):
+        return self.w["embed"][tokens]
+
     def residuals(self, tokens):
         """The residual stream after every layer: [layers, T, width]."""
         tokens = np.asarray(tokens)
         eps = self.cfg["norm"]["eps"]
         side = self.cfg.get("token_side")
-        x = self.w["embed"][tokens]
+        x = self.embedding_output(tokens)
         out = []
         for i, layer in enumerate(self.cfg["layers"]):
             p = f"l{i}."

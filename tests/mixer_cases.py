@@ -24,13 +24,82 @@ def parallel(left, right, ff=0):
             "mlp": {"kind": "dense", "ff": ff} if ff else None}
 
 
+def mingru(width, ff=0):
+    return {"type": "mingru", "mixer": {"width": width}, "mlp": {"kind": "dense", "ff": ff} if ff else None}
+
+
+def latent(heads, dim, vdim, q_rank, kv_rank, ff=0):
+    return {"type": "latent_attention", "mlp": {"kind": "dense", "ff": ff} if ff else None,
+            "mixer": {"heads": heads, "dim": dim, "vdim": vdim, "q_rank": q_rank, "kv_rank": kv_rank, "scale": 0.9 / dim ** 0.5}}
+
+
+def kunonex(layers, width=96, vocab=131, loop=None, eps=3e-5, logit_scale=0.7):
+    """loop = (start, stop, times)."""
+    return {"architecture": "Kunonex", "vocab": vocab, "width": width, "norm": {"eps": eps}, "logit_scale": logit_scale,
+            "loop": dict(zip(("start", "stop", "times"), loop)) if loop else None, "layers": layers}
+
+
 def config(layers, width=96, vocab=131, side=12, eps=3e-5):
     return {"architecture": "Sizilorn", "vocab": vocab, "width": width, "norm": {"eps": eps},
             "token_side": {"dim": side} if side else None, "layers": layers}
 
 
+def kunonex_weights(cfg, seed):
+    rng = np.random.default_rng(seed)
+    C, V = cfg["width"], cfg["vocab"]
+    w = {}
+
+    def mat(name, rows, cols, gain=1.0):
+        w[name] = rng.standard_normal((rows, cols)) * gain / np.sqrt(cols)
+
+    def around_one(name, n):
+        w[name] = 1.0 + 0.3 * rng.standard_normal(n)
+
+    def bias(name, n, dev=0.3):
+        w[name] = dev * rng.standard_normal(n)
+
+    w["embed"] = rng.standard_normal((V, C))
+    around_one("embed.norm", C)
+    if cfg["loop"]:
+        mat("loop.in", C, 2 * C)
+        bias("loop.step", (cfg["loop"]["times"], C))
+    for i, layer in enumerate(cfg["layers"]):
+        p, m = f"l{i}.", layer["mixer"]
+        around_one(p + "norm1", C)
+        w[p + "shift"] = rng.uniform(0, 1, C)
+        if layer["type"] == "mingru":
+            n = m["width"]
+            for s in "zxg":
+                mat(p + "mix." + s, n, C)
+            w[p + "mix.z.b"] = rng.uniform(-5.0, 1.0, n)
+            bias(p + "mix.x.b", n)
+            mat(p + "mix.o", C, n)
+        else:
+            mat(p + "mix.dq", m["q_rank"], C)
+            around_one(p + "mix.dq.norm", m["q_rank"])
+            mat(p + "mix.uq", m["heads"] * m["dim"], m["q_rank"], 2.0)
+            mat(p + "mix.dkv", m["kv_rank"], C)
+            around_one(p + "mix.dkv.norm", m["kv_rank"])
+            mat(p + "mix.uk", m["heads"] * m["dim"], m["kv_rank"], 1.5)
+            mat(p + "mix.uv", m["heads"] * m["vdim"], m["kv_rank"])
+            mat(p + "mix.g", m["heads"], C)
+            mat(p + "mix.o", C, m["heads"] * m["vdim"])
+        if layer["mlp"]:
+            ff = layer["mlp"]["ff"]
+            mat(p + "mlp.up", ff, C)
+            bias(p + "mlp.up.b", ff)
+            mat(p + "mlp.down", C, ff)
+            bias(p + "mlp.down.b", C)
+            w[p + "mlp.act"] = np.array([0.6, 0.4, -0.3, 0.2]) + 0.1 * rng.standard_normal(4)
+    around_one("final.norm", C)
+    mat("head", V, C)
+    return w
+
+
 def weights(cfg, seed=0, rank=5):
     """name -> float32 array holding bfloat16 values."""
+    if cfg["architecture"] == "Kunonex":
+        return {k: mixers.bf16(np.asarray(v, np.float32)) for k, v in kunonex_weights(cfg, seed).items()}
     rng = np.random.default_rng(seed)
     C, V, side = cfg["width"], cfg["vocab"], (cfg.get("token_side") or {}).get("dim", 0)
     w = {}

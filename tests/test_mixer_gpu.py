@@ -33,7 +33,7 @@ def checkpoint(tmp_path, cfg, seed=0, rank=5, change=None):
     if change:
         change(w)
         w = {k: mixers.bf16(np.asarray(v, np.float32)) for k, v in w.items()}
-    return mc.write(tmp_path / "m", cfg, w), mixers.MixerDecoder(cfg, w)
+    return mc.write(tmp_path / "m", cfg, w), mixers.decoder(cfg, w)
 
 
 def tokens_of(n, vocab, seed=3):
@@ -70,28 +70,86 @@ ALONE = {
 }
 
 
-@pytest.mark.parametrize("compute", DTYPES)
-@pytest.mark.parametrize("name", ALONE)
-def test_mechanism_alone(mk, tmp_path, name, compute):
+ALONE_BESIDE = {
+    # name: (layer, width, what is silenced)
+    "minGRU": (mc.mingru(70), 96, ()),
+    "minGRU wide state": (mc.mingru(300), 40, ()),
+    "minGRU few odd channels": (mc.mingru(5), 67, ()),
+    "minGRU beside a feed-forward": (mc.mingru(33, ff=90), 100, ()),
+    "latent odd sizes": (mc.latent(3, 40, 24, 33, 50), 70, ()),
+    "latent 128, wide values": (mc.latent(5, 20, 100, 12, 128), 96, ()),
+    "latent 256, twenty heads": (mc.latent(20, 16, 30, 40, 200), 64, ()),
+    "latent 512, one head": (mc.latent(1, 130, 70, 7, 300), 64, ()),
+    "latent 512, thirty heads": (mc.latent(30, 8, 8, 24, 512), 64, ()),
+    "latent, more than one head group": (mc.latent(37, 9, 12, 20, 30), 64, ()),
+    "latent, heads too wide to expand": (mc.latent(2, 270, 20, 30, 64), 64, ()),
+    "latent above the tensor-core kernel": (mc.latent(2, 24, 32, 30, 600), 64, ()),
+    "latent beside a feed-forward": (mc.latent(4, 64, 64, 50, 70, ff=130), 96, ()),
+    "feed-forward": (mc.mingru(8, ff=200), 66, ("l0.mix.o",)),
+    "feed-forward, odd width": (mc.latent(1, 8, 8, 8, 8, ff=37), 67, ("l0.mix.o",)),
+}
+
+
+def check_alone(folder, oracle, compute):
     """The residual stream after a layer with one mechanism at work, for a whole prompt, portions and single tokens."""
-    layer, width, side, silenced, rank = ALONE[name]
-    cfg = mc.config([layer], width=width, side=side)
-    folder, oracle = checkpoint(tmp_path, cfg, seed=7, rank=rank, change=silence(*silenced))
-    toks = tokens_of(75, cfg["vocab"])
+    toks = tokens_of(75, oracle.cfg["vocab"])
+    base = oracle.embedding_output(toks)
     want = oracle.residuals(toks)[0]
-    delta = want - oracle.w["embed"][toks]          # what the layer adds: the part under test
+    delta = want - base          # what the layer adds: the part under test
     model = mc.load(folder, compute)
     model.capture_residuals(True)
-    for portions in ([75], mc.cut(75, [2, 17, 1, 5, 33]), mc.cut(75, [1])):
+    for portions in ([75], mc.cut(75, [2, 17, 1, 5, 33]), mc.cut(75, [34, 2, 39]), mc.cut(75, [1])):
         s, at, got = model.new_session(), 0, []
         for k in portions:
             model.forward_batch([(s, toks[at:at + k], at)], want_logits=False, want_tokens=False, rows=[[]])
             got.append(model.residuals(k)[0])
             at += k
         s.close()
-        got = np.concatenate(got) - oracle.w["embed"][toks]
+        got = np.concatenate(got) - base
         e = np.sqrt(np.mean((got - delta) ** 2, axis=1) / np.mean(delta ** 2))
         assert e.max() <= mc.LIMIT[compute], f"{portions[:5]}: token {int(e.argmax())} off by {e.max():.2e}"
+    model.close()
+
+
+@pytest.mark.parametrize("compute", DTYPES)
+@pytest.mark.parametrize("name", ALONE)
+def test_mechanism_alone(mk, tmp_path, name, compute):
+    layer, width, side, silenced, rank = ALONE[name]
+    cfg = mc.config([layer], width=width, side=side)
+    check_alone(*checkpoint(tmp_path, cfg, seed=7, rank=rank, change=silence(*silenced)), compute)
+
+
+@pytest.mark.parametrize("compute", DTYPES)
+@pytest.mark.parametrize("name", ALONE_BESIDE)
+def test_mechanism_alone_in_layers_with_one_norm(mk, tmp_path, name, compute):
+    layer, width, silenced = ALONE_BESIDE[name]
+    check_alone(*checkpoint(tmp_path, mc.kunonex([layer], width=width), seed=7, change=silence(*silenced)), compute)
+
+
+@pytest.mark.parametrize("compute", DTYPES)
+def test_token_shift_reaches_the_mixer_only(mk, tmp_path, compute):
+    """A shift of one: the mixer sees nothing but the token before (zeros at first), the feed-forward nothing but the token."""
+    cfg = mc.kunonex([mc.mingru(20, ff=30)], width=50, vocab=40)
+
+    def change(w):
+        w["l0.shift"][:] = 1.0
+
+    folder, oracle = checkpoint(tmp_path, cfg, seed=9, change=change)
+    check_alone(folder, oracle, compute)
+
+
+@pytest.mark.parametrize("compute", DTYPES)
+@pytest.mark.parametrize("width", [64, 67])
+def test_sinusoidal_positions_far_out(mk, tmp_path, width, compute):
+    """The embedding output at positions up to the thousands: the layer adds nothing, so the stream after it is that output."""
+    cfg = mc.kunonex([mc.mingru(4)], width=width, vocab=20)
+    folder, oracle = checkpoint(tmp_path, cfg, seed=2, change=silence("l0.mix.o"))
+    toks = tokens_of(3000, 20)
+    model = mc.load(folder, compute, capacity=3008)
+    model.capture_residuals(True)
+    s = model.new_session()
+    model.forward_batch([(s, toks, 0)], want_logits=False, want_tokens=False, rows=[[]])
+    assert np.abs(model.residuals(3000)[0] - oracle.embedding_output(toks)).max() < 1e-5
     model.close()
 
 
@@ -101,6 +159,12 @@ MODELS = {
     "first": (mc.config([mc.wkv(3, 40), mc.parallel((4, 2, 64, 64, 32, True), (4, 2, 32, 48, 4), ff=150), mc.wkv(2, 64, ff=90)], width=104), 9),
     "second": (mc.config([mc.parallel((6, 2, 36, 20, 12, False), (3, 3, 48, 40, 2)), mc.wkv(5, 16), mc.parallel((8, 1, 32, 32, 32, True), (2, 2, 64, 64, 3), ff=64)],
                          width=67, vocab=201, side=5, eps=1e-5), 4),
+    "looped": (mc.kunonex([mc.mingru(40, ff=50), mc.latent(4, 32, 48, 30, 60, ff=150), mc.mingru(72), mc.latent(6, 20, 36, 24, 90)], width=104,
+                          loop=(1, 3, 3)), 0),
+    "loop over all layers": (mc.kunonex([mc.latent(2, 70, 20, 48, 130), mc.mingru(33, ff=41)], width=67, vocab=201, loop=(0, 2, 2), eps=1e-5,
+                                        logit_scale=1.3), 0),
+    "no loop": (mc.kunonex([mc.mingru(24, ff=60), mc.latent(20, 16, 16, 64, 40, ff=60)], width=64, logit_scale=1.0), 0),
+    "a loop of one pass": (mc.kunonex([mc.latent(3, 24, 24, 24, 24), mc.mingru(50, ff=32)], width=48, loop=(1, 2, 1)), 0),
     "time mixing only": (mc.config([mc.wkv(2, 32), mc.wkv(1, 72)], width=64, side=64), 20),
 }
 
@@ -113,7 +177,7 @@ def built(tmp_path_factory):
         if name not in made:
             cfg, rank = MODELS[name]
             w = mc.weights(cfg, seed=11, rank=rank)
-            made[name] = (mc.write(tmp_path_factory.mktemp("mixer") / "m", cfg, w), mixers.MixerDecoder(cfg, w), cfg)
+            made[name] = (mc.write(tmp_path_factory.mktemp("mixer") / "m", cfg, w), mixers.decoder(cfg, w), cfg)
         return made[name]
     return get
 
@@ -131,10 +195,14 @@ def test_prompt_portions_and_decoding_agree(mk, built, name, compute):
     model.close()
 
 
+BOTH = ["first", "looped"]   # a model of each layer form
+
+
 @pytest.mark.parametrize("compute", DTYPES)
-def test_unequal_batches_against_each_alone(mk, built, compute):
+@pytest.mark.parametrize("name", BOTH)
+def test_unequal_batches_against_each_alone(mk, built, name, compute):
     """Four sequences of different lengths, portions of some beside single tokens of others, one of them paused for a while."""
-    folder, oracle, cfg = built("first")
+    folder, oracle, cfg = built(name)
     seqs = [tokens_of(n, cfg["vocab"], seed=20 + n) for n in (130, 40, 3, 77)]
     want = [oracle.logits(t) for t in seqs]
     model = mc.load(folder, compute)
@@ -165,9 +233,10 @@ def test_unequal_batches_against_each_alone(mk, built, compute):
 
 
 @pytest.mark.parametrize("compute", DTYPES)
-def test_pages_and_slots_are_used_again(mk, built, compute):
+@pytest.mark.parametrize("name", BOTH)
+def test_pages_and_slots_are_used_again(mk, built, name, compute):
     """A pool and a slot array that only just hold the live sequences: every later one runs in what an earlier one left."""
-    folder, oracle, cfg = built("first")
+    folder, oracle, cfg = built(name)
     model = mc.load(folder, compute, capacity=128, lanes=2, slots=2)
     held = model.new_session()
     a = tokens_of(40, cfg["vocab"], seed=1)
@@ -225,6 +294,86 @@ def test_one_far_key_stands_out(mk, tmp_path, left, compute):
 
 
 @pytest.mark.parametrize("compute", DTYPES)
+@pytest.mark.parametrize("latent", [(4, 32, 48, 40, 40), (20, 24, 24, 100, 100), (2, 64, 64, 300, 300)])
+def test_one_far_key_stands_out_of_the_latents(mk, tmp_path, latent, compute):
+    """As above for latent attention: the query latent is the key latent of the embedding with its halves exchanged, and the
+    embeddings are large against the positions.  Histories of more than a few hundred keys are cut into shares when decoded."""
+    heads, dim, vdim, q_rank, kv_rank = latent
+    cfg = mc.kunonex([mc.latent(*latent)], width=80, vocab=60)
+
+    def change(w):
+        w["l0.mix.dq"][:] = np.roll(w["l0.mix.dkv"], 40, axis=1)
+        w["l0.mix.dq.norm"][:] = w["l0.mix.dkv.norm"]
+        w["l0.mix.uq"][:] = 2.0 * w["l0.mix.uk"]
+        w["embed"] *= 8.0
+        w["embed"][1] = np.roll(w["embed"][0], 40)
+        w["l0.norm1"][:] = 1.0
+        w["embed.norm"][:] = 1.0
+        w["l0.shift"][:] = 0.0
+
+    folder, oracle = checkpoint(tmp_path, cfg, seed=5, change=change)
+    model = mc.load(folder, compute, capacity=1200)
+    sought, asking, filler = 0, 1, np.random.default_rng(2).integers(2, 60, 1100)
+    for key, query in ((0, 1099), (15, 32), (16, 31), (31, 33), (32, 63), (16, 400), (255, 700), (256, 700), (63, 64), (128, 447), (0, 15), (0, 1), (7, 7)):
+        toks = filler[:query + 1].copy()
+        toks[key], toks[query] = sought, asking
+        want = oracle.logits(toks.tolist())[query]
+        if key < query:
+            without = toks.copy()
+            without[key] = 2
+            assert mc.row_errors(oracle.logits(without.tolist())[query], want) > 0.2      # a lost key shows
+        for portions in ([query + 1], [query, 1] if query else [1], mc.cut(query + 1, [48, 2])):
+            got = mc.run_portions(model, toks.tolist(), portions)[query]
+            assert mc.row_errors(got, want) <= mc.LIMIT[compute], (key, query, portions[:3])
+    model.close()
+
+
+@pytest.mark.parametrize("compute", DTYPES)
+def test_one_far_write_stays_in_the_mingru_state(mk, tmp_path, compute):
+    """Gates that hardly open but for one token: what it wrote is read hundreds of tokens later."""
+    cfg = mc.kunonex([mc.mingru(48)], width=64, vocab=50)
+
+    def change(w):
+        w["embed"] *= 8.0
+        w["embed"][:, 0] = -30.0
+        w["embed"][0, 0] = 30.0
+        w["embed.norm"][:] = 1.0
+        w["l0.norm1"][:] = 1.0
+        w["l0.shift"][:] = 0.0
+        w["l0.mix.z"] *= 0.05
+        w["l0.mix.z"][:, 0] = 4.0
+        w["l0.mix.z.b"][:] = -1.0
+
+    folder, oracle = checkpoint(tmp_path, cfg, seed=6, change=change)
+    toks = [0] + (1 + np.random.default_rng(4).integers(0, 49, 399)).tolist()
+    want = oracle.logits(toks)
+    lost = oracle.logits([1] + toks[1:])
+    assert mc.row_errors(lost[-40:], want[-40:]).min() > 10 * mc.LIMIT["float32"]
+    model = mc.load(folder, compute)
+    for portions in ([400], mc.cut(400, [37, 1, 2, 100]), mc.cut(400, [128, 129, 127, 8]), [64] + [1] * 336):
+        mc.assert_rows(mc.run_portions(model, toks, portions), want, compute, f"portions {portions[:4]}")
+    model.close()
+
+
+@pytest.mark.parametrize("lanes", [2, 9])
+def test_long_histories_decoded_in_shares(mk, built, lanes):
+    """A few sequences with a thousand tokens of history each, unequal, decoded together: their keys are shared out over CTAs."""
+    folder, oracle, cfg = built("looped")
+    seqs = [tokens_of(1000 - 111 * i, cfg["vocab"], seed=90 + i) for i in range(lanes)]
+    model = mc.load(folder, "bfloat16", capacity=lanes * 1008, lanes=lanes, slots=lanes)
+    sessions = [model.new_session() for _ in seqs]
+    for s, q in zip(sessions, seqs):
+        model.forward_batch([(s, q[:-4], 0)], want_logits=False, want_tokens=False, rows=[[]])
+    got = []
+    for t in range(4, 0, -1):
+        rows, _ = model.forward_batch([(s, [q[-t]], len(q) - t) for s, q in zip(sessions, seqs)], want_tokens=False)
+        got.append(rows)
+    for i, q in enumerate(seqs):
+        mc.assert_rows(np.stack([g[i] for g in got]), oracle.logits(q)[-4:], "bfloat16", f"sequence {i}")
+    model.close()
+
+
+@pytest.mark.parametrize("compute", DTYPES)
 def test_one_far_write_stays_in_the_recurrent_state(mk, tmp_path, compute):
     """Hardly any decay, no overwriting: what the first token wrote is read hundreds of tokens later by both recurrences."""
     cfg = mc.config([mc.wkv(2, 32), mc.parallel((2, 1, 16, 16, 8, False), (2, 1, 32, 32, 3))], width=64, vocab=50, side=0)
@@ -247,9 +396,10 @@ def test_one_far_write_stays_in_the_recurrent_state(mk, tmp_path, compute):
     model.close()
 
 
-def test_long_decoding_in_a_full_batch(mk, built):
+@pytest.mark.parametrize("name", BOTH)
+def test_long_decoding_in_a_full_batch(mk, built, name):
     """Four sequences decoded one token a tick for 300 ticks (the one-token kernels all the way), in bfloat16."""
-    folder, oracle, cfg = built("first")
+    folder, oracle, cfg = built(name)
     seqs = [tokens_of(300, cfg["vocab"], seed=70 + i) for i in range(4)]
     model = mc.load(folder, "bfloat16", capacity=4 * 304)
     sessions = [model.new_session() for _ in seqs]
@@ -266,8 +416,9 @@ def test_long_decoding_in_a_full_batch(mk, built):
 # ------------------------------------------------------------------------------------------------ sessions, sampling, engine
 
 @pytest.mark.parametrize("compute", DTYPES)
-def test_a_fork_carries_pages_and_state(mk, built, compute):
-    folder, oracle, cfg = built("first")
+@pytest.mark.parametrize("name", BOTH)
+def test_a_fork_carries_pages_and_state(mk, built, name, compute):
+    folder, oracle, cfg = built(name)
     toks = tokens_of(60, cfg["vocab"], seed=8)
     model = mc.load(folder, compute)
     a = model.new_session()
@@ -280,8 +431,9 @@ def test_a_fork_carries_pages_and_state(mk, built, compute):
     model.close()
 
 
-def test_a_refused_forward_leaves_the_state_alone(mk, built, capi):
-    folder, oracle, cfg = built("second")
+@pytest.mark.parametrize("name", ["second", "looped"])
+def test_a_refused_forward_leaves_the_state_alone(mk, built, capi, name):
+    folder, oracle, cfg = built(name)
     toks = tokens_of(50, cfg["vocab"], seed=9)
     model = mc.load(folder, "float32", capacity=128, lanes=1)
     s, other = model.new_session(), model.new_session()
@@ -295,7 +447,7 @@ def test_a_refused_forward_leaves_the_state_alone(mk, built, capi):
     model.close()
 
 
-@pytest.mark.parametrize("name", ["first", "second"])
+@pytest.mark.parametrize("name", ["first", "second", "looped", "loop over all layers", "no loop"])
 def test_greedy_generation_through_the_engine(mk, eng, built, name):
     """Requests of unequal length through the scheduler, more of them than slots; 32-bit, so that the plain statement's own
     argmax must come out wherever its first two logits are not a near-tie."""
@@ -316,9 +468,10 @@ def test_greedy_generation_through_the_engine(mk, eng, built, name):
     model.close()
 
 
-def test_device_sampling_and_recorded_logits(mk, eng, built):
+@pytest.mark.parametrize("name", BOTH)
+def test_device_sampling_and_recorded_logits(mk, eng, built, name):
     """Temperature / top-k / top-p on the device gives the same tokens as the host sampler on read-back logits."""
-    folder, oracle, cfg = built("first")
+    folder, oracle, cfg = built(name)
     outs = []
     for host in (False, True):
         model = mc.load(folder, "bfloat16")
@@ -331,14 +484,17 @@ def test_device_sampling_and_recorded_logits(mk, eng, built):
     assert outs[0] == outs[1]
 
 
-def test_residuals_after_every_layer(mk, built):
-    folder, oracle, cfg = built("second")
+@pytest.mark.parametrize("name", ["second", "looped", "loop over all layers"])
+def test_residuals_after_every_layer(mk, built, name):
+    """A looped layer counts once per pass."""
+    folder, oracle, cfg = built(name)
     toks = tokens_of(30, cfg["vocab"], seed=12)
     model = mc.load(folder, "float32")
     model.capture_residuals(True)
     s = model.new_session()
     model.forward_batch([(s, toks, 0)], want_tokens=False)
     got, want = model.residuals(30), oracle.residuals(toks)
+    assert got.shape == want.shape
     for l in range(len(want)):
         assert np.abs(got[l] - want[l]).max() <= 2e-5 * np.abs(want[l]).max()
     model.close()
@@ -364,8 +520,9 @@ def test_logit_rows_of_a_gguf_model(mk, eng, tmp_path):
 # ------------------------------------------------------------------------------------------------ the replay program
 
 @pytest.mark.parametrize("compute", DTYPES)
-def test_trace_replay(mk, built, tmp_path, compute):
-    folder, oracle, cfg = built("first")
+@pytest.mark.parametrize("name", BOTH)
+def test_trace_replay(mk, built, tmp_path, name, compute):
+    folder, oracle, cfg = built(name)
     a, b, c = (tokens_of(n, cfg["vocab"], seed=n) for n in (45, 20, 60))
     steps = [
         {"step": 0, "entries": [{"id": "a", "tokens": a[:17], "want": []}], "end": []},

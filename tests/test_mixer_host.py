@@ -80,6 +80,55 @@ def test_dyn_tanh_and_unit_and_gelu():
     assert np.allclose(mixers.gelu_tanh(np.array([0.0, 10.0, -10.0])), [0, 10, 0])
 
 
+def test_layer_norm_and_poly_norm_by_hand():
+    assert np.allclose(mixers.layer_norm(np.array([1.0, 3.0]), np.array([2.0, 0.5]), 0.0), [-2.0, 0.5])
+    assert np.allclose(mixers.layer_norm(np.array([1.0, 3.0]), np.ones(2), 3.0), [-0.5, 0.5])     # eps inside the root
+    z = np.array([3.0, -1.0])
+    # roots of the mean squares: sqrt(5), sqrt(41), sqrt(365)
+    want = 2.0 * z / np.sqrt(5) + 3.0 * z ** 2 / np.sqrt(41) - z ** 3 / np.sqrt(365) + 0.25
+    assert np.allclose(mixers.poly_norm(z, (2.0, 3.0, -1.0, 0.25), 0.0), want)
+
+
+def test_sinusoid_by_hand():
+    s = mixers.sinusoid([0, 1, 2000], 5)
+    assert np.allclose(s[0], [0, 1, 0, 1, 0])
+    f = 10000.0 ** -0.4
+    assert np.allclose(s[1], [np.sin(1), np.cos(1), np.sin(f), np.cos(f), np.sin(f * f)])
+    assert np.allclose(s[2, 2:4], [np.sin(2000 * f), np.cos(2000 * f)])
+
+
+def test_min_gru_by_hand():
+    z, u = np.array([[0.5], [0.25], [1.0]]), np.array([[1.5], [0.0], [-np.log(3.0)]])
+    out, S = mixers.min_gru(z, u)
+    # candidates 2, 1/2 and sigmoid(-log 3) = 1/4
+    assert np.allclose(out[:, 0], [1.0, 0.875, 0.25]) and np.allclose(S, [0.25])
+    rest, _ = mixers.min_gru(z[1:], u[1:], out[0])
+    assert np.allclose(rest, out[1:])
+
+
+def test_latent_attention_equals_attention_in_the_latent_space():
+    """Queries taken to the latent space and values taken out of it: the same numbers (what the kernels rely on)."""
+    rng = np.random.default_rng(0)
+    cfg = mc.latent(3, 7, 5, 6, 4)["mixer"]
+    W = {k[len("l0.mix."):]: v for k, v in mc.kunonex_weights(mc.kunonex([mc.latent(3, 7, 5, 6, 4)], width=10, vocab=11), 3).items() if k.startswith("l0.mix.")}
+    h = rng.standard_normal((9, 10))
+    want = mixers.latent_attention(h, W, cfg, 1e-5)
+    q = ((mixers.rms(h @ W["dq"].T, 1e-5) * W["dq.norm"]) @ W["uq"].T).reshape(9, 3, 7)
+    c = mixers.rms(h @ W["dkv"].T, 1e-5) * W["dkv.norm"]
+    lat = np.einsum("thd,hdr->thr", q, W["uk"].reshape(3, 7, 4))
+    o = mixers.causal_attention(lat, c[:, None, :], c[:, None, :], cfg["scale"])
+    v = np.einsum("thr,her->the", o, W["uv"].reshape(3, 5, 4)) * mixers.sigmoid(h @ W["g"].T)[:, :, None]
+    assert np.allclose(v.reshape(9, -1) @ W["o"].T, want)
+
+
+def test_looped_layers_run_in_order():
+    cfg = mc.kunonex([mc.mingru(3)] * 4, width=6, vocab=9, loop=(1, 3, 2))
+    m = mixers.decoder(cfg, mc.weights(cfg))
+    assert m.schedule() == [(0, None), (1, 0), (2, 0), (1, 1), (2, 1), (3, None)]
+    cfg["loop"] = None
+    assert mixers.decoder(cfg, {}).schedule() == [(i, None) for i in range(4)]
+
+
 @pytest.mark.parametrize("dims,base,scaling", [(8, 10000.0, None), (64, 500.0, mc.SCALING), (10, 1e6, dict(factor=2.0, low=0.5, high=6.0, original=4096))])
 def test_rotary_frequencies_of_the_loader(capi, dims, base, scaling):
     out = np.empty(dims // 2)
@@ -115,6 +164,59 @@ def test_inspect_reads_the_description(eng, tmp_path):
     w = mc.weights(mc.config(LAYERS, width=40))
     assert s["tensors_in_file"] == s["tensors_read"] == len(w)
     assert s["parameters"] == sum(a.size for a in w.values())
+
+
+BESIDE = [mc.mingru(24), mc.latent(4, 16, 20, 12, 10, ff=40), mc.mingru(40, ff=24)]
+
+
+def broken_beside(tmp_path, change_cfg=None, change_w=None):
+    cfg = json.loads(json.dumps(mc.kunonex(BESIDE, width=40, loop=(1, 3, 3))))
+    w = mc.weights(cfg)
+    if change_cfg:
+        change_cfg(cfg)
+    if change_w:
+        change_w(w)
+    return mc.write(tmp_path / "m", cfg, w)
+
+
+@pytest.mark.parametrize("loop,runs", [((1, 3, 3), 7), ((0, 3, 2), 6), ((0, 1, 1), 3), (None, 3)])
+def test_inspect_reads_layers_with_one_norm(eng, tmp_path, loop, runs):
+    cfg = mc.kunonex(BESIDE, width=40, loop=loop)
+    w = mc.weights(cfg)
+    s = eng.Model.inspect_mixer(mc.write(tmp_path / "m", cfg, w))
+    assert (s["architecture"], s["vocab_size"], s["hidden_size"], s["n_layers"], s["layer_runs"]) == ("Kunonex", 131, 40, 3, runs)
+    assert (s["mingru_layers"], s["latent_layers"], s["wkv_layers"], s["parallel_layers"], s["ffn_layers"], s["side_dim"]) == (2, 1, 0, 0, 2, 0)
+    assert s["tensors_in_file"] == s["tensors_read"] == len(w)
+    assert s["parameters"] == sum(a.size for a in w.values())
+
+
+@pytest.mark.parametrize("change,message", [
+    (lambda w: w.pop("l1.mix.uk"), "`l1.mix.uk` is missing"),
+    (lambda w: w.pop("embed.norm"), "`embed.norm` is missing"),
+    (lambda w: w.pop("l2.shift"), "`l2.shift` is missing"),
+    (lambda w: w.update({"loop.step": np.zeros((2, 40), np.float32)}), "`loop.step` has shape [2, 40], expected [3, 40]"),
+    (lambda w: w.update({"l1.mlp.act": np.zeros(3, np.float32)}), "`l1.mlp.act` has shape [3], expected [4]"),
+    (lambda w: w.update({"l0.mix.z.b": np.zeros(40, np.float32)}), "`l0.mix.z.b` has shape [40], expected [24]"),
+])
+def test_audit_names_the_tensor_of_layers_with_one_norm(eng, capi, tmp_path, change, message):
+    with pytest.raises(capi.MkError) as e:
+        eng.Model.inspect_mixer(broken_beside(tmp_path, change_w=change))
+    assert message in str(e.value)
+
+
+@pytest.mark.parametrize("change,message", [
+    (lambda c: c["layers"][0].update(type="wkv"), "config.layers[0].type `wkv` is not a known mixer"),
+    (lambda c: c["layers"][1]["mixer"].pop("q_rank"), "config.layers[1].mixer.q_rank is missing"),
+    (lambda c: c["layers"][1]["mlp"].update(kind="sparse"), "kind `sparse` is not supported"),
+    (lambda c: c["loop"].update(stop=4), "config.loop.stop is out of range"),
+    (lambda c: c["loop"].update(stop=1), "config.loop.stop is out of range"),
+    (lambda c: c["loop"].update(times=0), "config.loop.times is out of range"),
+    (lambda c: c.pop("logit_scale"), "config.logit_scale is missing"),
+])
+def test_reader_names_the_setting_of_layers_with_one_norm(eng, capi, tmp_path, change, message):
+    with pytest.raises(capi.MkError) as e:
+        eng.Model.inspect_mixer(broken_beside(tmp_path, change_cfg=change))
+    assert message in str(e.value)
 
 
 @pytest.mark.parametrize("change,message", [
