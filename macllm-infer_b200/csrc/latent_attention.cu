@@ -1,41 +1,118 @@
 // See latent_attention.h.
 //
-// Tensor-core kernel: one CTA per (query row, share of its keys, up to 32 heads).  The four warps each own a quarter of the
-// latent's columns: a warp's cp.async ring holds its columns of the next tiles of 32 rows, its queries' columns stay in registers,
-// its partial scores meet the other warps' in shared memory (the one barrier of a tile, double-buffered), every warp then forms
-// the same softmax weights and adds up its columns of the output from the rows it already holds.  A row is thus read once for
-// keys and values, and by one warp per column.  Scores, softmax and sums are f32; the weights enter the second product as the sum
-// of two f16 numbers.  When few rows are in flight their keys are shared out over several CTAs; the one that finishes last adds
-// the shares in order.
+// Tensor-core kernel (tcgen05): one CTA per (query row, share of its keys, up to 32 heads).  Tiles of 128 cached vectors arrive by
+// TMA, 128 bytes wide and swizzled, in chunks of 128 columns.  A tile is an operand twice: with the vectors' columns as the
+// reduction it gives the scores transposed (keys x heads), and read the other way round, with the keys as the reduction, it gives
+// the outputs transposed (columns x heads) - so the wide side of both products fills the tensor core's 128 rows and the few heads
+// are its columns.  Four groups of four warps, a quarter of the heads each, hold one key per thread: scores from tensor memory, the
+// heads' maxima over the keys by a folding exchange, softmax weights in f32, which go back to shared memory as two f16 numbers
+// each (high part and rest, as columns of their own, added up at the end).  A latent of 512 columns is too wide for a second tile
+// beside the first in shared memory, so two CTAs take half of the output columns each: both form all scores, and the chunks a CTA
+// needs for the scores only leave the ring at once.  The scores of the next tile are thus computed while the weights of this one
+// are being formed.  The running maximum moves only when a tile exceeds it by more than kSlack, so the accumulators
+// in tensor memory are hardly ever rescaled.  When few rows are in flight their keys are shared out over several CTAs; the one
+// that finishes last adds the shares in order.  Every wait is bounded (see hgemm_tc.cu).
 #include "latent_attention.h"
 #include "device_util.h"
+#include "hgemm_tc.h"
 #include <algorithm>
+#include <cuda.h>
 
 namespace mk {
 
 namespace {
 
-constexpr int LA_WARPS = 4;
-constexpr int LA_KT = 32;             // keys of a tile
-constexpr int LA_STAGES = 2;
-constexpr int LA_SP = LA_KT + 4;      // pitch of the partial scores
+constexpr int LU_KEYS = 128;          // keys of a tile
+constexpr int LU_COLS = 128;          // columns of a chunk
+constexpr int LU_CHUNK = LU_KEYS * LU_COLS * 2;
+constexpr int LU_BLOCK = LU_KEYS * 128;  // bytes of the 64 columns that share swizzled rows
+constexpr int LU_GROUPS = 4;           // softmax groups of four warps
+constexpr int LU_SOFTMAX = LU_GROUPS * 128;
+constexpr int LU_THREADS = LU_SOFTMAX + 64;  // and the loader's and the MMA issuer's warps
+constexpr float kSlack = 8.f;         // weights stay below e^8, well inside f16
+constexpr uint32_t LU_SPIN_LIMIT = 1u << 22;
 constexpr int LA_SMS = 148;
-constexpr int LA_TARGET_CTAS = LA_SMS * 2;
+constexpr int LA_TARGET_CTAS = LA_SMS;
 constexpr int LA_MIN_SHARE = 256;
 constexpr int LA_MAX_SHARES = 32;
 constexpr int LA_SHARED_ROWS = 256;   // ticks with more query rows are not cut into shares
 
-__device__ __forceinline__ uint32_t la_smem(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
-__device__ __forceinline__ void la_ldm4(uint32_t (&r)[4], const void* p) {
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(la_smem(p)));
+__device__ __forceinline__ uint32_t lu_smem(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
+__device__ __forceinline__ void lu_bar_init(uint64_t* bar, uint32_t count) { asm volatile("mbarrier.init.shared::cta.b64 [%0], %1;" ::"r"(lu_smem(bar)), "r"(count)); }
+__device__ __forceinline__ bool lu_bar_wait(uint64_t* bar, uint32_t parity) {
+    const uint32_t addr = lu_smem(bar);
+    for (uint32_t i = 0; i <= LU_SPIN_LIMIT; ++i) {
+        uint32_t done;
+        asm volatile(
+            "{\n\t.reg .pred p;\n\t"
+            "mbarrier.try_wait.parity.shared::cta.b64 p, [%1], %2;\n\t"
+            "selp.u32 %0, 1, 0, p;\n\t}"
+            : "=r"(done)
+            : "r"(addr), "r"(parity)
+            : "memory");
+        if (done) return true;
+    }
+    return false;
 }
-__device__ __forceinline__ void la_ldm4_trans(uint32_t (&r)[4], const void* p) {
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(la_smem(p)));
+__device__ __forceinline__ void lu_bar_arrive(uint64_t* bar) { asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];" ::"r"(lu_smem(bar)) : "memory"); }
+__device__ __forceinline__ void lu_bar_expect(uint64_t* bar, uint32_t bytes) {
+    asm volatile("mbarrier.arrive.expect_tx.shared::cta.b64 _, [%0], %1;" ::"r"(lu_smem(bar)), "r"(bytes) : "memory");
 }
-__device__ __forceinline__ void la_mma(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.f16.f16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
-                 : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
-                 : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+__device__ __forceinline__ void lu_tma(void* dst, const void* tmap, int x, int y, uint64_t* bar) {
+    asm volatile("cp.async.bulk.tensor.2d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3}], [%4];" ::"r"(lu_smem(dst)), "l"(tmap), "r"(x), "r"(y),
+                 "r"(lu_smem(bar))
+                 : "memory");
+}
+// Operand of 128-byte swizzled rows, 8-row groups 1024 bytes apart.  Reduction along the rows' bytes: lead is not used; reduction
+// from row to row: lead = distance of the next 64 elements of the other dimension.
+__device__ __forceinline__ uint64_t lu_desc(uint32_t addr, uint32_t lead) {
+    return (uint64_t)((addr >> 4) & 0x3FFF) | (uint64_t)(lead >> 4) << 16 | (uint64_t)(1024 >> 4) << 32 | (uint64_t)1 << 46 | (uint64_t)2 << 61;
+}
+__device__ __forceinline__ void lu_mma(uint32_t d, uint64_t a, uint64_t b, uint32_t idesc, bool accumulate) {
+    asm volatile(
+        "{\n\t.reg .pred p;\n\t"
+        "setp.ne.b32 p, %4, 0;\n\t"
+        "tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, p;\n\t}" ::"r"(d), "l"(a), "l"(b), "r"(idesc), "r"(accumulate ? 1u : 0u)
+        : "memory");
+}
+__device__ __forceinline__ void lu_commit(uint64_t* bar) {
+    asm volatile("tcgen05.commit.cta_group::1.mbarrier::arrive::one.shared::cluster.b64 [%0];" ::"r"(lu_smem(bar)) : "memory");
+}
+// N (4 or 8) columns of this thread's lane; the values are there after lu_tmem_wait.
+template <int N>
+__device__ __forceinline__ void lu_tmem_load(uint32_t at, uint32_t* r) {
+    if constexpr (N == 4)
+        asm volatile("tcgen05.ld.sync.aligned.32x32b.x4.b32 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(at) : "memory");
+    else
+        asm volatile("tcgen05.ld.sync.aligned.32x32b.x8.b32 {%0,%1,%2,%3,%4,%5,%6,%7}, [%8];"
+                     : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]), "=r"(r[4]), "=r"(r[5]), "=r"(r[6]), "=r"(r[7])
+                     : "r"(at)
+                     : "memory");
+}
+template <int N>
+__device__ __forceinline__ void lu_tmem_store(uint32_t at, const uint32_t* r) {
+    if constexpr (N == 4)
+        asm volatile("tcgen05.st.sync.aligned.32x32b.x4.b32 [%0], {%1,%2,%3,%4};" ::"r"(at), "r"(r[0]), "r"(r[1]), "r"(r[2]), "r"(r[3]) : "memory");
+    else
+        asm volatile("tcgen05.st.sync.aligned.32x32b.x8.b32 [%0], {%1,%2,%3,%4,%5,%6,%7,%8};" ::"r"(at), "r"(r[0]), "r"(r[1]), "r"(r[2]), "r"(r[3]), "r"(r[4]), "r"(r[5]),
+                     "r"(r[6]), "r"(r[7])
+                     : "memory");
+}
+__device__ __forceinline__ void lu_tmem_wait() { asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory"); }
+__device__ __forceinline__ void lu_fence_before() { asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory"); }
+__device__ __forceinline__ void lu_fence_after() { asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory"); }
+// Barrier of `threads` softmax threads; true when every one of them came with ok.
+__device__ __forceinline__ bool lu_agree(int barrier, int threads, bool ok) {
+    uint32_t all;
+    asm volatile(
+        "{\n\t.reg .pred p, q;\n\t"
+        "setp.ne.u32 q, %1, 0;\n\t"
+        "bar.red.and.pred p, %2, %3, q;\n\t"
+        "selp.u32 %0, 1, 0, p;\n\t}"
+        : "=r"(all)
+        : "r"(ok ? 1u : 0u), "r"(barrier), "r"(threads)
+        : "memory");
+    return all != 0;
 }
 __device__ __forceinline__ uint32_t la_pack(float x, float y) {
     const __half2 h = __floats2half2_rn(x, y);
@@ -46,6 +123,21 @@ __device__ __forceinline__ uint32_t la_rest(float x, float y, uint32_t rounded) 
     const float2 r = __half22float2(*reinterpret_cast<const __half2*>(&rounded));
     return la_pack(x - r.x, y - r.y);
 }
+// N values per lane, folded over the warp: lane l ends with the result of value l % N over all lanes.  Uses up v.
+template <int N, typename Op>
+__device__ __forceinline__ float lu_fold(float (&v)[N], int lane, Op op) {
+#pragma unroll
+    for (int s = N / 2; s > 0; s >>= 1) {
+        const bool up = (lane & s) != 0;
+#pragma unroll
+        for (int i = 0; i < N / 2; ++i)
+            if (i < s) v[i] = op(up ? v[i + s] : v[i], __shfl_xor_sync(0xffffffffu, up ? v[i] : v[i + s], s));
+    }
+    float r = v[0];
+#pragma unroll
+    for (int s = N; s < 32; s <<= 1) r = op(r, __shfl_xor_sync(0xffffffffu, r, s));
+    return r;
+}
 
 struct LatentEntry {
     int row, share, n_shares, pos, table_off, packed, first;
@@ -55,262 +147,338 @@ __device__ __forceinline__ LatentEntry load_entry(const int32_t* entries, int i)
     return LatentEntry{a.x, a.y, a.z, a.w, b.x, b.y, b.z};
 }
 
-template <int RANK, int MT>
-struct La {
-    static constexpr int CW = RANK / LA_WARPS;   // columns of a warp
-    static constexpr int PITCH = CW + 8;         // halves: conflict-free ldmatrix
-    static constexpr int KS = CW / 16;
-    static constexpr int NT = CW / 8;
-    static constexpr int STAGE = LA_KT * PITCH;  // halves of a warp's stage
-    static constexpr int SCORES = LA_WARPS * MT * 16 * LA_SP;
-    static constexpr size_t BYTES = (size_t)LA_WARPS * LA_STAGES * STAGE * 2 + (size_t)2 * SCORES * 4;
+// MB chunks of 128 columns, NH heads (16 or 32).
+template <int MB, int NH>
+struct Lu {
+    static constexpr int RANK = MB * LU_COLS;
+    static constexpr int STAGES = MB >= 4 && NH == 16 ? 6 : (MB >= 3 ? 5 : (MB == 2 ? 4 : 2));  // chunks in the ring
+    static constexpr int Q_BYTES = NH * RANK * 2;                                               // [column block][head][64]
+    static constexpr int P_BYTES = 2 * NH * LU_KEYS * 2;                                        // [key block][weights | rests][64]
+    static constexpr size_t BYTES = (size_t)STAGES * LU_CHUNK + Q_BYTES + P_BYTES + 1024 + 256;
+    static constexpr int CS = MB == 4 ? 2 : 1;   // CTAs that share the output columns
+    static constexpr int OWN = MB / CS;          // chunks of a CTA's own
+    static constexpr int S_COL = OWN * 2 * NH;   // tensor memory: outputs (high | rest) of every chunk, then two tiles' scores
+    static constexpr uint32_t TMEM = S_COL + 2 * NH <= 64 ? 64 : (S_COL + 2 * NH <= 128 ? 128 : (S_COL + 2 * NH <= 256 ? 256 : 512));
+    // chunks of the next tile that reach the ring while this tile's own ones are in use
+    static constexpr int AHEAD = STAGES - OWN < MB ? STAGES - OWN : MB;
 };
 
-template <int RANK, int MT>
-__global__ void __launch_bounds__(LA_WARPS * 32, 2) latent_tc_kernel(LatentAttnArgs a, int bt_shift) {
-    using L = La<RANK, MT>;
-    constexpr int CW = L::CW, PITCH = L::PITCH, KS = L::KS, NT = L::NT, HEADS = MT * 16;
-    extern __shared__ __align__(16) unsigned char la_raw[];
-    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, gid = lane >> 2, tq = lane & 3;
-    __half* ring = reinterpret_cast<__half*>(la_raw) + warp * LA_STAGES * L::STAGE;
-    float* scores = reinterpret_cast<float*>(la_raw + (size_t)LA_WARPS * LA_STAGES * L::STAGE * 2);
-    const int col0 = warp * CW, head0 = blockIdx.y * HEADS;
+template <int MB, int NH>
+__global__ void __launch_bounds__(LU_THREADS, 1) latent_umma_kernel(const __grid_constant__ CUtensorMap tm, LatentAttnArgs a, int bt_shift, int box_rows, int pool_rows) {
+    using L = Lu<MB, NH>;
+    constexpr int RANK = L::RANK, STAGES = L::STAGES, CS = L::CS, OWN = L::OWN, HG = NH / LU_GROUPS, LOADER = LU_SOFTMAX / 32;
+    extern __shared__ uint8_t lu_raw[];
+    uint8_t* ring = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(lu_raw) + 1023) & ~(uintptr_t)1023);
+    uint8_t* qs = ring + (size_t)STAGES * LU_CHUNK;
+    uint8_t* ps = qs + L::Q_BYTES;
+    uint64_t* full = reinterpret_cast<uint64_t*>(ps + L::P_BYTES);  // [STAGES] loader -> MMA
+    uint64_t* empty = full + STAGES;                                // [STAGES] MMA -> loader
+    uint64_t* q_full = empty + STAGES;                              // softmax -> MMA: queries
+    uint64_t* s_full = q_full + 1;                                  // [2] MMA -> softmax: scores
+    uint64_t* p_full = s_full + 2;                                  // softmax -> MMA: weights
+    uint64_t* o_done = p_full + 1;                                  // MMA -> softmax: the tile is in the outputs
+    __shared__ uint32_t tmem_slot;
+    __shared__ __align__(16) float s_warp[LU_SOFTMAX / 32][HG], s_factor[LA_MAX_SHARES][NH];
+    __shared__ int s_last;
+
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int head0 = blockIdx.y * NH, heads = min(NH, a.heads - head0);
+    const int part = blockIdx.z, col0 = part * OWN * LU_COLS;  // this CTA's output columns
+    // the i-th chunk of a tile to arrive: other CTAs' columns first, then the own ones
+    auto chunk_of = [&](int i) { return CS == 1 ? i : (i < MB - OWN ? (i >= part * OWN ? i + OWN : i) : part * OWN + i - (MB - OWN)); };
+    if (tid == 0) {
+        for (int i = 0; i < STAGES; ++i) {
+            lu_bar_init(&full[i], 1);
+            lu_bar_init(&empty[i], 1);
+        }
+        lu_bar_init(q_full, LU_SOFTMAX);
+        lu_bar_init(&s_full[0], 1);
+        lu_bar_init(&s_full[1], 1);
+        lu_bar_init(p_full, LU_SOFTMAX);
+        lu_bar_init(o_done, 1);
+        asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+    }
+    if (warp == LOADER) {
+        asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(lu_smem(&tmem_slot)), "r"(L::TMEM) : "memory");
+        asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
+    }
+    lu_fence_before();
+    __syncthreads();
+    lu_fence_after();
+    const uint32_t tmem = tmem_slot;
     pdl_trigger();
     pdl_wait();
     const LatentEntry e = load_entry(a.entries, blockIdx.x);
     const int len = e.pos + 1;
-    const int chunk = ((len + e.n_shares - 1) / e.n_shares + LA_KT - 1) / LA_KT * LA_KT;
+    const int chunk = ((len + e.n_shares - 1) / e.n_shares + LU_KEYS - 1) / LU_KEYS * LU_KEYS;
     const int k_lo = e.share * chunk, k_hi = min(len, k_lo + chunk);
-    const int tiles = k_hi > k_lo ? (k_hi - k_lo + LA_KT - 1) / LA_KT : 0;
+    const int tiles = k_hi > k_lo ? (k_hi - k_lo + LU_KEYS - 1) / LU_KEYS : 0;
 
-    // the warp's columns of the queries, as A fragments
-    uint32_t qf[MT][KS][4];
-#pragma unroll
-    for (int m = 0; m < MT; ++m)
-#pragma unroll
-        for (int k = 0; k < KS; ++k)
-#pragma unroll
-            for (int i = 0; i < 4; ++i) {
-                const int head = head0 + m * 16 + gid + (i & 1) * 8, c = col0 + k * 16 + 2 * tq + (i >> 1) * 8;
-                qf[m][k][i] = head < a.heads ? *reinterpret_cast<const uint32_t*>(a.q_h + ((int64_t)e.row * a.heads + head) * RANK + c) : 0u;
-            }
-
-    const __half* pool = static_cast<const __half*>(a.pool);
-    auto row_of = [&](int t) {  // pool row of this lane's key of tile t
-        const int pos = k_lo + t * LA_KT + lane;
-        return pos < k_hi ? ((int64_t)a.tables[e.table_off + (pos >> bt_shift)] << bt_shift) + (pos & ((1 << bt_shift) - 1)) : (int64_t)-1;
-    };
-    constexpr int CHUNKS = CW / 8;  // 16-byte pieces of a row
-    auto load = [&](int t, int64_t my_row) {
-        __half* dst = ring + (t % LA_STAGES) * L::STAGE;
-#pragma unroll
-        for (int i = 0; i < CHUNKS; ++i) {
-            const int j = i * 32 + lane, key = j / CHUNKS, c = (j % CHUNKS) * 8;
-            const int64_t row = __shfl_sync(0xffffffffu, my_row, key);
-            const int bytes = row >= 0 ? 16 : 0;  // keys past the end are zeros
-            asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(la_smem(dst + key * PITCH + c)), "l"(pool + (row >= 0 ? row : 0) * RANK + col0 + c),
-                         "r"(bytes)
-                         : "memory");
-        }
-    };
-
-    float o[MT][NT][4];
-#pragma unroll
-    for (int m = 0; m < MT; ++m)
-#pragma unroll
-        for (int j = 0; j < NT; ++j) o[m][j][0] = o[m][j][1] = o[m][j][2] = o[m][j][3] = 0.f;
-    float m_run[MT][2], l_run[MT][2];
-#pragma unroll
-    for (int m = 0; m < MT; ++m) {
-        m_run[m][0] = m_run[m][1] = -INFINITY;
-        l_run[m][0] = l_run[m][1] = 0.f;
-    }
-
-    int64_t next_row = 0;
-    if (tiles > 0) load(0, row_of(0));
-    asm volatile("cp.async.commit_group;" ::: "memory");
-    if (tiles > 1) next_row = row_of(1);
-    for (int t = 0; t < tiles; ++t) {
-        if (t + 1 < tiles) load(t + 1, next_row);
-        asm volatile("cp.async.commit_group;" ::: "memory");
-        if (t + 2 < tiles) next_row = row_of(t + 2);
-        asm volatile("cp.async.wait_group 1;" ::: "memory");
-        __syncwarp();
-        const __half* rows = ring + (t % LA_STAGES) * L::STAGE;
-        float* mine = scores + (t & 1) * L::SCORES;
-
-        // this warp's part of the scores
-        float s[MT][4][4];
-#pragma unroll
-        for (int m = 0; m < MT; ++m)
-#pragma unroll
-            for (int j = 0; j < 4; ++j) s[m][j][0] = s[m][j][1] = s[m][j][2] = s[m][j][3] = 0.f;
-#pragma unroll
-        for (int k = 0; k < KS; ++k)
-#pragma unroll
-            for (int j = 0; j < 4; j += 2) {
-                uint32_t b[4];
-                la_ldm4(b, rows + (j * 8 + (lane & 7) + (lane >> 4) * 8) * PITCH + k * 16 + ((lane >> 3) & 1) * 8);
-#pragma unroll
-                for (int m = 0; m < MT; ++m) {
-                    la_mma(s[m][j], qf[m][k], b[0], b[1]);
-                    la_mma(s[m][j + 1], qf[m][k], b[2], b[3]);
+    if (warp == LOADER) {
+        // ---- loader: a lane per box of box_rows keys x 64 columns (at most 32 of them)
+        const int boxes = LU_KEYS / box_rows;  // of a column block
+        const int block = lane / boxes, box = lane - block * boxes;
+        auto row_of = [&](int t) {
+            // boxes past the last key start behind the pool and are filled with zeros
+            const int pos = k_lo + t * LU_KEYS + box * box_rows;
+            return pos < k_hi ? (int)(a.tables[e.table_off + (pos >> bt_shift)] << bt_shift) + (pos & ((1 << bt_shift) - 1)) : pool_rows;
+        };
+        uint32_t it = 0;
+        bool ok = true;
+        int next = row_of(0);
+        for (int t = 0; t < tiles && ok; ++t) {
+            const int y = next;
+            if (t + 1 < tiles) next = row_of(t + 1);
+            for (int c = 0; c < MB && ok; ++c, ++it) {
+                const uint32_t st = it % STAGES, ph = (it / STAGES) & 1;
+                ok = lu_bar_wait(&empty[st], ph ^ 1);
+                if (!__all_sync(0xffffffffu, ok)) {
+                    if (lane == 0) atomicExch(a.status, 21);
+                    ok = false;
+                    break;
                 }
-            }
-#pragma unroll
-        for (int m = 0; m < MT; ++m)
-#pragma unroll
-            for (int j = 0; j < 4; ++j)
-#pragma unroll
-                for (int h = 0; h < 2; ++h)
-                    *reinterpret_cast<float2*>(mine + ((warp * MT + m) * 16 + gid + 8 * h) * LA_SP + j * 8 + 2 * tq) = make_float2(s[m][j][2 * h], s[m][j][2 * h + 1]);
-        __syncthreads();
-        const int pos0 = k_lo + t * LA_KT;
-#pragma unroll
-        for (int m = 0; m < MT; ++m) {
-            float mx[2] = {-INFINITY, -INFINITY};
-#pragma unroll
-            for (int j = 0; j < 4; ++j)
-#pragma unroll
-                for (int h = 0; h < 2; ++h) {
-                    float2 v = make_float2(0.f, 0.f);
-#pragma unroll
-                    for (int w = 0; w < LA_WARPS; ++w) {
-                        const float2 p = *reinterpret_cast<const float2*>(mine + ((w * MT + m) * 16 + gid + 8 * h) * LA_SP + j * 8 + 2 * tq);
-                        v.x += p.x;
-                        v.y += p.y;
-                    }
-                    const int pos = pos0 + j * 8 + 2 * tq;
-                    s[m][j][2 * h] = pos < k_hi ? v.x * a.scale : -INFINITY;
-                    s[m][j][2 * h + 1] = pos + 1 < k_hi ? v.y * a.scale : -INFINITY;
-                    mx[h] = fmaxf(mx[h], fmaxf(s[m][j][2 * h], s[m][j][2 * h + 1]));
-                }
-            float alpha[2];
-#pragma unroll
-            for (int h = 0; h < 2; ++h) {
-                mx[h] = fmaxf(mx[h], __shfl_xor_sync(0xffffffffu, mx[h], 1));
-                mx[h] = fmaxf(mx[h], __shfl_xor_sync(0xffffffffu, mx[h], 2));
-                const float m_new = fmaxf(m_run[m][h], mx[h]);  // finite: every tile has a visible key
-                alpha[h] = __expf(m_run[m][h] - m_new);
-                m_run[m][h] = m_new;
-                float sum = 0.f;
-#pragma unroll
-                for (int j = 0; j < 4; ++j)
-#pragma unroll
-                    for (int i = 0; i < 2; ++i) {
-                        const float p = __expf(s[m][j][2 * h + i] - m_new);
-                        s[m][j][2 * h + i] = p;
-                        sum += p;
-                    }
-                sum += __shfl_xor_sync(0xffffffffu, sum, 1);
-                sum += __shfl_xor_sync(0xffffffffu, sum, 2);
-                l_run[m][h] = l_run[m][h] * alpha[h] + sum;
-            }
-#pragma unroll
-            for (int j = 0; j < NT; ++j) {
-                o[m][j][0] *= alpha[0];
-                o[m][j][1] *= alpha[0];
-                o[m][j][2] *= alpha[1];
-                o[m][j][3] *= alpha[1];
+                if (lane == 0) lu_bar_expect(&full[st], (uint32_t)LU_CHUNK);
+                __syncwarp();
+                if (block < 2) lu_tma(ring + (size_t)st * LU_CHUNK + block * LU_BLOCK + box * box_rows * 128, &tm, chunk_of(c) * LU_COLS + block * 64, y, &full[st]);
+                __syncwarp();
             }
         }
+        if (!ok)  // copies still in flight land before the CTA goes
+            for (uint32_t i = it > STAGES ? it - STAGES : 0; i < it; ++i) lu_bar_wait(&full[i % STAGES], (i / STAGES) & 1);
+    } else if (warp == LOADER + 1) {
+        // ---- MMA issuer
+        if (lane == 0 && tiles > 0) {
+            const uint32_t i_scores = (1u << 4) | ((uint32_t)(NH >> 3) << 17) | (8u << 24);
+            const uint32_t i_out = (1u << 4) | (1u << 15) | ((uint32_t)(2 * NH >> 3) << 17) | (8u << 24);  // A read with the keys as the reduction
+            const uint32_t q_addr = lu_smem(qs), p_addr = lu_smem(ps), ring_addr = lu_smem(ring);
+            bool ok = true;
+            auto scores = [&](int t, int c0, int c1) {  // chunks c0 .. c1 - 1 of tile t's scores
+                for (int c = c0; c < c1; ++c) {
+                    const uint32_t it = (uint32_t)(t * MB + c), st = it % STAGES;
+                    if (!lu_bar_wait(&full[st], (it / STAGES) & 1)) {
+                        atomicExch(a.status, 22);
+                        ok = false;
+                        return;
+                    }
+                    lu_fence_after();
+                    const uint32_t q_chunk = q_addr + 2 * chunk_of(c) * (NH * 128);
 #pragma unroll
-        for (int kk = 0; kk < LA_KT / 16; ++kk) {
-            uint32_t pf[MT][4], pr[MT][4];
+                    for (int k = 0; k < LU_COLS / 16; ++k) {
+                        const uint32_t block = (uint32_t)k >> 2, step = ((uint32_t)k & 3) * 32;
+                        lu_mma(tmem + L::S_COL + (t & 1) * NH, lu_desc(ring_addr + st * LU_CHUNK + block * LU_BLOCK + step, 16),
+                               lu_desc(q_chunk + block * (NH * 128) + step, 16), i_scores, c > 0 || k > 0);
+                    }
+                    if (c < MB - OWN) lu_commit(&empty[st]);
+                }
+                if (c1 == MB) lu_commit(&s_full[t & 1]);
+            };
+            if (!lu_bar_wait(q_full, 0)) {
+                atomicExch(a.status, 26);
+                ok = false;
+            }
+            lu_fence_after();
+            if (ok) scores(0, 0, MB);
+            for (int t = 0; t < tiles && ok; ++t) {
+                if (t + 1 < tiles) scores(t + 1, 0, L::AHEAD);
+                if (!ok) break;
+                if (!lu_bar_wait(p_full, t & 1)) {
+                    atomicExch(a.status, 23);
+                    break;
+                }
+                lu_fence_after();
+                for (int c = 0; c < OWN; ++c) {
+                    const uint32_t st = (uint32_t)(t * MB + MB - OWN + c) % STAGES;
 #pragma unroll
-            for (int m = 0; m < MT; ++m)
+                    for (int k = 0; k < LU_KEYS / 16; ++k)
+                        lu_mma(tmem + c * 2 * NH, lu_desc(ring_addr + st * LU_CHUNK + k * 2048, LU_BLOCK),
+                               lu_desc(p_addr + (uint32_t)(k >> 2) * (2 * NH * 128) + ((uint32_t)k & 3) * 32, 16), i_out, t > 0 || k > 0);
+                    lu_commit(&empty[st]);
+                }
+                lu_commit(o_done);
+                if (L::AHEAD < MB && t + 1 < tiles) scores(t + 1, L::AHEAD, MB);
+            }
+        }
+    } else {
+        // ---- softmax: a group of 128 threads takes HG heads; thread = key of the tile, later column of a chunk
+        const int group = warp >> 2, gt = tid & 127, h0 = group * HG, bar = 1 + group;
+        // the queries, a head per row, 16-byte pieces
+#pragma unroll 4
+        for (int i = tid; i < NH * (RANK / 8); i += LU_SOFTMAX) {
+            const int h = i / (RANK / 8), c = i - h * (RANK / 8);
+            uint4 v = make_uint4(0u, 0u, 0u, 0u);
+            if (h < heads) v = *reinterpret_cast<const uint4*>(a.q_h + ((int64_t)e.row * a.heads + head0 + h) * RANK + c * 8);
+            *reinterpret_cast<uint4*>(qs + (c >> 3) * (NH * 128) + h * 128 + (((c & 7) ^ (h & 7)) << 4)) = v;
+        }
+        asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
+        lu_bar_arrive(q_full);
+
+        const uint32_t my_tmem = tmem + ((uint32_t)((warp & 3) * 32) << 16) + h0;
+        float m[HG], l[HG];
+#pragma unroll
+        for (int h = 0; h < HG; ++h) {
+            m[h] = -INFINITY;
+            l[h] = 0.f;
+        }
+        bool ok = true;
+        for (int t = 0; t < tiles; ++t) {
+            ok = ok && lu_bar_wait(&s_full[t & 1], (t >> 1) & 1);
+            __syncwarp();
+            lu_fence_after();
+            const bool visible = k_lo + t * LU_KEYS + gt < k_hi;
+            uint32_t raw[HG];
+            float s[HG], x[HG];
+            lu_tmem_load<HG>(my_tmem + L::S_COL + (t & 1) * NH, raw);
+            lu_tmem_wait();
+#pragma unroll
+            for (int h = 0; h < HG; ++h) x[h] = s[h] = visible ? __uint_as_float(raw[h]) * a.scale : -INFINITY;
+            const float top = lu_fold<HG>(x, lane, [](float p, float q) { return fmaxf(p, q); });
+            if (lane < HG) s_warp[warp][lane] = top;
+            ok = lu_agree(bar, 128, ok);
+            if (!ok) {
+                if (gt == 0) atomicExch(a.status, 24);
+                break;
+            }
+            bool moved = false;
+            float keep[HG];
+#pragma unroll
+            for (int h = 0; h < HG; h += 4) {
+                float4 v = *reinterpret_cast<const float4*>(&s_warp[group * 4][h]);
+#pragma unroll
+                for (int w = 1; w < 4; ++w) {
+                    const float4 u = *reinterpret_cast<const float4*>(&s_warp[group * 4 + w][h]);
+                    v = make_float4(fmaxf(v.x, u.x), fmaxf(v.y, u.y), fmaxf(v.z, u.z), fmaxf(v.w, u.w));
+                }
+                const float tile_max[4] = {v.x, v.y, v.z, v.w};
 #pragma unroll
                 for (int i = 0; i < 4; ++i) {
-                    const float x = s[m][2 * kk + (i >> 1)][(i & 1) * 2], y = s[m][2 * kk + (i >> 1)][(i & 1) * 2 + 1];
-                    pf[m][i] = la_pack(x, y);
-                    pr[m][i] = la_rest(x, y, pf[m][i]);
-                }
-#pragma unroll
-            for (int j = 0; j < NT; j += 2) {
-                uint32_t b[4];
-                la_ldm4_trans(b, rows + (kk * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * PITCH + j * 8 + (lane >> 4) * 8);
-#pragma unroll
-                for (int m = 0; m < MT; ++m) {
-                    la_mma(o[m][j], pf[m], b[0], b[1]);
-                    la_mma(o[m][j + 1], pf[m], b[2], b[3]);
-                    la_mma(o[m][j], pr[m], b[0], b[1]);
-                    la_mma(o[m][j + 1], pr[m], b[2], b[3]);
+                    keep[h + i] = 1.f;
+                    if (t == 0 || tile_max[i] > m[h + i] + kSlack) {  // the same in every thread
+                        keep[h + i] = t == 0 ? 0.f : __expf(m[h + i] - tile_max[i]);
+                        m[h + i] = tile_max[i];
+                        moved = true;
+                    }
                 }
             }
-        }
-        __syncwarp();  // the stage is refilled by the next iteration's load
-    }
-    asm volatile("cp.async.wait_group 0;" ::: "memory");
-
-    auto store = [&](int m, int h, int j, float x, float y, float f) {  // two neighbouring values of head row (m, h)
-        const int head = head0 + m * 16 + gid + 8 * h;
-        *reinterpret_cast<__nv_bfloat162*>(a.out.h + ((int64_t)head * a.n_rows + e.row) * RANK + col0 + j * 8 + 2 * tq) = __floats2bfloat162_rn(x * f, y * f);
-    };
-    if (e.n_shares == 1) {
+            // weights and rests of two heads at a time
+            uint32_t hi[HG / 2], lo[HG / 2];
 #pragma unroll
-        for (int m = 0; m < MT; ++m)
-#pragma unroll
-            for (int h = 0; h < 2; ++h) {
-                const int head = head0 + m * 16 + gid + 8 * h;
-                if (head >= a.heads) continue;
-                const float f = sigmoid_f(a.gate.at(e.packed, a.gate_col + head)) / l_run[m][h];
-#pragma unroll
-                for (int j = 0; j < NT; ++j) store(m, h, j, o[m][j][2 * h], o[m][j][2 * h + 1], f);
+            for (int h = 0; h < HG; h += 2) {
+                const float p0 = visible ? __expf(s[h] - m[h]) : 0.f, p1 = visible ? __expf(s[h + 1] - m[h + 1]) : 0.f;
+                l[h] = fmaf(l[h], keep[h], p0);
+                l[h + 1] = fmaf(l[h + 1], keep[h + 1], p1);
+                hi[h / 2] = la_pack(p0, p1);
+                lo[h / 2] = la_rest(p0, p1, hi[h / 2]);
             }
-        return;
-    }
-    const int groups = gridDim.y;
-    auto slot = [&](int entry) { return ((int64_t)entry * groups + blockIdx.y) * HEADS; };
-#pragma unroll
-    for (int m = 0; m < MT; ++m)
-#pragma unroll
-        for (int h = 0; h < 2; ++h) {
-            const int item = m * 16 + gid + 8 * h;
-            if (head0 + item >= a.heads) continue;
-            float* po = a.part_o + (slot(blockIdx.x) + item) * RANK + col0;
-#pragma unroll
-            for (int j = 0; j < NT; ++j) *reinterpret_cast<float2*>(po + j * 8 + 2 * tq) = make_float2(o[m][j][2 * h], o[m][j][2 * h + 1]);
-            if (warp == 0 && tq == 0) *reinterpret_cast<float2*>(a.part_ml + (slot(blockIdx.x) + item) * 2) = make_float2(m_run[m][h], l_run[m][h]);
-        }
-    __shared__ int s_last;
-    __threadfence();
-    __syncthreads();
-    if (tid == 0) {
-        int32_t* counter = a.counters + (int64_t)e.first * groups + blockIdx.y;
-        s_last = atomicAdd(counter, 1) == e.n_shares - 1 ? 1 : 0;
-        if (s_last) *counter = 0;
-    }
-    __syncthreads();
-    if (!s_last) return;
-    __threadfence();
+            if (t > 0) {
+                ok = lu_bar_wait(o_done, (t - 1) & 1);  // the weights' buffer is free and the outputs stand still
+                __syncwarp();
+                lu_fence_after();
+                if (moved) {
 #pragma unroll 1
-    for (int m = 0; m < MT; ++m)
-#pragma unroll 1
-        for (int h = 0; h < 2; ++h) {
-            const int item = m * 16 + gid + 8 * h, head = head0 + item;
-            if (head >= a.heads) continue;
-            float mx = -INFINITY;
-            for (int sh = 0; sh < e.n_shares; ++sh) mx = fmaxf(mx, __ldcg(a.part_ml + (slot(e.first + sh) + item) * 2));
-            float l = 0.f, acc[NT][2];
+                    for (int c = 0; c < OWN * 2; ++c) {
+                        lu_tmem_load<HG>(my_tmem + c * NH, raw);
+                        lu_tmem_wait();
 #pragma unroll
-            for (int j = 0; j < NT; ++j) acc[j][0] = acc[j][1] = 0.f;
-            for (int sh = 0; sh < e.n_shares; ++sh) {
-                const int64_t at = slot(e.first + sh) + item;
-                const float2 ml = __ldcg(reinterpret_cast<const float2*>(a.part_ml + at * 2));
-                if (ml.x == -INFINITY) continue;
-                const float f = __expf(ml.x - mx);
-                l += ml.y * f;
-#pragma unroll
-                for (int j = 0; j < NT; ++j) {
-                    const float2 v = __ldcg(reinterpret_cast<const float2*>(a.part_o + at * RANK + col0 + j * 8 + 2 * tq));
-                    acc[j][0] = fmaf(v.x, f, acc[j][0]);
-                    acc[j][1] = fmaf(v.y, f, acc[j][1]);
+                        for (int h = 0; h < HG; ++h) raw[h] = __float_as_uint(__uint_as_float(raw[h]) * keep[h]);
+                        lu_tmem_store<HG>(my_tmem + c * NH, raw);
+                    }
+                    asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory");
                 }
             }
-            const float f = sigmoid_f(a.gate.at(e.packed, a.gate_col + head)) / l;
+            uint8_t* col = ps + (gt >> 6) * (2 * NH * 128) + h0 * 128 + (gt & 7) * 2;
+            const int piece = (gt & 63) >> 3;
 #pragma unroll
-            for (int j = 0; j < NT; ++j) store(m, h, j, acc[j][0], acc[j][1], f);
+            for (int h = 0; h < HG; ++h) {
+                const int at = h * 128 + ((piece ^ ((h0 + h) & 7)) << 4);
+                *reinterpret_cast<uint16_t*>(col + at) = (uint16_t)(h & 1 ? hi[h / 2] >> 16 : hi[h / 2]);
+                *reinterpret_cast<uint16_t*>(col + NH * 128 + at) = (uint16_t)(h & 1 ? lo[h / 2] >> 16 : lo[h / 2]);
+            }
+            asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
+            lu_fence_before();
+            lu_bar_arrive(p_full);
         }
+        if (ok && tiles > 0) ok = lu_bar_wait(o_done, (tiles - 1) & 1);
+        __syncwarp();
+        lu_fence_after();
+        const float sum = lu_fold<HG>(l, lane, [](float p, float q) { return p + q; });
+        lu_agree(bar, 128, true);  // the maxima have been read
+        if (lane < HG) s_warp[warp][lane] = sum;
+        if (!lu_agree(bar, 128, ok) && gt == 0) atomicExch(a.status, 25);
+        auto slot = [&](int entry) { return ((int64_t)entry * gridDim.y + blockIdx.y) * NH; };
+        auto ml_at = [&](int entry, int h) { return a.part_ml + (slot(entry) * CS + part * NH + h) * 2; };
+        if (gt < HG && h0 + gt < heads) {  // thread gt finishes head h0 + gt
+            float total = 0.f, mine = -INFINITY;
+#pragma unroll
+            for (int w = 0; w < 4; ++w) total += s_warp[group * 4 + w][gt];
+#pragma unroll
+            for (int h = 0; h < HG; ++h)
+                if (h == gt) mine = m[h];
+            if (e.n_shares == 1) s_factor[0][h0 + gt] = sigmoid_f(a.gate.at(e.packed, a.gate_col + head0 + h0 + gt)) / total;
+            else *reinterpret_cast<float2*>(ml_at(blockIdx.x, h0 + gt)) = make_float2(mine, total);
+        }
+        lu_agree(bar, 128, true);
+#pragma unroll
+        for (int c = 0; c < OWN; ++c) {
+            uint32_t o[HG], rest[HG];
+            if (tiles > 0) {
+                lu_tmem_load<HG>(my_tmem + c * 2 * NH, o);
+                lu_tmem_load<HG>(my_tmem + c * 2 * NH + NH, rest);
+                lu_tmem_wait();
+            }
+#pragma unroll
+            for (int h = 0; h < HG; ++h) {
+                if (h0 + h >= heads) continue;
+                const float v = tiles > 0 ? __uint_as_float(o[h]) + __uint_as_float(rest[h]) : 0.f;
+                if (e.n_shares == 1)
+                    a.out.h[((int64_t)(head0 + h0 + h) * a.n_rows + e.row) * RANK + col0 + c * LU_COLS + gt] = __float2bfloat16_rn(v * s_factor[0][h0 + h]);
+                else
+                    a.part_o[(slot(blockIdx.x) + h0 + h) * RANK + col0 + c * LU_COLS + gt] = v;
+            }
+        }
+        if (e.n_shares > 1) {
+            __threadfence();
+            lu_agree(LU_GROUPS + 1, LU_SOFTMAX, true);
+            if (tid == 0) {
+                int32_t* counter = a.counters + ((int64_t)e.first * gridDim.y + blockIdx.y) * CS + part;
+                s_last = atomicAdd(counter, 1) == e.n_shares - 1 ? 1 : 0;
+                if (s_last) *counter = 0;
+            }
+            lu_agree(LU_GROUPS + 1, LU_SOFTMAX, true);
+            if (s_last) {
+                __threadfence();
+                if (tid < heads) {  // what every share of head `tid` is multiplied by
+                    float mx = -INFINITY, total = 0.f;
+                    for (int sh = 0; sh < e.n_shares; ++sh) mx = fmaxf(mx, __ldcg(ml_at(e.first + sh, tid)));
+                    for (int sh = 0; sh < e.n_shares; ++sh) {
+                        const float2 ml = __ldcg(reinterpret_cast<const float2*>(ml_at(e.first + sh, tid)));
+                        const float f = ml.x == -INFINITY ? 0.f : __expf(ml.x - mx);
+                        s_factor[sh][tid] = f;
+                        total = fmaf(ml.y, f, total);
+                    }
+                    const float g = sigmoid_f(a.gate.at(e.packed, a.gate_col + head0 + tid)) / total;
+                    for (int sh = 0; sh < e.n_shares; ++sh) s_factor[sh][tid] *= g;
+                }
+                lu_agree(LU_GROUPS + 1, LU_SOFTMAX, true);
+#pragma unroll 4
+                for (int i = tid; i < heads * (OWN * LU_COLS / 4); i += LU_SOFTMAX) {
+                    const int h = i / (OWN * LU_COLS / 4), c = col0 + (i - h * (OWN * LU_COLS / 4)) * 4;
+                    float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+                    for (int sh = 0; sh < e.n_shares; ++sh) {
+                        const float4 v = __ldcg(reinterpret_cast<const float4*>(a.part_o + (slot(e.first + sh) + h) * RANK + c));
+                        const float f = s_factor[sh][h];
+                        acc = make_float4(fmaf(v.x, f, acc.x), fmaf(v.y, f, acc.y), fmaf(v.z, f, acc.z), fmaf(v.w, f, acc.w));
+                    }
+                    a.out.put4((int64_t)(head0 + h) * a.n_rows + e.row, c, acc);
+                }
+            }
+        }
+    }
+    lu_fence_before();
+    __syncthreads();
+    if (warp == LOADER) {
+        lu_fence_after();
+        asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem), "r"(L::TMEM) : "memory");
+    }
 }
 
 // ------------------------------------------------------------------------------------------------ general kernel
@@ -445,36 +613,44 @@ __global__ void __launch_bounds__(256) split_rows_kernel(const float* x, int ldx
     }
 }
 
-template <int RANK, int MT>
-void launch_tc(const LatentAttnArgs& a, cudaStream_t s) {
-    constexpr size_t smem = La<RANK, MT>::BYTES;
+template <int MB, int NH>
+void launch_umma(const LatentAttnArgs& a, cudaStream_t s) {
+    constexpr size_t smem = Lu<MB, NH>::BYTES;
+    static_assert(smem <= (size_t)227 * 1024, "shared memory");
     int shift = 0;
     while ((1 << shift) < a.block_tokens) ++shift;
-    ensure_dynamic_smem(reinterpret_cast<const void*>(&latent_tc_kernel<RANK, MT>), smem);
-    launch_pdl(latent_tc_kernel<RANK, MT>, dim3((unsigned)a.n_entries, (unsigned)latent_tc_groups(a.heads)), dim3(LA_WARPS * 32), smem, s, a, shift);
+    ensure_dynamic_smem(reinterpret_cast<const void*>(&latent_umma_kernel<MB, NH>), smem);
+    launch_pdl(latent_umma_kernel<MB, NH>, dim3((unsigned)a.n_entries, (unsigned)latent_tc_groups(a.heads), (unsigned)Lu<MB, NH>::CS), dim3(LU_THREADS), smem, s,
+               *static_cast<const CUtensorMap*>(a.pool_map), a, shift, std::min(a.block_tokens, LU_KEYS), (int)a.pool_rows);
 }
 
-template <int RANK>
-void launch_tc_heads(const LatentAttnArgs& a, cudaStream_t s) {
-    if (latent_tc_heads(a.heads) == 16) launch_tc<RANK, 1>(a, s);
-    else launch_tc<RANK, 2>(a, s);
+template <int MB>
+void launch_umma_heads(const LatentAttnArgs& a, cudaStream_t s) {
+    if (latent_tc_heads(a.heads) == 16) launch_umma<MB, 16>(a, s);
+    else launch_umma<MB, 32>(a, s);
 }
 
 }  // namespace
 
 int latent_tc_rank(int kv_rank, int block_tokens) {
-    if (block_tokens <= 0 || (block_tokens & (block_tokens - 1)) != 0) return 0;
-    for (int r : {64, 128, 256, 512})
-        if (kv_rank <= r) return r;
-    return 0;
+    if (block_tokens < 8 || (block_tokens & (block_tokens - 1)) != 0) return 0;
+    const int r = (kv_rank + LU_COLS - 1) / LU_COLS * LU_COLS;
+    return r <= 4 * LU_COLS ? r : 0;
 }
+
+void latent_pool_map(void* out, const void* pool, int64_t rows, int rank, int block_tokens) {
+    if (rows > (int64_t)1 << 30) throw std::runtime_error("latent_pool_map: the pool has too many rows");
+    encode_tma_2d(out, false, pool, (uint64_t)rank, (uint64_t)rows, (uint64_t)rank * 2, 64, (uint32_t)std::min(block_tokens, LU_KEYS), true);
+}
+
+int latent_tc_ctas(int heads, int rank) { return latent_tc_groups(heads) * (rank == 4 * LU_COLS ? 2 : 1); }
 
 int latent_tc_heads(int heads) { return heads <= 16 ? 16 : 32; }
 
-int latent_max_shared_entries(int head_groups) { return std::max(LA_SHARED_ROWS + LA_SHARED_ROWS / 2, LA_TARGET_CTAS / head_groups) + 1; }
-int latent_max_entries(int tokens, int head_groups) { return std::max(tokens, latent_max_shared_entries(head_groups)); }
+int latent_max_shared_entries(int ctas) { return std::max(LA_SHARED_ROWS + LA_SHARED_ROWS / 2, LA_TARGET_CTAS / ctas) + 1; }
+int latent_max_entries(int tokens, int ctas) { return std::max(tokens, latent_max_shared_entries(ctas)); }
 
-void plan_latent_attention(const int32_t* start_pos, const int32_t* n_tokens, const int32_t* n_blocks, int lanes, int head_groups, int wide_from,
+void plan_latent_attention(const int32_t* start_pos, const int32_t* n_tokens, const int32_t* n_blocks, int lanes, int ctas, int wide_from,
                            bool shares, LatentPlan& plan) {
     plan.entries.clear();
     plan.rows.clear();
@@ -489,10 +665,11 @@ void plan_latent_attention(const int32_t* start_pos, const int32_t* n_tokens, co
     // a row more than twice as long as the mean is cut.
     int share = 1 << 30;
     if (shares && rows > 0 && rows <= LA_SHARED_ROWS) {
-        const bool filled = rows * head_groups >= LA_TARGET_CTAS;
-        const int slots = filled ? rows + rows / 2 : std::max(rows, LA_TARGET_CTAS / head_groups);
+        const bool filled = rows * ctas >= LA_TARGET_CTAS;
+        const int slots = filled ? rows + rows / 2 : std::max(rows, LA_TARGET_CTAS / ctas);
         share = (int)std::max<int64_t>(LA_MIN_SHARE, filled ? 2 * (keys / rows) : (keys + slots - 1) / slots);
-        for (;; share += LA_KT) {
+        share = (share + LU_KEYS - 1) / LU_KEYS * LU_KEYS;
+        for (;; share += LU_KEYS) {
             int64_t n = 0;
             for (int i = 0; i < lanes; ++i)
                 if (n_tokens[i] < wide_from)
@@ -518,11 +695,12 @@ void launch_latent_attention(const LatentAttnArgs& a, cudaStream_t s) {
     if (a.out.ld != a.rank) throw std::runtime_error("launch_latent_attention: the output's rows are as wide as the latent");
     if (a.q_h != nullptr) {
         if (!a.pool_f16 || a.out.h == nullptr) throw std::runtime_error("launch_latent_attention: f16 queries go with f16 pages and a bf16 output");
+        if (a.pool_map == nullptr || a.status == nullptr) throw std::runtime_error("launch_latent_attention: the tensor-core kernel needs the pool's map and a status word");
         switch (a.rank) {
-            case 64: launch_tc_heads<64>(a, s); break;
-            case 128: launch_tc_heads<128>(a, s); break;
-            case 256: launch_tc_heads<256>(a, s); break;
-            case 512: launch_tc_heads<512>(a, s); break;
+            case 128: launch_umma_heads<1>(a, s); break;
+            case 256: launch_umma_heads<2>(a, s); break;
+            case 384: launch_umma_heads<3>(a, s); break;
+            case 512: launch_umma_heads<4>(a, s); break;
             default: throw std::runtime_error("launch_latent_attention: unsupported rank");
         }
     } else {

@@ -14,6 +14,8 @@ struct LatentAttnArgs {
     const float* q_f = nullptr;      // the same in f32 (general kernel)
     const void* pool = nullptr;      // [blocks * block_tokens][rank]
     int pool_f16 = 1;
+    const void* pool_map = nullptr;  // host: latent_pool_map of the pool (tensor-core kernel)
+    int64_t pool_rows = 0;
     const uint32_t* tables = nullptr;
     // work list, 8 ints each, 32-byte aligned: (query row, share, n_shares, last visible position, table offset, packed row,
     // first entry of the query row, 0)
@@ -25,18 +27,23 @@ struct LatentAttnArgs {
     Shares gate;                     // a head's output is multiplied by sigmoid(gate[packed row][gate_col + head])
     int gate_col = 0;
     RowImage out;                    // row head * n_rows + query row, ld = rank
-    // shares (tensor-core kernel): unnormalised partial outputs [entry][heads padded][rank], (max, sum) pairs, and counters
-    // [entries][head groups] that are zero before the first call and after every call
+    // shares (tensor-core kernel): unnormalised partial outputs [entry][heads padded][rank], two (max, sum) pairs per head, and
+    // counters [entries][CTAs per entry] that are zero before the first call and after every call
     float* part_o = nullptr;
     float* part_ml = nullptr;
     int32_t* counters = nullptr;
+    int32_t* status = nullptr;       // receives a non-zero code when a bounded wait gave up
 };
 
-// The tensor-core kernel's rank for a latent of `kv_rank` values (64, 128, 256 or 512), or 0 when it does not cover the case.
+// The tensor-core kernel's rank for a latent of `kv_rank` values (a multiple of 128 up to 512), or 0 when it does not cover the
+// case.
 int latent_tc_rank(int kv_rank, int block_tokens);
-// Heads of one CTA of the tensor-core kernel, and CTAs per work item.
+// The descriptor (128 bytes, 64-byte aligned) through which that kernel loads an f16 pool of `rows` rows.
+void latent_pool_map(void* out, const void* pool, int64_t rows, int rank, int block_tokens);
+// Heads of one CTA of the tensor-core kernel, groups of that many, and CTAs per work item (a wide latent is shared by two).
 int latent_tc_heads(int heads);
 inline int latent_tc_groups(int heads) { return (heads + latent_tc_heads(heads) - 1) / latent_tc_heads(heads); }
+int latent_tc_ctas(int heads, int rank);
 constexpr int kLatentMaxRank = 1024;  // of the general kernel
 
 // Host-side work list: one entry per token of lane i with n_tokens[i] < wide_from, cut into key shares while that fills the GPU.
@@ -46,11 +53,11 @@ struct LatentPlan {
     int n_entries() const { return (int)entries.size() / 8; }
     int n_rows() const { return (int)rows.size(); }
 };
-void plan_latent_attention(const int32_t* start_pos, const int32_t* n_tokens, const int32_t* n_blocks, int lanes, int head_groups, int wide_from,
+void plan_latent_attention(const int32_t* start_pos, const int32_t* n_tokens, const int32_t* n_blocks, int lanes, int ctas, int wide_from,
                            bool shares, LatentPlan& plan);
 // Upper bounds for a tick of at most `tokens` tokens: entries, and entries with partial results.
-int latent_max_entries(int tokens, int head_groups);
-int latent_max_shared_entries(int head_groups);
+int latent_max_entries(int tokens, int ctas);
+int latent_max_shared_entries(int ctas);
 
 void launch_latent_attention(const LatentAttnArgs& a, cudaStream_t s);
 

@@ -316,7 +316,11 @@ void MixerLm::alloc_run(int run) {
             st.state.alloc(halves * (size_t)d.heads * d.vdim * linear_state_key_pad(d.dim) * 4);
             break;
         }
-        case MixerKind::Latent: pages(st.k_pool, 1); break;
+        case MixerKind::Latent:
+            pages(st.k_pool, 1);
+            if (latent_geo_[(size_t)w.geometry].tc)
+                latent_pool_map(st.pool_map, st.k_pool.ptr(), pool_->max_blocks() * cfg_.block_tokens, w.row_width, cfg_.block_tokens);
+            break;
         case MixerKind::MinGru: st.state.alloc(halves * (size_t)s.gru.width * 4); break;
     }
 }
@@ -326,7 +330,7 @@ void MixerLm::alloc_activations() {
     const int B = cfg_.max_batch_lanes, C = ms_.width;
     int64_t in_rows = 0, mix = 0, a_w = 0, b_w = 0, ff = 0, hd = 0, raw = 0, dqk = 0, dv = 0, dh = 0, attn = 0;
     int64_t q_lat = 0, uq = 0, lat = 0, cat = 0;  // widths of latent attention's rows, and of `out`'s input with both branches
-    int lat_groups = 1;
+    int lat_ctas = 1;
     int64_t lat_part = 0;
     for (size_t l = 0; l < lw_.size(); ++l) {
         const MixerLayerSpec& s = ms_.layers[l];
@@ -342,8 +346,8 @@ void MixerLm::alloc_activations() {
                 lat = std::max(lat, (int64_t)a.heads * w.row_width);
                 const LatentGeometry& g = latent_geo_[(size_t)w.geometry];
                 if (g.wide) attn = std::max(attn, (int64_t)a.heads * w.q_width);
-                lat_groups = std::max(lat_groups, g.groups);
-                if (g.tc) lat_part = std::max(lat_part, (int64_t)latent_max_shared_entries(g.groups) * g.groups * latent_tc_heads(a.heads) * w.row_width);
+                lat_ctas = std::max(lat_ctas, g.ctas);
+                if (g.tc) lat_part = std::max(lat_part, (int64_t)latent_max_shared_entries(g.ctas) * latent_tc_groups(a.heads) * latent_tc_heads(a.heads) * w.row_width);
             }
             continue;
         }
@@ -391,7 +395,7 @@ void MixerLm::alloc_activations() {
     if (lat_part > 0) {
         lat_part_o_.alloc((size_t)lat_part * 4);
         lat_part_ml_.alloc((size_t)lat_part / 64 * 2 * 4);
-        lat_counters_.alloc((size_t)latent_max_shared_entries(1) * lat_groups * 4);
+        lat_counters_.alloc((size_t)latent_max_shared_entries(1) * lat_ctas * 4);
         lat_counters_.zero(stream_);
     }
     attn_.alloc((size_t)(T * attn) * 4);
@@ -416,7 +420,7 @@ void MixerLm::alloc_activations() {
             extra += (size_t)(T + B) * 8 + 64;
         }
     }
-    for (const LatentGeometry& g : latent_geo_) extra += (size_t)latent_max_entries((int)T, g.groups) * 32 + (size_t)T * 4 + 32;
+    for (const LatentGeometry& g : latent_geo_) extra += (size_t)latent_max_entries((int)T, g.ctas) * 32 + (size_t)T * 4 + 32;
     if (!latent_geo_.empty()) extra += (size_t)B * sizeof(LaneHeader) + (size_t)(T + B) * 8 + (size_t)T * 4 + (size_t)(pool_->max_blocks() + B) * 4 + 64;
     attn_part_o_.alloc(part_o);
     attn_part_ml_.alloc(part_ml);

@@ -86,6 +86,7 @@ private:
     struct RunState {
         DevBuf k_pool, v_pool;  // latent attention: k_pool only
         DevBuf state, kept, tail;
+        alignas(64) unsigned char pool_map[128] = {};  // latent attention on the tensor cores (see latent_pool_map)
     };
     // Layers with the same heads share a tick's attention work list.
     struct Geometry {
@@ -98,7 +99,7 @@ private:
     };
     // Latent-attention layers with the same kernel and grid share a tick's work list.
     struct LatentGeometry {
-        int groups = 1;      // CTAs per entry
+        int ctas = 1;        // CTAs per entry
         bool tc = false;     // tensor-core kernel
         bool wide = false;   // lanes with many tokens run on expanded keys and values
         LatentPlan plan;
@@ -139,7 +140,7 @@ private:
     Shares matmul(const Dense& W, const RowImage& x, int T, DevBuf& y, int scratch);
     void matmul_scatter(const Dense& W, const RowImage& x, int T, const MatmulScatter& to);
     void set_norm(RowUpdateArgs& a, const Norm& n) const;
-    int latent_geometry(int groups, bool tc, bool wide);
+    int latent_geometry(int ctas, bool tc, bool wide);
     void plan_latent(Tick& t, const std::vector<int32_t>& start, const std::vector<int32_t>& n_tokens, const std::vector<int32_t>& n_blocks, KvReservation& r);
 
     // Branch outputs not yet added to the residual stream.

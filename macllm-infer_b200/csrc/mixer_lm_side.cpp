@@ -76,11 +76,11 @@ void MixerLm::load_side_by_side(const SafetensorsFile& f, int l) {
     upload_dense(f, out, C, w.mix_cols + s.ff, w.out);
 }
 
-int MixerLm::latent_geometry(int groups, bool tc, bool wide) {
+int MixerLm::latent_geometry(int ctas, bool tc, bool wide) {
     for (size_t i = 0; i < latent_geo_.size(); ++i)
-        if (latent_geo_[i].groups == groups && latent_geo_[i].tc == tc && latent_geo_[i].wide == wide) return (int)i;
+        if (latent_geo_[i].ctas == ctas && latent_geo_[i].tc == tc && latent_geo_[i].wide == wide) return (int)i;
     LatentGeometry g;
-    g.groups = groups;
+    g.ctas = ctas;
     g.tc = tc;
     g.wide = wide;
     latent_geo_.push_back(std::move(g));
@@ -106,7 +106,7 @@ void MixerLm::load_latent(const SafetensorsFile& f, int l) {
                 wide = true;
                 w.q_width = d;
             }
-    w.geometry = latent_geometry(tc_rank > 0 ? latent_tc_groups(H) : 1, tc_rank > 0, wide);
+    w.geometry = latent_geometry(tc_rank > 0 ? latent_tc_ctas(H, w.row_width) : 1, tc_rank > 0, wide);
     if (wide && iota_.size() == 0) {
         std::vector<uint32_t> n((size_t)(pool_->max_blocks() + cfg_.max_batch_lanes));
         for (size_t i = 0; i < n.size(); ++i) n[i] = (uint32_t)i;
@@ -148,7 +148,7 @@ void MixerLm::load_latent(const SafetensorsFile& f, int l) {
 void MixerLm::plan_latent(Tick& t, const std::vector<int32_t>& start, const std::vector<int32_t>& n_tokens, const std::vector<int32_t>& n_blocks, KvReservation& r) {
     bool any_wide = false;
     for (LatentGeometry& g : latent_geo_) {
-        plan_latent_attention(start.data(), n_tokens.data(), n_blocks.data(), t.B, g.groups, g.wide ? kWideFrom : INT_MAX, g.tc, g.plan);
+        plan_latent_attention(start.data(), n_tokens.data(), n_blocks.data(), t.B, g.ctas, g.wide ? kWideFrom : INT_MAX, g.tc, g.plan);
         g.off_entries = stage_bytes(t, g.plan.entries.data(), g.plan.entries.size() * 4);
         g.off_rows = stage_bytes(t, g.plan.rows.data(), g.plan.rows.size() * 4);
         any_wide |= g.wide;
@@ -321,6 +321,9 @@ void MixerLm::run_latent(const Tick& t, int run, const Shares& y, const RowImage
         else a.q_f = q_lat_.as<float>();
         a.pool = rs_[(size_t)run].k_pool.ptr();
         a.pool_f16 = cfg_.kv_f16 ? 1 : 0;
+        a.pool_map = rs_[(size_t)run].pool_map;
+        a.pool_rows = pool_->max_blocks() * cfg_.block_tokens;
+        a.status = status_.as<int32_t>();
         a.tables = t.bd.tables;
         a.entries = reinterpret_cast<const int32_t*>(t.dp + g.off_entries);
         a.n_entries = g.plan.n_entries();
