@@ -1,22 +1,19 @@
 // See latent_attention.h.
 //
-// Tensor-core kernel (tcgen05): one CTA per (query row, share of its keys, up to 32 heads).  Tiles of 128 cached vectors arrive by
-// TMA, 128 bytes wide and swizzled, in chunks of 128 columns.  A tile is an operand twice: with the vectors' columns as the
-// reduction it gives the scores transposed (keys x heads), and read the other way round, with the keys as the reduction, it gives
-// the outputs transposed (columns x heads) - so the wide side of both products fills the tensor core's 128 rows and the few heads
-// are its columns.  Four groups of four warps, a quarter of the heads each, hold one key per thread: scores from tensor memory, the
-// heads' maxima over the keys by a folding exchange, softmax weights in f32, which go back to shared memory as two f16 numbers
-// each (high part and rest, as columns of their own, added up at the end).  A latent of 512 columns is too wide for a second tile
-// beside the first in shared memory, so two CTAs take half of the output columns each: both form all scores, and the chunks a CTA
-// needs for the scores only leave the ring at once.  The scores of the next tile are thus computed while the weights of this one
-// are being formed.  The running maximum moves only when a tile exceeds it by more than kSlack, so the accumulators
-// in tensor memory are hardly ever rescaled.  When few rows are in flight their keys are shared out over several CTAs; the one
-// that finishes last adds the shares in order.  Every wait is bounded (see hgemm_tc.cu).
+// Tensor-core kernel (tcgen05): one CTA per (query row, share of its keys, up to 32 heads).  Tiles of 128 cached vectors arrive in
+// chunks of 128 columns as 128-byte swizzled rows, by 16-byte cp.async (TMA boxes as small as a page's part of a chunk brought
+// them no faster).  A tile is an operand twice: with the vectors' columns as the reduction it gives the scores transposed (keys x
+// heads), and read the other way round, with the keys as the reduction, it gives the outputs transposed (columns x heads) - so the
+// wide side of both products fills the tensor core's 128 rows and the few heads are its columns.  Four groups of four warps, a
+// quarter of the heads each, hold one key per thread: scores from tensor memory, the heads' maxima over the keys by a folding
+// exchange, softmax weights in f32, which go back to shared memory as two f16 numbers each (high part and rest, as columns of
+// their own, added up at the end).  The MMA issuer takes what is ready first, the weights of a tile or the next chunk of the tile
+// after it, so scores go ahead of outputs as far as the ring holds them.  The running maximum moves only when a tile exceeds it by
+// more than kSlack, so the accumulators in tensor memory are hardly ever rescaled.  When few rows are in flight their keys are
+// shared out over several CTAs; the one that finishes last adds the shares in order.  Every wait is bounded (see hgemm_tc.cu).
 #include "latent_attention.h"
 #include "device_util.h"
-#include "hgemm_tc.h"
 #include <algorithm>
-#include <cuda.h>
 
 namespace mk {
 
@@ -28,7 +25,8 @@ constexpr int LU_CHUNK = LU_KEYS * LU_COLS * 2;
 constexpr int LU_BLOCK = LU_KEYS * 128;  // bytes of the 64 columns that share swizzled rows
 constexpr int LU_GROUPS = 4;           // softmax groups of four warps
 constexpr int LU_SOFTMAX = LU_GROUPS * 128;
-constexpr int LU_THREADS = LU_SOFTMAX + 64;  // and the loader's and the MMA issuer's warps
+constexpr int LU_LOADERS = 128;
+constexpr int LU_THREADS = LU_SOFTMAX + LU_LOADERS + 32;  // and the MMA issuer's warp
 constexpr float kSlack = 8.f;         // weights stay below e^8, well inside f16
 constexpr uint32_t LU_SPIN_LIMIT = 1u << 22;
 constexpr int LA_SMS = 148;
@@ -54,14 +52,24 @@ __device__ __forceinline__ bool lu_bar_wait(uint64_t* bar, uint32_t parity) {
     }
     return false;
 }
-__device__ __forceinline__ void lu_bar_arrive(uint64_t* bar) { asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];" ::"r"(lu_smem(bar)) : "memory"); }
-__device__ __forceinline__ void lu_bar_expect(uint64_t* bar, uint32_t bytes) {
-    asm volatile("mbarrier.arrive.expect_tx.shared::cta.b64 _, [%0], %1;" ::"r"(lu_smem(bar)), "r"(bytes) : "memory");
+__device__ __forceinline__ bool lu_bar_test(uint64_t* bar, uint32_t parity) {
+    uint32_t done;
+    asm volatile(
+        "{\n\t.reg .pred p;\n\t"
+        "mbarrier.test_wait.parity.shared::cta.b64 p, [%1], %2;\n\t"
+        "selp.u32 %0, 1, 0, p;\n\t}"
+        : "=r"(done)
+        : "r"(lu_smem(bar)), "r"(parity)
+        : "memory");
+    return done != 0;
 }
-__device__ __forceinline__ void lu_tma(void* dst, const void* tmap, int x, int y, uint64_t* bar) {
-    asm volatile("cp.async.bulk.tensor.2d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3}], [%4];" ::"r"(lu_smem(dst)), "l"(tmap), "r"(x), "r"(y),
-                 "r"(lu_smem(bar))
-                 : "memory");
+__device__ __forceinline__ void lu_bar_arrive(uint64_t* bar) { asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];" ::"r"(lu_smem(bar)) : "memory"); }
+// 16 bytes (zeros when there is no source), counted on the barrier together with the thread's other copies by lu_copies_arrive.
+__device__ __forceinline__ void lu_copy16(uint32_t dst, const void* src, bool valid) {
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(valid ? 16 : 0) : "memory");
+}
+__device__ __forceinline__ void lu_copies_arrive(uint64_t* bar) {
+    asm volatile("cp.async.mbarrier.arrive.noinc.shared::cta.b64 [%0];" ::"r"(lu_smem(bar)) : "memory");
 }
 // Operand of 128-byte swizzled rows, 8-row groups 1024 bytes apart.  Reduction along the rows' bytes: lead is not used; reduction
 // from row to row: lead = distance of the next 64 elements of the other dimension.
@@ -155,18 +163,16 @@ struct Lu {
     static constexpr int Q_BYTES = NH * RANK * 2;                                               // [column block][head][64]
     static constexpr int P_BYTES = 2 * NH * LU_KEYS * 2;                                        // [key block][weights | rests][64]
     static constexpr size_t BYTES = (size_t)STAGES * LU_CHUNK + Q_BYTES + P_BYTES + 1024 + 256;
-    static constexpr int CS = MB == 4 ? 2 : 1;   // CTAs that share the output columns
-    static constexpr int OWN = MB / CS;          // chunks of a CTA's own
-    static constexpr int S_COL = OWN * 2 * NH;   // tensor memory: outputs (high | rest) of every chunk, then two tiles' scores
-    static constexpr uint32_t TMEM = S_COL + 2 * NH <= 64 ? 64 : (S_COL + 2 * NH <= 128 ? 128 : (S_COL + 2 * NH <= 256 ? 256 : 512));
-    // chunks of the next tile that reach the ring while this tile's own ones are in use
-    static constexpr int AHEAD = STAGES - OWN < MB ? STAGES - OWN : MB;
+    static constexpr int S_COL = MB * 2 * NH;  // tensor memory: outputs (high | rest) of every chunk, then two tiles' scores
+    static constexpr int END_COL = S_COL + 2 * NH;
+    static constexpr uint32_t TMEM = END_COL <= 64 ? 64 : END_COL <= 128 ? 128 : (END_COL <= 256 ? 256 : 512);
+    static_assert(END_COL <= 512, "tensor memory");
 };
 
 template <int MB, int NH>
-__global__ void __launch_bounds__(LU_THREADS, 1) latent_umma_kernel(const __grid_constant__ CUtensorMap tm, LatentAttnArgs a, int bt_shift, int box_rows, int pool_rows) {
+__global__ void __launch_bounds__(LU_THREADS, 1) latent_umma_kernel(LatentAttnArgs a, int bt_shift) {
     using L = Lu<MB, NH>;
-    constexpr int RANK = L::RANK, STAGES = L::STAGES, CS = L::CS, OWN = L::OWN, HG = NH / LU_GROUPS, LOADER = LU_SOFTMAX / 32;
+    constexpr int RANK = L::RANK, STAGES = L::STAGES, HG = NH / LU_GROUPS, LOADER = LU_SOFTMAX / 32;
     extern __shared__ uint8_t lu_raw[];
     uint8_t* ring = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(lu_raw) + 1023) & ~(uintptr_t)1023);
     uint8_t* qs = ring + (size_t)STAGES * LU_CHUNK;
@@ -179,16 +185,13 @@ __global__ void __launch_bounds__(LU_THREADS, 1) latent_umma_kernel(const __grid
     uint64_t* o_done = p_full + 1;                                  // MMA -> softmax: the tile is in the outputs
     __shared__ uint32_t tmem_slot;
     __shared__ __align__(16) float s_warp[LU_SOFTMAX / 32][HG], s_factor[LA_MAX_SHARES][NH];
-    __shared__ int s_last;
+    __shared__ int s_last, s_rows[2][LU_KEYS];
 
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int head0 = blockIdx.y * NH, heads = min(NH, a.heads - head0);
-    const int part = blockIdx.z, col0 = part * OWN * LU_COLS;  // this CTA's output columns
-    // the i-th chunk of a tile to arrive: other CTAs' columns first, then the own ones
-    auto chunk_of = [&](int i) { return CS == 1 ? i : (i < MB - OWN ? (i >= part * OWN ? i + OWN : i) : part * OWN + i - (MB - OWN)); };
     if (tid == 0) {
         for (int i = 0; i < STAGES; ++i) {
-            lu_bar_init(&full[i], 1);
+            lu_bar_init(&full[i], LU_LOADERS);
             lu_bar_init(&empty[i], 1);
         }
         lu_bar_init(q_full, LU_SOFTMAX);
@@ -214,80 +217,63 @@ __global__ void __launch_bounds__(LU_THREADS, 1) latent_umma_kernel(const __grid
     const int k_lo = e.share * chunk, k_hi = min(len, k_lo + chunk);
     const int tiles = k_hi > k_lo ? (k_hi - k_lo + LU_KEYS - 1) / LU_KEYS : 0;
 
-    if (warp == LOADER) {
-        // ---- loader: a lane per box of box_rows keys x 64 columns (at most 32 of them)
-        const int boxes = LU_KEYS / box_rows;  // of a column block
-        const int block = lane / boxes, box = lane - block * boxes;
+    if (warp >= LOADER && warp < LOADER + LU_LOADERS / 32) {
+        // ---- loaders: pool rows of a tile's keys first (one per thread), then 16-byte pieces of the rows
+        static_assert(LU_LOADERS == LU_KEYS, "a loader thread looks up one key");
+        const int lt = tid - LU_SOFTMAX, piece = lt & 15, key0 = lt >> 4;
+        const __half* pool = static_cast<const __half*>(a.pool) + piece * 8;
+        const uint32_t dst0 = lu_smem(ring) + (piece >> 3) * LU_BLOCK;
         auto row_of = [&](int t) {
-            // boxes past the last key start behind the pool and are filled with zeros
-            const int pos = k_lo + t * LU_KEYS + box * box_rows;
-            return pos < k_hi ? (int)(a.tables[e.table_off + (pos >> bt_shift)] << bt_shift) + (pos & ((1 << bt_shift) - 1)) : pool_rows;
+            const int pos = k_lo + t * LU_KEYS + lt;
+            return pos < k_hi ? (int)(a.tables[e.table_off + (pos >> bt_shift)] << bt_shift) + (pos & ((1 << bt_shift) - 1)) : -1;
         };
         uint32_t it = 0;
         bool ok = true;
-        int next = row_of(0);
-        for (int t = 0; t < tiles && ok; ++t) {
-            const int y = next;
-            if (t + 1 < tiles) next = row_of(t + 1);
-            for (int c = 0; c < MB && ok; ++c, ++it) {
-                const uint32_t st = it % STAGES, ph = (it / STAGES) & 1;
-                ok = lu_bar_wait(&empty[st], ph ^ 1);
-                if (!__all_sync(0xffffffffu, ok)) {
-                    if (lane == 0) atomicExch(a.status, 21);
-                    ok = false;
-                    break;
+        if (tiles > 0) s_rows[0][lt] = row_of(0);
+        for (int t = 0; t < tiles; ++t) {
+            ok = lu_agree(LU_GROUPS + 2, LU_LOADERS, ok);  // this tile's rows are there, nobody reads the other buffer any more
+            if (!ok) break;
+            if (t + 1 < tiles) s_rows[(t + 1) & 1][lt] = row_of(t + 1);
+            for (int c = 0; c < MB; ++c, ++it) {
+                const uint32_t st = it % STAGES;
+                ok = lu_bar_wait(&empty[st], ((it / STAGES) & 1) ^ 1);
+                if (!ok) break;
+                const uint32_t dst = dst0 + st * LU_CHUNK;
+                const __half* src = pool + c * LU_COLS;
+#pragma unroll
+                for (int j = 0; j < LU_KEYS / 8; ++j) {
+                    const int key = j * 8 + key0, row = s_rows[t & 1][key];
+                    lu_copy16(dst + key * 128 + (((piece & 7) ^ (key & 7)) << 4), src + (int64_t)max(row, 0) * RANK, row >= 0);
                 }
-                if (lane == 0) lu_bar_expect(&full[st], (uint32_t)LU_CHUNK);
-                __syncwarp();
-                if (block < 2) lu_tma(ring + (size_t)st * LU_CHUNK + block * LU_BLOCK + box * box_rows * 128, &tm, chunk_of(c) * LU_COLS + block * 64, y, &full[st]);
-                __syncwarp();
+                lu_copies_arrive(&full[st]);
             }
         }
-        if (!ok)  // copies still in flight land before the CTA goes
-            for (uint32_t i = it > STAGES ? it - STAGES : 0; i < it; ++i) lu_bar_wait(&full[i % STAGES], (i / STAGES) & 1);
-    } else if (warp == LOADER + 1) {
+        if (!ok) atomicExch(a.status, 21);
+        asm volatile("cp.async.wait_all;" ::: "memory");
+    } else if (warp == LOADER + LU_LOADERS / 32) {
         // ---- MMA issuer
         if (lane == 0 && tiles > 0) {
             const uint32_t i_scores = (1u << 4) | ((uint32_t)(NH >> 3) << 17) | (8u << 24);
             const uint32_t i_out = (1u << 4) | (1u << 15) | ((uint32_t)(2 * NH >> 3) << 17) | (8u << 24);  // A read with the keys as the reduction
             const uint32_t q_addr = lu_smem(qs), p_addr = lu_smem(ps), ring_addr = lu_smem(ring);
             bool ok = true;
-            auto scores = [&](int t, int c0, int c1) {  // chunks c0 .. c1 - 1 of tile t's scores
-                for (int c = c0; c < c1; ++c) {
-                    const uint32_t it = (uint32_t)(t * MB + c), st = it % STAGES;
-                    if (!lu_bar_wait(&full[st], (it / STAGES) & 1)) {
-                        atomicExch(a.status, 22);
-                        ok = false;
-                        return;
-                    }
-                    lu_fence_after();
-                    const uint32_t q_chunk = q_addr + 2 * chunk_of(c) * (NH * 128);
-#pragma unroll
-                    for (int k = 0; k < LU_COLS / 16; ++k) {
-                        const uint32_t block = (uint32_t)k >> 2, step = ((uint32_t)k & 3) * 32;
-                        lu_mma(tmem + L::S_COL + (t & 1) * NH, lu_desc(ring_addr + st * LU_CHUNK + block * LU_BLOCK + step, 16),
-                               lu_desc(q_chunk + block * (NH * 128) + step, 16), i_scores, c > 0 || k > 0);
-                    }
-                    if (c < MB - OWN) lu_commit(&empty[st]);
-                }
-                if (c1 == MB) lu_commit(&s_full[t & 1]);
-            };
-            if (!lu_bar_wait(q_full, 0)) {
-                atomicExch(a.status, 26);
-                ok = false;
-            }
-            lu_fence_after();
-            if (ok) scores(0, 0, MB);
-            for (int t = 0; t < tiles && ok; ++t) {
-                if (t + 1 < tiles) scores(t + 1, 0, L::AHEAD);
-                if (!ok) break;
-                if (!lu_bar_wait(p_full, t & 1)) {
-                    atomicExch(a.status, 23);
-                    break;
-                }
+            auto scores = [&](int t, int c) {  // chunk c of tile t's scores; the chunk is there
+                const uint32_t st = (uint32_t)(t * MB + c) % STAGES;
+                asm volatile("fence.proxy.async.shared::cta;" ::: "memory");  // the copies are ordinary writes
                 lu_fence_after();
-                for (int c = 0; c < OWN; ++c) {
-                    const uint32_t st = (uint32_t)(t * MB + MB - OWN + c) % STAGES;
+                const uint32_t q_chunk = q_addr + 2 * c * (NH * 128);
+#pragma unroll
+                for (int k = 0; k < LU_COLS / 16; ++k) {
+                    const uint32_t block = (uint32_t)k >> 2, step = ((uint32_t)k & 3) * 32;
+                    lu_mma(tmem + L::S_COL + (t & 1) * NH, lu_desc(ring_addr + st * LU_CHUNK + block * LU_BLOCK + step, 16),
+                           lu_desc(q_chunk + block * (NH * 128) + step, 16), i_scores, c > 0 || k > 0);
+                }
+                if (c == MB - 1) lu_commit(&s_full[t & 1]);
+            };
+            auto outputs = [&](int t) {  // tile t's part of the outputs; the weights are there
+                lu_fence_after();
+                for (int c = 0; c < MB; ++c) {
+                    const uint32_t st = (uint32_t)(t * MB + c) % STAGES;
 #pragma unroll
                     for (int k = 0; k < LU_KEYS / 16; ++k)
                         lu_mma(tmem + c * 2 * NH, lu_desc(ring_addr + st * LU_CHUNK + k * 2048, LU_BLOCK),
@@ -295,8 +281,35 @@ __global__ void __launch_bounds__(LU_THREADS, 1) latent_umma_kernel(const __grid
                     lu_commit(&empty[st]);
                 }
                 lu_commit(o_done);
-                if (L::AHEAD < MB && t + 1 < tiles) scores(t + 1, L::AHEAD, MB);
+            };
+            auto full_of = [&](int t, int c) { return &full[(uint32_t)(t * MB + c) % STAGES]; };
+            auto full_parity = [&](int t, int c) { return ((uint32_t)(t * MB + c) / STAGES) & 1; };
+            ok = lu_bar_wait(q_full, 0);
+            lu_fence_after();
+            for (int c = 0; c < MB && ok; ++c) {
+                ok = lu_bar_wait(full_of(0, c), full_parity(0, c));
+                if (ok) scores(0, c);
             }
+            // From here on whatever is ready first: the weights of tile t, or the next chunk of tile t + 1.  Chunks that find no room
+            // beside tile t come only after its outputs.
+            for (int t = 0; t < tiles && ok; ++t) {
+                bool summed = false;
+                int c = t + 1 < tiles ? 0 : MB;
+                for (uint32_t spins = 0; ok && (!summed || c < MB);) {
+                    if (!summed && lu_bar_test(p_full, t & 1)) {
+                        outputs(t);
+                        summed = true;
+                        spins = 0;
+                    }
+                    if (c < MB && lu_bar_test(full_of(t + 1, c), full_parity(t + 1, c))) {
+                        scores(t + 1, c);
+                        ++c;
+                        spins = 0;
+                    }
+                    ok = ++spins < LU_SPIN_LIMIT;
+                }
+            }
+            if (!ok) atomicExch(a.status, 22);
         }
     } else {
         // ---- softmax: a group of 128 threads takes HG heads; thread = key of the tile, later column of a chunk
@@ -375,7 +388,7 @@ __global__ void __launch_bounds__(LU_THREADS, 1) latent_umma_kernel(const __grid
                 lu_fence_after();
                 if (moved) {
 #pragma unroll 1
-                    for (int c = 0; c < OWN * 2; ++c) {
+                    for (int c = 0; c < MB * 2; ++c) {
                         lu_tmem_load<HG>(my_tmem + c * NH, raw);
                         lu_tmem_wait();
 #pragma unroll
@@ -405,7 +418,7 @@ __global__ void __launch_bounds__(LU_THREADS, 1) latent_umma_kernel(const __grid
         if (lane < HG) s_warp[warp][lane] = sum;
         if (!lu_agree(bar, 128, ok) && gt == 0) atomicExch(a.status, 25);
         auto slot = [&](int entry) { return ((int64_t)entry * gridDim.y + blockIdx.y) * NH; };
-        auto ml_at = [&](int entry, int h) { return a.part_ml + (slot(entry) * CS + part * NH + h) * 2; };
+        auto ml_at = [&](int entry, int h) { return a.part_ml + (slot(entry) + h) * 2; };
         if (gt < HG && h0 + gt < heads) {  // thread gt finishes head h0 + gt
             float total = 0.f, mine = -INFINITY;
 #pragma unroll
@@ -418,7 +431,7 @@ __global__ void __launch_bounds__(LU_THREADS, 1) latent_umma_kernel(const __grid
         }
         lu_agree(bar, 128, true);
 #pragma unroll
-        for (int c = 0; c < OWN; ++c) {
+        for (int c = 0; c < MB; ++c) {
             uint32_t o[HG], rest[HG];
             if (tiles > 0) {
                 lu_tmem_load<HG>(my_tmem + c * 2 * NH, o);
@@ -430,16 +443,16 @@ __global__ void __launch_bounds__(LU_THREADS, 1) latent_umma_kernel(const __grid
                 if (h0 + h >= heads) continue;
                 const float v = tiles > 0 ? __uint_as_float(o[h]) + __uint_as_float(rest[h]) : 0.f;
                 if (e.n_shares == 1)
-                    a.out.h[((int64_t)(head0 + h0 + h) * a.n_rows + e.row) * RANK + col0 + c * LU_COLS + gt] = __float2bfloat16_rn(v * s_factor[0][h0 + h]);
+                    a.out.h[((int64_t)(head0 + h0 + h) * a.n_rows + e.row) * RANK + c * LU_COLS + gt] = __float2bfloat16_rn(v * s_factor[0][h0 + h]);
                 else
-                    a.part_o[(slot(blockIdx.x) + h0 + h) * RANK + col0 + c * LU_COLS + gt] = v;
+                    a.part_o[(slot(blockIdx.x) + h0 + h) * RANK + c * LU_COLS + gt] = v;
             }
         }
         if (e.n_shares > 1) {
             __threadfence();
             lu_agree(LU_GROUPS + 1, LU_SOFTMAX, true);
             if (tid == 0) {
-                int32_t* counter = a.counters + ((int64_t)e.first * gridDim.y + blockIdx.y) * CS + part;
+                int32_t* counter = a.counters + (int64_t)e.first * gridDim.y + blockIdx.y;
                 s_last = atomicAdd(counter, 1) == e.n_shares - 1 ? 1 : 0;
                 if (s_last) *counter = 0;
             }
@@ -460,8 +473,8 @@ __global__ void __launch_bounds__(LU_THREADS, 1) latent_umma_kernel(const __grid
                 }
                 lu_agree(LU_GROUPS + 1, LU_SOFTMAX, true);
 #pragma unroll 4
-                for (int i = tid; i < heads * (OWN * LU_COLS / 4); i += LU_SOFTMAX) {
-                    const int h = i / (OWN * LU_COLS / 4), c = col0 + (i - h * (OWN * LU_COLS / 4)) * 4;
+                for (int i = tid; i < heads * (MB * LU_COLS / 4); i += LU_SOFTMAX) {
+                    const int h = i / (MB * LU_COLS / 4), c = (i - h * (MB * LU_COLS / 4)) * 4;
                     float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
                     for (int sh = 0; sh < e.n_shares; ++sh) {
                         const float4 v = __ldcg(reinterpret_cast<const float4*>(a.part_o + (slot(e.first + sh) + h) * RANK + c));
@@ -620,8 +633,7 @@ void launch_umma(const LatentAttnArgs& a, cudaStream_t s) {
     int shift = 0;
     while ((1 << shift) < a.block_tokens) ++shift;
     ensure_dynamic_smem(reinterpret_cast<const void*>(&latent_umma_kernel<MB, NH>), smem);
-    launch_pdl(latent_umma_kernel<MB, NH>, dim3((unsigned)a.n_entries, (unsigned)latent_tc_groups(a.heads), (unsigned)Lu<MB, NH>::CS), dim3(LU_THREADS), smem, s,
-               *static_cast<const CUtensorMap*>(a.pool_map), a, shift, std::min(a.block_tokens, LU_KEYS), (int)a.pool_rows);
+    launch_pdl(latent_umma_kernel<MB, NH>, dim3((unsigned)a.n_entries, (unsigned)latent_tc_groups(a.heads)), dim3(LU_THREADS), smem, s, a, shift);
 }
 
 template <int MB>
@@ -633,17 +645,10 @@ void launch_umma_heads(const LatentAttnArgs& a, cudaStream_t s) {
 }  // namespace
 
 int latent_tc_rank(int kv_rank, int block_tokens) {
-    if (block_tokens < 8 || (block_tokens & (block_tokens - 1)) != 0) return 0;
+    if (block_tokens <= 0 || (block_tokens & (block_tokens - 1)) != 0) return 0;
     const int r = (kv_rank + LU_COLS - 1) / LU_COLS * LU_COLS;
     return r <= 4 * LU_COLS ? r : 0;
 }
-
-void latent_pool_map(void* out, const void* pool, int64_t rows, int rank, int block_tokens) {
-    if (rows > (int64_t)1 << 30) throw std::runtime_error("latent_pool_map: the pool has too many rows");
-    encode_tma_2d(out, false, pool, (uint64_t)rank, (uint64_t)rows, (uint64_t)rank * 2, 64, (uint32_t)std::min(block_tokens, LU_KEYS), true);
-}
-
-int latent_tc_ctas(int heads, int rank) { return latent_tc_groups(heads) * (rank == 4 * LU_COLS ? 2 : 1); }
 
 int latent_tc_heads(int heads) { return heads <= 16 ? 16 : 32; }
 
@@ -695,7 +700,7 @@ void launch_latent_attention(const LatentAttnArgs& a, cudaStream_t s) {
     if (a.out.ld != a.rank) throw std::runtime_error("launch_latent_attention: the output's rows are as wide as the latent");
     if (a.q_h != nullptr) {
         if (!a.pool_f16 || a.out.h == nullptr) throw std::runtime_error("launch_latent_attention: f16 queries go with f16 pages and a bf16 output");
-        if (a.pool_map == nullptr || a.status == nullptr) throw std::runtime_error("launch_latent_attention: the tensor-core kernel needs the pool's map and a status word");
+        if (a.status == nullptr) throw std::runtime_error("launch_latent_attention: the tensor-core kernel needs a status word");
         switch (a.rank) {
             case 128: launch_umma_heads<1>(a, s); break;
             case 256: launch_umma_heads<2>(a, s); break;

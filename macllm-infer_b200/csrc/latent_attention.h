@@ -14,8 +14,6 @@ struct LatentAttnArgs {
     const float* q_f = nullptr;      // the same in f32 (general kernel)
     const void* pool = nullptr;      // [blocks * block_tokens][rank]
     int pool_f16 = 1;
-    const void* pool_map = nullptr;  // host: latent_pool_map of the pool (tensor-core kernel)
-    int64_t pool_rows = 0;
     const uint32_t* tables = nullptr;
     // work list, 8 ints each, 32-byte aligned: (query row, share, n_shares, last visible position, table offset, packed row,
     // first entry of the query row, 0)
@@ -27,7 +25,7 @@ struct LatentAttnArgs {
     Shares gate;                     // a head's output is multiplied by sigmoid(gate[packed row][gate_col + head])
     int gate_col = 0;
     RowImage out;                    // row head * n_rows + query row, ld = rank
-    // shares (tensor-core kernel): unnormalised partial outputs [entry][heads padded][rank], two (max, sum) pairs per head, and
+    // shares (tensor-core kernel): unnormalised partial outputs [entry][heads padded][rank], (max, sum) pairs, and
     // counters [entries][CTAs per entry] that are zero before the first call and after every call
     float* part_o = nullptr;
     float* part_ml = nullptr;
@@ -38,12 +36,9 @@ struct LatentAttnArgs {
 // The tensor-core kernel's rank for a latent of `kv_rank` values (a multiple of 128 up to 512), or 0 when it does not cover the
 // case.
 int latent_tc_rank(int kv_rank, int block_tokens);
-// The descriptor (128 bytes, 64-byte aligned) through which that kernel loads an f16 pool of `rows` rows.
-void latent_pool_map(void* out, const void* pool, int64_t rows, int rank, int block_tokens);
-// Heads of one CTA of the tensor-core kernel, groups of that many, and CTAs per work item (a wide latent is shared by two).
+// Heads of one CTA of the tensor-core kernel, and CTAs per work item.
 int latent_tc_heads(int heads);
 inline int latent_tc_groups(int heads) { return (heads + latent_tc_heads(heads) - 1) / latent_tc_heads(heads); }
-int latent_tc_ctas(int heads, int rank);
 constexpr int kLatentMaxRank = 1024;  // of the general kernel
 
 // Host-side work list: one entry per token of lane i with n_tokens[i] < wide_from, cut into key shares while that fills the GPU.

@@ -316,11 +316,7 @@ void MixerLm::alloc_run(int run) {
             st.state.alloc(halves * (size_t)d.heads * d.vdim * linear_state_key_pad(d.dim) * 4);
             break;
         }
-        case MixerKind::Latent:
-            pages(st.k_pool, 1);
-            if (latent_geo_[(size_t)w.geometry].tc)
-                latent_pool_map(st.pool_map, st.k_pool.ptr(), pool_->max_blocks() * cfg_.block_tokens, w.row_width, cfg_.block_tokens);
-            break;
+        case MixerKind::Latent: pages(st.k_pool, 1); break;
         case MixerKind::MinGru: st.state.alloc(halves * (size_t)s.gru.width * 4); break;
     }
 }

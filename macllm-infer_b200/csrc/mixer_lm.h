@@ -86,7 +86,6 @@ private:
     struct RunState {
         DevBuf k_pool, v_pool;  // latent attention: k_pool only
         DevBuf state, kept, tail;
-        alignas(64) unsigned char pool_map[128] = {};  // latent attention on the tensor cores (see latent_pool_map)
     };
     // Layers with the same heads share a tick's attention work list.
     struct Geometry {

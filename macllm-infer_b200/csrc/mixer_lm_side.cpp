@@ -106,7 +106,7 @@ void MixerLm::load_latent(const SafetensorsFile& f, int l) {
                 wide = true;
                 w.q_width = d;
             }
-    w.geometry = latent_geometry(tc_rank > 0 ? latent_tc_ctas(H, w.row_width) : 1, tc_rank > 0, wide);
+    w.geometry = latent_geometry(tc_rank > 0 ? latent_tc_groups(H) : 1, tc_rank > 0, wide);
     if (wide && iota_.size() == 0) {
         std::vector<uint32_t> n((size_t)(pool_->max_blocks() + cfg_.max_batch_lanes));
         for (size_t i = 0; i < n.size(); ++i) n[i] = (uint32_t)i;
@@ -321,8 +321,6 @@ void MixerLm::run_latent(const Tick& t, int run, const Shares& y, const RowImage
         else a.q_f = q_lat_.as<float>();
         a.pool = rs_[(size_t)run].k_pool.ptr();
         a.pool_f16 = cfg_.kv_f16 ? 1 : 0;
-        a.pool_map = rs_[(size_t)run].pool_map;
-        a.pool_rows = pool_->max_blocks() * cfg_.block_tokens;
         a.status = status_.as<int32_t>();
         a.tables = t.bd.tables;
         a.entries = reinterpret_cast<const int32_t*>(t.dp + g.off_entries);
