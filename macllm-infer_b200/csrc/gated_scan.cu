@@ -1,8 +1,8 @@
 // See gated_scan.h.
 //
-// A row is an affine map S -> a S + b of every channel, so rows compose: prompts run in tiles of 256 rows, 16 channels per CTA.
-// A thread folds eight consecutive rows of one channel, one warp per channel then scans the 32 folded maps with shuffles, and the
-// threads walk their eight rows again from the state they now know.  The next tile's projections are on their way meanwhile.
+// A row is an affine map S -> a S + b of every channel, so rows compose: prompts run in tiles of 128 rows, 16 channels per CTA.
+// A thread folds four consecutive rows of one channel, one warp per channel then scans the 32 folded maps with shuffles, and the
+// threads walk their four rows again from the state they now know.  The next tile's projections are on their way meanwhile.
 // a = 1 - z lies in (0, 1) and b is what the gate lets in, so composing loses nothing but rounding.  Short lanes take a thread per
 // channel that walks the rows.
 #include "gated_scan.h"
@@ -14,7 +14,7 @@ namespace {
 
 constexpr int GS_CH = 16;       // channels of a CTA
 constexpr int GS_SLICES = 32;   // row slices of a tile, one per lane of the scanning warp
-constexpr int GS_ROWS = 8;      // rows of a slice
+constexpr int GS_ROWS = 4;      // rows of a slice
 constexpr int GS_TILE = GS_SLICES * GS_ROWS;
 constexpr int GS_THREADS = GS_CH * GS_SLICES;
 constexpr int GS_SHORT = 8;     // lanes up to this many rows are walked row by row
