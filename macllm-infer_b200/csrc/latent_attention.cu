@@ -210,12 +210,18 @@ __global__ void __launch_bounds__(LU_THREADS, 1) latent_umma_kernel(LatentAttnAr
     lu_fence_after();
     const uint32_t tmem = tmem_slot;
     pdl_trigger();
-    pdl_wait();
+    // work list and block tables were staged by the host: they need not wait for the predecessor
     const LatentEntry e = load_entry(a.entries, blockIdx.x);
     const int len = e.pos + 1;
     const int chunk = ((len + e.n_shares - 1) / e.n_shares + LU_KEYS - 1) / LU_KEYS * LU_KEYS;
     const int k_lo = e.share * chunk, k_hi = min(len, k_lo + chunk);
     const int tiles = k_hi > k_lo ? (k_hi - k_lo + LU_KEYS - 1) / LU_KEYS : 0;
+    auto row_of = [&](int t, int key) {  // pool row of a tile's key, -1 past the last one
+        const int pos = k_lo + t * LU_KEYS + key;
+        return pos < k_hi ? (int)(a.tables[e.table_off + (pos >> bt_shift)] << bt_shift) + (pos & ((1 << bt_shift) - 1)) : -1;
+    };
+    if (warp >= LOADER && warp < LOADER + LU_LOADERS / 32 && tiles > 0) s_rows[0][tid - LU_SOFTMAX] = row_of(0, tid - LU_SOFTMAX);
+    pdl_wait();
 
     if (warp >= LOADER && warp < LOADER + LU_LOADERS / 32) {
         // ---- loaders: pool rows of a tile's keys first (one per thread), then 16-byte pieces of the rows
@@ -223,17 +229,12 @@ __global__ void __launch_bounds__(LU_THREADS, 1) latent_umma_kernel(LatentAttnAr
         const int lt = tid - LU_SOFTMAX, piece = lt & 15, key0 = lt >> 4;
         const __half* pool = static_cast<const __half*>(a.pool) + piece * 8;
         const uint32_t dst0 = lu_smem(ring) + (piece >> 3) * LU_BLOCK;
-        auto row_of = [&](int t) {
-            const int pos = k_lo + t * LU_KEYS + lt;
-            return pos < k_hi ? (int)(a.tables[e.table_off + (pos >> bt_shift)] << bt_shift) + (pos & ((1 << bt_shift) - 1)) : -1;
-        };
         uint32_t it = 0;
         bool ok = true;
-        if (tiles > 0) s_rows[0][lt] = row_of(0);
         for (int t = 0; t < tiles; ++t) {
             ok = lu_agree(LU_GROUPS + 2, LU_LOADERS, ok);  // this tile's rows are there, nobody reads the other buffer any more
             if (!ok) break;
-            if (t + 1 < tiles) s_rows[(t + 1) & 1][lt] = row_of(t + 1);
+            if (t + 1 < tiles) s_rows[(t + 1) & 1][lt] = row_of(t + 1, lt);
             for (int c = 0; c < MB; ++c, ++it) {
                 const uint32_t st = it % STAGES;
                 ok = lu_bar_wait(&empty[st], ((it / STAGES) & 1) ^ 1);
@@ -261,23 +262,23 @@ __global__ void __launch_bounds__(LU_THREADS, 1) latent_umma_kernel(LatentAttnAr
                 const uint32_t st = (uint32_t)(t * MB + c) % STAGES;
                 asm volatile("fence.proxy.async.shared::cta;" ::: "memory");  // the copies are ordinary writes
                 lu_fence_after();
-                const uint32_t q_chunk = q_addr + 2 * c * (NH * 128);
+                // descriptors hold addresses in 16-byte units
+                const uint64_t keys = lu_desc(ring_addr + st * LU_CHUNK, 16), queries = lu_desc(q_addr + 2 * c * (NH * 128), 16);
+                const uint32_t d = tmem + L::S_COL + (t & 1) * NH;
 #pragma unroll
-                for (int k = 0; k < LU_COLS / 16; ++k) {
-                    const uint32_t block = (uint32_t)k >> 2, step = ((uint32_t)k & 3) * 32;
-                    lu_mma(tmem + L::S_COL + (t & 1) * NH, lu_desc(ring_addr + st * LU_CHUNK + block * LU_BLOCK + step, 16),
-                           lu_desc(q_chunk + block * (NH * 128) + step, 16), i_scores, c > 0 || k > 0);
-                }
+                for (int k = 0; k < LU_COLS / 16; ++k)
+                    lu_mma(d, keys + (k >> 2) * (LU_BLOCK / 16) + (k & 3) * 2, queries + (k >> 2) * (NH * 8) + (k & 3) * 2, i_scores, c > 0 || k > 0);
                 if (c == MB - 1) lu_commit(&s_full[t & 1]);
             };
             auto outputs = [&](int t) {  // tile t's part of the outputs; the weights are there
                 lu_fence_after();
+                const uint64_t weights = lu_desc(p_addr, 16);
                 for (int c = 0; c < MB; ++c) {
                     const uint32_t st = (uint32_t)(t * MB + c) % STAGES;
+                    const uint64_t values = lu_desc(ring_addr + st * LU_CHUNK, LU_BLOCK);
 #pragma unroll
                     for (int k = 0; k < LU_KEYS / 16; ++k)
-                        lu_mma(tmem + c * 2 * NH, lu_desc(ring_addr + st * LU_CHUNK + k * 2048, LU_BLOCK),
-                               lu_desc(p_addr + (uint32_t)(k >> 2) * (2 * NH * 128) + ((uint32_t)k & 3) * 32, 16), i_out, t > 0 || k > 0);
+                        lu_mma(tmem + c * 2 * NH, values + k * 128, weights + (k >> 2) * (2 * NH * 8) + (k & 3) * 2, i_out, t > 0 || k > 0);
                     lu_commit(&empty[st]);
                 }
                 lu_commit(o_done);
