@@ -172,11 +172,16 @@ typedef struct mk_mixer_summary {
     int32_t wkv_layers, parallel_layers, ffn_layers, side_dim;
     int32_t latent_layers, mingru_layers;
     int32_t layer_runs; /* executions of a layer per forward: a looped layer counts once per pass */
+    int32_t mlstm_layers, attention_layers, experts; /* experts: of the layer that has most, 0 = no mixture */
     int64_t tensors_in_file, tensors_read, parameters;
 } mk_mixer_summary;
 int32_t mk_mixer_inspect(const char* dir, mk_mixer_summary* out);
 /* Rotary frequencies [dims / 2] (radians per position); `scaling` = {factor, low, high, original} or NULL. */
 int32_t mk_rotary_frequencies(int32_t dims, double base, const double* scaling, double* out);
+/* The same stretched between the pairs that turn `fast` and `slow` times over the original context; *amplitude = the factor of
+ * cosine and sine. */
+int32_t mk_rotary_frequencies_yarn(int32_t dims, double base, double factor, double original, double fast, double slow, double* out,
+                                   double* amplitude);
 
 /* LoadedRuntime::load (src/runtime.rs:104-145): loads a checkpoint with the registered format that recognises it - a GGUF file
  * (first shard of a family), or a folder with config.json and model.safetensors whose config names a registered

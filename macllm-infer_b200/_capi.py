@@ -49,7 +49,8 @@ class GgufSummary(C.Structure):
 class MixerSummary(C.Structure):
     _fields_ = [("architecture", C.c_char * 32), ("vocab_size", C.c_int32), ("hidden_size", C.c_int32), ("n_layers", C.c_int32),
                 ("wkv_layers", C.c_int32), ("parallel_layers", C.c_int32), ("ffn_layers", C.c_int32), ("side_dim", C.c_int32),
-                ("latent_layers", C.c_int32), ("mingru_layers", C.c_int32), ("layer_runs", C.c_int32), ("tensors_in_file", C.c_int64), ("tensors_read", C.c_int64), ("parameters", C.c_int64)]
+                ("latent_layers", C.c_int32), ("mingru_layers", C.c_int32), ("layer_runs", C.c_int32),
+                ("mlstm_layers", C.c_int32), ("attention_layers", C.c_int32), ("experts", C.c_int32), ("tensors_in_file", C.c_int64), ("tensors_read", C.c_int64), ("parameters", C.c_int64)]
 
 
 class RuntimeSpec(C.Structure):
@@ -264,6 +265,7 @@ SIGNATURES = {
     "mk_model_read_residuals": (_i32, [P, P, _i64, C.POINTER(_i32)]),
     "mk_mixer_inspect": (_i32, [C.c_char_p, C.POINTER(MixerSummary)]),
     "mk_rotary_frequencies": (_i32, [_i32, C.c_double, P, P]),
+    "mk_rotary_frequencies_yarn": (_i32, [_i32, C.c_double, C.c_double, C.c_double, C.c_double, C.c_double, P, P]),
     "mk_state_slots_query": (_i32, [P, C.POINTER(_i32), C.POINTER(_i32)]),
     "mk_k_moe_route": (_i32, [P, _i32, _i32, _i32, P, P]),
 }

@@ -5,7 +5,7 @@
 // 614-709 is its scalar CPU form; metal/paged_decode.metal:189-489 the Metal forms) and the dense
 // fallback the CPU/CUDA backends take (dense_causal_attention, src/decoder.rs:4580-4670, with the
 // visibility rule of src/decoder.rs:4515-4532: key j is visible to the query at absolute position p
-// iff j <= p and, on sliding layers, p - j < window).  One query tile of one lane and one KV head
+// iff j <= p and, on sliding layers, p - j < window; on chunked layers iff j and p lie in the same chunk).  One query tile of one lane and one KV head
 // per CTA, so the K/V pages of that head are loaded once for the whole query group (all q heads that
 // map to the KV head, query head h reads KV head h / groups).  Scores, softmax and the weighted sum
 // are f32; the softmax is the online (running max / running sum) form.
@@ -58,9 +58,7 @@ __global__ void __launch_bounds__(AT_WARPS * 32) attn_tile_kernel(AttnArgs a) {
 
     const int p_first = hdr.start_pos + row0;
     const int p_last = p_first + n_rows - 1;
-    int k_begin = 0;
-    if (a.window > 0) k_begin = max(0, p_first - a.window + 1);
-    k_begin = (k_begin / AT_KEYS) * AT_KEYS;
+    const int k_begin = attention_first_key(p_first, a.window, a.chunk) / AT_KEYS * AT_KEYS;
     const int k_end = p_last + 1;
 
     float m_run[AT_IPW], l_run[AT_IPW], acc[AT_IPW][AT_DPL];
@@ -103,7 +101,7 @@ __global__ void __launch_bounds__(AT_WARPS * 32) attn_tile_kernel(AttnArgs a) {
             int r = item / g;
             int p = p_first + r;
             int key = kt + lane;
-            bool visible = key <= p && (a.window == 0 || p - key < a.window);
+            bool visible = key <= p && key >= attention_first_key(p, a.window, a.chunk);
             float s = -INFINITY;
             if (visible) {
                 const float4* qv = reinterpret_cast<const float4*>(Qs + item * d);
@@ -149,6 +147,10 @@ __global__ void __launch_bounds__(AT_WARPS * 32) attn_tile_kernel(AttnArgs a) {
         int r = item / g, hq = item - r * g;
         float* o = a.out + (int64_t)(q_off + row0 + r) * ldo + (kvh * g + hq) * d;
         float inv = 1.0f / l_run[ii];
+        if (a.sink != nullptr) {
+            const float z = a.sink[kvh * g + hq], m = fmaxf(m_run[ii], z), f = expf(m_run[ii] - m);
+            inv = f / (l_run[ii] * f + expf(z - m));
+        }
 #pragma unroll
         for (int j = 0; j < AT_DPL; ++j) {
             int c = lane + 32 * j;

@@ -56,6 +56,12 @@ __device__ __forceinline__ uint32_t pack_half2_rest(float x, float y, uint32_t r
     return pack_half2(x - r.x, y - r.y);
 }
 
+// 1 / denominator of a row with running maximum m and sum l of exp(score - m), when the softmax also counts exp(sink).
+__device__ __forceinline__ float sink_scale(float m, float l, float sink) {
+    const float top = fmaxf(m, sink), f = __expf(m - top);
+    return f / (l * f + __expf(sink - top));
+}
+
 // One CTA.  D = head_dim, WARPS warps of 16 items each, KT keys per shared-memory tile.
 // SPLIT = false: work item = tiles[blockIdx.x] = (lane, first query row); the CTA walks every visible key
 //                and writes normalised outputs.
@@ -119,7 +125,7 @@ __global__ void __launch_bounds__(WARPS * 32) attn_tc_kernel(AttnTcArgs a) {
 
     // key range of this CTA
     const int p_first = hdr.start_pos + row0, p_last = p_first + n_rows - 1;
-    int k_lo = a.window > 0 ? max(0, p_first - a.window + 1) : 0;
+    int k_lo = attention_first_key(p_first, a.window, a.chunk);
     int k_hi = p_last + 1;
     if (SPLIT) {
         int len = k_hi - k_lo;
@@ -157,13 +163,14 @@ __global__ void __launch_bounds__(WARPS * 32) attn_tc_kernel(AttnTcArgs a) {
 
     // the two accumulator rows of this thread: items warp*16 + gid and + 8
     int item_r[2] = {warp * 16 + gid, warp * 16 + gid + 8};
-    int pos_r[2];
+    int pos_r[2], lo_r[2];  // position and first visible key of the two rows
     bool live_r[2];
 #pragma unroll
     for (int h = 0; h < 2; ++h) {
         int hq = item_r[h] / rows_per_head, r = item_r[h] - hq * rows_per_head;
         live_r[h] = hq < g && r < n_rows;
         pos_r[h] = p_first + r;
+        lo_r[h] = attention_first_key(pos_r[h], a.window, a.chunk);
     }
 
     if (n_tiles > 0) load_tile(0, 0);
@@ -203,7 +210,7 @@ __global__ void __launch_bounds__(WARPS * 32) attn_tc_kernel(AttnTcArgs a) {
                 int pos = tile_pos + j * 8 + 2 * tq + (e & 1);
                 float v = s[j][e] * a.scale;
                 if (a.softcap != 0.f) v = tanhf(v / a.softcap) * a.softcap;
-                bool vis = live_r[h] && pos >= k_lo && pos < k_hi && pos <= pos_r[h] && (a.window == 0 || pos_r[h] - pos < a.window);
+                bool vis = live_r[h] && pos >= k_lo && pos < k_hi && pos <= pos_r[h] && pos >= lo_r[h];
                 v = vis ? v : -INFINITY;
                 s[j][e] = v;
                 tmax[h] = fmaxf(tmax[h], v);
@@ -274,6 +281,7 @@ __global__ void __launch_bounds__(WARPS * 32) attn_tc_kernel(AttnTcArgs a) {
             if (!live_r[h]) continue;
             int hq = item_r[h] / rows_per_head, r = item_r[h] - hq * rows_per_head;
             float inv = 1.0f / l_run[h];
+            if (a.sink != nullptr) inv = sink_scale(m_run[h], l_run[h], a.sink[kvh * g + hq]);
             const int64_t at = (int64_t)(q_off + row0 + r) * ldo + (kvh * g + hq) * D;
             if (a.out != nullptr) {
 #pragma unroll
@@ -384,7 +392,7 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(AttnTcArgs a) {
     }
 
     const int p = start_pos;  // the query's position
-    int k_lo = a.window > 0 ? max(0, p - a.window + 1) : 0;
+    int k_lo = attention_first_key(p, a.window, a.chunk);
     int k_hi = p + 1;
     {
         int len = k_hi - k_lo;
@@ -613,7 +621,7 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(AttnTcArgs a) {
         finish([&](int idx) {
             float m, l;
             float o = merged_local(idx, m, l);
-            return o / l;
+            return a.sink != nullptr ? o * sink_scale(m, l, a.sink[kvh * g + idx / D]) : o / l;
         });
     } else {
         for (int idx = tid; idx < g * D; idx += 128) {
@@ -654,7 +662,7 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(AttnTcArgs a) {
                         o += __ldcg(a.part_o + ps * D + c) * f;
                     }
                 }
-                return o / l;
+                return a.sink != nullptr ? o * sink_scale(m, l, a.sink[kvh * g + item]) : o / l;
             });
         }
     }
@@ -739,7 +747,8 @@ int attention_tc_tile_rows(int q_heads, int kv_heads) { return 16 * attention_tc
 int attention_tc_max_entries(int lanes, int kv_heads) { return std::max(lanes + lanes / 2, kAttnTargetCtas / std::max(1, kv_heads)) + 1; }
 
 void plan_attention_tc(const int32_t* start_pos, const int32_t* n_tokens, const int32_t* n_blocks, int lanes, int q_heads,
-                       int kv_heads, AttnTcPlan& plan) {
+                       int kv_heads, AttnTcPlan& plan, int chunk) {
+    auto visible = [&](int i) { return start_pos[i] + 1 - attention_first_key(start_pos[i], 0, chunk); };  // keys of a one-token lane
     plan.tiles.clear();
     plan.entries.clear();
     plan.dec_lanes.clear();
@@ -749,7 +758,7 @@ void plan_attention_tc(const int32_t* start_pos, const int32_t* n_tokens, const 
     int n_dec = 0;
     int64_t total_keys = 0;
     for (int i = 0; i < lanes; ++i)
-        if (n_tokens[i] == 1) { ++n_dec; total_keys += start_pos[i] + 1; }
+        if (n_tokens[i] == 1) { ++n_dec; total_keys += visible(i); }
     // Once the lanes alone give every SM a CTA, sharing keys out only adds merge work and repeated query preparation
     // (measured at 64 lanes x 4 KV heads with histories within twice their mean: +1.4 % on the whole benchmark
     // without shares).  Then only a lane more than twice as long as the mean is cut, so that one long history among
@@ -762,14 +771,14 @@ void plan_attention_tc(const int32_t* start_pos, const int32_t* n_tokens, const 
     for (;;) {
         int64_t ctas = 0;
         for (int i = 0; i < lanes; ++i)
-            if (n_tokens[i] == 1) ctas += shares_of(start_pos[i] + 1);
+            if (n_tokens[i] == 1) ctas += shares_of(visible(i));
         if (ctas <= slots || share > (1 << 20)) break;
         share += 64;
     }
     int q_off = 0, table_off = 0;
     for (int i = 0; i < lanes; q_off += n_tokens[i], table_off += n_blocks[i], ++i) {
         if (n_tokens[i] == 1) {
-            const int splits = shares_of(start_pos[i] + 1);
+            const int splits = shares_of(visible(i));
             const int first = plan.n_entries();
             for (int sidx = 0; sidx < splits; ++sidx) {
                 const int32_t rec[8] = {i, sidx, splits, start_pos[i], table_off, q_off, first, 0};
@@ -789,6 +798,7 @@ int launch_paged_attention_tc(const AttnTcArgs& a_in, cudaStream_t s) {
     if (!attention_tc_supported(a.q_heads, a.kv_heads, a.d, a.block_tokens, true))
         throw std::runtime_error("launch_paged_attention_tc: unsupported shape");
     if (a.out == nullptr && a.out_h == nullptr && a.qout.qs == nullptr) throw std::runtime_error("launch_paged_attention_tc: no output");
+    if (a.sink != nullptr && a.n_dec_lanes > 0) throw std::runtime_error("launch_paged_attention_tc: the separate merge pass knows no sink");
     if (a.out == nullptr && a.n_dec_lanes > 0) throw std::runtime_error("launch_paged_attention_tc: the separate merge pass writes f32 rows");
     a.bt_shift = 0;
     while ((1 << a.bt_shift) < a.block_tokens) ++a.bt_shift;

@@ -41,6 +41,8 @@ struct AttnTcArgs {
     int bt_shift = 0;         // log2(block_tokens), filled in by the launcher
     float scale = 1.f, softcap = 0.f;
     int window = 0;
+    int chunk = 0;              // > 0: a position sees the keys of its own chunk only (chunks counted from position 0)
+    const float* sink = nullptr;  // [q_heads]: one more term exp(sink) in the denominator; null: none
     // attention weights enter the product with V as the sum of two f16 numbers (about 22 bits) instead of one
     int exact_weights = 0;
 };
@@ -66,8 +68,9 @@ struct AttnTcPlan {
     int n_dec_lanes() const { return (int)dec_lanes.size() / 3; }
 };
 // n_blocks[i] = entries of lane i's block table (tables are concatenated in lane order, tokens packed in lane order).
+// chunk: see AttnTcArgs.
 void plan_attention_tc(const int32_t* start_pos, const int32_t* n_tokens, const int32_t* n_blocks, int lanes, int q_heads,
-                       int kv_heads, AttnTcPlan& plan);
+                       int kv_heads, AttnTcPlan& plan, int chunk = 0);
 // Upper bound of plan.n_entries() for a tick of at most `lanes` lanes.
 int attention_tc_max_entries(int lanes, int kv_heads);
 

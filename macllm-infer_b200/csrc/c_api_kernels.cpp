@@ -287,7 +287,7 @@ int32_t mk_k_gated_ffn(int32_t type, const void* gate_w, const void* up_w, int64
         status.zero(nullptr);
         HgemmScratch hs;
         hs.status = status.as<int32_t>();
-        auto run = [&] { launch_hgemm_tc_gated(image, a.xh, T, act, dy.as<__half>(), (int)F, hs, nullptr); };
+        auto run = [&] { launch_hgemm_tc_gated(image, a.xh, T, GatedAct{act == 0 ? GatedAct::Silu : GatedAct::GeluTanh}, dy.as<__half>(), (int)F, hs, nullptr); };
         run();
         if (iters > 0 && avg_ms != nullptr) {
             DevBuf flush((size_t)256 << 20);  // larger than the L2

@@ -113,8 +113,11 @@ int32_t mk_mixer_inspect(const char* dir, mk_mixer_summary* out) {
                 case MixerKind::Parallel: ++out->parallel_layers; break;
                 case MixerKind::Latent: ++out->latent_layers; break;
                 case MixerKind::MinGru: ++out->mingru_layers; break;
+                case MixerKind::Mlstm: ++out->mlstm_layers; break;
+                case MixerKind::Attention: ++out->attention_layers; break;
             }
             out->ffn_layers += l.ff > 0 ? 1 : 0;
+            out->experts = std::max(out->experts, (int32_t)l.moe.experts);
         }
         out->side_dim = s.side_dim;
         out->layer_runs = (int32_t)s.runs().size();
@@ -124,13 +127,29 @@ int32_t mk_mixer_inspect(const char* dir, mk_mixer_summary* out) {
     });
 }
 
+int32_t mk_rotary_frequencies_yarn(int32_t dims, double base, double factor, double original, double fast, double slow, double* out, double* amplitude) {
+    return guarded([&] {
+        RotarySpec r;
+        r.dims = dims;
+        r.base = base;
+        r.scaling = RotaryScaling::Yarn;
+        r.factor = factor;
+        r.original = original;
+        r.high = fast;
+        r.low = slow;
+        const std::vector<double> f = rotary_frequencies(r);
+        std::copy(f.begin(), f.end(), out);
+        *amplitude = rotary_amplitude(r);
+    });
+}
+
 int32_t mk_rotary_frequencies(int32_t dims, double base, const double* scaling, double* out) {
     return guarded([&] {
         RotarySpec r;
         r.dims = dims;
         r.base = base;
         if (scaling != nullptr) {
-            r.scaled = true;
+            r.scaling = RotaryScaling::Turns;
             r.factor = scaling[0];
             r.low = scaling[1];
             r.high = scaling[2];

@@ -180,8 +180,11 @@ struct HgParams {
     float* partial;
     int32_t* status;
     // gated epilogue (splits == 1): weight rows 2j / 2j+1 are the gate / up projections of feature j and the kernel
-    // writes yh[t][j] = f16(act(gate) * up) instead of y; 0 = off, 1 = SiLU, 2 = tanh GELU
+    // writes yh[t][j] = f16(act(gate, up)) instead of y; 0 = off, otherwise 1 + GatedAct::Kind
     int gated;
+    float act_limit;
+    const float* act_pre;
+    const float* act_post;
     __half* yh;
     int ldyh;
     int bf16;  // both operands (and yh) are bfloat16
@@ -191,6 +194,18 @@ struct HgParams {
     int group_tiles;
     int scattered;  // the result goes where `scatter` says (splits == 1)
     MatmulScatter scatter;
+    // activation rows grouped by expert: row_tiles row tiles per expert, item = (expert, row tile, token tile of its rows)
+    int experts;
+    int expert_rows;          // true rows of an expert's matrix
+    const int32_t* offsets;   // [experts + 1]
+};
+constexpr int HG_MAX_EXPERTS = 1024;
+
+// One output tile: the first weight row, the first activation row, and the bounds of what counts.
+struct HgTile {
+    int w_row, row0;          // weight row of the tile (within the whole image), output row it becomes
+    int x_row, tok0, tok_end; // activation row of the tile (box), its first output row, end of the output rows
+    int rows;                 // end of the output columns
 };
 
 __device__ __forceinline__ int group_row0(const HgParams& p, int m_tile) {
@@ -227,6 +242,8 @@ hgemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant_
     using L = HgSmem<BN, STAGES>;
     constexpr int LD_COLS = BN >= 32 ? 32 : BN;
     extern __shared__ uint8_t hg_smem_raw[];
+    __shared__ int32_t first_item[HG_MAX_EXPERTS + 1];  // grouped by expert: items of the experts before
+    __shared__ int32_t first_row[HG_MAX_EXPERTS + 1];
     uint8_t* tiles = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(hg_smem_raw) + 1023) & ~(uintptr_t)1023);
     uint64_t* bars = reinterpret_cast<uint64_t*>(tiles + (size_t)STAGES * L::STAGE_BYTES);
     uint64_t* full = bars;                  // [STAGES]  loader -> MMA
@@ -238,7 +255,7 @@ hgemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant_
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int k_blocks = p.K / HG_BK;
     const int mn_tiles = p.row_tiles * p.n_tiles;
-    const int total_items = mn_tiles * p.splits;
+    int total_items = mn_tiles * p.splits;
     constexpr uint32_t TMEM_COLS = 2 * BN < 32 ? 32 : 2 * BN;
 
     if (threadIdx.x == 0) {
@@ -267,13 +284,62 @@ hgemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant_
     // (the activations) it loads next.  Every other access to global memory of this kernel (the epilogue's
     // stores) is ordered after those loads through the mbarriers.
     pdl_trigger();
+    if (p.experts > 0) {
+        // the row ranges are the predecessor's: one warp turns them into item numbers
+        pdl_wait();
+        if (warp == 0) {
+            int carry = 0;
+            for (int base = 0; base < p.experts; base += 32) {
+                const int e = base + lane;
+                int lo = 0, n = 0;
+                if (e < p.experts) {
+                    lo = p.offsets[e];
+                    n = (p.offsets[e + 1] - lo + BN - 1) / BN * p.row_tiles;
+                }
+                int inc = n;
+#pragma unroll
+                for (int o = 1; o < 32; o <<= 1) {
+                    const int v = __shfl_up_sync(0xffffffffu, inc, o);
+                    if (lane >= o) inc += v;
+                }
+                if (e < p.experts) {
+                    first_item[e] = carry + inc - n;
+                    first_row[e] = lo;
+                }
+                carry += __shfl_sync(0xffffffffu, inc, 31);
+            }
+            if (lane == 0) {
+                first_item[p.experts] = carry;
+                first_row[p.experts] = p.offsets[p.experts];
+            }
+        }
+        __syncthreads();
+        total_items = first_item[p.experts];
+    }
 
     // work item -> (row tile, token tile, K share); token tiles vary fastest, so the CTAs that run side by side cover
     // a few row tiles across every token tile: each weight box comes from HBM once and the activations stay in L2
-    auto decode = [&](int item, int& m_tile, int& n_tile, int& kb0, int& kb1) {
-        int mn = item % mn_tiles, split = item / mn_tiles;
-        m_tile = mn / p.n_tiles;
-        n_tile = mn % p.n_tiles;
+    auto decode = [&](int item, HgTile& t, int& kb0, int& kb1) {
+        if (p.experts > 0) {
+            int e = 0;  // the last expert whose items begin at or before this one, experts without rows have none
+            for (int step = HG_MAX_EXPERTS; step > 0; step >>= 1)
+                if (e + step < p.experts && first_item[e + step] <= item) e += step;
+            const int mn = item - first_item[e], n_tiles = (first_row[e + 1] - first_row[e] + BN - 1) / BN, m_tile = mn / n_tiles;
+            t.w_row = (e * p.row_tiles + m_tile) * HG_BM;
+            t.row0 = m_tile * HG_BM;
+            t.x_row = t.tok0 = first_row[e] + mn % n_tiles * BN;
+            t.tok_end = first_row[e + 1];
+            t.rows = p.expert_rows;
+            kb0 = 0;
+            kb1 = k_blocks;
+            return;
+        }
+        const int mn = item % mn_tiles, split = item / mn_tiles, m_tile = mn / p.n_tiles;
+        t.w_row = t.row0 = m_tile * HG_BM;
+        t.tok0 = mn % p.n_tiles * BN;
+        t.x_row = group_row0(p, m_tile) + t.tok0;
+        t.tok_end = p.T;
+        t.rows = p.rows;
         kb0 = split * p.kb_per_split;
         kb1 = min(k_blocks, kb0 + p.kb_per_split);
     };
@@ -282,12 +348,12 @@ hgemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant_
         // ---- loader
         if (lane == 0) {
             uint32_t it = 0;
-            bool ok = true, waited = false;
+            bool ok = true, waited = p.experts > 0;
             int held_x[STAGES], held_y[STAGES];  // activation boxes of the stages filled before the wait
             for (int item = blockIdx.x; item < total_items && ok; item += gridDim.x) {
-                int m_tile, n_tile, kb0, kb1;
-                decode(item, m_tile, n_tile, kb0, kb1);
-                const int x_row = group_row0(p, m_tile) + n_tile * BN;
+                HgTile tile;
+                int kb0, kb1;
+                decode(item, tile, kb0, kb1);
                 for (int kb = kb0; kb < kb1; ++kb, ++it) {
                     const uint32_t st = it % STAGES, ph = (it / STAGES) & 1;
                     if (it == STAGES && !waited) {  // the ring is full of weights: now the activations
@@ -304,12 +370,12 @@ hgemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant_
                     uint8_t* a_dst = tiles + (size_t)st * L::STAGE_BYTES;
                     uint8_t* b_dst = a_dst + L::A_BYTES;
                     mbar_expect_tx(&full[st], (uint32_t)L::STAGE_BYTES);
-                    tma_load_2d(a_dst, &tm_w, kb * HG_BK, m_tile * HG_BM, &full[st]);
+                    tma_load_2d(a_dst, &tm_w, kb * HG_BK, tile.w_row, &full[st]);
                     if (waited) {
-                        tma_load_2d(b_dst, &tm_x, kb * HG_BK, x_row, &full[st]);
+                        tma_load_2d(b_dst, &tm_x, kb * HG_BK, tile.x_row, &full[st]);
                     } else {
                         held_x[st] = kb * HG_BK;
-                        held_y[st] = x_row;
+                        held_y[st] = tile.x_row;
                     }
                 }
             }
@@ -326,8 +392,9 @@ hgemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant_
             uint32_t it = 0, tile_it = 0;
             bool ok = true;
             for (int item = blockIdx.x; item < total_items && ok; item += gridDim.x, ++tile_it) {
-                int m_tile, n_tile, kb0, kb1;
-                decode(item, m_tile, n_tile, kb0, kb1);
+                HgTile tile;
+                int kb0, kb1;
+                decode(item, tile, kb0, kb1);
                 const uint32_t acc = tile_it & 1, acc_ph = (tile_it >> 1) & 1;
                 if (!mbar_wait(&acc_empty[acc], acc_ph ^ 1, HG_SPIN_LIMIT)) {
                     atomicExch(p.status, 12);
@@ -360,11 +427,13 @@ hgemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant_
         // ---- epilogue: warps 2..5 own TMEM lane quadrants (warp % 4)
         const int quad = warp & 3;
         const int etid = (int)threadIdx.x - 64;  // 0..127 among the epilogue threads
+        if (p.act_post != nullptr) pdl_wait();   // the factors of the rows come from a predecessor
         uint32_t tile_it = 0;
         for (int item = blockIdx.x; item < total_items; item += gridDim.x, ++tile_it) {
-            int m_tile, n_tile, kb0, kb1;
-            decode(item, m_tile, n_tile, kb0, kb1);
-            const int split = item / mn_tiles;
+            HgTile tile;
+            int kb0, kb1;
+            decode(item, tile, kb0, kb1);
+            const int split = p.splits > 1 ? item / mn_tiles : 0;
             const uint32_t acc = tile_it & 1, acc_ph = (tile_it >> 1) & 1;
             // every epilogue warp waits for itself, then the four agree on the outcome, so that a wait that
             // gave up takes all of them out of the loop together (they meet again at named barrier 1)
@@ -383,13 +452,13 @@ hgemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant_
                 break;
             }
             asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-            const int row = m_tile * HG_BM + quad * 32 + lane;
-            const int tok0 = n_tile * BN;
+            const int row = tile.row0 + quad * 32 + lane;
+            const int tok0 = tile.tok0;
             float* dst = p.splits > 1 ? p.partial + (int64_t)split * p.T * p.rows : p.y;
             const int ld = p.splits > 1 ? p.rows : p.ldy;
 #pragma unroll 1
             for (int cb = 0; cb < BN; cb += LD_COLS) {
-                if (tok0 + cb >= p.T) break;  // uniform over the CTA: nothing but padding from here on
+                if (tok0 + cb >= tile.tok_end) break;  // uniform over the CTA: nothing but padding from here on
                 uint32_t r[32];
                 tmem_ld32(tmem_base + ((uint32_t)(quad * 32) << 16) + acc * BN + (uint32_t)cb, r);
                 asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
@@ -405,26 +474,33 @@ hgemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant_
                         float g = odd ? theirs : __uint_as_float(r[i]);
                         float u = odd ? __uint_as_float(r[i + 1]) : theirs;
                         int tok = tok0 + cb + i + (odd ? 1 : 0);
-                        if (row < p.rows && tok < p.T) {
-                            float a = p.gated == 1 ? hg_silu(g) : hg_gelu_tanh(g);
-                            if (p.bf16) reinterpret_cast<__nv_bfloat16*>(p.yh)[(int64_t)tok * p.ldyh + feature] = __float2bfloat16_rn(a * u);
-                            else p.yh[(int64_t)tok * p.ldyh + feature] = __float2half_rn(a * u);
+                        if (row < tile.rows && tok < tile.tok_end) {
+                            float a;
+                            if (p.gated == 1 + GatedAct::Clamped) {
+                                const float pre = p.act_pre != nullptr ? p.act_pre[tok] : 1.0f;
+                                a = clamped_gate_f(pre * g, pre * u, p.act_limit);
+                                if (p.act_post != nullptr) a *= p.act_post[tok];
+                            } else {
+                                a = (p.gated == 1 + GatedAct::Silu ? hg_silu(g) : hg_gelu_tanh(g)) * u;
+                            }
+                            if (p.bf16) reinterpret_cast<__nv_bfloat16*>(p.yh)[(int64_t)tok * p.ldyh + feature] = __float2bfloat16_rn(a);
+                            else p.yh[(int64_t)tok * p.ldyh + feature] = __float2half_rn(a);
                         }
                     }
                 } else if (p.scattered != 0) {
-                    const int64_t col = row < p.rows ? p.scatter.column(row) : -1;
+                    const int64_t col = row < tile.rows ? p.scatter.column(row) : -1;
                     if (col >= 0) {
 #pragma unroll
                         for (int i = 0; i < 32; ++i) {
                             const int tok = tok0 + cb + i;
-                            if (tok < p.T) p.scatter.put(p.scatter.row(tok) + col, __uint_as_float(r[i]));
+                            if (tok < tile.tok_end) p.scatter.put(p.scatter.row(tok) + col, __uint_as_float(r[i]));
                         }
                     }
-                } else if (row < p.rows) {
+                } else if (row < tile.rows) {
 #pragma unroll
                     for (int i = 0; i < 32; ++i) {
                         int tok = tok0 + cb + i;
-                        if (tok < p.T) {
+                        if (tok < tile.tok_end) {
                             float v = __uint_as_float(r[i]);
                             if (p.splits == 1) v = finish_value(v, p);
                             dst[(int64_t)tok * ld + row] = v;
@@ -630,35 +706,53 @@ HgemmPlan hgemm_tc_plan(int64_t rows, int64_t cols, int T, int max_splits) {
 
 namespace {
 int launch_hgemm_any(const HalfWeight& W, const __half* xh, int T, float* y, int ldy, float out_scale, float softcap,
-                     const HgemmScratch& ws, cudaStream_t s, int max_splits, int gated, __half* yh, int ldyh,
-                     const MatmulScatter* scatter = nullptr);
+                     const HgemmScratch& ws, cudaStream_t s, int max_splits, const GatedAct* act, __half* yh, int ldyh,
+                     const MatmulScatter* scatter = nullptr, const ExpertRows* experts = nullptr);
 }
 
 int launch_hgemm_tc(const HalfWeight& W, const __half* xh, int T, float* y, int ldy, float out_scale, float softcap,
                     const HgemmScratch& ws, cudaStream_t s, int max_splits) {
-    return launch_hgemm_any(W, xh, T, y, ldy, out_scale, softcap, ws, s, max_splits, 0, nullptr, 0);
+    return launch_hgemm_any(W, xh, T, y, ldy, out_scale, softcap, ws, s, max_splits, nullptr, nullptr, 0);
 }
 
 void launch_hgemm_tc_scatter(const HalfWeight& W, const __half* xh, int T, const MatmulScatter& to, const HgemmScratch& ws, cudaStream_t s) {
     if (to.out == nullptr || to.part_rows <= 0) throw std::runtime_error("launch_hgemm_tc_scatter: no destination");
-    launch_hgemm_any(W, xh, T, nullptr, 0, 1.0f, 0.f, ws, s, 1, 0, nullptr, 0, &to);
+    launch_hgemm_any(W, xh, T, nullptr, 0, 1.0f, 0.f, ws, s, 1, nullptr, nullptr, 0, &to);
 }
 
-void launch_hgemm_tc_gated(const HalfWeight& W, const __half* xh, int T, int act, __half* yh, int ldyh, const HgemmScratch& ws,
+void launch_hgemm_tc_gated(const HalfWeight& W, const __half* xh, int T, const GatedAct& act, __half* yh, int ldyh, const HgemmScratch& ws,
                            cudaStream_t s) {
     if (W.rows % 2 != 0 || yh == nullptr) throw std::runtime_error("launch_hgemm_tc_gated: needs an interleaved gate/up image and an output");
-    launch_hgemm_any(W, xh, T, nullptr, 0, 1.0f, 0.f, ws, s, 1, act == 0 ? 1 : 2, yh, ldyh);
+    launch_hgemm_any(W, xh, T, nullptr, 0, 1.0f, 0.f, ws, s, 1, &act, yh, ldyh);
+}
+
+void launch_hgemm_tc_experts(const HalfWeight& W, const ExpertRows& experts, const __half* xh, int T, float* y, int ldy, const GatedAct* act, __half* yh,
+                             int ldyh, const HgemmScratch& ws, cudaStream_t s) {
+    if (experts.experts <= 0 || experts.experts > HG_MAX_EXPERTS || experts.offsets == nullptr || experts.rows_padded % HG_BM != 0 ||
+        W.rows != (int64_t)experts.experts * experts.rows_padded || W.n_groups != 1)
+        throw std::runtime_error("launch_hgemm_tc_experts: at most 1024 experts of whole 128-row tiles");
+    if ((act != nullptr) != (yh != nullptr)) throw std::runtime_error("launch_hgemm_tc_experts: the gated form writes its own output");
+    launch_hgemm_any(W, xh, T, y, ldy, 1.0f, 0.f, ws, s, 1, act, yh, ldyh, nullptr, &experts);
 }
 
 namespace {
 int launch_hgemm_any(const HalfWeight& W, const __half* xh, int T, float* y, int ldy, float out_scale, float softcap,
-                     const HgemmScratch& ws, cudaStream_t s, int max_splits, int gated, __half* yh, int ldyh,
-                     const MatmulScatter* scatter) {
+                     const HgemmScratch& ws, cudaStream_t s, int max_splits, const GatedAct* act, __half* yh, int ldyh,
+                     const MatmulScatter* scatter, const ExpertRows* experts) {
     if (T <= 0) return 1;
     if (!W.ready) throw std::runtime_error("launch_hgemm_tc: the f16 image of the matrix was not built");
     if (xh == nullptr) throw std::runtime_error("launch_hgemm_tc: f16 activations missing");
     if (out_scale != 1.0f || softcap != 0.f || ws.partial == nullptr) max_splits = 1;
     HgemmPlan pl = hgemm_tc_plan(W.rows, W.cols, T, max_splits);
+    if (experts != nullptr) {
+        // token tiles about as wide as an expert has rows: what lies behind them belongs to the next one and is computed for nothing
+        const int mean = (T + experts->experts - 1) / experts->experts;
+        pl.bn = mean <= 48 ? 64 : (mean <= 160 ? 128 : 256);
+        pl.row_tiles = experts->rows_padded / HG_BM;
+        pl.n_tiles = 1;
+        pl.splits = 1;
+        pl.kb_per_split = (int)(W.cols / HG_BK);
+    }
     if (pl.splits > 1 && pl.partial_floats > ws.partial_floats) {
         pl.splits = 1;
         pl.kb_per_split = (int)(W.cols / HG_BK);
@@ -679,7 +773,13 @@ int launch_hgemm_any(const HalfWeight& W, const __half* xh, int T, float* y, int
     p.kb_per_split = pl.kb_per_split;
     p.partial = ws.partial;
     p.status = ws.status;
-    p.gated = gated;
+    p.gated = act != nullptr ? 1 + act->kind : 0;
+    p.act_limit = act != nullptr ? act->limit : 0.f;
+    p.act_pre = act != nullptr ? act->pre : nullptr;
+    p.act_post = act != nullptr ? act->post : nullptr;
+    p.experts = experts != nullptr ? experts->experts : 0;
+    p.expert_rows = experts != nullptr ? experts->rows : 0;
+    p.offsets = experts != nullptr ? experts->offsets : nullptr;
     p.yh = yh;
     p.ldyh = ldyh;
     p.bf16 = W.bf16 ? 1 : 0;
@@ -688,7 +788,8 @@ int launch_hgemm_any(const HalfWeight& W, const __half* xh, int T, float* y, int
     p.group_tiles = W.group_tiles;
     p.scattered = scatter != nullptr ? 1 : 0;
     if (scatter != nullptr) p.scatter = *scatter;
-    const int grid = std::min(device_sm_count(), p.row_tiles * p.n_tiles * p.splits);
+    const int most_items = experts != nullptr ? p.row_tiles * (std::min(T, experts->experts) + T / pl.bn) : p.row_tiles * p.n_tiles * p.splits;
+    const int grid = std::min(device_sm_count(), most_items);
     const CUtensorMap& tw = *reinterpret_cast<const CUtensorMap*>(W.tmap);
     if (pl.bn == 256) launch_hg<256, 4>(tw, tx, p, grid, s);
     else if (pl.bn == 128) launch_hg<128, 6>(tw, tx, p, grid, s);

@@ -2,6 +2,7 @@
 #pragma once
 #include "common.cuh"
 #include "device_util.h"
+#include "row_types.cuh"
 
 namespace mk {
 
@@ -62,11 +63,21 @@ int launch_hgemm_tc(const HalfWeight& W, const __half* xh, int T, float* y, int 
 void launch_hgemm_tc_scatter(const HalfWeight& W, const __half* xh, int T, const MatmulScatter& to, const HgemmScratch& ws, cudaStream_t s);
 
 // Gated feed-forward front half in one kernel: with W an interleaved gate/up image (2F rows),
-// yh[t][j] = f16(act(sum_k xh[t][k] gate[j][k]) * sum_k xh[t][k] up[j][k]), j < F; act 0 = SiLU, otherwise tanh GELU.
+// yh[t][j] = f16(act(sum_k xh[t][k] gate[j][k], sum_k xh[t][k] up[j][k])), j < F (see GatedAct).
 // The two sums are the f32 accumulators of the plain GEMM and the activation is evaluated like the separate SwiGLU
 // kernel does, so the halves written equal the ones that kernel derives from the plain GEMM's output.  (bf16 for a bf16
 // image.)
-void launch_hgemm_tc_gated(const HalfWeight& W, const __half* xh, int T, int act, __half* yh, int ldyh, const HgemmScratch& ws,
+void launch_hgemm_tc_gated(const HalfWeight& W, const __half* xh, int T, const GatedAct& act, __half* yh, int ldyh, const HgemmScratch& ws,
                            cudaStream_t s);
+
+// Rows grouped by expert: W stacks the matrices of `experts` experts, rows_padded rows each (a multiple of 128, of which `rows`
+// count); rows [offsets[e], offsets[e + 1]) of xh [T][cols] and of the result meet expert e's.  The ranges are read on the device.
+// With `act` the matrices are interleaved gate/up rows and the result is yh (act->pre / post by grouped row), else y.
+struct ExpertRows {
+    int experts = 0, rows_padded = 0, rows = 0;
+    const int32_t* offsets = nullptr;  // device, [experts + 1]
+};
+void launch_hgemm_tc_experts(const HalfWeight& W, const ExpertRows& experts, const __half* xh, int T, float* y, int ldy, const GatedAct* act, __half* yh,
+                             int ldyh, const HgemmScratch& ws, cudaStream_t s);
 
 }  // namespace mk

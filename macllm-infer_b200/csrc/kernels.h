@@ -94,6 +94,8 @@ struct RopeKvArgs {
     int ldq_out = 0;
     const float* q_norm_w = nullptr;  // [d] or null
     const float* k_norm_w = nullptr;  // [d] or null
+    // launch_rope_kv_rows: biases, and norm weights over all heads at once ([q_heads * d], [kv_heads * d])
+    const float *q_bias = nullptr, *k_bias = nullptr, *v_bias = nullptr;
     float norm_eps = 1e-6f;
     const float* cos_t = nullptr;  // [capacity][rotary_dim/2], null on NoPE layers
     const float* sin_t = nullptr;
@@ -110,6 +112,8 @@ struct RopeKvArgs {
     int interleaved = 0; // rotate the pairs (2i, 2i + 1) instead of (i, i + rotary_dim / 2)
 };
 void launch_rope_kv(const RopeKvArgs& a, cudaStream_t s);
+// The same for projections with biases whose query and key norms run over all heads at once (q_out required).
+void launch_rope_kv_rows(const RopeKvArgs& a, cudaStream_t s);
 
 // Copy `rows` token rows of every layer and head from block src to block dst (copy-on-write).
 void launch_cow_copy(void* k_pool, void* v_pool, int kv_f16, int64_t src_block, int64_t dst_block, int rows,
@@ -128,8 +132,19 @@ struct AttnArgs {
     int64_t pool_blocks = 0;  // see kv_page_index
     float scale = 1.f, softcap = 0.f;
     int window = 0;  // 0 = full causal
+    int chunk = 0;   // > 0: a position sees the keys of its own chunk only (chunks counted from position 0)
+    const float* sink = nullptr;  // [q_heads]: one more term exp(sink) in the denominator; null: none
     int q_tile = 0;
 };
+// The first key the position sees.
+__host__ __device__ __forceinline__ int attention_first_key(int position, int window, int chunk) {
+    int lo = window > 0 && position >= window ? position - window + 1 : 0;
+    if (chunk > 0) {
+        const int c = position - position % chunk;
+        lo = c > lo ? c : lo;
+    }
+    return lo;
+}
 void launch_paged_attention(const AttnArgs& a, cudaStream_t s);
 int attention_q_tile(int q_heads, int kv_heads);
 

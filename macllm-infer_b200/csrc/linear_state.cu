@@ -9,6 +9,7 @@
 // and leave the head norm to a second kernel; ticks of short lanes give a whole head to one CTA, which then finishes the output
 // row itself: there the state's way through the SM is what counts.
 #include "linear_state.h"
+#include "recurrent_core.cuh"
 #include <algorithm>
 
 namespace mk {
@@ -17,6 +18,16 @@ namespace {
 
 constexpr int LS_WIDE_WARPS = 4;  // warps of a CTA that owns part of a head
 constexpr int LS_MAX_FINISH_V = 128;
+
+enum LsRule : int { LS_WKV, LS_DELTA, LS_MLSTM };
+template <LsRule RULE>
+struct LsArgs;
+template <>
+struct LsArgs<LS_WKV> { using type = WkvScanArgs; };
+template <>
+struct LsArgs<LS_DELTA> { using type = DeltaScanArgs; };
+template <>
+struct LsArgs<LS_MLSTM> { using type = MlstmScanArgs; };
 
 __device__ __forceinline__ void ls_cp_async16(void* dst, const void* src) {
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
@@ -67,48 +78,55 @@ __device__ __forceinline__ float fold8(const float (&v)[8], int t) {
     return r;
 }
 
-// One head's row o[0 .. vdim) of packed row `row`, by one warp; gate[v] and norm weights nw[v] of the head.
+// One head's row o[0 .. vdim) of packed row `row`, by one warp; gate[v] and norm weights nw[v] of the head, den: its denominator.
 template <typename Gate>
-__device__ __forceinline__ void finish_head_row(const LinearStateArgs& a, const float* o, Gate gate, const float* nw, int64_t row, int head, int lane) {
+__device__ __forceinline__ void finish_head_row(const LinearStateArgs& a, const float* o, float den, Gate gate, const float* nw, int64_t row, int head, int lane) {
     float ss = 0.f;
-    for (int v = lane; v < a.vdim; v += 32) ss += o[v] * o[v];
+    for (int v = lane; v < a.vdim; v += 32) ss += (o[v] / den) * (o[v] / den);
     ss = warp_sum(ss);
     const float root = sqrtf(ss / (float)a.vdim + a.eps);
-    for (int v = lane; v < a.vdim; v += 32) a.image.put(row, head * a.vdim + v, o[v] / root * nw[v] * silu_f(gate(v)));
+    for (int v = lane; v < a.vdim; v += 32) {
+        const float g = gate(v);
+        a.image.put(row, head * a.vdim + v, o[v] / den / root * nw[v] * (a.gate_sigmoid ? sigmoid_f(g) : silu_f(g)));
+    }
     if (head == a.heads - 1)
         for (int c = a.heads * a.vdim + lane; c < a.image.end(); c += 32) a.image.put(row, c, 0.f);
 }
 
-template <int KD, bool WKV, bool FINISH>
+template <int KD, LsRule RULE, bool FINISH>
 struct Ls {
+    static constexpr bool WKV = RULE == LS_WKV;
+    static constexpr int EXTRA = RULE == LS_MLSTM ? 1 : 0;   // columns of the state beside the values
     static constexpr int KS = !FINISH && KD >= 64 ? 16 : 8;  // threads of a column pair
     static constexpr int KE = KD / KS;                       // keys of a thread
     static constexpr int COLS = 32 / KS * 2;                 // value columns of a warp
     static constexpr int TT = FINISH ? 4 : 16;               // rows of a chunk
     static constexpr int KROWS = WKV ? 3 : 2;                // r, k, decay  /  q, k
-    static constexpr int MAX_THREADS = FINISH ? LS_MAX_FINISH_V / COLS * 32 : LS_WIDE_WARPS * 32;
-    static constexpr int MIN_CTAS = FINISH ? (KD >= 128 ? 2 : 3) : 1;
-    // stage: KROWS key-wide rows, the value row, the gate row (FINISH), decay and beta (delta rule)
+    static constexpr int MAX_THREADS = FINISH ? (LS_MAX_FINISH_V / COLS + EXTRA) * 32 : LS_WIDE_WARPS * 32;
+    static constexpr int MIN_CTAS = FINISH ? (KD >= 128 ? 2 : 3) - EXTRA : 1;
+    // stage: KROWS key-wide rows, the value row, the gate row (FINISH), decay, write and floor of the denominator (not WKV)
     static __host__ __device__ constexpr int row_floats(int cols) { return KROWS * KD + cols * (FINISH ? 2 : 1) + (WKV ? 0 : 4); }
     static __host__ __device__ constexpr int stage_floats(int cols) { return TT * row_floats(cols); }
     // two stages; FINISH: the output rows and the head's norm weights
     static __host__ __device__ constexpr size_t bytes(int cols) { return (2 * (size_t)stage_floats(cols) + (FINISH ? (size_t)(TT + 1) * cols : 0)) * 4; }
 };
 
-template <int KD, bool WKV, bool FINISH>
-__global__ void __launch_bounds__(Ls<KD, WKV, FINISH>::MAX_THREADS, Ls<KD, WKV, FINISH>::MIN_CTAS)
-linear_state_kernel(const __grid_constant__ WkvScanArgs wa, const __grid_constant__ DeltaScanArgs da) {
-    using L = Ls<KD, WKV, FINISH>;
+template <int KD, LsRule RULE, bool FINISH>
+__global__ void __launch_bounds__(Ls<KD, RULE, FINISH>::MAX_THREADS, Ls<KD, RULE, FINISH>::MIN_CTAS)
+linear_state_kernel(const __grid_constant__ typename LsArgs<RULE>::type ra) {
+    using L = Ls<KD, RULE, FINISH>;
+    constexpr bool WKV = L::WKV;
     constexpr int TT = L::TT, KS = L::KS, KE = L::KE, NJ = KE / 4;
     extern __shared__ __align__(16) float ls_smem[];
-    const LinearStateArgs& a = WKV ? wa.common : da.common;
+    const LinearStateArgs& a = ra.common;
+    const int state_cols = a.vdim + L::EXTRA;
 
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, ks = lane & (KS - 1);
     const int cols = (int)(blockDim.x >> 5) * L::COLS;                 // columns of this CTA
     const int col0 = blockIdx.x * cols;
     const int head = blockIdx.y;
     const int c_loc = warp * L::COLS + lane / KS * 2;                  // first of the thread's two columns, within the CTA
-    const int my_cols = min(cols, a.vdim - col0);
+    const int my_cols = max(0, min(cols, a.vdim - col0));              // of them values
     float* s_o = ls_smem + 2 * L::stage_floats(cols);                  // FINISH: [TT][cols]
     float* s_nw = s_o + TT * cols;                                     // FINISH: [cols]
 
@@ -117,11 +135,11 @@ linear_state_kernel(const __grid_constant__ WkvScanArgs wa, const __grid_constan
     pdl_trigger();
     const StateLane sl = a.lanes.at(blockIdx.z);
     float S[2][KE];
-    const int64_t head_state = (int64_t)a.vdim * KD;
+    const int64_t head_state = (int64_t)state_cols * KD;
 #pragma unroll
     for (int c = 0; c < 2; ++c) {
         const int v = col0 + c_loc + c;
-        const bool live = sl.in >= 0 && v < a.vdim;
+        const bool live = sl.in >= 0 && v < state_cols;
         const float4* src = reinterpret_cast<const float4*>(a.state + ((int64_t)sl.in * a.heads + head) * head_state + (int64_t)v * KD);
 #pragma unroll
         for (int j = 0; j < NJ; ++j) {
@@ -130,12 +148,17 @@ linear_state_kernel(const __grid_constant__ WkvScanArgs wa, const __grid_constan
         }
     }
     float U[WKV ? KE : 1];
-    if (WKV) {
+    if constexpr (WKV) {
 #pragma unroll
         for (int e = 0; e < KE; ++e) {
             const int i = (e >> 2) * 4 * KS + ks * 4 + (e & 3);
-            U[WKV ? e : 0] = i < a.dim ? wa.bonus[head * a.dim + i] : 0.f;
+            U[e] = i < a.dim ? ra.bonus[head * a.dim + i] : 0.f;
         }
+    }
+    // mLSTM: the first warp turns the gates of a chunk's rows into decay, write and floor, a row per lane
+    float run_max = 0.f;
+    if constexpr (RULE == LS_MLSTM) {
+        if (warp == 0 && sl.in >= 0) run_max = ra.running_max[(int64_t)sl.in * a.heads + head];
     }
     if (FINISH)
         for (int v = threadIdx.x; v < a.vdim; v += blockDim.x) s_nw[v] = a.norm_w[(a.norm_per_head ? head * a.vdim : 0) + v];
@@ -144,11 +167,15 @@ linear_state_kernel(const __grid_constant__ WkvScanArgs wa, const __grid_constan
         for (int i = threadIdx.x; i < 2 * L::stage_floats(cols); i += blockDim.x) ls_smem[i] = 0.f;
         __syncthreads();
     }
+    if (RULE == LS_MLSTM && a.vdim >= col0 && a.vdim < col0 + cols)  // the normaliser's value
+        for (int i = threadIdx.x; i < 2 * TT; i += blockDim.x)
+            ls_smem[i / TT * L::stage_floats(cols) + TT * L::KROWS * KD + i % TT * cols + a.vdim - col0] = 1.f;
     pdl_wait();
 
     const int first = sl.first, n = sl.n;
-    const int kv_head = WKV ? head : head / (a.heads / da.kv_heads);
     const bool vec = (a.dim & 3) == 0 && (a.vdim & 3) == 0;
+    const int raw_width = RULE == LS_MLSTM ? linear_state_raw_width(a.vdim) : a.vdim;
+    const float q_scale = RULE == LS_MLSTM ? rsqrtf((float)a.dim) : 1.f;
     auto stage = [&](int which) { return ls_smem + which * L::stage_floats(cols); };
     auto fetch = [&](int chunk) {
         float* s = stage(chunk & 1);
@@ -156,29 +183,62 @@ linear_state_kernel(const __grid_constant__ WkvScanArgs wa, const __grid_constan
         const int m = min(TT, n - chunk * TT);
         float* s_v = s + TT * L::KROWS * KD;
         float* s_g = s_v + TT * cols;
-        if (WKV) {
-            const Shares& y = wa.rkv;
-            const int h0 = head * a.dim;
+        float* s_c = s_v + TT * cols * (FINISH ? 2 : 1);
+        // the first key-wide row, the second and the values, from a matmul's output
+        auto fetch_heads = [&](const Shares& y, int x_col, int k_col, int v_col) {
             if (y.n == 1) {
                 const bool yv = vec && (y.ld & 3) == 0;
-                fetch_rows(s, KD, m, a.dim, yv, [&](int r) { return y.p + (r0 + r) * y.ld + wa.r_col + h0; });
-                fetch_rows(s + TT * KD, KD, m, a.dim, yv, [&](int r) { return y.p + (r0 + r) * y.ld + wa.k_col + h0; });
-                fetch_rows(s_v, cols, m, my_cols, yv && (my_cols & 3) == 0, [&](int r) { return y.p + (r0 + r) * y.ld + wa.v_col + h0 + col0; });
+                fetch_rows(s, KD, m, a.dim, yv, [&](int r) { return y.p + (r0 + r) * y.ld + x_col; });
+                fetch_rows(s + TT * KD, KD, m, a.dim, yv, [&](int r) { return y.p + (r0 + r) * y.ld + k_col; });
+                fetch_rows(s_v, cols, m, my_cols, yv && (my_cols & 3) == 0, [&](int r) { return y.p + (r0 + r) * y.ld + v_col; });
             } else {
-                sum_rows(s, KD, m, a.dim, y, r0, wa.r_col + h0);
-                sum_rows(s + TT * KD, KD, m, a.dim, y, r0, wa.k_col + h0);
-                sum_rows(s_v, cols, m, my_cols, y, r0, wa.v_col + h0 + col0);
+                sum_rows(s, KD, m, a.dim, y, r0, x_col);
+                sum_rows(s + TT * KD, KD, m, a.dim, y, r0, k_col);
+                sum_rows(s_v, cols, m, my_cols, y, r0, v_col);
             }
-            fetch_rows(s + 2 * TT * KD, KD, m, a.dim, vec, [&](int r) { return wa.decay + (r0 + r) * a.heads * a.dim + h0; });
+        };
+        if constexpr (RULE == LS_WKV) {
+            const int h0 = head * a.dim;
+            fetch_heads(ra.rkv, ra.r_col + h0, ra.k_col + h0, ra.v_col + h0 + col0);
+            fetch_rows(s + 2 * TT * KD, KD, m, a.dim, vec, [&](int r) { return ra.decay + (r0 + r) * a.heads * a.dim + h0; });
+        } else if constexpr (RULE == LS_MLSTM) {
+            const int h0 = head * a.dim;
+            fetch_heads(ra.y, ra.q_col + h0, ra.k_col + h0, ra.v_col + head * a.vdim + col0);
+            if (warp == 0) {
+                float f = 0.f, i = -INFINITY;
+                if (lane < m) {
+                    i = ra.cap * tanhf((ra.y.at(r0 + lane, ra.i_col + head) + ra.i_bias[head]) / ra.cap);
+                    f = -recurrent::softplus_stable(-ra.cap * tanhf((ra.y.at(r0 + lane, ra.f_col + head) + ra.f_bias[head]) / ra.cap));
+                }
+                // row t's maximum is max(sum of f up to t + the chunk's first maximum, running maximum of i with f added since)
+                float sum = f, top = i;
+#pragma unroll
+                for (int o = 1; o < TT; o <<= 1) {
+                    const float ps = __shfl_up_sync(0xffffffffu, sum, o), pt = __shfl_up_sync(0xffffffffu, top, o);
+                    if (lane >= o) {
+                        top = fmaxf(pt + sum, top);
+                        sum += ps;
+                    }
+                }
+                const float mt = fmaxf(run_max + sum, top);
+                float before = __shfl_up_sync(0xffffffffu, mt, 1);
+                if (lane == 0) before = run_max;
+                if (lane < m) {
+                    s_c[4 * lane] = expf(f + before - mt);
+                    s_c[4 * lane + 1] = expf(i - mt);
+                    s_c[4 * lane + 2] = expf(-mt);
+                }
+                run_max = __shfl_sync(0xffffffffu, mt, m - 1);
+            }
         } else {
-            const int64_t kw = (int64_t)da.kv_heads * a.dim, vw = (int64_t)a.heads * a.vdim;
-            fetch_rows(s, KD, m, a.dim, vec, [&](int r) { return da.q + (r0 + r) * kw + kv_head * a.dim; });
-            fetch_rows(s + TT * KD, KD, m, a.dim, vec, [&](int r) { return da.k + (r0 + r) * kw + kv_head * a.dim; });
-            fetch_rows(s_v, cols, m, my_cols, vec && (my_cols & 3) == 0, [&](int r) { return da.v + (r0 + r) * vw + head * a.vdim + col0; });
-            float* s_c = s_v + TT * cols * (FINISH ? 2 : 1);
+            const int kv_head = head / (a.heads / ra.kv_heads);
+            const int64_t kw = (int64_t)ra.kv_heads * a.dim, vw = (int64_t)a.heads * a.vdim;
+            fetch_rows(s, KD, m, a.dim, vec, [&](int r) { return ra.q + (r0 + r) * kw + kv_head * a.dim; });
+            fetch_rows(s + TT * KD, KD, m, a.dim, vec, [&](int r) { return ra.k + (r0 + r) * kw + kv_head * a.dim; });
+            fetch_rows(s_v, cols, m, my_cols, vec && (my_cols & 3) == 0, [&](int r) { return ra.v + (r0 + r) * vw + head * a.vdim + col0; });
             for (int r = threadIdx.x; r < m; r += blockDim.x) {
-                ls_cp_async4(s_c + 4 * r, da.decay + (r0 + r) * a.heads + head);
-                ls_cp_async4(s_c + 4 * r + 1, da.beta + (r0 + r) * a.heads + head);
+                ls_cp_async4(s_c + 4 * r, ra.decay + (r0 + r) * a.heads + head);
+                ls_cp_async4(s_c + 4 * r + 1, ra.beta + (r0 + r) * a.heads + head);
             }
         }
         if (FINISH) sum_rows(s_g, cols, m, a.vdim, a.gate, r0, a.gate_col + head * a.vdim);
@@ -243,7 +303,16 @@ linear_state_kernel(const __grid_constant__ WkvScanArgs wa, const __grid_constan
         };
         auto step = [&](const Row& r, float& out0, float& out1) {
             float o0 = 0.f, o1 = 0.f;
-            if constexpr (WKV) {
+            if constexpr (RULE == LS_MLSTM) {
+                const float u0 = r.gb.y * r.v.x, u1 = r.gb.y * r.v.y;
+#pragma unroll
+                for (int e = 0; e < KE; ++e) {
+                    S[0][e] = fmaf(r.y[e], u0, r.gb.x * S[0][e]);
+                    S[1][e] = fmaf(r.y[e], u1, r.gb.x * S[1][e]);
+                    o0 = fmaf(S[0][e], r.x[e], o0);
+                    o1 = fmaf(S[1][e], r.x[e], o1);
+                }
+            } else if constexpr (WKV) {
 #pragma unroll
                 for (int e = 0; e < KE; ++e) {
                     const float uk = U[e] * r.y[e];
@@ -288,13 +357,18 @@ linear_state_kernel(const __grid_constant__ WkvScanArgs wa, const __grid_constan
                     step(r, part[2 * i], part[2 * i + 1]);
                 }
             }
-            const float o = fold8<KS>(part, ks);
+            float o = fold8<KS>(part, ks);
             const int t = ks >> 1, c = c_loc + (ks & 1);
-            if (t < m && c < a.vdim) s_o[t * cols + c] = o;
+            if (RULE == LS_MLSTM) {
+                o *= q_scale;
+                if (c == a.vdim && t < m) o = fmaxf(fabsf(o), s_c[4 * t + 2]) + 1e-6f;
+            }
+            if (t < m && c < state_cols) s_o[t * cols + c] = o;
             __syncthreads();
             const float* s_g = s_v + TT * cols;
             for (int t = warp; t < m; t += (int)(blockDim.x >> 5))
-                finish_head_row(a, s_o + t * cols, [&](int v) { return s_g[t * cols + v]; }, s_nw, first + ch * TT + t, head, lane);
+                finish_head_row(a, s_o + t * cols, RULE == LS_MLSTM ? s_o[t * cols + a.vdim] : 1.f, [&](int v) { return s_g[t * cols + v]; }, s_nw,
+                                first + ch * TT + t, head, lane);
             __syncthreads();  // the stage is free for the chunk after next
         } else {
             Row rows[2];
@@ -307,10 +381,14 @@ linear_state_kernel(const __grid_constant__ WkvScanArgs wa, const __grid_constan
                     load_row(min(t0 + i + 1, TT - 1), rows[(i + 1) & 1]);
                     step(rows[i & 1], part[2 * i], part[2 * i + 1]);
                 }
-                const float o = fold8<KS>(part, ks);
+                float o = fold8<KS>(part, ks);
                 const int t = t0 + ((ks & 7) >> 1), c = c_loc + (ks & 1);
-                if (ks < 8 && t < m && col0 + c < a.vdim)
-                    a.out[(int64_t)(first + ch * TT + t) * a.heads * a.vdim + head * a.vdim + col0 + c] = o;
+                if (RULE == LS_MLSTM) {
+                    o *= q_scale;
+                    if (col0 + c == a.vdim && t < m) o = fmaxf(fabsf(o), s_c[4 * t + 2]) + 1e-6f;
+                }
+                if (ks < 8 && t < m && col0 + c < state_cols)
+                    a.out[((int64_t)(first + ch * TT + t) * a.heads + head) * raw_width + col0 + c] = o;
             }
             __syncthreads();  // the stage is free for the chunk after next
         }
@@ -319,10 +397,13 @@ linear_state_kernel(const __grid_constant__ WkvScanArgs wa, const __grid_constan
 #pragma unroll
     for (int c = 0; c < 2; ++c) {
         const int v = col0 + c_loc + c;
-        if (v >= a.vdim) continue;
+        if (v >= state_cols) continue;
         float4* dst = reinterpret_cast<float4*>(a.state + ((int64_t)sl.out * a.heads + head) * head_state + (int64_t)v * KD);
 #pragma unroll
         for (int j = 0; j < NJ; ++j) __stcs(dst + j * KS + ks, make_float4(S[c][4 * j], S[c][4 * j + 1], S[c][4 * j + 2], S[c][4 * j + 3]));
+    }
+    if constexpr (RULE == LS_MLSTM) {
+        if (blockIdx.x == 0 && threadIdx.x == 0) ra.running_max[(int64_t)sl.out * a.heads + head] = run_max;
     }
 }
 
@@ -333,7 +414,9 @@ __global__ void __launch_bounds__(128) head_norm_gate_kernel(LinearStateArgs a, 
     if (i >= (int64_t)rows * a.heads) return;
     const int64_t row = i / a.heads;
     const int head = (int)(i % a.heads);
-    finish_head_row(a, a.out + row * a.heads * a.vdim + head * a.vdim, [&](int v) { return a.gate.at(row, a.gate_col + head * a.vdim + v); },
+    const int width = a.normalised ? linear_state_raw_width(a.vdim) : a.vdim;
+    const float* o = a.out + (row * a.heads + head) * width;
+    finish_head_row(a, o, a.normalised ? o[a.vdim] : 1.f, [&](int v) { return a.gate.at(row, a.gate_col + head * a.vdim + v); },
                     a.norm_w + (a.norm_per_head ? head * a.vdim : 0), row, head, threadIdx.x & 31);
 }
 
@@ -349,7 +432,12 @@ __global__ void __launch_bounds__(128) head_norm_gate_vec_kernel(LinearStateArgs
     const bool mine = live && v < a.vdim;
     float4 o = make_float4(0.f, 0.f, 0.f, 0.f), g = o, w = o;
     if (mine) {
-        o = *reinterpret_cast<const float4*>(a.out + row * a.heads * a.vdim + head * a.vdim + v);
+        const float* src = a.out + (row * a.heads + head) * (a.normalised ? linear_state_raw_width(a.vdim) : a.vdim);
+        o = *reinterpret_cast<const float4*>(src + v);
+        if (a.normalised) {
+            const float den = src[a.vdim];
+            o = make_float4(o.x / den, o.y / den, o.z / den, o.w / den);
+        }
         g = a.gate.at4(row, a.gate_col + head * a.vdim + v);
         w = *reinterpret_cast<const float4*>(a.norm_w + (a.norm_per_head ? head * a.vdim : 0) + v);
     }
@@ -357,39 +445,41 @@ __global__ void __launch_bounds__(128) head_norm_gate_vec_kernel(LinearStateArgs
 #pragma unroll
     for (int x = 1; x < G; x <<= 1) ss += __shfl_xor_sync(0xffffffffu, ss, x);
     const float root = sqrtf(ss / (float)a.vdim + a.eps);
-    if (mine)
-        a.image.put4(row, head * a.vdim + v, make_float4(o.x / root * w.x * silu_f(g.x), o.y / root * w.y * silu_f(g.y), o.z / root * w.z * silu_f(g.z),
-                                                         o.w / root * w.w * silu_f(g.w)));
+    if (mine) {
+        g = a.gate_sigmoid ? make_float4(sigmoid_f(g.x), sigmoid_f(g.y), sigmoid_f(g.z), sigmoid_f(g.w)) : make_float4(silu_f(g.x), silu_f(g.y), silu_f(g.z), silu_f(g.w));
+        a.image.put4(row, head * a.vdim + v, make_float4(o.x / root * w.x * g.x, o.y / root * w.y * g.y, o.z / root * w.z * g.z, o.w / root * w.w * g.w));
+    }
     if (live && head == a.heads - 1)
         for (int c = a.heads * a.vdim + (int)(threadIdx.x % G); c < a.image.end(); c += G) a.image.put(row, c, 0.f);
 }
 
-template <int KD, bool WKV, bool FINISH>
-void launch_variant(const WkvScanArgs& wa, const DeltaScanArgs& da, cudaStream_t s) {
-    const LinearStateArgs& a = WKV ? wa.common : da.common;
-    using L = Ls<KD, WKV, FINISH>;
-    const int warps = FINISH ? (a.vdim + L::COLS - 1) / L::COLS : LS_WIDE_WARPS;
+template <int KD, LsRule RULE, bool FINISH>
+void launch_variant(const typename LsArgs<RULE>::type& ra, cudaStream_t s) {
+    const LinearStateArgs& a = ra.common;
+    using L = Ls<KD, RULE, FINISH>;
+    const int state_cols = a.vdim + L::EXTRA;
+    const int warps = FINISH ? (state_cols + L::COLS - 1) / L::COLS : LS_WIDE_WARPS;
     const int cols = warps * L::COLS;
     const size_t smem = L::bytes(cols);
-    auto* kernel = linear_state_kernel<KD, WKV, FINISH>;
+    auto* kernel = linear_state_kernel<KD, RULE, FINISH>;
     ensure_dynamic_smem(reinterpret_cast<const void*>(kernel), smem);
-    const dim3 grid((unsigned)((a.vdim + cols - 1) / cols), (unsigned)a.heads, (unsigned)a.lanes.lanes);
-    launch_pdl(kernel, grid, dim3((unsigned)warps * 32), smem, s, wa, da);
+    const dim3 grid((unsigned)((state_cols + cols - 1) / cols), (unsigned)a.heads, (unsigned)a.lanes.lanes);
+    launch_pdl(kernel, grid, dim3((unsigned)warps * 32), smem, s, ra);
     MK_LAUNCH_CHECK();
 }
 
-template <bool WKV>
-void launch_scan(const WkvScanArgs& wa, const DeltaScanArgs& da, cudaStream_t s) {
-    const LinearStateArgs& a = WKV ? wa.common : da.common;
+template <LsRule RULE>
+void launch_scan(const typename LsArgs<RULE>::type& ra, cudaStream_t s) {
+    const LinearStateArgs& a = ra.common;
     if (a.lanes.lanes <= 0) return;
     if (a.heads > 65535 || a.lanes.lanes > 65535) throw std::runtime_error("linear-attention scan: at most 65535 heads and lanes");
     const bool finish = a.image.h != nullptr || a.image.f != nullptr;
     if (finish && !linear_state_can_finish(a.dim, a.vdim)) throw std::runtime_error("linear-attention scan: the finishing form takes dimensions up to 128");
     switch (linear_state_key_pad(a.dim)) {
-        case 32: finish ? launch_variant<32, WKV, true>(wa, da, s) : launch_variant<32, WKV, false>(wa, da, s); break;
-        case 64: finish ? launch_variant<64, WKV, true>(wa, da, s) : launch_variant<64, WKV, false>(wa, da, s); break;
-        case 128: finish ? launch_variant<128, WKV, true>(wa, da, s) : launch_variant<128, WKV, false>(wa, da, s); break;
-        default: launch_variant<256, WKV, false>(wa, da, s); break;
+        case 32: finish ? launch_variant<32, RULE, true>(ra, s) : launch_variant<32, RULE, false>(ra, s); break;
+        case 64: finish ? launch_variant<64, RULE, true>(ra, s) : launch_variant<64, RULE, false>(ra, s); break;
+        case 128: finish ? launch_variant<128, RULE, true>(ra, s) : launch_variant<128, RULE, false>(ra, s); break;
+        default: launch_variant<256, RULE, false>(ra, s); break;
     }
 }
 
@@ -403,11 +493,13 @@ int linear_state_key_pad(int dim) {
 
 bool linear_state_can_finish(int dim, int vdim) { return dim <= 128 && vdim <= LS_MAX_FINISH_V; }
 
-void launch_wkv_scan(const WkvScanArgs& a, cudaStream_t s) { launch_scan<true>(a, DeltaScanArgs{}, s); }
+void launch_wkv_scan(const WkvScanArgs& a, cudaStream_t s) { launch_scan<LS_WKV>(a, s); }
+
+void launch_mlstm_scan(const MlstmScanArgs& a, cudaStream_t s) { launch_scan<LS_MLSTM>(a, s); }
 
 void launch_delta_scan(const DeltaScanArgs& a, cudaStream_t s) {
     if (a.kv_heads <= 0 || a.common.heads % a.kv_heads != 0) throw std::runtime_error("delta-rule scan: heads must be a multiple of kv_heads");
-    launch_scan<false>(WkvScanArgs{}, a, s);
+    launch_scan<LS_DELTA>(a, s);
 }
 
 void launch_head_norm_gate(const LinearStateArgs& a, int rows, cudaStream_t s) {

@@ -1,7 +1,8 @@
 // Linear-attention recurrences over ragged lanes with slot-held state: WKV time mixing (a decay per key channel and a bonus for
-// the current token) and the gated delta rule (one decay per head, grouped query / key heads).  State layout per slot half:
-// [heads][value columns][KD] f32, value-major, KD = the key dimension padded to 32, 64, 128 or 256 - a column's keys are
-// contiguous, so a decode tick streams the state with 16-byte accesses.
+// the current token), the gated delta rule (one decay per head, grouped query / key heads) and the matrix memory of mLSTM (one
+// decay per head from exponential gates, a normaliser).  State layout per slot half: [heads][value columns][KD] f32, value-major,
+// KD = the key dimension padded to 32, 64, 128 or 256 - a column's keys are contiguous, so a decode tick streams the state with
+// 16-byte accesses.  mLSTM has one column more than values: the normaliser, whose value is always 1.
 #pragma once
 #include "row_types.cuh"
 
@@ -10,13 +11,15 @@ namespace mk {
 // The padded key dimension of the state (throws above 256).
 int linear_state_key_pad(int dim);
 
-// What both share.  With `image` set the kernel also finishes the mixer's output - each head's row divided by its root mean
-// square, times norm_w, times silu(gate) - and writes the next matmul's input; otherwise the raw rows go to `out`.
+// What all share.  With `image` set the kernel also finishes the mixer's output - each head's row divided by its root mean
+// square, times norm_w, times silu(gate) or sigmoid(gate) - and writes the next matmul's input; otherwise the raw rows go to `out`.
 struct LinearStateArgs {
     StateLanes lanes;
     float* state = nullptr;
     int heads = 0, dim = 0, vdim = 0;
-    float* out = nullptr;            // [rows][heads * vdim]
+    float* out = nullptr;            // [rows][heads][vdim], normalised: [rows][heads][linear_state_raw_width(vdim)]
+    int normalised = 0;              // a raw head row ends with its denominator (mLSTM): divided by it before the norm
+    int gate_sigmoid = 0;            // sigmoid(gate) instead of silu(gate)
     RowImage image;                  // [rows][heads * vdim]
     const float* norm_w = nullptr;   // [heads * vdim], or [vdim] shared by the heads
     int norm_per_head = 0;           // norm_w has its own part for every head
@@ -46,6 +49,23 @@ struct DeltaScanArgs {
     const float* beta = nullptr;     // [rows][heads]
 };
 void launch_delta_scan(const DeltaScanArgs& a, cudaStream_t s);
+
+// Raw row of a normalised head: its values, then the denominator.
+__host__ __device__ inline int linear_state_raw_width(int vdim) { return (vdim + 4) / 4 * 4; }
+
+// Per head: i = cap tanh((zi + i_bias) / cap), f = log sigmoid(cap tanh((zf + f_bias) / cap));
+// m' = max(f + m, i);  S <- exp(f + m - m') S + exp(i - m') k v^T, n likewise with k alone, m <- m' (0 at the start);
+// o = S^T q / (max(|n . q|, exp(-m)) + 1e-6), q times dim^-1/2.
+struct MlstmScanArgs {
+    LinearStateArgs common;
+    Shares y;                        // columns q_col / k_col + head * dim + i, v_col + head * vdim + v, i_col / f_col + head
+    int q_col = 0, k_col = 0, v_col = 0, i_col = 0, f_col = 0;
+    const float* i_bias = nullptr;   // [heads]
+    const float* f_bias = nullptr;
+    float cap = 1.f;
+    float* running_max = nullptr;    // [slot halves][heads]
+};
+void launch_mlstm_scan(const MlstmScanArgs& a, cudaStream_t s);
 
 // Whether the finishing form (LinearStateArgs::image) exists for these sizes.
 bool linear_state_can_finish(int dim, int vdim);

@@ -12,7 +12,8 @@ namespace mk {
 namespace {
 
 const std::vector<const char*> class_names = {"hgemm_tc", "hgemm_tc_splitk", "f32_matmul", "wkv_scan", "delta_scan", "paged_attention", "rope_kv_scatter",
-                                              "row_update", "delta_prep", "wkv_decay", "latent_attention", "mingru_scan", "latent_prep", "latent_rows", "gates", "embed", "build_batch", "argmax"};
+                                              "row_update", "delta_prep", "wkv_decay", "latent_attention", "mingru_scan", "latent_prep", "latent_rows",
+                                              "mlstm_scan", "moe_gemm", "moe_rows", "gates", "embed", "build_batch", "argmax"};
 
 bool is_mixer_checkpoint(const std::string& dir) {
     struct stat st;
@@ -34,7 +35,7 @@ MixerLm::MixerLm(const std::string& dir, const ModelConfig& cfg) : DeviceLm(cfg,
     f32_ = cfg.compute_f32;
     esz_ = f32_ ? 4 : 2;
     if (f32_) cfg_.kv_f16 = false;
-    if (cfg.ep_size > 1) throw std::runtime_error("expert parallelism asked for a model without experts");
+    if (cfg.ep_size > 1) throw std::runtime_error("expert parallelism is not supported for mixer-built decoders");
     open_device();
     spec_.vocab = ms_.vocab;
     runs_ = ms_.runs();
@@ -81,7 +82,7 @@ void MixerLm::place(const SafetensorsFile& f, const Part& p, int cols, int ld, s
 }
 
 void MixerLm::upload_matrix(const std::vector<float>& m, int64_t rows, int ld, int64_t true_bytes, Dense& out, const std::vector<int64_t>& group_rows,
-                            int groups, bool per_token) {
+                            int groups, double share_per_token) {
     out.rows = rows;
     out.ld = ld;
     out.bytes = true_bytes;
@@ -98,11 +99,11 @@ void MixerLm::upload_matrix(const std::vector<float>& m, int64_t rows, int ld, i
     else if (groups > 0) build_bf16_weight_groups(m.data(), rows, ld, groups, out.half, stream_);
     else build_bf16_weight(m.data(), rows, ld, out.half, stream_, group_rows);
     spec_.weight_bytes += out.bytes;
-    if (per_token) spec_.weight_bytes_per_token += out.bytes * passes_;
+    spec_.weight_bytes_per_token += (int64_t)((double)out.bytes * share_per_token) * passes_;
 }
 
 void MixerLm::upload_dense(const SafetensorsFile& f, const std::vector<Part>& parts, int64_t rows, int cols, Dense& out,
-                           const std::vector<int64_t>& group_rows) {
+                           const std::vector<int64_t>& group_rows, double share_per_token) {
     const int ld = pad_to(cols, 64);
     std::vector<float> m((size_t)(rows * ld), 0.f);
     int64_t bytes = 0;
@@ -110,25 +111,26 @@ void MixerLm::upload_dense(const SafetensorsFile& f, const std::vector<Part>& pa
         place(f, p, cols, ld, m);
         bytes += (int64_t)p.rows * (p.cols > 0 ? p.cols : cols) * esz_;
     }
-    upload_matrix(m, rows, ld, bytes, out, group_rows, 0);
+    upload_matrix(m, rows, ld, bytes, out, group_rows, 0, share_per_token);
 }
 
 int MixerLm::rope_table(const RotarySpec& r) {
     for (size_t i = 0; i < rope_.size(); ++i)
-        if (rope_[i]->spec == r) return (int)i;
+        if (rope_[i]->spec.same_table(r)) return (int)i;
     auto t = std::make_unique<RopeTable>();
     t->spec = r;
     if (r.dims > 0) {
         // angles in f64, so that a far position is as exact as a near one
         const std::vector<double> freq = rotary_frequencies(r);
+        const double amplitude = rotary_amplitude(r);
         const int64_t positions = pool_->max_blocks() * pool_->block_tokens(), half = r.dims / 2;
         std::vector<float> c((size_t)(positions * half)), s((size_t)(positions * half));
 #pragma omp parallel for
         for (int64_t p = 0; p < positions; ++p)
             for (int64_t i = 0; i < half; ++i) {
                 const double a = (double)p * freq[(size_t)i];
-                c[(size_t)(p * half + i)] = (float)std::cos(a);
-                s[(size_t)(p * half + i)] = (float)std::sin(a);
+                c[(size_t)(p * half + i)] = (float)(amplitude * std::cos(a));
+                s[(size_t)(p * half + i)] = (float)(amplitude * std::sin(a));
             }
         upload_f32(c, t->cos_t);
         upload_f32(s, t->sin_t);
@@ -142,6 +144,7 @@ int MixerLm::geometry_of(const AttentionSpec& a) {
     Geometry g;
     g.heads = a.heads;
     g.kv_heads = a.kv_heads;
+    g.chunk = a.chunk;
     // the tensor-core kernels take rows of 64, 128 or 256; narrower heads are padded with zeros in the pools
     for (int d : {64, 128, 256})
         if (need <= d && !g.tc && attention_tc_supported(a.heads, a.kv_heads, d, cfg_.block_tokens, cfg_.kv_f16)) {
@@ -152,7 +155,7 @@ int MixerLm::geometry_of(const AttentionSpec& a) {
     if (g.row_width > 256) throw std::runtime_error("attention head dimensions above 256 are not supported");
     if (a.heads / a.kv_heads > 64) throw std::runtime_error("more than 64 query heads per key/value head are not supported");
     for (size_t i = 0; i < geo_.size(); ++i)
-        if (geo_[i].heads == g.heads && geo_[i].kv_heads == g.kv_heads && geo_[i].row_width == g.row_width) return (int)i;
+        if (geo_[i].heads == g.heads && geo_[i].kv_heads == g.kv_heads && geo_[i].row_width == g.row_width && geo_[i].chunk == g.chunk) return (int)i;
     geo_.push_back(std::move(g));
     return (int)geo_.size() - 1;
 }
@@ -189,6 +192,7 @@ void MixerLm::load(const SafetensorsFile& f) {
         upload_f32(f.values("loop.step", {ms_.loop.times, C}), loop_step_);
     }
     for (int l = 0; l < (int)ms_.layers.size(); ++l) {
+        if (ms_.layers[(size_t)l].weights_of >= 0) continue;
         passes_ = (int)std::count_if(runs_.begin(), runs_.end(), [&](const LayerRun& r) { return r.layer == l; });
         load_layer(f, l);
     }
@@ -200,7 +204,8 @@ void MixerLm::load(const SafetensorsFile& f) {
 void MixerLm::load_layer(const SafetensorsFile& f, int l) {
     const MixerLayerSpec& s = ms_.layers[(size_t)l];
     Layer& w = lw_[(size_t)l];
-    if (ms_.side_by_side) return load_side_by_side(f, l);
+    if (ms_.side_by_side()) return load_side_by_side(f, l);
+    if (ms_.norm_place == NormPlace::Output) return load_output_norm(f, l);
     const int C = ms_.width;
     const std::string p = "l" + std::to_string(l) + ".", m = p + "mix.";
     upload_norm(f, p + "norm1", w.norm1);
@@ -303,7 +308,7 @@ void MixerLm::alloc_run(int run) {
         pool.zero(stream_);
         spec_.kv_bytes_per_token += bytes / cfg_.block_tokens;
     };
-    if (s.kind == MixerKind::Wkv || ms_.side_by_side) st.kept.alloc(halves * (size_t)ms_.width * 4);  // the token shift's row
+    if (s.kind == MixerKind::Wkv || ms_.side_by_side()) st.kept.alloc(halves * (size_t)ms_.width * 4);  // the token shift's row
     switch (s.kind) {
         case MixerKind::Wkv:
             st.state.alloc(halves * (size_t)s.wkv.heads * s.wkv.dim * linear_state_key_pad(s.wkv.dim) * 4);
@@ -318,6 +323,14 @@ void MixerLm::alloc_run(int run) {
         }
         case MixerKind::Latent: pages(st.k_pool, 1); break;
         case MixerKind::MinGru: st.state.alloc(halves * (size_t)s.gru.width * 4); break;
+        case MixerKind::Mlstm:
+            st.state.alloc(halves * (size_t)s.mlstm.heads * (s.mlstm.vdim + 1) * linear_state_key_pad(s.mlstm.dim) * 4);
+            st.running_max.alloc(halves * (size_t)s.mlstm.heads * 4);
+            break;
+        case MixerKind::Attention:
+            pages(st.k_pool, s.attn.kv_heads);
+            pages(st.v_pool, s.attn.kv_heads);
+            break;
     }
 }
 
@@ -328,11 +341,30 @@ void MixerLm::alloc_activations() {
     int64_t q_lat = 0, uq = 0, lat = 0, cat = 0;  // widths of latent attention's rows, and of `out`'s input with both branches
     int lat_ctas = 1;
     int64_t lat_part = 0;
+    int64_t pairs = 0, experts = 0, expert_ff = 0, expert_gu = 0;  // routed rows, experts, widths of an expert's activations
     for (size_t l = 0; l < lw_.size(); ++l) {
         const MixerLayerSpec& s = ms_.layers[l];
         const Layer& w = lw_[l];
         in_rows = std::max(in_rows, w.in.rows);
-        if (ms_.side_by_side) {
+        if (s.ff > 0 && ms_.ff_kind == FfKind::Moe) {
+            pairs = std::max(pairs, T * s.moe.top);
+            experts = std::max(experts, (int64_t)s.moe.experts);
+            in_rows = std::max(in_rows, w.router.rows);
+            expert_ff = std::max(expert_ff, (int64_t)w.experts_down.ld);
+            expert_gu = std::max(expert_gu, w.experts_gu.rows / std::max(1, s.moe.experts));
+        }
+        if (s.kind == MixerKind::Mlstm) {
+            b_w = std::max(b_w, (int64_t)s.mlstm.heads * s.mlstm.vdim);
+            raw = std::max(raw, (int64_t)s.mlstm.heads * linear_state_raw_width(s.mlstm.vdim));
+        } else if (s.kind == MixerKind::Attention) {
+            a_w = std::max(a_w, (int64_t)s.attn.heads * s.attn.vdim);
+            attn = std::max(attn, (int64_t)s.attn.heads * w.row_width);
+        }
+        if (ms_.norm_place == NormPlace::Output) {
+            ff = std::max(ff, (int64_t)s.moe.shared_ff);
+            continue;
+        }
+        if (ms_.side_by_side()) {
             mix = 2;
             cat = std::max(cat, (int64_t)w.out.ld);
             if (s.kind == MixerKind::Latent) {
@@ -377,7 +409,20 @@ void MixerLm::alloc_activations() {
     y_in_.alloc((size_t)(T * std::max<int64_t>(in_rows, ms_.side_dim)) * 4);
     y_a_.alloc((size_t)(T * C) * 4);
     y_b_.alloc((size_t)(T * C) * 4);
-    if (f32_) y_gu_.alloc((size_t)(T * 2 * ff) * 4);
+    if (f32_) y_gu_.alloc((size_t)std::max(T * 2 * ff, pairs * expert_gu) * 4);
+    if (pairs > 0) {
+        img_rows_.alloc((size_t)(pairs * ldc) * esz_);
+        img_expert_ff_.alloc((size_t)(pairs * expert_ff) * esz_);
+        routed_.alloc((size_t)(pairs * C) * 4);
+        moe_words_.alloc((size_t)(5 * pairs + experts + 1 + T) * 4);
+        moe_.sel = moe_words_.as<int32_t>();
+        moe_.pos_of_pair = moe_.sel + pairs;
+        moe_.token_of_pos = moe_.pos_of_pair + pairs;
+        moe_.offsets = moe_.token_of_pos + pairs;
+        moe_.weight = reinterpret_cast<float*>(moe_.offsets + experts + 1);
+        moe_.weight_of_pos = moe_.weight + pairs;
+        moe_.shared_gate = moe_.weight_of_pos + pairs;
+    }
     decay_.alloc((size_t)(T * hd) * 4);
     raw_.alloc((size_t)(T * raw) * 4);
     q_rot_.alloc((size_t)(T * attn) * 4);
@@ -495,6 +540,11 @@ void MixerLm::apply_pending(RowUpdateArgs& a, Pending& p, bool other_buffer) {
         a.add_w[i] = p.w[i];
     }
     a.add_bias = p.bias;
+    if (p.routed_k > 0) {
+        a.routed = routed_.as<float>();
+        a.routed_at = p.routed_at;
+        a.routed_k = p.routed_k;
+    }
     a.add_coef = p.coef;
     a.add_eps = ms_.eps;
     if (p.n > 0) {
@@ -562,25 +612,12 @@ void MixerLm::run_wkv(const Tick& t, int run, Pending& pend) {
     pend.y[0] = matmul(w.out, img, T, y_a_, 1);
 }
 
-void MixerLm::run_parallel(const Tick& t, int run, Pending& pend, const std::vector<LmLane>& lanes) {
+void MixerLm::attend(const Tick& t, int run, const AttentionSpec& s, const Shares& y, const std::vector<LmLane>& lanes) {
     const int l = runs_[(size_t)run].layer;
     RunState& st = rs_[(size_t)run];
-    const AttentionSpec& s = ms_.layers[(size_t)l].attn;
-    const DeltaSpec& d = ms_.layers[(size_t)l].delta;
     Layer& w = lw_[(size_t)l];
-    const int T = t.T, C = ms_.width, D = w.row_width, bt = cfg_.block_tokens;
-    RowUpdateArgs u;
-    u.rows = T;
-    apply_pending(u, pend, false);
-    set_norm(u, w.norm1);
-    u.normed = image(img_h_, w.in.ld);
-    prof_begin(KC_ROW_UPDATE, (double)T * C * (8.0 + 4.0 * u.n_add + esz_), 0);
-    launch_row_update(u, stream_);
-    prof_end();
-    const Shares y = matmul(w.in, u.normed, T, y_in_, 0);
-    ++launches_;
-
-    // ---- attention: head norms, rotation, page write, softmax, head gate
+    const int T = t.T, D = w.row_width, bt = cfg_.block_tokens;
+    const bool whole = s.qk_norm == QkNorm::Whole;
     Geometry& g = geo_[(size_t)w.geometry];
     RopeKvArgs ra;
     ra.q = const_cast<float*>(y.p) + w.c_q;
@@ -594,6 +631,11 @@ void MixerLm::run_parallel(const Tick& t, int run, Pending& pend, const std::vec
     ra.q_norm_w = w.q_norm.as<float>();
     ra.k_norm_w = w.k_norm.as<float>();
     ra.norm_eps = ms_.eps;
+    if (s.biases) {
+        ra.q_bias = w.q_b.as<float>();
+        ra.k_bias = w.k_b.as<float>();
+        ra.v_bias = w.v_b.as<float>();
+    }
     if (s.rot.dims > 0) {
         ra.cos_t = rope_[(size_t)w.rope]->cos_t.as<float>();
         ra.sin_t = rope_[(size_t)w.rope]->sin_t.as<float>();
@@ -616,18 +658,22 @@ void MixerLm::run_parallel(const Tick& t, int run, Pending& pend, const std::vec
     ra.layer = 0;
     ra.pool_blocks = pool_->max_blocks();
     // ticks of one-token lanes: the attention kernel prepares its own rows
-    const bool fuse_rope = g.tc && g.plan.n_tiles() == 0 && g.plan.n_entries() > 0 && g.plan.n_dec_lanes() == 0;
+    const bool fuse_rope = !whole && g.tc && g.plan.n_tiles() == 0 && g.plan.n_entries() > 0 && g.plan.n_dec_lanes() == 0;
     const double kv_esz = cfg_.kv_f16 ? 2.0 : 4.0;
     if (!fuse_rope) {
         prof_begin(KC_ROPE_KV, (double)T * s.heads * (s.dim + D) * 4.0 + (double)T * s.kv_heads * (s.dim + s.vdim + 0.5 * kv_esz * D) * 4.0, 0);
-        launch_rope_kv(ra, stream_);
+        if (whole) launch_rope_kv_rows(ra, stream_);
+        else launch_rope_kv(ra, stream_);
         prof_end();
         ++launches_;
     }
     double kv_tokens = 0, flops = 0;
     for (const LmLane& ln : lanes) {
-        kv_tokens += (double)ln.start_pos + ln.n_tokens;
-        flops += 2.0 * s.heads * (s.dim + s.vdim) * ((double)ln.n_tokens * ln.start_pos + 0.5 * ln.n_tokens * ln.n_tokens);
+        const int lo = attention_first_key(ln.start_pos, 0, s.chunk);
+        kv_tokens += (double)ln.start_pos + ln.n_tokens - lo;
+        double pairs = (double)ln.n_tokens * (ln.start_pos - lo) + 0.5 * ln.n_tokens * ln.n_tokens;
+        if (s.chunk > 0) pairs = std::min(pairs, (double)ln.n_tokens * 0.5 * (s.chunk + 1));
+        flops += 2.0 * s.heads * (s.dim + s.vdim) * pairs;
     }
     prof_begin(KC_ATTN, kv_tokens * 2 * s.kv_heads * D * kv_esz + 8.0 * T * s.heads * D, flops);
     if (g.tc) {
@@ -655,6 +701,9 @@ void MixerLm::run_parallel(const Tick& t, int run, Pending& pend, const std::vec
         ta.layers = 1;
         ta.pool_blocks = ra.pool_blocks;
         ta.scale = s.scale;
+        ta.softcap = s.softcap;
+        ta.chunk = s.chunk;
+        ta.sink = s.sink ? w.sink.as<float>() : nullptr;
         ta.exact_weights = 1;
         if (fuse_rope) {
             ta.fused_rope = 1;
@@ -679,11 +728,36 @@ void MixerLm::run_parallel(const Tick& t, int run, Pending& pend, const std::vec
         at.layers = 1;
         at.pool_blocks = ra.pool_blocks;
         at.scale = s.scale;
+        at.softcap = s.softcap;
+        at.chunk = s.chunk;
+        at.sink = s.sink ? w.sink.as<float>() : nullptr;
         at.q_tile = attention_q_tile(s.heads, s.kv_heads);
         launch_paged_attention(at, stream_);
         ++launches_;
     }
     prof_end();
+}
+
+void MixerLm::run_parallel(const Tick& t, int run, Pending& pend, const std::vector<LmLane>& lanes) {
+    const int l = runs_[(size_t)run].layer;
+    RunState& st = rs_[(size_t)run];
+    const AttentionSpec& s = ms_.layers[(size_t)l].attn;
+    const DeltaSpec& d = ms_.layers[(size_t)l].delta;
+    Layer& w = lw_[(size_t)l];
+    const int T = t.T, C = ms_.width, D = w.row_width;
+    RowUpdateArgs u;
+    u.rows = T;
+    apply_pending(u, pend, false);
+    set_norm(u, w.norm1);
+    u.normed = image(img_h_, w.in.ld);
+    prof_begin(KC_ROW_UPDATE, (double)T * C * (8.0 + 4.0 * u.n_add + esz_), 0);
+    launch_row_update(u, stream_);
+    prof_end();
+    const Shares y = matmul(w.in, u.normed, T, y_in_, 0);
+    ++launches_;
+
+    // ---- attention: head norms, rotation, page write, softmax, head gate
+    attend(t, run, s, y, lanes);
     const RowImage img_a = image(img_a_, w.out.ld);
     prof_begin(KC_GATES, (double)T * s.heads * (D * 4.0 + s.vdim * (double)esz_), 0);
     launch_head_gate(attn_.as<float>(), T, s.heads, D, s.vdim, y, w.c_g, img_a, stream_);
@@ -779,7 +853,7 @@ void MixerLm::run_forward(const std::vector<LmLane>& lanes, KvReservation& r, ui
     }
     for (Geometry& g : geo_) {
         if (g.tc) {
-            plan_attention_tc(sp.data(), nt.data(), nb.data(), B, g.heads, g.kv_heads, g.plan);
+            plan_attention_tc(sp.data(), nt.data(), nb.data(), B, g.heads, g.kv_heads, g.plan, g.chunk);
             if (g.plan.n_entries() > attn_max_entries_) throw std::runtime_error("attention work list exceeds its scratch");
             g.off_entries = stage_bytes(t, g.plan.entries.data(), g.plan.entries.size() * 4);
             g.off_tiles = stage_bytes(t, g.plan.tiles.data(), g.plan.tiles.size() * 4);
@@ -834,7 +908,7 @@ void MixerLm::run_forward(const std::vector<LmLane>& lanes, KvReservation& r, ui
         if (ms_.loop.times > 0) e.image = image(img_loop_, loop_in_.ld).part(loop_in_.ld / 2, loop_in_.ld / 2);
         launch_embed_norm(e, stream_);
     } else {
-        launch_embed(table, t.ids, T, 1.f, x_[cur_].as<float>(), stream_);
+        launch_embed(table, t.ids, T, ms_.embedding_scale, x_[cur_].as<float>(), stream_);
     }
     prof_end();
     ++launches_;
@@ -847,10 +921,11 @@ void MixerLm::run_forward(const std::vector<LmLane>& lanes, KvReservation& r, ui
         const MixerLayerSpec& s = ms_.layers[(size_t)l];
         Layer& w = lw_[(size_t)l];
         if (runs_[(size_t)run].first) begin_pass(t, runs_[(size_t)run].pass, pend);
-        if (ms_.side_by_side) run_side_by_side(t, run, pend, lanes);
+        if (ms_.side_by_side()) run_side_by_side(t, run, pend, lanes);
+        else if (ms_.norm_place == NormPlace::Output) run_output_norm(t, run, pend, lanes);
         else if (s.kind == MixerKind::Wkv) run_wkv(t, run, pend);
         else run_parallel(t, run, pend, lanes);
-        if (s.ff > 0 && !ms_.side_by_side) {
+        if (s.ff > 0 && ms_.norm_place == NormPlace::Input) {
             RowUpdateArgs u;
             u.rows = T;
             apply_pending(u, pend, false);
@@ -870,7 +945,7 @@ void MixerLm::run_forward(const std::vector<LmLane>& lanes, KvReservation& r, ui
                 prof_begin(T <= 64 ? KC_GEMM_NARROW : KC_GEMM, (double)w.gate_up.bytes + 2.0 * T * C + 2.0 * T * s.ff, 2.0 * T * (double)w.gate_up.rows * w.gate_up.ld);
                 HgemmScratch ws;
                 ws.status = status_.as<int32_t>();
-                launch_hgemm_tc_gated(w.gate_up.half, reinterpret_cast<const __half*>(u.normed.h), T, 0, reinterpret_cast<__half*>(img.h), img.ld, ws, stream_);
+                launch_hgemm_tc_gated(w.gate_up.half, reinterpret_cast<const __half*>(u.normed.h), T, GatedAct{}, reinterpret_cast<__half*>(img.h), img.ld, ws, stream_);
                 prof_end();
             }
             launches_ += 2;
@@ -922,11 +997,12 @@ void MixerLm::run_forward(const std::vector<LmLane>& lanes, KvReservation& r, ui
         prof_begin(f32_ ? KC_F32_MATMUL : (R <= 64 ? KC_GEMM_NARROW : KC_GEMM), (double)head_.bytes + (double)esz_ * R * C + 4.0 * R * ms_.vocab,
                    2.0 * R * (double)ms_.vocab * C);
         if (f32_) {
-            launch_f32_matmul(head_.f32.as<float>(), head_.rows, head_.ld, u.normed.f, R, logits_.as<float>(), ms_.vocab, 1, nullptr, stream_, 0, ms_.logit_scale);
+            launch_f32_matmul(head_.f32.as<float>(), head_.rows, head_.ld, u.normed.f, R, logits_.as<float>(), ms_.vocab, 1, nullptr, stream_, 0, ms_.logit_scale, nullptr,
+                              ms_.logit_softcap);
         } else {
             HgemmScratch ws;
             ws.status = status_.as<int32_t>();
-            launch_hgemm_tc(head_.half, reinterpret_cast<const __half*>(u.normed.h), R, logits_.as<float>(), ms_.vocab, ms_.logit_scale, 0.f, ws, stream_, 1);
+            launch_hgemm_tc(head_.half, reinterpret_cast<const __half*>(u.normed.h), R, logits_.as<float>(), ms_.vocab, ms_.logit_scale, ms_.logit_softcap, ws, stream_, 1);
         }
         prof_end();
         ++launches_;
@@ -940,7 +1016,7 @@ void MixerLm::copy_state(int from, int to) {
     MK_CUDA(cudaSetDevice(cfg_.device));
     const size_t halves = (size_t)state_slots_->capacity() * 2;
     for (RunState& st : rs_)
-        for (DevBuf* b : {&st.state, &st.kept, &st.tail}) {
+        for (DevBuf* b : {&st.state, &st.kept, &st.tail, &st.running_max}) {
             if (b->size() == 0) continue;
             const size_t n = b->size() / halves;
             MK_CUDA(cudaMemcpyAsync(b->as<uint8_t>() + (size_t)to * n, b->as<uint8_t>() + (size_t)from * n, n, cudaMemcpyDeviceToDevice, stream_));

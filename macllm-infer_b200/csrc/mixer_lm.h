@@ -11,6 +11,7 @@
 #include "linear_state.h"
 #include "mixer_ops.h"
 #include "mixer_spec.h"
+#include "moe_rows.h"
 
 namespace mk {
 
@@ -81,15 +82,23 @@ private:
         // feed-forward beside the mixer
         int c_ff = 0;
         DevBuf up_b, down_b, poly;
+        // biases of the attention projections, a denominator term per head
+        DevBuf q_b, k_b, v_b, o_b, sink;
+        // mLSTM (columns c_q, c_k, c_v, c_g and these)
+        int c_i = 0, c_f = 0;
+        DevBuf i_b, f_b;
+        // mixture of experts: router rows (the shared expert's gate behind them), gate/up and down matrices of all experts; the
+        // shared expert's are gate_up and down
+        Dense router, experts_gu, experts_down;
     };
     // What one execution of a layer keeps between forwards: pages, and the two halves of every state slot.
     struct RunState {
         DevBuf k_pool, v_pool;  // latent attention: k_pool only
-        DevBuf state, kept, tail;
+        DevBuf state, kept, tail, running_max;
     };
     // Layers with the same heads share a tick's attention work list.
     struct Geometry {
-        int heads = 0, kv_heads = 0, row_width = 0;
+        int heads = 0, kv_heads = 0, row_width = 0, chunk = 0;
         bool tc = false;
         AttnTcPlan plan;
         size_t off_tiles = 0, off_entries = 0, off_dec = 0;
@@ -116,18 +125,21 @@ private:
         DevBuf cos_t, sin_t;
     };
     enum KClass { KC_GEMM = 0, KC_GEMM_NARROW, KC_F32_MATMUL, KC_WKV_SCAN, KC_DELTA_SCAN, KC_ATTN, KC_ROPE_KV, KC_ROW_UPDATE, KC_DELTA_PREP, KC_WKV_DECAY,
-                  KC_LATENT_ATTN, KC_MINGRU, KC_LATENT_PREP, KC_LATENT_ROWS, KC_GATES, KC_EMBED, KC_BATCH, KC_SAMPLE, KC_COUNT };
+                  KC_LATENT_ATTN, KC_MINGRU, KC_LATENT_PREP, KC_LATENT_ROWS, KC_MLSTM_SCAN, KC_MOE_GEMM, KC_MOE_ROWS, KC_GATES, KC_EMBED, KC_BATCH,
+                  KC_SAMPLE, KC_COUNT };
 
     void load(const SafetensorsFile& f);
     void load_layer(const SafetensorsFile& f, int l);
     void load_latent(const SafetensorsFile& f, int l);
     void load_side_by_side(const SafetensorsFile& f, int l);
+    void load_output_norm(const SafetensorsFile& f, int l);
+    void load_moe(const SafetensorsFile& f, int l);
     void alloc_run(int run);
     void upload_dense(const SafetensorsFile& f, const std::vector<Part>& parts, int64_t rows, int cols, Dense& out,
-                      const std::vector<int64_t>& group_rows = {});
-    // `groups` > 0: equal parts with an input each.  per_token: counted in the bytes of a token's pass.
+                      const std::vector<int64_t>& group_rows = {}, double share_per_token = 1.0);
+    // `groups` > 0: equal parts with an input each.  share_per_token: how much of it a token's pass reads.
     void upload_matrix(const std::vector<float>& m, int64_t rows, int ld, int64_t true_bytes, Dense& out, const std::vector<int64_t>& group_rows, int groups,
-                       bool per_token = true);
+                       double share_per_token = 1.0);
     int passes_ = 1;  // how often a token's pass runs what is being loaded
     void place(const SafetensorsFile& f, const Part& p, int cols, int ld, std::vector<float>& m);
     void upload_f32(const std::vector<float>& v, DevBuf& out);
@@ -148,15 +160,23 @@ private:
         Shares y[2];
         const float* w[2] = {nullptr, nullptr};
         const float* bias = nullptr;  // of a single branch
+        const int32_t* routed_at = nullptr;  // of a single branch: rows of routed_ to add (see RowUpdateArgs)
+        int routed_k = 0;
         float coef = 1.f;
         bool replace = false;         // they take the stream's place
     };
     void apply_pending(RowUpdateArgs& a, Pending& p, bool other_buffer);
     void run_wkv(const Tick& t, int run, Pending& p);
     void run_parallel(const Tick& t, int run, Pending& p, const std::vector<LmLane>& lanes);
+    // Queries, keys and values out of the projections `y`, page write and attention: leaves the heads' outputs in attn_.
+    void attend(const Tick& t, int run, const AttentionSpec& s, const Shares& y, const std::vector<LmLane>& lanes);
     // layers whose mixer and feed-forward read one norm
     void begin_pass(const Tick& t, int pass, Pending& p);
     void run_side_by_side(const Tick& t, int run, Pending& p, const std::vector<LmLane>& lanes);
+    // layers whose norms sit on what the sublayers give
+    void run_output_norm(const Tick& t, int run, Pending& p, const std::vector<LmLane>& lanes);
+    void run_mlstm(const Tick& t, int run, const Shares& y, const RowImage& out);
+    void run_moe(const Tick& t, int layer, Pending& p);
     void run_latent(const Tick& t, int run, const Shares& y, const RowImage& out, const std::vector<LmLane>& lanes);
     void run_latent_wide(const Tick& t, int run, const Shares& y, const RowImage& out);
 
@@ -183,6 +203,9 @@ private:
     DevBuf img_loop_, img_q_, img_uq_, q_lat_, img_lat_, img_cat_, wide_in_, wide_kv_;
     DevBuf lat_part_o_, lat_part_ml_, lat_counters_;
     DevBuf partial_[3];
+    // mixture of experts: the tick's routing, rows grouped by expert, their activations and results
+    MoeRows moe_;
+    DevBuf moe_words_, img_rows_, img_expert_ff_, routed_;
     DevBuf attn_part_o_, attn_part_ml_, attn_counters_;
     int attn_max_entries_ = 0;
     int cur_ = 0;             // which of x_ holds the residual stream

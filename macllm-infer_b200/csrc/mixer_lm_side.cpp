@@ -139,7 +139,7 @@ void MixerLm::load_latent(const SafetensorsFile& f, int l) {
         std::vector<float> t((size_t)(rows * w.row_width), 0.f);
         place(f, {m + "uk", H * a.dim, 0, 1, 0, a.kv_rank, a.dim, w.q_width}, a.kv_rank, w.row_width, t);
         place(f, {m + "uv", H * a.vdim, H * w.q_width, 1, 0, a.kv_rank, a.vdim, w.q_width}, a.kv_rank, w.row_width, t);
-        upload_matrix(t, rows, w.row_width, uk_bytes + uv_bytes, w.ukv, {}, 0, false);
+        upload_matrix(t, rows, w.row_width, uk_bytes + uv_bytes, w.ukv, {}, 0, 0.0);
     }
 }
 

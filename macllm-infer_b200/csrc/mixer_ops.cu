@@ -53,6 +53,29 @@ __device__ __forceinline__ void zero_tail(const RowImage& im, int64_t row, int w
     for (int c = width + threadIdx.x; c < im.end(); c += blockDim.x) im.put(row, c, 0.f);
 }
 
+// VEC values of branch b of a row: the matmul's, the chosen experts' and the bias.
+template <int VEC>
+__device__ __forceinline__ Pack<VEC> branch_pack(const RowUpdateArgs& a, int b, int64_t row, int c) {
+    Pack<VEC> y;
+    if (a.add[b].p != nullptr) {
+        y = share_pack<VEC>(a.add[b], row, c);
+    } else {
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) y.v[i] = 0.f;
+    }
+    for (int j = 0; j < a.routed_k; ++j) {
+        const Pack<VEC> e = load_pack<VEC>(a.routed + (int64_t)a.routed_at[row * a.routed_k + j] * a.width + c);
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) y.v[i] += e.v[i];
+    }
+    if (a.add_bias != nullptr) {
+        const Pack<VEC> e = load_pack<VEC>(a.add_bias + c);
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) y.v[i] += e.v[i];
+    }
+    return y;
+}
+
 // The updated row into `dst` (shared memory): x + coef * (branches + bias).  Normed branches are staged in `dst` / `other` first.
 template <int VEC>
 __device__ __forceinline__ void updated_row(const RowUpdateArgs& a, int64_t row, float* dst, float* other, float* red) {
@@ -64,7 +87,7 @@ __device__ __forceinline__ void updated_row(const RowUpdateArgs& a, int64_t row,
             float* st = b == 0 ? dst : other;
             float ss = 0.f;
             for (int c = threadIdx.x * VEC; c < a.width; c += step) {
-                const Pack<VEC> y = share_pack<VEC>(a.add[b], row, c);
+                const Pack<VEC> y = branch_pack<VEC>(a, b, row, c);
                 store_pack<VEC>(st + c, y);
 #pragma unroll
                 for (int i = 0; i < VEC; ++i) ss = fmaf(y.v[i], y.v[i], ss);
@@ -93,12 +116,7 @@ __device__ __forceinline__ void updated_row(const RowUpdateArgs& a, int64_t row,
 #pragma unroll
             for (int i = 0; i < VEC; ++i) v.v[i] = fmaf(a.add_coef, sum.v[i], v.v[i]);
         } else if (a.n_add > 0) {
-            Pack<VEC> y = share_pack<VEC>(a.add[0], row, c);
-            if (a.add_bias != nullptr) {
-                const Pack<VEC> b = load_pack<VEC>(a.add_bias + c);
-#pragma unroll
-                for (int i = 0; i < VEC; ++i) y.v[i] += b.v[i];
-            }
+            const Pack<VEC> y = branch_pack<VEC>(a, 0, row, c);
 #pragma unroll
             for (int i = 0; i < VEC; ++i) v.v[i] = fmaf(a.add_coef, y.v[i], v.v[i]);
         }
@@ -106,21 +124,23 @@ __device__ __forceinline__ void updated_row(const RowUpdateArgs& a, int64_t row,
     }
 }
 
-// Mean and root of (variance + eps) of a staged row, for the layer norm.
+// Mean and root of (variance + eps) of a staged row, for the layer norm; root of (mean square + eps) for the RMS norm.
 struct RowStats {
     float mean = 0.f, root = 1.f;
 };
 template <int VEC>
-__device__ __forceinline__ RowStats row_stats(const float* x, int width, float eps, float* red) {
+__device__ __forceinline__ RowStats row_stats(const float* x, int width, float eps, float* red, bool centred = true) {
     const int step = RU_THREADS * VEC;
     float s = 0.f;
-    for (int c = threadIdx.x * VEC; c < width; c += step) {
-        const Pack<VEC> v = load_pack<VEC>(x + c);
-#pragma unroll
-        for (int i = 0; i < VEC; ++i) s += v.v[i];
-    }
     RowStats r;
-    r.mean = block_sum(s, red) / (float)width;
+    if (centred) {
+        for (int c = threadIdx.x * VEC; c < width; c += step) {
+            const Pack<VEC> v = load_pack<VEC>(x + c);
+#pragma unroll
+            for (int i = 0; i < VEC; ++i) s += v.v[i];
+        }
+        r.mean = block_sum(s, red) / (float)width;
+    }
     s = 0.f;
     for (int c = threadIdx.x * VEC; c < width; c += step) {
         const Pack<VEC> v = load_pack<VEC>(x + c);
@@ -135,7 +155,7 @@ template <int VEC>
 __device__ __forceinline__ Pack<VEC> norm_pack(const RowUpdateArgs& a, const RowStats& st, const Pack<VEC>& x, int c) {
     Pack<VEC> h;
     const Pack<VEC> w = load_pack<VEC>(a.norm_w + c);
-    if (a.norm == NormKind::Layer) {
+    if (a.norm != NormKind::DynTanh) {
 #pragma unroll
         for (int i = 0; i < VEC; ++i) h.v[i] = (x.v[i] - st.mean) / st.root * w.v[i];
     } else {
@@ -169,7 +189,8 @@ __global__ void __launch_bounds__(RU_THREADS) row_update_kernel(RowUpdateArgs a)
     if (a.norm == NormKind::None) return;
     // a thread has written the columns of `cur` that it reads itself; block_sum's barriers are all the sums need
     RowStats st, st_prev;
-    if (a.norm == NormKind::Layer) st = row_stats<VEC>(cur, a.width, a.norm_eps, red);
+    const bool stats = a.norm != NormKind::DynTanh, centred = a.norm == NormKind::Layer;
+    if (stats) st = row_stats<VEC>(cur, a.width, a.norm_eps, red, centred);
     if (a.n_mix == 0) {
         for (int c = threadIdx.x * VEC; c < a.width; c += step) put_pack<VEC>(a.normed, r, c, norm_pack<VEC>(a, st, load_pack<VEC>(cur + c), c));
         zero_tail(a.normed, r, a.width);
@@ -181,7 +202,7 @@ __global__ void __launch_bounds__(RU_THREADS) row_update_kernel(RowUpdateArgs a)
     const bool inside = row > first;
     if (inside) {
         updated_row<VEC>(a, row - 1, prv, other, red);
-        if (a.norm == NormKind::Layer) st_prev = row_stats<VEC>(prv, a.width, a.norm_eps, red);
+        if (stats) st_prev = row_stats<VEC>(prv, a.width, a.norm_eps, red, centred);
     }
     for (int c = threadIdx.x * VEC; c < a.width; c += step) {
         const Pack<VEC> h = norm_pack<VEC>(a, st, load_pack<VEC>(cur + c), c);
@@ -359,12 +380,12 @@ __global__ void __launch_bounds__(DP_WARPS * 32) delta_prep_kernel(DeltaPrepArgs
 // ------------------------------------------------------------------------------------------------ gates
 
 __global__ void __launch_bounds__(256) head_gate_kernel(const float* attn, int heads, int row_width, int vdim, Shares gate, int gate_col, RowImage out,
-                                                        const int32_t* rows) {
+                                                        const int32_t* rows, OutputGate kind, int vec_gate) {
     extern __shared__ float hg_gate[];
     pdl_trigger();
     pdl_wait();
     const int64_t row = rows != nullptr ? rows[blockIdx.x] : blockIdx.x;
-    for (int h = threadIdx.x; h < heads; h += blockDim.x) hg_gate[h] = sigmoid_f(gate.at(row, gate_col + h));
+    for (int h = threadIdx.x; h < heads; h += blockDim.x) hg_gate[h] = kind == OutputGate::Head ? sigmoid_f(gate.at(row, gate_col + h)) : 1.f;
     __syncthreads();
     const float* src = attn + row * heads * row_width;
     if ((vdim & 3) == 0) {  // out.end() is a multiple of 64, a head's row of 4
@@ -373,8 +394,15 @@ __global__ void __launch_bounds__(256) head_gate_kernel(const float* attn, int h
             float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
             if (h < heads) {
                 v = *reinterpret_cast<const float4*>(src + h * row_width + (c - h * vdim));
-                const float g = hg_gate[h];
-                v = make_float4(v.x * g, v.y * g, v.z * g, v.w * g);
+                if (kind == OutputGate::Value) {
+                    float4 g;
+                    if (vec_gate) g = gate.at4(row, gate_col + c);
+                    else g = make_float4(gate.at(row, gate_col + c), gate.at(row, gate_col + c + 1), gate.at(row, gate_col + c + 2), gate.at(row, gate_col + c + 3));
+                    v = make_float4(v.x * sigmoid_f(g.x), v.y * sigmoid_f(g.y), v.z * sigmoid_f(g.z), v.w * sigmoid_f(g.w));
+                } else {
+                    const float g = hg_gate[h];
+                    v = make_float4(v.x * g, v.y * g, v.z * g, v.w * g);
+                }
             }
             out.put4(row, c, v);
         }
@@ -382,7 +410,9 @@ __global__ void __launch_bounds__(256) head_gate_kernel(const float* attn, int h
     }
     for (int c = threadIdx.x; c < out.end(); c += blockDim.x) {
         const int h = c / vdim;
-        out.put(row, c, h < heads ? src[h * row_width + (c - h * vdim)] * hg_gate[h] : 0.f);
+        float v = 0.f;
+        if (h < heads) v = src[h * row_width + (c - h * vdim)] * (kind == OutputGate::Value ? sigmoid_f(gate.at(row, gate_col + c)) : hg_gate[h]);
+        out.put(row, c, v);
     }
 }
 
@@ -402,11 +432,19 @@ __global__ void __launch_bounds__(128) side_gate_kernel(Shares z, int dim, const
     }
 }
 
-__global__ void __launch_bounds__(256) gated_act_kernel(Shares gu, int ff, RowImage out) {
+__global__ void __launch_bounds__(256) gated_act_kernel(Shares gu, int ff, RowImage out, GatedAct act) {
     pdl_trigger();
     pdl_wait();
     const int64_t row = blockIdx.x;
-    for (int c = threadIdx.x; c < out.end(); c += blockDim.x) out.put(row, c, c < ff ? silu_f(gu.at(row, 2 * c)) * gu.at(row, 2 * c + 1) : 0.f);
+    const float pre = act.pre != nullptr ? act.pre[row] : 1.f, post = act.post != nullptr ? act.post[row] : 1.f;
+    for (int c = threadIdx.x; c < out.end(); c += blockDim.x) {
+        float v = 0.f;
+        if (c < ff) {
+            const float g = gu.at(row, 2 * c), u = gu.at(row, 2 * c + 1);
+            v = act.kind == GatedAct::Clamped ? clamped_gate_f(pre * g, pre * u, act.limit) * post : (act.kind == GatedAct::Silu ? silu_f(g) : gelu_tanh_f(g)) * u;
+        }
+        out.put(row, c, v);
+    }
 }
 
 // ------------------------------------------------------------------------------------------------ embedding with positions
@@ -538,13 +576,21 @@ constexpr int FM_TILE = 64, FM_K = 16;
 
 // 64 x 64 outputs per CTA, 4 x 4 per thread.
 __global__ void __launch_bounds__(256) f32_matmul_kernel(const float* __restrict__ w, int64_t rows, int cols, const float* __restrict__ x, int T, float* y,
-                                                         int ldy, float scale, int n_groups, int group_tiles, int4 end_lo, int4 end_hi,
-                                                         MatmulScatter to) {
+                                                         int ldy, float scale, float softcap, int n_groups, int group_tiles, int4 end_lo, int4 end_hi,
+                                                         MatmulScatter to, const int32_t* __restrict__ offsets, int64_t matrix_rows) {
     __shared__ float ws[FM_K][FM_TILE + 4], xs[FM_K][FM_TILE + 4];
     pdl_trigger();
     pdl_wait();
     const int64_t n0 = (int64_t)blockIdx.x * FM_TILE;
     const int t0 = blockIdx.y * FM_TILE;
+    if (offsets != nullptr) {  // rows grouped by expert: matrix blockIdx.z
+        const int e = blockIdx.z, first = offsets[e];
+        T = offsets[e + 1] - first;
+        if (t0 >= T) return;
+        w += e * matrix_rows * cols;
+        x += (int64_t)first * cols;
+        y += (int64_t)first * ldy;
+    }
     const int ends[kMaxRowGroups] = {end_lo.x, end_lo.y, end_lo.z, end_lo.w, end_hi.x, end_hi.y, end_hi.z, end_hi.w};
     int g = 0;
     if (group_tiles > 0) g = (int)(n0 / 128 / group_tiles);
@@ -583,7 +629,8 @@ __global__ void __launch_bounds__(256) f32_matmul_kernel(const float* __restrict
             const int64_t n = n0 + tx * 4 + j;
             if (t >= T || n >= rows) continue;
             if (to.out == nullptr) {
-                y[(int64_t)t * ldy + n] = acc[i][j] * scale;
+                const float v = acc[i][j] * scale;
+                y[(int64_t)t * ldy + n] = softcap != 0.f ? softcap * tanhf(v / softcap) : v;
                 continue;
             }
             const int64_t col = to.column(n);
@@ -596,7 +643,8 @@ __global__ void __launch_bounds__(256) f32_matmul_kernel(const float* __restrict
 void launch_row_update(const RowUpdateArgs& a, cudaStream_t s) {
     if (a.rows <= 0) return;
     if (a.n_mix > 0 && (a.x == a.x_out || a.row_index != nullptr)) throw std::runtime_error("launch_row_update: a token shift needs its own output buffer and packed rows");
-    if (a.add_bias != nullptr && (a.n_add != 1 || a.add_w[0] != nullptr)) throw std::runtime_error("launch_row_update: a bias goes with one plain branch");
+    if (a.add_bias != nullptr && a.n_add != 1) throw std::runtime_error("launch_row_update: a bias goes with one branch");
+    if (a.routed_k > 0 && (a.n_add != 1 || a.add_w[0] == nullptr || a.routed == nullptr)) throw std::runtime_error("launch_row_update: experts' rows go with one normed branch");
     if (a.n_add == 2 && (a.add_w[0] == nullptr || a.add_w[1] == nullptr)) throw std::runtime_error("launch_row_update: two branches are both normed");
     bool vec = a.width % 4 == 0;
     for (int b = 0; b < a.n_add; ++b)
@@ -632,9 +680,10 @@ void launch_delta_prep(const DeltaPrepArgs& a, cudaStream_t s) {
 }
 
 void launch_head_gate(const float* attn, int rows, int heads, int row_width, int vdim, const Shares& gate, int gate_col, const RowImage& out,
-                      cudaStream_t s, const int32_t* row_list) {
+                      cudaStream_t s, const int32_t* row_list, OutputGate kind) {
     if (rows <= 0) return;
-    launch_pdl(head_gate_kernel, dim3((unsigned)rows), dim3(256), (size_t)heads * 4, s, attn, heads, row_width, vdim, gate, gate_col, out, row_list);
+    const int vec_gate = gate_col % 4 == 0 && gate.ld % 4 == 0 && gate.stride % 4 == 0 && (reinterpret_cast<uintptr_t>(gate.p) & 15) == 0 ? 1 : 0;
+    launch_pdl(head_gate_kernel, dim3((unsigned)rows), dim3(256), (size_t)heads * 4, s, attn, heads, row_width, vdim, gate, gate_col, out, row_list, kind, vec_gate);
     MK_LAUNCH_CHECK();
 }
 
@@ -645,9 +694,9 @@ void launch_side_gate(const Shares& z, int rows, int dim, const uint32_t* ids, c
     MK_LAUNCH_CHECK();
 }
 
-void launch_gated_act(const Shares& gu, int rows, int ff, const RowImage& out, cudaStream_t s) {
+void launch_gated_act(const Shares& gu, int rows, int ff, const RowImage& out, cudaStream_t s, const GatedAct& act) {
     if (rows <= 0) return;
-    launch_pdl(gated_act_kernel, dim3((unsigned)rows), dim3(256), 0, s, gu, ff, out);
+    launch_pdl(gated_act_kernel, dim3((unsigned)rows), dim3(256), 0, s, gu, ff, out, act);
     MK_LAUNCH_CHECK();
 }
 
@@ -673,13 +722,21 @@ void launch_latent_prep(const LatentPrepArgs& a, cudaStream_t s) {
 }
 
 void launch_f32_matmul(const float* w, int64_t rows, int cols, const float* x, int T, float* y, int ldy, int n_groups, const int* group_end,
-                       cudaStream_t s, int group_tiles, float scale, const MatmulScatter* to) {
+                       cudaStream_t s, int group_tiles, float scale, const MatmulScatter* to, float softcap) {
     if (T <= 0) return;
     int e[kMaxRowGroups] = {};
     for (int g = 0; g < n_groups && n_groups > 1 && group_tiles == 0; ++g) e[g] = group_end[g];
     const dim3 grid((unsigned)((rows + FM_TILE - 1) / FM_TILE), (unsigned)((T + FM_TILE - 1) / FM_TILE));
-    launch_pdl(f32_matmul_kernel, grid, dim3(256), 0, s, w, rows, cols, x, T, y, ldy, scale, n_groups, group_tiles, make_int4(e[0], e[1], e[2], e[3]),
-               make_int4(e[4], e[5], e[6], e[7]), to != nullptr ? *to : MatmulScatter{});
+    launch_pdl(f32_matmul_kernel, grid, dim3(256), 0, s, w, rows, cols, x, T, y, ldy, scale, softcap, n_groups, group_tiles, make_int4(e[0], e[1], e[2], e[3]),
+               make_int4(e[4], e[5], e[6], e[7]), to != nullptr ? *to : MatmulScatter{}, nullptr, (int64_t)0);
+    MK_LAUNCH_CHECK();
+}
+
+void launch_f32_matmul_experts(const float* w, int experts, const int32_t* offsets, int64_t rows, int64_t matrix_rows, int cols, const float* x, int T, float* y,
+                               int ldy, cudaStream_t s) {
+    if (T <= 0) return;
+    const dim3 grid((unsigned)((rows + FM_TILE - 1) / FM_TILE), (unsigned)((T + FM_TILE - 1) / FM_TILE), (unsigned)experts);
+    launch_pdl(f32_matmul_kernel, grid, dim3(256), 0, s, w, rows, cols, x, T, y, ldy, 1.f, 0.f, 1, 0, int4{}, int4{}, MatmulScatter{}, offsets, matrix_rows);
     MK_LAUNCH_CHECK();
 }
 

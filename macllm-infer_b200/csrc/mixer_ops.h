@@ -10,7 +10,8 @@ namespace mk {
 
 // One CTA per row r (x row = row_index ? row_index[r] : r):
 //   x_out = x + coef * sum over branches b of (add_w[b] ? rms(add[b]) * add_w[b] : add[b])      (n_add branches; x = 0 when null)
-//   (a single plain branch may carry a bias [width])
+//   (a single branch may carry a bias [width], added before its norm; a single normed branch also the rows of the experts a token
+//    chose, added up before its norm - its own matrix may then be missing)
 //   raw    <- x_out                        (optional image)
 //   h       = norm(x_out);  normed <- h    (optional image, n_mix = 0)
 //   mixes[i] <- h + (h' - h) * mu[i]       (n_mix images of `rows` rows each, one after the other), h' = h of the sequence's
@@ -26,11 +27,14 @@ struct RowUpdateArgs {
     Shares add[2];
     const float* add_w[2] = {nullptr, nullptr};
     const float* add_bias = nullptr;
+    const float* routed = nullptr;       // [rows of all experts][width]
+    const int32_t* routed_at = nullptr;  // [token][routed_k]: where a token's rows are
+    int routed_k = 0;
     float add_coef = 1.f, add_eps = 0.f;
     RowImage raw;
     NormKind norm = NormKind::None;
     float alpha = 1.f;          // DynTanh
-    float norm_eps = 0.f;       // Layer
+    float norm_eps = 0.f;       // Layer, Rms
     const float* norm_w = nullptr;
     const float* norm_b = nullptr;  // DynTanh
     RowImage normed;
@@ -64,21 +68,26 @@ struct DeltaPrepArgs {
 void launch_delta_prep(const DeltaPrepArgs& a, cudaStream_t s);
 
 // out[t][h * vdim + i] = attn[t][h * row_width + i] * sigmoid(gate[t][gate_col + h]), t = row_list[0 .. rows) or 0 .. rows - 1
+// (OutputGate::Value: sigmoid(gate[t][gate_col + h * vdim + i]); None: no factor)
 void launch_head_gate(const float* attn, int rows, int heads, int row_width, int vdim, const Shares& gate, int gate_col, const RowImage& out,
-                      cudaStream_t s, const int32_t* row_list = nullptr);
+                      cudaStream_t s, const int32_t* row_list = nullptr, OutputGate kind = OutputGate::Head);
 
 // out[t][j] = gelu_tanh(z[t][j]) * table[ids[t]][slice + j], j < dim; table [vocab][table_ld] as bfloat16 bits (or f32)
 void launch_side_gate(const Shares& z, int rows, int dim, const uint32_t* ids, const void* table, int table_f32, int64_t table_ld, int slice,
                       const RowImage& out, cudaStream_t s);
 
-// out[t][j] = silu(gu[t][2j]) * gu[t][2j + 1], j < ff: gate and up rows interleaved
-void launch_gated_act(const Shares& gu, int rows, int ff, const RowImage& out, cudaStream_t s);
+// out[t][j] = act(gu[t][2j], gu[t][2j + 1]), j < ff: gate and up rows interleaved
+void launch_gated_act(const Shares& gu, int rows, int ff, const RowImage& out, cudaStream_t s, const GatedAct& act = {});
 
 // y[t][n] = sum_k x[t][k] w[n][k] in f32, k ascending.  x is [n_groups][T][cols]; weight row n reads input g of its group, whose
 // rows end at 128 * group_end[g], or are 128 * group_tiles each (see HalfWeight).  `to` scatters the result instead (see
-// MatmulScatter).
+// MatmulScatter).  The result is multiplied by `scale` and, with a soft cap c, becomes c * tanh(y / c).
 void launch_f32_matmul(const float* w, int64_t rows, int cols, const float* x, int T, float* y, int ldy, int n_groups, const int* group_end,
-                       cudaStream_t s, int group_tiles = 0, float scale = 1.f, const MatmulScatter* to = nullptr);
+                       cudaStream_t s, int group_tiles = 0, float scale = 1.f, const MatmulScatter* to = nullptr, float softcap = 0.f);
+// The same over rows grouped by expert: rows [offsets[e], offsets[e + 1]) of x and y meet matrix e of `experts`, rows x cols each,
+// matrix_rows apart.  T: rows of all experts.
+void launch_f32_matmul_experts(const float* w, int experts, const int32_t* offsets, int64_t rows, int64_t matrix_rows, int cols, const float* x, int T, float* y,
+                               int ldy, cudaStream_t s);
 
 // The embedding output of models with sinusoidal positions:  e = table[ids[t]] + sinusoid(positions[t]);  x = layer norm of e, in
 // f32 to x [rows][width] and as a matmul input to `image` (optional).  freq[i] is the frequency of column pair i in f64: the angle

@@ -1,5 +1,6 @@
 // See mixer_spec.h.
 #include "mixer_spec.h"
+#include <algorithm>
 #include <cmath>
 #include <fstream>
 #include <map>
@@ -21,8 +22,9 @@ int size_of(const Json& v, int lo = 1, int hi = 1 << 24) {
     return (int)n;
 }
 
-RotarySpec read_rotary(const Json& mixer, int head_dim) {
+RotarySpec read_rotary(const Json& mixer, int head_dim, RotaryScaling scaling = RotaryScaling::Turns, bool interleaved = true) {
     RotarySpec r;
+    r.interleaved = interleaved;
     const Json* rot = mixer.find("rot");
     if (rot == nullptr || rot->is_null()) return r;
     r.dims = size_of(rot->at("dims"), 0, head_dim);
@@ -31,12 +33,14 @@ RotarySpec read_rotary(const Json& mixer, int head_dim) {
     if (!(r.base > 0)) throw std::runtime_error(rot->where() + ".base must be positive");
     const Json* s = rot->find("scaling");
     if (s != nullptr && !s->is_null()) {
-        r.scaled = true;
+        if (scaling == RotaryScaling::None) throw std::runtime_error(s->where() + " is not supported here");
+        r.scaling = scaling;
         r.factor = s->at("factor").number();
-        r.low = s->at("low").number();
-        r.high = s->at("high").number();
+        r.low = s->at(scaling == RotaryScaling::Yarn ? "slow" : "low").number();
+        r.high = s->at(scaling == RotaryScaling::Yarn ? "fast" : "high").number();
         r.original = s->at("original").number();
         if (!(r.factor > 0 && r.original > 0)) throw std::runtime_error(s->where() + " needs a positive factor and original context");
+        if (scaling == RotaryScaling::Yarn && !(r.low > 0 && r.high > 0 && r.base != 1.0)) throw std::runtime_error(s->where() + " needs positive turns");
     }
     return r;
 }
@@ -123,7 +127,7 @@ MixerSpec read_kunonex(const Json& c, const SafetensorsFile&) {
     s.width = size_of(c.at("width"));
     s.norm = NormKind::Layer;
     s.ff_kind = FfKind::Poly;
-    s.side_by_side = true;
+    s.norm_place = NormPlace::Shared;
     s.sinusoid_positions = true;
     s.eps = number_of(c.at("norm").at("eps"));
     if (!(s.eps >= 0.f)) throw std::runtime_error("config norm.eps must not be negative");
@@ -161,6 +165,107 @@ MixerSpec read_kunonex(const Json& c, const SafetensorsFile&) {
 }
 
 const RegisterMixerArchitecture register_kunonex("Kunonex", read_kunonex);
+
+MoeSpec read_moe(const Json& mlp) {
+    if (mlp.at("kind").str() != "moe") throw std::runtime_error(mlp.where() + ".kind `" + mlp.at("kind").str() + "` is not supported");
+    auto limit = [](const Json& j) {
+        const float v = number_of(j.at("limit"));
+        if (!(v >= 0.f)) throw std::runtime_error(j.where() + ".limit must not be negative");
+        return v;
+    };
+    MoeSpec m;
+    const Json &r = mlp.at("router"), &e = mlp.at("expert");
+    m.experts = size_of(r.at("experts"), 1, 1024);
+    m.top = size_of(r.at("top"), 1, std::min(m.experts, 32));
+    m.ff = size_of(e.at("ff"));
+    m.limit = limit(e);
+    const Json* sh = mlp.find("shared");
+    if (sh != nullptr && !sh->is_null()) {
+        m.shared_ff = size_of(sh->at("ff"));
+        m.shared_limit = limit(*sh);
+    }
+    return m;
+}
+
+// Tevanex: mLSTM layers and two kinds of chunked attention over a mixture of experts, norms on what the sublayers give, layers that
+// run another layer's tensors again.
+MixerSpec read_tevanex(const Json& c, const SafetensorsFile&) {
+    MixerSpec s;
+    s.arch = "Tevanex";
+    s.vocab = size_of(c.at("vocab"));
+    s.width = size_of(c.at("width"));
+    s.norm = NormKind::Rms;
+    s.norm_place = NormPlace::Output;
+    s.ff_kind = FfKind::Moe;
+    s.eps = number_of(c.at("norm").at("eps"));
+    if (!(s.eps >= 0.f)) throw std::runtime_error("config norm.eps must not be negative");
+    s.embedding_scale = number_of(c.at("embedding").at("scale"));
+    s.residual_mult = number_of(c.at("residual_mult"));
+    s.logit_scale = number_of(c.at("logit_scale"));
+    s.logit_softcap = number_of(c.at("logit_softcap"));
+    if (!(s.logit_softcap > 0.f)) throw std::runtime_error("config.logit_softcap must be positive");
+    const auto& layers = c.at("layers").items();
+    if (layers.empty()) throw std::runtime_error("config lists no layers");
+    for (const Json& j : layers) {
+        const Json& m = j.at("mixer");
+        const std::string type = j.at("type").str();
+        MixerLayerSpec l;
+        if (type == "mlstm") {
+            l.kind = MixerKind::Mlstm;
+            l.mlstm.heads = size_of(m.at("heads"));
+            l.mlstm.dim = size_of(m.at("dim"));
+            l.mlstm.vdim = size_of(m.at("vdim"));
+            l.mlstm.gate_cap = number_of(m.at("gate_cap"));
+            if (!(l.mlstm.gate_cap > 0.f)) throw std::runtime_error(m.where() + ".gate_cap must be positive");
+        } else if (type == "attention" || type == "attention_2") {
+            const bool capped = type == "attention_2";
+            l.kind = MixerKind::Attention;
+            AttentionSpec& a = l.attn;
+            a.heads = size_of(m.at("heads"));
+            a.kv_heads = size_of(m.at("kv_heads"));
+            a.dim = size_of(m.at("dim"));
+            a.vdim = size_of(m.at("vdim"));
+            a.scale = number_of(m.at("scale"));
+            a.chunk = size_of(m.at("mask").at("size"), 1, 1 << 30);
+            a.biases = true;
+            a.qk_norm = QkNorm::Whole;
+            a.sink = !capped;
+            a.gate = capped ? OutputGate::Value : OutputGate::None;
+            a.rot = read_rotary(m, a.dim, capped ? RotaryScaling::Yarn : RotaryScaling::None, capped);
+            if (capped) {
+                a.softcap = number_of(m.at("softcap"));
+                if (!(a.softcap > 0.f)) throw std::runtime_error(m.where() + ".softcap must be positive");
+            }
+            check_groups(m, a.heads, a.kv_heads);
+        } else {
+            throw std::runtime_error(j.where() + ".type `" + type + "` is not a known mixer");
+        }
+        const Json* mlp = j.find("mlp");
+        if (mlp != nullptr && !mlp->is_null()) {
+            l.moe = read_moe(*mlp);
+            l.ff = l.moe.ff;
+        }
+        const Json* of = j.find("weights_of");
+        if (of != nullptr && !of->is_null()) l.weights_of = size_of(*of, 0, (int)layers.size() - 1);
+        s.layers.push_back(l);
+    }
+    for (size_t i = 0; i < s.layers.size(); ++i) {
+        // the layer that owns the tensors, through any number of references
+        int root = (int)i;
+        for (size_t steps = 0; s.layers[(size_t)root].weights_of >= 0; ++steps) {
+            if (steps > s.layers.size()) throw std::runtime_error(layers[i].where() + ".weights_of goes round in a circle");
+            root = s.layers[(size_t)root].weights_of;
+        }
+        if (root == (int)i) continue;
+        const MixerLayerSpec &a = s.layers[i], &b = s.layers[(size_t)root];
+        if (a.kind != b.kind || a.ff != b.ff) throw std::runtime_error(layers[i].where() + ".weights_of names a layer of another kind");
+        s.layers[i] = b;
+        s.layers[i].weights_of = root;
+    }
+    return s;
+}
+
+const RegisterMixerArchitecture register_tevanex("Tevanex", read_tevanex);
 
 }  // namespace
 
@@ -201,6 +306,7 @@ std::vector<std::pair<std::string, std::vector<int64_t>>> mixer_tensors(const Mi
     if (s.side_dim > 0) add("side.embed", {V, (int64_t)s.layers.size() * s.side_dim});
     for (size_t i = 0; i < s.layers.size(); ++i) {
         const MixerLayerSpec& l = s.layers[i];
+        if (l.weights_of >= 0) continue;
         const std::string p = "l" + std::to_string(i) + ".", m = p + "mix.";
         norm(p + "norm1");
         if (l.kind == MixerKind::Wkv) {
@@ -233,6 +339,34 @@ std::vector<std::pair<std::string, std::vector<int64_t>>> mixer_tensors(const Mi
             }
             add(m + "g", {n, C});
             add(m + "o", {C, n});
+        } else if (l.kind == MixerKind::Mlstm) {
+            const MlstmSpec& x = l.mlstm;
+            const int64_t kw = (int64_t)x.heads * x.dim, vw = (int64_t)x.heads * x.vdim;
+            add(m + "q", {kw, C});
+            add(m + "k", {kw, C});
+            add(m + "v", {vw, C});
+            add(m + "g", {vw, C});
+            for (const char* gate : {"i", "f"}) {
+                add(m + gate, {x.heads, C});
+                add(m + gate + ".b", {x.heads});
+            }
+            add(m + "norm", {vw});
+            add(m + "o", {C, vw});
+        } else if (l.kind == MixerKind::Attention) {
+            const AttentionSpec& a = l.attn;
+            const int64_t qw = (int64_t)a.heads * a.dim, kw = (int64_t)a.kv_heads * a.dim, vw = (int64_t)a.kv_heads * a.vdim, ow = (int64_t)a.heads * a.vdim;
+            auto linear = [&](const char* name, int64_t rows, int64_t cols) {
+                add(m + name, {rows, cols});
+                if (a.biases) add(m + name + ".b", {rows});
+            };
+            linear("q", qw, C);
+            linear("k", kw, C);
+            linear("v", vw, C);
+            linear("o", C, ow);
+            add(m + "q.norm", {a.qk_norm == QkNorm::Whole ? qw : a.dim});
+            add(m + "k.norm", {a.qk_norm == QkNorm::Whole ? kw : a.dim});
+            if (a.sink) add(m + "sink", {a.heads});
+            if (a.gate != OutputGate::None) add(m + "g", {a.gate == OutputGate::Value ? ow : (int64_t)a.heads, C});
         } else {
             const AttentionSpec& a = l.attn;
             const DeltaSpec& d = l.delta;
@@ -259,9 +393,22 @@ std::vector<std::pair<std::string, std::vector<int64_t>>> mixer_tensors(const Mi
             add(m + "right.o", {C, dv});
             add(m + "right.out", {C});
         }
-        if (s.side_by_side) add(p + "shift", {C});
-        if (l.ff > 0) {
-            if (!s.side_by_side) norm(p + "norm2");
+        if (s.side_by_side()) add(p + "shift", {C});
+        if (l.ff > 0 && s.ff_kind == FfKind::Moe) {
+            norm(p + "norm2");
+            auto expert = [&](const std::string& name, int64_t ff) {
+                add(name + ".gate", {ff, C});
+                add(name + ".up", {ff, C});
+                add(name + ".down", {C, ff});
+            };
+            for (int e = 0; e < l.moe.experts; ++e) expert(p + "mlp.e" + std::to_string(e), l.moe.ff);
+            add(p + "mlp.router", {l.moe.experts, C});
+            if (l.moe.shared_ff > 0) {
+                expert(p + "mlp.shared", l.moe.shared_ff);
+                add(p + "mlp.shared.sg", {1, C});
+            }
+        } else if (l.ff > 0) {
+            if (!s.side_by_side()) norm(p + "norm2");
             if (s.ff_kind == FfKind::Gated) add(p + "mlp.gate", {l.ff, C});
             add(p + "mlp.up", {l.ff, C});
             add(p + "mlp.down", {C, l.ff});
@@ -287,7 +434,9 @@ std::vector<LayerRun> MixerSpec::runs() const {
     const int n = (int)layers.size();
     for (int l = 0; l < n;) {
         if (loop.times == 0 || l != loop.start) {
-            out.push_back(LayerRun{l++, -1, false});
+            const int of = layers[(size_t)l].weights_of;
+            out.push_back(LayerRun{of >= 0 ? of : l, -1, false});
+            ++l;
             continue;
         }
         for (int pass = 0; pass < loop.times; ++pass)
@@ -310,9 +459,18 @@ MixerAudit validate_mixer_tensors(const MixerSpec& s, const SafetensorsFile& f) 
 std::vector<double> rotary_frequencies(const RotarySpec& r) {
     std::vector<double> f((size_t)(r.dims / 2));
     const double two_pi = 2.0 * std::acos(-1.0);
+    double first = 0.0, span = 1.0;  // Yarn: the pair from which frequencies are stretched, and over how many pairs
+    if (r.scaling == RotaryScaling::Yarn) {
+        auto pair_that_turns = [&](double turns) { return r.dims * std::log(r.original / (two_pi * turns)) / (2.0 * std::log(r.base)); };
+        first = std::max(std::floor(pair_that_turns(r.high)), 0.0);
+        span = std::max(std::min(std::ceil(pair_that_turns(r.low)), r.dims - 1.0) - first, 0.001);
+    }
     for (int i = 0; i < r.dims / 2; ++i) {
         double v = std::pow(r.base, -2.0 * i / r.dims);
-        if (r.scaled) {
+        if (r.scaling == RotaryScaling::Yarn) {
+            const double stretched = std::min(std::max((i - first) / span, 0.0), 1.0);
+            v = v / r.factor * stretched + v * (1.0 - stretched);
+        } else if (r.scaling == RotaryScaling::Turns) {
             const double wavelength = two_pi / v;
             if (wavelength > r.original / r.low) {
                 v /= r.factor;
@@ -325,5 +483,7 @@ std::vector<double> rotary_frequencies(const RotarySpec& r) {
     }
     return f;
 }
+
+double rotary_amplitude(const RotarySpec& r) { return r.scaling == RotaryScaling::Yarn ? 0.1 * std::log(r.factor) + 1.0 : 1.0; }
 
 }  // namespace mk

@@ -10,28 +10,45 @@
 
 namespace mk {
 
-enum class NormKind { None, DynTanh, Layer };
+enum class NormKind { None, DynTanh, Layer, Rms };
+
+// How the frequencies of long wavelengths are divided by `factor`, by the turns a pair makes over the original context.
+//   Turns: below `low` turns whole, above `high` not at all, in between blended by the number of turns.
+//   Yarn:  the same between the pairs that turn `high` and `low` times, blended by the pair's index; cosine and sine are
+//          multiplied by 0.1 ln(factor) + 1.
+enum class RotaryScaling { None, Turns, Yarn };
 
 // Rotary positions on the first `dims` dimensions of a head; dims = 0: none.
 struct RotarySpec {
     int dims = 0;
     double base = 10000.0;
     bool interleaved = true;  // pairs (2i, 2i + 1); false: (i, i + dims / 2)
-    // stretch of the long wavelengths: below `low` turns over the original context by `factor`, above `high` not at all
-    bool scaled = false;
+    RotaryScaling scaling = RotaryScaling::None;
     double factor = 1.0, low = 1.0, high = 1.0, original = 1.0;
-    bool operator==(const RotarySpec& o) const {
-        return dims == o.dims && base == o.base && interleaved == o.interleaved && scaled == o.scaled &&
-               (!scaled || (factor == o.factor && low == o.low && high == o.high && original == o.original));
+    // the same angles and amplitude (the layout of the pairs aside)
+    bool same_table(const RotarySpec& o) const {
+        return dims == o.dims && base == o.base && scaling == o.scaling &&
+               (scaling == RotaryScaling::None || (factor == o.factor && low == o.low && high == o.high && original == o.original));
     }
 };
 // The frequency of every pair, in radians per position.
 std::vector<double> rotary_frequencies(const RotarySpec& r);
+// What cosine and sine are multiplied by.
+double rotary_amplitude(const RotarySpec& r);
 
-// Grouped-query attention; per-head query / key RMS norm before the rotation, a sigmoid gate per head on the output.
+enum class OutputGate { None, Head, Value };     // a sigmoid gate per head, or per value, on what attention gives
+enum class QkNorm { Head, Whole };               // RMS norm of queries and keys per head, or over all heads at once
+
+// Grouped-query attention; query / key RMS norm before the rotation.
 struct AttentionSpec {
     int heads = 0, kv_heads = 0, dim = 0, vdim = 0;
     float scale = 1.f;
+    float softcap = 0.f;      // scores pass through softcap * tanh(. / softcap); 0: as they are
+    int chunk = 0;            // a position sees the keys of its own chunk only, chunks counted from position 0; 0: all before it
+    bool sink = false;        // one learned term per head in the softmax denominator
+    bool biases = false;      // of the query, key, value and output projections
+    QkNorm qk_norm = QkNorm::Head;
+    OutputGate gate = OutputGate::Head;
     RotarySpec rot;
 };
 
@@ -57,9 +74,28 @@ struct MinGruSpec {
     int width = 0;
 };
 
-enum class MixerKind { Wkv, Parallel, Latent, MinGru };  // Parallel: attention and the gated delta rule side by side
+// Matrix memory with exponential gates: a log input and a log forget gate per head, held within +-gate_cap, and a running maximum
+// that keeps the state in range.
+struct MlstmSpec {
+    int heads = 0, dim = 0, vdim = 0;
+    float gate_cap = 1.f;
+};
 
-enum class FfKind { Gated, Poly };  // silu(gate) * up; a cubic of up, every power over its own root mean square
+// Mixture of experts: the `top` experts with the largest sigmoid scores, each reading score * row; gate and up rows held within a
+// limit.  A shared expert with a sigmoid gate per token runs beside them (shared_ff = 0: none).
+struct MoeSpec {
+    int experts = 0, top = 0, ff = 0, shared_ff = 0;
+    float limit = 0.f, shared_limit = 0.f;
+};
+
+enum class MixerKind { Wkv, Parallel, Latent, MinGru, Mlstm, Attention };  // Parallel: attention and the gated delta rule side by side
+
+enum class FfKind { Gated, Poly, Moe };  // silu(gate) * up; a cubic of up, every power over its own root mean square; experts
+
+// Where a layer's norms sit.  Input: in front of the mixer and of the feed-forward.  Shared: one in front of both, which read the
+// same row side by side; the mixer's input is mixed with the previous token's normed row (token shift).  Output: on what the mixer
+// and the feed-forward give, which read the stream itself.
+enum class NormPlace { Input, Shared, Output };
 
 struct MixerLayerSpec {
     MixerKind kind = MixerKind::Wkv;
@@ -68,7 +104,10 @@ struct MixerLayerSpec {
     DeltaSpec delta;
     LatentSpec latent;
     MinGruSpec gru;
-    int ff = 0;  // width of the feed-forward, 0: the layer has none
+    MlstmSpec mlstm;
+    int ff = 0;  // width of the feed-forward (of one expert), 0: the layer has none
+    MoeSpec moe;
+    int weights_of = -1;  // >= 0: the layer has no tensors and runs that layer's, with a cache and a state of its own
 };
 
 // Layers start .. stop - 1 run `times` times in a row, every pass with a cache and a state of its own.  A pass begins with
@@ -77,7 +116,7 @@ struct LoopSpec {
     int start = 0, stop = 0, times = 0;  // times = 0: no loop
 };
 
-// One execution of a layer: pass < 0 outside of the loop; first: the layer a pass begins with.
+// One execution of a layer: pass < 0 outside of the loop; first: the layer a pass begins with.  `layer` owns the tensors.
 struct LayerRun {
     int layer = 0, pass = -1;
     bool first = false;
@@ -89,11 +128,12 @@ struct MixerSpec {
     float eps = 1e-6f;
     NormKind norm = NormKind::DynTanh;
     FfKind ff_kind = FfKind::Gated;
-    // false: mixer and feed-forward one after the other, a norm in front of each.  true: both read one normed row and their sum
-    // is added; the mixer's input is mixed with the previous token's normed row (token shift).
-    bool side_by_side = false;
+    NormPlace norm_place = NormPlace::Input;
+    bool side_by_side() const { return norm_place == NormPlace::Shared; }
     bool sinusoid_positions = false;  // added to the embedding, which a norm then follows
-    float logit_scale = 1.f;
+    float embedding_scale = 1.f;
+    float residual_mult = 1.f;        // of every sublayer's output (NormPlace::Output)
+    float logit_scale = 1.f, logit_softcap = 0.f;  // logits <- softcap * tanh(scale * logits / softcap), 0: scale only
     LoopSpec loop;
     std::vector<MixerLayerSpec> layers;
     std::vector<LayerRun> runs() const;  // in the order of execution

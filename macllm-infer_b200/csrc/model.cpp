@@ -942,7 +942,7 @@ void Model::run_forward(const std::vector<LmLane>& lanes, KvReservation& r, uint
             } else if (gated_gemm) {
                 prof_begin(KC_HGEMM, 2.0 * (double)w.gu_half.rows * (double)w.gu_half.cols + 2.0 * T * H + 2.0 * T * ms_.ffn,
                            2.0 * T * (double)w.gu_half.rows * (double)w.gu_half.cols);
-                launch_hgemm_tc_gated(w.gu_half, xf.xh, T, ls.act, f_xh_.as<__half>(), ms_.ffn, hgemm_scratch(), stream_);
+                launch_hgemm_tc_gated(w.gu_half, xf.xh, T, GatedAct{ls.act == 0 ? GatedAct::Silu : GatedAct::GeluTanh}, f_xh_.as<__half>(), ms_.ffn, hgemm_scratch(), stream_);
                 prof_end();
                 ++launches_;
             } else if (stream_gu) {

@@ -82,9 +82,26 @@ struct StateLanes {
 #endif
 };
 
+// How a gated feed-forward joins its gate and up sums.
+//   Silu: silu(g) * u.  GeluTanh: gelu(g) * u.
+//   Clamped: g and u times `pre` of the row (the weight of a mixture of experts, which multiplies the expert's input), held within
+//   `limit` (g from above only), g * sigmoid(1.702 g) * (u + 1), times `post` of the row (the gate of a shared expert).
+struct GatedAct {
+    enum Kind : int { Silu = 0, GeluTanh = 1, Clamped = 2 };
+    int kind = Silu;
+    float limit = 0.f;
+    const float* pre = nullptr;   // [rows], null: 1
+    const float* post = nullptr;  // [rows], null: 1
+};
+
 #ifdef __CUDACC__
 __device__ __forceinline__ float sigmoid_f(float z) { return 1.0f / (1.0f + expf(-z)); }
 __device__ __forceinline__ float silu_f(float z) { return z / (1.0f + expf(-z)); }
+__device__ __forceinline__ float clamped_gate_f(float g, float u, float limit) {
+    g = fminf(g, limit);
+    u = fminf(fmaxf(u, -limit), limit);
+    return g * sigmoid_f(1.702f * g) * (u + 1.0f);
+}
 __device__ __forceinline__ float gelu_tanh_f(float z) { return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z))); }
 #endif
 

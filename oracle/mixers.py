@@ -1,4 +1,4 @@
-"""Plain NumPy statement of the mixer-built decoders (the Sizilorn and Kunonex designs and their parts), test infrastructure only.
+"""Plain NumPy statement of the mixer-built decoders (the Sizilorn, Kunonex and Tevanex designs and their parts), test infrastructure only.
 
 One function per mechanism, whole sequences at once, float64 unless the caller passes other arrays; recurrences are written
 token by token.  Nothing here is shared with the CUDA path.  Shapes: x, h [T, width]; a head-wise array [T, heads, dim].
@@ -86,6 +86,30 @@ def rotate_interleaved(x, positions, dims, freqs):
     return out
 
 
+def yarn_frequencies(dims, base, factor, original, fast, slow):
+    """Frequencies stretched by `factor` where a pair turns less than `slow` times over the original context, kept where it
+    turns more than `fast` times, blended linearly in between; and the factor of cosine and sine."""
+    f = base ** (-2.0 * np.arange(dims // 2) / dims)
+
+    def pair_that_turns(t):
+        return dims * np.log(original / (2.0 * np.pi * t)) / (2.0 * np.log(base))
+
+    lo, hi = max(np.floor(pair_that_turns(fast)), 0.0), min(np.ceil(pair_that_turns(slow)), dims - 1.0)
+    stretched = np.clip((np.arange(dims // 2) - lo) / max(hi - lo, 0.001), 0.0, 1.0)
+    return f / factor * stretched + f * (1.0 - stretched), 0.1 * np.log(factor) + 1.0
+
+
+def rotate_half(x, positions, dims, freqs):
+    """x [T, heads, dim]: the pairs (i, i + dims / 2) of the first `dims` dimensions turn by position * freqs[i]."""
+    a = np.asarray(positions, np.float64)[:, None] * freqs[None, :]
+    c, s = np.cos(a)[:, None, :], np.sin(a)[:, None, :]
+    out, n = x.copy(), dims // 2
+    u, v = x[..., :n], x[..., n:dims]
+    out[..., :n] = u * c - v * s
+    out[..., n:dims] = v * c + u * s
+    return out
+
+
 # ------------------------------------------------------------------------------------------------ attention
 
 def causal_attention(q, k, v, scale):
@@ -117,6 +141,59 @@ def gated_attention(h, W, cfg, eps):
     o = causal_attention(q, k, v, cfg["scale"])
     o = o * sigmoid(h @ W["g"].T)[:, :, None]
     return o.reshape(T, H * e) @ W["o"].T
+
+
+def chunked_attention(q, k, v, scale, chunk, softcap=None, sink=None):
+    """q [T, H, d], k [T, G, d], v [T, G, e]; a position sees the keys of its own chunk up to itself.  softcap: scores pass
+    through softcap * tanh(. / softcap); sink [H]: one more term exp(sink) in every denominator."""
+    T, H, _ = q.shape
+    group = H // k.shape[1]
+    out = np.empty((T, H, v.shape[2]), q.dtype)
+    for h in range(H):
+        for t in range(T):
+            lo = t // chunk * chunk
+            s = k[lo:t + 1, h // group] @ q[t, h] * scale
+            if softcap is not None:
+                s = softcap * np.tanh(s / softcap)
+            top = s.max() if sink is None else max(s.max(), sink[h])
+            p = np.exp(s - top)
+            den = p.sum() + (0.0 if sink is None else np.exp(sink[h] - top))
+            out[t, h] = p @ v[lo:t + 1, h // group] / den
+    return out
+
+
+def projected_heads(h, W, cfg, eps):
+    """q, k, v with biases; the RMS norm of q and k runs over all heads at once."""
+    T = h.shape[0]
+    q = rms(h @ W["q"].T + W["q.b"], eps) * W["q.norm"]
+    k = rms(h @ W["k"].T + W["k.b"], eps) * W["k.norm"]
+    v = h @ W["v"].T + W["v.b"]
+    return q.reshape(T, cfg["heads"], cfg["dim"]), k.reshape(T, cfg["kv_heads"], cfg["dim"]), v.reshape(T, cfg["kv_heads"], cfg["vdim"])
+
+
+def sink_attention(h, W, cfg, eps):
+    """Chunked attention with a sink per head and half-split rotation."""
+    q, k, v = projected_heads(h, W, cfg, eps)
+    rot, pos = cfg["rot"], np.arange(h.shape[0])
+    f = rope_frequencies(rot["dims"], rot["base"])
+    q, k = rotate_half(q, pos, rot["dims"], f), rotate_half(k, pos, rot["dims"], f)
+    o = chunked_attention(q, k, v, cfg["scale"], cfg["mask"]["size"], sink=W["sink"])
+    return o.reshape(len(pos), -1) @ W["o"].T + W["o.b"]
+
+
+def capped_attention(h, W, cfg, eps):
+    """Chunked attention with capped scores, adjacent-pair rotation stretched to a longer context, and an element-wise gate."""
+    q, k, v = projected_heads(h, W, cfg, eps)
+    rot, pos = cfg["rot"], np.arange(h.shape[0])
+    f, m = yarn_frequencies(rot["dims"], rot["base"], **rot["scaling"])
+
+    def turn(x):
+        r = rotate_interleaved(x, pos, rot["dims"], f)
+        r[..., :rot["dims"]] *= m
+        return r
+
+    o = chunked_attention(turn(q), turn(k), v, cfg["scale"], cfg["mask"]["size"], softcap=cfg["softcap"])
+    return (o.reshape(len(pos), -1) * sigmoid(h @ W["g"].T)) @ W["o"].T + W["o.b"]
 
 
 def latent_attention(h, W, cfg, eps):
@@ -217,6 +294,39 @@ def wkv_mixer(h, W, cfg, eps):
     return (rms(o, eps).reshape(T, H * d) * W["norm"] * silu(mix["g"] @ W["g"].T)) @ W["o"].T
 
 
+# ------------------------------------------------------------------------------------------------ mLSTM
+
+def mlstm_gates(zi, zf, cap):
+    """Log input gate and log forget gate from their projections (biases included)."""
+    return cap * np.tanh(zi / cap), -softplus(-cap * np.tanh(zf / cap))
+
+
+def mlstm_rule(q, k, v, i, f, state=None):
+    """q, k [T, H, d], v [T, H, e], i, f [T, H].  State (S [H, d, e], n [H, d], m [H]) is kept times exp(-m), m the running
+    maximum of the logarithms, 0 at the start.  Returns (o [T, H, e], state)."""
+    T, H, d = k.shape
+    S, n, m = (np.zeros((H, d, v.shape[2]), v.dtype), np.zeros((H, d), v.dtype), np.zeros(H, v.dtype)) if state is None else [a.copy() for a in state]
+    o = np.empty_like(v)
+    for t in range(T):
+        top = np.maximum(f[t] + m, i[t])
+        keep, write = np.exp(f[t] + m - top), np.exp(i[t] - top)
+        S = keep[:, None, None] * S + write[:, None, None] * k[t][:, :, None] * v[t][:, None, :]
+        n = keep[:, None] * n + write[:, None] * k[t]
+        m = top
+        den = np.maximum(np.abs(np.einsum("hd,hd->h", n, q[t])), np.exp(-m)) + 1e-6
+        o[t] = np.einsum("hde,hd->he", S, q[t]) / den[:, None]
+    return o, (S, n, m)
+
+
+def mlstm_mixer(h, W, cfg, eps):
+    T = h.shape[0]
+    H, d, e = cfg["heads"], cfg["dim"], cfg["vdim"]
+    q, k = (h @ W["q"].T).reshape(T, H, d) / np.sqrt(d), (h @ W["k"].T).reshape(T, H, d)
+    i, f = mlstm_gates(h @ W["i"].T + W["i.b"], h @ W["f"].T + W["f.b"], cfg["gate_cap"])
+    o, _ = mlstm_rule(q, k, (h @ W["v"].T).reshape(T, H, e), i, f)
+    return (rms(o, eps).reshape(T, H * e) * W["norm"] * sigmoid(h @ W["g"].T)) @ W["o"].T
+
+
 # ------------------------------------------------------------------------------------------------ minGRU
 
 def min_gru(z, u, state=None):
@@ -249,6 +359,32 @@ def poly_mlp(h, W, eps):
 
 def gated_mlp(h, W):
     return (silu(h @ W["gate"].T) * (h @ W["up"].T)) @ W["down"].T
+
+
+def clamped_mlp(h, W, limit):
+    """Gate and up rows held within a limit, the gate through z * sigmoid(1.702 z), the up rows plus one."""
+    g = np.minimum(h @ W["gate"].T, limit)
+    u = np.clip(h @ W["up"].T, -limit, limit)
+    return (g * sigmoid(1.702 * g) * (u + 1.0)) @ W["down"].T
+
+
+def routed(h, W, top):
+    """Chosen experts and their weights [T, top]: the largest sigmoid scores, as they are."""
+    s = sigmoid(h @ W["router"].T)
+    chosen = np.argsort(-s, axis=1, kind="stable")[:, :top]
+    return chosen, np.take_along_axis(s, chosen, axis=1)
+
+
+def moe_mlp(h, W, cfg):
+    """Every chosen expert reads its weight times the row; a shared expert with a gate per token runs beside them."""
+    sub = lambda p: {k[len(p):]: v for k, v in W.items() if k.startswith(p)}
+    chosen, weight = routed(h, W, cfg["router"]["top"])
+    out = sigmoid(h @ W["shared.sg"].T) * clamped_mlp(h, sub("shared."), cfg["shared"]["limit"])
+    for e in range(cfg["router"]["experts"]):
+        t, j = np.nonzero(chosen == e)
+        if len(t):
+            out[t] += clamped_mlp(weight[t, j][:, None] * h[t], sub(f"e{e}."), cfg["expert"]["limit"])
+    return out
 
 
 def token_side(x, e, W, eps):
@@ -338,8 +474,39 @@ class KunonexDecoder(MixerDecoder):
         return super().logits(tokens) * self.cfg["logit_scale"]
 
 
+class TevanexDecoder(MixerDecoder):
+    """mLSTM layers and two kinds of chunked attention over a mixture of experts; norms on what a sublayer gives, not on what it
+    reads; layers that run another one's tensors again."""
+
+    def _norm(self, name, x):
+        return rms(x, self.cfg["norm"]["eps"]) * self.w[name]
+
+    def embedding_output(self, tokens):
+        return self.w["embed"][tokens] * self.cfg["embedding"]["scale"]
+
+    def residuals(self, tokens):
+        """The residual stream after every layer: [layers, T, width]."""
+        eps, m = self.cfg["norm"]["eps"], self.cfg["residual_mult"]
+        x = self.embedding_output(np.asarray(tokens))
+        out = []
+        for i, layer in enumerate(self.cfg["layers"]):
+            while self.cfg["layers"][i].get("weights_of") is not None:
+                i = self.cfg["layers"][i]["weights_of"]
+            p = f"l{i}."
+            mixer = {"mlstm": mlstm_mixer, "attention": sink_attention, "attention_2": capped_attention}[layer["type"]]
+            x = x + m * self._norm(p + "norm1", mixer(x, self._sub(p + "mix."), layer["mixer"], eps))
+            if layer.get("mlp"):
+                x = x + m * self._norm(p + "norm2", moe_mlp(x, self._sub(p + "mlp."), layer["mlp"]))
+            out.append(x)
+        return np.stack(out)
+
+    def logits(self, tokens):
+        cap = self.cfg["logit_softcap"]
+        return cap * np.tanh(super().logits(tokens) * self.cfg["logit_scale"] / cap)
+
+
 def decoder(config, tensors, dtype=np.float64):
-    return {"Sizilorn": MixerDecoder, "Kunonex": KunonexDecoder}[config["architecture"]](config, tensors, dtype)
+    return {"Sizilorn": MixerDecoder, "Kunonex": KunonexDecoder, "Tevanex": TevanexDecoder}[config["architecture"]](config, tensors, dtype)
 
 
 def read_safetensors(path):
