@@ -1,6 +1,6 @@
 """Throughput of mixer-built decoders (random weights, layers of real-model sizes) beside the closest GGUF family of the same
-width, heads, feed-forward and layer count (looped layers counted once per pass) with dense BF16 matrices.  Used by
-`bench.py --mixer`.
+width, heads, feed-forward and layer count (looped layers counted once per pass): dense BF16 matrices, or, beside mixtures of experts,
+the sparse family with its own quantised ones.  Used by `bench.py --mixer`.
 
 Every figure is device time (CUDA events around the tick, median over the timed ticks); the weights of a tick are several
 times the L2.  The per-class table comes from separate ticks with an event pair around every launch; `roofline` there is the
@@ -73,7 +73,49 @@ BESIDE_SHAPES = [
 ]
 
 
+@dataclass
+class ExpertShape:
+    """Groups of four layers - capped attention, two of mLSTM, sink attention - over a mixture of experts."""
+    name: str
+    width: int
+    groups: int
+    heads: int           # of attention
+    kv_heads: int
+    dim: int
+    chunk: int
+    mem_heads: int       # of mLSTM
+    mem_dim: int
+    mem_vdim: int
+    experts: int
+    top: int
+    ff: int
+    vocab: int = 32000
+
+    @property
+    def runs(self) -> int:
+        return 4 * self.groups
+
+
+EXPERT_SHAPES = [
+    ExpertShape("w2048", 2048, 1, 16, 4, 128, 8192, 8, 128, 256, 64, 8, 768),
+    ExpertShape("w4096", 4096, 1, 32, 8, 128, 8192, 16, 128, 256, 16, 2, 2048),
+]
+
+
+def expert_layers(s) -> list:
+    mlp = {"kind": "moe", "router": {"experts": s.experts, "top": s.top}, "expert": {"ff": s.ff, "limit": 7.0}, "shared": {"ff": s.ff, "limit": 7.0}}
+    attn = {"heads": s.heads, "kv_heads": s.kv_heads, "dim": s.dim, "vdim": s.dim, "scale": s.dim ** -0.5, "mask": {"size": s.chunk}}
+    sink = {"type": "attention", "mlp": mlp, "mixer": {**attn, "rot": {"base": 10000.0, "dims": s.dim}}}
+    capped = {"type": "attention_2", "mlp": mlp, "mixer": {**attn, "softcap": 30.0, "rot": {
+        "base": 500000.0, "dims": s.dim, "scaling": {"factor": 8.0, "original": 8192, "fast": 32.0, "slow": 1.0}}}}
+    mem = {"type": "mlstm", "mlp": mlp, "mixer": {"heads": s.mem_heads, "dim": s.mem_dim, "vdim": s.mem_vdim, "gate_cap": 15.0}}
+    return [capped, mem, mem, sink] * s.groups
+
+
 def config_of(s) -> dict:
+    if isinstance(s, ExpertShape):
+        return {"architecture": "Tevanex", "vocab": s.vocab, "width": s.width, "norm": {"eps": 1e-6}, "embedding": {"scale": 1.0}, "residual_mult": 0.5,
+                "logit_scale": 1.0, "logit_softcap": 30.0, "layers": expert_layers(s)}
     if isinstance(s, BesideShape):
         mlp = {"kind": "dense", "ff": s.ff}
         lat = {"type": "latent_attention", "mlp": mlp, "mixer": {"heads": s.heads, "dim": s.dim, "vdim": s.dim, "q_rank": s.q_rank, "kv_rank": s.kv_rank,
@@ -109,6 +151,40 @@ def tensor_shapes(s) -> dict[str, tuple]:
             vec(name + ".alpha", mean=0.7, dev=0.0)
 
     out["embed"] = ((V, C), 0.0, 1.0)
+    if isinstance(s, ExpertShape):
+        for i, layer in enumerate(expert_layers(s)):
+            p, m = f"l{i}.", layer["mixer"]
+            vec(p + "norm1", C)
+            vec(p + "norm2", C)
+            qw, vw = m["heads"] * m["dim"], m["heads"] * m["vdim"]
+            G = m.get("kv_heads", m["heads"])
+            mat(p + "mix.q", qw, C)
+            mat(p + "mix.k", G * m["dim"], C)
+            mat(p + "mix.v", G * m["vdim"], C)
+            mat(p + "mix.o", C, vw)
+            if layer["type"] != "attention":
+                mat(p + "mix.g", vw, C)
+            if layer["type"] == "mlstm":
+                vec(p + "mix.norm", vw)
+                for x, mean in (("i", -1.0), ("f", 4.0)):
+                    mat(p + "mix." + x, m["heads"], C)
+                    vec(p + f"mix.{x}.b", m["heads"], mean=mean)
+            else:
+                for x, n in (("q", qw), ("k", G * m["dim"]), ("v", G * m["vdim"]), ("o", C)):
+                    vec(p + f"mix.{x}.b", n, mean=0.0)
+                vec(p + "mix.q.norm", qw)
+                vec(p + "mix.k.norm", G * m["dim"])
+            if layer["type"] == "attention":
+                vec(p + "mix.sink", m["heads"])
+            for name in [f"e{e}" for e in range(s.experts)] + ["shared"]:
+                mat(p + f"mlp.{name}.gate", s.ff, C)
+                mat(p + f"mlp.{name}.up", s.ff, C)
+                mat(p + f"mlp.{name}.down", C, s.ff)
+            mat(p + "mlp.router", s.experts, C)
+            mat(p + "mlp.shared.sg", 1, C)
+        vec("final.norm", C)
+        mat("head", V, C)
+        return out
     if beside:
         norm("embed.norm")
         mat("loop.in", C, 2 * C)
@@ -213,6 +289,9 @@ def write_checkpoint(folder: Path, s) -> Path:
 
 
 def closest_spec(s) -> seed_gguf.SeedSpec:
+    if isinstance(s, ExpertShape):
+        return seed_gguf.SeedSpec("qwen3moe", s.runs, s.width, s.heads, s.kv_heads, s.dim, 4 * s.ff, s.vocab, context=16384, theta=1e6, eps=1e-6, experts=s.experts,
+                                  experts_used=s.top, expert_ffn=s.ff, name=f"closest-{s.name}")
     layers = s.runs if isinstance(s, BesideShape) else 2 * s.pairs
     return seed_gguf.SeedSpec("qwen3", layers, s.width, s.heads, s.kv_heads, s.dim, s.ff, s.vocab, context=16384, theta=1e6, eps=1e-6,
                               matrix_type=capi.TYPE_BF16, high_type=capi.TYPE_BF16, name=f"closest-{s.name}")
@@ -278,7 +357,7 @@ def measure(model, vocab: int, prompt: int, lanes: int, context: int, warmup: in
     return out
 
 
-DESIGNS = {"sizilorn": ("Sizilorn", SHAPES), "kunonex": ("Kunonex", BESIDE_SHAPES)}
+DESIGNS = {"sizilorn": ("Sizilorn", SHAPES), "kunonex": ("Kunonex", BESIDE_SHAPES), "tevanex": ("Tevanex", EXPERT_SHAPES)}
 
 
 def run(peaks: dict, warmup: int, steps: int, design="sizilorn", prompt=2048, lanes=64, context=1024) -> list[dict]:
@@ -299,7 +378,7 @@ def run(peaks: dict, warmup: int, steps: int, design="sizilorn", prompt=2048, la
                     weights = seed_gguf.weight_bytes(closest_spec(s))["per_token"]
                 r = measure(model, s.vocab, prompt, lanes, context, warmup, steps, peaks)
                 sp = model.spec()
-                results.append(dict(shape=s.name, model=title if kind == design else "qwen3 family, dense BF16 matrices", layers=int(sp.n_layers),
+                results.append(dict(shape=s.name, model=title if kind == design else ("qwen3moe family, Q4_K / Q6_K matrices" if isinstance(s, ExpertShape) else "qwen3 family, dense BF16 matrices"), layers=int(sp.n_layers),
                                     width=int(sp.hidden_size), weight_gb=round(weights / 1e9, 3), **r))
                 model.close()
     return results

@@ -379,7 +379,9 @@ def moe_mlp(h, W, cfg):
     """Every chosen expert reads its weight times the row; a shared expert with a gate per token runs beside them."""
     sub = lambda p: {k[len(p):]: v for k, v in W.items() if k.startswith(p)}
     chosen, weight = routed(h, W, cfg["router"]["top"])
-    out = sigmoid(h @ W["shared.sg"].T) * clamped_mlp(h, sub("shared."), cfg["shared"]["limit"])
+    out = np.zeros_like(h)
+    if cfg.get("shared"):
+        out = sigmoid(h @ W["shared.sg"].T) * clamped_mlp(h, sub("shared."), cfg["shared"]["limit"])
     for e in range(cfg["router"]["experts"]):
         t, j = np.nonzero(chosen == e)
         if len(t):

@@ -44,6 +44,121 @@ def config(layers, width=96, vocab=131, side=12, eps=3e-5):
             "token_side": {"dim": side} if side else None, "layers": layers}
 
 
+def experts(n, top, ff, limit=1.0, shared=None):
+    """shared = (ff, limit) of the expert every token runs."""
+    return {"kind": "moe", "router": {"experts": n, "top": top}, "expert": {"ff": ff, "limit": limit},
+            "shared": {"ff": shared[0], "limit": shared[1]} if shared else None}
+
+
+def mlstm(heads, dim, vdim, cap=4.0, mlp=None):
+    return {"type": "mlstm", "mixer": {"heads": heads, "dim": dim, "vdim": vdim, "gate_cap": cap}, "mlp": mlp}
+
+
+YARN = dict(factor=4.0, original=64, fast=8.0, slow=1.0)
+
+
+def sink_attention(heads, kv_heads, dim, vdim, rot, chunk, mlp=None):
+    return {"type": "attention", "mlp": mlp, "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": 0.9 / dim ** 0.5,
+                                                       "mask": {"size": chunk}, "rot": {"base": 500.0, "dims": rot}}}
+
+
+def capped_attention(heads, kv_heads, dim, vdim, rot, chunk, softcap=2.5, mlp=None, yarn=YARN):
+    m = sink_attention(heads, kv_heads, dim, vdim, rot, chunk, mlp)
+    m["type"] = "attention_2"
+    m["mixer"]["softcap"] = softcap
+    m["mixer"]["rot"]["scaling"] = dict(yarn)
+    return m
+
+
+def again(layers, i):
+    """An entry that runs layer i's tensors again."""
+    return {**layers[i], "weights_of": i}
+
+
+def tevanex(layers, width=96, vocab=131, eps=3e-5, embed=1.7, mult=0.6, logit_scale=0.8, softcap=9.0):
+    return {"architecture": "Tevanex", "vocab": vocab, "width": width, "norm": {"eps": eps}, "embedding": {"scale": embed},
+            "residual_mult": mult, "logit_scale": logit_scale, "logit_softcap": softcap, "layers": layers}
+
+
+ROUTING = 8   # channels that only embeddings write and routers read, so that a choice is a token's and never close; one more is constant
+
+
+def tevanex_weights(cfg, seed):
+    rng = np.random.default_rng(seed)
+    C, V = cfg["width"], cfg["vocab"]
+    w = {}
+
+    def mat(name, rows, cols, gain=1.0):
+        w[name] = rng.standard_normal((rows, cols)) * gain / np.sqrt(cols)
+
+    def around_one(name, n):
+        w[name] = 1.0 + 0.3 * rng.standard_normal(n)
+
+    def bias(name, n, dev=0.3):
+        w[name] = dev * rng.standard_normal(n)
+
+    w["embed"] = rng.standard_normal((V, C))
+    w["embed"][:, ROUTING] = 1.0
+    routers = []
+    for i, layer in enumerate(cfg["layers"]):
+        if layer.get("weights_of") is not None:
+            continue
+        p, m = f"l{i}.", layer["mixer"]
+        H, d, e = m["heads"], m["dim"], m["vdim"]
+        if layer["type"] == "mlstm":
+            mat(p + "mix.q", H * d, C)
+            mat(p + "mix.k", H * d, C)
+            mat(p + "mix.v", H * e, C)
+            # the constant channel gives queries and keys a common part: denominators are sums without much cancellation
+            w[p + "mix.q"][:, ROUTING] = w[p + "mix.k"][:, ROUTING] = rng.standard_normal(H * d)
+            mat(p + "mix.g", H * e, C)
+            for s, b in (("i", -1.0), ("f", 3.0)):
+                mat(p + "mix." + s, H, C)
+                w[p + "mix." + s + ".b"] = b + rng.standard_normal(H)
+            around_one(p + "mix.norm", H * e)
+        else:
+            G = m["kv_heads"]
+            for s, n in (("q", H * d), ("k", G * d), ("v", G * e)):
+                mat(p + "mix." + s, n, C)
+                bias(p + "mix." + s + ".b", n)
+            w[p + "mix.q.norm"] = 1.5 + 0.3 * rng.standard_normal(H * d)
+            w[p + "mix.k.norm"] = 1.5 + 0.3 * rng.standard_normal(G * d)
+            bias(p + "mix.o.b", C)
+            if layer["type"] == "attention":
+                w[p + "mix.sink"] = 1.5 + rng.standard_normal(H)
+            else:
+                mat(p + "mix.g", H * e, C)
+        mat(p + "mix.o", C, H * e)
+        around_one(p + "norm1", C)
+        w[p + "norm1"][:ROUTING + 1] = 0.0
+        if layer["mlp"]:
+            x = layer["mlp"]
+            around_one(p + "norm2", C)
+            w[p + "norm2"][:ROUTING + 1] = 0.0
+            for name, ff in [(f"e{j}", x["expert"]["ff"]) for j in range(x["router"]["experts"])] + ([("shared", x["shared"]["ff"])] if x["shared"] else []):
+                mat(p + f"mlp.{name}.gate", ff, C)
+                mat(p + f"mlp.{name}.up", ff, C)
+                mat(p + f"mlp.{name}.down", C, ff)
+            if x["shared"]:
+                mat(p + "mlp.shared.sg", 1, C)
+            r = np.zeros((x["router"]["experts"], C))
+            r[:, :ROUTING] = mixers.bf16(rng.standard_normal((len(r), ROUTING)).astype(np.float32) / np.sqrt(ROUTING) / cfg["embedding"]["scale"])
+            w[p + "mlp.router"] = r
+            routers.append((r, x["router"]["top"]))
+    # a token's last chosen and first left-out logits are well apart in every layer
+    for t in range(V):
+        for _ in range(100000):
+            z = [np.sort(r @ (w["embed"][t] * cfg["embedding"]["scale"]))[::-1] for r, _ in routers]
+            if all(k == len(s) or s[k - 1] - s[k] > 0.06 for s, (_, k) in zip(z, routers)):
+                break
+            w["embed"][t, :ROUTING] = 1.5 * rng.standard_normal(ROUTING)
+        else:
+            raise AssertionError("no embedding with clear choices was found")
+    around_one("final.norm", C)
+    mat("head", V, C, 2.0)
+    return w
+
+
 def kunonex_weights(cfg, seed):
     rng = np.random.default_rng(seed)
     C, V = cfg["width"], cfg["vocab"]
@@ -100,6 +215,8 @@ def weights(cfg, seed=0, rank=5):
     """name -> float32 array holding bfloat16 values."""
     if cfg["architecture"] == "Kunonex":
         return {k: mixers.bf16(np.asarray(v, np.float32)) for k, v in kunonex_weights(cfg, seed).items()}
+    if cfg["architecture"] == "Tevanex":
+        return {k: mixers.bf16(np.asarray(v, np.float32)) for k, v in tevanex_weights(cfg, seed).items()}
     rng = np.random.default_rng(seed)
     C, V, side = cfg["width"], cfg["vocab"], (cfg.get("token_side") or {}).get("dim", 0)
     w = {}

@@ -90,6 +90,30 @@ ALONE_BESIDE = {
 }
 
 
+ALONE_OUTPUT = {
+    # name: (layer, width, what is silenced)
+    "mLSTM": (mc.mlstm(3, 64, 64), 96, ()),
+    "mLSTM odd sizes": (mc.mlstm(2, 43, 37), 70, ()),
+    "mLSTM 128, tight cap": (mc.mlstm(2, 128, 128, cap=0.8), 96, ()),
+    "mLSTM narrow keys, wide values": (mc.mlstm(1, 12, 200), 64, ()),
+    "mLSTM wide keys": (mc.mlstm(2, 200, 72, cap=12.0), 64, ()),
+    "mLSTM two values": (mc.mlstm(5, 9, 2), 64, ()),
+    "sink, chunk of a page": (mc.sink_attention(4, 2, 64, 64, 64, 16), 96, ()),
+    "sink, odd chunk, partly turned": (mc.sink_attention(8, 2, 48, 24, 22, 33), 96, ()),
+    "sink, three heads per key": (mc.sink_attention(6, 2, 20, 36, 20, 10), 70, ()),
+    "sink, chunk of one": (mc.sink_attention(2, 2, 128, 96, 64, 1), 64, ()),
+    "sink, one chunk for all": (mc.sink_attention(8, 1, 32, 128, 30, 4096), 64, ()),
+    "capped, chunk of a tile": (mc.capped_attention(4, 2, 64, 64, 64, 32), 96, ()),
+    "capped, odd chunk, partly turned": (mc.capped_attention(8, 4, 40, 24, 26, 27, softcap=0.7), 96, ()),
+    "capped, odd width, five heads": (mc.capped_attention(5, 5, 21, 33, 12, 50, softcap=30.0), 67, ()),
+    "capped, 256 wide": (mc.capped_attention(2, 1, 200, 130, 128, 7, yarn=dict(factor=16.0, original=512, fast=32.0, slow=2.0)), 64, ()),
+    "experts, one of five": (mc.mlstm(1, 8, 8, mlp=mc.experts(5, 1, 37, 0.5)), 66, ("l0.norm1",)),
+    "experts, seven of forty and a shared one": (mc.mlstm(1, 8, 8, mlp=mc.experts(40, 7, 24, 2.0, (90, 0.3))), 96, ("l0.norm1",)),
+    "experts, all of three": (mc.mlstm(1, 8, 8, mlp=mc.experts(3, 3, 130, 0.7, (20, 3.0))), 130, ("l0.norm1",)),
+    "experts behind a mixer": (mc.sink_attention(2, 1, 16, 16, 8, 12, mlp=mc.experts(6, 2, 64, 1.0, (64, 1.0))), 64, ()),
+}
+
+
 def check_alone(folder, oracle, compute):
     """The residual stream after a layer with one mechanism at work, for a whole prompt, portions and single tokens."""
     toks = tokens_of(75, oracle.cfg["vocab"])
@@ -127,6 +151,13 @@ def test_mechanism_alone_in_layers_with_one_norm(mk, tmp_path, name, compute):
 
 
 @pytest.mark.parametrize("compute", DTYPES)
+@pytest.mark.parametrize("name", ALONE_OUTPUT)
+def test_mechanism_alone_in_layers_with_norms_on_outputs(mk, tmp_path, name, compute):
+    layer, width, silenced = ALONE_OUTPUT[name]
+    check_alone(*checkpoint(tmp_path, mc.tevanex([layer], width=width), seed=7, change=silence(*silenced)), compute)
+
+
+@pytest.mark.parametrize("compute", DTYPES)
 def test_token_shift_reaches_the_mixer_only(mk, tmp_path, compute):
     """A shift of one: the mixer sees nothing but the token before (zeros at first), the feed-forward nothing but the token."""
     cfg = mc.kunonex([mc.mingru(20, ff=30)], width=50, vocab=40)
@@ -155,6 +186,9 @@ def test_sinusoidal_positions_far_out(mk, tmp_path, width, compute):
 
 # ------------------------------------------------------------------------------------------------ whole models
 
+_EXPERTS = [mc.mlstm(4, 32, 48, mlp=mc.experts(6, 2, 40, 0.8, (60, 1.2))), mc.sink_attention(4, 2, 64, 40, 64, 24, mlp=mc.experts(12, 1, 64)),
+            mc.capped_attention(8, 2, 64, 64, 32, 48, mlp=mc.experts(4, 4, 33, 1.5, (33, 1.5))), mc.mlstm(2, 64, 130)]
+
 MODELS = {
     "first": (mc.config([mc.wkv(3, 40), mc.parallel((4, 2, 64, 64, 32, True), (4, 2, 32, 48, 4), ff=150), mc.wkv(2, 64, ff=90)], width=104), 9),
     "second": (mc.config([mc.parallel((6, 2, 36, 20, 12, False), (3, 3, 48, 40, 2)), mc.wkv(5, 16), mc.parallel((8, 1, 32, 32, 32, True), (2, 2, 64, 64, 3), ff=64)],
@@ -165,6 +199,9 @@ MODELS = {
                                         logit_scale=1.3), 0),
     "no loop": (mc.kunonex([mc.mingru(24, ff=60), mc.latent(20, 16, 16, 64, 40, ff=60)], width=64, logit_scale=1.0), 0),
     "a loop of one pass": (mc.kunonex([mc.latent(3, 24, 24, 24, 24), mc.mingru(50, ff=32)], width=48, loop=(1, 2, 1)), 0),
+    "experts": (mc.tevanex(_EXPERTS + [mc.again(_EXPERTS, 1), mc.again(_EXPERTS, 0)], width=104), 0),
+    "experts, odd sizes": (mc.tevanex([mc.capped_attention(6, 2, 44, 36, 28, 50, mlp=mc.experts(5, 3, 37)), mc.mlstm(3, 40, 21, mlp=mc.experts(9, 2, 50, 0.6, (70, 0.4))),
+                                       mc.sink_attention(8, 1, 32, 80, 32, 20)], width=67, vocab=201, eps=1e-5, embed=2.3, mult=0.35, logit_scale=1.4, softcap=3.0), 0),
     "time mixing only": (mc.config([mc.wkv(2, 32), mc.wkv(1, 72)], width=64, side=64), 20),
 }
 
@@ -195,7 +232,7 @@ def test_prompt_portions_and_decoding_agree(mk, built, name, compute):
     model.close()
 
 
-BOTH = ["first", "looped"]   # a model of each layer form
+BOTH = ["first", "looped", "experts"]   # a model of each layer form
 
 
 @pytest.mark.parametrize("compute", DTYPES)
@@ -431,7 +468,7 @@ def test_a_fork_carries_pages_and_state(mk, built, name, compute):
     model.close()
 
 
-@pytest.mark.parametrize("name", ["second", "looped"])
+@pytest.mark.parametrize("name", ["second", "looped", "experts"])
 def test_a_refused_forward_leaves_the_state_alone(mk, built, capi, name):
     folder, oracle, cfg = built(name)
     toks = tokens_of(50, cfg["vocab"], seed=9)
@@ -447,7 +484,7 @@ def test_a_refused_forward_leaves_the_state_alone(mk, built, capi, name):
     model.close()
 
 
-@pytest.mark.parametrize("name", ["first", "second", "looped", "loop over all layers", "no loop"])
+@pytest.mark.parametrize("name", ["first", "second", "looped", "loop over all layers", "no loop", "experts", "experts, odd sizes"])
 def test_greedy_generation_through_the_engine(mk, eng, built, name):
     """Requests of unequal length through the scheduler, more of them than slots; 32-bit, so that the plain statement's own
     argmax must come out wherever its first two logits are not a near-tie."""
@@ -484,7 +521,7 @@ def test_device_sampling_and_recorded_logits(mk, eng, built, name):
     assert outs[0] == outs[1]
 
 
-@pytest.mark.parametrize("name", ["second", "looped", "loop over all layers"])
+@pytest.mark.parametrize("name", ["second", "looped", "loop over all layers", "experts", "experts, odd sizes"])
 def test_residuals_after_every_layer(mk, built, name):
     """A looped layer counts once per pass."""
     folder, oracle, cfg = built(name)
