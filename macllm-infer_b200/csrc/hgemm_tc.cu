@@ -167,10 +167,20 @@ __global__ void dequant_f16_kernel(QWeight W, __half* out, int64_t row_stride) {
 
 // ---- the GEMM ------------------------------------------------------------------------------------
 
-struct HgParams {
-    int T, K, rows;
+// Grouped form: one of the two matrices of a launch.
+struct HgPart {
+    int row_tiles, rows;      // row tiles of an expert's matrix, its true rows
+    int T, k_blocks;          // rows (the second part), K blocks
     float* y;
     int ldy;
+    __half* yh;
+    int ldyh;
+    float act_limit;          // of GatedAct::Clamped
+    const float *act_pre, *act_post;
+};
+
+struct HgParams {
+    int T, K, rows;
     float out_scale, softcap;
     int row_tiles, n_tiles;
     // split-K (narrow batches, long K): work item = (output tile, K share); every share writes its f32
@@ -182,11 +192,6 @@ struct HgParams {
     // gated epilogue (splits == 1): weight rows 2j / 2j+1 are the gate / up projections of feature j and the kernel
     // writes yh[t][j] = f16(act(gate, up)) instead of y; 0 = off, otherwise 1 + GatedAct::Kind
     int gated;
-    float act_limit;
-    const float* act_pre;
-    const float* act_post;
-    __half* yh;
-    int ldyh;
     int bf16;  // both operands (and yh) are bfloat16
     // stacked projections with inputs of their own: the first row of input g in the activation matrix is g * T
     int n_groups;
@@ -194,10 +199,12 @@ struct HgParams {
     int group_tiles;
     int scattered;  // the result goes where `scatter` says (splits == 1)
     MatmulScatter scatter;
-    // activation rows grouped by expert: row_tiles row tiles per expert, item = (expert, row tile, token tile of its rows)
+    // activation rows grouped by expert, beside them a matrix that rows of its own meet all of (see HgPart); item = (part, expert,
+    // row tile, token tile of the expert's rows)
     int experts;
-    int expert_rows;          // true rows of an expert's matrix
+    int box_rows;             // rows of an activation box
     const int32_t* offsets;   // [experts + 1]
+    HgPart part[2];
 };
 constexpr int HG_MAX_EXPERTS = 1024;
 
@@ -206,7 +213,14 @@ struct HgTile {
     int w_row, row0;          // weight row of the tile (within the whole image), output row it becomes
     int x_row, tok0, tok_end; // activation row of the tile (box), its first output row, end of the output rows
     int rows;                 // end of the output columns
+    int part;                 // grouped: 0 experts, 1 the matrix beside them
 };
+
+// Rows shared out evenly over as few tiles of at most `most` rows as hold them, in steps of 16.
+__device__ __forceinline__ int even_tile(int n, int most) {
+    const int tiles = (n + most - 1) / most;
+    return ((n + tiles - 1) / tiles + 15) & ~15;
+}
 
 __device__ __forceinline__ int group_row0(const HgParams& p, int m_tile) {
     if (p.n_groups == 1) return 0;
@@ -238,7 +252,8 @@ __device__ __forceinline__ float hg_gelu_tanh(float x) {
 
 template <int BN, int STAGES>
 __global__ void __launch_bounds__(HG_THREADS, 1)
-hgemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__ CUtensorMap tm_x, HgParams p) {
+hgemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__ CUtensorMap tm_x, const __grid_constant__ CUtensorMap tm_w1,
+                const __grid_constant__ CUtensorMap tm_x1, const __grid_constant__ HgParams p) {
     using L = HgSmem<BN, STAGES>;
     constexpr int LD_COLS = BN >= 32 ? 32 : BN;
     extern __shared__ uint8_t hg_smem_raw[];
@@ -288,13 +303,14 @@ hgemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant_
         // the row ranges are the predecessor's: one warp turns them into item numbers
         pdl_wait();
         if (warp == 0) {
-            int carry = 0;
+            const HgPart& every = p.part[1];
+            int carry = every.T > 0 ? (every.T + BN - 1) / BN * every.row_tiles : 0;
             for (int base = 0; base < p.experts; base += 32) {
                 const int e = base + lane;
                 int lo = 0, n = 0;
                 if (e < p.experts) {
                     lo = p.offsets[e];
-                    n = (p.offsets[e + 1] - lo + BN - 1) / BN * p.row_tiles;
+                    n = (p.offsets[e + 1] - lo + BN - 1) / BN * p.part[0].row_tiles;
                 }
                 int inc = n;
 #pragma unroll
@@ -321,19 +337,28 @@ hgemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant_
     // a few row tiles across every token tile: each weight box comes from HBM once and the activations stay in L2
     auto decode = [&](int item, HgTile& t, int& kb0, int& kb1) {
         if (p.experts > 0) {
-            int e = 0;  // the last expert whose items begin at or before this one, experts without rows have none
-            for (int step = HG_MAX_EXPERTS; step > 0; step >>= 1)
-                if (e + step < p.experts && first_item[e + step] <= item) e += step;
-            const int mn = item - first_item[e], n_tiles = (first_row[e + 1] - first_row[e] + BN - 1) / BN, m_tile = mn / n_tiles;
-            t.w_row = (e * p.row_tiles + m_tile) * HG_BM;
+            int e = 0, first = 0, row = 0, n = p.part[1].T;
+            t.part = item < first_item[0] ? 1 : 0;
+            if (t.part == 0) {
+                // the last expert whose items begin at or before this one; experts without rows have none
+                for (int step = HG_MAX_EXPERTS; step > 0; step >>= 1)
+                    if (e + step < p.experts && first_item[e + step] <= item) e += step;
+                first = first_item[e];
+                row = first_row[e];
+                n = first_row[e + 1] - row;
+            }
+            const HgPart& part = p.part[t.part];
+            const int mn = item - first, n_tiles = (n + BN - 1) / BN, m_tile = mn / n_tiles, each = even_tile(n, BN);
+            t.w_row = (e * part.row_tiles + m_tile) * HG_BM;
             t.row0 = m_tile * HG_BM;
-            t.x_row = t.tok0 = first_row[e] + mn % n_tiles * BN;
-            t.tok_end = first_row[e + 1];
-            t.rows = p.expert_rows;
+            t.x_row = t.tok0 = row + mn % n_tiles * each;
+            t.tok_end = min(row + n, t.tok0 + each);
+            t.rows = part.rows;
             kb0 = 0;
-            kb1 = k_blocks;
+            kb1 = part.k_blocks;
             return;
         }
+        t.part = 0;
         const int mn = item % mn_tiles, split = item / mn_tiles, m_tile = mn / p.n_tiles;
         t.w_row = t.row0 = m_tile * HG_BM;
         t.tok0 = mn % p.n_tiles * BN;
@@ -369,6 +394,15 @@ hgemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant_
                     }
                     uint8_t* a_dst = tiles + (size_t)st * L::STAGE_BYTES;
                     uint8_t* b_dst = a_dst + L::A_BYTES;
+                    if (p.experts > 0) {
+                        // as many activation boxes as the tile has rows for
+                        const int boxes = (max(tile.tok_end - tile.tok0, 1) + p.box_rows - 1) / p.box_rows;
+                        mbar_expect_tx(&full[st], (uint32_t)(L::A_BYTES + boxes * p.box_rows * HG_BK * 2));
+                        tma_load_2d(a_dst, tile.part == 0 ? &tm_w : &tm_w1, kb * HG_BK, tile.w_row, &full[st]);
+                        for (int b = 0; b < boxes; ++b)
+                            tma_load_2d(b_dst + b * p.box_rows * HG_BK * 2, tile.part == 0 ? &tm_x : &tm_x1, kb * HG_BK, tile.x_row + b * p.box_rows, &full[st]);
+                        continue;
+                    }
                     mbar_expect_tx(&full[st], (uint32_t)L::STAGE_BYTES);
                     tma_load_2d(a_dst, &tm_w, kb * HG_BK, tile.w_row, &full[st]);
                     if (waited) {
@@ -388,7 +422,7 @@ hgemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant_
     } else if (warp == 1) {
         // ---- MMA issuer
         if (lane == 0) {
-            const uint32_t idesc = (1u << 4) | (p.bf16 ? (1u << 7) | (1u << 10) : 0u) | ((uint32_t)(BN >> 3) << 17) | ((uint32_t)(HG_BM >> 4) << 24);
+            const uint32_t idesc_wide = (1u << 4) | (p.bf16 ? (1u << 7) | (1u << 10) : 0u) | ((uint32_t)(HG_BM >> 4) << 24);
             uint32_t it = 0, tile_it = 0;
             bool ok = true;
             for (int item = blockIdx.x; item < total_items && ok; item += gridDim.x, ++tile_it) {
@@ -402,6 +436,9 @@ hgemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant_
                 }
                 asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
                 const uint32_t d_tmem = tmem_base + acc * BN;
+                // grouped: no wider than the tile's rows, in steps of 16
+                const uint32_t wide = p.experts > 0 ? (uint32_t)((tile.tok_end - tile.tok0 + 15) & ~15) : (uint32_t)BN;
+                const uint32_t idesc = idesc_wide | ((wide >> 3) << 17);
                 for (int kb = kb0; kb < kb1; ++kb, ++it) {
                     const uint32_t st = it % STAGES, ph = (it / STAGES) & 1;
                     if (!mbar_wait(&full[st], ph, HG_SPIN_LIMIT)) {
@@ -427,7 +464,7 @@ hgemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant_
         // ---- epilogue: warps 2..5 own TMEM lane quadrants (warp % 4)
         const int quad = warp & 3;
         const int etid = (int)threadIdx.x - 64;  // 0..127 among the epilogue threads
-        if (p.act_post != nullptr) pdl_wait();   // the factors of the rows come from a predecessor
+        if (p.part[0].act_post != nullptr) pdl_wait();   // the factors of the rows come from a predecessor
         uint32_t tile_it = 0;
         for (int item = blockIdx.x; item < total_items; item += gridDim.x, ++tile_it) {
             HgTile tile;
@@ -454,8 +491,9 @@ hgemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant_
             asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
             const int row = tile.row0 + quad * 32 + lane;
             const int tok0 = tile.tok0;
-            float* dst = p.splits > 1 ? p.partial + (int64_t)split * p.T * p.rows : p.y;
-            const int ld = p.splits > 1 ? p.rows : p.ldy;
+            const HgPart& part = p.part[tile.part];  // where a whole tile goes and its activation's constants (both forms)
+            float* dst = p.splits > 1 ? p.partial + (int64_t)split * p.T * p.rows : part.y;
+            const int ld = p.splits > 1 ? p.rows : part.ldy;
 #pragma unroll 1
             for (int cb = 0; cb < BN; cb += LD_COLS) {
                 if (tok0 + cb >= tile.tok_end) break;  // uniform over the CTA: nothing but padding from here on
@@ -477,14 +515,14 @@ hgemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant_
                         if (row < tile.rows && tok < tile.tok_end) {
                             float a;
                             if (p.gated == 1 + GatedAct::Clamped) {
-                                const float pre = p.act_pre != nullptr ? p.act_pre[tok] : 1.0f;
-                                a = clamped_gate_f(pre * g, pre * u, p.act_limit);
-                                if (p.act_post != nullptr) a *= p.act_post[tok];
+                                const float pre = part.act_pre != nullptr ? part.act_pre[tok] : 1.0f;
+                                a = clamped_gate_f(pre * g, pre * u, part.act_limit);
+                                if (part.act_post != nullptr) a *= part.act_post[tok];
                             } else {
                                 a = (p.gated == 1 + GatedAct::Silu ? hg_silu(g) : hg_gelu_tanh(g)) * u;
                             }
-                            if (p.bf16) reinterpret_cast<__nv_bfloat16*>(p.yh)[(int64_t)tok * p.ldyh + feature] = __float2bfloat16_rn(a);
-                            else p.yh[(int64_t)tok * p.ldyh + feature] = __float2half_rn(a);
+                            if (p.bf16) reinterpret_cast<__nv_bfloat16*>(part.yh)[(int64_t)tok * part.ldyh + feature] = __float2bfloat16_rn(a);
+                            else part.yh[(int64_t)tok * part.ldyh + feature] = __float2half_rn(a);
                         }
                     }
                 } else if (p.scattered != 0) {
@@ -554,11 +592,17 @@ void encode_half_matrix(CUtensorMap* out, const void* base, int64_t n_rows, int6
 }
 
 template <int BN, int STAGES>
-void launch_hg(const CUtensorMap& tw, const CUtensorMap& tx, const HgParams& p, int grid, cudaStream_t s) {
+void launch_hg(const CUtensorMap& tw, const CUtensorMap& tx, const CUtensorMap& tw1, const CUtensorMap& tx1, const HgParams& p, int grid, cudaStream_t s) {
     constexpr size_t smem = HgSmem<BN, STAGES>::TOTAL;
     ensure_dynamic_smem(reinterpret_cast<const void*>(&hgemm_tc_kernel<BN, STAGES>), smem);
-    launch_pdl(hgemm_tc_kernel<BN, STAGES>, dim3(grid), dim3(HG_THREADS), smem, s, tw, tx, p);
+    launch_pdl(hgemm_tc_kernel<BN, STAGES>, dim3(grid), dim3(HG_THREADS), smem, s, tw, tx, tw1, tx1, p);
     MK_LAUNCH_CHECK();
+}
+
+void launch_hg_width(int bn, const CUtensorMap& tw, const CUtensorMap& tx, const CUtensorMap& tw1, const CUtensorMap& tx1, const HgParams& p, int grid, cudaStream_t s) {
+    if (bn == 256) launch_hg<256, 4>(tw, tx, tw1, tx1, p, grid, s);
+    else if (bn == 128) launch_hg<128, 6>(tw, tx, tw1, tx1, p, grid, s);
+    else launch_hg<64, 8>(tw, tx, tw1, tx1, p, grid, s);
 }
 
 }  // namespace
@@ -707,7 +751,7 @@ HgemmPlan hgemm_tc_plan(int64_t rows, int64_t cols, int T, int max_splits) {
 namespace {
 int launch_hgemm_any(const HalfWeight& W, const __half* xh, int T, float* y, int ldy, float out_scale, float softcap,
                      const HgemmScratch& ws, cudaStream_t s, int max_splits, const GatedAct* act, __half* yh, int ldyh,
-                     const MatmulScatter* scatter = nullptr, const ExpertRows* experts = nullptr);
+                     const MatmulScatter* scatter = nullptr);
 }
 
 int launch_hgemm_tc(const HalfWeight& W, const __half* xh, int T, float* y, int ldy, float out_scale, float softcap,
@@ -726,45 +770,92 @@ void launch_hgemm_tc_gated(const HalfWeight& W, const __half* xh, int T, const G
     launch_hgemm_any(W, xh, T, nullptr, 0, 1.0f, 0.f, ws, s, 1, &act, yh, ldyh);
 }
 
-void launch_hgemm_tc_experts(const HalfWeight& W, const ExpertRows& experts, const __half* xh, int T, float* y, int ldy, const GatedAct* act, __half* yh,
-                             int ldyh, const HgemmScratch& ws, cudaStream_t s) {
-    if (experts.experts <= 0 || experts.experts > HG_MAX_EXPERTS || experts.offsets == nullptr || experts.rows_padded % HG_BM != 0 ||
-        W.rows != (int64_t)experts.experts * experts.rows_padded || W.n_groups != 1)
-        throw std::runtime_error("launch_hgemm_tc_experts: at most 1024 experts of whole 128-row tiles");
-    if ((act != nullptr) != (yh != nullptr)) throw std::runtime_error("launch_hgemm_tc_experts: the gated form writes its own output");
-    launch_hgemm_any(W, xh, T, y, ldy, 1.0f, 0.f, ws, s, 1, act, yh, ldyh, nullptr, &experts);
+void launch_hgemm_tc_experts(const ExpertRows& experts, const ExpertRows* every, const HgemmScratch& ws, cudaStream_t s) {
+    if (experts.experts <= 0 || experts.experts > HG_MAX_EXPERTS || experts.offsets == nullptr) throw std::runtime_error("launch_hgemm_tc_experts: 1 to 1024 experts");
+    if (experts.T <= 0) return;
+    HgParams p{};
+    CUtensorMap tx[2];
+    const CUtensorMap* tw[2] = {};
+    int most_items = 0;
+    // token tiles about as wide as an expert has rows
+    const int mean = (experts.T + experts.experts - 1) / experts.experts;
+    const int bn = mean <= 48 ? 64 : (mean <= 160 ? 128 : 256);
+    p.box_rows = bn == 64 ? 16 : 64;
+    for (int i = 0; i < 2; ++i) {
+        const ExpertRows* e = i == 0 ? &experts : every;
+        if (e == nullptr) {
+            tw[1] = tw[0];
+            tx[1] = tx[0];
+            continue;
+        }
+        const HalfWeight& W = *e->W;
+        if (!W.ready || e->xh == nullptr || e->rows_padded % HG_BM != 0 || W.rows != (int64_t)e->experts * e->rows_padded || W.n_groups != 1)
+            throw std::runtime_error("launch_hgemm_tc_experts: matrices of whole 128-row tiles and their rows");
+        if ((e->act != nullptr) != (e->yh != nullptr) || (experts.act != nullptr) != (e->act != nullptr) || W.bf16 != experts.W->bf16 || (i == 1 && e->experts != 1))
+            throw std::runtime_error("launch_hgemm_tc_experts: the two parts differ in form");
+        tw[i] = reinterpret_cast<const CUtensorMap*>(W.tmap);
+        encode_half_matrix(&tx[i], e->xh, e->T, W.cols, p.box_rows, W.bf16);
+        HgPart& part = p.part[i];
+        part.row_tiles = e->rows_padded / HG_BM;
+        part.rows = e->rows;
+        part.T = i == 1 ? e->T : 0;
+        part.k_blocks = (int)(W.cols / HG_BK);
+        part.y = e->y;
+        part.ldy = e->ldy;
+        part.yh = e->yh;
+        part.ldyh = e->ldyh;
+        if (e->act != nullptr) {
+            part.act_limit = e->act->limit;
+            part.act_pre = e->act->pre;
+            part.act_post = e->act->post;
+        }
+        most_items += part.row_tiles * (std::min(e->T, e->experts) + e->T / bn);
+    }
+    p.T = experts.T;
+    p.K = (int)experts.W->cols;
+    p.rows = (int)experts.W->rows;
+    p.out_scale = 1.f;
+    p.row_tiles = p.part[0].row_tiles;
+    p.n_tiles = 1;
+    p.splits = 1;
+    p.kb_per_split = p.part[0].k_blocks;
+    p.status = ws.status;
+    p.gated = experts.act != nullptr ? 1 + experts.act->kind : 0;
+    p.bf16 = experts.W->bf16 ? 1 : 0;
+    p.n_groups = 1;
+    p.experts = experts.experts;
+    p.offsets = experts.offsets;
+    launch_hg_width(bn, *tw[0], tx[0], *tw[1], tx[1], p, std::min(device_sm_count(), most_items), s);
 }
 
 namespace {
 int launch_hgemm_any(const HalfWeight& W, const __half* xh, int T, float* y, int ldy, float out_scale, float softcap,
                      const HgemmScratch& ws, cudaStream_t s, int max_splits, const GatedAct* act, __half* yh, int ldyh,
-                     const MatmulScatter* scatter, const ExpertRows* experts) {
+                     const MatmulScatter* scatter) {
     if (T <= 0) return 1;
     if (!W.ready) throw std::runtime_error("launch_hgemm_tc: the f16 image of the matrix was not built");
     if (xh == nullptr) throw std::runtime_error("launch_hgemm_tc: f16 activations missing");
     if (out_scale != 1.0f || softcap != 0.f || ws.partial == nullptr) max_splits = 1;
     HgemmPlan pl = hgemm_tc_plan(W.rows, W.cols, T, max_splits);
-    if (experts != nullptr) {
-        // token tiles about as wide as an expert has rows: what lies behind them belongs to the next one and is computed for nothing
-        const int mean = (T + experts->experts - 1) / experts->experts;
-        pl.bn = mean <= 48 ? 64 : (mean <= 160 ? 128 : 256);
-        pl.row_tiles = experts->rows_padded / HG_BM;
-        pl.n_tiles = 1;
-        pl.splits = 1;
-        pl.kb_per_split = (int)(W.cols / HG_BK);
-    }
     if (pl.splits > 1 && pl.partial_floats > ws.partial_floats) {
         pl.splits = 1;
         pl.kb_per_split = (int)(W.cols / HG_BK);
     }
     alignas(64) CUtensorMap tx;
     encode_half_matrix(&tx, xh, (int64_t)T * W.n_groups, W.cols, pl.bn, W.bf16);
-    HgParams p;
+    HgParams p{};
     p.T = T;
     p.K = (int)W.cols;
     p.rows = (int)W.rows;
-    p.y = y;
-    p.ldy = ldy;
+    p.part[0].y = y;
+    p.part[0].ldy = ldy;
+    p.part[0].yh = yh;
+    p.part[0].ldyh = ldyh;
+    if (act != nullptr) {
+        p.part[0].act_limit = act->limit;
+        p.part[0].act_pre = act->pre;
+        p.part[0].act_post = act->post;
+    }
     p.out_scale = out_scale;
     p.softcap = softcap;
     p.row_tiles = pl.row_tiles;
@@ -774,26 +865,15 @@ int launch_hgemm_any(const HalfWeight& W, const __half* xh, int T, float* y, int
     p.partial = ws.partial;
     p.status = ws.status;
     p.gated = act != nullptr ? 1 + act->kind : 0;
-    p.act_limit = act != nullptr ? act->limit : 0.f;
-    p.act_pre = act != nullptr ? act->pre : nullptr;
-    p.act_post = act != nullptr ? act->post : nullptr;
-    p.experts = experts != nullptr ? experts->experts : 0;
-    p.expert_rows = experts != nullptr ? experts->rows : 0;
-    p.offsets = experts != nullptr ? experts->offsets : nullptr;
-    p.yh = yh;
-    p.ldyh = ldyh;
     p.bf16 = W.bf16 ? 1 : 0;
     p.n_groups = W.n_groups;
     for (int g = 0; g < kMaxRowGroups; ++g) p.group_end[g] = W.group_end[g];
     p.group_tiles = W.group_tiles;
     p.scattered = scatter != nullptr ? 1 : 0;
     if (scatter != nullptr) p.scatter = *scatter;
-    const int most_items = experts != nullptr ? p.row_tiles * (std::min(T, experts->experts) + T / pl.bn) : p.row_tiles * p.n_tiles * p.splits;
-    const int grid = std::min(device_sm_count(), most_items);
+    const int grid = std::min(device_sm_count(), p.row_tiles * p.n_tiles * p.splits);
     const CUtensorMap& tw = *reinterpret_cast<const CUtensorMap*>(W.tmap);
-    if (pl.bn == 256) launch_hg<256, 4>(tw, tx, p, grid, s);
-    else if (pl.bn == 128) launch_hg<128, 6>(tw, tx, p, grid, s);
-    else launch_hg<64, 8>(tw, tx, p, grid, s);
+    launch_hg_width(pl.bn, tw, tx, tw, tx, p, grid, s);
     return pl.splits;
 }
 }  // namespace

@@ -74,10 +74,18 @@ void launch_hgemm_tc_gated(const HalfWeight& W, const __half* xh, int T, const G
 // count); rows [offsets[e], offsets[e + 1]) of xh [T][cols] and of the result meet expert e's.  The ranges are read on the device.
 // With `act` the matrices are interleaved gate/up rows and the result is yh (act->pre / post by grouped row), else y.
 struct ExpertRows {
+    const HalfWeight* W = nullptr;
     int experts = 0, rows_padded = 0, rows = 0;
     const int32_t* offsets = nullptr;  // device, [experts + 1]
+    const __half* xh = nullptr;
+    int T = 0;                         // rows of all experts
+    float* y = nullptr;
+    int ldy = 0;
+    const GatedAct* act = nullptr;
+    __half* yh = nullptr;
+    int ldyh = 0;
 };
-void launch_hgemm_tc_experts(const HalfWeight& W, const ExpertRows& experts, const __half* xh, int T, float* y, int ldy, const GatedAct* act, __half* yh,
-                             int ldyh, const HgemmScratch& ws, cudaStream_t s);
+// `every` (optional): one more matrix in the same launch, which all its T rows meet (experts = 1, no offsets).
+void launch_hgemm_tc_experts(const ExpertRows& experts, const ExpertRows* every, const HgemmScratch& ws, cudaStream_t s);
 
 }  // namespace mk

@@ -102,8 +102,8 @@ struct Ls {
     static constexpr int COLS = 32 / KS * 2;                 // value columns of a warp
     static constexpr int TT = FINISH ? 4 : 16;               // rows of a chunk
     static constexpr int KROWS = WKV ? 3 : 2;                // r, k, decay  /  q, k
-    static constexpr int MAX_THREADS = FINISH ? (LS_MAX_FINISH_V / COLS + EXTRA) * 32 : LS_WIDE_WARPS * 32;
-    static constexpr int MIN_CTAS = FINISH ? (KD >= 128 ? 2 : 3) - EXTRA : 1;
+    static constexpr int MAX_THREADS = FINISH ? LS_MAX_FINISH_V / COLS * 32 : LS_WIDE_WARPS * 32;
+    static constexpr int MIN_CTAS = FINISH ? (KD >= 128 ? 2 : 3) : 1;
     // stage: KROWS key-wide rows, the value row, the gate row (FINISH), decay, write and floor of the denominator (not WKV)
     static __host__ __device__ constexpr int row_floats(int cols) { return KROWS * KD + cols * (FINISH ? 2 : 1) + (WKV ? 0 : 4); }
     static __host__ __device__ constexpr int stage_floats(int cols) { return TT * row_floats(cols); }
@@ -357,18 +357,13 @@ linear_state_kernel(const __grid_constant__ typename LsArgs<RULE>::type ra) {
                     step(r, part[2 * i], part[2 * i + 1]);
                 }
             }
-            float o = fold8<KS>(part, ks);
+            const float o = fold8<KS>(part, ks);
             const int t = ks >> 1, c = c_loc + (ks & 1);
-            if (RULE == LS_MLSTM) {
-                o *= q_scale;
-                if (c == a.vdim && t < m) o = fmaxf(fabsf(o), s_c[4 * t + 2]) + 1e-6f;
-            }
-            if (t < m && c < state_cols) s_o[t * cols + c] = o;
+            if (t < m && c < a.vdim) s_o[t * cols + c] = o;
             __syncthreads();
             const float* s_g = s_v + TT * cols;
             for (int t = warp; t < m; t += (int)(blockDim.x >> 5))
-                finish_head_row(a, s_o + t * cols, RULE == LS_MLSTM ? s_o[t * cols + a.vdim] : 1.f, [&](int v) { return s_g[t * cols + v]; }, s_nw,
-                                first + ch * TT + t, head, lane);
+                finish_head_row(a, s_o + t * cols, 1.f, [&](int v) { return s_g[t * cols + v]; }, s_nw, first + ch * TT + t, head, lane);
             __syncthreads();  // the stage is free for the chunk after next
         } else {
             Row rows[2];
@@ -475,10 +470,19 @@ void launch_scan(const typename LsArgs<RULE>::type& ra, cudaStream_t s) {
     if (a.heads > 65535 || a.lanes.lanes > 65535) throw std::runtime_error("linear-attention scan: at most 65535 heads and lanes");
     const bool finish = a.image.h != nullptr || a.image.f != nullptr;
     if (finish && !linear_state_can_finish(a.dim, a.vdim)) throw std::runtime_error("linear-attention scan: the finishing form takes dimensions up to 128");
-    switch (linear_state_key_pad(a.dim)) {
-        case 32: finish ? launch_variant<32, RULE, true>(ra, s) : launch_variant<32, RULE, false>(ra, s); break;
-        case 64: finish ? launch_variant<64, RULE, true>(ra, s) : launch_variant<64, RULE, false>(ra, s); break;
-        case 128: finish ? launch_variant<128, RULE, true>(ra, s) : launch_variant<128, RULE, false>(ra, s); break;
+    const int pad = linear_state_key_pad(a.dim);
+    if constexpr (RULE != LS_MLSTM) {
+        if (finish) {
+            if (pad == 32) launch_variant<32, RULE, true>(ra, s);
+            else if (pad == 64) launch_variant<64, RULE, true>(ra, s);
+            else launch_variant<128, RULE, true>(ra, s);
+            return;
+        }
+    }
+    switch (pad) {
+        case 32: launch_variant<32, RULE, false>(ra, s); break;
+        case 64: launch_variant<64, RULE, false>(ra, s); break;
+        case 128: launch_variant<128, RULE, false>(ra, s); break;
         default: launch_variant<256, RULE, false>(ra, s); break;
     }
 }
@@ -495,7 +499,23 @@ bool linear_state_can_finish(int dim, int vdim) { return dim <= 128 && vdim <= L
 
 void launch_wkv_scan(const WkvScanArgs& a, cudaStream_t s) { launch_scan<LS_WKV>(a, s); }
 
-void launch_mlstm_scan(const MlstmScanArgs& a, cudaStream_t s) { launch_scan<LS_MLSTM>(a, s); }
+int launch_mlstm_scan(const MlstmScanArgs& a, cudaStream_t s) {
+    if (a.longest <= 1) {
+        launch_mlstm_step(a, s);
+        return 1;
+    }
+    MlstmScanArgs raw = a;
+    raw.common.image = RowImage{};
+    LinearStateArgs finish = a.common;
+    if (a.tensor_cores != 0) {
+        launch_mlstm_chunks(raw, s);
+    } else {
+        launch_scan<LS_MLSTM>(raw, s);
+        finish.normalised = 1;
+    }
+    launch_head_norm_gate(finish, a.rows, s);
+    return 2;
+}
 
 void launch_delta_scan(const DeltaScanArgs& a, cudaStream_t s) {
     if (a.kv_heads <= 0 || a.common.heads % a.kv_heads != 0) throw std::runtime_error("delta-rule scan: heads must be a multiple of kv_heads");

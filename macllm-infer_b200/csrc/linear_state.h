@@ -64,8 +64,15 @@ struct MlstmScanArgs {
     const float* f_bias = nullptr;
     float cap = 1.f;
     float* running_max = nullptr;    // [slot halves][heads]
+    int32_t* counters = nullptr;     // [lanes][heads], zero before the first call; every call leaves them zero
+    int rows = 0, longest = 0;       // of all lanes, of the longest one
+    int tensor_cores = 0;            // prompts as products of 64-row chunks, else row by row in f32; queries, keys and values are rounded to bfloat16
 };
-void launch_mlstm_scan(const MlstmScanArgs& a, cudaStream_t s);
+// Always finishes (common.image is set, common.out is scratch).  Returns the number of kernels launched.
+int launch_mlstm_scan(const MlstmScanArgs& a, cudaStream_t s);
+// The forms behind it (mlstm.cu): one-token lanes, finished; chunks of prompts, whose raw rows are [heads][vdim] and divided already.
+void launch_mlstm_step(const MlstmScanArgs& a, cudaStream_t s);
+void launch_mlstm_chunks(const MlstmScanArgs& a, cudaStream_t s);
 
 // Whether the finishing form (LinearStateArgs::image) exists for these sizes.
 bool linear_state_can_finish(int dim, int vdim);

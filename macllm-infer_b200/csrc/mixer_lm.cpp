@@ -13,7 +13,7 @@ namespace {
 
 const std::vector<const char*> class_names = {"hgemm_tc", "hgemm_tc_splitk", "f32_matmul", "wkv_scan", "delta_scan", "paged_attention", "rope_kv_scatter",
                                               "row_update", "delta_prep", "wkv_decay", "latent_attention", "mingru_scan", "latent_prep", "latent_rows",
-                                              "mlstm_scan", "moe_gemm", "moe_rows", "gates", "embed", "build_batch", "argmax"};
+                                              "mlstm_scan", "moe_gemm", "moe_route", "moe_gather", "gates", "embed", "build_batch", "argmax"};
 
 bool is_mixer_checkpoint(const std::string& dir) {
     struct stat st;
@@ -341,6 +341,7 @@ void MixerLm::alloc_activations() {
     int64_t q_lat = 0, uq = 0, lat = 0, cat = 0;  // widths of latent attention's rows, and of `out`'s input with both branches
     int lat_ctas = 1;
     int64_t lat_part = 0;
+    int64_t mlstm_heads = 0;
     int64_t pairs = 0, experts = 0, expert_ff = 0, expert_gu = 0;  // routed rows, experts, widths of an expert's activations
     for (size_t l = 0; l < lw_.size(); ++l) {
         const MixerLayerSpec& s = ms_.layers[l];
@@ -354,6 +355,7 @@ void MixerLm::alloc_activations() {
             expert_gu = std::max(expert_gu, w.experts_gu.rows / std::max(1, s.moe.experts));
         }
         if (s.kind == MixerKind::Mlstm) {
+            mlstm_heads = std::max(mlstm_heads, (int64_t)s.mlstm.heads);
             b_w = std::max(b_w, (int64_t)s.mlstm.heads * s.mlstm.vdim);
             raw = std::max(raw, (int64_t)s.mlstm.heads * linear_state_raw_width(s.mlstm.vdim));
         } else if (s.kind == MixerKind::Attention) {
@@ -361,7 +363,7 @@ void MixerLm::alloc_activations() {
             attn = std::max(attn, (int64_t)s.attn.heads * w.row_width);
         }
         if (ms_.norm_place == NormPlace::Output) {
-            ff = std::max(ff, (int64_t)s.moe.shared_ff);
+            ff = std::max(ff, (int64_t)pad_to(s.moe.shared_ff, 64));
             continue;
         }
         if (ms_.side_by_side()) {
@@ -410,15 +412,20 @@ void MixerLm::alloc_activations() {
     y_a_.alloc((size_t)(T * C) * 4);
     y_b_.alloc((size_t)(T * C) * 4);
     if (f32_) y_gu_.alloc((size_t)std::max(T * 2 * ff, pairs * expert_gu) * 4);
+    mlstm_counters_.alloc((size_t)(B * mlstm_heads) * 4);
+    mlstm_counters_.zero(stream_);
     if (pairs > 0) {
         img_rows_.alloc((size_t)(pairs * ldc) * esz_);
         img_expert_ff_.alloc((size_t)(pairs * expert_ff) * esz_);
-        routed_.alloc((size_t)(pairs * C) * 4);
-        moe_words_.alloc((size_t)(5 * pairs + experts + 1 + T) * 4);
+        routed_.alloc((size_t)((pairs + T) * C) * 4);
+        moe_words_.alloc((size_t)(5 * pairs + 3 * experts + 1 + T) * 4);
+        moe_words_.zero(stream_);  // the counts
         moe_.sel = moe_words_.as<int32_t>();
-        moe_.pos_of_pair = moe_.sel + pairs;
-        moe_.token_of_pos = moe_.pos_of_pair + pairs;
-        moe_.offsets = moe_.token_of_pos + pairs;
+        moe_.rank = moe_.sel + pairs;
+        moe_.pos_of_pair = moe_.rank + pairs;
+        moe_.count = moe_.pos_of_pair + pairs;
+        moe_.counts = (int)experts;
+        moe_.offsets = moe_.count + 2 * experts;
         moe_.weight = reinterpret_cast<float*>(moe_.offsets + experts + 1);
         moe_.weight_of_pos = moe_.weight + pairs;
         moe_.shared_gate = moe_.weight_of_pos + pairs;

@@ -125,7 +125,7 @@ private:
         DevBuf cos_t, sin_t;
     };
     enum KClass { KC_GEMM = 0, KC_GEMM_NARROW, KC_F32_MATMUL, KC_WKV_SCAN, KC_DELTA_SCAN, KC_ATTN, KC_ROPE_KV, KC_ROW_UPDATE, KC_DELTA_PREP, KC_WKV_DECAY,
-                  KC_LATENT_ATTN, KC_MINGRU, KC_LATENT_PREP, KC_LATENT_ROWS, KC_MLSTM_SCAN, KC_MOE_GEMM, KC_MOE_ROWS, KC_GATES, KC_EMBED, KC_BATCH,
+                  KC_LATENT_ATTN, KC_MINGRU, KC_LATENT_PREP, KC_LATENT_ROWS, KC_MLSTM_SCAN, KC_MOE_GEMM, KC_MOE_ROUTE, KC_MOE_GATHER, KC_GATES, KC_EMBED, KC_BATCH,
                   KC_SAMPLE, KC_COUNT };
 
     void load(const SafetensorsFile& f);
@@ -205,7 +205,9 @@ private:
     DevBuf partial_[3];
     // mixture of experts: the tick's routing, rows grouped by expert, their activations and results
     MoeRows moe_;
+    int moe_half_ = 0;  // of the counts, alternates from layer to layer
     DevBuf moe_words_, img_rows_, img_expert_ff_, routed_;
+    DevBuf mlstm_counters_;
     DevBuf attn_part_o_, attn_part_ml_, attn_counters_;
     int attn_max_entries_ = 0;
     int cur_ = 0;             // which of x_ holds the residual stream

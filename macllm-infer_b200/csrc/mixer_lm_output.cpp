@@ -83,8 +83,8 @@ void MixerLm::load_moe(const SafetensorsFile& f, int l) {
     upload_dense(f, gate_up, (int64_t)s.experts * gu, C, w.experts_gu, {}, share);
     upload_dense(f, downs, (int64_t)s.experts * down, s.ff, w.experts_down, {}, share);
     if (s.shared_ff > 0) {
-        upload_dense(f, {{m + "shared.gate", s.shared_ff, 0, 2}, {m + "shared.up", s.shared_ff, 1, 2}}, 2 * (int64_t)s.shared_ff, C, w.gate_up);
-        upload_dense(f, {{m + "shared.down", C, 0}}, C, s.shared_ff, w.down);
+        upload_dense(f, {{m + "shared.gate", s.shared_ff, 0, 2}, {m + "shared.up", s.shared_ff, 1, 2}}, pad_to(2 * s.shared_ff, 128), C, w.gate_up);
+        upload_dense(f, {{m + "shared.down", C, 0}}, down, s.shared_ff, w.down);
     }
 }
 
@@ -137,7 +137,6 @@ void MixerLm::run_mlstm(const Tick& t, int run, const Shares& y, const RowImage&
     a.common.dim = s.dim;
     a.common.vdim = s.vdim;
     a.common.out = raw_.as<float>();
-    a.common.normalised = 1;
     a.common.gate_sigmoid = 1;
     a.common.norm_w = w.head_norm.as<float>();
     a.common.norm_per_head = 1;
@@ -154,20 +153,15 @@ void MixerLm::run_mlstm(const Tick& t, int run, const Shares& y, const RowImage&
     a.f_bias = w.f_b.as<float>();
     a.cap = s.gate_cap;
     a.running_max = st.running_max.as<float>();
-    const bool finish = short_lanes_ && linear_state_can_finish(s.dim, s.vdim);
-    if (finish) a.common.image = out;
+    a.common.image = out;
+    a.counters = mlstm_counters_.as<int32_t>();
+    a.rows = T;
+    a.longest = longest_;
+    a.tensor_cores = f32_ ? 0 : 1;
     const double vw = (double)s.heads * s.vdim, kw = (double)s.heads * s.dim;
-    prof_begin(KC_MLSTM_SCAN, 4.0 * T * (2.0 * kw + vw) + T * vw * (finish ? 4.0 + esz_ : 4.0) + 8.0 * t.B * (vw + s.heads) * s.dim, 6.0 * T * vw * s.dim);
-    launch_mlstm_scan(a, stream_);
+    prof_begin(KC_MLSTM_SCAN, 4.0 * T * (2.0 * kw + 2.0 * vw) + T * vw * esz_ + 8.0 * t.B * (vw + s.heads) * s.dim, 6.0 * T * vw * s.dim);
+    launches_ += launch_mlstm_scan(a, stream_);
     prof_end();
-    ++launches_;
-    if (!finish) {
-        a.common.image = out;
-        prof_begin(KC_GATES, T * vw * (8.0 + esz_), 0);
-        launch_head_norm_gate(a.common, T, stream_);
-        prof_end();
-        ++launches_;
-    }
 }
 
 void MixerLm::run_moe(const Tick& t, int layer, Pending& pend) {
@@ -182,77 +176,110 @@ void MixerLm::run_moe(const Tick& t, int layer, Pending& pend) {
     launch_row_update(u, stream_);
     prof_end();
     ++launches_;
-    const Shares z = matmul(w.router, u.raw, T, y_in_, 0);
+    const bool shared = s.shared_ff > 0;
     MoeRows rows = moe_;
-    if (s.shared_ff == 0) rows.shared_gate = nullptr;
-    prof_begin(KC_MOE_ROWS, (double)T * s.experts * 4.0 + 2.0 * P * C * (double)esz_, 0);
-    launches_ += launch_moe_rows(z, T, s.experts, s.top, rows, status_.as<int32_t>(), stream_);
-    launch_moe_gather(f32_ ? (const void*)u.raw.f : (const void*)u.raw.h, T, s.top, (int64_t)w.router.ld * esz_, rows, img_rows_.ptr(), stream_);
+    if (!shared) rows.shared_gate = nullptr;
+    const int half = moe_half_;
+    moe_half_ ^= 1;
+    if (moe_router_is_narrow(T, s.experts, w.router.ld)) {
+        prof_begin(KC_MOE_ROUTE, (double)w.router.bytes + (double)T * C * esz_, 2.0 * T * (double)C * (s.experts + 1));
+        launch_moe_router(u.raw, f32_ ? w.router.f32.ptr() : w.router.half.values.ptr(), T, s.experts, s.top, rows, half, status_.as<int32_t>(), stream_);
+        prof_end();
+    } else {
+        const Shares z = matmul(w.router, u.raw, T, y_in_, 0);
+        prof_begin(KC_MOE_ROUTE, (double)T * (s.experts + 1) * 4.0, 0);
+        launch_moe_route(z, T, s.experts, s.top, rows, half, status_.as<int32_t>(), stream_);
+        prof_end();
+    }
+    prof_begin(KC_MOE_GATHER, (double)(T + P) * C * esz_, 0);
+    launch_moe_gather(f32_ ? (const void*)u.raw.f : (const void*)u.raw.h, T, s.experts, s.top, (int64_t)w.router.ld * esz_, rows, half, img_rows_.ptr(), stream_);
     prof_end();
-    ++launches_;
+    launches_ += 2;
 
-    // experts: a token's weight multiplies what goes in, so the gate and up sums of a grouped row
-    const RowImage in = image(img_rows_, w.experts_gu.ld), act = image(img_expert_ff_, w.experts_down.ld);
-    GatedAct ga;
-    ga.kind = GatedAct::Clamped;
+    // A token's weight multiplies what goes into an expert, so the gate and up sums of a grouped row; the shared expert's gate
+    // multiplies what comes out, so the input of its last matrix.
+    const RowImage in = image(img_rows_, w.experts_gu.ld), act = image(img_expert_ff_, w.experts_down.ld), every = image(img_ff_, shared ? w.down.ld : 64);
+    float* routed = routed_.as<float>();
+    float* of_every = routed + (size_t)P * C;
+    GatedAct ga, gs;
+    ga.kind = gs.kind = GatedAct::Clamped;
     ga.limit = s.limit;
     ga.pre = rows.weight_of_pos;
-    const int gu_rows = pad_to(2 * s.ff, 128), down_rows = pad_to(C, 128);
+    gs.limit = s.shared_limit;
+    gs.post = rows.shared_gate;
+    const int gu_rows = pad_to(2 * s.ff, 128), shared_rows = pad_to(2 * s.shared_ff, 128), down_rows = pad_to(C, 128);
     const double met = std::min<double>(s.experts, P);  // experts with rows, at most
-    const double gu_bytes = (double)w.experts_gu.bytes / s.experts * met, down_bytes = (double)w.experts_down.bytes / s.experts * met;
+    const double gu_bytes = (double)w.experts_gu.bytes / s.experts * met + w.gate_up.bytes, down_bytes = (double)w.experts_down.bytes / s.experts * met + w.down.bytes;
+    const double ff_rows = (double)P * s.ff + (double)T * s.shared_ff;
+    const double gu_io = (double)esz_ * ((P + (shared ? T : 0.0)) * C + ff_rows), down_io = esz_ * ff_rows + 4.0 * (P + (shared ? T : 0.0)) * C;
     if (f32_) {
-        prof_begin(KC_MOE_GEMM, gu_bytes + down_bytes + 4.0 * P * (2.0 * C + 5.0 * s.ff), 6.0 * P * (double)C * s.ff);
-        launch_f32_matmul_experts(w.experts_gu.f32.as<float>(), s.experts, rows.offsets, gu_rows, gu_rows, w.experts_gu.ld, in.f, P, y_gu_.as<float>(), gu_rows, stream_);
+        prof_begin(KC_MOE_GEMM, gu_bytes + down_bytes + gu_io + down_io, 6.0 * C * ff_rows);
         Shares gu;
         gu.p = y_gu_.as<float>();
         gu.ld = gu_rows;
+        launch_f32_matmul_experts(w.experts_gu.f32.as<float>(), s.experts, rows.offsets, gu_rows, gu_rows, w.experts_gu.ld, in.f, P, y_gu_.as<float>(), gu_rows, stream_);
         launch_gated_act(gu, P, s.ff, act, stream_, ga);
-        launch_f32_matmul_experts(w.experts_down.f32.as<float>(), s.experts, rows.offsets, C, down_rows, w.experts_down.ld, act.f, P, routed_.as<float>(), C, stream_);
-        prof_end();
+        launch_f32_matmul_experts(w.experts_down.f32.as<float>(), s.experts, rows.offsets, C, down_rows, w.experts_down.ld, act.f, P, routed, C, stream_);
         launches_ += 3;
+        if (shared) {
+            gu.ld = shared_rows;
+            launch_f32_matmul(w.gate_up.f32.as<float>(), shared_rows, w.gate_up.ld, u.raw.f, T, y_gu_.as<float>(), shared_rows, 1, nullptr, stream_);
+            launch_gated_act(gu, T, s.shared_ff, every, stream_, gs);
+            launch_f32_matmul(w.down.f32.as<float>(), C, w.down.ld, every.f, T, of_every, C, 1, nullptr, stream_);
+            launches_ += 3;
+        }
+        prof_end();
     } else {
         HgemmScratch ws;
         ws.status = status_.as<int32_t>();
-        ExpertRows er;
+        ExpertRows er, es;  // the experts; beside them the one every token runs
+        er.W = &w.experts_gu.half;
         er.experts = s.experts;
-        er.offsets = rows.offsets;
         er.rows = er.rows_padded = gu_rows;
-        prof_begin(KC_MOE_GEMM, gu_bytes + 2.0 * P * (C + s.ff), 4.0 * P * (double)C * s.ff);
-        launch_hgemm_tc_experts(w.experts_gu.half, er, reinterpret_cast<const __half*>(in.h), P, nullptr, 0, &ga, reinterpret_cast<__half*>(act.h), act.ld, ws, stream_);
+        er.offsets = rows.offsets;
+        er.xh = reinterpret_cast<const __half*>(in.h);
+        er.T = P;
+        er.act = &ga;
+        er.yh = reinterpret_cast<__half*>(act.h);
+        er.ldyh = act.ld;
+        es.W = &w.gate_up.half;
+        es.experts = 1;
+        es.rows = es.rows_padded = shared_rows;
+        es.xh = reinterpret_cast<const __half*>(u.raw.h);
+        es.T = T;
+        es.act = &gs;
+        es.yh = reinterpret_cast<__half*>(every.h);
+        es.ldyh = every.ld;
+        prof_begin(KC_MOE_GEMM, gu_bytes + gu_io, 4.0 * C * ff_rows);
+        launch_hgemm_tc_experts(er, shared ? &es : nullptr, ws, stream_);
         prof_end();
-        er.rows = C;
-        er.rows_padded = down_rows;
-        prof_begin(KC_MOE_GEMM, down_bytes + P * (2.0 * s.ff + 4.0 * C), 2.0 * P * (double)C * s.ff);
-        launch_hgemm_tc_experts(w.experts_down.half, er, reinterpret_cast<const __half*>(act.h), P, routed_.as<float>(), C, nullptr, nullptr, 0, ws, stream_);
+        er.W = &w.experts_down.half;
+        er.xh = er.yh;
+        er.y = routed;
+        es.W = &w.down.half;
+        es.xh = es.yh;
+        es.y = of_every;
+        for (ExpertRows* e : {&er, &es}) {
+            e->rows = C;
+            e->rows_padded = down_rows;
+            e->ldy = C;
+            e->act = nullptr;
+            e->yh = nullptr;
+        }
+        prof_begin(KC_MOE_GEMM, down_bytes + down_io, 2.0 * C * ff_rows);
+        launch_hgemm_tc_experts(er, shared ? &es : nullptr, ws, stream_);
         prof_end();
         launches_ += 2;
     }
     pend.n = 1;
+    if (shared) {
+        pend.y[0].p = of_every;
+        pend.y[0].ld = C;
+    }
     pend.routed_at = rows.pos_of_pair;
     pend.routed_k = s.top;
     pend.w[0] = w.norm2.w.as<float>();
     pend.coef = ms_.residual_mult;
-    if (s.shared_ff == 0) return;
-
-    // the expert every token runs, times its gate
-    const RowImage img = image(img_ff_, w.down.ld);
-    ga.limit = s.shared_limit;
-    ga.pre = nullptr;
-    ga.post = rows.shared_gate;
-    if (f32_) {
-        const Shares gu = matmul(w.gate_up, u.raw, T, y_gu_, 0);
-        prof_begin(KC_GATES, 12.0 * T * s.shared_ff, 0);
-        launch_gated_act(gu, T, s.shared_ff, img, stream_, ga);
-        prof_end();
-    } else {
-        prof_begin(T <= 64 ? KC_GEMM_NARROW : KC_GEMM, (double)w.gate_up.bytes + 2.0 * T * (C + s.shared_ff), 4.0 * T * (double)s.shared_ff * C);
-        HgemmScratch ws;
-        ws.status = status_.as<int32_t>();
-        launch_hgemm_tc_gated(w.gate_up.half, reinterpret_cast<const __half*>(u.raw.h), T, ga, reinterpret_cast<__half*>(img.h), img.ld, ws, stream_);
-        prof_end();
-    }
-    ++launches_;
-    pend.y[0] = matmul(w.down, img, T, y_b_, 2);
 }
 
 }  // namespace mk

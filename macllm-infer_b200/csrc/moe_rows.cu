@@ -1,7 +1,8 @@
 // See moe_rows.h.
 //
-// Narrow ticks route and group in one CTA: a warp takes a token, the choices stay in shared memory, a counting sort gives every
-// pair its row.  Wide ticks route with a warp per token over the whole GPU and group with moe_group_kernel.
+// A token's choices take their places among their expert's rows by counting up; where those rows begin follows from the counts when
+// the rows are gathered.  So two launches route and group a tick of any size.  Places depend on the order in which tokens come to
+// count, results do not: a row meets its expert's matrix wherever it lies.
 #include "moe_rows.h"
 #include "kernels.h"
 #include <climits>
@@ -11,26 +12,28 @@ namespace mk {
 namespace {
 
 constexpr int MR_MAX_EXPERTS = 1024;
-constexpr int MR_PAIRS = 1024;    // pairs of a tick that one CTA routes and groups
 constexpr int MR_MAX_TOP = 32;
+constexpr int MR_THREADS = 256;
 
-// One token by one warp: fn(choice, expert, weight) from lane 0, best first.
-template <typename Fn>
-__device__ __forceinline__ void route_token(const Shares& logits, int t, int experts, int k, float* shared_gate, int32_t* status, int lane, Fn fn) {
+// One token by one warp; logit(e) is valid up to `experts` (the shared expert's gate).
+template <typename Logit>
+__device__ __forceinline__ void route_token(Logit logit, int t, int experts, int k, const MoeRows& r, int half, int32_t* status, int lane) {
     float v[MR_MAX_EXPERTS / 32];
     int cnt = 0;
     bool bad = false;
     for (int e = lane; e < experts; e += 32) {
-        float x = logits.at(t, e);
+        float x = logit(e);
         if (!isfinite(x)) {
             bad = true;
             x = -3.402823466e38f;
         }
         v[cnt++] = x;
     }
-    if (lane == 0 && shared_gate != nullptr) shared_gate[t] = sigmoid_f(logits.at(t, experts));
+    if (lane == 0 && r.shared_gate != nullptr) r.shared_gate[t] = sigmoid_f(logit(experts));
     if (__any_sync(0xffffffffu, bad) && lane == 0) atomicCAS(status, 0, kMoeRouteStatus | (t & 0xFFFF));
     unsigned taken = 0;  // bit c: this lane's c-th expert was chosen
+    float my_logit = 0.f;
+    int mine = 0;        // lane i keeps choice i
     for (int i = 0; i < k; ++i) {
         float bv = -INFINITY;
         int be = INT_MAX;
@@ -49,104 +52,147 @@ __device__ __forceinline__ void route_token(const Shares& logits, int t, int exp
             }
         }
         if ((be & 31) == lane) taken |= 1u << (be >> 5);
-        if (lane == 0) fn(i, be, sigmoid_f(bv));
+        if (lane == i) {
+            my_logit = bv;
+            mine = be;
+        }
+    }
+    if (lane < k) {
+        const int64_t p = (int64_t)t * k + lane;
+        r.sel[p] = mine;
+        r.weight[p] = sigmoid_f(my_logit);
+        r.rank[p] = atomicAdd(r.count + half * r.counts + mine, 1);
     }
 }
 
-__global__ void __launch_bounds__(128) moe_route_rows_kernel(Shares logits, int T, int experts, int k, MoeRows r, int32_t* status) {
+__global__ void __launch_bounds__(128) moe_route_rows_kernel(Shares logits, int T, int experts, int k, MoeRows r, int half, int32_t* status) {
     pdl_trigger();
     pdl_wait();
     const int t = blockIdx.x * 4 + (threadIdx.x >> 5);
     if (t >= T) return;
-    route_token(logits, t, experts, k, r.shared_gate, status, threadIdx.x & 31, [&](int i, int e, float w) {
-        r.sel[(int64_t)t * k + i] = e;
-        r.weight[(int64_t)t * k + i] = w;
-    });
+    route_token([&](int e) { return logits.at(t, e); }, t, experts, k, r, half, status, threadIdx.x & 31);
 }
 
-__global__ void __launch_bounds__(1024) moe_route_group_kernel(Shares logits, int T, int experts, int k, MoeRows r, int32_t* status) {
-    __shared__ int32_t sel[MR_PAIRS], count[MR_MAX_EXPERTS], start[MR_MAX_EXPERTS + 1];
-    __shared__ float weight[MR_PAIRS];
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, pairs = T * k;
-    for (int e = threadIdx.x; e < experts; e += 1024) count[e] = 0;
+// Eight neighbouring columns.
+__device__ __forceinline__ void load8(const __nv_bfloat16* p, float (&v)[8]) {
+    const uint4 u = *reinterpret_cast<const uint4*>(p);
+    const uint32_t w[4] = {u.x, u.y, u.z, u.w};
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+        v[2 * i] = __uint_as_float(w[i] << 16);
+        v[2 * i + 1] = __uint_as_float(w[i] & 0xffff0000u);
+    }
+}
+__device__ __forceinline__ void load8(const float* p, float (&v)[8]) {
+    const float4 a = reinterpret_cast<const float4*>(p)[0], b = reinterpret_cast<const float4*>(p)[1];
+    v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w;
+    v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
+}
+
+// One CTA per token: a warp per router row, then the first warp routes.  Shared memory: experts + 1 logits.
+template <typename W>
+__global__ void __launch_bounds__(MR_THREADS) moe_router_kernel(RowImage x, const W* __restrict__ w, int experts, int k, MoeRows r, int half, int32_t* status) {
+    extern __shared__ float mr_logit[];
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int64_t t = blockIdx.x;
+    const int ld = x.ld, rows = experts + (r.shared_gate != nullptr ? 1 : 0);
+    const W* row;
+    if constexpr (sizeof(W) == 2) row = x.h + t * ld;
+    else row = x.f + t * ld;
     pdl_trigger();
     pdl_wait();
+    for (int e = warp; e < rows; e += MR_THREADS / 32) {
+        float sum = 0.f;
+#pragma unroll 4
+        for (int c = lane * 8; c < ld; c += 256) {  // ld is a multiple of 64
+            float a[8], b[8];
+            load8(row + c, a);
+            load8(w + (int64_t)e * ld + c, b);
+#pragma unroll
+            for (int i = 0; i < 8; ++i) sum = fmaf(a[i], b[i], sum);
+        }
+        sum = warp_sum(sum);
+        if (lane == 0) mr_logit[e] = sum;
+    }
     __syncthreads();
-    for (int t = warp; t < T; t += 32)
-        route_token(logits, t, experts, k, r.shared_gate, status, lane, [&](int i, int e, float w) {
-            sel[t * k + i] = e;
-            weight[t * k + i] = w;
-            atomicAdd(&count[e], 1);
-        });
-    __syncthreads();
-    if (warp == 0) {  // exclusive scan, 32 experts at a time
+    if (warp == 0) route_token([&](int e) { return mr_logit[e]; }, (int)t, experts, k, r, half, status, lane);
+}
+
+// One CTA per token.
+__global__ void __launch_bounds__(MR_THREADS) moe_gather_kernel(const uint4* x, int experts, int k, int64_t chunks, MoeRows r, int half, uint4* out) {
+    __shared__ int at[MR_MAX_TOP];
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int64_t t = blockIdx.x;
+    pdl_trigger();
+    pdl_wait();
+    const int32_t* count = r.count + half * r.counts;
+    for (int j = warp; j < k; j += MR_THREADS / 32) {
+        const int64_t p = t * k + j;
+        const int e = r.sel[p];
+        int before = 0;
+        for (int i = lane; i < e; i += 32) before += count[i];
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) before += __shfl_xor_sync(0xffffffffu, before, o);
+        if (lane == 0) {
+            const int pos = before + r.rank[p];
+            at[j] = pos;
+            r.pos_of_pair[p] = pos;
+            r.weight_of_pos[pos] = r.weight[p];
+        }
+    }
+    if (t == 0 && warp == MR_THREADS / 32 - 1) {  // where every expert's rows begin; the other half of the counts for the next call
         int carry = 0;
         for (int base = 0; base < experts; base += 32) {
             const int e = base + lane, c = e < experts ? count[e] : 0;
             int inc = c;
 #pragma unroll
             for (int o = 1; o < 32; o <<= 1) {
-                const int x = __shfl_up_sync(0xffffffffu, inc, o);
-                if (lane >= o) inc += x;
+                const int v = __shfl_up_sync(0xffffffffu, inc, o);
+                if (lane >= o) inc += v;
             }
-            if (e < experts) start[e] = carry + inc - c;
+            if (e < experts) r.offsets[e] = carry + inc - c;
             carry += __shfl_sync(0xffffffffu, inc, 31);
         }
-        if (lane == 0) start[experts] = carry;
+        if (lane == 0) r.offsets[experts] = carry;
+        for (int e = lane; e < r.counts; e += 32) r.count[(half ^ 1) * r.counts + e] = 0;
     }
     __syncthreads();
-    for (int e = threadIdx.x; e <= experts; e += 1024) r.offsets[e] = start[e];
-    for (int p = threadIdx.x; p < pairs; p += 1024) {
-        r.sel[p] = sel[p];
-        r.weight[p] = weight[p];
-    }
-    // a pair's place among its expert's pairs is the number of earlier ones
-    const unsigned below = (1u << lane) - 1u;
-    for (int e = warp; e < experts; e += 32) {
-        int pos = start[e];
-        if (count[e] == 0) continue;
-        for (int base = 0; base < pairs; base += 32) {
-            const int p = base + lane;
-            const bool mine = p < pairs && sel[p] == e;
-            const unsigned m = __ballot_sync(0xffffffffu, mine);
-            if (mine) {
-                const int at = pos + __popc(m & below);
-                r.pos_of_pair[p] = at;
-                r.token_of_pos[at] = p / k;
-            }
-            pos += __popc(m);
-        }
+    for (int64_t c = threadIdx.x; c < chunks; c += MR_THREADS) {
+        const uint4 v = x[t * chunks + c];
+        for (int j = 0; j < k; ++j) out[at[j] * chunks + c] = v;
     }
 }
 
-__global__ void __launch_bounds__(128) moe_gather_kernel(const uint4* x, int k, int64_t chunks, MoeRows r, uint4* out) {
-    pdl_trigger();
-    pdl_wait();
-    const int64_t p = blockIdx.x, at = r.pos_of_pair[p], t = p / k;
-    for (int64_t c = threadIdx.x; c < chunks; c += 128) out[at * chunks + c] = x[t * chunks + c];
-    if (threadIdx.x == 0) r.weight_of_pos[at] = r.weight[p];
+void check(int experts, int k) {
+    if (experts <= 0 || experts > MR_MAX_EXPERTS || k <= 0 || k > MR_MAX_TOP || k > experts) throw std::runtime_error("mixture of experts: at most 1024 experts and 32 choices");
 }
 
 }  // namespace
 
-int launch_moe_rows(const Shares& logits, int T, int experts, int k, const MoeRows& rows, int32_t* status, cudaStream_t s) {
-    if (T <= 0) return 0;
-    if (experts > MR_MAX_EXPERTS || k > MR_MAX_TOP || k > experts) throw std::runtime_error("launch_moe_rows: at most 1024 experts and 32 choices");
-    if (T * k <= MR_PAIRS) {
-        launch_pdl(moe_route_group_kernel, dim3(1), dim3(1024), 0, s, logits, T, experts, k, rows, status);
-        MK_LAUNCH_CHECK();
-        return 1;
-    }
-    launch_pdl(moe_route_rows_kernel, dim3((unsigned)((T + 3) / 4)), dim3(128), 0, s, logits, T, experts, k, rows, status);
+void launch_moe_route(const Shares& logits, int T, int experts, int k, const MoeRows& rows, int half, int32_t* status, cudaStream_t s) {
+    if (T <= 0) return;
+    check(experts, k);
+    launch_pdl(moe_route_rows_kernel, dim3((unsigned)((T + 3) / 4)), dim3(128), 0, s, logits, T, experts, k, rows, half, status);
     MK_LAUNCH_CHECK();
-    launch_moe_group(rows.sel, T, k, experts, rows.offsets, rows.pos_of_pair, rows.token_of_pos, s);
-    return 2;
 }
 
-void launch_moe_gather(const void* x, int T, int k, int64_t bytes, const MoeRows& rows, void* out, cudaStream_t s) {
+bool moe_router_is_narrow(int T, int experts, int cols) { return T <= 64 && (int64_t)(experts + 1) * cols <= (int64_t)320 * 1024; }
+
+void launch_moe_router(const RowImage& x, const void* w, int T, int experts, int k, const MoeRows& rows, int half, int32_t* status, cudaStream_t s) {
+    if (T <= 0) return;
+    check(experts, k);
+    const size_t smem = (size_t)(experts + 1) * 4;
+    if (x.h != nullptr)
+        launch_pdl(moe_router_kernel<__nv_bfloat16>, dim3((unsigned)T), dim3(MR_THREADS), smem, s, x, static_cast<const __nv_bfloat16*>(w), experts, k, rows, half, status);
+    else
+        launch_pdl(moe_router_kernel<float>, dim3((unsigned)T), dim3(MR_THREADS), smem, s, x, static_cast<const float*>(w), experts, k, rows, half, status);
+    MK_LAUNCH_CHECK();
+}
+
+void launch_moe_gather(const void* x, int T, int experts, int k, int64_t bytes, const MoeRows& rows, int half, void* out, cudaStream_t s) {
     if (T <= 0) return;
     if (bytes % 16 != 0) throw std::runtime_error("launch_moe_gather: rows must be multiples of 16 bytes");
-    launch_pdl(moe_gather_kernel, dim3((unsigned)(T * k)), dim3(128), 0, s, static_cast<const uint4*>(x), k, bytes / 16, rows, static_cast<uint4*>(out));
+    launch_pdl(moe_gather_kernel, dim3((unsigned)T), dim3(MR_THREADS), 0, s, static_cast<const uint4*>(x), experts, k, bytes / 16, rows, half, static_cast<uint4*>(out));
     MK_LAUNCH_CHECK();
 }
 

@@ -242,7 +242,7 @@ def test_wide_ticks_route_like_narrow_ones(mk, tmp_path, mlp, compute):
 
 def test_every_token_on_one_expert(mk, tmp_path):
     """All rows of a tick meet one expert, and the other experts none."""
-    cfg = mc.tevanex([mc.mlstm(1, 8, 8, mlp=mc.experts(9, 1, 48, 0.8, (30, 0.8)))], width=64, vocab=40)
+    cfg = mc.tevanex([mc.capped_attention(2, 1, 32, 32, 16, 64, mlp=mc.experts(9, 1, 48, 0.8, (30, 0.8)))], width=64, vocab=40)
 
     def change(w):
         w["l0.mlp.router"] *= 0.1
