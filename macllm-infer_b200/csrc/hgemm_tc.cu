@@ -246,6 +246,11 @@ __device__ __forceinline__ float finish_value(float v, const HgParams& p) {
 
 // The activations of the gated feed-forward, as the SwiGLU kernel of quantize.cu computes them.
 __device__ __forceinline__ float hg_silu(float x) { return x / (1.0f + expf(-x)); }
+__device__ __forceinline__ float hg_clamped(float g, float u, float limit) {  // clamped_gate_f to what the 16-bit result needs
+    g = fminf(g, limit);
+    u = fminf(fmaxf(u, -limit), limit);
+    return __fdividef(g, 1.0f + __expf(-1.702f * g)) * (u + 1.0f);
+}
 __device__ __forceinline__ float hg_gelu_tanh(float x) {
     return 0.5f * x * (1.0f + tanhf(0.7978845608028654f * x * (1.0f + 0.044715f * x * x)));
 }
@@ -497,6 +502,12 @@ hgemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant_
 #pragma unroll 1
             for (int cb = 0; cb < BN; cb += LD_COLS) {
                 if (tok0 + cb >= tile.tok_end) break;  // uniform over the CTA: nothing but padding from here on
+                // the factors of the chunk's tokens, one per lane, on their way with the accumulators
+                float pre = 1.0f, post = 1.0f;
+                if (p.gated == 1 + GatedAct::Clamped && tok0 + cb + lane < tile.tok_end) {
+                    if (part.act_pre != nullptr) pre = part.act_pre[tok0 + cb + lane];
+                    if (part.act_post != nullptr) post = part.act_post[tok0 + cb + lane];
+                }
                 uint32_t r[32];
                 tmem_ld32(tmem_base + ((uint32_t)(quad * 32) << 16) + acc * BN + (uint32_t)cb, r);
                 asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
@@ -512,12 +523,11 @@ hgemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant_
                         float g = odd ? theirs : __uint_as_float(r[i]);
                         float u = odd ? __uint_as_float(r[i + 1]) : theirs;
                         int tok = tok0 + cb + i + (odd ? 1 : 0);
+                        const float w_in = __shfl_sync(0xffffffffu, pre, i + (odd ? 1 : 0)), w_out = __shfl_sync(0xffffffffu, post, i + (odd ? 1 : 0));
                         if (row < tile.rows && tok < tile.tok_end) {
                             float a;
                             if (p.gated == 1 + GatedAct::Clamped) {
-                                const float pre = part.act_pre != nullptr ? part.act_pre[tok] : 1.0f;
-                                a = clamped_gate_f(pre * g, pre * u, part.act_limit);
-                                if (part.act_post != nullptr) a *= part.act_post[tok];
+                                a = hg_clamped(w_in * g, w_in * u, part.act_limit) * w_out;
                             } else {
                                 a = (p.gated == 1 + GatedAct::Silu ? hg_silu(g) : hg_gelu_tanh(g)) * u;
                             }

@@ -200,7 +200,7 @@ __global__ void __launch_bounds__(MS_WARPS * 32, 4) mlstm_step_kernel(const __gr
 // ------------------------------------------------------------------------------------------------ prompts
 
 constexpr int MC_ROWS = 64;      // rows of a chunk
-constexpr int MC_WARPS = 8;
+constexpr int MC_WARPS = 16;
 constexpr int MC_THREADS = MC_WARPS * 32;
 
 __device__ __forceinline__ uint32_t mc_smem(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
@@ -226,16 +226,66 @@ __device__ __forceinline__ void mc_split(float x, float y, uint32_t& hi, uint32_
     lo = *reinterpret_cast<const uint32_t*>(&l);
 }
 
+// acc[N] (16 rows x 8 N columns) += A B over 16 STEPS inner indices, B in one or two parts.
+//   a_at(step): fragment of A.  b_at(step, tile): where the tile's 16 inner indices begin, its columns (or, TRANS, its inner indices)
+//   PITCH apart.
+// Pairs of tiles share a load; a single tile takes two steps per load.
+template <int N, int STEPS, bool TRANS, int PITCH, typename A, typename B>
+__device__ __forceinline__ void mc_product(float (&acc)[N][4], int lane, A a_at, B b_at, const __nv_bfloat16* b_hi, const __nv_bfloat16* b_lo) {
+    // lane's row of the four 8 x 8 matrices of a load
+    const int pair = TRANS ? ((lane & 7) + ((lane >> 3) & 1) * 8) * PITCH + (lane >> 4) * 8 : ((lane & 7) + (lane >> 4) * 8) * PITCH + ((lane >> 3) & 1) * 8;
+    const int single = TRANS ? lane * PITCH : (lane & 7) * PITCH + (lane >> 3) * 8;
+    auto load = [&](uint32_t (&r)[4], const __nv_bfloat16* p) {
+        if (TRANS) mc_ldmatrix_t(r, p);
+        else mc_ldmatrix(r, p);
+    };
+    if constexpr (N % 2 == 0) {
+#pragma unroll
+        for (int k = 0; k < STEPS; ++k) {
+            uint32_t af[4], bf[4];
+            a_at(k, af);
+#pragma unroll
+            for (int j = 0; j < N; j += 2) {
+                load(bf, b_hi + b_at(k, j) + pair);
+                mc_mma(acc[j], af, bf[0], bf[1]);
+                mc_mma(acc[j + 1], af, bf[2], bf[3]);
+                if (b_lo != nullptr) {
+                    load(bf, b_lo + b_at(k, j) + pair);
+                    mc_mma(acc[j], af, bf[0], bf[1]);
+                    mc_mma(acc[j + 1], af, bf[2], bf[3]);
+                }
+            }
+        }
+    } else {
+        static_assert(N == 1 && STEPS % 2 == 0, "a single tile takes pairs of steps");
+#pragma unroll
+        for (int k = 0; k < STEPS; k += 2) {
+            uint32_t a0[4], a1[4], bf[4];
+            a_at(k, a0);
+            a_at(k + 1, a1);
+            load(bf, b_hi + b_at(k, 0) + single);
+            mc_mma(acc[0], a0, bf[0], bf[1]);
+            mc_mma(acc[0], a1, bf[2], bf[3]);
+            if (b_lo != nullptr) {
+                load(bf, b_lo + b_at(k, 0) + single);
+                mc_mma(acc[0], a0, bf[0], bf[1]);
+                mc_mma(acc[0], a1, bf[2], bf[3]);
+            }
+        }
+    }
+}
+
 template <int KD, int C>
 struct Chunk {
     static constexpr int KP = KD + 8, CP = C + 8, PP = MC_ROWS + 8;  // padded rows (bfloat16): conflict-free ldmatrix
     static constexpr int COL_GROUPS = C / 16, KEY_GROUPS = MC_WARPS / COL_GROUPS, KEYS = KD / KEY_GROUPS;  // of the state, by warp
+    static constexpr int N_PARTS = MC_THREADS / (KD / 2);            // row groups of the normaliser's sums
     static constexpr bool STAGED = KD <= 128;                        // the next chunk's projections are on their way meanwhile
     static constexpr int HALVES = 2 * MC_ROWS * KP + 3 * MC_ROWS * CP + 2 * MC_ROWS * PP + 2 * C * KP;
-    static constexpr int FLOATS = 11 * MC_ROWS + KD + 4;
+    static constexpr int FLOATS = 12 * MC_ROWS + KD + N_PARTS * KD + 4;
     static constexpr int STAGE = STAGED ? MC_ROWS * (2 * KD + C) : 0;
     static constexpr size_t BYTES = (size_t)HALVES * 2 + (size_t)(FLOATS + STAGE) * 4;
-    static_assert(KEYS % 16 == 0, "a warp takes pairs of key tiles");
+    static_assert(KEYS % 8 == 0 && C % 32 == 0, "whole tiles");
 };
 
 // Grid (column slices of C, heads, lanes).
@@ -243,7 +293,7 @@ template <int KD, int C>
 __global__ void __launch_bounds__(MC_THREADS, 1) mlstm_chunk_kernel(const __grid_constant__ MlstmScanArgs a, int vec) {
     using P = Chunk<KD, C>;
     constexpr int KP = P::KP, CP = P::CP, PP = P::PP, R = MC_ROWS;
-    constexpr int NT = C / 16;            // output tiles of a warp: 16 rows x C / 2 columns
+    constexpr int NT = C / 32;            // output tiles of a warp: 16 rows x C / 4 columns
     constexpr int NK = P::KEYS / 8;       // state tiles of a warp: 16 columns x KEYS keys
     extern __shared__ __align__(16) unsigned char mc_raw[];
     __nv_bfloat16* Q = reinterpret_cast<__nv_bfloat16*>(mc_raw);   // [R][KP]
@@ -255,9 +305,10 @@ __global__ void __launch_bounds__(MC_THREADS, 1) mlstm_chunk_kernel(const __grid
     __nv_bfloat16* Pl = Ph + R * PP;
     __nv_bfloat16* Sh = Pl + R * PP;                                // the state the chunk starts from, [C][KP] in two parts
     __nv_bfloat16* Sl = Sh + C * KP;
-    float* c_hi = reinterpret_cast<float*>(Sl + C * KP);            // c_s and e_t in two parts each
-    float *c_lo = c_hi + R, *e_hi = c_lo + R, *e_lo = e_hi + R, *s_g = e_lo + R, *s_w = s_g + R, *s_floor = s_w + R;
-    float *s_sum = s_floor + R /* [2][R] */, *s_nq = s_sum + 2 * R, *s_n = s_nq + R + R /* spare */, *s_keep = s_n + KD;
+    float2* s_c = reinterpret_cast<float2*>(Sl + C * KP);           // c_s and e_t in units of ln 2, two parts each
+    float2* s_e = s_c + R;
+    float *s_g = reinterpret_cast<float*>(s_e + R), *s_w = s_g + R, *s_floor = s_w + R, *s_nq = s_floor + R;
+    float *s_sum = s_nq + R /* [4][R] */, *s_n = s_sum + 4 * R, *s_np = s_n + KD /* [N_PARTS][KD] */, *s_keep = s_np + P::N_PARTS * KD;
     float* stage = s_keep + 4;                                      // [R][KD], [R][KD], [R][C]
 
     const LinearStateArgs& cm = a.common;
@@ -265,7 +316,7 @@ __global__ void __launch_bounds__(MC_THREADS, 1) mlstm_chunk_kernel(const __grid
     const int col0 = blockIdx.x * C, head = blockIdx.y, cols = min(C, cm.vdim - col0);
     const int64_t head_state = (int64_t)(cm.vdim + 1) * KD;
     const int sc0 = warp % P::COL_GROUPS * 16, sk0 = warp / P::COL_GROUPS * P::KEYS;  // the warp's part of the state
-    const int row0 = (warp & 3) * 16, half = warp >> 2;                               // its part of a chunk's rows
+    const int row0 = (warp & 3) * 16, quarter = warp >> 2;                            // its part of a chunk's rows
 
     pdl_trigger();
     const StateLane sl = cm.lanes.at(blockIdx.z);
@@ -305,16 +356,18 @@ __global__ void __launch_bounds__(MC_THREADS, 1) mlstm_chunk_kernel(const __grid
     const bool staged = P::STAGED && vec;
     float *st_q = stage, *st_k = stage + R * KD, *st_v = stage + 2 * R * KD;
     auto request = [&](int chunk) {
-        const int64_t r0 = sl.first + (int64_t)chunk * R;
-        const int m = min(R, n - chunk * R), kp = cm.dim >> 2, vp = cols >> 2;
-        for (int i = threadIdx.x; i < m * kp; i += MC_THREADS) {
-            const int r = i / kp, c = (i - r * kp) * 4;
-            mc_cp_async16(st_q + r * KD + c, a.y.p + (r0 + r) * a.y.ld + qc + c);
-            mc_cp_async16(st_k + r * KD + c, a.y.p + (r0 + r) * a.y.ld + kc + c);
+        const float* y = a.y.p + ((int64_t)sl.first + (int64_t)chunk * R) * a.y.ld;
+        const int m = min(R, n - chunk * R);
+        for (int i = threadIdx.x; i < m * (KD / 4); i += MC_THREADS) {
+            const int r = i / (KD / 4), c = i % (KD / 4) * 4;
+            if (c < cm.dim) {
+                mc_cp_async16(st_q + r * KD + c, y + (int64_t)r * a.y.ld + qc + c);
+                mc_cp_async16(st_k + r * KD + c, y + (int64_t)r * a.y.ld + kc + c);
+            }
         }
-        for (int i = threadIdx.x; i < m * vp; i += MC_THREADS) {
-            const int r = i / vp, c = (i - r * vp) * 4;
-            mc_cp_async16(st_v + r * C + c, a.y.p + (r0 + r) * a.y.ld + vc + c);
+        for (int i = threadIdx.x; i < m * (C / 4); i += MC_THREADS) {
+            const int r = i / (C / 4), c = i % (C / 4) * 4;
+            if (c < cols) mc_cp_async16(st_v + r * C + c, y + (int64_t)r * a.y.ld + vc + c);
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
@@ -337,13 +390,13 @@ __global__ void __launch_bounds__(MC_THREADS, 1) mlstm_chunk_kernel(const __grid
         if (warp == 0) fetch_gates(0);
     }
     const float q_scale = rsqrtf((float)cm.dim);
-    const int raw_width = cm.vdim;
 
     for (int ch = 0; ch < chunks; ++ch) {
         const int64_t r0 = sl.first + (int64_t)ch * R;
         const int m = min(R, n - ch * R);
         if (warp == 0) {
             // sums and running maxima of the chunk's rows, two per lane, in f64: differences of far sums stay exact
+            constexpr double kLog2e = 1.4426950408889634074;
             double f1 = (double)lf[0] + lf[1];
 #pragma unroll
             for (int o = 1; o < 32; o <<= 1) {
@@ -372,10 +425,10 @@ __global__ void __launch_bounds__(MC_THREADS, 1) mlstm_chunk_kernel(const __grid
 #pragma unroll
             for (int h = 0; h < 2; ++h) {
                 const int r = 2 * lane + h;
-                c_hi[r] = (float)c[h];
-                c_lo[r] = c[h] == -INFINITY ? 0.f : (float)(c[h] - (double)c_hi[r]);
-                e_hi[r] = (float)e[h];
-                e_lo[r] = (float)(e[h] - (double)e_hi[r]);
+                const double c2 = c[h] * kLog2e, e2 = e[h] * kLog2e;
+                const float ch_hi = (float)c2, eh_hi = (float)e2;
+                s_c[r] = make_float2(ch_hi, c[h] == -INFINITY ? 0.f : (float)(c2 - (double)ch_hi));
+                s_e[r] = make_float2(eh_hi, (float)(e2 - (double)eh_hi));
                 s_g[r] = expf((float)(run_max - e[h]));
                 s_w[r] = expf((float)(c[h] - e_last));
                 s_floor[r] = expf(-mt[h]);
@@ -388,7 +441,7 @@ __global__ void __launch_bounds__(MC_THREADS, 1) mlstm_chunk_kernel(const __grid
         __syncthreads();  // the staged rows, the gates; everyone is through with the chunk before
         if (staged) {
             for (int i = threadIdx.x; i < R * (KD / 4); i += MC_THREADS) {
-                const int r = i / (KD / 4), c = (i - r * (KD / 4)) * 4;
+                const int r = i / (KD / 4), c = i % (KD / 4) * 4;
                 float4 x = make_float4(0.f, 0.f, 0.f, 0.f), y = x;
                 if (r < m && c < cm.dim) {
                     x = *reinterpret_cast<const float4*>(st_q + r * KD + c);
@@ -401,144 +454,137 @@ __global__ void __launch_bounds__(MC_THREADS, 1) mlstm_chunk_kernel(const __grid
             }
         } else {
             for (int i = threadIdx.x; i < R * KD; i += MC_THREADS) {
-                const int r = i / KD, c = i - r * KD;
+                const int r = i / KD, c = i % KD;
                 const bool live = r < m && c < cm.dim;
                 Q[r * KP + c] = __float2bfloat16_rn(live ? a.y.at(r0 + r, qc + c) : 0.f);
                 K[r * KP + c] = __float2bfloat16_rn(live ? a.y.at(r0 + r, kc + c) : 0.f);
             }
         }
         for (int i = threadIdx.x; i < R * (C / 2); i += MC_THREADS) {
-            const int r = i / (C / 2), c = (i - r * (C / 2)) * 2;
-            float x = 0.f, y = 0.f;
+            const int r = i / (C / 2), c = i % (C / 2) * 2;
+            float2 x = make_float2(0.f, 0.f);
             if (r < m) {
-                if (c < cols) x = staged ? st_v[r * C + c] : a.y.at(r0 + r, vc + c);
-                if (c + 1 < cols) y = staged ? st_v[r * C + c + 1] : a.y.at(r0 + r, vc + c + 1);
+                if (staged) {
+                    if (c < cols) x = *reinterpret_cast<const float2*>(st_v + r * C + c);
+                } else {
+                    if (c < cols) x.x = a.y.at(r0 + r, vc + c);
+                    if (c + 1 < cols) x.y = a.y.at(r0 + r, vc + c + 1);
+                }
             }
-            const __nv_bfloat162 v = __floats2bfloat162_rn(x, y);
+            const __nv_bfloat162 v = __floats2bfloat162_rn(x.x, x.y);
             *reinterpret_cast<__nv_bfloat162*>(V + r * CP + c) = v;
             uint32_t hi, lo;
             mc_split(s_w[r] * __low2float(v), s_w[r] * __high2float(v), hi, lo);
             *reinterpret_cast<uint32_t*>(Wh + r * CP + c) = hi;
             *reinterpret_cast<uint32_t*>(Wl + r * CP + c) = lo;
         }
+        if (ch > 0)  // the normaliser the chunk starts from: what was kept and the sums of the chunk before, by row groups
+            for (int i = threadIdx.x; i < KD; i += MC_THREADS) {
+                float x = s_n[i];
+#pragma unroll
+                for (int p = 0; p < P::N_PARTS; ++p) x += s_np[p * KD + i];
+                s_n[i] = x;
+            }
         __syncthreads();  // the staging rows are free, the operands are there
         if (ch + 1 < chunks) {
             if (staged) request(ch + 1);
             if (warp == 0) fetch_gates(ch + 1);
         }
+        auto q_fragment = [&](int k, uint32_t (&r)[4]) { mc_ldmatrix(r, Q + (row0 + (lane & 15)) * KP + k * 16 + (lane >> 4) * 8); };
 
-        // D (Q K^T): 16 rows x 32 keys per warp, keys behind the rows are zeros
+        // D (Q K^T): 16 rows x 16 keys per warp, keys behind the rows are zeros
         {
-            float sc[4][4] = {};
-            const int k0 = half * 32;
-            if (k0 <= row0 + 15) {
+            float sc[2][4] = {}, sum[2] = {0.f, 0.f};
+            const int k0 = quarter * 16;
+            uint32_t hi[2][2] = {}, lo[2][2] = {};
+            if (k0 <= row0) {
+                mc_product<2, KD / 16, false, KP>(sc, lane, q_fragment, [&](int k, int j) { return (k0 + j * 8) * KP + k * 16; }, K, nullptr);
+                const float2 e[2] = {s_e[row0 + gid], s_e[row0 + gid + 8]};
 #pragma unroll
-                for (int kk = 0; kk < KD / 16; ++kk) {
-                    uint32_t af[4];
-                    mc_ldmatrix(af, Q + (row0 + (lane & 15)) * KP + kk * 16 + (lane >> 4) * 8);
+                for (int j = 0; j < 2; ++j) {
+                    const int s = k0 + j * 8 + 2 * tq;
+                    const float4 c = *reinterpret_cast<const float4*>(s_c + s);
 #pragma unroll
-                    for (int j = 0; j < 4; j += 2) {
-                        uint32_t bf[4];
-                        mc_ldmatrix(bf, K + (k0 + j * 8 + (lane & 7) + (lane >> 4) * 8) * KP + kk * 16 + ((lane >> 3) & 1) * 8);
-                        mc_mma(sc[j], af, bf[0], bf[1]);
-                        mc_mma(sc[j + 1], af, bf[2], bf[3]);
+                    for (int h = 0; h < 2; ++h) {
+                        const int t = row0 + gid + 8 * h;
+                        const float d0 = s <= t ? exp2f((c.x - e[h].x) + (c.y - e[h].y)) : 0.f, d1 = s + 1 <= t ? exp2f((c.z - e[h].x) + (c.w - e[h].y)) : 0.f;
+                        const float p0 = sc[j][2 * h] * q_scale * d0, p1 = sc[j][2 * h + 1] * q_scale * d1;
+                        sum[h] += p0 + p1;
+                        mc_split(p0, p1, hi[j][h], lo[j][h]);
                     }
                 }
             }
-            float sum[2] = {0.f, 0.f};
 #pragma unroll
-            for (int j = 0; j < 4; ++j)
+            for (int j = 0; j < 2; ++j)
 #pragma unroll
                 for (int h = 0; h < 2; ++h) {
-                    const int t = row0 + gid + 8 * h, s = k0 + j * 8 + 2 * tq;
-                    float p[2];
-#pragma unroll
-                    for (int x = 0; x < 2; ++x) {
-                        const float d = s + x <= t ? expf((c_hi[s + x] - e_hi[t]) + (c_lo[s + x] - e_lo[t])) : 0.f;
-                        p[x] = sc[j][2 * h + x] * q_scale * d;
-                        sum[h] += p[x];
-                    }
-                    uint32_t hi, lo;
-                    mc_split(p[0], p[1], hi, lo);
-                    *reinterpret_cast<uint32_t*>(Ph + t * PP + s) = hi;
-                    *reinterpret_cast<uint32_t*>(Pl + t * PP + s) = lo;
+                    const int at = (row0 + gid + 8 * h) * PP + k0 + j * 8 + 2 * tq;
+                    *reinterpret_cast<uint32_t*>(Ph + at) = hi[j][h];
+                    *reinterpret_cast<uint32_t*>(Pl + at) = lo[j][h];
                 }
 #pragma unroll
             for (int h = 0; h < 2; ++h) {
                 sum[h] += __shfl_xor_sync(0xffffffffu, sum[h], 1);
                 sum[h] += __shfl_xor_sync(0xffffffffu, sum[h], 2);
-                if (tq == 0) s_sum[half * R + row0 + gid + 8 * h] = sum[h];
+                if (tq == 0) s_sum[quarter * R + row0 + gid + 8 * h] = sum[h];
             }
-            // n . q of the normaliser the chunk starts from: four threads per row
-            const int t = threadIdx.x >> 2, part = threadIdx.x & 3;
+            // n . q of the normaliser the chunk starts from: eight threads per row
+            const int t = threadIdx.x >> 3, part = threadIdx.x & 7;
             float nq = 0.f;
-#pragma unroll 8
-            for (int c = part * 2; c < KD; c += 8) {
+#pragma unroll
+            for (int c = part * 2; c < KD; c += 16) {
                 const __nv_bfloat162 q2 = *reinterpret_cast<const __nv_bfloat162*>(Q + t * KP + c);
-                nq = fmaf(__low2float(q2), s_n[c], fmaf(__high2float(q2), s_n[c + 1], nq));
+                const float2 n2 = *reinterpret_cast<const float2*>(s_n + c);
+                nq = fmaf(__low2float(q2), n2.x, fmaf(__high2float(q2), n2.y, nq));
             }
-            nq += __shfl_xor_sync(0xffffffffu, nq, 1);
-            nq += __shfl_xor_sync(0xffffffffu, nq, 2);
+#pragma unroll
+            for (int x = 1; x < 8; x <<= 1) nq += __shfl_xor_sync(0xffffffffu, nq, x);
             if (part == 0) s_nq[t] = nq;
         }
         __syncthreads();
 
-        // outputs: 16 rows x C / 2 columns per warp
+        // outputs: 16 rows x C / 4 columns per warp
         {
             float o[NT][4] = {};
-            const int n0 = half * (C / 2);
-#pragma unroll
-            for (int kk = 0; kk < KD / 16; ++kk) {
-                uint32_t af[4];
-                mc_ldmatrix(af, Q + (row0 + (lane & 15)) * KP + kk * 16 + (lane >> 4) * 8);
-#pragma unroll
-                for (int j = 0; j < NT; j += 2) {
-                    const int at = (n0 + j * 8 + (lane & 7) + (lane >> 4) * 8) * KP + kk * 16 + ((lane >> 3) & 1) * 8;
-                    uint32_t bf[4];
-                    mc_ldmatrix(bf, Sh + at);
-                    mc_mma(o[j], af, bf[0], bf[1]);
-                    mc_mma(o[j + 1], af, bf[2], bf[3]);
-                    mc_ldmatrix(bf, Sl + at);
-                    mc_mma(o[j], af, bf[0], bf[1]);
-                    mc_mma(o[j + 1], af, bf[2], bf[3]);
-                }
-            }
+            const int n0 = quarter * (C / 4);
+            mc_product<NT, KD / 16, false, KP>(o, lane, q_fragment, [&](int k, int j) { return (n0 + j * 8) * KP + k * 16; }, Sh, Sl);
             float g[2], den[2];
 #pragma unroll
             for (int h = 0; h < 2; ++h) {
                 const int t = row0 + gid + 8 * h;
                 g[h] = s_g[t] * q_scale;
-                den[h] = fmaxf(fabsf(s_sum[t] + s_sum[R + t] + g[h] * s_nq[t]), s_floor[t]) + 1e-6f;
+                const float nq = s_sum[t] + s_sum[R + t] + s_sum[2 * R + t] + s_sum[3 * R + t] + g[h] * s_nq[t];
+                den[h] = fmaxf(fabsf(nq), s_floor[t]) + 1e-6f;
             }
 #pragma unroll
             for (int j = 0; j < NT; ++j)
 #pragma unroll
                 for (int x = 0; x < 4; ++x) o[j][x] *= g[x >> 1];
-            for (int kk = 0; kk <= (row0 >> 4); ++kk) {
-                uint32_t ph[4], pl[4];
-                const int at = (row0 + (lane & 15)) * PP + kk * 16 + (lane >> 4) * 8;
-                mc_ldmatrix(ph, Ph + at);
-                mc_ldmatrix(pl, Pl + at);
+            // the weights behind the rows are zeros: only what lies before counts, 32 keys at a time
+            auto v_at = [&](int k, int j) { return k * 16 * CP + n0 + j * 8; };
 #pragma unroll
-                for (int j = 0; j < NT; j += 2) {
-                    uint32_t bf[4];
-                    mc_ldmatrix_t(bf, V + (kk * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * CP + n0 + j * 8 + (lane >> 4) * 8);
-                    mc_mma(o[j], ph, bf[0], bf[1]);
-                    mc_mma(o[j + 1], ph, bf[2], bf[3]);
-                    mc_mma(o[j], pl, bf[0], bf[1]);
-                    mc_mma(o[j + 1], pl, bf[2], bf[3]);
-                }
+            for (int part = 0; part < 2; ++part) {
+                const __nv_bfloat16* Pp = part == 0 ? Ph : Pl;
+                auto p_fragment = [&](int k, uint32_t (&r)[4]) { mc_ldmatrix(r, Pp + (row0 + (lane & 15)) * PP + k * 16 + (lane >> 4) * 8); };
+                if (row0 < 32) mc_product<NT, 2, true, CP>(o, lane, p_fragment, v_at, V, nullptr);
+                else mc_product<NT, 4, true, CP>(o, lane, p_fragment, v_at, V, nullptr);
             }
 #pragma unroll
             for (int h = 0; h < 2; ++h) {
                 const int t = row0 + gid + 8 * h;
                 if (t >= m) continue;
-                float* out = cm.out + ((r0 + t) * cm.heads + head) * raw_width + col0;
+                float* out = cm.out + ((r0 + t) * cm.heads + head) * cm.vdim + col0;
+                const float inv = 1.0f / den[h];
 #pragma unroll
                 for (int j = 0; j < NT; ++j) {
                     const int c = n0 + j * 8 + 2 * tq;
-                    if (c < cols) out[c] = o[j][2 * h] / den[h];
-                    if (c + 1 < cols) out[c + 1] = o[j][2 * h + 1] / den[h];
+                    const float x = o[j][2 * h] * inv, y = o[j][2 * h + 1] * inv;
+                    if (vec) {
+                        if (c < cols) *reinterpret_cast<float2*>(out + c) = make_float2(x, y);
+                    } else {
+                        if (c < cols) out[c] = x;
+                        if (c + 1 < cols) out[c + 1] = y;
+                    }
                 }
             }
         }
@@ -548,27 +594,28 @@ __global__ void __launch_bounds__(MC_THREADS, 1) mlstm_chunk_kernel(const __grid
         for (int j = 0; j < NK; ++j)
 #pragma unroll
             for (int x = 0; x < 4; ++x) S[j][x] *= keep;
+        auto k_at = [&](int k, int j) { return k * 16 * KP + sk0 + j * 8; };
 #pragma unroll
-        for (int kk = 0; kk < R / 16; ++kk) {
-            uint32_t wh[4], wl[4];
-            const int at = (kk * 16 + (lane >> 4) * 8 + (lane & 7)) * CP + sc0 + ((lane >> 3) & 1) * 8;
-            mc_ldmatrix_t(wh, Wh + at);
-            mc_ldmatrix_t(wl, Wl + at);
-#pragma unroll
-            for (int j = 0; j < NK; j += 2) {
-                uint32_t bf[4];
-                mc_ldmatrix_t(bf, K + (kk * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * KP + sk0 + j * 8 + (lane >> 4) * 8);
-                mc_mma(S[j], wh, bf[0], bf[1]);
-                mc_mma(S[j + 1], wh, bf[2], bf[3]);
-                mc_mma(S[j], wl, bf[0], bf[1]);
-                mc_mma(S[j + 1], wl, bf[2], bf[3]);
-            }
+        for (int part = 0; part < 2; ++part) {
+            const __nv_bfloat16* Wp = part == 0 ? Wh : Wl;
+            auto w_fragment = [&](int k, uint32_t (&r)[4]) { mc_ldmatrix_t(r, Wp + (k * 16 + (lane >> 4) * 8 + (lane & 7)) * CP + sc0 + ((lane >> 3) & 1) * 8); };
+            mc_product<NK, R / 16, true, KP>(S, lane, w_fragment, k_at, K, nullptr);
         }
-        for (int i = threadIdx.x; i < KD; i += MC_THREADS) {
-            float x = s_n[i] * keep;
-#pragma unroll 8
-            for (int t = 0; t < R; ++t) x = fmaf(s_w[t], __bfloat162float(K[t * KP + i]), x);
-            s_n[i] = x;  // read again behind the next barrier only
+        {
+            const int pair = threadIdx.x % (KD / 2) * 2, part = threadIdx.x / (KD / 2);
+            constexpr int ROWS = R / P::N_PARTS;
+            float x = 0.f, y = 0.f;
+#pragma unroll
+            for (int t = part * ROWS; t < (part + 1) * ROWS; ++t) {
+                const __nv_bfloat162 k2 = *reinterpret_cast<const __nv_bfloat162*>(K + t * KP + pair);
+                x = fmaf(s_w[t], __low2float(k2), x);
+                y = fmaf(s_w[t], __high2float(k2), y);
+            }
+            *reinterpret_cast<float2*>(s_np + part * KD + pair) = make_float2(x, y);
+            if (part == 0) {
+                s_n[pair] *= keep;  // the sums are added behind the next barrier
+                s_n[pair + 1] *= keep;
+            }
         }
         __syncthreads();  // the old state was read by everyone
         if (ch + 1 < chunks) publish_state();
@@ -583,7 +630,12 @@ __global__ void __launch_bounds__(MC_THREADS, 1) mlstm_chunk_kernel(const __grid
             if (col < cm.vdim) *reinterpret_cast<float2*>(dst + (int64_t)col * KD + sk0 + j * 8 + 2 * tq) = make_float2(S[j][2 * h], S[j][2 * h + 1]);
         }
     if (blockIdx.x == 0) {
-        for (int i = threadIdx.x; i < KD; i += MC_THREADS) dst[(int64_t)cm.vdim * KD + i] = s_n[i];
+        for (int i = threadIdx.x; i < KD; i += MC_THREADS) {
+            float x = s_n[i];
+            if (chunks > 0)
+                for (int p = 0; p < P::N_PARTS; ++p) x += s_np[p * KD + i];
+            dst[(int64_t)cm.vdim * KD + i] = x;
+        }
         if (threadIdx.x == 0) a.running_max[(int64_t)sl.out * cm.heads + head] = run_max;
     }
 }

@@ -6,6 +6,7 @@
 #include "moe_rows.h"
 #include "kernels.h"
 #include <climits>
+#include <type_traits>
 
 namespace mk {
 
@@ -15,30 +16,30 @@ constexpr int MR_MAX_EXPERTS = 1024;
 constexpr int MR_MAX_TOP = 32;
 constexpr int MR_THREADS = 256;
 
-// One token by one warp; logit(e) is valid up to `experts` (the shared expert's gate).
-template <typename Logit>
+// One token by one warp, PER experts per lane; logit(e) is valid up to `experts` (the shared expert's gate).
+template <int PER, typename Logit>
 __device__ __forceinline__ void route_token(Logit logit, int t, int experts, int k, const MoeRows& r, int half, int32_t* status, int lane) {
-    float v[MR_MAX_EXPERTS / 32];
-    int cnt = 0;
+    float v[PER];
     bool bad = false;
-    for (int e = lane; e < experts; e += 32) {
-        float x = logit(e);
-        if (!isfinite(x)) {
+#pragma unroll
+    for (int c = 0; c < PER; ++c) {
+        const int e = lane + 32 * c;
+        v[c] = e < experts ? logit(e) : -INFINITY;
+        if (e < experts && !isfinite(v[c])) {
             bad = true;
-            x = -3.402823466e38f;
+            v[c] = -3.402823466e38f;
         }
-        v[cnt++] = x;
     }
     if (lane == 0 && r.shared_gate != nullptr) r.shared_gate[t] = sigmoid_f(logit(experts));
     if (__any_sync(0xffffffffu, bad) && lane == 0) atomicCAS(status, 0, kMoeRouteStatus | (t & 0xFFFF));
-    unsigned taken = 0;  // bit c: this lane's c-th expert was chosen
     float my_logit = 0.f;
     int mine = 0;        // lane i keeps choice i
     for (int i = 0; i < k; ++i) {
         float bv = -INFINITY;
         int be = INT_MAX;
-        for (int c = 0; c < cnt; ++c)
-            if (!(taken >> c & 1u) && v[c] > bv) {
+#pragma unroll
+        for (int c = 0; c < PER; ++c)
+            if (v[c] > bv) {
                 bv = v[c];
                 be = lane + 32 * c;
             }
@@ -51,7 +52,9 @@ __device__ __forceinline__ void route_token(Logit logit, int t, int experts, int
                 be = oe;
             }
         }
-        if ((be & 31) == lane) taken |= 1u << (be >> 5);
+#pragma unroll
+        for (int c = 0; c < PER; ++c)
+            if (be == lane + 32 * c) v[c] = -INFINITY;
         if (lane == i) {
             my_logit = bv;
             mine = be;
@@ -65,12 +68,13 @@ __device__ __forceinline__ void route_token(Logit logit, int t, int experts, int
     }
 }
 
+template <int PER>
 __global__ void __launch_bounds__(128) moe_route_rows_kernel(Shares logits, int T, int experts, int k, MoeRows r, int half, int32_t* status) {
     pdl_trigger();
     pdl_wait();
     const int t = blockIdx.x * 4 + (threadIdx.x >> 5);
     if (t >= T) return;
-    route_token([&](int e) { return logits.at(t, e); }, t, experts, k, r, half, status, threadIdx.x & 31);
+    route_token<PER>([&](int e) { return logits.at(t, e); }, t, experts, k, r, half, status, threadIdx.x & 31);
 }
 
 // Eight neighbouring columns.
@@ -89,9 +93,12 @@ __device__ __forceinline__ void load8(const float* p, float (&v)[8]) {
     v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
 }
 
-// One CTA per token: a warp per router row, then the first warp routes.  Shared memory: experts + 1 logits.
-template <typename W>
-__global__ void __launch_bounds__(MR_THREADS) moe_router_kernel(RowImage x, const W* __restrict__ w, int experts, int k, MoeRows r, int half, int32_t* status) {
+constexpr int MR_ROUTER_THREADS = 512;
+
+// One CTA per token: a warp takes four router rows at once, then the first warp routes.  Shared memory: experts + 4 logits.
+template <typename W, int PER>
+__global__ void __launch_bounds__(MR_ROUTER_THREADS) moe_router_kernel(RowImage x, const W* __restrict__ w, int experts, int k, MoeRows r, int half,
+                                                                       int32_t* status) {
     extern __shared__ float mr_logit[];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int64_t t = blockIdx.x;
@@ -101,21 +108,30 @@ __global__ void __launch_bounds__(MR_THREADS) moe_router_kernel(RowImage x, cons
     else row = x.f + t * ld;
     pdl_trigger();
     pdl_wait();
-    for (int e = warp; e < rows; e += MR_THREADS / 32) {
-        float sum = 0.f;
-#pragma unroll 4
-        for (int c = lane * 8; c < ld; c += 256) {  // ld is a multiple of 64
-            float a[8], b[8];
-            load8(row + c, a);
-            load8(w + (int64_t)e * ld + c, b);
+    for (int e = warp * 4; e < rows; e += MR_ROUTER_THREADS / 32 * 4) {
+        const W* we[4];
 #pragma unroll
-            for (int i = 0; i < 8; ++i) sum = fmaf(a[i], b[i], sum);
+        for (int i = 0; i < 4; ++i) we[i] = w + (int64_t)min(e + i, rows - 1) * ld;
+        float sum[4] = {};
+#pragma unroll 2
+        for (int c = lane * 8; c < ld; c += 256) {  // ld is a multiple of 64
+            float a[8], b[4][8];
+            load8(row + c, a);
+#pragma unroll
+            for (int i = 0; i < 4; ++i) load8(we[i] + c, b[i]);
+#pragma unroll
+            for (int i = 0; i < 4; ++i)
+#pragma unroll
+                for (int j = 0; j < 8; ++j) sum[i] = fmaf(a[j], b[i][j], sum[i]);
         }
-        sum = warp_sum(sum);
-        if (lane == 0) mr_logit[e] = sum;
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            sum[i] = warp_sum(sum[i]);
+            if (lane == 0) mr_logit[e + i] = sum[i];
+        }
     }
     __syncthreads();
-    if (warp == 0) route_token([&](int e) { return mr_logit[e]; }, (int)t, experts, k, r, half, status, lane);
+    if (warp == 0) route_token<PER>([&](int e) { return mr_logit[e]; }, (int)t, experts, k, r, half, status, lane);
 }
 
 // One CTA per token.
@@ -167,12 +183,24 @@ void check(int experts, int k) {
     if (experts <= 0 || experts > MR_MAX_EXPERTS || k <= 0 || k > MR_MAX_TOP || k > experts) throw std::runtime_error("mixture of experts: at most 1024 experts and 32 choices");
 }
 
+// fn(constant): experts per lane of a routing warp.
+template <typename Fn>
+void per_lane(int experts, Fn fn) {
+    if (experts <= 32) fn(std::integral_constant<int, 1>{});
+    else if (experts <= 64) fn(std::integral_constant<int, 2>{});
+    else if (experts <= 128) fn(std::integral_constant<int, 4>{});
+    else if (experts <= 256) fn(std::integral_constant<int, 8>{});
+    else fn(std::integral_constant<int, MR_MAX_EXPERTS / 32>{});
+}
+
 }  // namespace
 
 void launch_moe_route(const Shares& logits, int T, int experts, int k, const MoeRows& rows, int half, int32_t* status, cudaStream_t s) {
     if (T <= 0) return;
     check(experts, k);
-    launch_pdl(moe_route_rows_kernel, dim3((unsigned)((T + 3) / 4)), dim3(128), 0, s, logits, T, experts, k, rows, half, status);
+    per_lane(experts, [&](auto per) {
+        launch_pdl(moe_route_rows_kernel<per.value>, dim3((unsigned)((T + 3) / 4)), dim3(128), 0, s, logits, T, experts, k, rows, half, status);
+    });
     MK_LAUNCH_CHECK();
 }
 
@@ -181,11 +209,14 @@ bool moe_router_is_narrow(int T, int experts, int cols) { return T <= 64 && (int
 void launch_moe_router(const RowImage& x, const void* w, int T, int experts, int k, const MoeRows& rows, int half, int32_t* status, cudaStream_t s) {
     if (T <= 0) return;
     check(experts, k);
-    const size_t smem = (size_t)(experts + 1) * 4;
-    if (x.h != nullptr)
-        launch_pdl(moe_router_kernel<__nv_bfloat16>, dim3((unsigned)T), dim3(MR_THREADS), smem, s, x, static_cast<const __nv_bfloat16*>(w), experts, k, rows, half, status);
-    else
-        launch_pdl(moe_router_kernel<float>, dim3((unsigned)T), dim3(MR_THREADS), smem, s, x, static_cast<const float*>(w), experts, k, rows, half, status);
+    const size_t smem = (size_t)(experts + 8) * 4;
+    const dim3 grid((unsigned)T), block(MR_ROUTER_THREADS);
+    per_lane(experts, [&](auto per) {
+        if (x.h != nullptr)
+            launch_pdl(moe_router_kernel<__nv_bfloat16, per.value>, grid, block, smem, s, x, static_cast<const __nv_bfloat16*>(w), experts, k, rows, half, status);
+        else
+            launch_pdl(moe_router_kernel<float, per.value>, grid, block, smem, s, x, static_cast<const float*>(w), experts, k, rows, half, status);
+    });
     MK_LAUNCH_CHECK();
 }
 

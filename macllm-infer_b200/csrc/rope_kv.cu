@@ -53,21 +53,38 @@ __global__ void __launch_bounds__(RK_WARPS * 32) rope_kv_kernel(RopeKvArgs a) {
     }
 }
 
-constexpr int RR_THREADS = 256;
-
-// One CTA per token: all heads of the token in shared memory (kv_heads * (d + dv) + q_heads * d floats).
-template <typename KV>
-__global__ void __launch_bounds__(RR_THREADS) rope_kv_rows_kernel(RopeKvArgs a) {
+// One CTA per token: all heads of the token in shared memory ((q_heads + kv_heads) * d + kv_heads * dv floats).
+// vec: every row starts on 16 bytes and head widths are multiples of four.
+template <typename KV, int THREADS>
+__global__ void __launch_bounds__(THREADS) rope_kv_rows_kernel(RopeKvArgs a, int vec) {
     extern __shared__ __align__(16) float rr_row[];
-    __shared__ float red[32];
+    __shared__ float red[2][32];
     pdl_trigger();
     pdl_wait();
     const int t = blockIdx.x, dv = a.dv > 0 ? a.dv : a.d, D = rope_row_width(a);
     const int qw = a.q_heads * a.d, kw = a.kv_heads * a.d, vw = a.kv_heads * dv;
     float *xq = rr_row, *xk = xq + qw, *xv = xk + kw;
+    // a projection's row: the shares' sum and the bias; returns the thread's sum of squares
     auto load = [&](float* dst, const float* src, int n, int parts, int64_t stride, const float* bias) {
         float ss = 0.f;
-        for (int c = threadIdx.x; c < n; c += RR_THREADS) {
+        if (vec) {
+            for (int c = threadIdx.x * 4; c < n; c += THREADS * 4) {
+                float4 v = *reinterpret_cast<const float4*>(src + c);
+#pragma unroll 8
+                for (int p = 1; p < parts; ++p) {
+                    const float4 w = *reinterpret_cast<const float4*>(src + (int64_t)p * stride + c);
+                    v = make_float4(v.x + w.x, v.y + w.y, v.z + w.z, v.w + w.w);
+                }
+                if (bias != nullptr) {
+                    const float4 b = *reinterpret_cast<const float4*>(bias + c);
+                    v = make_float4(v.x + b.x, v.y + b.y, v.z + b.z, v.w + b.w);
+                }
+                *reinterpret_cast<float4*>(dst + c) = v;
+                ss = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, ss))));
+            }
+            return ss;
+        }
+        for (int c = threadIdx.x; c < n; c += THREADS) {
             float v = src[c];
             for (int p = 1; p < parts; ++p) v += src[(int64_t)p * stride + c];
             if (bias != nullptr) v += bias[c];
@@ -76,11 +93,23 @@ __global__ void __launch_bounds__(RR_THREADS) rope_kv_rows_kernel(RopeKvArgs a) 
         }
         return ss;
     };
-    const float sq = load(xq, a.q + (int64_t)t * a.ldq, qw, a.qk_splits, a.qk_split_stride, a.q_bias);
-    const float sk = load(xk, a.k + (int64_t)t * a.ldk, kw, a.qk_splits, a.qk_split_stride, a.k_bias);
+    float sq = load(xq, a.q + (int64_t)t * a.ldq, qw, a.qk_splits, a.qk_split_stride, a.q_bias);
+    float sk = load(xk, a.k + (int64_t)t * a.ldk, kw, a.qk_splits, a.qk_split_stride, a.k_bias);
     load(xv, a.v + (int64_t)t * a.ldv, vw, a.v_splits, a.v_split_stride, a.v_bias);
-    const float rq = sqrtf(block_sum(sq, red) / (float)qw + a.norm_eps);
-    const float rk = sqrtf(block_sum(sk, red) / (float)kw + a.norm_eps);  // its barriers also publish the rows
+    sq = warp_sum(sq);
+    sk = warp_sum(sk);
+    if ((threadIdx.x & 31) == 0) {
+        red[0][threadIdx.x >> 5] = sq;
+        red[1][threadIdx.x >> 5] = sk;
+    }
+    __syncthreads();
+    sq = sk = 0.f;
+#pragma unroll
+    for (int w = 0; w < THREADS / 32; ++w) {
+        sq += red[0][w];
+        sk += red[1][w];
+    }
+    const float rq = sqrtf(sq / (float)qw + a.norm_eps), rk = sqrtf(sk / (float)kw + a.norm_eps);
     const int rd = a.cos_t != nullptr ? a.rotary_dim : 0, half = rd / 2;
     const float* cs = a.cos_t + (rd > 0 ? (int64_t)a.positions[t] * half : 0);
     const float* sn = a.sin_t + (rd > 0 ? (int64_t)a.positions[t] * half : 0);
@@ -95,18 +124,28 @@ __global__ void __launch_bounds__(RR_THREADS) rope_kv_rows_kernel(RopeKvArgs a) 
         return first ? own * cs[i] - other * sn[i] : own * cs[i] + other * sn[i];
     };
     float* q_out = a.q_out + (int64_t)t * a.ldq_out;
-    for (int i = threadIdx.x; i < a.q_heads * D; i += RR_THREADS) {
+#pragma unroll 4
+    for (int i = threadIdx.x; i < a.q_heads * D; i += THREADS) {
         const int h = i / D, c = i - h * D;
         q_out[i] = c < a.d ? turned(xq + h * a.d, a.q_norm_w + h * a.d, rq, c) : 0.f;
     }
     const int64_t slot = a.slots[t], blk = slot / a.block_tokens, row = slot % a.block_tokens;
     KV *kp = reinterpret_cast<KV*>(a.k_pool), *vp = reinterpret_cast<KV*>(a.v_pool);
-    for (int i = threadIdx.x; i < a.kv_heads * D; i += RR_THREADS) {
+    const int64_t page = kv_page_index(blk, a.layer, a.layers, a.pool_blocks) * a.kv_heads;
+#pragma unroll 2
+    for (int i = threadIdx.x; i < a.kv_heads * D; i += THREADS) {
         const int h = i / D, c = i - h * D;
-        const int64_t at = ((kv_page_index(blk, a.layer, a.layers, a.pool_blocks) * a.kv_heads + h) * a.block_tokens + row) * (int64_t)D + c;
+        const int64_t at = ((page + h) * a.block_tokens + row) * (int64_t)D + c;
         kp[at] = to_kv<KV>(c < a.d ? turned(xk + h * a.d, a.k_norm_w + h * a.d, rk, c) : 0.f);
         vp[at] = to_kv<KV>(c < dv ? xv[h * dv + c] : 0.f);
     }
+}
+
+template <typename KV, int THREADS>
+void launch_rope_rows(const RopeKvArgs& a, size_t smem, int vec, cudaStream_t s) {
+    auto* kernel = rope_kv_rows_kernel<KV, THREADS>;
+    ensure_dynamic_smem(reinterpret_cast<const void*>(kernel), smem);
+    launch_pdl(kernel, dim3((unsigned)a.T), dim3(THREADS), smem, s, a, vec);
 }
 
 template <typename KV>
@@ -143,9 +182,18 @@ void launch_rope_kv_rows(const RopeKvArgs& a, cudaStream_t s) {
     if (a.q_out == nullptr || a.q_norm_w == nullptr || a.k_norm_w == nullptr) throw std::runtime_error("launch_rope_kv_rows: needs norm weights and a query output");
     const size_t smem = ((size_t)a.q_heads * a.d + (size_t)a.kv_heads * (a.d + (a.dv > 0 ? a.dv : a.d))) * 4;
     if (smem > (size_t)200 * 1024) throw std::runtime_error("launch_rope_kv_rows: the projections are too wide");
-    auto* kernel = a.kv_f16 ? rope_kv_rows_kernel<__half> : rope_kv_rows_kernel<float>;
-    ensure_dynamic_smem(reinterpret_cast<const void*>(kernel), smem);
-    launch_pdl(kernel, dim3((unsigned)a.T), dim3(RR_THREADS), smem, s, a);
+    const int dv = a.dv > 0 ? a.dv : a.d;
+    auto on16 = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
+    const int vec = a.d % 4 == 0 && dv % 4 == 0 && a.ldq % 4 == 0 && a.ldk % 4 == 0 && a.ldv % 4 == 0 && a.qk_split_stride % 4 == 0 && a.v_split_stride % 4 == 0 &&
+                    on16(a.q) && on16(a.k) && on16(a.v) && on16(a.q_bias) && on16(a.k_bias) && on16(a.v_bias) ? 1 : 0;
+    // ticks of a few rows: a row's latency counts, so many threads share it
+    if (a.T <= 148) {
+        if (a.kv_f16) launch_rope_rows<__half, 1024>(a, smem, vec, s);
+        else launch_rope_rows<float, 1024>(a, smem, vec, s);
+    } else {
+        if (a.kv_f16) launch_rope_rows<__half, 256>(a, smem, vec, s);
+        else launch_rope_rows<float, 256>(a, smem, vec, s);
+    }
     MK_LAUNCH_CHECK();
 }
 
