@@ -7,15 +7,18 @@
 // once at load time: w = f16(dequant(block)), one rounding per weight.  The GEMM is then the plain
 // y[t][n] = sum_k xh[t][k] * wh[n][k] with f32 accumulation in tensor memory.
 //
-// One persistent CTA per SM, 192 threads in three roles:
+// One persistent CTA per SM, 320 threads in three roles:
 //   warp 0   - one lane issues TMA loads (cp.async.bulk.tensor, 128-byte swizzle) of a 128 x 64 weight
 //              box and a BN x 64 activation box per stage into a ring of shared-memory stages;
 //   warp 1   - one lane issues the MMAs (tcgen05.mma kind::f16, M = 128 weight rows, N = BN tokens,
 //              four K = 16 steps per stage), commits each stage back to the loader, and commits the tile
 //              to the epilogue; two accumulators in tensor memory alternate so the next tile's main
 //              loop runs under the previous tile's epilogue;
-//   warps 2-5 - read the accumulator (tcgen05.ld, one lane per weight row), apply scale / soft cap and
-//              store f32 results (32 consecutive rows of one token per store instruction).
+//   warps 2-9 - read the accumulator (tcgen05.ld, one lane per weight row, two warps per lane quadrant that take
+//              every other 32 columns), apply scale / soft cap and store f32 results (32 consecutive rows of one
+//              token per store instruction).  A tile's main loop is as long as K, its epilogue is not: with short K
+//              it is the epilogue's instructions that count, hence eight warps and whole 32-column groups without
+//              a test per column.
 // Every mbarrier wait is bounded; a wait that gives up records a status word and the role leaves its
 // loop, the other roles run into their own limits, and tensor memory is always released.
 #include "hgemm_tc.h"
@@ -30,7 +33,8 @@ namespace {
 
 constexpr int HG_BM = 128;
 constexpr int HG_BK = 64;  // 64 halves = 128 bytes = one swizzle row
-constexpr int HG_THREADS = 192;
+constexpr int HG_EPI_THREADS = 256;
+constexpr int HG_THREADS = 64 + HG_EPI_THREADS;
 constexpr uint32_t HG_SPIN_LIMIT = 1u << 22;
 
 __device__ __forceinline__ uint32_t smem_u32(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
@@ -285,7 +289,7 @@ hgemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant_
         }
         for (int i = 0; i < 2; ++i) {
             mbar_init(&acc_full[i], 1);
-            mbar_init(&acc_empty[i], 128);
+            mbar_init(&acc_empty[i], HG_EPI_THREADS);
         }
         asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
     }
@@ -466,9 +470,10 @@ hgemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant_
             }
         }
     } else {
-        // ---- epilogue: warps 2..5 own TMEM lane quadrants (warp % 4)
-        const int quad = warp & 3;
-        const int etid = (int)threadIdx.x - 64;  // 0..127 among the epilogue threads
+        // ---- epilogue: warps 2..9 own TMEM lane quadrants (warp % 4), two each
+        const int quad = warp & 3, odd_group = (warp - 2) >> 2;
+        const int etid = (int)threadIdx.x - 64;  // among the epilogue threads
+        const bool plain = p.out_scale == 1.0f && p.softcap == 0.f;
         if (p.part[0].act_post != nullptr) pdl_wait();   // the factors of the rows come from a predecessor
         uint32_t tile_it = 0;
         for (int item = blockIdx.x; item < total_items; item += gridDim.x, ++tile_it) {
@@ -477,17 +482,17 @@ hgemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant_
             decode(item, tile, kb0, kb1);
             const int split = p.splits > 1 ? item / mn_tiles : 0;
             const uint32_t acc = tile_it & 1, acc_ph = (tile_it >> 1) & 1;
-            // every epilogue warp waits for itself, then the four agree on the outcome, so that a wait that
+            // every epilogue warp waits for itself, then all agree on the outcome, so that a wait that
             // gave up takes all of them out of the loop together (they meet again at named barrier 1)
             const uint32_t got = mbar_wait(&acc_full[acc], acc_ph, HG_SPIN_LIMIT) ? 1u : 0u;
             uint32_t all_got;
             asm volatile(
                 "{\n\t.reg .pred p, q;\n\t"
                 "setp.ne.u32 q, %1, 0;\n\t"
-                "bar.red.and.pred p, 1, 128, q;\n\t"
+                "bar.red.and.pred p, 1, %2, q;\n\t"
                 "selp.u32 %0, 1, 0, p;\n\t}"
                 : "=r"(all_got)
-                : "r"(got)
+                : "r"(got), "n"(HG_EPI_THREADS)
                 : "memory");
             if (!all_got) {
                 if (etid == 0) atomicExch(p.status, 14);
@@ -500,8 +505,8 @@ hgemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant_
             float* dst = p.splits > 1 ? p.partial + (int64_t)split * p.T * p.rows : part.y;
             const int ld = p.splits > 1 ? p.rows : part.ldy;
 #pragma unroll 1
-            for (int cb = 0; cb < BN; cb += LD_COLS) {
-                if (tok0 + cb >= tile.tok_end) break;  // uniform over the CTA: nothing but padding from here on
+            for (int cb = odd_group * LD_COLS; cb < BN; cb += 2 * LD_COLS) {
+                if (tok0 + cb >= tile.tok_end) break;  // uniform over the warp: nothing but padding from here on
                 // the factors of the chunk's tokens, one per lane, on their way with the accumulators
                 float pre = 1.0f, post = 1.0f;
                 if (p.gated == 1 + GatedAct::Clamped && tok0 + cb + lane < tile.tok_end) {
@@ -516,6 +521,7 @@ hgemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant_
                     // the odd lane the odd ones, after one exchange per pair of columns
                     const bool odd = (lane & 1) != 0;
                     const int feature = row >> 1;
+                    const bool weighed = part.act_pre != nullptr || part.act_post != nullptr;
 #pragma unroll
                     for (int i = 0; i < 32; i += 2) {
                         float mine = __uint_as_float(odd ? r[i] : r[i + 1]);       // what the partner needs
@@ -523,7 +529,11 @@ hgemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant_
                         float g = odd ? theirs : __uint_as_float(r[i]);
                         float u = odd ? __uint_as_float(r[i + 1]) : theirs;
                         int tok = tok0 + cb + i + (odd ? 1 : 0);
-                        const float w_in = __shfl_sync(0xffffffffu, pre, i + (odd ? 1 : 0)), w_out = __shfl_sync(0xffffffffu, post, i + (odd ? 1 : 0));
+                        float w_in = 1.0f, w_out = 1.0f;
+                        if (weighed) {  // uniform
+                            w_in = __shfl_sync(0xffffffffu, pre, i + (odd ? 1 : 0));
+                            w_out = __shfl_sync(0xffffffffu, post, i + (odd ? 1 : 0));
+                        }
                         if (row < tile.rows && tok < tile.tok_end) {
                             float a;
                             if (p.gated == 1 + GatedAct::Clamped) {
@@ -544,6 +554,10 @@ hgemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant_
                             if (tok < tile.tok_end) p.scatter.put(p.scatter.row(tok) + col, __uint_as_float(r[i]));
                         }
                     }
+                } else if (row < tile.rows && plain && tok0 + cb + 32 <= tile.tok_end) {
+                    float* out = dst + (int64_t)(tok0 + cb) * ld + row;
+#pragma unroll
+                    for (int i = 0; i < 32; ++i, out += ld) *out = __uint_as_float(r[i]);
                 } else if (row < tile.rows) {
 #pragma unroll
                     for (int i = 0; i < 32; ++i) {
