@@ -75,6 +75,10 @@ struct MatmulScatter {
     int64_t ld_part = 0, ld_row = 0, ld_block = 0;
     int block_shift = 31;
     const int32_t* row_map = nullptr;
+    // weight rows from rest_from on (a multiple of 32) go as f32 to rest[t * ld_rest + n - rest_from] instead
+    float* rest = nullptr;
+    int rest_from = 0;
+    int64_t ld_rest = 0;
 #ifdef __CUDACC__
     // Offset of weight row n's values, or -1 when they are not kept.
     __device__ __forceinline__ int64_t column(int64_t n) const {

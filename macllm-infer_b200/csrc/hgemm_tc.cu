@@ -545,6 +545,21 @@ hgemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant_
                             else part.yh[(int64_t)tok * part.ldyh + feature] = __float2half_rn(a);
                         }
                     }
+                } else if (p.scattered != 0 && p.scatter.rest != nullptr && row >= p.scatter.rest_from) {
+                    float* out = p.scatter.rest + (int64_t)(tok0 + cb) * p.scatter.ld_rest + row - p.scatter.rest_from;
+                    if (row < tile.rows) {
+#pragma unroll
+                        for (int i = 0; i < 32; ++i, out += p.scatter.ld_rest)
+                            if (tok0 + cb + i < tile.tok_end) *out = __uint_as_float(r[i]);
+                    }
+                } else if (p.scattered != 0 && p.scatter.type == MatmulScatter::BF16 && p.scatter.row_map == nullptr && p.scatter.block_shift == 31) {
+                    const int64_t col = row < tile.rows ? p.scatter.column(row) : -1;
+                    if (col >= 0) {
+                        __nv_bfloat16* out = static_cast<__nv_bfloat16*>(p.scatter.out) + (int64_t)(tok0 + cb) * p.scatter.ld_row + col;
+#pragma unroll
+                        for (int i = 0; i < 32; ++i, out += p.scatter.ld_row)
+                            if (tok0 + cb + i < tile.tok_end) *out = __float2bfloat16_rn(__uint_as_float(r[i]));
+                    }
                 } else if (p.scattered != 0) {
                     const int64_t col = row < tile.rows ? p.scatter.column(row) : -1;
                     if (col >= 0) {

@@ -500,14 +500,14 @@ bool linear_state_can_finish(int dim, int vdim) { return dim <= 128 && vdim <= L
 void launch_wkv_scan(const WkvScanArgs& a, cudaStream_t s) { launch_scan<LS_WKV>(a, s); }
 
 int launch_mlstm_scan(const MlstmScanArgs& a, cudaStream_t s) {
-    if (a.longest <= 1) {
+    if (a.longest <= 1 && a.yh == nullptr) {
         launch_mlstm_step(a, s);
         return 1;
     }
     MlstmScanArgs raw = a;
     raw.common.image = RowImage{};
     LinearStateArgs finish = a.common;
-    if (a.tensor_cores != 0) {
+    if (a.yh != nullptr) {
         launch_mlstm_chunks(raw, s);
     } else {
         launch_scan<LS_MLSTM>(raw, s);

@@ -60,15 +60,18 @@ struct MlstmScanArgs {
     LinearStateArgs common;
     Shares y;                        // columns q_col / k_col + head * dim + i, v_col + head * vdim + v, i_col / f_col + head
     int q_col = 0, k_col = 0, v_col = 0, i_col = 0, f_col = 0;
+    const __nv_bfloat16* yh = nullptr;  // q, k and v come from these rows [rows][ldh] instead (16-byte aligned, ldh a multiple of 8):
+    int ldh = 0;                        // what the chunked form reads
     const float* i_bias = nullptr;   // [heads]
     const float* f_bias = nullptr;
     float cap = 1.f;
     float* running_max = nullptr;    // [slot halves][heads]
     int32_t* counters = nullptr;     // [lanes][heads], zero before the first call; every call leaves them zero
     int rows = 0, longest = 0;       // of all lanes, of the longest one
-    int tensor_cores = 0;            // prompts as products of 64-row chunks, else row by row in f32; queries, keys and values are rounded to bfloat16
+    int rounded = 0;                 // queries, keys and values are rounded to bfloat16 (as the chunked form has them)
 };
-// Always finishes (common.image is set, common.out is scratch).  Returns the number of kernels launched.
+// One-token lanes, prompts in chunks (yh set), prompts row by row in f32 (otherwise).  Always finishes (common.image is set,
+// common.out is scratch).  Returns the number of kernels launched.
 int launch_mlstm_scan(const MlstmScanArgs& a, cudaStream_t s);
 // The forms behind it (mlstm.cu): one-token lanes, finished; chunks of prompts, whose raw rows are [heads][vdim] and divided already.
 void launch_mlstm_step(const MlstmScanArgs& a, cudaStream_t s);

@@ -341,7 +341,7 @@ void MixerLm::alloc_activations() {
     int64_t q_lat = 0, uq = 0, lat = 0, cat = 0;  // widths of latent attention's rows, and of `out`'s input with both branches
     int lat_ctas = 1;
     int64_t lat_part = 0;
-    int64_t mlstm_heads = 0;
+    int64_t mlstm_heads = 0, qkv = 0;
     int64_t pairs = 0, experts = 0, expert_ff = 0, expert_gu = 0;  // routed rows, experts, widths of an expert's activations
     for (size_t l = 0; l < lw_.size(); ++l) {
         const MixerLayerSpec& s = ms_.layers[l];
@@ -356,6 +356,7 @@ void MixerLm::alloc_activations() {
         }
         if (s.kind == MixerKind::Mlstm) {
             mlstm_heads = std::max(mlstm_heads, (int64_t)s.mlstm.heads);
+            qkv = std::max(qkv, (int64_t)w.c_g);
             b_w = std::max(b_w, (int64_t)s.mlstm.heads * s.mlstm.vdim);
             raw = std::max(raw, (int64_t)s.mlstm.heads * linear_state_raw_width(s.mlstm.vdim));
         } else if (s.kind == MixerKind::Attention) {
@@ -414,6 +415,7 @@ void MixerLm::alloc_activations() {
     if (f32_) y_gu_.alloc((size_t)std::max(T * 2 * ff, pairs * expert_gu) * 4);
     mlstm_counters_.alloc((size_t)(B * mlstm_heads) * 4);
     mlstm_counters_.zero(stream_);
+    if (!f32_) img_qkv_.alloc((size_t)(T * qkv) * 2);
     if (pairs > 0) {
         img_rows_.alloc((size_t)(pairs * ldc) * esz_);
         img_expert_ff_.alloc((size_t)(pairs * expert_ff) * esz_);

@@ -175,7 +175,7 @@ private:
     void run_side_by_side(const Tick& t, int run, Pending& p, const std::vector<LmLane>& lanes);
     // layers whose norms sit on what the sublayers give
     void run_output_norm(const Tick& t, int run, Pending& p, const std::vector<LmLane>& lanes);
-    void run_mlstm(const Tick& t, int run, const Shares& y, const RowImage& out);
+    void run_mlstm(const Tick& t, int run, const RowImage& in, const RowImage& out);
     void run_moe(const Tick& t, int layer, Pending& p);
     void run_latent(const Tick& t, int run, const Shares& y, const RowImage& out, const std::vector<LmLane>& lanes);
     void run_latent_wide(const Tick& t, int run, const Shares& y, const RowImage& out);
@@ -207,7 +207,7 @@ private:
     MoeRows moe_;
     int moe_half_ = 0;  // of the counts, alternates from layer to layer
     DevBuf moe_words_, img_rows_, img_expert_ff_, routed_;
-    DevBuf mlstm_counters_;
+    DevBuf mlstm_counters_, img_qkv_;
     DevBuf attn_part_o_, attn_part_ml_, attn_counters_;
     int attn_max_entries_ = 0;
     int cur_ = 0;             // which of x_ holds the residual stream

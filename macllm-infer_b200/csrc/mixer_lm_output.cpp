@@ -18,7 +18,7 @@ void MixerLm::load_output_norm(const SafetensorsFile& f, int l) {
     auto part = [&](const char* name, int rows) {
         const int here = at;
         parts.push_back({m + name, rows, here});
-        at = pad_to(at + rows, 4);
+        at = pad_to(at + rows, 8);
         return here;
     };
     if (s.kind == MixerKind::Mlstm) {
@@ -27,6 +27,7 @@ void MixerLm::load_output_norm(const SafetensorsFile& f, int l) {
         w.c_q = part("q", kw);
         w.c_k = part("k", kw);
         w.c_v = part("v", vw);
+        at = pad_to(at, 128);  // what stays in f32 on prompts begins here
         w.c_g = part("g", vw);
         w.c_i = part("i", x.heads);
         w.c_f = part("f", x.heads);
@@ -103,12 +104,12 @@ void MixerLm::run_output_norm(const Tick& t, int run, Pending& pend, const std::
     launch_row_update(u, stream_);
     prof_end();
     ++launches_;
-    const Shares y = matmul(w.in, u.raw, T, y_in_, 0);
     RowImage mixed;
     if (s.kind == MixerKind::Mlstm) {
         mixed = image(img_b_, w.out.ld);
-        run_mlstm(t, run, y, mixed);
+        run_mlstm(t, run, u.raw, mixed);
     } else {
+        const Shares y = matmul(w.in, u.raw, T, y_in_, 0);
         mixed = image(img_a_, w.out.ld);
         attend(t, run, s.attn, y, lanes);
         const double gate = s.attn.gate == OutputGate::Value ? 4.0 : 0.0;
@@ -125,12 +126,34 @@ void MixerLm::run_output_norm(const Tick& t, int run, Pending& pend, const std::
     if (s.ff > 0) run_moe(t, l, pend);
 }
 
-void MixerLm::run_mlstm(const Tick& t, int run, const Shares& y, const RowImage& out) {
+void MixerLm::run_mlstm(const Tick& t, int run, const RowImage& in, const RowImage& out) {
     const int l = runs_[(size_t)run].layer, T = t.T;
     const MlstmSpec& s = ms_.layers[(size_t)l].mlstm;
     Layer& w = lw_[(size_t)l];
     RunState& st = rs_[(size_t)run];
     MlstmScanArgs a;
+    const bool chunked = !f32_ && longest_ > 1;
+    Shares y;
+    int from = 0;  // the first projection column that `y` holds
+    if (chunked) {
+        // queries, keys and values leave the matmul as bfloat16, the gates as f32
+        from = w.c_g;
+        MatmulScatter to;
+        to.out = img_qkv_.ptr();
+        to.type = MatmulScatter::BF16;
+        to.part_rows = to.part_valid = from;
+        to.ld_row = from;
+        to.rest = y_in_.as<float>();
+        to.rest_from = from;
+        to.ld_rest = w.in.rows - from;
+        matmul_scatter(w.in, in, T, to);
+        y.p = y_in_.as<float>();
+        y.ld = (int)to.ld_rest;
+        a.yh = img_qkv_.as<__nv_bfloat16>();
+        a.ldh = from;
+    } else {
+        y = matmul(w.in, in, T, y_in_, 0);
+    }
     a.common.lanes = state_lanes_;
     a.common.state = st.state.as<float>();
     a.common.heads = s.heads;
@@ -142,13 +165,13 @@ void MixerLm::run_mlstm(const Tick& t, int run, const Shares& y, const RowImage&
     a.common.norm_per_head = 1;
     a.common.eps = ms_.eps;
     a.common.gate = y;
-    a.common.gate_col = w.c_g;
+    a.common.gate_col = w.c_g - from;
     a.y = y;
     a.q_col = w.c_q;
     a.k_col = w.c_k;
     a.v_col = w.c_v;
-    a.i_col = w.c_i;
-    a.f_col = w.c_f;
+    a.i_col = w.c_i - from;
+    a.f_col = w.c_f - from;
     a.i_bias = w.i_b.as<float>();
     a.f_bias = w.f_b.as<float>();
     a.cap = s.gate_cap;
@@ -157,9 +180,9 @@ void MixerLm::run_mlstm(const Tick& t, int run, const Shares& y, const RowImage&
     a.counters = mlstm_counters_.as<int32_t>();
     a.rows = T;
     a.longest = longest_;
-    a.tensor_cores = f32_ ? 0 : 1;
+    a.rounded = f32_ ? 0 : 1;
     const double vw = (double)s.heads * s.vdim, kw = (double)s.heads * s.dim;
-    prof_begin(KC_MLSTM_SCAN, 4.0 * T * (2.0 * kw + 2.0 * vw) + T * vw * esz_ + 8.0 * t.B * (vw + s.heads) * s.dim, 6.0 * T * vw * s.dim);
+    prof_begin(KC_MLSTM_SCAN, (chunked ? 2.0 : 4.0) * T * (2.0 * kw + vw) + 4.0 * T * vw + T * vw * esz_ + 8.0 * t.B * (vw + s.heads) * s.dim, 6.0 * T * vw * s.dim);
     launches_ += launch_mlstm_scan(a, stream_);
     prof_end();
 }

@@ -8,7 +8,7 @@
 // running maximum and m_0, S, n what the chunk starts from,
 //   c_s = i_s - F_s,  e_t = m_t - F_t:   D_ts = exp(c_s - e_t) (s <= t),  g_t = exp(m_0 - e_t),
 //   o_t = sum_s D_ts (q_t . k_s) v_s + g_t S^T q_t,   S' = g_last S + sum_s exp(c_s - e_last) k_s v_s^T,
-// every exponent at most 0.  q, k and v are bfloat16 numbers; what the recurrence adds to them - D (Q K^T), the written values and the
+// every exponent at most 0.  q, k and v are bfloat16 numbers, as the projection's epilogue leaves them; what the recurrence adds to them - D (Q K^T), the written values and the
 // state - enters a product as the sum of two bfloat16 numbers (16 bits and more), and the state itself stays in f32 registers.
 #include "linear_state.h"
 #include "device_util.h"
@@ -93,7 +93,7 @@ __global__ void __launch_bounds__(MS_WARPS * 32, 4) mlstm_step_kernel(const __gr
     const int64_t row = sl.first;
     float4 q[NJ], k[NJ];
     // the numbers a prompt's chunks would multiply
-    auto operand = [&](float x) { return a.tensor_cores ? __bfloat162float(__float2bfloat16_rn(x)) : x; };
+    auto operand = [&](float x) { return a.rounded ? __bfloat162float(__float2bfloat16_rn(x)) : x; };
     auto keys = [&](int col, int j) {
         const int d = (j * LPC + lk) * 4;
         float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
@@ -201,7 +201,10 @@ __global__ void __launch_bounds__(MS_WARPS * 32, 4) mlstm_step_kernel(const __gr
 
 constexpr int MC_ROWS = 64;      // rows of a chunk
 constexpr int MC_WARPS = 16;
-constexpr int MC_THREADS = MC_WARPS * 32;
+constexpr int MC_THREADS = MC_WARPS * 32;           // that compute; one more warp keeps the gates a chunk ahead
+
+// All warps of the CTA, the gates' one included.
+__device__ __forceinline__ void mc_sync() { asm volatile("bar.sync 1, %0;" ::"n"(MC_THREADS + 32) : "memory"); }
 
 __device__ __forceinline__ uint32_t mc_smem(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
 __device__ __forceinline__ void mc_ldmatrix(uint32_t (&r)[4], const __nv_bfloat16* p) {
@@ -215,8 +218,9 @@ __device__ __forceinline__ void mc_mma(float (&c)[4], const uint32_t (&a)[4], ui
                  : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
                  : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
-__device__ __forceinline__ void mc_cp_async16(void* dst, const void* src) {
-    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(mc_smem(dst)), "l"(src) : "memory");
+__device__ __forceinline__ void mc_cp_async16(void* dst, const void* src, bool valid) {
+    const int bytes = valid ? 16 : 0;  // 0: the 16 bytes become zeros
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(mc_smem(dst)), "l"(src), "r"(bytes) : "memory");
 }
 // x and y as bfloat16 numbers, and what that left of them.
 __device__ __forceinline__ void mc_split(float x, float y, uint32_t& hi, uint32_t& lo) {
@@ -280,36 +284,96 @@ struct Chunk {
     static constexpr int KP = KD + 8, CP = C + 8, PP = MC_ROWS + 8;  // padded rows (bfloat16): conflict-free ldmatrix
     static constexpr int COL_GROUPS = C / 16, KEY_GROUPS = MC_WARPS / COL_GROUPS, KEYS = KD / KEY_GROUPS;  // of the state, by warp
     static constexpr int N_PARTS = MC_THREADS / (KD / 2);            // row groups of the normaliser's sums
-    static constexpr bool STAGED = KD <= 128;                        // the next chunk's projections are on their way meanwhile
-    static constexpr int HALVES = 2 * MC_ROWS * KP + 3 * MC_ROWS * CP + 2 * MC_ROWS * PP + 2 * C * KP;
-    static constexpr int FLOATS = 12 * MC_ROWS + KD + N_PARTS * KD + 4;
-    static constexpr int STAGE = STAGED ? MC_ROWS * (2 * KD + C) : 0;
-    static constexpr size_t BYTES = (size_t)HALVES * 2 + (size_t)(FLOATS + STAGE) * 4;
-    static_assert(KEYS % 8 == 0 && C % 32 == 0, "whole tiles");
+    static constexpr int INPUTS = MC_ROWS * (2 * KP + CP);           // one chunk's q, k, v
+    static constexpr int HALVES = 2 * INPUTS + 2 * MC_ROWS * CP + 2 * MC_ROWS * PP + 2 * C * KP;
+    static constexpr int GATES = 7 * MC_ROWS + 4;                    // one chunk's
+    static constexpr int FLOATS = 2 * GATES + 5 * MC_ROWS + KD + N_PARTS * KD;
+    static constexpr size_t BYTES = (size_t)HALVES * 2 + (size_t)FLOATS * 4;
+    static_assert(KEYS % 8 == 0 && C % 32 == 0 && BYTES <= 227 * 1024, "whole tiles that fit");
 };
 
-// Grid (column slices of C, heads, lanes).
+// What the chunk's exponents are made of (see the top), by row.
+struct ChunkGates {
+    float2 *c, *e;                    // in units of ln 2, two parts each
+    float *g, *w, *floor, *keep;
+    __device__ __forceinline__ explicit ChunkGates(float* at) {
+        c = reinterpret_cast<float2*>(at);
+        e = c + MC_ROWS;
+        g = reinterpret_cast<float*>(e + MC_ROWS);
+        w = g + MC_ROWS;
+        floor = w + MC_ROWS;
+        keep = floor + MC_ROWS;
+    }
+};
+
+// One warp, two rows per lane: the gates of `m` rows behind a running maximum, which it moves on.  Sums and maxima in f64:
+// differences of far sums stay exact.
+__device__ __forceinline__ void chunk_gates(const MlstmScanArgs& a, int64_t first, int m, int head, float& run_max, const ChunkGates& out, int lane) {
+    constexpr double kLog2e = 1.4426950408889634074;
+    double li[2], lf[2];
+#pragma unroll
+    for (int h = 0; h < 2; ++h) {
+        const int r = 2 * lane + h;
+        li[h] = r < m ? (double)log_input_gate(a, first + r, head) : -INFINITY;  // rows past the end change neither sums nor maxima
+        lf[h] = r < m ? (double)log_forget_gate(a, first + r, head) : 0.0;
+    }
+    double f1 = lf[0] + lf[1];
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+        const double p = __shfl_up_sync(0xffffffffu, f1, o);
+        if (lane >= o) f1 += p;
+    }
+    const double F[2] = {f1 - lf[1], f1};
+    const double c[2] = {li[0] - F[0], li[1] - F[1]};
+    double best = fmax(c[0], c[1]);
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+        const double p = __shfl_up_sync(0xffffffffu, best, o);
+        if (lane >= o) best = fmax(best, p);
+    }
+    double earlier = __shfl_up_sync(0xffffffffu, best, 1);
+    if (lane == 0) earlier = -INFINITY;
+    const double top[2] = {F[0] + fmax((double)run_max, fmax(earlier, c[0])), F[1] + fmax((double)run_max, best)};
+    double e[2];
+    float mt[2];
+#pragma unroll
+    for (int h = 0; h < 2; ++h) {
+        mt[h] = (float)top[h];
+        e[h] = (double)mt[h] - F[h];
+    }
+    const double e_last = __shfl_sync(0xffffffffu, e[1], 31);
+#pragma unroll
+    for (int h = 0; h < 2; ++h) {
+        const int r = 2 * lane + h;
+        const double c2 = c[h] * kLog2e, e2 = e[h] * kLog2e;
+        const float c_hi = (float)c2, e_hi = (float)e2;
+        out.c[r] = make_float2(c_hi, r < m ? (float)(c2 - (double)c_hi) : 0.f);
+        out.e[r] = make_float2(e_hi, (float)(e2 - (double)e_hi));
+        out.g[r] = expf((float)(run_max - e[h]));
+        out.w[r] = expf((float)(c[h] - e_last));
+        out.floor[r] = expf(-mt[h]);
+    }
+    if (lane == 0) *out.keep = expf((float)(run_max - e_last));
+    run_max = __shfl_sync(0xffffffffu, mt[1], 31);
+}
+
+// Grid (column slices of C, heads, lanes).  vec: rows of q, k and v in whole 16-byte pieces.
 template <int KD, int C>
-__global__ void __launch_bounds__(MC_THREADS, 1) mlstm_chunk_kernel(const __grid_constant__ MlstmScanArgs a, int vec) {
+__global__ void __launch_bounds__(MC_THREADS + 32, 1) mlstm_chunk_kernel(const __grid_constant__ MlstmScanArgs a, int vec) {
     using P = Chunk<KD, C>;
     constexpr int KP = P::KP, CP = P::CP, PP = P::PP, R = MC_ROWS;
     constexpr int NT = C / 32;            // output tiles of a warp: 16 rows x C / 4 columns
     constexpr int NK = P::KEYS / 8;       // state tiles of a warp: 16 columns x KEYS keys
     extern __shared__ __align__(16) unsigned char mc_raw[];
-    __nv_bfloat16* Q = reinterpret_cast<__nv_bfloat16*>(mc_raw);   // [R][KP]
-    __nv_bfloat16* K = Q + R * KP;                                  // [R][KP]
-    __nv_bfloat16* V = K + R * KP;                                  // [R][CP]
-    __nv_bfloat16* Wh = V + R * CP;                                 // written values, [R][CP] in two parts
+    __nv_bfloat16* inputs = reinterpret_cast<__nv_bfloat16*>(mc_raw);  // [2]: q [R][KP], k [R][KP], v [R][CP]
+    __nv_bfloat16* Wh = inputs + 2 * P::INPUTS;                     // written values, [R][CP] in two parts
     __nv_bfloat16* Wl = Wh + R * CP;
     __nv_bfloat16* Ph = Wl + R * CP;                                // D (Q K^T), [R][PP] in two parts
     __nv_bfloat16* Pl = Ph + R * PP;
     __nv_bfloat16* Sh = Pl + R * PP;                                // the state the chunk starts from, [C][KP] in two parts
     __nv_bfloat16* Sl = Sh + C * KP;
-    float2* s_c = reinterpret_cast<float2*>(Sl + C * KP);           // c_s and e_t in units of ln 2, two parts each
-    float2* s_e = s_c + R;
-    float *s_g = reinterpret_cast<float*>(s_e + R), *s_w = s_g + R, *s_floor = s_w + R, *s_nq = s_floor + R;
-    float *s_sum = s_nq + R /* [4][R] */, *s_n = s_sum + 4 * R, *s_np = s_n + KD /* [N_PARTS][KD] */, *s_keep = s_np + P::N_PARTS * KD;
-    float* stage = s_keep + 4;                                      // [R][KD], [R][KD], [R][C]
+    float* gates = reinterpret_cast<float*>(Sl + C * KP);           // [2]
+    float *s_nq = gates + 2 * P::GATES, *s_sum = s_nq + R /* [4][R] */, *s_n = s_sum + 4 * R, *s_np = s_n + KD /* [N_PARTS][KD] */;
 
     const LinearStateArgs& cm = a.common;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, gid = lane >> 2, tq = lane & 3;
@@ -320,6 +384,24 @@ __global__ void __launch_bounds__(MC_THREADS, 1) mlstm_chunk_kernel(const __grid
 
     pdl_trigger();
     const StateLane sl = cm.lanes.at(blockIdx.z);
+    const int n = sl.n, chunks = (n + R - 1) / R;
+
+    if (warp == MC_WARPS) {
+        // the gates' warp: a chunk ahead of the others, whom it meets at every barrier
+        float run_max = sl.in >= 0 ? a.running_max[(int64_t)sl.in * cm.heads + head] : 0.f;
+        pdl_wait();
+        for (int ch = 0; ch <= chunks; ++ch) {
+            if (ch < chunks) chunk_gates(a, sl.first + (int64_t)ch * R, min(R, n - ch * R), head, run_max, ChunkGates(gates + (ch & 1) * P::GATES), lane);
+            if (ch > 0) {
+                mc_sync();
+                mc_sync();
+            }
+            if (ch < chunks) mc_sync();
+        }
+        if (blockIdx.x == 0 && lane == 0) a.running_max[(int64_t)sl.out * cm.heads + head] = run_max;
+        return;
+    }
+
     float S[NK][4];
     {
         const float* src = cm.state + ((int64_t)sl.in * cm.heads + head) * head_state;
@@ -335,7 +417,6 @@ __global__ void __launch_bounds__(MC_THREADS, 1) mlstm_chunk_kernel(const __grid
             }
         for (int i = threadIdx.x; i < KD; i += MC_THREADS) s_n[i] = sl.in >= 0 ? src[(int64_t)cm.vdim * KD + i] : 0.f;
     }
-    float run_max = sl.in >= 0 ? a.running_max[(int64_t)sl.in * cm.heads + head] : 0.f;  // warp 0's counts
     auto publish_state = [&] {
 #pragma unroll
         for (int j = 0; j < NK; ++j)
@@ -351,144 +432,64 @@ __global__ void __launch_bounds__(MC_THREADS, 1) mlstm_chunk_kernel(const __grid
     publish_state();
     pdl_wait();
 
-    const int n = sl.n, chunks = (n + R - 1) / R;
     const int qc = a.q_col + head * cm.dim, kc = a.k_col + head * cm.dim, vc = a.v_col + head * cm.vdim + col0;
-    const bool staged = P::STAGED && vec;
-    float *st_q = stage, *st_k = stage + R * KD, *st_v = stage + 2 * R * KD;
+    // a chunk's q, k and v on their way; rows past the end and columns past the head are zeros
     auto request = [&](int chunk) {
-        const float* y = a.y.p + ((int64_t)sl.first + (int64_t)chunk * R) * a.y.ld;
+        __nv_bfloat16* Q = inputs + (chunk & 1) * P::INPUTS;
+        __nv_bfloat16 *K = Q + R * KP, *V = K + R * KP;
+        const __nv_bfloat16* y = a.yh + ((int64_t)sl.first + (int64_t)chunk * R) * a.ldh;
         const int m = min(R, n - chunk * R);
-        for (int i = threadIdx.x; i < m * (KD / 4); i += MC_THREADS) {
-            const int r = i / (KD / 4), c = i % (KD / 4) * 4;
-            if (c < cm.dim) {
-                mc_cp_async16(st_q + r * KD + c, y + (int64_t)r * a.y.ld + qc + c);
-                mc_cp_async16(st_k + r * KD + c, y + (int64_t)r * a.y.ld + kc + c);
+        if (vec) {
+#pragma unroll
+            for (int i = threadIdx.x; i < R * (KD / 8); i += MC_THREADS) {
+                const int r = i / (KD / 8), c = i % (KD / 8) * 8;
+                const bool live = r < m && c < cm.dim;
+                const __nv_bfloat16* src = y + (live ? (int64_t)r * a.ldh + c : 0);
+                mc_cp_async16(Q + r * KP + c, src + qc, live);
+                mc_cp_async16(K + r * KP + c, src + kc, live);
             }
-        }
-        for (int i = threadIdx.x; i < m * (C / 4); i += MC_THREADS) {
-            const int r = i / (C / 4), c = i % (C / 4) * 4;
-            if (c < cols) mc_cp_async16(st_v + r * C + c, y + (int64_t)r * a.y.ld + vc + c);
+            for (int i = threadIdx.x; i < R * (C / 8); i += MC_THREADS) {
+                const int r = i / (C / 8), c = i % (C / 8) * 8;
+                const bool live = r < m && c < cols;
+                mc_cp_async16(V + r * CP + c, y + vc + (live ? (int64_t)r * a.ldh + c : 0), live);
+            }
+        } else {
+            const __nv_bfloat16 zero = __float2bfloat16_rn(0.f);
+            for (int i = threadIdx.x; i < R * KD; i += MC_THREADS) {
+                const int r = i / KD, c = i % KD;
+                const bool live = r < m && c < cm.dim;
+                Q[r * KP + c] = live ? y[(int64_t)r * a.ldh + qc + c] : zero;
+                K[r * KP + c] = live ? y[(int64_t)r * a.ldh + kc + c] : zero;
+            }
+            for (int i = threadIdx.x; i < R * C; i += MC_THREADS) {
+                const int r = i / C, c = i % C;
+                V[r * CP + c] = r < m && c < cols ? y[(int64_t)r * a.ldh + vc + c] : zero;
+            }
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
-    // the gates of rows 2 lane and 2 lane + 1 (warp 0), a chunk ahead
-    float li[2], lf[2];
-    auto fetch_gates = [&](int chunk) {
-#pragma unroll
-        for (int h = 0; h < 2; ++h) {
-            const int r = chunk * R + 2 * lane + h;
-            li[h] = -INFINITY;
-            lf[h] = 0.f;
-            if (r < n) {
-                li[h] = log_input_gate(a, sl.first + r, head);
-                lf[h] = log_forget_gate(a, sl.first + r, head);
-            }
-        }
-    };
-    if (chunks > 0) {
-        if (staged) request(0);
-        if (warp == 0) fetch_gates(0);
-    }
+    if (chunks > 0) request(0);
     const float q_scale = rsqrtf((float)cm.dim);
+    const bool even = (cm.vdim & 1) == 0;
 
     for (int ch = 0; ch < chunks; ++ch) {
         const int64_t r0 = sl.first + (int64_t)ch * R;
         const int m = min(R, n - ch * R);
-        if (warp == 0) {
-            // sums and running maxima of the chunk's rows, two per lane, in f64: differences of far sums stay exact
-            constexpr double kLog2e = 1.4426950408889634074;
-            double f1 = (double)lf[0] + lf[1];
+        const ChunkGates gt(gates + (ch & 1) * P::GATES);
+        const __nv_bfloat16* Q = inputs + (ch & 1) * P::INPUTS;
+        const __nv_bfloat16 *K = Q + R * KP, *V = K + R * KP;
+        asm volatile("cp.async.wait_group 0;" ::: "memory");
+        mc_sync();  // the chunk's inputs and gates, the state and the normaliser it starts from
+        if (ch + 1 < chunks) request(ch + 1);
+        // what the rows write: v times the weight that is left of it at the chunk's end
 #pragma unroll
-            for (int o = 1; o < 32; o <<= 1) {
-                const double p = __shfl_up_sync(0xffffffffu, f1, o);
-                if (lane >= o) f1 += p;
-            }
-            const double F[2] = {f1 - lf[1], f1};
-            const double c[2] = {li[0] - F[0], li[1] - F[1]};
-            double best = fmax(c[0], c[1]);
-#pragma unroll
-            for (int o = 1; o < 32; o <<= 1) {
-                const double p = __shfl_up_sync(0xffffffffu, best, o);
-                if (lane >= o) best = fmax(best, p);
-            }
-            double earlier = __shfl_up_sync(0xffffffffu, best, 1);
-            if (lane == 0) earlier = -INFINITY;
-            const double top[2] = {F[0] + fmax((double)run_max, fmax(earlier, c[0])), F[1] + fmax((double)run_max, best)};
-            double e[2];
-            float mt[2];
-#pragma unroll
-            for (int h = 0; h < 2; ++h) {
-                mt[h] = (float)top[h];
-                e[h] = (double)mt[h] - F[h];
-            }
-            const double e_last = __shfl_sync(0xffffffffu, e[1], 31);  // rows past the end change neither sums nor maxima
-#pragma unroll
-            for (int h = 0; h < 2; ++h) {
-                const int r = 2 * lane + h;
-                const double c2 = c[h] * kLog2e, e2 = e[h] * kLog2e;
-                const float ch_hi = (float)c2, eh_hi = (float)e2;
-                s_c[r] = make_float2(ch_hi, c[h] == -INFINITY ? 0.f : (float)(c2 - (double)ch_hi));
-                s_e[r] = make_float2(eh_hi, (float)(e2 - (double)eh_hi));
-                s_g[r] = expf((float)(run_max - e[h]));
-                s_w[r] = expf((float)(c[h] - e_last));
-                s_floor[r] = expf(-mt[h]);
-            }
-            if (lane == 0) *s_keep = expf((float)(run_max - e_last));
-            run_max = __shfl_sync(0xffffffffu, mt[1], 31);
-        }
-        // q, k, v as bfloat16, rows past the end as zeros
-        if (staged) asm volatile("cp.async.wait_group 0;" ::: "memory");
-        __syncthreads();  // the staged rows, the gates; everyone is through with the chunk before
-        if (staged) {
-            for (int i = threadIdx.x; i < R * (KD / 4); i += MC_THREADS) {
-                const int r = i / (KD / 4), c = i % (KD / 4) * 4;
-                float4 x = make_float4(0.f, 0.f, 0.f, 0.f), y = x;
-                if (r < m && c < cm.dim) {
-                    x = *reinterpret_cast<const float4*>(st_q + r * KD + c);
-                    y = *reinterpret_cast<const float4*>(st_k + r * KD + c);
-                }
-                const __nv_bfloat162 x0 = __floats2bfloat162_rn(x.x, x.y), x1 = __floats2bfloat162_rn(x.z, x.w);
-                const __nv_bfloat162 y0 = __floats2bfloat162_rn(y.x, y.y), y1 = __floats2bfloat162_rn(y.z, y.w);
-                *reinterpret_cast<uint2*>(Q + r * KP + c) = make_uint2(*reinterpret_cast<const uint32_t*>(&x0), *reinterpret_cast<const uint32_t*>(&x1));
-                *reinterpret_cast<uint2*>(K + r * KP + c) = make_uint2(*reinterpret_cast<const uint32_t*>(&y0), *reinterpret_cast<const uint32_t*>(&y1));
-            }
-        } else {
-            for (int i = threadIdx.x; i < R * KD; i += MC_THREADS) {
-                const int r = i / KD, c = i % KD;
-                const bool live = r < m && c < cm.dim;
-                Q[r * KP + c] = __float2bfloat16_rn(live ? a.y.at(r0 + r, qc + c) : 0.f);
-                K[r * KP + c] = __float2bfloat16_rn(live ? a.y.at(r0 + r, kc + c) : 0.f);
-            }
-        }
         for (int i = threadIdx.x; i < R * (C / 2); i += MC_THREADS) {
             const int r = i / (C / 2), c = i % (C / 2) * 2;
-            float2 x = make_float2(0.f, 0.f);
-            if (r < m) {
-                if (staged) {
-                    if (c < cols) x = *reinterpret_cast<const float2*>(st_v + r * C + c);
-                } else {
-                    if (c < cols) x.x = a.y.at(r0 + r, vc + c);
-                    if (c + 1 < cols) x.y = a.y.at(r0 + r, vc + c + 1);
-                }
-            }
-            const __nv_bfloat162 v = __floats2bfloat162_rn(x.x, x.y);
-            *reinterpret_cast<__nv_bfloat162*>(V + r * CP + c) = v;
+            const __nv_bfloat162 v = *reinterpret_cast<const __nv_bfloat162*>(V + r * CP + c);
             uint32_t hi, lo;
-            mc_split(s_w[r] * __low2float(v), s_w[r] * __high2float(v), hi, lo);
+            mc_split(gt.w[r] * __low2float(v), gt.w[r] * __high2float(v), hi, lo);
             *reinterpret_cast<uint32_t*>(Wh + r * CP + c) = hi;
             *reinterpret_cast<uint32_t*>(Wl + r * CP + c) = lo;
-        }
-        if (ch > 0)  // the normaliser the chunk starts from: what was kept and the sums of the chunk before, by row groups
-            for (int i = threadIdx.x; i < KD; i += MC_THREADS) {
-                float x = s_n[i];
-#pragma unroll
-                for (int p = 0; p < P::N_PARTS; ++p) x += s_np[p * KD + i];
-                s_n[i] = x;
-            }
-        __syncthreads();  // the staging rows are free, the operands are there
-        if (ch + 1 < chunks) {
-            if (staged) request(ch + 1);
-            if (warp == 0) fetch_gates(ch + 1);
         }
         auto q_fragment = [&](int k, uint32_t (&r)[4]) { mc_ldmatrix(r, Q + (row0 + (lane & 15)) * KP + k * 16 + (lane >> 4) * 8); };
 
@@ -499,11 +500,11 @@ __global__ void __launch_bounds__(MC_THREADS, 1) mlstm_chunk_kernel(const __grid
             uint32_t hi[2][2] = {}, lo[2][2] = {};
             if (k0 <= row0) {
                 mc_product<2, KD / 16, false, KP>(sc, lane, q_fragment, [&](int k, int j) { return (k0 + j * 8) * KP + k * 16; }, K, nullptr);
-                const float2 e[2] = {s_e[row0 + gid], s_e[row0 + gid + 8]};
+                const float2 e[2] = {gt.e[row0 + gid], gt.e[row0 + gid + 8]};
 #pragma unroll
                 for (int j = 0; j < 2; ++j) {
                     const int s = k0 + j * 8 + 2 * tq;
-                    const float4 c = *reinterpret_cast<const float4*>(s_c + s);
+                    const float4 c = *reinterpret_cast<const float4*>(gt.c + s);
 #pragma unroll
                     for (int h = 0; h < 2; ++h) {
                         const int t = row0 + gid + 8 * h;
@@ -541,7 +542,7 @@ __global__ void __launch_bounds__(MC_THREADS, 1) mlstm_chunk_kernel(const __grid
             for (int x = 1; x < 8; x <<= 1) nq += __shfl_xor_sync(0xffffffffu, nq, x);
             if (part == 0) s_nq[t] = nq;
         }
-        __syncthreads();
+        mc_sync();
 
         // outputs: 16 rows x C / 4 columns per warp
         {
@@ -552,9 +553,9 @@ __global__ void __launch_bounds__(MC_THREADS, 1) mlstm_chunk_kernel(const __grid
 #pragma unroll
             for (int h = 0; h < 2; ++h) {
                 const int t = row0 + gid + 8 * h;
-                g[h] = s_g[t] * q_scale;
+                g[h] = gt.g[t] * q_scale;
                 const float nq = s_sum[t] + s_sum[R + t] + s_sum[2 * R + t] + s_sum[3 * R + t] + g[h] * s_nq[t];
-                den[h] = fmaxf(fabsf(nq), s_floor[t]) + 1e-6f;
+                den[h] = fmaxf(fabsf(nq), gt.floor[t]) + 1e-6f;
             }
 #pragma unroll
             for (int j = 0; j < NT; ++j)
@@ -579,7 +580,7 @@ __global__ void __launch_bounds__(MC_THREADS, 1) mlstm_chunk_kernel(const __grid
                 for (int j = 0; j < NT; ++j) {
                     const int c = n0 + j * 8 + 2 * tq;
                     const float x = o[j][2 * h] * inv, y = o[j][2 * h + 1] * inv;
-                    if (vec) {
+                    if (even) {
                         if (c < cols) *reinterpret_cast<float2*>(out + c) = make_float2(x, y);
                     } else {
                         if (c < cols) out[c] = x;
@@ -589,7 +590,7 @@ __global__ void __launch_bounds__(MC_THREADS, 1) mlstm_chunk_kernel(const __grid
             }
         }
         // the state behind the chunk: 16 columns x KEYS keys per warp
-        const float keep = *s_keep;
+        const float keep = *gt.keep;
 #pragma unroll
         for (int j = 0; j < NK; ++j)
 #pragma unroll
@@ -608,17 +609,19 @@ __global__ void __launch_bounds__(MC_THREADS, 1) mlstm_chunk_kernel(const __grid
 #pragma unroll
             for (int t = part * ROWS; t < (part + 1) * ROWS; ++t) {
                 const __nv_bfloat162 k2 = *reinterpret_cast<const __nv_bfloat162*>(K + t * KP + pair);
-                x = fmaf(s_w[t], __low2float(k2), x);
-                y = fmaf(s_w[t], __high2float(k2), y);
+                x = fmaf(gt.w[t], __low2float(k2), x);
+                y = fmaf(gt.w[t], __high2float(k2), y);
             }
             *reinterpret_cast<float2*>(s_np + part * KD + pair) = make_float2(x, y);
-            if (part == 0) {
-                s_n[pair] *= keep;  // the sums are added behind the next barrier
-                s_n[pair + 1] *= keep;
-            }
         }
-        __syncthreads();  // the old state was read by everyone
-        if (ch + 1 < chunks) publish_state();
+        mc_sync();  // the old state was read by everyone
+        publish_state();
+        for (int i = threadIdx.x; i < KD; i += MC_THREADS) {
+            float x = s_n[i] * keep;
+#pragma unroll
+            for (int p = 0; p < P::N_PARTS; ++p) x += s_np[p * KD + i];
+            s_n[i] = x;
+        }
     }
 
     float* dst = cm.state + ((int64_t)sl.out * cm.heads + head) * head_state;
@@ -630,13 +633,7 @@ __global__ void __launch_bounds__(MC_THREADS, 1) mlstm_chunk_kernel(const __grid
             if (col < cm.vdim) *reinterpret_cast<float2*>(dst + (int64_t)col * KD + sk0 + j * 8 + 2 * tq) = make_float2(S[j][2 * h], S[j][2 * h + 1]);
         }
     if (blockIdx.x == 0) {
-        for (int i = threadIdx.x; i < KD; i += MC_THREADS) {
-            float x = s_n[i];
-            if (chunks > 0)
-                for (int p = 0; p < P::N_PARTS; ++p) x += s_np[p * KD + i];
-            dst[(int64_t)cm.vdim * KD + i] = x;
-        }
-        if (threadIdx.x == 0) a.running_max[(int64_t)sl.out * cm.heads + head] = run_max;
+        for (int i = threadIdx.x; i < KD; i += MC_THREADS) dst[(int64_t)cm.vdim * KD + i] = s_n[i];  // written by the same thread
     }
 }
 
@@ -661,8 +658,10 @@ void launch_chunk_cols(const MlstmScanArgs& a, cudaStream_t s) {
     const LinearStateArgs& c = a.common;
     auto* kernel = mlstm_chunk_kernel<KD, C>;
     ensure_dynamic_smem(reinterpret_cast<const void*>(kernel), Chunk<KD, C>::BYTES);
+    const bool vec = a.ldh % 8 == 0 && c.dim % 8 == 0 && c.vdim % 8 == 0 && a.q_col % 8 == 0 && a.k_col % 8 == 0 && a.v_col % 8 == 0 &&
+                     (reinterpret_cast<uintptr_t>(a.yh) & 15) == 0;
     const dim3 grid((unsigned)((c.vdim + C - 1) / C), (unsigned)c.heads, (unsigned)c.lanes.lanes);
-    launch_pdl(kernel, grid, dim3(MC_THREADS), Chunk<KD, C>::BYTES, s, a, aligned_heads(a) && a.y.n == 1 ? 1 : 0);
+    launch_pdl(kernel, grid, dim3(MC_THREADS + 32), Chunk<KD, C>::BYTES, s, a, vec ? 1 : 0);
     MK_LAUNCH_CHECK();
 }
 

@@ -113,7 +113,7 @@ __global__ void __launch_bounds__(MR_ROUTER_THREADS) moe_router_kernel(RowImage 
 #pragma unroll
         for (int i = 0; i < 4; ++i) we[i] = w + (int64_t)min(e + i, rows - 1) * ld;
         float sum[4] = {};
-#pragma unroll 2
+#pragma unroll 4
         for (int c = lane * 8; c < ld; c += 256) {  // ld is a multiple of 64
             float a[8], b[4][8];
             load8(row + c, a);
