@@ -56,6 +56,11 @@ __device__ __forceinline__ uint32_t pack_half2_rest(float x, float y, uint32_t r
     return pack_half2(x - r.x, y - r.y);
 }
 
+// cap * tanh(v / cap) as cap - 2 cap / (1 + exp(2 v / cap)): off by a few 1e-7 of the cap, which is what a score's own rounding costs.
+__device__ __forceinline__ float capped(float v, float cap, float two_over_cap) {
+    return cap - __fdividef(2.0f * cap, 1.0f + __expf(fminf(v * two_over_cap, 80.0f)));
+}
+
 // 1 / denominator of a row with running maximum m and sum l of exp(score - m), when the softmax also counts exp(sink).
 __device__ __forceinline__ float sink_scale(float m, float l, float sink) {
     const float top = fmaxf(m, sink), f = __expf(m - top);
@@ -84,6 +89,7 @@ __global__ void __launch_bounds__(WARPS * 32) attn_tc_kernel(AttnTcArgs a) {
     const int gid = lane >> 2, tq = lane & 3;
     const int kvh = blockIdx.y;
     const int g = a.q_heads / a.kv_heads;
+    const float two_over_cap = a.softcap != 0.f ? 2.0f / a.softcap : 0.f;
     pdl_trigger();
     pdl_wait();
 
@@ -209,7 +215,7 @@ __global__ void __launch_bounds__(WARPS * 32) attn_tc_kernel(AttnTcArgs a) {
                 int h = e >> 1;
                 int pos = tile_pos + j * 8 + 2 * tq + (e & 1);
                 float v = s[j][e] * a.scale;
-                if (a.softcap != 0.f) v = tanhf(v / a.softcap) * a.softcap;
+                if (a.softcap != 0.f) v = capped(v, a.softcap, two_over_cap);
                 bool vis = live_r[h] && pos >= k_lo && pos < k_hi && pos <= pos_r[h] && pos >= lo_r[h];
                 v = vis ? v : -INFINITY;
                 s[j][e] = v;
@@ -338,6 +344,7 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(AttnTcArgs a) {
     const int gid = lane >> 2, tq = lane & 3;
     const int kvh = blockIdx.y;
     const int g = a.q_heads / a.kv_heads;
+    const float two_over_cap = a.softcap != 0.f ? 2.0f / a.softcap : 0.f;
     pdl_trigger();
     pdl_wait();
     // one 32-byte record per work item, so that nothing but the block table and the queries is a dependent load
@@ -483,7 +490,7 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(AttnTcArgs a) {
                 int h = e >> 1;
                 int pos = tile_pos + j * 8 + 2 * tq + (e & 1);
                 float v = sc[j][e] * a.scale;
-                if (a.softcap != 0.f) v = tanhf(v / a.softcap) * a.softcap;
+                if (a.softcap != 0.f) v = capped(v, a.softcap, two_over_cap);
                 bool vis = full_tile || (live_r[h] && pos >= k_lo && pos < k_hi);  // k_lo / k_hi carry causality and the window
                 v = vis ? v : -INFINITY;
                 sc[j][e] = v;
