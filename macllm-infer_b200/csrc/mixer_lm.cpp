@@ -896,6 +896,10 @@ void MixerLm::run_forward(const std::vector<LmLane>& lanes, KvReservation& r, ui
             ++launches_;
         }
     cur_ = 0;
+    if (moe_.counts > 0) {  // whatever a forward that failed half-way left of its counts
+        MK_CUDA(cudaMemsetAsync(moe_.count, 0, (size_t)moe_.counts * 2 * 4, stream_));
+        moe_half_ = 0;
+    }
     QWeight table;
     table.type = f32_ ? QT_F32 : QT_BF16;
     table.rows = ms_.vocab;

@@ -107,8 +107,8 @@ def expert_layers(s) -> list:
     attn = {"heads": s.heads, "kv_heads": s.kv_heads, "dim": s.dim, "vdim": s.dim, "scale": s.dim ** -0.5, "mask": {"size": s.chunk}}
     sink = {"type": "attention", "mlp": mlp, "mixer": {**attn, "rot": {"base": 10000.0, "dims": s.dim}}}
     capped = {"type": "attention_2", "mlp": mlp, "mixer": {**attn, "softcap": 30.0, "rot": {
-        "base": 500000.0, "dims": s.dim, "scaling": {"factor": 8.0, "original": 8192, "fast": 32.0, "slow": 1.0}}}}
-    mem = {"type": "mlstm", "mlp": mlp, "mixer": {"heads": s.mem_heads, "dim": s.mem_dim, "vdim": s.mem_vdim, "gate_cap": 15.0}}
+        "base": 500000.0, "dims": s.dim, "scaling": {"factor": 16.0, "original": 4096, "fast": 24.0, "slow": 1.5}}}}
+    mem = {"type": "mlstm", "mlp": mlp, "mixer": {"heads": s.mem_heads, "dim": s.mem_dim, "vdim": s.mem_vdim, "gate_cap": 12.0}}
     return [capped, mem, mem, sink] * s.groups
 
 
