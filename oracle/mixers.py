@@ -1,4 +1,4 @@
-"""Plain NumPy statement of the mixer-built decoders (the Sizilorn, Kunonex and Tevanex designs and their parts), test infrastructure only.
+"""Plain NumPy statement of the mixer-built decoders (the Sizilorn, Kunonex, Tevanex and Mamivik designs and their parts), test infrastructure only.
 
 One function per mechanism, whole sequences at once, float64 unless the caller passes other arrays; recurrences are written
 token by token.  Nothing here is shared with the CUDA path.  Shapes: x, h [T, width]; a head-wise array [T, heads, dim].
@@ -207,6 +207,54 @@ def latent_attention(h, W, cfg, eps):
     return o.reshape(T, H * cfg["vdim"]) @ W["o"].T
 
 
+def windowed_attention(q, k, v, scale, window, sink=None):
+    """q [T, H, d], k [T, G, d], v [T, G, e]; a position sees itself and the window - 1 keys before it.  sink [H]: one more term
+    exp(sink) in every denominator."""
+    T, H, _ = q.shape
+    group = H // k.shape[1]
+    out = np.empty((T, H, v.shape[2]), q.dtype)
+    for h in range(H):
+        for t in range(T):
+            lo = max(0, t - window + 1)
+            s = k[lo:t + 1, h // group] @ q[t, h] * scale
+            top = s.max() if sink is None else max(s.max(), sink[h])
+            p = np.exp(s - top)
+            den = p.sum() + (0.0 if sink is None else np.exp(sink[h] - top))
+            out[t, h] = p @ v[lo:t + 1, h // group] / den
+    return out
+
+
+def shared_kv_attention(h, W, cfg):
+    """Windowed grouped-query attention whose values are the keys before their rotation; biases on queries and keys."""
+    T, rot = h.shape[0], cfg["rot"]
+    q = (h @ W["q"].T + W["q.b"]).reshape(T, cfg["heads"], cfg["dim"])
+    k = (h @ W["k"].T + W["k.b"]).reshape(T, cfg["kv_heads"], cfg["dim"])
+    f = rope_frequencies(rot["dims"], rot["base"])
+
+    def turn(x):
+        return rotate_half(x, np.arange(T), rot["dims"], f)
+
+    o = windowed_attention(turn(q), turn(k), k, cfg["scale"], cfg["mask"]["size"])
+    return o.reshape(T, -1) @ W["o"].T
+
+
+def rotated_latent_attention(h, W, cfg, eps):
+    """Windowed latent attention with a second, rotated key part that all heads share, a sink per head and a gate per value."""
+    T, H, d, r, rank = h.shape[0], cfg["heads"], cfg["dim"], cfg["rot_dim"], cfg["kv_rank"]
+    q = ((rms(h @ W["dq"].T, eps) * W["dq.norm"]) @ W["uq"].T).reshape(T, H, d + r)
+    down = h @ W["dkv"].T
+    c, turned = rms(down[:, :rank], eps) * W["dkv.norm"], down[:, None, rank:]
+    f, m = yarn_frequencies(r, cfg["rot"]["base"], **cfg["rot"]["scaling"]) if cfg["rot"].get("scaling") else (rope_frequencies(r, cfg["rot"]["base"]), 1.0)
+
+    def turn(x):
+        return m * rotate_half(x, np.arange(T), r, f)
+
+    k = np.concatenate([(c @ W["uk"].T).reshape(T, H, d), np.repeat(turn(turned), H, axis=1)], axis=2)
+    q = np.concatenate([q[..., :d], turn(q[..., d:])], axis=2)
+    o = windowed_attention(q, k, (c @ W["uv"].T).reshape(T, H, cfg["vdim"]), cfg["scale"], cfg["mask"]["size"], W["sink"])
+    return (o.reshape(T, -1) * sigmoid(h @ W["g"].T)) @ W["o"].T
+
+
 # ------------------------------------------------------------------------------------------------ gated delta rule
 
 def causal_conv(x, taps):
@@ -259,6 +307,43 @@ def parallel_mixer(h, W, cfg, eps):
     left = gated_attention(h, sub("left."), cfg["left"], eps)
     right = gated_delta(h, sub("right."), cfg["right"], eps)
     return 0.5 * (rms(left, eps) * W["left.out"] + rms(right, eps) * W["right.out"])
+
+
+# ------------------------------------------------------------------------------------------------ delta rule with channel gates
+
+def bounded_decay(h, w1, w2, w0):
+    """A decay per channel between exp(-exp(-1/2)) and 1."""
+    return np.exp(-np.exp(-0.5) * sigmoid(np.tanh(h @ w1.T) @ w2.T + w0))
+
+
+def channel_delta_rule(r, k, v, w, a, state=None):
+    """r, k, v, w, a [T, H, d]: decay w and removal rate a per key channel; the removal reads along the unit key, the write takes
+    the key as it is, and both see the old state.  Returns (o [T, H, d], state)."""
+    T, H, d = k.shape
+    S = np.zeros((H, d, v.shape[2]), k.dtype) if state is None else state.copy()
+    o = np.empty_like(v)
+    for t in range(T):
+        u = unit(k[t])
+        seen = np.einsum("hkv,hk->hv", S, u)
+        S = w[t][:, :, None] * S - (a[t] * u)[:, :, None] * seen[:, None, :] + k[t][:, :, None] * v[t][:, None, :]
+        o[t] = np.einsum("hkv,hk->hv", S, r[t])
+    return o, S
+
+
+def channel_delta_mixer(h, W, cfg, eps):
+    T = h.shape[0]
+    H, d = cfg["heads"], cfg["dim"]
+    r, k, v = ((h @ W[s].T).reshape(T, H, d) for s in "rkv")
+    w = bounded_decay(h, W["w1"], W["w2"], W["w0"]).reshape(T, H, d)
+    a = sigmoid(h @ W["a"].T + W["a.b"]).reshape(T, H, d)
+    o, _ = channel_delta_rule(r, k, v, w, a)
+    return (rms(o, eps).reshape(T, H * d) * W["norm"] * sigmoid(h @ W["g"].T)) @ W["o"].T
+
+
+def scaled_parallel_mixer(h, W, cfg, eps):
+    """Two branches over one input, each times its own constant."""
+    sub = lambda p: {k[len(p):]: v for k, v in W.items() if k.startswith(p)}
+    return cfg["left_scale"] * shared_kv_attention(h, sub("left."), cfg["left"]) + cfg["right_scale"] * channel_delta_mixer(h, sub("right."), cfg["right"], eps)
 
 
 # ------------------------------------------------------------------------------------------------ WKV time mixing
@@ -359,6 +444,10 @@ def poly_mlp(h, W, eps):
 
 def gated_mlp(h, W):
     return (silu(h @ W["gate"].T) * (h @ W["up"].T)) @ W["down"].T
+
+
+def gelu_mlp(h, W):
+    return (gelu_tanh(h @ W["gate"].T) * (h @ W["up"].T)) @ W["down"].T
 
 
 def clamped_mlp(h, W, limit):
@@ -507,8 +596,32 @@ class TevanexDecoder(MixerDecoder):
         return cap * np.tanh(super().logits(tokens) * self.cfg["logit_scale"] / cap)
 
 
+class MamivikDecoder(MixerDecoder):
+    """RMS norms with one number each; a short convolution in front of every mixer; windowed attention beside a delta rule with a
+    decay and a removal rate per channel, and windowed latent attention with a rotated part."""
+
+    def _norm(self, name, x):
+        return rms(x, self.cfg["norm"]["eps"]) * self.w[name]
+
+    def residuals(self, tokens):
+        """The residual stream after every layer: [layers, T, width]."""
+        eps = self.cfg["norm"]["eps"]
+        x = self.embedding_output(np.asarray(tokens))
+        out = []
+        for i, layer in enumerate(self.cfg["layers"]):
+            p = f"l{i}."
+            h = self._norm(p + "norm1", x)
+            h = h + causal_conv(h, self.w[p + "canon1"])
+            mixer = {"parallel": scaled_parallel_mixer, "latent_attention": rotated_latent_attention}[layer["type"]]
+            x = x + mixer(h, self._sub(p + "mix."), layer["mixer"], eps)
+            if layer.get("mlp"):
+                x = x + gelu_mlp(self._norm(p + "norm2", x), self._sub(p + "mlp."))
+            out.append(x)
+        return np.stack(out)
+
+
 def decoder(config, tensors, dtype=np.float64):
-    return {"Sizilorn": MixerDecoder, "Kunonex": KunonexDecoder, "Tevanex": TevanexDecoder}[config["architecture"]](config, tensors, dtype)
+    return {"Sizilorn": MixerDecoder, "Kunonex": KunonexDecoder, "Tevanex": TevanexDecoder, "Mamivik": MamivikDecoder}[config["architecture"]](config, tensors, dtype)
 
 
 def read_safetensors(path):
