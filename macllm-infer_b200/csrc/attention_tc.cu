@@ -73,17 +73,19 @@ __device__ __forceinline__ float sink_scale(float m, float l, float sink) {
 // SPLIT = true : work item = entries[blockIdx.x] = (lane, split, n_splits) of a one-token lane; the CTA walks
 //                its share of the keys and writes an unnormalised partial.
 // EXACT: the attention weights are split into two f16 operands, so that they reach the product with V in (nearly) f32.
-template <int D, int WARPS, int KT, bool SPLIT, bool EXACT>
+// DV: width of the values that count (rows of K, V and the output are D apart).
+template <int D, int DV, int WARPS, int KT, bool SPLIT, bool EXACT>
 __global__ void __launch_bounds__(WARPS * 32) attn_tc_kernel(AttnTcArgs a) {
     constexpr int DP = D + 8;              // padded row (halves): conflict-free ldmatrix
+    constexpr int VP = DV + 8;
     constexpr int M = 16 * WARPS;
     constexpr int NT_S = KT / 8;           // score n-tiles per warp
-    constexpr int NT_O = D / 8;            // output n-tiles per warp
-    constexpr int CHUNKS = D / 8;          // 16-byte chunks per K or V row
+    constexpr int NT_O = DV / 8;           // output n-tiles per warp
+    constexpr int CHUNKS = D / 8;          // 16-byte chunks per K row
     extern __shared__ __align__(16) unsigned char smem_raw[];
     __half* Qs = reinterpret_cast<__half*>(smem_raw);          // [M][DP]
     __half* Ks = Qs + M * DP;                                   // [2][KT][DP]
-    __half* Vs = Ks + 2 * KT * DP;                              // [2][KT][DP]
+    __half* Vs = Ks + 2 * KT * DP;                              // [2][KT][VP]
 
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int gid = lane >> 2, tq = lane & 3;
@@ -119,6 +121,17 @@ __global__ void __launch_bounds__(WARPS * 32) attn_tc_kernel(AttnTcArgs a) {
         if (hq < g && r < n_rows) {
             const float* src = a.q + (int64_t)(q_off + row0 + r) * ldq + (kvh * g + hq) * D + c;
             float4 x0 = *reinterpret_cast<const float4*>(src), x1 = *reinterpret_cast<const float4*>(src + 4);
+            if (!SPLIT && c >= a.rot_from && c < a.rot_from + a.rot_dims) {
+                const int64_t pair0 = (int64_t)(hdr.start_pos + row0 + r) * (a.rot_dims / 2) + (c - a.rot_from) / 2;
+                float* p[4][2] = {{&x0.x, &x0.y}, {&x0.z, &x0.w}, {&x1.x, &x1.y}, {&x1.z, &x1.w}};
+#pragma unroll
+                for (int i = 0; i < 4; ++i) {
+                    if (c - a.rot_from + 2 * i >= a.rot_dims) break;
+                    const float cs = a.cos_t[pair0 + i], sn = a.sin_t[pair0 + i], u = *p[i][0], v = *p[i][1];
+                    *p[i][0] = u * cs - v * sn;
+                    *p[i][1] = v * cs + u * sn;
+                }
+            }
             h[0] = __floats2half2_rn(x0.x, x0.y);
             h[1] = __floats2half2_rn(x0.z, x0.w);
             h[2] = __floats2half2_rn(x1.x, x1.y);
@@ -146,7 +159,7 @@ __global__ void __launch_bounds__(WARPS * 32) attn_tc_kernel(AttnTcArgs a) {
     const __half* vp = reinterpret_cast<const __half*>(a.v_pool);
     auto load_tile = [&](int t, int stage) {
         __half* kd = Ks + stage * KT * DP;
-        __half* vd = Vs + stage * KT * DP;
+        __half* vd = Vs + stage * KT * VP;
         for (int i = tid; i < KT * CHUNKS; i += WARPS * 32) {
             int key = i / CHUNKS, c = (i - key * CHUNKS) * 8;
             int pos = k_begin + t * KT + key;
@@ -158,7 +171,7 @@ __global__ void __launch_bounds__(WARPS * 32) attn_tc_kernel(AttnTcArgs a) {
                         (pos & (a.block_tokens - 1))) * (int64_t)D + c;
             }
             cp_async16(kd + key * DP + c, kp + base, valid);
-            cp_async16(vd + key * DP + c, vp + base, valid);
+            if (DV == D || c < DV) cp_async16(vd + key * VP + c, vp + base, valid);
         }
     };
 
@@ -187,7 +200,7 @@ __global__ void __launch_bounds__(WARPS * 32) attn_tc_kernel(AttnTcArgs a) {
         cp_async_wait<1>();
         __syncthreads();
         const __half* kt = Ks + (t & 1) * KT * DP;
-        const __half* vt = Vs + (t & 1) * KT * DP;
+        const __half* vt = Vs + (t & 1) * KT * VP;
 
         // S = Q K^T
         float s[NT_S][4];
@@ -268,7 +281,7 @@ __global__ void __launch_bounds__(WARPS * 32) attn_tc_kernel(AttnTcArgs a) {
 #pragma unroll
             for (int j = 0; j < NT_O; j += 2) {
                 uint32_t bf[4];
-                ldmatrix_x4_trans(bf, vt + (kk * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * DP + j * 8 + (lane >> 4) * 8);
+                ldmatrix_x4_trans(bf, vt + (kk * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * VP + j * 8 + (lane >> 4) * 8);
                 mma16816(o_acc[j], pf, bf[0], bf[1]);
                 mma16816(o_acc[j + 1], pf, bf[2], bf[3]);
                 if constexpr (EXACT) {
@@ -704,20 +717,20 @@ __global__ void attn_combine_kernel(AttnTcArgs a, int D) {
     }
 }
 
-template <int D, int WARPS, int KT, bool SPLIT, bool EXACT>
+template <int D, int DV, int WARPS, int KT, bool SPLIT, bool EXACT>
 void launch_variant(const AttnTcArgs& a, int n_work, cudaStream_t s) {
-    constexpr size_t smem = (size_t)(16 * WARPS + 4 * KT) * (D + 8) * sizeof(__half);
-    ensure_dynamic_smem(reinterpret_cast<const void*>(&attn_tc_kernel<D, WARPS, KT, SPLIT, EXACT>), smem);
+    constexpr size_t smem = ((size_t)(16 * WARPS + 2 * KT) * (D + 8) + (size_t)2 * KT * (DV + 8)) * sizeof(__half);
+    ensure_dynamic_smem(reinterpret_cast<const void*>(&attn_tc_kernel<D, DV, WARPS, KT, SPLIT, EXACT>), smem);
     dim3 grid((unsigned)n_work, (unsigned)a.kv_heads);
-    launch_pdl(attn_tc_kernel<D, WARPS, KT, SPLIT, EXACT>, grid, dim3(WARPS * 32), smem, s, a);
+    launch_pdl(attn_tc_kernel<D, DV, WARPS, KT, SPLIT, EXACT>, grid, dim3(WARPS * 32), smem, s, a);
     MK_LAUNCH_CHECK();
 }
 
 template <int D, bool EXACT>
 void launch_for_dim(const AttnTcArgs& a, int warps, cudaStream_t s) {
     if (a.n_tiles > 0) {
-        if (warps == 8) launch_variant<D, 8, 64, false, EXACT>(a, a.n_tiles, s);
-        else launch_variant<D, 4, 32, false, EXACT>(a, a.n_tiles, s);  // 32-key tiles: half the shared memory, twice the CTAs per SM (measured +0.4 % on the whole benchmark)
+        if (warps == 8) launch_variant<D, D, 8, 64, false, EXACT>(a, a.n_tiles, s);
+        else launch_variant<D, D, 4, 32, false, EXACT>(a, a.n_tiles, s);  // 32-key tiles: half the shared memory, twice the CTAs per SM (measured +0.4 % on the whole benchmark)
     }
     if (a.n_entries > 0) {
         constexpr int STAGES = D >= 256 ? 2 : 3;
@@ -749,13 +762,21 @@ bool attention_tc_supported(int q_heads, int kv_heads, int head_dim, int block_t
 // eight warps measured slower (fewer, longer CTAs) than four.
 int attention_tc_warps(int q_heads, int kv_heads) { return q_heads / kv_heads == 8 ? 8 : 4; }
 
+int attention_tc_prefill_width(int q_heads, int kv_heads, int dim, int vdim, int block_tokens) {
+    if (!attention_tc_supported(q_heads, kv_heads, 64, block_tokens, true)) return 0;
+    const int need = std::max(dim, vdim);
+    for (int d : {64, 128, 192, 256})
+        if (need <= d && (d != 192 || (vdim <= 128 && attention_tc_warps(q_heads, kv_heads) == 4))) return d;
+    return 0;
+}
+
 int attention_tc_tile_rows(int q_heads, int kv_heads) { return 16 * attention_tc_warps(q_heads, kv_heads) / (q_heads / kv_heads); }
 
 int attention_tc_max_entries(int lanes, int kv_heads) { return std::max(lanes + lanes / 2, kAttnTargetCtas / std::max(1, kv_heads)) + 1; }
 
 void plan_attention_tc(const int32_t* start_pos, const int32_t* n_tokens, const int32_t* n_blocks, int lanes, int q_heads,
-                       int kv_heads, AttnTcPlan& plan, int chunk) {
-    auto visible = [&](int i) { return start_pos[i] + 1 - attention_first_key(start_pos[i], 0, chunk); };  // keys of a one-token lane
+                       int kv_heads, AttnTcPlan& plan, int chunk, int window) {
+    auto visible = [&](int i) { return start_pos[i] + 1 - attention_first_key(start_pos[i], window, chunk); };  // keys of a one-token lane
     plan.tiles.clear();
     plan.entries.clear();
     plan.dec_lanes.clear();
@@ -802,8 +823,12 @@ void plan_attention_tc(const int32_t* start_pos, const int32_t* n_tokens, const 
 
 int launch_paged_attention_tc(const AttnTcArgs& a_in, cudaStream_t s) {
     AttnTcArgs a = a_in;
-    if (!attention_tc_supported(a.q_heads, a.kv_heads, a.d, a.block_tokens, true))
+    const bool prefill_192 = a.d == 192 && a.n_entries == 0 && a.n_dec_lanes == 0 && a.dv > 0 && a.dv <= 128 && a.exact_weights &&
+                             attention_tc_prefill_width(a.q_heads, a.kv_heads, 192, a.dv, a.block_tokens) == 192;
+    if (!prefill_192 && !attention_tc_supported(a.q_heads, a.kv_heads, a.d, a.block_tokens, true))
         throw std::runtime_error("launch_paged_attention_tc: unsupported shape");
+    if (a.rot_dims > 0 && (a.n_entries > 0 || a.rot_from % 8 != 0 || a.cos_t == nullptr || a.sin_t == nullptr))
+        throw std::runtime_error("launch_paged_attention_tc: queries turn on their way into prefill tiles only");
     if (a.out == nullptr && a.out_h == nullptr && a.qout.qs == nullptr) throw std::runtime_error("launch_paged_attention_tc: no output");
     if (a.sink != nullptr && a.n_dec_lanes > 0) throw std::runtime_error("launch_paged_attention_tc: the separate merge pass knows no sink");
     if (a.out == nullptr && a.n_dec_lanes > 0) throw std::runtime_error("launch_paged_attention_tc: the separate merge pass writes f32 rows");
@@ -813,6 +838,9 @@ int launch_paged_attention_tc(const AttnTcArgs& a_in, cudaStream_t s) {
     switch (a.d) {
         case 64: a.exact_weights ? launch_for_dim<64, true>(a, warps, s) : launch_for_dim<64, false>(a, warps, s); break;
         case 128: a.exact_weights ? launch_for_dim<128, true>(a, warps, s) : launch_for_dim<128, false>(a, warps, s); break;
+        case 192:
+            if (a.n_tiles > 0) launch_variant<192, 128, 4, 32, false, true>(a, a.n_tiles, s);
+            break;
         case 256: a.exact_weights ? launch_for_dim<256, true>(a, warps, s) : launch_for_dim<256, false>(a, warps, s); break;
         default: throw std::runtime_error("launch_paged_attention_tc: unsupported head_dim");
     }

@@ -40,15 +40,23 @@ struct AttnTcArgs {
     int64_t pool_blocks = 0;  // see kv_page_index
     int bt_shift = 0;         // log2(block_tokens), filled in by the launcher
     float scale = 1.f, softcap = 0.f;
-    int window = 0;
+    int window = 0;             // > 0: a position sees itself and the window - 1 keys before it
     int chunk = 0;              // > 0: a position sees the keys of its own chunk only (chunks counted from position 0)
     const float* sink = nullptr;  // [q_heads]: one more term exp(sink) in the denominator; null: none
     // attention weights enter the product with V as the sum of two f16 numbers (about 22 bits) instead of one
     int exact_weights = 0;
+    // prefill tiles only: width of a value head inside its row of d values (0: d), and dimensions rot_from .. rot_from + rot_dims - 1
+    // of the queries, which turn in adjacent pairs while the queries are read (tables [positions][rot_dims / 2])
+    int dv = 0;
+    int rot_from = 0, rot_dims = 0;   // rot_from: a multiple of 8
+    const float *cos_t = nullptr, *sin_t = nullptr;
 };
 
 // f16 pools, head_dim 64/128/256, 1/2/4/8 query heads per KV head, block_tokens a power of two >= 16.
 bool attention_tc_supported(int q_heads, int kv_heads, int head_dim, int block_tokens, bool kv_f16);
+// The head width (row of the pools) with which lanes of several tokens can run heads of `dim` query / key and `vdim` value
+// dimensions; besides the widths above 192 with values of up to 128.  0: none.
+int attention_tc_prefill_width(int q_heads, int kv_heads, int dim, int vdim, int block_tokens);
 // Query rows of one prefill tile (the CTA covers rows x group heads = 16 * warps items).
 int attention_tc_tile_rows(int q_heads, int kv_heads);
 int attention_tc_warps(int q_heads, int kv_heads);
@@ -68,9 +76,9 @@ struct AttnTcPlan {
     int n_dec_lanes() const { return (int)dec_lanes.size() / 3; }
 };
 // n_blocks[i] = entries of lane i's block table (tables are concatenated in lane order, tokens packed in lane order).
-// chunk: see AttnTcArgs.
+// chunk, window: see AttnTcArgs.
 void plan_attention_tc(const int32_t* start_pos, const int32_t* n_tokens, const int32_t* n_blocks, int lanes, int q_heads,
-                       int kv_heads, AttnTcPlan& plan, int chunk = 0);
+                       int kv_heads, AttnTcPlan& plan, int chunk = 0, int window = 0);
 // Upper bound of plan.n_entries() for a tick of at most `lanes` lanes.
 int attention_tc_max_entries(int lanes, int kv_heads);
 

@@ -110,7 +110,8 @@ int32_t mk_mixer_inspect(const char* dir, mk_mixer_summary* out) {
         for (const MixerLayerSpec& l : s.layers) {
             switch (l.kind) {
                 case MixerKind::Wkv: ++out->wkv_layers; break;
-                case MixerKind::Parallel: ++out->parallel_layers; break;
+                case MixerKind::Parallel:
+                case MixerKind::ScaledParallel: ++out->parallel_layers; break;
                 case MixerKind::Latent: ++out->latent_layers; break;
                 case MixerKind::MinGru: ++out->mingru_layers; break;
                 case MixerKind::Mlstm: ++out->mlstm_layers; break;

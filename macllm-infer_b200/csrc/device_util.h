@@ -79,7 +79,19 @@ struct MatmulScatter {
     float* rest = nullptr;
     int rest_from = 0;
     int64_t ld_rest = 0;
+    // value (t, p, i) is multiplied by sigmoid(sum over s < gate_n of gate[s * gate_stride + t' * gate_ld + p * part_valid + i])
+    const float* gate = nullptr;
+    int gate_n = 1, gate_ld = 0;
+    int64_t gate_stride = 0;
 #ifdef __CUDACC__
+    __device__ __forceinline__ float gate_sum(int t, int64_t n) const {
+        if (row_map != nullptr) t = row_map[t];
+        const int64_t p = n / part_rows, i = n - p * part_rows;
+        const float* g = gate + (int64_t)t * gate_ld + p * part_valid + i;
+        float z = *g;
+        for (int s = 1; s < gate_n; ++s) z += g[s * gate_stride];
+        return z;
+    }
     // Offset of weight row n's values, or -1 when they are not kept.
     __device__ __forceinline__ int64_t column(int64_t n) const {
         const int64_t p = n / part_rows, i = n - p * part_rows;

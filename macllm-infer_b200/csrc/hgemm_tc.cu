@@ -249,6 +249,7 @@ __device__ __forceinline__ float finish_value(float v, const HgParams& p) {
 }
 
 // The activations of the gated feed-forward, as the SwiGLU kernel of quantize.cu computes them.
+__device__ __forceinline__ float hg_sigmoid(float x) { return __fdividef(1.0f, 1.0f + __expf(-x)); }  // to what a 16-bit result needs
 __device__ __forceinline__ float hg_silu(float x) { return x / (1.0f + expf(-x)); }
 __device__ __forceinline__ float hg_clamped(float g, float u, float limit) {  // clamped_gate_f to what the 16-bit result needs
     g = fminf(g, limit);
@@ -474,7 +475,7 @@ hgemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant_
         const int quad = warp & 3, odd_group = (warp - 2) >> 2;
         const int etid = (int)threadIdx.x - 64;  // among the epilogue threads
         const bool plain = p.out_scale == 1.0f && p.softcap == 0.f;
-        if (p.part[0].act_post != nullptr) pdl_wait();   // the factors of the rows come from a predecessor
+        if (p.part[0].act_post != nullptr || (p.scattered != 0 && p.scatter.gate != nullptr)) pdl_wait();   // the factors of the rows come from a predecessor
         uint32_t tile_it = 0;
         for (int item = blockIdx.x; item < total_items; item += gridDim.x, ++tile_it) {
             HgTile tile;
@@ -516,6 +517,16 @@ hgemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant_
                 uint32_t r[32];
                 tmem_ld32(tmem_base + ((uint32_t)(quad * 32) << 16) + acc * BN + (uint32_t)cb, r);
                 asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
+                if (p.scattered != 0 && p.scatter.gate != nullptr && row < tile.rows && p.scatter.column(row) >= 0) {
+                    float z[8];
+#pragma unroll
+                    for (int i0 = 0; i0 < 32; i0 += 8) {
+#pragma unroll
+                        for (int i = 0; i < 8; ++i) z[i] = tok0 + cb + i0 + i < tile.tok_end ? p.scatter.gate_sum(tok0 + cb + i0 + i, row) : 0.f;
+#pragma unroll
+                        for (int i = 0; i < 8; ++i) r[i0 + i] = __float_as_uint(__uint_as_float(r[i0 + i]) * hg_sigmoid(z[i]));
+                    }
+                }
                 if (p.gated != 0) {
                     // lanes 2i / 2i+1 hold gate / up of one feature: the even lane finishes the even token columns,
                     // the odd lane the odd ones, after one exchange per pair of columns

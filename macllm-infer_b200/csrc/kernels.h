@@ -94,7 +94,7 @@ struct RopeKvArgs {
     int ldq_out = 0;
     const float* q_norm_w = nullptr;  // [d] or null
     const float* k_norm_w = nullptr;  // [d] or null
-    // launch_rope_kv_rows: biases, and norm weights over all heads at once ([q_heads * d], [kv_heads * d])
+    // biases (optional); launch_rope_kv_rows takes norm weights over all heads at once ([q_heads * d], [kv_heads * d])
     const float *q_bias = nullptr, *k_bias = nullptr, *v_bias = nullptr;
     float norm_eps = 1e-6f;
     const float* cos_t = nullptr;  // [capacity][rotary_dim/2], null on NoPE layers

@@ -12,6 +12,7 @@
 // more than kSlack, so the accumulators in tensor memory are hardly ever rescaled.  When few rows are in flight their keys are
 // shared out over several CTAs; the one that finishes last adds the shares in order.  Every wait is bounded (see hgemm_tc.cu).
 #include "latent_attention.h"
+#include "kernels.h"
 #include "device_util.h"
 #include <algorithm>
 
@@ -155,24 +156,36 @@ __device__ __forceinline__ LatentEntry load_entry(const int32_t* entries, int i)
     return LatentEntry{a.x, a.y, a.z, a.w, b.x, b.y, b.z};
 }
 
-// MB chunks of 128 columns, NH heads (16 or 32).
-template <int MB, int NH>
+// What the softmax's denominator, exp(m) l without it, is with one more term exp(sink): exp(m) times the result.
+__device__ __forceinline__ float la_with_sink(const float* sink, int head, float m, float l) {
+    return sink == nullptr ? l : l + __expf(fminf(sink[head] - m, 80.f));
+}
+// Two neighbouring query columns at `turn` of the rotation tables.
+__device__ __forceinline__ float2 la_turn(float2 v, const LatentAttnArgs& a, int64_t turn) {
+    const float cs = a.cos_t[turn], sn = a.sin_t[turn];
+    return make_float2(v.x * cs - v.y * sn, v.y * cs + v.x * sn);
+}
+
+// MB chunks of 128 value columns, then XB blocks of 64 columns that count in the scores only; NH heads (16 or 32).
+template <int MB, int NH, int XB>
 struct Lu {
-    static constexpr int RANK = MB * LU_COLS;
-    static constexpr int STAGES = MB >= 4 && NH == 16 ? 6 : (MB >= 3 ? 5 : (MB == 2 ? 4 : 2));  // chunks in the ring
+    static constexpr int VALUES = MB * LU_COLS, RANK = VALUES + XB * 64;
+    static constexpr int CHUNKS = MB + (XB > 0 ? 1 : 0);   // of a tile; the last one may be half as wide
+    static constexpr int BASE = MB >= 4 && NH == 16 ? 6 : (MB >= 3 ? 5 : (MB == 2 ? 4 : 2));
+    static constexpr int STAGES = XB > 0 && MB == 1 ? 4 : BASE;                                 // chunks in the ring
     static constexpr int Q_BYTES = NH * RANK * 2;                                               // [column block][head][64]
     static constexpr int P_BYTES = 2 * NH * LU_KEYS * 2;                                        // [key block][weights | rests][64]
     static constexpr size_t BYTES = (size_t)STAGES * LU_CHUNK + Q_BYTES + P_BYTES + 1024 + 256;
     static constexpr int S_COL = MB * 2 * NH;  // tensor memory: outputs (high | rest) of every chunk, then two tiles' scores
     static constexpr int END_COL = S_COL + 2 * NH;
     static constexpr uint32_t TMEM = END_COL <= 64 ? 64 : END_COL <= 128 ? 128 : (END_COL <= 256 ? 256 : 512);
-    static_assert(END_COL <= 512, "tensor memory");
+    static_assert(END_COL <= 512 && STAGES >= CHUNKS, "tensor memory; a tile fits in the ring");
 };
 
-template <int MB, int NH>
+template <int MB, int NH, int XB>
 __global__ void __launch_bounds__(LU_THREADS, 1) latent_umma_kernel(LatentAttnArgs a, int bt_shift) {
-    using L = Lu<MB, NH>;
-    constexpr int RANK = L::RANK, STAGES = L::STAGES, HG = NH / LU_GROUPS, LOADER = LU_SOFTMAX / 32;
+    using L = Lu<MB, NH, XB>;
+    constexpr int RANK = L::RANK, VALUES = L::VALUES, CHUNKS = L::CHUNKS, STAGES = L::STAGES, HG = NH / LU_GROUPS, LOADER = LU_SOFTMAX / 32;
     extern __shared__ uint8_t lu_raw[];
     uint8_t* ring = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(lu_raw) + 1023) & ~(uintptr_t)1023);
     uint8_t* qs = ring + (size_t)STAGES * LU_CHUNK;
@@ -212,9 +225,9 @@ __global__ void __launch_bounds__(LU_THREADS, 1) latent_umma_kernel(LatentAttnAr
     pdl_trigger();
     // work list and block tables were staged by the host: they need not wait for the predecessor
     const LatentEntry e = load_entry(a.entries, blockIdx.x);
-    const int len = e.pos + 1;
+    const int first_key = attention_first_key(e.pos, a.window, 0), len = e.pos + 1 - first_key;
     const int chunk = ((len + e.n_shares - 1) / e.n_shares + LU_KEYS - 1) / LU_KEYS * LU_KEYS;
-    const int k_lo = e.share * chunk, k_hi = min(len, k_lo + chunk);
+    const int k_lo = first_key + e.share * chunk, k_hi = min(e.pos + 1, k_lo + chunk);
     const int tiles = k_hi > k_lo ? (k_hi - k_lo + LU_KEYS - 1) / LU_KEYS : 0;
     auto row_of = [&](int t, int key) {  // pool row of a tile's key, -1 past the last one
         const int pos = k_lo + t * LU_KEYS + key;
@@ -235,10 +248,14 @@ __global__ void __launch_bounds__(LU_THREADS, 1) latent_umma_kernel(LatentAttnAr
             ok = lu_agree(LU_GROUPS + 2, LU_LOADERS, ok);  // this tile's rows are there, nobody reads the other buffer any more
             if (!ok) break;
             if (t + 1 < tiles) s_rows[(t + 1) & 1][lt] = row_of(t + 1, lt);
-            for (int c = 0; c < MB; ++c, ++it) {
+            for (int c = 0; c < CHUNKS; ++c, ++it) {
                 const uint32_t st = it % STAGES;
                 ok = lu_bar_wait(&empty[st], ((it / STAGES) & 1) ^ 1);
                 if (!ok) break;
+                if (XB == 1 && c == MB && piece >= 8) {  // half a chunk
+                    lu_copies_arrive(&full[st]);
+                    continue;
+                }
                 const uint32_t dst = dst0 + st * LU_CHUNK;
                 const __half* src = pool + c * LU_COLS;
 #pragma unroll
@@ -259,22 +276,25 @@ __global__ void __launch_bounds__(LU_THREADS, 1) latent_umma_kernel(LatentAttnAr
             const uint32_t q_addr = lu_smem(qs), p_addr = lu_smem(ps), ring_addr = lu_smem(ring);
             bool ok = true;
             auto scores = [&](int t, int c) {  // chunk c of tile t's scores; the chunk is there
-                const uint32_t st = (uint32_t)(t * MB + c) % STAGES;
+                const uint32_t st = (uint32_t)(t * CHUNKS + c) % STAGES;
                 asm volatile("fence.proxy.async.shared::cta;" ::: "memory");  // the copies are ordinary writes
                 lu_fence_after();
                 // descriptors hold addresses in 16-byte units
                 const uint64_t keys = lu_desc(ring_addr + st * LU_CHUNK, 16), queries = lu_desc(q_addr + 2 * c * (NH * 128), 16);
                 const uint32_t d = tmem + L::S_COL + (t & 1) * NH;
 #pragma unroll
-                for (int k = 0; k < LU_COLS / 16; ++k)
+                for (int k = 0; k < LU_COLS / 16; ++k) {
+                    if (XB == 1 && k >= 4 && c == MB) break;
                     lu_mma(d, keys + (k >> 2) * (LU_BLOCK / 16) + (k & 3) * 2, queries + (k >> 2) * (NH * 8) + (k & 3) * 2, i_scores, c > 0 || k > 0);
-                if (c == MB - 1) lu_commit(&s_full[t & 1]);
+                }
+                if (XB > 0 && c == MB) lu_commit(&empty[st]);  // nothing else reads it
+                if (c == CHUNKS - 1) lu_commit(&s_full[t & 1]);
             };
             auto outputs = [&](int t) {  // tile t's part of the outputs; the weights are there
                 lu_fence_after();
                 const uint64_t weights = lu_desc(p_addr, 16);
                 for (int c = 0; c < MB; ++c) {
-                    const uint32_t st = (uint32_t)(t * MB + c) % STAGES;
+                    const uint32_t st = (uint32_t)(t * CHUNKS + c) % STAGES;
                     const uint64_t values = lu_desc(ring_addr + st * LU_CHUNK, LU_BLOCK);
 #pragma unroll
                     for (int k = 0; k < LU_KEYS / 16; ++k)
@@ -283,11 +303,11 @@ __global__ void __launch_bounds__(LU_THREADS, 1) latent_umma_kernel(LatentAttnAr
                 }
                 lu_commit(o_done);
             };
-            auto full_of = [&](int t, int c) { return &full[(uint32_t)(t * MB + c) % STAGES]; };
-            auto full_parity = [&](int t, int c) { return ((uint32_t)(t * MB + c) / STAGES) & 1; };
+            auto full_of = [&](int t, int c) { return &full[(uint32_t)(t * CHUNKS + c) % STAGES]; };
+            auto full_parity = [&](int t, int c) { return ((uint32_t)(t * CHUNKS + c) / STAGES) & 1; };
             ok = lu_bar_wait(q_full, 0);
             lu_fence_after();
-            for (int c = 0; c < MB && ok; ++c) {
+            for (int c = 0; c < CHUNKS && ok; ++c) {
                 ok = lu_bar_wait(full_of(0, c), full_parity(0, c));
                 if (ok) scores(0, c);
             }
@@ -295,14 +315,14 @@ __global__ void __launch_bounds__(LU_THREADS, 1) latent_umma_kernel(LatentAttnAr
             // beside tile t come only after its outputs.
             for (int t = 0; t < tiles && ok; ++t) {
                 bool summed = false;
-                int c = t + 1 < tiles ? 0 : MB;
-                for (uint32_t spins = 0; ok && (!summed || c < MB);) {
+                int c = t + 1 < tiles ? 0 : CHUNKS;
+                for (uint32_t spins = 0; ok && (!summed || c < CHUNKS);) {
                     if (!summed && lu_bar_test(p_full, t & 1)) {
                         outputs(t);
                         summed = true;
                         spins = 0;
                     }
-                    if (c < MB && lu_bar_test(full_of(t + 1, c), full_parity(t + 1, c))) {
+                    if (c < CHUNKS && lu_bar_test(full_of(t + 1, c), full_parity(t + 1, c))) {
                         scores(t + 1, c);
                         ++c;
                         spins = 0;
@@ -321,6 +341,17 @@ __global__ void __launch_bounds__(LU_THREADS, 1) latent_umma_kernel(LatentAttnAr
             const int h = i / (RANK / 8), c = i - h * (RANK / 8);
             uint4 v = make_uint4(0u, 0u, 0u, 0u);
             if (h < heads) v = *reinterpret_cast<const uint4*>(a.q_h + ((int64_t)e.row * a.heads + head0 + h) * RANK + c * 8);
+            const int turned = c * 8 - a.rot0;
+            if (turned >= 0 && turned < a.rot_dims) {
+                uint32_t w[4] = {v.x, v.y, v.z, v.w};
+#pragma unroll
+                for (int i = 0; i < 4; ++i) {
+                    if (turned + 2 * i >= a.rot_dims) break;
+                    const float2 x = la_turn(__half22float2(*reinterpret_cast<const __half2*>(&w[i])), a, (int64_t)e.pos * (a.rot_dims / 2) + turned / 2 + i);
+                    w[i] = la_pack(x.x, x.y);
+                }
+                v = make_uint4(w[0], w[1], w[2], w[3]);
+            }
             *reinterpret_cast<uint4*>(qs + (c >> 3) * (NH * 128) + h * 128 + (((c & 7) ^ (h & 7)) << 4)) = v;
         }
         asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
@@ -419,6 +450,7 @@ __global__ void __launch_bounds__(LU_THREADS, 1) latent_umma_kernel(LatentAttnAr
         if (lane < HG) s_warp[warp][lane] = sum;
         if (!lu_agree(bar, 128, ok) && gt == 0) atomicExch(a.status, 25);
         auto slot = [&](int entry) { return ((int64_t)entry * gridDim.y + blockIdx.y) * NH; };
+        auto gate_of = [&](int h) { return a.gate.p != nullptr ? sigmoid_f(a.gate.at(e.packed, a.gate_col + head0 + h)) : 1.f; };
         auto ml_at = [&](int entry, int h) { return a.part_ml + (slot(entry) + h) * 2; };
         if (gt < HG && h0 + gt < heads) {  // thread gt finishes head h0 + gt
             float total = 0.f, mine = -INFINITY;
@@ -427,7 +459,7 @@ __global__ void __launch_bounds__(LU_THREADS, 1) latent_umma_kernel(LatentAttnAr
 #pragma unroll
             for (int h = 0; h < HG; ++h)
                 if (h == gt) mine = m[h];
-            if (e.n_shares == 1) s_factor[0][h0 + gt] = sigmoid_f(a.gate.at(e.packed, a.gate_col + head0 + h0 + gt)) / total;
+            if (e.n_shares == 1) s_factor[0][h0 + gt] = gate_of(h0 + gt) / la_with_sink(a.sink, head0 + h0 + gt, mine, total);
             else *reinterpret_cast<float2*>(ml_at(blockIdx.x, h0 + gt)) = make_float2(mine, total);
         }
         lu_agree(bar, 128, true);
@@ -444,9 +476,9 @@ __global__ void __launch_bounds__(LU_THREADS, 1) latent_umma_kernel(LatentAttnAr
                 if (h0 + h >= heads) continue;
                 const float v = tiles > 0 ? __uint_as_float(o[h]) + __uint_as_float(rest[h]) : 0.f;
                 if (e.n_shares == 1)
-                    a.out.h[((int64_t)(head0 + h0 + h) * a.n_rows + e.row) * RANK + c * LU_COLS + gt] = __float2bfloat16_rn(v * s_factor[0][h0 + h]);
+                    a.out.h[((int64_t)(head0 + h0 + h) * a.n_rows + e.row) * VALUES + c * LU_COLS + gt] = __float2bfloat16_rn(v * s_factor[0][h0 + h]);
                 else
-                    a.part_o[(slot(blockIdx.x) + h0 + h) * RANK + c * LU_COLS + gt] = v;
+                    a.part_o[(slot(blockIdx.x) + h0 + h) * VALUES + c * LU_COLS + gt] = v;
             }
         }
         if (e.n_shares > 1) {
@@ -469,7 +501,7 @@ __global__ void __launch_bounds__(LU_THREADS, 1) latent_umma_kernel(LatentAttnAr
                         s_factor[sh][tid] = f;
                         total = fmaf(ml.y, f, total);
                     }
-                    const float g = sigmoid_f(a.gate.at(e.packed, a.gate_col + head0 + tid)) / total;
+                    const float g = gate_of(tid) / la_with_sink(a.sink, head0 + tid, mx, total);
                     for (int sh = 0; sh < e.n_shares; ++sh) s_factor[sh][tid] *= g;
                 }
                 lu_agree(LU_GROUPS + 1, LU_SOFTMAX, true);
@@ -478,7 +510,7 @@ __global__ void __launch_bounds__(LU_THREADS, 1) latent_umma_kernel(LatentAttnAr
                     const int h = i / (MB * LU_COLS / 4), c = (i - h * (MB * LU_COLS / 4)) * 4;
                     float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
                     for (int sh = 0; sh < e.n_shares; ++sh) {
-                        const float4 v = __ldcg(reinterpret_cast<const float4*>(a.part_o + (slot(e.first + sh) + h) * RANK + c));
+                        const float4 v = __ldcg(reinterpret_cast<const float4*>(a.part_o + (slot(e.first + sh) + h) * VALUES + c));
                         const float f = s_factor[sh][h];
                         acc = make_float4(fmaf(v.x, f, acc.x), fmaf(v.y, f, acc.y), fmaf(v.z, f, acc.z), fmaf(v.w, f, acc.w));
                     }
@@ -514,7 +546,7 @@ __device__ __forceinline__ float la_widen<__half>(__half v) { return __half2floa
 template <typename KV>
 __global__ void __launch_bounds__(LG_WARPS * 32) latent_general_kernel(LatentAttnArgs a) {
     extern __shared__ __align__(16) float lg_smem[];
-    const int R = a.rank, pitch = R + 4;
+    const int R = a.rank, V = a.values, pitch = R + 4;
     float* qs = lg_smem;                              // [16][R]
     float* ks = qs + LG_WARPS * LG_ITEMS * R;         // [LG_KEYS][pitch]
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -523,7 +555,13 @@ __global__ void __launch_bounds__(LG_WARPS * 32) latent_general_kernel(LatentAtt
     const LatentEntry e = load_entry(a.entries, blockIdx.x);
     const int head0 = blockIdx.y * LG_WARPS * LG_ITEMS, heads = min(LG_WARPS * LG_ITEMS, a.heads - head0);
     const float* q = a.q_f + ((int64_t)e.row * a.heads + head0) * R;
-    for (int i = threadIdx.x; i < heads * R; i += LG_WARPS * 32) qs[i] = q[i];
+    for (int i = threadIdx.x * 2; i < heads * R; i += LG_WARPS * 64) {
+        float2 x = *reinterpret_cast<const float2*>(q + i);
+        const int c = i % R - a.rot0;
+        if (c >= 0 && c < a.rot_dims) x = la_turn(x, a, (int64_t)e.pos * (a.rot_dims / 2) + c / 2);
+        *reinterpret_cast<float2*>(qs + i) = x;
+    }
+    const int first_key = attention_first_key(e.pos, a.window, 0);
     float m_run[LG_ITEMS], l_run[LG_ITEMS], acc[LG_ITEMS][LG_COLS];
 #pragma unroll
     for (int i = 0; i < LG_ITEMS; ++i) {
@@ -533,7 +571,7 @@ __global__ void __launch_bounds__(LG_WARPS * 32) latent_general_kernel(LatentAtt
         for (int j = 0; j < LG_COLS; ++j) acc[i][j] = 0.f;
     }
     const KV* pool = static_cast<const KV*>(a.pool);
-    for (int k0 = 0; k0 <= e.pos; k0 += LG_KEYS) {
+    for (int k0 = first_key; k0 <= e.pos; k0 += LG_KEYS) {
         __syncthreads();
         for (int key = warp; key < LG_KEYS; key += LG_WARPS) {
             const int pos = k0 + key;
@@ -576,7 +614,7 @@ __global__ void __launch_bounds__(LG_WARPS * 32) latent_general_kernel(LatentAtt
                 const float* v = ks + key * pitch + lane;
 #pragma unroll
                 for (int j = 0; j < LG_COLS; ++j)
-                    if (j * 32 < R) acc[i][j] = fmaf(pk, v[j * 32], acc[i][j]);
+                    if (j * 32 < V) acc[i][j] = fmaf(pk, v[j * 32], acc[i][j]);
             }
         }
     }
@@ -584,10 +622,11 @@ __global__ void __launch_bounds__(LG_WARPS * 32) latent_general_kernel(LatentAtt
     for (int i = 0; i < LG_ITEMS; ++i) {
         const int item = warp + LG_WARPS * i;
         if (item >= heads) continue;
-        const float f = sigmoid_f(a.gate.at(e.packed, a.gate_col + head0 + item)) / l_run[i];
+        const float gate = a.gate.p != nullptr ? sigmoid_f(a.gate.at(e.packed, a.gate_col + head0 + item)) : 1.f;
+        const float f = gate / (a.sink != nullptr ? l_run[i] + expf(fminf(a.sink[head0 + item] - m_run[i], 80.f)) : l_run[i]);
 #pragma unroll
         for (int j = 0; j < LG_COLS; ++j)
-            if (j * 32 < R) a.out.put((int64_t)(head0 + item) * a.n_rows + e.row, j * 32 + lane, acc[i][j] * f);
+            if (j * 32 < V) a.out.put((int64_t)(head0 + item) * a.n_rows + e.row, j * 32 + lane, acc[i][j] * f);
     }
 }
 
@@ -627,28 +666,50 @@ __global__ void __launch_bounds__(256) split_rows_kernel(const float* x, int ldx
     }
 }
 
-template <int MB, int NH>
+template <int MB, int NH, int XB>
 void launch_umma(const LatentAttnArgs& a, cudaStream_t s) {
-    constexpr size_t smem = Lu<MB, NH>::BYTES;
+    constexpr size_t smem = Lu<MB, NH, XB>::BYTES;
     static_assert(smem <= (size_t)227 * 1024, "shared memory");
     int shift = 0;
     while ((1 << shift) < a.block_tokens) ++shift;
-    ensure_dynamic_smem(reinterpret_cast<const void*>(&latent_umma_kernel<MB, NH>), smem);
-    launch_pdl(latent_umma_kernel<MB, NH>, dim3((unsigned)a.n_entries, (unsigned)latent_tc_groups(a.heads)), dim3(LU_THREADS), smem, s, a, shift);
+    ensure_dynamic_smem(reinterpret_cast<const void*>(&latent_umma_kernel<MB, NH, XB>), smem);
+    launch_pdl(latent_umma_kernel<MB, NH, XB>, dim3((unsigned)a.n_entries, (unsigned)latent_tc_groups(a.heads)), dim3(LU_THREADS), smem, s, a, shift);
+}
+
+template <int MB, int NH>
+void launch_umma_extra(const LatentAttnArgs& a, cudaStream_t s) {
+    switch (a.rank - a.values) {
+        case 0: launch_umma<MB, NH, 0>(a, s); break;
+        case 64: launch_umma<MB, NH, 1>(a, s); break;
+        case 128: launch_umma<MB, NH, 2>(a, s); break;
+        default: throw std::runtime_error("launch_latent_attention: unsupported row width");
+    }
 }
 
 template <int MB>
 void launch_umma_heads(const LatentAttnArgs& a, cudaStream_t s) {
-    if (latent_tc_heads(a.heads) == 16) launch_umma<MB, 16>(a, s);
-    else launch_umma<MB, 32>(a, s);
+    if (latent_tc_heads(a.heads) == 16) launch_umma_extra<MB, 16>(a, s);
+    else launch_umma_extra<MB, 32>(a, s);
 }
 
 }  // namespace
 
-int latent_tc_rank(int kv_rank, int block_tokens) {
-    if (block_tokens <= 0 || (block_tokens & (block_tokens - 1)) != 0) return 0;
-    const int r = (kv_rank + LU_COLS - 1) / LU_COLS * LU_COLS;
-    return r <= 4 * LU_COLS ? r : 0;
+LatentColumns latent_tc_columns(int kv_rank, int rot_width, int block_tokens) {
+    LatentColumns c;
+    if (block_tokens <= 0 || (block_tokens & (block_tokens - 1)) != 0) return c;
+    c.values = (kv_rank + LU_COLS - 1) / LU_COLS * LU_COLS;
+    c.rot0 = (kv_rank + 7) / 8 * 8;  // behind the vector, in its padding where there is room
+    const int row = std::max(c.values, rot_width > 0 ? (c.rot0 + rot_width + 63) / 64 * 64 : 0);
+    if (c.values <= 4 * LU_COLS && row <= c.values + 128) c.row = row;
+    return c;
+}
+
+LatentColumns latent_general_columns(int kv_rank, int rot_width) {
+    LatentColumns c;
+    c.values = (kv_rank + 63) / 64 * 64;
+    c.rot0 = (kv_rank + 7) / 8 * 8;
+    c.row = std::max(c.values, rot_width > 0 ? (c.rot0 + rot_width + 63) / 64 * 64 : 0);
+    return c;
 }
 
 int latent_tc_heads(int heads) { return heads <= 16 ? 16 : 32; }
@@ -657,15 +718,16 @@ int latent_max_shared_entries(int ctas) { return std::max(LA_SHARED_ROWS + LA_SH
 int latent_max_entries(int tokens, int ctas) { return std::max(tokens, latent_max_shared_entries(ctas)); }
 
 void plan_latent_attention(const int32_t* start_pos, const int32_t* n_tokens, const int32_t* n_blocks, int lanes, int ctas, int wide_from,
-                           bool shares, LatentPlan& plan) {
+                           bool shares, LatentPlan& plan, int window) {
     plan.entries.clear();
     plan.rows.clear();
+    auto seen = [&](int pos) { return pos + 1 - attention_first_key(pos, window, 0); };  // keys of a position
     int rows = 0;
     int64_t keys = 0;
     for (int i = 0; i < lanes; ++i)
         if (n_tokens[i] < wide_from) {
             rows += n_tokens[i];
-            keys += (int64_t)n_tokens[i] * start_pos[i] + (int64_t)n_tokens[i] * (n_tokens[i] + 1) / 2;
+            for (int t = 0; t < n_tokens[i]; ++t) keys += seen(start_pos[i] + t);
         }
     // Every CTA should walk about the same number of keys and all of them fit on the GPU at once.  Once the rows alone fill it, only
     // a row more than twice as long as the mean is cut.
@@ -679,7 +741,7 @@ void plan_latent_attention(const int32_t* start_pos, const int32_t* n_tokens, co
             int64_t n = 0;
             for (int i = 0; i < lanes; ++i)
                 if (n_tokens[i] < wide_from)
-                    for (int t = 0; t < n_tokens[i]; ++t) n += std::min<int64_t>(LA_MAX_SHARES, (start_pos[i] + t + share) / share);
+                    for (int t = 0; t < n_tokens[i]; ++t) n += std::min<int64_t>(LA_MAX_SHARES, (seen(start_pos[i] + t) - 1 + share) / share);
             if (n <= slots) break;
         }
     }
@@ -687,7 +749,7 @@ void plan_latent_attention(const int32_t* start_pos, const int32_t* n_tokens, co
     for (int i = 0; i < lanes; packed += n_tokens[i], table_off += n_blocks[i], ++i) {
         if (n_tokens[i] >= wide_from) continue;
         for (int t = 0; t < n_tokens[i]; ++t) {
-            const int pos = start_pos[i] + t, n = std::max(1, std::min(LA_MAX_SHARES, (int)(((int64_t)pos + share) / share)));
+            const int pos = start_pos[i] + t, n = std::max(1, std::min(LA_MAX_SHARES, (int)(((int64_t)seen(pos) - 1 + share) / share)));
             const int first = plan.n_entries(), row = plan.n_rows();
             for (int k = 0; k < n; ++k)
                 for (int32_t v : {row, k, n, pos, table_off, packed + t, first, 0}) plan.entries.push_back(v);
@@ -696,13 +758,17 @@ void plan_latent_attention(const int32_t* start_pos, const int32_t* n_tokens, co
     }
 }
 
-void launch_latent_attention(const LatentAttnArgs& a, cudaStream_t s) {
+void launch_latent_attention(const LatentAttnArgs& in, cudaStream_t s) {
+    LatentAttnArgs a = in;
     if (a.n_entries <= 0) return;
-    if (a.out.ld != a.rank) throw std::runtime_error("launch_latent_attention: the output's rows are as wide as the latent");
+    if (a.values == 0) a.values = a.rank;
+    if (a.out.ld != a.values) throw std::runtime_error("launch_latent_attention: the output's rows are as wide as the latent");
+    if (a.rot_dims > 0 && (a.rot0 % 8 != 0 || a.rot_dims % 2 != 0 || a.cos_t == nullptr || a.sin_t == nullptr))
+        throw std::runtime_error("launch_latent_attention: a rotation starts at a multiple of 8 columns and needs its tables");
     if (a.q_h != nullptr) {
         if (!a.pool_f16 || a.out.h == nullptr) throw std::runtime_error("launch_latent_attention: f16 queries go with f16 pages and a bf16 output");
         if (a.status == nullptr) throw std::runtime_error("launch_latent_attention: the tensor-core kernel needs a status word");
-        switch (a.rank) {
+        switch (a.values) {
             case 128: launch_umma_heads<1>(a, s); break;
             case 256: launch_umma_heads<2>(a, s); break;
             case 384: launch_umma_heads<3>(a, s); break;
@@ -710,7 +776,7 @@ void launch_latent_attention(const LatentAttnArgs& a, cudaStream_t s) {
             default: throw std::runtime_error("launch_latent_attention: unsupported rank");
         }
     } else {
-        if (a.rank % 32 != 0 || a.rank > kLatentMaxRank) throw std::runtime_error("launch_latent_attention: latents above 1024 values are not supported");
+        if (a.rank % 64 != 0 || a.values % 32 != 0 || a.rank > kLatentMaxRank) throw std::runtime_error("launch_latent_attention: latents above 1024 values are not supported");
         const size_t smem = ((size_t)LG_WARPS * LG_ITEMS * a.rank + (size_t)LG_KEYS * (a.rank + 4)) * 4;
         auto* kernel = a.pool_f16 ? latent_general_kernel<__half> : latent_general_kernel<float>;
         const dim3 grid((unsigned)a.n_entries, (unsigned)((a.heads + LG_WARPS * LG_ITEMS - 1) / (LG_WARPS * LG_ITEMS)));

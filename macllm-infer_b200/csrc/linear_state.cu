@@ -19,7 +19,7 @@ namespace {
 constexpr int LS_WIDE_WARPS = 4;  // warps of a CTA that owns part of a head
 constexpr int LS_MAX_FINISH_V = 128;
 
-enum LsRule : int { LS_WKV, LS_DELTA, LS_MLSTM };
+enum LsRule : int { LS_WKV, LS_DELTA, LS_MLSTM, LS_CHANNEL };
 template <LsRule RULE>
 struct LsArgs;
 template <>
@@ -28,6 +28,8 @@ template <>
 struct LsArgs<LS_DELTA> { using type = DeltaScanArgs; };
 template <>
 struct LsArgs<LS_MLSTM> { using type = MlstmScanArgs; };
+template <>
+struct LsArgs<LS_CHANNEL> { using type = ChannelDeltaArgs; };
 
 __device__ __forceinline__ void ls_cp_async16(void* dst, const void* src) {
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
@@ -87,7 +89,7 @@ __device__ __forceinline__ void finish_head_row(const LinearStateArgs& a, const 
     const float root = sqrtf(ss / (float)a.vdim + a.eps);
     for (int v = lane; v < a.vdim; v += 32) {
         const float g = gate(v);
-        a.image.put(row, head * a.vdim + v, o[v] / den / root * nw[v] * (a.gate_sigmoid ? sigmoid_f(g) : silu_f(g)));
+        a.image.put(row, head * a.vdim + v, o[v] / den / root * nw[v] * (a.gate_sigmoid ? sigmoid_f(g) : silu_f(g)) * a.out_scale);
     }
     if (head == a.heads - 1)
         for (int c = a.heads * a.vdim + lane; c < a.image.end(); c += 32) a.image.put(row, c, 0.f);
@@ -95,17 +97,18 @@ __device__ __forceinline__ void finish_head_row(const LinearStateArgs& a, const 
 
 template <int KD, LsRule RULE, bool FINISH>
 struct Ls {
-    static constexpr bool WKV = RULE == LS_WKV;
+    static constexpr bool WKV = RULE == LS_WKV, CHANNEL = RULE == LS_CHANNEL;
+    static constexpr bool ROW_DECAY = WKV || CHANNEL;        // a decay per key, as a row of its own
     static constexpr int EXTRA = RULE == LS_MLSTM ? 1 : 0;   // columns of the state beside the values
     static constexpr int KS = !FINISH && KD >= 64 ? 16 : 8;  // threads of a column pair
     static constexpr int KE = KD / KS;                       // keys of a thread
     static constexpr int COLS = 32 / KS * 2;                 // value columns of a warp
     static constexpr int TT = FINISH ? 4 : 16;               // rows of a chunk
-    static constexpr int KROWS = WKV ? 3 : 2;                // r, k, decay  /  q, k
+    static constexpr int KROWS = CHANNEL ? 4 : (WKV ? 3 : 2);  // r, k, decay, removal  /  r, k, decay  /  q, k
     static constexpr int MAX_THREADS = FINISH ? LS_MAX_FINISH_V / COLS * 32 : LS_WIDE_WARPS * 32;
-    static constexpr int MIN_CTAS = FINISH ? (KD >= 128 ? 2 : 3) : 1;
-    // stage: KROWS key-wide rows, the value row, the gate row (FINISH), decay, write and floor of the denominator (not WKV)
-    static __host__ __device__ constexpr int row_floats(int cols) { return KROWS * KD + cols * (FINISH ? 2 : 1) + (WKV ? 0 : 4); }
+    static constexpr int MIN_CTAS = FINISH && !CHANNEL ? (KD >= 128 ? 2 : 3) : 1;
+    // stage: KROWS key-wide rows, the value row, the gate row (FINISH), decay, write and floor of the denominator (not ROW_DECAY)
+    static __host__ __device__ constexpr int row_floats(int cols) { return KROWS * KD + cols * (FINISH ? 2 : 1) + (ROW_DECAY ? 0 : 4); }
     static __host__ __device__ constexpr int stage_floats(int cols) { return TT * row_floats(cols); }
     // two stages; FINISH: the output rows and the head's norm weights
     static __host__ __device__ constexpr size_t bytes(int cols) { return (2 * (size_t)stage_floats(cols) + (FINISH ? (size_t)(TT + 1) * cols : 0)) * 4; }
@@ -115,7 +118,7 @@ template <int KD, LsRule RULE, bool FINISH>
 __global__ void __launch_bounds__(Ls<KD, RULE, FINISH>::MAX_THREADS, Ls<KD, RULE, FINISH>::MIN_CTAS)
 linear_state_kernel(const __grid_constant__ typename LsArgs<RULE>::type ra) {
     using L = Ls<KD, RULE, FINISH>;
-    constexpr bool WKV = L::WKV;
+    constexpr bool WKV = L::WKV, CHANNEL = L::CHANNEL, ROW_DECAY = L::ROW_DECAY;
     constexpr int TT = L::TT, KS = L::KS, KE = L::KE, NJ = KE / 4;
     extern __shared__ __align__(16) float ls_smem[];
     const LinearStateArgs& a = ra.common;
@@ -201,6 +204,11 @@ linear_state_kernel(const __grid_constant__ typename LsArgs<RULE>::type ra) {
             const int h0 = head * a.dim;
             fetch_heads(ra.rkv, ra.r_col + h0, ra.k_col + h0, ra.v_col + h0 + col0);
             fetch_rows(s + 2 * TT * KD, KD, m, a.dim, vec, [&](int r) { return ra.decay + (r0 + r) * a.heads * a.dim + h0; });
+        } else if constexpr (CHANNEL) {
+            const int h0 = head * a.dim;
+            fetch_heads(ra.y, ra.r_col + h0, ra.k_col + h0, ra.v_col + head * a.vdim + col0);
+            fetch_rows(s + 2 * TT * KD, KD, m, a.dim, vec, [&](int r) { return ra.decay + (r0 + r) * a.heads * a.dim + h0; });
+            fetch_rows(s + 3 * TT * KD, KD, m, a.dim, vec, [&](int r) { return ra.removal + (r0 + r) * a.heads * a.dim + h0; });
         } else if constexpr (RULE == LS_MLSTM) {
             const int h0 = head * a.dim;
             fetch_heads(ra.y, ra.q_col + h0, ra.k_col + h0, ra.v_col + head * a.vdim + col0);
@@ -265,19 +273,20 @@ linear_state_kernel(const __grid_constant__ typename LsArgs<RULE>::type ra) {
                 for (int i = threadIdx.x; i < KD; i += blockDim.x) {
                     s[t * KD + i] = 0.f;
                     s[TT * KD + t * KD + i] = 0.f;
-                    if (WKV) s[2 * TT * KD + t * KD + i] = 1.f;
+                    if (ROW_DECAY) s[2 * TT * KD + t * KD + i] = 1.f;
+                    if (CHANNEL) s[3 * TT * KD + t * KD + i] = 0.f;
                 }
                 for (int i = threadIdx.x; i < cols; i += blockDim.x) s_v[t * cols + i] = 0.f;
-                if (!WKV && threadIdx.x == 0) {
+                if (!ROW_DECAY && threadIdx.x == 0) {
                     s_c[4 * t] = 1.f;
                     s_c[4 * t + 1] = 0.f;
                 }
             }
         }
         __syncthreads();
-        // one row's vectors: r | q in x, k in y, decay in w (WKV)
+        // one row's vectors: r | q in x, k in y, decay in w (WKV, CHANNEL), removal in b (CHANNEL)
         struct Row {
-            float x[KE], y[KE], w[WKV ? KE : 1];
+            float x[KE], y[KE], w[ROW_DECAY ? KE : 1], b[CHANNEL ? KE : 1];
             float2 v, gb;
         };
         auto load_row = [&](int t, Row& r) {
@@ -289,7 +298,7 @@ linear_state_kernel(const __grid_constant__ typename LsArgs<RULE>::type ra) {
                 r.y[4 * j] = y.x; r.y[4 * j + 1] = y.y; r.y[4 * j + 2] = y.z; r.y[4 * j + 3] = y.w;
                 r.x[4 * j] = x.x; r.x[4 * j + 1] = x.y; r.x[4 * j + 2] = x.z; r.x[4 * j + 3] = x.w;
             }
-            if constexpr (WKV) {
+            if constexpr (ROW_DECAY) {
                 const float4* w4 = reinterpret_cast<const float4*>(s + 2 * TT * KD + t * KD) + ks;
 #pragma unroll
                 for (int j = 0; j < NJ; ++j) {
@@ -298,6 +307,14 @@ linear_state_kernel(const __grid_constant__ typename LsArgs<RULE>::type ra) {
                 }
             } else {
                 r.gb = *reinterpret_cast<const float2*>(s_c + 4 * t);
+            }
+            if constexpr (CHANNEL) {
+                const float4* b4 = reinterpret_cast<const float4*>(s + 3 * TT * KD + t * KD) + ks;
+#pragma unroll
+                for (int j = 0; j < NJ; ++j) {
+                    const float4 b = b4[j * KS];
+                    r.b[4 * j] = b.x; r.b[4 * j + 1] = b.y; r.b[4 * j + 2] = b.z; r.b[4 * j + 3] = b.w;
+                }
             }
             r.v = *reinterpret_cast<const float2*>(s_v + t * cols + c_loc);
         };
@@ -333,6 +350,18 @@ linear_state_kernel(const __grid_constant__ typename LsArgs<RULE>::type ra) {
                 for (int x = 1; x < KS; x <<= 1) {
                     m0 += __shfl_xor_sync(0xffffffffu, m0, x);
                     m1 += __shfl_xor_sync(0xffffffffu, m1, x);
+                }
+                if constexpr (CHANNEL) {
+#pragma unroll
+                    for (int e = 0; e < KE; ++e) {
+                        S[0][e] = fmaf(-r.b[e], m0, fmaf(r.w[e], S[0][e], r.y[e] * r.v.x));
+                        S[1][e] = fmaf(-r.b[e], m1, fmaf(r.w[e], S[1][e], r.y[e] * r.v.y));
+                        o0 = fmaf(S[0][e], r.x[e], o0);
+                        o1 = fmaf(S[1][e], r.x[e], o1);
+                    }
+                    out0 = o0;
+                    out1 = o1;
+                    return;
                 }
                 const float u0 = r.gb.y * (r.v.x - r.gb.x * m0), u1 = r.gb.y * (r.v.y - r.gb.x * m1);
 #pragma unroll
@@ -441,6 +470,7 @@ __global__ void __launch_bounds__(128) head_norm_gate_vec_kernel(LinearStateArgs
     for (int x = 1; x < G; x <<= 1) ss += __shfl_xor_sync(0xffffffffu, ss, x);
     const float root = sqrtf(ss / (float)a.vdim + a.eps);
     if (mine) {
+        w = make_float4(w.x * a.out_scale, w.y * a.out_scale, w.z * a.out_scale, w.w * a.out_scale);
         g = a.gate_sigmoid ? make_float4(sigmoid_f(g.x), sigmoid_f(g.y), sigmoid_f(g.z), sigmoid_f(g.w)) : make_float4(silu_f(g.x), silu_f(g.y), silu_f(g.z), silu_f(g.w));
         a.image.put4(row, head * a.vdim + v, make_float4(o.x / root * w.x * g.x, o.y / root * w.y * g.y, o.z / root * w.z * g.z, o.w / root * w.w * g.w));
     }
@@ -520,6 +550,11 @@ int launch_mlstm_scan(const MlstmScanArgs& a, cudaStream_t s) {
 void launch_delta_scan(const DeltaScanArgs& a, cudaStream_t s) {
     if (a.kv_heads <= 0 || a.common.heads % a.kv_heads != 0) throw std::runtime_error("delta-rule scan: heads must be a multiple of kv_heads");
     launch_scan<LS_DELTA>(a, s);
+}
+
+void launch_channel_delta_scan(const ChannelDeltaArgs& a, cudaStream_t s) {
+    if (a.common.dim != a.common.vdim) throw std::runtime_error("delta-rule scan with channel gates: square heads only");
+    launch_scan<LS_CHANNEL>(a, s);
 }
 
 void launch_head_norm_gate(const LinearStateArgs& a, int rows, cudaStream_t s) {

@@ -1,6 +1,6 @@
 // Linear-attention recurrences over ragged lanes with slot-held state: WKV time mixing (a decay per key channel and a bonus for
-// the current token), the gated delta rule (one decay per head, grouped query / key heads) and the matrix memory of mLSTM (one
-// decay per head from exponential gates, a normaliser).  State layout per slot half: [heads][value columns][KD] f32, value-major,
+// the current token), the gated delta rule (one decay per head, grouped query / key heads), the matrix memory of mLSTM (one
+// decay per head from exponential gates, a normaliser) and the delta rule with a decay and a removal rate per key channel.  State layout per slot half: [heads][value columns][KD] f32, value-major,
 // KD = the key dimension padded to 32, 64, 128 or 256 - a column's keys are contiguous, so a decode tick streams the state with
 // 16-byte accesses.  mLSTM has one column more than values: the normaliser, whose value is always 1.
 #pragma once
@@ -20,6 +20,7 @@ struct LinearStateArgs {
     float* out = nullptr;            // [rows][heads][vdim], normalised: [rows][heads][linear_state_raw_width(vdim)]
     int normalised = 0;              // a raw head row ends with its denominator (mLSTM): divided by it before the norm
     int gate_sigmoid = 0;            // sigmoid(gate) instead of silu(gate)
+    float out_scale = 1.f;           // of the finished rows
     RowImage image;                  // [rows][heads * vdim]
     const float* norm_w = nullptr;   // [heads * vdim], or [vdim] shared by the heads
     int norm_per_head = 0;           // norm_w has its own part for every head
@@ -76,6 +77,17 @@ int launch_mlstm_scan(const MlstmScanArgs& a, cudaStream_t s);
 // The forms behind it (mlstm.cu): one-token lanes, finished; chunks of prompts, whose raw rows are [heads][vdim] and divided already.
 void launch_mlstm_step(const MlstmScanArgs& a, cudaStream_t s);
 void launch_mlstm_chunks(const MlstmScanArgs& a, cudaStream_t s);
+
+// S <- diag(w) S - (a u)(u^T S) + k v^T with both terms reading the old state, u the head's unit key;  o = S^T r.  With
+// removal = a k / (sum k^2 + 1e-6) the middle term is removal (k^T S).
+struct ChannelDeltaArgs {
+    LinearStateArgs common;
+    Shares y;                        // columns r_col / k_col / v_col + head * dim + i
+    int r_col = 0, k_col = 0, v_col = 0;
+    const float* decay = nullptr;    // [rows][heads * dim]
+    const float* removal = nullptr;  // [rows][heads * dim]
+};
+void launch_channel_delta_scan(const ChannelDeltaArgs& a, cudaStream_t s);
 
 // Whether the finishing form (LinearStateArgs::image) exists for these sizes.
 bool linear_state_can_finish(int dim, int vdim);

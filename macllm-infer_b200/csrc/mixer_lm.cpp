@@ -13,7 +13,7 @@ namespace {
 
 const std::vector<const char*> class_names = {"hgemm_tc", "hgemm_tc_splitk", "f32_matmul", "wkv_scan", "delta_scan", "paged_attention", "rope_kv_scatter",
                                               "row_update", "delta_prep", "wkv_decay", "latent_attention", "mingru_scan", "latent_prep", "latent_rows",
-                                              "mlstm_scan", "moe_gemm", "moe_route", "moe_gather", "gates", "embed", "build_batch", "argmax"};
+                                              "mlstm_scan", "moe_gemm", "moe_route", "moe_gather", "gates", "channel_gates", "embed", "build_batch", "argmax"};
 
 bool is_mixer_checkpoint(const std::string& dir) {
     struct stat st;
@@ -65,7 +65,8 @@ void MixerLm::upload_f32(const std::vector<float>& v, DevBuf& out) {
 }
 
 void MixerLm::upload_norm(const SafetensorsFile& f, const std::string& name, Norm& out) {
-    upload_f32(f.values(name, {ms_.width}), out.w);
+    if (ms_.one_number_norms) upload_f32(std::vector<float>((size_t)ms_.width, f.values(name, {}).at(0)), out.w);
+    else upload_f32(f.values(name, {ms_.width}), out.w);
     if (ms_.norm != NormKind::DynTanh) return;
     upload_f32(f.values(name + ".b", {ms_.width}), out.b);
     out.alpha = f.values(name + ".alpha", {}).at(0);
@@ -76,7 +77,12 @@ void MixerLm::place(const SafetensorsFile& f, const Part& p, int cols, int ld, s
     const std::vector<float> v = f.values(p.name, {p.rows, n});
 #pragma omp parallel for
     for (int r = 0; r < p.rows; ++r) {
-        const int64_t row = p.at + (int64_t)(r / block) * p.pitch + (int64_t)(r % block) * p.step;
+        int in_block = r % block;
+        if (p.turn_from >= 0 && in_block >= p.turn_from) {
+            const int i = in_block - p.turn_from, half = p.turn_dims / 2;
+            in_block = p.turn_to + (i >= p.turn_dims ? i : (i < half ? 2 * i : 2 * (i - half) + 1));
+        }
+        const int64_t row = p.at + (int64_t)(r / block) * p.pitch + (int64_t)in_block * p.step;
         memcpy(&m[(size_t)(row * ld + p.col)], &v[(size_t)r * n], (size_t)n * 4);
     }
 }
@@ -145,6 +151,7 @@ int MixerLm::geometry_of(const AttentionSpec& a) {
     g.heads = a.heads;
     g.kv_heads = a.kv_heads;
     g.chunk = a.chunk;
+    g.window = a.window;
     // the tensor-core kernels take rows of 64, 128 or 256; narrower heads are padded with zeros in the pools
     for (int d : {64, 128, 256})
         if (need <= d && !g.tc && attention_tc_supported(a.heads, a.kv_heads, d, cfg_.block_tokens, cfg_.kv_f16)) {
@@ -155,7 +162,7 @@ int MixerLm::geometry_of(const AttentionSpec& a) {
     if (g.row_width > 256) throw std::runtime_error("attention head dimensions above 256 are not supported");
     if (a.heads / a.kv_heads > 64) throw std::runtime_error("more than 64 query heads per key/value head are not supported");
     for (size_t i = 0; i < geo_.size(); ++i)
-        if (geo_[i].heads == g.heads && geo_[i].kv_heads == g.kv_heads && geo_[i].row_width == g.row_width && geo_[i].chunk == g.chunk) return (int)i;
+        if (geo_[i].heads == g.heads && geo_[i].kv_heads == g.kv_heads && geo_[i].row_width == g.row_width && geo_[i].chunk == g.chunk && geo_[i].window == g.window) return (int)i;
     geo_.push_back(std::move(g));
     return (int)geo_.size() - 1;
 }
@@ -206,6 +213,7 @@ void MixerLm::load_layer(const SafetensorsFile& f, int l) {
     Layer& w = lw_[(size_t)l];
     if (ms_.side_by_side()) return load_side_by_side(f, l);
     if (ms_.norm_place == NormPlace::Output) return load_output_norm(f, l);
+    if (ms_.conv_taps > 0) return load_conv_input(f, l);
     const int C = ms_.width;
     const std::string p = "l" + std::to_string(l) + ".", m = p + "mix.";
     upload_norm(f, p + "norm1", w.norm1);
@@ -222,14 +230,7 @@ void MixerLm::load_layer(const SafetensorsFile& f, int l) {
             mu.insert(mu.end(), v.begin(), v.end());
         }
         upload_f32(mu, w.mu);
-        const std::vector<float> w2 = f.values(m + "w2", {HD, R});
-        std::vector<float> w2t((size_t)HD * R);
-        for (int c = 0; c < HD; ++c)
-            for (int j = 0; j < R; ++j) w2t[(size_t)j * HD + c] = w2[(size_t)c * R + j];
-        upload_f32(w2t, w.w2t);
-        spec_.weight_bytes += (int64_t)HD * R * 4;
-        spec_.weight_bytes_per_token += (int64_t)HD * R * 4;
-        upload_f32(f.values(m + "w0", {HD}), w.w0);
+        upload_low_rank(f, m, HD, R, w);
         upload_f32(f.values(m + "u", {s.wkv.heads, s.wkv.dim}), w.bonus);
         upload_f32(f.values(m + "norm", {HD}), w.head_norm);
         upload_dense(f, {{m + "o", C, 0}}, C, HD, w.out);
@@ -296,6 +297,18 @@ void MixerLm::load_layer(const SafetensorsFile& f, int l) {
     }
 }
 
+// The second half of a low-rank projection and its bias, for the kernels that keep it in f32.
+void MixerLm::upload_low_rank(const SafetensorsFile& f, const std::string& prefix, int channels, int rank, Layer& w) {
+    const std::vector<float> w2 = f.values(prefix + "w2", {channels, rank});
+    std::vector<float> w2t(w2.size());
+    for (int c = 0; c < channels; ++c)
+        for (int j = 0; j < rank; ++j) w2t[(size_t)j * channels + c] = w2[(size_t)c * rank + j];
+    upload_f32(w2t, w.w2t);
+    spec_.weight_bytes += (int64_t)channels * rank * 4;
+    spec_.weight_bytes_per_token += (int64_t)channels * rank * 4;
+    upload_f32(f.values(prefix + "w0", {channels}), w.w0);
+}
+
 void MixerLm::alloc_run(int run) {
     const int l = runs_[(size_t)run].layer;
     const MixerLayerSpec& s = ms_.layers[(size_t)l];
@@ -309,6 +322,7 @@ void MixerLm::alloc_run(int run) {
         spec_.kv_bytes_per_token += bytes / cfg_.block_tokens;
     };
     if (s.kind == MixerKind::Wkv || ms_.side_by_side()) st.kept.alloc(halves * (size_t)ms_.width * 4);  // the token shift's row
+    if (ms_.conv_taps > 1) st.kept.alloc(halves * (size_t)(ms_.conv_taps - 1) * ms_.width * 4);
     switch (s.kind) {
         case MixerKind::Wkv:
             st.state.alloc(halves * (size_t)s.wkv.heads * s.wkv.dim * linear_state_key_pad(s.wkv.dim) * 4);
@@ -321,6 +335,11 @@ void MixerLm::alloc_run(int run) {
             st.state.alloc(halves * (size_t)d.heads * d.vdim * linear_state_key_pad(d.dim) * 4);
             break;
         }
+        case MixerKind::ScaledParallel:
+            pages(st.k_pool, s.attn.kv_heads);
+            pages(st.v_pool, s.attn.kv_heads);
+            st.state.alloc(halves * (size_t)s.channel_delta.heads * s.channel_delta.dim * linear_state_key_pad(s.channel_delta.dim) * 4);
+            break;
         case MixerKind::Latent: pages(st.k_pool, 1); break;
         case MixerKind::MinGru: st.state.alloc(halves * (size_t)s.gru.width * 4); break;
         case MixerKind::Mlstm:
@@ -341,7 +360,7 @@ void MixerLm::alloc_activations() {
     int64_t q_lat = 0, uq = 0, lat = 0, cat = 0;  // widths of latent attention's rows, and of `out`'s input with both branches
     int lat_ctas = 1;
     int64_t lat_part = 0;
-    int64_t mlstm_heads = 0, qkv = 0;
+    int64_t mlstm_heads = 0, qkv = 0, removal = 0;
     int64_t pairs = 0, experts = 0, expert_ff = 0, expert_gu = 0;  // routed rows, experts, widths of an expert's activations
     for (size_t l = 0; l < lw_.size(); ++l) {
         const MixerLayerSpec& s = ms_.layers[l];
@@ -367,21 +386,22 @@ void MixerLm::alloc_activations() {
             ff = std::max(ff, (int64_t)pad_to(s.moe.shared_ff, 64));
             continue;
         }
+        if (s.kind == MixerKind::Latent) {
+            const LatentSpec& a = s.latent;
+            q_lat = std::max(q_lat, (int64_t)w.uq.ld);
+            uq = std::max(uq, (int64_t)a.heads * w.q_width);
+            lat = std::max(lat, (int64_t)a.heads * w.row_width);
+            const LatentGeometry& g = latent_geo_[(size_t)w.geometry];
+            if (g.wide) attn = std::max(attn, (int64_t)a.heads * w.q_width);
+            lat_ctas = std::max(lat_ctas, g.ctas);
+            if (g.tc) lat_part = std::max(lat_part, (int64_t)latent_max_shared_entries(g.ctas) * latent_tc_groups(a.heads) * latent_tc_heads(a.heads) * w.value_width);
+        }
         if (ms_.side_by_side()) {
             mix = 2;
             cat = std::max(cat, (int64_t)w.out.ld);
-            if (s.kind == MixerKind::Latent) {
-                const LatentSpec& a = s.latent;
-                q_lat = std::max(q_lat, (int64_t)w.uq.ld);
-                uq = std::max(uq, (int64_t)a.heads * w.q_width);
-                lat = std::max(lat, (int64_t)a.heads * w.row_width);
-                const LatentGeometry& g = latent_geo_[(size_t)w.geometry];
-                if (g.wide) attn = std::max(attn, (int64_t)a.heads * w.q_width);
-                lat_ctas = std::max(lat_ctas, g.ctas);
-                if (g.tc) lat_part = std::max(lat_part, (int64_t)latent_max_shared_entries(g.ctas) * latent_tc_groups(a.heads) * latent_tc_heads(a.heads) * w.row_width);
-            }
             continue;
         }
+        if (ms_.conv_taps > 0) cat = std::max(cat, (int64_t)w.out.ld);
         ff = std::max(ff, (int64_t)s.ff);
         if (s.kind == MixerKind::Wkv) {
             mix = 5;
@@ -398,6 +418,12 @@ void MixerLm::alloc_activations() {
             dqk = std::max(dqk, (int64_t)s.delta.kv_heads * s.delta.dim);
             dv = std::max(dv, n);
             dh = std::max(dh, (int64_t)s.delta.heads);
+        } else if (s.kind == MixerKind::ScaledParallel) {
+            attn = std::max(attn, (int64_t)s.attn.heads * w.row_width);
+            const int64_t n = (int64_t)s.channel_delta.heads * s.channel_delta.dim;
+            removal = std::max(removal, n);
+            hd = std::max(hd, n);
+            raw = std::max(raw, n);
         }
     }
     const int64_t ldc = pad_to(C, 64);
@@ -433,6 +459,7 @@ void MixerLm::alloc_activations() {
         moe_.shared_gate = moe_.weight_of_pos + pairs;
     }
     decay_.alloc((size_t)(T * hd) * 4);
+    removal_.alloc((size_t)(T * removal) * 4);
     raw_.alloc((size_t)(T * raw) * 4);
     q_rot_.alloc((size_t)(T * attn) * 4);
     img_q_.alloc((size_t)(T * q_lat) * esz_);
@@ -471,7 +498,7 @@ void MixerLm::alloc_activations() {
         }
     }
     for (const LatentGeometry& g : latent_geo_) extra += (size_t)latent_max_entries((int)T, g.ctas) * 32 + (size_t)T * 4 + 32;
-    if (!latent_geo_.empty()) extra += (size_t)B * sizeof(LaneHeader) + (size_t)(T + B) * 8 + (size_t)T * 4 + (size_t)(pool_->max_blocks() + B) * 4 + 64;
+    extra += wide_.size() * ((size_t)B * sizeof(LaneHeader) + (size_t)(T + B) * 8 + (size_t)T * 4 + (size_t)(pool_->max_blocks() + B) * 4 + 64);
     attn_part_o_.alloc(part_o);
     attn_part_ml_.alloc(part_ml);
     attn_counters_.alloc(counters);
@@ -631,7 +658,7 @@ void MixerLm::attend(const Tick& t, int run, const AttentionSpec& s, const Share
     RopeKvArgs ra;
     ra.q = const_cast<float*>(y.p) + w.c_q;
     ra.k = y.p + w.c_k;
-    ra.v = y.p + w.c_v;
+    ra.v = y.p + (s.keys_are_values ? w.c_k : w.c_v);
     ra.ldq = ra.ldk = ra.ldv = y.ld;
     ra.qk_splits = ra.v_splits = y.n;
     ra.qk_split_stride = ra.v_split_stride = y.stride;
@@ -643,7 +670,7 @@ void MixerLm::attend(const Tick& t, int run, const AttentionSpec& s, const Share
     if (s.biases) {
         ra.q_bias = w.q_b.as<float>();
         ra.k_bias = w.k_b.as<float>();
-        ra.v_bias = w.v_b.as<float>();
+        ra.v_bias = (s.keys_are_values ? w.k_b : w.v_b).as<float>();
     }
     if (s.rot.dims > 0) {
         ra.cos_t = rope_[(size_t)w.rope]->cos_t.as<float>();
@@ -678,10 +705,13 @@ void MixerLm::attend(const Tick& t, int run, const AttentionSpec& s, const Share
     }
     double kv_tokens = 0, flops = 0;
     for (const LmLane& ln : lanes) {
-        const int lo = attention_first_key(ln.start_pos, 0, s.chunk);
+        const int lo = attention_first_key(ln.start_pos, s.window, s.chunk);
         kv_tokens += (double)ln.start_pos + ln.n_tokens - lo;
         double pairs = (double)ln.n_tokens * (ln.start_pos - lo) + 0.5 * ln.n_tokens * ln.n_tokens;
-        if (s.chunk > 0) pairs = std::min(pairs, (double)ln.n_tokens * 0.5 * (s.chunk + 1));
+        if (s.window > 0) {
+            pairs = 0;
+            for (int k = 0; k < ln.n_tokens; ++k) pairs += ln.start_pos + k + 1 - attention_first_key(ln.start_pos + k, s.window, s.chunk);
+        } else if (s.chunk > 0) pairs = std::min(pairs, (double)ln.n_tokens * 0.5 * (s.chunk + 1));
         flops += 2.0 * s.heads * (s.dim + s.vdim) * pairs;
     }
     prof_begin(KC_ATTN, kv_tokens * 2 * s.kv_heads * D * kv_esz + 8.0 * T * s.heads * D, flops);
@@ -712,6 +742,7 @@ void MixerLm::attend(const Tick& t, int run, const AttentionSpec& s, const Share
         ta.scale = s.scale;
         ta.softcap = s.softcap;
         ta.chunk = s.chunk;
+        ta.window = s.window;
         ta.sink = s.sink ? w.sink.as<float>() : nullptr;
         ta.exact_weights = 1;
         if (fuse_rope) {
@@ -739,6 +770,7 @@ void MixerLm::attend(const Tick& t, int run, const AttentionSpec& s, const Share
         at.scale = s.scale;
         at.softcap = s.softcap;
         at.chunk = s.chunk;
+        at.window = s.window;
         at.sink = s.sink ? w.sink.as<float>() : nullptr;
         at.q_tile = attention_q_tile(s.heads, s.kv_heads);
         launch_paged_attention(at, stream_);
@@ -862,7 +894,7 @@ void MixerLm::run_forward(const std::vector<LmLane>& lanes, KvReservation& r, ui
     }
     for (Geometry& g : geo_) {
         if (g.tc) {
-            plan_attention_tc(sp.data(), nt.data(), nb.data(), B, g.heads, g.kv_heads, g.plan, g.chunk);
+            plan_attention_tc(sp.data(), nt.data(), nb.data(), B, g.heads, g.kv_heads, g.plan, g.chunk, g.window);
             if (g.plan.n_entries() > attn_max_entries_) throw std::runtime_error("attention work list exceeds its scratch");
             g.off_entries = stage_bytes(t, g.plan.entries.data(), g.plan.entries.size() * 4);
             g.off_tiles = stage_bytes(t, g.plan.tiles.data(), g.plan.tiles.size() * 4);
@@ -936,6 +968,7 @@ void MixerLm::run_forward(const std::vector<LmLane>& lanes, KvReservation& r, ui
         if (runs_[(size_t)run].first) begin_pass(t, runs_[(size_t)run].pass, pend);
         if (ms_.side_by_side()) run_side_by_side(t, run, pend, lanes);
         else if (ms_.norm_place == NormPlace::Output) run_output_norm(t, run, pend, lanes);
+        else if (ms_.conv_taps > 0) run_conv_input(t, run, pend, lanes);
         else if (s.kind == MixerKind::Wkv) run_wkv(t, run, pend);
         else run_parallel(t, run, pend, lanes);
         if (s.ff > 0 && ms_.norm_place == NormPlace::Input) {
@@ -948,17 +981,19 @@ void MixerLm::run_forward(const std::vector<LmLane>& lanes, KvReservation& r, ui
             launch_row_update(u, stream_);
             prof_end();
             const RowImage img = image(img_ff_, w.down.ld);
+            GatedAct act;
+            act.kind = ms_.ff_kind == FfKind::GatedGelu ? GatedAct::GeluTanh : GatedAct::Silu;
             if (f32_) {
                 const Shares gu = matmul(w.gate_up, u.normed, T, y_gu_, 0);
                 prof_begin(KC_GATES, 12.0 * T * s.ff, 0);
-                launch_gated_act(gu, T, s.ff, img, stream_);
+                launch_gated_act(gu, T, s.ff, img, stream_, act);
                 prof_end();
             } else {
-                // silu(gate) * up in the matmul's epilogue
+                // act(gate) * up in the matmul's epilogue
                 prof_begin(T <= 64 ? KC_GEMM_NARROW : KC_GEMM, (double)w.gate_up.bytes + 2.0 * T * C + 2.0 * T * s.ff, 2.0 * T * (double)w.gate_up.rows * w.gate_up.ld);
                 HgemmScratch ws;
                 ws.status = status_.as<int32_t>();
-                launch_hgemm_tc_gated(w.gate_up.half, reinterpret_cast<const __half*>(u.normed.h), T, GatedAct{}, reinterpret_cast<__half*>(img.h), img.ld, ws, stream_);
+                launch_hgemm_tc_gated(w.gate_up.half, reinterpret_cast<const __half*>(u.normed.h), T, act, reinterpret_cast<__half*>(img.h), img.ld, ws, stream_);
                 prof_end();
             }
             launches_ += 2;

@@ -46,7 +46,9 @@ private:
         DevBuf w, b;
     };
     // Part of a stacked matrix: `rows` rows of tensor `name`, placed from row `at` on, `step` rows apart; with `block` set, runs of
-    // `block` rows begin `pitch` rows apart.  Columns from `col` on, `cols` of them (0: the matrix's).
+    // `block` rows begin `pitch` rows apart.  Columns from `col` on, `cols` of them (0: the matrix's).  With turn_from >= 0 the rows of a
+    // run from turn_from on go to turn_to on, the first turn_dims of them in an order that makes the halves' pairs (i, i + turn_dims / 2)
+    // neighbours: a rotation then turns adjacent rows.
     struct Part {
         std::string name;
         int rows;
@@ -54,6 +56,7 @@ private:
         int step = 1;
         int col = 0, cols = 0;
         int block = 0, pitch = 0;
+        int turn_from = -1, turn_to = 0, turn_dims = 0;
     };
     struct Layer {
         Norm norm1, norm2;
@@ -76,7 +79,13 @@ private:
         Dense uq, uk, uv, ukv;
         int c_kv = 0;         // column of the key/value latent (c_q: of the query latent)
         int q_width = 0;      // padded width of a query head
+        int value_width = 0;  // columns of `row_width` that values come from
+        int rot0 = 0, q_rot0 = 0, c_rot = 0;  // rotated part: its column in a page row and in a query head, its projection's column
         int mix_cols = 0;     // columns of the mixer in `out`'s input; the feed-forward's follow
+        // delta rule with channel gates (columns d_q: r, d_k, d_v, d_a, d_g, c_low; w2t, w0 as WKV's)
+        DevBuf a_b;
+        // the short convolution in front of the mixer, [taps][width]
+        DevBuf input_conv;
         // minGRU (columns c_q: z, c_v: x, c_g: g)
         DevBuf z_b, x_b;
         // feed-forward beside the mixer
@@ -98,7 +107,7 @@ private:
     };
     // Layers with the same heads share a tick's attention work list.
     struct Geometry {
-        int heads = 0, kv_heads = 0, row_width = 0, chunk = 0;
+        int heads = 0, kv_heads = 0, row_width = 0, chunk = 0, window = 0;
         bool tc = false;
         AttnTcPlan plan;
         size_t off_tiles = 0, off_entries = 0, off_dec = 0;
@@ -110,12 +119,15 @@ private:
         int ctas = 1;        // CTAs per entry
         bool tc = false;     // tensor-core kernel
         bool wide = false;   // lanes with many tokens run on expanded keys and values
+        int window = 0;
+        int lanes = 0;       // wide: which of wide_
         LatentPlan plan;
         size_t off_entries = 0, off_rows = 0;
     };
-    // The tick's lanes that run on expanded keys and values.
+    // The tick's lanes that run on expanded keys and values, of the layers with the same window.
     struct WideLanes {
-        std::vector<LaneHeader> hdr;          // by lane; table_off: first expanded block
+        int window = 0;
+        std::vector<LaneHeader> hdr;          // by lane; table_off: where block 0 would be among the expanded ones
         std::vector<int32_t> tiles, rows, blocks;
         size_t off_hdr = 0, off_tiles = 0, off_rows = 0, off_blocks = 0;
         double keys = 0, pairs = 0;           // of the profile: keys expanded, (query, key) pairs
@@ -125,7 +137,7 @@ private:
         DevBuf cos_t, sin_t;
     };
     enum KClass { KC_GEMM = 0, KC_GEMM_NARROW, KC_F32_MATMUL, KC_WKV_SCAN, KC_DELTA_SCAN, KC_ATTN, KC_ROPE_KV, KC_ROW_UPDATE, KC_DELTA_PREP, KC_WKV_DECAY,
-                  KC_LATENT_ATTN, KC_MINGRU, KC_LATENT_PREP, KC_LATENT_ROWS, KC_MLSTM_SCAN, KC_MOE_GEMM, KC_MOE_ROUTE, KC_MOE_GATHER, KC_GATES, KC_EMBED, KC_BATCH,
+                  KC_LATENT_ATTN, KC_MINGRU, KC_LATENT_PREP, KC_LATENT_ROWS, KC_MLSTM_SCAN, KC_MOE_GEMM, KC_MOE_ROUTE, KC_MOE_GATHER, KC_GATES, KC_CHANNEL_GATES, KC_EMBED, KC_BATCH,
                   KC_SAMPLE, KC_COUNT };
 
     void load(const SafetensorsFile& f);
@@ -151,7 +163,7 @@ private:
     Shares matmul(const Dense& W, const RowImage& x, int T, DevBuf& y, int scratch);
     void matmul_scatter(const Dense& W, const RowImage& x, int T, const MatmulScatter& to);
     void set_norm(RowUpdateArgs& a, const Norm& n) const;
-    int latent_geometry(int ctas, bool tc, bool wide);
+    int latent_geometry(int ctas, bool tc, bool wide, int window);
     void plan_latent(Tick& t, const std::vector<int32_t>& start, const std::vector<int32_t>& n_tokens, const std::vector<int32_t>& n_blocks, KvReservation& r);
 
     // Branch outputs not yet added to the residual stream.
@@ -170,6 +182,11 @@ private:
     void run_parallel(const Tick& t, int run, Pending& p, const std::vector<LmLane>& lanes);
     // Queries, keys and values out of the projections `y`, page write and attention: leaves the heads' outputs in attn_.
     void attend(const Tick& t, int run, const AttentionSpec& s, const Shares& y, const std::vector<LmLane>& lanes);
+    // layers whose mixer reads a short convolution over its norm
+    void load_conv_input(const SafetensorsFile& f, int l);
+    void run_conv_input(const Tick& t, int run, Pending& p, const std::vector<LmLane>& lanes);
+    void run_channel_delta(const Tick& t, int run, const Shares& y, const RowImage& out);
+    void upload_low_rank(const SafetensorsFile& f, const std::string& prefix, int channels, int rank, Layer& w);
     // layers whose mixer and feed-forward read one norm
     void begin_pass(const Tick& t, int pass, Pending& p);
     void run_side_by_side(const Tick& t, int run, Pending& p, const std::vector<LmLane>& lanes);
@@ -179,6 +196,8 @@ private:
     void run_moe(const Tick& t, int layer, Pending& p);
     void run_latent(const Tick& t, int run, const Shares& y, const RowImage& out, const std::vector<LmLane>& lanes);
     void run_latent_wide(const Tick& t, int run, const Shares& y, const RowImage& out);
+    void latent_prep_args(const Tick& t, int run, const Shares& y, LatentPrepArgs& p);
+    int latent_qkv(const std::string& mix, const LatentSpec& s, Layer& w, std::vector<Part>& parts, int at) const;
 
     MixerSpec ms_;
     bool f32_ = false;
@@ -192,12 +211,12 @@ private:
     Norm final_norm_;
     std::vector<Geometry> geo_;
     std::vector<LatentGeometry> latent_geo_;
-    WideLanes wide_;
+    std::vector<WideLanes> wide_;
     std::vector<std::unique_ptr<RopeTable>> rope_;
 
     // activations of one tick
     DevBuf x_[2], mixes_, img_h_, img_a_, img_b_, img_ff_, img_side_;
-    DevBuf y_in_, y_a_, y_b_, y_gu_, decay_, raw_, q_rot_, attn_, dq_, dk_, dv_, dbeta_, ddecay_;
+    DevBuf y_in_, y_a_, y_b_, y_gu_, decay_, removal_, raw_, q_rot_, attn_, dq_, dk_, dv_, dbeta_, ddecay_;
     // layers with one norm: loop entry, latents, per-head queries, queries and outputs in the latent space, mixer | feed-forward,
     // expanded keys and values (and the vectors they come from)
     DevBuf img_loop_, img_q_, img_uq_, q_lat_, img_lat_, img_cat_, wide_in_, wide_kv_;

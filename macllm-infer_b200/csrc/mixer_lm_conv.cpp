@@ -1,0 +1,170 @@
+// Layers of mixer-built decoders whose mixer reads its normed input plus a short causal convolution of it: windowed attention with
+// shared keys and values beside the delta rule with channel gates, and windowed latent attention with a rotated part.  Both branches
+// of the former share one output matmul over their columns, to which each comes times its constant.  See mixer_lm.h.
+#include "mixer_lm.h"
+
+namespace mk {
+
+// ---------------------------------------------------------------------------- load
+
+void MixerLm::load_conv_input(const SafetensorsFile& f, int l) {
+    const MixerLayerSpec& s = ms_.layers[(size_t)l];
+    Layer& w = lw_[(size_t)l];
+    const int C = ms_.width, taps = ms_.conv_taps;
+    const std::string p = "l" + std::to_string(l) + ".", m = p + "mix.";
+    upload_norm(f, p + "norm1", w.norm1);
+    const std::vector<float> conv = f.values(p + "canon1", {C, taps});
+    std::vector<float> by_tap(conv.size());
+    for (int c = 0; c < C; ++c)
+        for (int j = 0; j < taps; ++j) by_tap[(size_t)j * C + c] = conv[(size_t)c * taps + j];
+    upload_f32(by_tap, w.input_conv);
+
+    std::vector<Part> parts;
+    int at = 0;
+    if (s.kind == MixerKind::Latent) {
+        at = latent_qkv(m, s.latent, w, parts, at);
+        load_latent(f, l);
+        upload_dense(f, parts, at, C, w.in);
+        w.mix_cols = s.latent.heads * s.latent.vdim;
+        upload_dense(f, {{m + "o", C, 0}}, C, w.mix_cols, w.out);
+    } else {
+        const AttentionSpec& a = s.attn;
+        const ChannelDeltaSpec& d = s.channel_delta;
+        const std::string L = m + "left.", R = m + "right.";
+        const int qw = a.heads * a.dim, kw = a.kv_heads * a.dim, n = d.heads * d.dim;
+        auto part = [&](const std::string& name, int rows) {
+            const int here = at;
+            parts.push_back({name, rows, here});
+            at = pad_to(at + rows, 4);
+            return here;
+        };
+        w.c_q = part(L + "q", qw);
+        w.c_k = part(L + "k", kw);
+        w.d_q = part(R + "r", n);
+        w.d_k = part(R + "k", n);
+        w.d_v = part(R + "v", n);
+        w.d_a = part(R + "a", n);
+        w.d_g = part(R + "g", n);
+        w.c_low = part(R + "w1", d.rank);
+        upload_dense(f, parts, at, C, w.in);
+        upload_f32(f.values(L + "q.b", {qw}), w.q_b);
+        upload_f32(f.values(L + "k.b", {kw}), w.k_b);
+        w.geometry = geometry_of(a);
+        w.row_width = geo_[(size_t)w.geometry].row_width;
+        w.rope = rope_table(a.rot);
+        linear_state_key_pad(d.dim);  // refuses head dimensions the recurrence does not take
+        upload_low_rank(f, R, n, d.rank, w);
+        upload_f32(f.values(R + "a.b", {n}), w.a_b);
+        upload_f32(f.values(R + "norm", {n}), w.head_norm);
+        w.mix_cols = pad_to(a.heads * a.vdim, 64);
+        upload_dense(f, {{L + "o", C, 0, 1, 0, a.heads * a.vdim}, {R + "o", C, 0, 1, w.mix_cols, n}}, C, w.mix_cols + n, w.out);
+    }
+    if (s.ff > 0) {
+        upload_norm(f, p + "norm2", w.norm2);
+        upload_dense(f, {{p + "mlp.gate", s.ff, 0, 2}, {p + "mlp.up", s.ff, 1, 2}}, 2 * (int64_t)s.ff, C, w.gate_up);
+        upload_dense(f, {{p + "mlp.down", C, 0}}, C, s.ff, w.down);
+    }
+}
+
+// ---------------------------------------------------------------------------- forward
+
+void MixerLm::run_conv_input(const Tick& t, int run, Pending& pend, const std::vector<LmLane>& lanes) {
+    const int l = runs_[(size_t)run].layer;
+    const MixerLayerSpec& s = ms_.layers[(size_t)l];
+    Layer& w = lw_[(size_t)l];
+    RunState& st = rs_[(size_t)run];
+    const int T = t.T, C = ms_.width;
+    RowUpdateArgs u;
+    u.rows = T;
+    apply_pending(u, pend, true);
+    set_norm(u, w.norm1);
+    u.normed = image(img_h_, w.in.ld);
+    u.taps = ms_.conv_taps;
+    u.conv = w.input_conv.as<float>();
+    u.lanes = state_lanes_;
+    u.token_lane = t.bd.token_lane;
+    u.kept = st.kept.as<float>();
+    prof_begin(KC_ROW_UPDATE, (double)T * C * (8.0 + 4.0 * u.n_add + esz_), 0);
+    launch_row_update(u, stream_);
+    prof_end();
+    ++launches_;
+    const Shares y = matmul(w.in, u.normed, T, y_in_, 0);
+    const RowImage both = image(img_cat_, w.out.ld);
+    if (s.kind == MixerKind::Latent) {
+        LatentPrepArgs p;
+        latent_prep_args(t, run, y, p);
+        prof_begin(KC_LATENT_PREP, (double)T * (p.q_rank + p.kv_rank + p.rot_width) * (4.0 + esz_), 0);
+        launch_latent_prep(p, stream_);
+        prof_end();
+        ++launches_;
+        run_latent(t, run, y, both, lanes);
+    } else {
+        attend(t, run, s.attn, y, lanes);
+        prof_begin(KC_GATES, (double)T * s.attn.heads * s.attn.vdim * (4.0 + esz_), 0);
+        launch_head_gate(attn_.as<float>(), T, s.attn.heads, w.row_width, s.attn.vdim, Shares{}, 0, both.part(0, w.mix_cols), stream_, nullptr, s.attn.gate, s.left_scale);
+        prof_end();
+        ++launches_;
+        run_channel_delta(t, run, y, both.part(w.mix_cols, w.out.ld - w.mix_cols));
+    }
+    pend.n = 1;
+    pend.y[0] = matmul(w.out, both, T, y_a_, 1);
+}
+
+void MixerLm::run_channel_delta(const Tick& t, int run, const Shares& y, const RowImage& out) {
+    const int l = runs_[(size_t)run].layer, T = t.T;
+    const MixerLayerSpec& s = ms_.layers[(size_t)l];
+    const ChannelDeltaSpec& d = s.channel_delta;
+    Layer& w = lw_[(size_t)l];
+    const double n = (double)d.heads * d.dim;
+    ChannelGatesArgs g;
+    g.y = y;
+    g.k_col = w.d_k;
+    g.a_col = w.d_a;
+    g.low_col = w.c_low;
+    g.rows = T;
+    g.heads = d.heads;
+    g.dim = d.dim;
+    g.rank = d.rank;
+    g.w2t = w.w2t.as<float>();
+    g.w0 = w.w0.as<float>();
+    g.a_bias = w.a_b.as<float>();
+    g.decay = decay_.as<float>();
+    g.removal = removal_.as<float>();
+    prof_begin(KC_CHANNEL_GATES, T * (4.0 * n + d.rank) * 4.0 + n * d.rank * 4.0, 2.0 * T * n * d.rank);
+    launch_channel_gates(g, stream_);
+    prof_end();
+    ChannelDeltaArgs a;
+    a.common.lanes = state_lanes_;
+    a.common.state = rs_[(size_t)run].state.as<float>();
+    a.common.heads = d.heads;
+    a.common.dim = a.common.vdim = d.dim;
+    a.common.out = raw_.as<float>();
+    a.common.gate_sigmoid = 1;
+    a.common.out_scale = s.right_scale;
+    a.common.norm_w = w.head_norm.as<float>();
+    a.common.norm_per_head = 1;
+    a.common.eps = ms_.eps;
+    a.common.gate = y;
+    a.common.gate_col = w.d_g;
+    a.y = y;
+    a.r_col = w.d_q;
+    a.k_col = w.d_k;
+    a.v_col = w.d_v;
+    a.decay = g.decay;
+    a.removal = g.removal;
+    const bool finish = short_lanes_ && linear_state_can_finish(d.dim, d.dim);
+    if (finish) a.common.image = out;
+    prof_begin(KC_DELTA_SCAN, 4.0 * T * 6.0 * n + 8.0 * t.B * n * d.dim, 10.0 * T * n * d.dim);
+    launch_channel_delta_scan(a, stream_);
+    prof_end();
+    launches_ += 2;
+    if (!finish) {
+        a.common.image = out;
+        prof_begin(KC_GATES, T * n * (8.0 + esz_), 0);
+        launch_head_norm_gate(a.common, T, stream_);
+        prof_end();
+        ++launches_;
+    }
+}
+
+}  // namespace mk

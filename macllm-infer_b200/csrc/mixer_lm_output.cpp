@@ -48,8 +48,8 @@ void MixerLm::load_output_norm(const SafetensorsFile& f, int l) {
             upload_f32(f.values(m + "q.b", {qw}), w.q_b);
             upload_f32(f.values(m + "k.b", {kw}), w.k_b);
             upload_f32(f.values(m + "v.b", {vw}), w.v_b);
-            upload_f32(f.values(m + "o.b", {C}), w.o_b);
         }
+        if (a.out_bias) upload_f32(f.values(m + "o.b", {C}), w.o_b);
         upload_f32(f.values(m + "q.norm", {a.qk_norm == QkNorm::Whole ? qw : a.dim}), w.q_norm);
         upload_f32(f.values(m + "k.norm", {a.qk_norm == QkNorm::Whole ? kw : a.dim}), w.k_norm);
         if (a.sink) upload_f32(f.values(m + "sink", {a.heads}), w.sink);
@@ -117,7 +117,7 @@ void MixerLm::run_output_norm(const Tick& t, int run, Pending& pend, const std::
         launch_head_gate(attn_.as<float>(), T, s.attn.heads, w.row_width, s.attn.vdim, y, w.c_g, mixed, stream_, nullptr, s.attn.gate);
         prof_end();
         ++launches_;
-        if (s.attn.biases) pend.bias = w.o_b.as<float>();
+        if (s.attn.out_bias) pend.bias = w.o_b.as<float>();
     }
     pend.n = 1;
     pend.y[0] = matmul(w.out, mixed, T, y_a_, 1);

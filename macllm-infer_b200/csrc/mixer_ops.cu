@@ -224,6 +224,117 @@ __global__ void __launch_bounds__(RU_THREADS) row_update_kernel(RowUpdateArgs a)
     for (int m = 0; m < a.n_mix; ++m) zero_tail(a.mixes, (int64_t)m * a.rows + r, a.width);
 }
 
+// Rows of a short convolution: a CTA takes ROWS consecutive rows and the taps - 1 before them (of the first one's lane), updates them
+// all into shared memory behind one barrier for their sums of squares, and then walks its columns.  A thread reads the staged columns
+// it has written itself.
+template <int VEC, int ROWS>
+__global__ void __launch_bounds__(RU_THREADS) conv_update_kernel(RowUpdateArgs a) {
+    extern __shared__ __align__(16) float cu_smem[];   // [ROWS + taps - 1][width], then [ROWS + taps - 1] sums per warp and inverse roots
+    constexpr int BATCH = ROWS >= 4 ? 4 : ROWS;
+    constexpr int WARPS = RU_THREADS / 32;
+    const int hist = a.taps - 1, staged = ROWS + hist, W = a.width;
+    float* red = cu_smem + (int64_t)staged * W;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, step = RU_THREADS * VEC;
+    pdl_trigger();
+    pdl_wait();
+    const int r0 = blockIdx.x * ROWS, r1 = min(a.rows, r0 + ROWS);
+    StateLane sl = a.lanes.at(a.token_lane[r0]);
+    const int lo = max(max(0, sl.first), r0 - hist), n = r1 - lo;
+    for (int i0 = 0; i0 < n; i0 += BATCH) {
+        float ss[BATCH];
+#pragma unroll
+        for (int u = 0; u < BATCH; ++u) ss[u] = 0.f;
+        for (int c = threadIdx.x * VEC; c < W; c += step) {
+            Pack<VEC> v[BATCH];
+#pragma unroll
+            for (int u = 0; u < BATCH; ++u) {
+                if (i0 + u >= n) continue;
+                v[u] = load_pack<VEC>(a.x + (int64_t)(lo + i0 + u) * W + c);
+            }
+            if (a.n_add > 0) {
+#pragma unroll
+                for (int u = 0; u < BATCH; ++u) {
+                    if (i0 + u >= n) continue;
+                    const Pack<VEC> y = branch_pack<VEC>(a, 0, lo + i0 + u, c);
+#pragma unroll
+                    for (int i = 0; i < VEC; ++i) v[u].v[i] = fmaf(a.add_coef, y.v[i], v[u].v[i]);
+                }
+            }
+#pragma unroll
+            for (int u = 0; u < BATCH; ++u) {
+                if (i0 + u >= n) continue;
+                const int row = lo + i0 + u;
+                if (row >= r0 && a.x_out != nullptr) store_pack<VEC>(a.x_out + (int64_t)row * W + c, v[u]);
+                store_pack<VEC>(cu_smem + (int64_t)(i0 + u) * W + c, v[u]);
+#pragma unroll
+                for (int i = 0; i < VEC; ++i) ss[u] = fmaf(v[u].v[i], v[u].v[i], ss[u]);
+            }
+        }
+#pragma unroll
+        for (int u = 0; u < BATCH; ++u) {
+            const float s = warp_sum(ss[u]);
+            if (lane == 0 && i0 + u < n) red[(i0 + u) * WARPS + warp] = s;
+        }
+    }
+    __syncthreads();
+    // every thread needs every row's root: each of the first threads adds one up
+    float* root = red + staged * WARPS;
+    for (int i = threadIdx.x; i < n; i += RU_THREADS) {
+        float s = 0.f;
+#pragma unroll
+        for (int w = 0; w < WARPS; ++w) s += red[i * WARPS + w];
+        root[i] = sqrtf(s / (float)W + a.norm_eps);
+    }
+    __syncthreads();
+    for (int r = r0; r < r1; ++r) {
+        if (r >= sl.first + sl.n) sl = a.lanes.at(a.token_lane[r]);
+        const bool last = r == sl.first + sl.n - 1;
+        for (int c = threadIdx.x * VEC; c < W; c += step) {
+            const Pack<VEC> w = load_pack<VEC>(a.norm_w + c);
+            auto normed = [&](int row) {  // h of a row of the lane, or of one before this tick
+                Pack<VEC> h;
+                if (row >= sl.first) {
+                    h = load_pack<VEC>(cu_smem + (int64_t)(row - lo) * W + c);
+                    const float d = root[row - lo];
+#pragma unroll
+                    for (int i = 0; i < VEC; ++i) h.v[i] = h.v[i] / d * w.v[i];
+                } else if (sl.in >= 0) {
+                    h = load_pack<VEC>(a.kept + ((int64_t)sl.in * hist + hist + row - sl.first) * W + c);
+                } else {
+#pragma unroll
+                    for (int i = 0; i < VEC; ++i) h.v[i] = 0.f;
+                }
+                return h;
+            };
+            Pack<VEC> sum;
+            const Pack<VEC> own = normed(r);
+#pragma unroll
+            for (int i = 0; i < VEC; ++i) sum.v[i] = 0.f;
+#pragma unroll 4
+            for (int j = 0; j < a.taps; ++j) {
+                const Pack<VEC> k = load_pack<VEC>(a.conv + (int64_t)j * W + c);
+                const Pack<VEC> h = j == hist ? own : normed(r - hist + j);
+#pragma unroll
+                for (int i = 0; i < VEC; ++i) sum.v[i] = fmaf(k.v[i], h.v[i], sum.v[i]);
+            }
+#pragma unroll
+            for (int i = 0; i < VEC; ++i) sum.v[i] += own.v[i];
+            put_pack<VEC>(a.normed, r, c, sum);
+            if (last)
+                for (int t = 0; t < hist; ++t) store_pack<VEC>(a.kept + ((int64_t)sl.out * hist + t) * W + c, normed(r - hist + 1 + t));
+        }
+        zero_tail(a.normed, r, W);
+    }
+}
+
+template <int VEC, int ROWS>
+void launch_conv_rows(const RowUpdateArgs& a, cudaStream_t s) {
+    const size_t staged = (size_t)ROWS + a.taps - 1, smem = (staged * a.width + staged * (RU_THREADS / 32 + 1)) * 4;
+    if (smem > (size_t)220 * 1024) throw std::runtime_error("launch_row_update: the model is too wide for its short convolution");
+    ensure_dynamic_smem(reinterpret_cast<const void*>(&conv_update_kernel<VEC, ROWS>), smem);
+    launch_pdl(conv_update_kernel<VEC, ROWS>, dim3((unsigned)((a.rows + ROWS - 1) / ROWS)), dim3(RU_THREADS), smem, s, a);
+}
+
 // ------------------------------------------------------------------------------------------------ WKV decay
 
 constexpr int WD_COLS = 128;       // channels (threads) of a CTA
@@ -280,6 +391,84 @@ void launch_decay_rows(const Shares& low, int low_col, int rows, int rank, int c
     ensure_dynamic_smem(reinterpret_cast<const void*>(&wkv_decay_kernel<ROWS>), smem);
     const dim3 grid((unsigned)((channels + WD_COLS - 1) / WD_COLS), (unsigned)((rows + ROWS - 1) / ROWS));
     launch_pdl(wkv_decay_kernel<ROWS>, grid, dim3(WD_COLS), smem, s, low, low_col, rows, rank, channels, w2t, w0, decay);
+    MK_LAUNCH_CHECK();
+}
+
+// ------------------------------------------------------------------------------------------------ channel gates of the delta rule
+
+// A CTA takes ROWS rows and whole heads of up to CG_COLS channels together, a channel per thread.
+constexpr int CG_COLS = 256;
+
+template <int ROWS>
+__global__ void __launch_bounds__(CG_COLS) channel_gates_kernel(ChannelGatesArgs a, int tile_heads) {
+    extern __shared__ __align__(16) float cg_smem[];
+    const int cols = tile_heads * a.dim, channels = a.heads * a.dim;
+    float* z = cg_smem;                       // [rank][ROWS]
+    float* ks = z + a.rank * ROWS;            // [ROWS][cols]
+    float* inv = ks + ROWS * cols;            // [ROWS][tile_heads]
+    const int r0 = blockIdx.y * ROWS, c = blockIdx.x * cols + threadIdx.x;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
+    const bool live = (int)threadIdx.x < cols && c < channels;
+    pdl_trigger();
+    pdl_wait();
+    for (int i = threadIdx.x; i < a.rank * ROWS; i += blockDim.x) {
+        const int r = i / a.rank, j = i - r * a.rank;
+        z[j * ROWS + r] = r0 + r < a.rows ? tanhf(a.y.at(r0 + r, a.low_col + j)) : 0.f;
+    }
+    float k[ROWS], gate[ROWS];
+#pragma unroll
+    for (int r = 0; r < ROWS; ++r) {
+        const bool there = live && r0 + r < a.rows;
+        k[r] = there ? a.y.at(r0 + r, a.k_col + c) : 0.f;
+        gate[r] = there ? a.y.at(r0 + r, a.a_col + c) : 0.f;
+        if ((int)threadIdx.x < cols) ks[r * cols + threadIdx.x] = k[r];
+    }
+    __syncthreads();
+    for (int i = warp; i < ROWS * tile_heads; i += warps) {
+        const float* row = ks + i / tile_heads * cols + i % tile_heads * a.dim;
+        float ss = 0.f;
+        for (int d = lane; d < a.dim; d += 32) ss = fmaf(row[d], row[d], ss);
+        ss = warp_sum(ss);
+        if (lane == 0) inv[i] = 1.0f / (ss + 1e-6f);
+    }
+    float acc[ROWS];
+#pragma unroll
+    for (int r = 0; r < ROWS; ++r) acc[r] = 0.f;
+    if (live) {
+#pragma unroll 8
+        for (int j = 0; j < a.rank; ++j) {
+            const float w = a.w2t[(int64_t)j * channels + c];
+#pragma unroll
+            for (int r = 0; r < ROWS; r += 4) {
+                const float4 v = *reinterpret_cast<const float4*>(z + j * ROWS + r);
+                acc[r] = fmaf(v.x, w, acc[r]);
+                acc[r + 1] = fmaf(v.y, w, acc[r + 1]);
+                acc[r + 2] = fmaf(v.z, w, acc[r + 2]);
+                acc[r + 3] = fmaf(v.w, w, acc[r + 3]);
+            }
+        }
+    }
+    __syncthreads();
+    if (!live) return;
+    const float w0 = a.w0[c], bias = a.a_bias[c], span = expf(-0.5f);
+    const int head = threadIdx.x / a.dim;
+#pragma unroll
+    for (int r = 0; r < ROWS; ++r) {
+        if (r0 + r >= a.rows) break;
+        const int64_t at = (int64_t)(r0 + r) * channels + c;
+        a.decay[at] = expf(-span * sigmoid_f(acc[r] + w0));
+        a.removal[at] = sigmoid_f(gate[r] + bias) * k[r] * inv[r * tile_heads + head];
+    }
+}
+
+template <int ROWS>
+void launch_channel_rows(const ChannelGatesArgs& a, cudaStream_t s) {
+    const int tile_heads = std::min(a.heads, std::max(1, 128 / a.dim)), cols = tile_heads * a.dim;
+    const size_t smem = ((size_t)a.rank * ROWS + (size_t)ROWS * (cols + tile_heads)) * 4;
+    if (smem > (size_t)220 * 1024) throw std::runtime_error("launch_channel_gates: the low rank is too large");
+    ensure_dynamic_smem(reinterpret_cast<const void*>(&channel_gates_kernel<ROWS>), smem);
+    const dim3 grid((unsigned)((a.heads + tile_heads - 1) / tile_heads), (unsigned)((a.rows + ROWS - 1) / ROWS));
+    launch_pdl(channel_gates_kernel<ROWS>, grid, dim3((unsigned)((cols + 31) / 32 * 32)), smem, s, a, tile_heads);
     MK_LAUNCH_CHECK();
 }
 
@@ -380,12 +569,12 @@ __global__ void __launch_bounds__(DP_WARPS * 32) delta_prep_kernel(DeltaPrepArgs
 // ------------------------------------------------------------------------------------------------ gates
 
 __global__ void __launch_bounds__(256) head_gate_kernel(const float* attn, int heads, int row_width, int vdim, Shares gate, int gate_col, RowImage out,
-                                                        const int32_t* rows, OutputGate kind, int vec_gate) {
+                                                        const int32_t* rows, OutputGate kind, int vec_gate, float scale) {
     extern __shared__ float hg_gate[];
     pdl_trigger();
     pdl_wait();
     const int64_t row = rows != nullptr ? rows[blockIdx.x] : blockIdx.x;
-    for (int h = threadIdx.x; h < heads; h += blockDim.x) hg_gate[h] = kind == OutputGate::Head ? sigmoid_f(gate.at(row, gate_col + h)) : 1.f;
+    for (int h = threadIdx.x; h < heads; h += blockDim.x) hg_gate[h] = scale * (kind == OutputGate::Head ? sigmoid_f(gate.at(row, gate_col + h)) : 1.f);
     __syncthreads();
     const float* src = attn + row * heads * row_width;
     if ((vdim & 3) == 0) {  // out.end() is a multiple of 64, a head's row of 4
@@ -398,7 +587,7 @@ __global__ void __launch_bounds__(256) head_gate_kernel(const float* attn, int h
                     float4 g;
                     if (vec_gate) g = gate.at4(row, gate_col + c);
                     else g = make_float4(gate.at(row, gate_col + c), gate.at(row, gate_col + c + 1), gate.at(row, gate_col + c + 2), gate.at(row, gate_col + c + 3));
-                    v = make_float4(v.x * sigmoid_f(g.x), v.y * sigmoid_f(g.y), v.z * sigmoid_f(g.z), v.w * sigmoid_f(g.w));
+                    v = make_float4(scale * v.x * sigmoid_f(g.x), scale * v.y * sigmoid_f(g.y), scale * v.z * sigmoid_f(g.z), scale * v.w * sigmoid_f(g.w));
                 } else {
                     const float g = hg_gate[h];
                     v = make_float4(v.x * g, v.y * g, v.z * g, v.w * g);
@@ -411,7 +600,7 @@ __global__ void __launch_bounds__(256) head_gate_kernel(const float* attn, int h
     for (int c = threadIdx.x; c < out.end(); c += blockDim.x) {
         const int h = c / vdim;
         float v = 0.f;
-        if (h < heads) v = src[h * row_width + (c - h * vdim)] * (kind == OutputGate::Value ? sigmoid_f(gate.at(row, gate_col + c)) : hg_gate[h]);
+        if (h < heads) v = src[h * row_width + (c - h * vdim)] * (kind == OutputGate::Value ? scale * sigmoid_f(gate.at(row, gate_col + c)) : hg_gate[h]);
         out.put(row, c, v);
     }
 }
@@ -564,7 +753,16 @@ __global__ void __launch_bounds__(LP_THREADS) latent_prep_kernel(LatentPrepArgs 
     zero_tail(a.q_image, row, a.q_rank);
     const int64_t at = a.slots[row] * a.kv_width;
     for (int c = threadIdx.x; c < a.kv_width; c += LP_THREADS) {
-        const float v = c < a.kv_rank ? kv[c] / rk * a.kv_norm[c] : 0.f;
+        float v = c < a.kv_rank ? kv[c] / rk * a.kv_norm[c] : 0.f;
+        const int i = c - a.rot0;
+        if (a.rot_width > 0 && i >= 0 && i < a.rot_width) {
+            v = a.y.at(row, a.rot_col + i);
+            if (i < a.rot_dims) {
+                const int64_t turn = (int64_t)a.positions[row] * (a.rot_dims / 2) + (i >> 1);
+                const float other = a.y.at(row, a.rot_col + (i ^ 1)), cs = a.cos_t[turn], sn = a.sin_t[turn];
+                v = (i & 1) == 0 ? v * cs - other * sn : v * cs + other * sn;
+            }
+        }
         if (a.pool_f16) static_cast<__half*>(a.pool)[at + c] = __float2half_rn(v);
         else static_cast<float*>(a.pool)[at + c] = v;
     }
@@ -634,7 +832,7 @@ __global__ void __launch_bounds__(256) f32_matmul_kernel(const float* __restrict
                 continue;
             }
             const int64_t col = to.column(n);
-            if (col >= 0) to.put(to.row(t) + col, acc[i][j]);
+            if (col >= 0) to.put(to.row(t) + col, to.gate != nullptr ? acc[i][j] * sigmoid_f(to.gate_sum(t, n)) : acc[i][j]);
         }
 }
 
@@ -645,10 +843,22 @@ void launch_row_update(const RowUpdateArgs& a, cudaStream_t s) {
     if (a.n_mix > 0 && (a.x == a.x_out || a.row_index != nullptr)) throw std::runtime_error("launch_row_update: a token shift needs its own output buffer and packed rows");
     if (a.add_bias != nullptr && a.n_add != 1) throw std::runtime_error("launch_row_update: a bias goes with one branch");
     if (a.routed_k > 0 && (a.n_add != 1 || a.add_w[0] == nullptr || a.routed == nullptr)) throw std::runtime_error("launch_row_update: experts' rows go with one normed branch");
+    if (a.taps > 0 && (a.x == nullptr || a.x == a.x_out || a.row_index != nullptr || a.n_mix > 0 || a.n_add > 1 || a.add_w[0] != nullptr || a.norm != NormKind::Rms || a.raw.h != nullptr || a.raw.f != nullptr))
+        throw std::runtime_error("launch_row_update: a short convolution needs its own output buffer, packed rows, one plain branch and an RMS norm");
     if (a.n_add == 2 && (a.add_w[0] == nullptr || a.add_w[1] == nullptr)) throw std::runtime_error("launch_row_update: two branches are both normed");
     bool vec = a.width % 4 == 0;
     for (int b = 0; b < a.n_add; ++b)
         vec = vec && a.add[b].ld % 4 == 0 && a.add[b].stride % 4 == 0 && (reinterpret_cast<uintptr_t>(a.add[b].p) & 15) == 0;
+    if (a.taps > 0) {
+        // wide ticks: as many rows per CTA as leave room for two CTAs
+        auto fits = [&](int rows) { return (size_t)(rows + a.taps - 1) * a.width * 4 <= (size_t)112 * 1024; };
+        if (!vec) launch_conv_rows<1, 1>(a, s);
+        else if (a.rows > 512 && fits(8)) launch_conv_rows<4, 8>(a, s);
+        else if (a.rows > 256 && fits(4)) launch_conv_rows<4, 4>(a, s);
+        else launch_conv_rows<4, 1>(a, s);
+        MK_LAUNCH_CHECK();
+        return;
+    }
     const size_t smem = (size_t)a.width * 4 * (1 + (a.n_mix > 0 ? 1 : 0) + (a.n_add == 2 ? 1 : 0));
     if (smem > (size_t)200 * 1024) throw std::runtime_error("launch_row_update: the model is too wide");
     if (vec) {
@@ -667,6 +877,13 @@ void launch_wkv_decay(const Shares& low, int low_col, int rows, int rank, int ch
     else launch_decay_rows<8>(low, low_col, rows, rank, channels, w2t, w0, decay, s);
 }
 
+void launch_channel_gates(const ChannelGatesArgs& a, cudaStream_t s) {
+    if (a.rows <= 0) return;
+    if (a.dim > CG_COLS) throw std::runtime_error("launch_channel_gates: head dimensions above 256 are not supported");
+    if (a.rows > 256) launch_channel_rows<16>(a, s);
+    else launch_channel_rows<4>(a, s);
+}
+
 void launch_delta_prep(const DeltaPrepArgs& a, cudaStream_t s) {
     if (a.rows <= 0) return;
     if (a.dim > DP_MAX_DIM || a.vdim > DP_MAX_DIM) throw std::runtime_error("launch_delta_prep: head dimensions above 256 are not supported");
@@ -680,10 +897,10 @@ void launch_delta_prep(const DeltaPrepArgs& a, cudaStream_t s) {
 }
 
 void launch_head_gate(const float* attn, int rows, int heads, int row_width, int vdim, const Shares& gate, int gate_col, const RowImage& out,
-                      cudaStream_t s, const int32_t* row_list, OutputGate kind) {
+                      cudaStream_t s, const int32_t* row_list, OutputGate kind, float scale) {
     if (rows <= 0) return;
     const int vec_gate = gate_col % 4 == 0 && gate.ld % 4 == 0 && gate.stride % 4 == 0 && (reinterpret_cast<uintptr_t>(gate.p) & 15) == 0 ? 1 : 0;
-    launch_pdl(head_gate_kernel, dim3((unsigned)rows), dim3(256), (size_t)heads * 4, s, attn, heads, row_width, vdim, gate, gate_col, out, row_list, kind, vec_gate);
+    launch_pdl(head_gate_kernel, dim3((unsigned)rows), dim3(256), (size_t)heads * 4, s, attn, heads, row_width, vdim, gate, gate_col, out, row_list, kind, vec_gate, scale);
     MK_LAUNCH_CHECK();
 }
 

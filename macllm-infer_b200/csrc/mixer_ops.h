@@ -1,6 +1,6 @@
-// The steps between the matmuls of mixer-built decoders: residual update with norm and token shift, the decay of WKV time
-// mixing, the short convolution and unit norms of the gated delta rule, output gates, the per-layer token input - and the
-// 32-bit matmul for models computed in f32 throughout.
+// The steps between the matmuls of mixer-built decoders: residual update with norm and token shift or short convolution, the decay
+// of WKV time mixing, the short convolution and unit norms of the gated delta rule, the channel gates of the other delta rule,
+// output gates, the per-layer token input - and the 32-bit matmul for models computed in f32 throughout.
 #pragma once
 #include "mixer_spec.h"
 #include "device_util.h"
@@ -44,11 +44,31 @@ struct RowUpdateArgs {
     StateLanes lanes;
     const int32_t* token_lane = nullptr;
     float* kept = nullptr;      // [slot halves][width]
+    // taps > 0:  normed <- h + sum_j conv[j] h of the row taps - 1 - j before (zeros before the sequence's start), the rows' norm
+    // recomputed like the token shift's; `kept` then holds the last taps - 1 rows, [slot halves][taps - 1][width].  At most one
+    // un-normed branch; an RMS norm.
+    int taps = 0;
+    const float* conv = nullptr;  // [taps][width]
 };
 void launch_row_update(const RowUpdateArgs& a, cudaStream_t s);
 
 // decay[t][c] = exp(-exp(sum_j tanh(low[t][j]) w2[c][j] + w0[c])), everything in f32.  w2t is w2 transposed, [rank][channels].
 void launch_wkv_decay(const Shares& low, int low_col, int rows, int rank, int channels, const float* w2t, const float* w0, float* decay, cudaStream_t s);
+
+// What the delta rule with channel gates needs beside its projections, everything in f32, per row and key channel c of a head:
+//   decay   = exp(-exp(-1/2) sigmoid(sum_j tanh(y[low_col + j]) w2[c][j] + w0[c]))
+//   removal = sigmoid(y[a_col + c] + a_bias[c]) k[c] / (sum of the head's k^2 + 1e-6),  k = y[k_col + c]
+struct ChannelGatesArgs {
+    Shares y;
+    int k_col = 0, a_col = 0, low_col = 0;
+    int rows = 0, heads = 0, dim = 0, rank = 0;
+    const float* w2t = nullptr;     // w2 transposed, [rank][heads * dim]
+    const float* w0 = nullptr;      // [heads * dim]
+    const float* a_bias = nullptr;  // [heads * dim]
+    float* decay = nullptr;         // [rows][heads * dim]
+    float* removal = nullptr;
+};
+void launch_channel_gates(const ChannelGatesArgs& a, cudaStream_t s);
 
 // The gated delta rule's inputs from the raw projections y: a causal convolution of `taps` taps per channel over q | k | v and
 // silu, unit norm per head of q and k (q also times dim^-1/2), beta = sigmoid(b), decay = exp(softplus(a + dt_bias) * log_decay).
@@ -68,9 +88,9 @@ struct DeltaPrepArgs {
 void launch_delta_prep(const DeltaPrepArgs& a, cudaStream_t s);
 
 // out[t][h * vdim + i] = attn[t][h * row_width + i] * sigmoid(gate[t][gate_col + h]), t = row_list[0 .. rows) or 0 .. rows - 1
-// (OutputGate::Value: sigmoid(gate[t][gate_col + h * vdim + i]); None: no factor)
+// (OutputGate::Value: sigmoid(gate[t][gate_col + h * vdim + i]); None: no factor), all of it times `scale`
 void launch_head_gate(const float* attn, int rows, int heads, int row_width, int vdim, const Shares& gate, int gate_col, const RowImage& out,
-                      cudaStream_t s, const int32_t* row_list = nullptr, OutputGate kind = OutputGate::Head);
+                      cudaStream_t s, const int32_t* row_list = nullptr, OutputGate kind = OutputGate::Head, float scale = 1.f);
 
 // out[t][j] = gelu_tanh(z[t][j]) * table[ids[t]][slice + j], j < dim; table [vocab][table_ld] as bfloat16 bits (or f32)
 void launch_side_gate(const Shares& z, int rows, int dim, const uint32_t* ids, const void* table, int table_f32, int64_t table_ld, int slice,
@@ -107,7 +127,8 @@ struct EmbedNormArgs {
 void launch_embed_norm(const EmbedNormArgs& a, cudaStream_t s);
 
 // What a row's projections need before the next matmuls, one CTA per (row, part):
-//   part 1 (q_rank > 0): the query latent RMS-normed into q_image, the key/value latent RMS-normed into its page
+//   part 1 (q_rank > 0): the query latent RMS-normed into q_image, the key/value latent RMS-normed into its page; behind it, at
+//                        column rot0, the shared key part of rot_width columns, whose first rot_dims turn in adjacent pairs
 //   part 2 (ff > 0):     poly = a N(z) + b N(z^2) + c N(z^3) + e over z = y[ff_col ..] + ff_bias, N = division by the row's root
 //                        mean square
 struct LatentPrepArgs {
@@ -122,6 +143,9 @@ struct LatentPrepArgs {
     const int64_t* slots = nullptr;
     void* pool = nullptr;                       // [blocks * block_tokens][kv_width]
     int pool_f16 = 1;
+    int rot_col = 0, rot0 = 0, rot_width = 0, rot_dims = 0;
+    const float *cos_t = nullptr, *sin_t = nullptr;  // [positions][rot_dims / 2]
+    const int32_t* positions = nullptr;
     int ff_col = 0, ff = 0;
     const float* ff_bias = nullptr;
     const float* poly = nullptr;                // [4]

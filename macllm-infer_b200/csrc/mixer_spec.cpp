@@ -49,6 +49,13 @@ void check_groups(const Json& where, int heads, int kv_heads) {
     if (heads % kv_heads != 0) throw std::runtime_error(where.where() + ": heads must be a multiple of kv_heads");
 }
 
+// A size that only a tensor's shape gives.
+int matrix_rows(const SafetensorsFile& f, const std::string& name) {
+    const StTensor* t = f.find(name);
+    if (t == nullptr || t->shape.size() != 2) throw std::runtime_error("tensor `" + name + "` must be a matrix");
+    return (int)t->shape[0];
+}
+
 // Width of a layer's feed-forward, 0: none.
 int read_dense_ff(const Json& layer) {
     const Json* mlp = layer.find("mlp");
@@ -80,10 +87,7 @@ MixerSpec read_sizilorn(const Json& c, const SafetensorsFile& f) {
             l.kind = MixerKind::Wkv;
             l.wkv.heads = size_of(m.at("heads"));
             l.wkv.dim = size_of(m.at("dim"));
-            const std::string w1 = "l" + std::to_string(i) + ".mix.w1";
-            const StTensor* t = f.find(w1);
-            if (t == nullptr || t->shape.size() != 2) throw std::runtime_error("tensor `" + w1 + "` must be a matrix");
-            l.wkv.rank = (int)t->shape[0];
+            l.wkv.rank = matrix_rows(f, "l" + std::to_string(i) + ".mix.w1");
         } else if (type == "parallel") {
             l.kind = MixerKind::Parallel;
             const Json& a = m.at("left");
@@ -227,7 +231,7 @@ MixerSpec read_tevanex(const Json& c, const SafetensorsFile&) {
             a.vdim = size_of(m.at("vdim"));
             a.scale = number_of(m.at("scale"));
             a.chunk = size_of(m.at("mask").at("size"), 1, 1 << 30);
-            a.biases = true;
+            a.biases = a.out_bias = true;
             a.qk_norm = QkNorm::Whole;
             a.sink = !capped;
             a.gate = capped ? OutputGate::Value : OutputGate::None;
@@ -267,6 +271,70 @@ MixerSpec read_tevanex(const Json& c, const SafetensorsFile&) {
 
 const RegisterMixerArchitecture register_tevanex("Tevanex", read_tevanex);
 
+// Mamivik: a short convolution in front of every mixer, windowed attention with shared keys and values beside the delta rule with
+// channel gates, and windowed latent attention with a rotated part, a sink and a gate per value.
+MixerSpec read_mamivik(const Json& c, const SafetensorsFile& f) {
+    MixerSpec s;
+    s.arch = "Mamivik";
+    s.vocab = size_of(c.at("vocab"));
+    s.width = size_of(c.at("width"));
+    s.norm = NormKind::Rms;
+    s.one_number_norms = true;
+    s.ff_kind = FfKind::GatedGelu;
+    s.eps = number_of(c.at("norm").at("eps"));
+    if (!(s.eps >= 0.f)) throw std::runtime_error("config norm.eps must not be negative");
+    s.conv_taps = size_of(c.at("canon").at("taps"), 1, 64);
+    const auto& layers = c.at("layers").items();
+    if (layers.empty()) throw std::runtime_error("config lists no layers");
+    for (const Json& j : layers) {
+        const Json& m = j.at("mixer");
+        const std::string type = j.at("type").str();
+        MixerLayerSpec l;
+        if (type == "parallel") {
+            l.kind = MixerKind::ScaledParallel;
+            l.left_scale = number_of(m.at("left_scale"));
+            l.right_scale = number_of(m.at("right_scale"));
+            const Json &a = m.at("left"), &d = m.at("right");
+            l.attn.heads = size_of(a.at("heads"));
+            l.attn.kv_heads = size_of(a.at("kv_heads"));
+            check_groups(a, l.attn.heads, l.attn.kv_heads);
+            l.attn.dim = size_of(a.at("dim"));
+            l.attn.vdim = size_of(a.at("vdim"));
+            if (l.attn.vdim != l.attn.dim) throw std::runtime_error(a.where() + ".vdim must be dim, the values being the keys");
+            l.attn.scale = number_of(a.at("scale"));
+            l.attn.window = size_of(a.at("mask").at("size"), 1, 1 << 30);
+            l.attn.biases = l.attn.keys_are_values = true;
+            l.attn.qk_norm = QkNorm::None;
+            l.attn.gate = OutputGate::None;
+            l.attn.rot = read_rotary(a, l.attn.dim, RotaryScaling::None, false);
+            l.channel_delta.heads = size_of(d.at("heads"));
+            l.channel_delta.dim = size_of(d.at("dim"));
+            l.channel_delta.rank = matrix_rows(f, "l" + std::to_string(s.layers.size()) + ".mix.right.w1");
+        } else if (type == "latent_attention") {
+            l.kind = MixerKind::Latent;
+            LatentSpec& a = l.latent;
+            a.heads = size_of(m.at("heads"));
+            a.dim = size_of(m.at("dim"));
+            a.vdim = size_of(m.at("vdim"));
+            a.q_rank = size_of(m.at("q_rank"));
+            a.kv_rank = size_of(m.at("kv_rank"));
+            a.scale = number_of(m.at("scale"));
+            a.rot_dim = size_of(m.at("rot_dim"));
+            a.rot = read_rotary(m, a.rot_dim, RotaryScaling::Yarn, false);
+            a.window = size_of(m.at("mask").at("size"), 1, 1 << 30);
+            a.sink = true;
+            a.gate = OutputGate::Value;
+        } else {
+            throw std::runtime_error(j.where() + ".type `" + type + "` is not a known mixer");
+        }
+        l.ff = read_dense_ff(j);
+        s.layers.push_back(l);
+    }
+    return s;
+}
+
+const RegisterMixerArchitecture register_mamivik("Mamivik", read_mamivik);
+
 }  // namespace
 
 RegisterMixerArchitecture::RegisterMixerArchitecture(const std::string& name, MixerSpecReader reader) { readers()[name] = std::move(reader); }
@@ -291,7 +359,8 @@ std::vector<std::pair<std::string, std::vector<int64_t>>> mixer_tensors(const Mi
     const int64_t C = s.width, V = s.vocab;
     auto add = [&](const std::string& name, std::vector<int64_t> shape) { out.emplace_back(name, std::move(shape)); };
     auto norm = [&](const std::string& name) {
-        add(name, {C});
+        if (s.one_number_norms) add(name, {});
+        else add(name, {C});
         if (s.norm == NormKind::DynTanh) {
             add(name + ".b", {C});
             add(name + ".alpha", {});
@@ -321,15 +390,16 @@ std::vector<std::pair<std::string, std::vector<int64_t>>> mixer_tensors(const Mi
             add(m + "o", {C, n});
         } else if (l.kind == MixerKind::Latent) {
             const LatentSpec& a = l.latent;
-            const int64_t qw = (int64_t)a.heads * a.dim, vw = (int64_t)a.heads * a.vdim;
+            const int64_t kw = (int64_t)a.heads * a.dim, vw = (int64_t)a.heads * a.vdim;
             add(m + "dq", {a.q_rank, C});
             add(m + "dq.norm", {a.q_rank});
-            add(m + "uq", {qw, a.q_rank});
-            add(m + "dkv", {a.kv_rank, C});
+            add(m + "uq", {(int64_t)a.heads * (a.dim + a.rot_dim), a.q_rank});
+            add(m + "dkv", {a.kv_rank + a.rot_dim, C});
             add(m + "dkv.norm", {a.kv_rank});
-            add(m + "uk", {qw, a.kv_rank});
+            add(m + "uk", {kw, a.kv_rank});
             add(m + "uv", {vw, a.kv_rank});
-            add(m + "g", {a.heads, C});
+            if (a.sink) add(m + "sink", {a.heads});
+            if (a.gate != OutputGate::None) add(m + "g", {a.gate == OutputGate::Value ? vw : (int64_t)a.heads, C});
             add(m + "o", {C, vw});
         } else if (l.kind == MixerKind::MinGru) {
             const int64_t n = l.gru.width;
@@ -362,11 +432,28 @@ std::vector<std::pair<std::string, std::vector<int64_t>>> mixer_tensors(const Mi
             linear("q", qw, C);
             linear("k", kw, C);
             linear("v", vw, C);
-            linear("o", C, ow);
+            add(m + "o", {C, ow});
+            if (a.out_bias) add(m + "o.b", {C});
             add(m + "q.norm", {a.qk_norm == QkNorm::Whole ? qw : a.dim});
             add(m + "k.norm", {a.qk_norm == QkNorm::Whole ? kw : a.dim});
             if (a.sink) add(m + "sink", {a.heads});
             if (a.gate != OutputGate::None) add(m + "g", {a.gate == OutputGate::Value ? ow : (int64_t)a.heads, C});
+        } else if (l.kind == MixerKind::ScaledParallel) {
+            const AttentionSpec& a = l.attn;
+            const ChannelDeltaSpec& d = l.channel_delta;
+            const int64_t qw = (int64_t)a.heads * a.dim, kw = (int64_t)a.kv_heads * a.dim, n = (int64_t)d.heads * d.dim;
+            add(m + "left.q", {qw, C});
+            add(m + "left.q.b", {qw});
+            add(m + "left.k", {kw, C});
+            add(m + "left.k.b", {kw});
+            add(m + "left.o", {C, (int64_t)a.heads * a.vdim});
+            for (const char* x : {"r", "k", "v", "g", "a"}) add(m + "right." + x, {n, C});
+            add(m + "right.a.b", {n});
+            add(m + "right.w1", {d.rank, C});
+            add(m + "right.w2", {n, d.rank});
+            add(m + "right.w0", {n});
+            add(m + "right.norm", {n});
+            add(m + "right.o", {C, n});
         } else {
             const AttentionSpec& a = l.attn;
             const DeltaSpec& d = l.delta;
@@ -394,6 +481,7 @@ std::vector<std::pair<std::string, std::vector<int64_t>>> mixer_tensors(const Mi
             add(m + "right.out", {C});
         }
         if (s.side_by_side()) add(p + "shift", {C});
+        if (s.conv_taps > 0) add(p + "canon1", {C, s.conv_taps});
         if (l.ff > 0 && s.ff_kind == FfKind::Moe) {
             norm(p + "norm2");
             auto expert = [&](const std::string& name, int64_t ff) {
@@ -409,7 +497,7 @@ std::vector<std::pair<std::string, std::vector<int64_t>>> mixer_tensors(const Mi
             }
         } else if (l.ff > 0) {
             if (!s.side_by_side()) norm(p + "norm2");
-            if (s.ff_kind == FfKind::Gated) add(p + "mlp.gate", {l.ff, C});
+            if (s.ff_kind != FfKind::Poly) add(p + "mlp.gate", {l.ff, C});
             add(p + "mlp.up", {l.ff, C});
             add(p + "mlp.down", {C, l.ff});
             if (s.ff_kind == FfKind::Poly) {

@@ -37,7 +37,7 @@ std::vector<double> rotary_frequencies(const RotarySpec& r);
 double rotary_amplitude(const RotarySpec& r);
 
 enum class OutputGate { None, Head, Value };     // a sigmoid gate per head, or per value, on what attention gives
-enum class QkNorm { Head, Whole };               // RMS norm of queries and keys per head, or over all heads at once
+enum class QkNorm { None, Head, Whole };         // RMS norm of queries and keys per head, or over all heads at once
 
 // Grouped-query attention; query / key RMS norm before the rotation.
 struct AttentionSpec {
@@ -45,8 +45,11 @@ struct AttentionSpec {
     float scale = 1.f;
     float softcap = 0.f;      // scores pass through softcap * tanh(. / softcap); 0: as they are
     int chunk = 0;            // a position sees the keys of its own chunk only, chunks counted from position 0; 0: all before it
+    int window = 0;           // a position sees itself and the window - 1 keys before it; 0: all before it
     bool sink = false;        // one learned term per head in the softmax denominator
-    bool biases = false;      // of the query, key, value and output projections
+    bool biases = false;      // of the query, key and value projections
+    bool out_bias = false;    // of the output projection
+    bool keys_are_values = false;  // no value projection: the values are the keys before their rotation
     QkNorm qk_norm = QkNorm::Head;
     OutputGate gate = OutputGate::Head;
     RotarySpec rot;
@@ -62,11 +65,22 @@ struct WkvSpec {
     int heads = 0, dim = 0, rank = 0;  // rank of the decay's low-rank projection
 };
 
+// The delta rule with a decay and a removal rate per key channel (see ChannelDeltaArgs); square heads.
+struct ChannelDeltaSpec {
+    int heads = 0, dim = 0, rank = 0;  // rank of the decay's low-rank projection
+};
+
 // Attention whose keys and values are two projections of one cached vector of `kv_rank` values per token; queries come from a
-// latent of `q_rank` values.  No positions; a sigmoid gate per head on the output.
+// latent of `q_rank` values.  With rot_dim > 0 queries have that many dimensions more per head, and a token has one more key part
+// of that width, shared by the heads and cached beside the vector; these dimensions turn with the position, the others do not.
 struct LatentSpec {
     int heads = 0, dim = 0, vdim = 0, q_rank = 0, kv_rank = 0;
     float scale = 1.f;
+    int rot_dim = 0;
+    RotarySpec rot;                      // of the rot_dim dimensions
+    int window = 0;                      // as AttentionSpec's
+    bool sink = false;
+    OutputGate gate = OutputGate::Head;
 };
 
 // Element-wise gated recurrence over `width` channels whose gates read the current token only.
@@ -88,9 +102,12 @@ struct MoeSpec {
     float limit = 0.f, shared_limit = 0.f;
 };
 
-enum class MixerKind { Wkv, Parallel, Latent, MinGru, Mlstm, Attention };  // Parallel: attention and the gated delta rule side by side
+// Parallel: attention and the gated delta rule side by side.  ScaledParallel: attention and the delta rule with channel gates side by
+// side, each branch times a constant.
+enum class MixerKind { Wkv, Parallel, Latent, MinGru, Mlstm, Attention, ScaledParallel };
 
-enum class FfKind { Gated, Poly, Moe };  // silu(gate) * up; a cubic of up, every power over its own root mean square; experts
+// silu(gate) * up; gelu(gate) * up; a cubic of up, every power over its own root mean square; experts
+enum class FfKind { Gated, GatedGelu, Poly, Moe };
 
 // Where a layer's norms sit.  Input: in front of the mixer and of the feed-forward.  Shared: one in front of both, which read the
 // same row side by side; the mixer's input is mixed with the previous token's normed row (token shift).  Output: on what the mixer
@@ -105,6 +122,8 @@ struct MixerLayerSpec {
     LatentSpec latent;
     MinGruSpec gru;
     MlstmSpec mlstm;
+    ChannelDeltaSpec channel_delta;
+    float left_scale = 1.f, right_scale = 1.f;  // ScaledParallel
     int ff = 0;  // width of the feed-forward (of one expert), 0: the layer has none
     MoeSpec moe;
     int weights_of = -1;  // >= 0: the layer has no tensors and runs that layer's, with a cache and a state of its own
@@ -130,6 +149,8 @@ struct MixerSpec {
     FfKind ff_kind = FfKind::Gated;
     NormPlace norm_place = NormPlace::Input;
     bool side_by_side() const { return norm_place == NormPlace::Shared; }
+    bool one_number_norms = false;    // a norm has one weight for all channels
+    int conv_taps = 0;                // > 0: the mixers read h + conv(h), a causal convolution per channel behind norm1 (NormPlace::Input)
     bool sinusoid_positions = false;  // added to the embedding, which a norm then follows
     float embedding_scale = 1.f;
     float residual_mult = 1.f;        // of every sublayer's output (NormPlace::Output)

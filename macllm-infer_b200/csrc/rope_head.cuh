@@ -1,4 +1,4 @@
-// One head vector of one token on its way from the projection to the attention: summation of split-K shares, the
+// One head vector of one token on its way from the projection to the attention: summation of split-K shares, an optional bias, the
 // optional per-head RMSNorm (SelfAttention::project_packed_qkv, src/decoder.rs:1137-1154, applied BEFORE the rotation)
 // and the half-split rotation (RotaryEmbedding::apply, src/decoder.rs:203-257).  Shared by the stand-alone
 // RoPE + KV-scatter kernel and by the decode attention kernel that prepares its own rows, so that both produce the
@@ -36,6 +36,11 @@ __device__ __forceinline__ void rope_head_prepare(const RopeKvArgs& a, int kind,
             for (int sp = 1; sp < n_parts; ++sp) v += src[(int64_t)sp * part_stride + i];
             x[i] = v;
         }
+    }
+    const float* bias = kind == 0 ? a.q_bias : (kind == 1 ? a.k_bias : a.v_bias);
+    if (bias != nullptr) {
+        __syncwarp();
+        for (int i = lane; i < d; i += 32) x[i] += bias[hh * d + i];
     }
     for (int i = d + lane; i < rope_row_width(a); i += 32) x[i] = 0.f;
     __syncwarp();
