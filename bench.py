@@ -27,7 +27,7 @@ has no exchange step for them); the sparse-MoE workload runs expert parallelism 
 serves its own requests and each MoE layer exchanges the routed rows (`config.ep`; `--ep off` for replicas).  The
 reported time is the max over ranks.  `--http-clients N` adds a step through the `/completion` endpoint (`http` key),
 `--microbench` prints the Q4_K matmul GB/s of the decode shapes instead, `--mixer` the prefill and decode throughput of
-a mixer-built decoder design (`--mixer sizilorn`, the default, `--mixer kunonex` or `--mixer tevanex`; layers at real-model sizes, random weights)
+a mixer-built decoder design (`--mixer sizilorn`, the default, `--mixer kunonex`, `--mixer tevanex` or `--mixer mamivik`; layers at real-model sizes, random weights)
 beside the closest GGUF family of equal size.
 """
 from __future__ import annotations
@@ -642,7 +642,7 @@ def main():
                          "resident; N > 1: expert parallelism over the same ranks)")
     ap.add_argument("--no-profiled-step", action="store_true", help="skip the extra step that times every launch")
     ap.add_argument("--microbench", action="store_true", help="Q4_K matmul GB/s on the decode shapes instead of the workload")
-    ap.add_argument("--mixer", nargs="?", const="sizilorn", choices=["sizilorn", "kunonex", "tevanex"],
+    ap.add_argument("--mixer", nargs="?", const="sizilorn", choices=["sizilorn", "kunonex", "tevanex", "mamivik"],
                     help="prefill / decode throughput of a mixer-built decoder design beside the closest GGUF family instead of the workload")
     args = ap.parse_args()
 

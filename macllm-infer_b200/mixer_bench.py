@@ -102,6 +102,49 @@ EXPERT_SHAPES = [
 ]
 
 
+@dataclass
+class ConvShape:
+    """Groups of four layers behind a short convolution: attention beside the delta rule with channel gates, twice, latent attention with
+    a rotated part, and the first kind again."""
+    name: str
+    width: int
+    groups: int
+    heads: int
+    kv_heads: int
+    dim: int
+    delta_heads: int
+    delta_dim: int
+    rank: int
+    q_rank: int
+    kv_rank: int
+    rot_dim: int
+    window: int
+    ff: int
+    vocab: int = 32000
+
+    @property
+    def runs(self) -> int:
+        return 4 * self.groups
+
+
+CONV_SHAPES = [
+    ConvShape("w2048", 2048, 2, 16, 4, 128, 16, 128, 64, 1024, 512, 64, 8192, 8192),
+    ConvShape("w4096", 4096, 1, 32, 8, 128, 32, 128, 64, 1536, 512, 64, 8192, 12288),
+]
+
+
+def conv_layers(s) -> list:
+    mlp = {"kind": "dense", "ff": s.ff}
+    par = {"type": "parallel", "mlp": mlp, "mixer": {
+        "left": {"heads": s.heads, "kv_heads": s.kv_heads, "dim": s.dim, "vdim": s.dim, "scale": s.dim ** -0.5, "mask": {"size": s.window},
+                 "rot": {"base": 500000.0, "dims": s.dim // 4}},
+        "right": {"heads": s.delta_heads, "dim": s.delta_dim}, "left_scale": 0.7, "right_scale": 0.7}}
+    lat = {"type": "latent_attention", "mlp": mlp, "mixer": {
+        "heads": s.heads, "dim": s.dim, "vdim": s.dim, "q_rank": s.q_rank, "kv_rank": s.kv_rank, "rot_dim": s.rot_dim, "scale": (s.dim + s.rot_dim) ** -0.5,
+        "mask": {"size": s.window}, "rot": {"base": 10000.0, "dims": s.rot_dim, "scaling": {"factor": 16.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}}
+    return [par, par, lat, par] * s.groups
+
+
 def expert_layers(s) -> list:
     mlp = {"kind": "moe", "router": {"experts": s.experts, "top": s.top}, "expert": {"ff": s.ff, "limit": 7.0}, "shared": {"ff": s.ff, "limit": 7.0}}
     attn = {"heads": s.heads, "kv_heads": s.kv_heads, "dim": s.dim, "vdim": s.dim, "scale": s.dim ** -0.5, "mask": {"size": s.chunk}}
@@ -113,6 +156,8 @@ def expert_layers(s) -> list:
 
 
 def config_of(s) -> dict:
+    if isinstance(s, ConvShape):
+        return {"architecture": "Mamivik", "vocab": s.vocab, "width": s.width, "norm": {"eps": 1e-6}, "canon": {"taps": 4}, "layers": conv_layers(s)}
     if isinstance(s, ExpertShape):
         return {"architecture": "Tevanex", "vocab": s.vocab, "width": s.width, "norm": {"eps": 1e-6}, "embedding": {"scale": 1.0}, "residual_mult": 0.5,
                 "logit_scale": 1.0, "logit_softcap": 30.0, "layers": expert_layers(s)}
@@ -151,6 +196,44 @@ def tensor_shapes(s) -> dict[str, tuple]:
             vec(name + ".alpha", mean=0.7, dev=0.0)
 
     out["embed"] = ((V, C), 0.0, 1.0)
+    if isinstance(s, ConvShape):
+        for i, layer in enumerate(conv_layers(s)):
+            p, m = f"l{i}.", layer["mixer"]
+            vec(p + "norm1")
+            vec(p + "norm2")
+            out[p + "canon1"] = ((C, 4), 0.0, 0.3)
+            if layer["type"] == "parallel":
+                L, R, n = p + "mix.left.", p + "mix.right.", s.delta_heads * s.delta_dim
+                for x, rows in (("q", s.heads * s.dim), ("k", s.kv_heads * s.dim)):
+                    mat(L + x, rows, C)
+                    vec(L + x + ".b", rows, mean=0.0)
+                mat(L + "o", C, s.heads * s.dim)
+                for x in "rkvga":
+                    mat(R + x, n, C)
+                vec(R + "a.b", n, mean=0.0)
+                mat(R + "w1", s.rank, C)
+                mat(R + "w2", n, s.rank)
+                vec(R + "w0", n, mean=-3.0, dev=1.0)
+                vec(R + "norm", n)
+                mat(R + "o", C, n)
+            else:
+                n = s.heads * s.dim
+                mat(p + "mix.dq", s.q_rank, C)
+                vec(p + "mix.dq.norm", s.q_rank)
+                mat(p + "mix.uq", n + s.heads * s.rot_dim, s.q_rank)
+                mat(p + "mix.dkv", s.kv_rank + s.rot_dim, C)
+                vec(p + "mix.dkv.norm", s.kv_rank)
+                mat(p + "mix.uk", n, s.kv_rank)
+                mat(p + "mix.uv", n, s.kv_rank)
+                vec(p + "mix.sink", s.heads)
+                mat(p + "mix.g", n, C)
+                mat(p + "mix.o", C, n)
+            mat(p + "mlp.gate", s.ff, C)
+            mat(p + "mlp.up", s.ff, C)
+            mat(p + "mlp.down", C, s.ff)
+        vec("final.norm")
+        mat("head", V, C)
+        return out
     if isinstance(s, ExpertShape):
         for i, layer in enumerate(expert_layers(s)):
             p, m = f"l{i}.", layer["mixer"]
@@ -292,7 +375,7 @@ def closest_spec(s) -> seed_gguf.SeedSpec:
     if isinstance(s, ExpertShape):
         return seed_gguf.SeedSpec("qwen3moe", s.runs, s.width, s.heads, s.kv_heads, s.dim, 4 * s.ff, s.vocab, context=16384, theta=1e6, eps=1e-6, experts=s.experts,
                                   experts_used=s.top, expert_ffn=s.ff, name=f"closest-{s.name}")
-    layers = s.runs if isinstance(s, BesideShape) else 2 * s.pairs
+    layers = s.runs if isinstance(s, (BesideShape, ConvShape)) else 2 * s.pairs
     return seed_gguf.SeedSpec("qwen3", layers, s.width, s.heads, s.kv_heads, s.dim, s.ff, s.vocab, context=16384, theta=1e6, eps=1e-6,
                               matrix_type=capi.TYPE_BF16, high_type=capi.TYPE_BF16, name=f"closest-{s.name}")
 
@@ -357,7 +440,7 @@ def measure(model, vocab: int, prompt: int, lanes: int, context: int, warmup: in
     return out
 
 
-DESIGNS = {"sizilorn": ("Sizilorn", SHAPES), "kunonex": ("Kunonex", BESIDE_SHAPES), "tevanex": ("Tevanex", EXPERT_SHAPES)}
+DESIGNS = {"sizilorn": ("Sizilorn", SHAPES), "kunonex": ("Kunonex", BESIDE_SHAPES), "tevanex": ("Tevanex", EXPERT_SHAPES), "mamivik": ("Mamivik", CONV_SHAPES)}
 
 
 def run(peaks: dict, warmup: int, steps: int, design="sizilorn", prompt=2048, lanes=64, context=1024) -> list[dict]:

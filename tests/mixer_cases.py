@@ -211,8 +211,87 @@ def kunonex_weights(cfg, seed):
     return w
 
 
+def scaled_parallel(left, right, window, scales=(0.8, 0.5), ff=0, base=500.0, scale=None):
+    """left = (heads, kv_heads, dim, rot dims), right = (heads, dim)."""
+    h, g, d, rd = left
+    return {"type": "parallel", "mlp": {"kind": "dense", "ff": ff} if ff else None,
+            "mixer": {"left": {"heads": h, "kv_heads": g, "dim": d, "vdim": d, "scale": scale or 0.9 / d ** 0.5, "mask": {"size": window},
+                               "rot": {"base": base, "dims": rd}},
+                      "right": {"heads": right[0], "dim": right[1]}, "left_scale": scales[0], "right_scale": scales[1]}}
+
+
+def rotated_latent(heads, dim, vdim, q_rank, kv_rank, rot_dim, window, ff=0, scaling=YARN, base=500.0, scale=None):
+    return {"type": "latent_attention", "mlp": {"kind": "dense", "ff": ff} if ff else None,
+            "mixer": {"heads": heads, "dim": dim, "vdim": vdim, "q_rank": q_rank, "kv_rank": kv_rank, "rot_dim": rot_dim,
+                      "scale": scale or 0.9 / (dim + rot_dim) ** 0.5, "mask": {"size": window},
+                      "rot": {"base": base, "dims": rot_dim, "scaling": dict(scaling) if scaling else None}}}
+
+
+def mamivik(layers, width=96, vocab=131, taps=3, eps=3e-5):
+    return {"architecture": "Mamivik", "vocab": vocab, "width": width, "norm": {"eps": eps}, "canon": {"taps": taps}, "layers": layers}
+
+
+def mamivik_weights(cfg, seed, rank):
+    rng = np.random.default_rng(seed)
+    C, V, taps = cfg["width"], cfg["vocab"], cfg["canon"]["taps"]
+    w = {}
+
+    def mat(name, rows, cols, gain=1.0):
+        w[name] = rng.standard_normal((rows, cols)) * gain / np.sqrt(cols)
+
+    def around_one(name, *shape):
+        w[name] = 1.0 + 0.3 * rng.standard_normal(shape)
+
+    w["embed"] = rng.standard_normal((V, C))
+    for i, layer in enumerate(cfg["layers"]):
+        p, m = f"l{i}.", layer["mixer"]
+        around_one(p + "norm1")
+        w[p + "canon1"] = rng.standard_normal((C, taps)) * 0.6 / np.sqrt(taps)
+        if layer["type"] == "parallel":
+            a, L, R = m["left"], p + "mix.left.", p + "mix.right."
+            n = m["right"]["heads"] * m["right"]["dim"]
+            for x, heads in (("q", a["heads"]), ("k", a["kv_heads"])):
+                mat(L + x, heads * a["dim"], C, 1.3)
+                w[L + x + ".b"] = 0.4 * rng.standard_normal(heads * a["dim"])
+            mat(L + "o", C, a["heads"] * a["dim"])
+            for x in "kvga":
+                mat(R + x, n, C)
+            # queries that have something in common with the keys: what the heads give is a sum without much cancellation, from the
+            # first token on
+            w[R + "r"] = 0.8 * w[R + "k"] + 0.6 * rng.standard_normal((n, C)) / np.sqrt(C)
+            w[R + "a.b"] = rng.standard_normal(n)
+            mat(R + "w1", rank, C)
+            mat(R + "w2", n, rank)
+            w[R + "w0"] = rng.uniform(-6.0, 2.0, n)
+            around_one(R + "norm", n)
+            mat(R + "o", C, n)
+        else:
+            H, q_rank, kv_rank = m["heads"], m["q_rank"], m["kv_rank"]
+            mat(p + "mix.dq", q_rank, C)
+            around_one(p + "mix.dq.norm", q_rank)
+            mat(p + "mix.uq", H * (m["dim"] + m["rot_dim"]), q_rank, 1.5)
+            mat(p + "mix.dkv", kv_rank + m["rot_dim"], C)
+            around_one(p + "mix.dkv.norm", kv_rank)
+            mat(p + "mix.uk", H * m["dim"], kv_rank, 1.2)
+            mat(p + "mix.uv", H * m["vdim"], kv_rank)
+            w[p + "mix.sink"] = 1.0 + rng.standard_normal(H)
+            mat(p + "mix.g", H * m["vdim"], C)
+            mat(p + "mix.o", C, H * m["vdim"])
+        if layer["mlp"]:
+            ff = layer["mlp"]["ff"]
+            around_one(p + "norm2")
+            mat(p + "mlp.gate", ff, C)
+            mat(p + "mlp.up", ff, C)
+            mat(p + "mlp.down", C, ff)
+    around_one("final.norm")
+    mat("head", V, C)
+    return w
+
+
 def weights(cfg, seed=0, rank=5):
     """name -> float32 array holding bfloat16 values."""
+    if cfg["architecture"] == "Mamivik":
+        return {k: mixers.bf16(np.asarray(v, np.float32)) for k, v in mamivik_weights(cfg, seed, rank).items()}
     if cfg["architecture"] == "Kunonex":
         return {k: mixers.bf16(np.asarray(v, np.float32)) for k, v in kunonex_weights(cfg, seed).items()}
     if cfg["architecture"] == "Tevanex":

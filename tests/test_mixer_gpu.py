@@ -114,6 +114,39 @@ ALONE_OUTPUT = {
 }
 
 
+ALONE_CONV = {
+    # name: (layer, width, taps, what is silenced, rank)
+    "shared keys and values": (mc.scaled_parallel((4, 2, 64, 32), (1, 8), 20), 96, 4, ("l0.mix.right.o",), 5),
+    "shared keys and values, three heads per key": (mc.scaled_parallel((6, 2, 20, 8), (1, 8), 9), 70, 3, ("l0.mix.right.o",), 5),
+    "shared keys and values, window of one": (mc.scaled_parallel((2, 2, 32, 32), (1, 8), 1), 64, 2, ("l0.mix.right.o",), 5),
+    "shared keys and values, 128, one key head": (mc.scaled_parallel((8, 1, 128, 64), (1, 8), 33), 96, 4, ("l0.mix.right.o",), 5),
+    "shared keys and values, odd head": (mc.scaled_parallel((5, 5, 21, 6), (1, 8), 300), 67, 5, ("l0.mix.right.o",), 5),
+    "shared keys and values, no turning": (mc.scaled_parallel((4, 4, 40, 0), (1, 8), 16), 64, 1, ("l0.mix.right.o",), 5),
+    "channel delta": (mc.scaled_parallel((2, 1, 16, 8), (3, 64), 9), 96, 4, ("l0.mix.left.o",), 16),
+    "channel delta, odd heads": (mc.scaled_parallel((2, 1, 16, 8), (5, 43), 9), 70, 3, ("l0.mix.left.o",), 3),
+    "channel delta, one head": (mc.scaled_parallel((2, 1, 16, 8), (1, 24), 9), 64, 2, ("l0.mix.left.o",), 7),
+    "channel delta 128": (mc.scaled_parallel((2, 1, 16, 8), (2, 128), 9), 128, 4, ("l0.mix.left.o",), 64),
+    "channel delta, wide head, wide rank": (mc.scaled_parallel((2, 1, 16, 8), (2, 136), 9), 96, 1, ("l0.mix.left.o",), 130),
+    "channel delta 256": (mc.scaled_parallel((2, 1, 16, 8), (1, 256), 9), 64, 4, ("l0.mix.left.o",), 4),
+    "channel delta, many small heads": (mc.scaled_parallel((2, 1, 16, 8), (19, 12), 9), 64, 4, ("l0.mix.left.o",), 8),
+    "both scaled branches": (mc.scaled_parallel((4, 2, 40, 16), (4, 24), 20, scales=(-0.7, 1.6)), 100, 4, (), 5),
+    "rotated latents": (mc.rotated_latent(4, 32, 48, 40, 56, 16, 24), 96, 4, (), 5),
+    "rotated latents, odd sizes": (mc.rotated_latent(3, 37, 24, 33, 45, 10, 17), 70, 3, (), 5),
+    "rotated latents, turned part wider": (mc.rotated_latent(5, 12, 100, 12, 64, 60, 300), 96, 2, (), 5),
+    "rotated latents behind 128": (mc.rotated_latent(2, 40, 20, 30, 128, 32, 40), 64, 4, (), 5),
+    "rotated latents, whole extra chunk": (mc.rotated_latent(2, 64, 64, 30, 128, 96, 40), 64, 4, (), 5),
+    "rotated latents behind 256, twenty heads": (mc.rotated_latent(20, 16, 30, 40, 250, 24, 50), 64, 4, (), 5),
+    "rotated latents behind 384": (mc.rotated_latent(2, 16, 16, 20, 384, 64, 19), 64, 4, (), 5),
+    "rotated latents behind 512, 192 wide": (mc.rotated_latent(3, 128, 128, 64, 512, 64, 48), 96, 4, (), 5),
+    "rotated latents behind 512, more than one head group": (mc.rotated_latent(37, 9, 12, 20, 512, 8, 60), 64, 4, (), 5),
+    "rotated latents above the tensor-core kernel": (mc.rotated_latent(2, 24, 32, 30, 600, 16, 30), 64, 4, (), 5),
+    "rotated latents, heads too wide to expand": (mc.rotated_latent(2, 250, 20, 30, 64, 16, 30), 64, 4, (), 5),
+    "rotated latents, window of one": (mc.rotated_latent(2, 16, 16, 20, 40, 8, 1), 64, 4, (), 5),
+    "rotated latents, plain rotation": (mc.rotated_latent(4, 24, 24, 32, 40, 24, 40, scaling=None), 64, 4, (), 5),
+    "gelu feed-forward": (mc.scaled_parallel((2, 1, 16, 8), (1, 8), 9, ff=200), 66, 4, ("l0.mix.left.o", "l0.mix.right.o"), 5),
+}
+
+
 def check_alone(folder, oracle, compute):
     """The residual stream after a layer with one mechanism at work, for a whole prompt, portions and single tokens."""
     toks = tokens_of(75, oracle.cfg["vocab"])
@@ -155,6 +188,13 @@ def test_mechanism_alone_in_layers_with_one_norm(mk, tmp_path, name, compute):
 def test_mechanism_alone_in_layers_with_norms_on_outputs(mk, tmp_path, name, compute):
     layer, width, silenced = ALONE_OUTPUT[name]
     check_alone(*checkpoint(tmp_path, mc.tevanex([layer], width=width), seed=7, change=silence(*silenced)), compute)
+
+
+@pytest.mark.parametrize("compute", DTYPES)
+@pytest.mark.parametrize("name", ALONE_CONV)
+def test_mechanism_alone_in_layers_behind_a_convolution(mk, tmp_path, name, compute):
+    layer, width, taps, silenced, rank = ALONE_CONV[name]
+    check_alone(*checkpoint(tmp_path, mc.mamivik([layer], width=width, taps=taps), seed=7, rank=rank, change=silence(*silenced)), compute)
 
 
 @pytest.mark.parametrize("compute", DTYPES)
@@ -202,6 +242,10 @@ MODELS = {
     "experts": (mc.tevanex(_EXPERTS + [mc.again(_EXPERTS, 1), mc.again(_EXPERTS, 0)], width=104), 0),
     "experts, odd sizes": (mc.tevanex([mc.capped_attention(6, 2, 44, 36, 28, 50, mlp=mc.experts(5, 3, 37)), mc.mlstm(3, 40, 21, mlp=mc.experts(9, 2, 50, 0.6, (70, 0.4))),
                                        mc.sink_attention(8, 1, 32, 80, 32, 20)], width=67, vocab=201, eps=1e-5, embed=2.3, mult=0.35, logit_scale=1.4, softcap=3.0), 0),
+    "convolved": (mc.mamivik([mc.scaled_parallel((4, 2, 64, 16), (3, 48), 37, ff=150), mc.rotated_latent(4, 32, 40, 30, 56, 16, 50, ff=90),
+                              mc.scaled_parallel((8, 2, 32, 32), (2, 64), 21, scales=(1.3, 0.4))], width=104, taps=4), 9),
+    "convolved, odd sizes": (mc.mamivik([mc.rotated_latent(6, 20, 36, 24, 130, 14, 23), mc.scaled_parallel((6, 2, 36, 12), (3, 40), 60, ff=37),
+                                         mc.rotated_latent(2, 70, 20, 48, 90, 40, 100, ff=64, scaling=None)], width=67, vocab=201, taps=6, eps=1e-5), 4),
     "time mixing only": (mc.config([mc.wkv(2, 32), mc.wkv(1, 72)], width=64, side=64), 20),
 }
 
@@ -232,7 +276,7 @@ def test_prompt_portions_and_decoding_agree(mk, built, name, compute):
     model.close()
 
 
-BOTH = ["first", "looped", "experts"]   # a model of each layer form
+BOTH = ["first", "looped", "experts", "convolved"]   # a model of each layer form
 
 
 @pytest.mark.parametrize("compute", DTYPES)
@@ -468,7 +512,7 @@ def test_a_fork_carries_pages_and_state(mk, built, name, compute):
     model.close()
 
 
-@pytest.mark.parametrize("name", ["second", "looped", "experts"])
+@pytest.mark.parametrize("name", ["second", "looped", "experts", "convolved"])
 def test_a_refused_forward_leaves_the_state_alone(mk, built, capi, name):
     folder, oracle, cfg = built(name)
     toks = tokens_of(50, cfg["vocab"], seed=9)
@@ -484,7 +528,7 @@ def test_a_refused_forward_leaves_the_state_alone(mk, built, capi, name):
     model.close()
 
 
-@pytest.mark.parametrize("name", ["first", "second", "looped", "loop over all layers", "no loop", "experts", "experts, odd sizes"])
+@pytest.mark.parametrize("name", ["first", "second", "looped", "loop over all layers", "no loop", "experts", "experts, odd sizes", "convolved", "convolved, odd sizes"])
 def test_greedy_generation_through_the_engine(mk, eng, built, name):
     """Requests of unequal length through the scheduler, more of them than slots; 32-bit, so that the plain statement's own
     argmax must come out wherever its first two logits are not a near-tie."""
@@ -521,7 +565,7 @@ def test_device_sampling_and_recorded_logits(mk, eng, built, name):
     assert outs[0] == outs[1]
 
 
-@pytest.mark.parametrize("name", ["second", "looped", "loop over all layers", "experts", "experts, odd sizes"])
+@pytest.mark.parametrize("name", ["second", "looped", "loop over all layers", "experts", "experts, odd sizes", "convolved", "convolved, odd sizes"])
 def test_residuals_after_every_layer(mk, built, name):
     """A looped layer counts once per pass."""
     folder, oracle, cfg = built(name)
