@@ -20,7 +20,7 @@ BUILD = HERE / "build"
 LIB = HERE / "libmacllm_b200.so"
 SERVING_LIB = HERE / "libmacllm_b200_serving.so"
 # the translation units behind a safetensors checkpoint; the rest serves GGUF files and kernel-level callers
-SERVING = ["attention.cu", "attention_tc.cu", "batch.cu", "c_api_core.cpp", "c_api_model.cpp", "device_lm.cpp", "embed.cu", "engine.cpp", "gated_scan.cu", "hgemm_tc.cu",
+SERVING = ["attention.cu", "attention_tc.cu", "batch.cu", "channel_delta.cu", "c_api_core.cpp", "c_api_model.cpp", "device_lm.cpp", "embed.cu", "engine.cpp", "gated_scan.cu", "hgemm_tc.cu",
            "json.cpp", "kv_pool.cpp", "latent_attention.cu", "linear_state.cu", "mixer_lm.cpp", "mixer_lm_conv.cpp", "mixer_lm_output.cpp", "mixer_lm_side.cpp", "mixer_ops.cu", "mixer_spec.cpp", "mlstm.cu", "model_registry.cpp", "moe_rows.cu", "paged_lm.cpp",
            "rope_kv.cu", "safetensors_file.cpp", "sample.cu", "seed_model.cpp", "device_info.cpp", "weights.cpp"]
 

@@ -86,8 +86,42 @@ struct ChannelDeltaArgs {
     int r_col = 0, k_col = 0, v_col = 0;
     const float* decay = nullptr;    // [rows][heads * dim]
     const float* removal = nullptr;  // [rows][heads * dim]
+    // for the forms that make decay and removal themselves (see ChannelGatesArgs): the columns of the removal rates' and of the
+    // low-rank input, and the weights; w2h: w2t as bfloat16, taken instead when it is there
+    int a_col = 0, low_col = 0, rank = 0;
+    const float *w2t = nullptr, *w0 = nullptr, *a_bias = nullptr;
+    const __nv_bfloat16* w2h = nullptr;
 };
+// Row by row, from `decay` and `removal`.
 void launch_channel_delta_scan(const ChannelDeltaArgs& a, cudaStream_t s);
+// One-token lanes, from the projections; finishes (common.image is set).
+bool channel_delta_can_step(int dim, int rank);
+void launch_channel_delta_step(const ChannelDeltaArgs& a, cudaStream_t s);
+#ifdef __CUDACC__
+// The decay of a channel from the logit of its low-rank projection: exp(-exp(-1/2) sigmoid(z)).
+__device__ __forceinline__ float channel_decay_f(float z) { return expf(-0.60653066f * sigmoid_f(z)); }
+
+// N values per lane summed over LPC lanes (a power of two): lane l ends with value(s) first .. first + returned - 1 in v[0 ..].
+template <int N, int LPC>
+__device__ __forceinline__ int fold_lanes(float (&v)[N], int lane, int& first) {
+    int n = N;
+    first = 0;
+#pragma unroll
+    for (int x = 1; x < LPC; x <<= 1) {
+        if (n > 1) {
+            n >>= 1;
+            const bool up = (lane & x) != 0;
+#pragma unroll
+            for (int i = 0; i < N / 2; ++i)
+                if (i < n) v[i] = (up ? v[i + n] : v[i]) + __shfl_xor_sync(0xffffffffu, up ? v[i] : v[i + n], x);
+            first += up ? n : 0;
+        } else {
+            v[0] += __shfl_xor_sync(0xffffffffu, v[0], x);
+        }
+    }
+    return n;
+}
+#endif
 
 // Whether the finishing form (LinearStateArgs::image) exists for these sizes.
 bool linear_state_can_finish(int dim, int vdim);

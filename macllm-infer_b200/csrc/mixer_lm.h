@@ -83,7 +83,7 @@ private:
         int rot0 = 0, q_rot0 = 0, c_rot = 0;  // rotated part: its column in a page row and in a query head, its projection's column
         int mix_cols = 0;     // columns of the mixer in `out`'s input; the feed-forward's follow
         // delta rule with channel gates (columns d_q: r, d_k, d_v, d_a, d_g, c_low; w2t, w0 as WKV's)
-        DevBuf a_b;
+        DevBuf a_b, w2h;
         // the short convolution in front of the mixer, [taps][width]
         DevBuf input_conv;
         // minGRU (columns c_q: z, c_v: x, c_g: g)

@@ -54,6 +54,14 @@ void MixerLm::load_conv_input(const SafetensorsFile& f, int l) {
         w.rope = rope_table(a.rot);
         linear_state_key_pad(d.dim);  // refuses head dimensions the recurrence does not take
         upload_low_rank(f, R, n, d.rank, w);
+        if (!f32_) {
+            const std::vector<uint16_t> w2 = f.bf16_values(R + "w2", {n, d.rank});
+            std::vector<uint16_t> t(w2.size());
+            for (int c = 0; c < n; ++c)
+                for (int j = 0; j < d.rank; ++j) t[(size_t)j * n + c] = w2[(size_t)c * d.rank + j];
+            w.w2h.upload(t.data(), t.size() * 2, stream_);
+            MK_CUDA(cudaStreamSynchronize(stream_));
+        }
         upload_f32(f.values(R + "a.b", {n}), w.a_b);
         upload_f32(f.values(R + "norm", {n}), w.head_norm);
         w.mix_cols = pad_to(a.heads * a.vdim, 64);
@@ -116,23 +124,6 @@ void MixerLm::run_channel_delta(const Tick& t, int run, const Shares& y, const R
     const ChannelDeltaSpec& d = s.channel_delta;
     Layer& w = lw_[(size_t)l];
     const double n = (double)d.heads * d.dim;
-    ChannelGatesArgs g;
-    g.y = y;
-    g.k_col = w.d_k;
-    g.a_col = w.d_a;
-    g.low_col = w.c_low;
-    g.rows = T;
-    g.heads = d.heads;
-    g.dim = d.dim;
-    g.rank = d.rank;
-    g.w2t = w.w2t.as<float>();
-    g.w0 = w.w0.as<float>();
-    g.a_bias = w.a_b.as<float>();
-    g.decay = decay_.as<float>();
-    g.removal = removal_.as<float>();
-    prof_begin(KC_CHANNEL_GATES, T * (4.0 * n + d.rank) * 4.0 + n * d.rank * 4.0, 2.0 * T * n * d.rank);
-    launch_channel_gates(g, stream_);
-    prof_end();
     ChannelDeltaArgs a;
     a.common.lanes = state_lanes_;
     a.common.state = rs_[(size_t)run].state.as<float>();
@@ -150,11 +141,44 @@ void MixerLm::run_channel_delta(const Tick& t, int run, const Shares& y, const R
     a.r_col = w.d_q;
     a.k_col = w.d_k;
     a.v_col = w.d_v;
+    a.a_col = w.d_a;
+    a.low_col = w.c_low;
+    a.rank = d.rank;
+    a.w2t = w.w2t.as<float>();
+    a.w2h = w.w2h.as<__nv_bfloat16>();
+    a.w0 = w.w0.as<float>();
+    a.a_bias = w.a_b.as<float>();
+    const double state_io = 8.0 * t.B * n * d.dim;
+    if (longest_ <= 1 && channel_delta_can_step(d.dim, d.rank)) {
+        a.common.image = out;
+        prof_begin(KC_DELTA_SCAN, 4.0 * T * 5.0 * n + T * n * esz_ + n * d.rank * (f32_ ? 4.0 : 2.0) + state_io, T * n * (10.0 * d.dim + 2.0 * d.rank));
+        launch_channel_delta_step(a, stream_);
+        prof_end();
+        ++launches_;
+        return;
+    }
+    ChannelGatesArgs g;
+    g.y = y;
+    g.k_col = w.d_k;
+    g.a_col = w.d_a;
+    g.low_col = w.c_low;
+    g.rows = T;
+    g.heads = d.heads;
+    g.dim = d.dim;
+    g.rank = d.rank;
+    g.w2t = a.w2t;
+    g.w0 = a.w0;
+    g.a_bias = a.a_bias;
+    g.decay = decay_.as<float>();
+    g.removal = removal_.as<float>();
+    prof_begin(KC_CHANNEL_GATES, T * (4.0 * n + d.rank) * 4.0 + n * d.rank * 4.0, 2.0 * T * n * d.rank);
+    launch_channel_gates(g, stream_);
+    prof_end();
     a.decay = g.decay;
     a.removal = g.removal;
     const bool finish = short_lanes_ && linear_state_can_finish(d.dim, d.dim);
     if (finish) a.common.image = out;
-    prof_begin(KC_DELTA_SCAN, 4.0 * T * 6.0 * n + 8.0 * t.B * n * d.dim, 10.0 * T * n * d.dim);
+    prof_begin(KC_DELTA_SCAN, 4.0 * T * 6.0 * n + state_io, 10.0 * T * n * d.dim);
     launch_channel_delta_scan(a, stream_);
     prof_end();
     launches_ += 2;

@@ -1,6 +1,7 @@
 // See mixer_ops.h.
 #include "mixer_ops.h"
 #include "device_util.h"
+#include "linear_state.h"
 #include "recurrent_core.cuh"
 #include <algorithm>
 
@@ -450,13 +451,13 @@ __global__ void __launch_bounds__(CG_COLS) channel_gates_kernel(ChannelGatesArgs
     }
     __syncthreads();
     if (!live) return;
-    const float w0 = a.w0[c], bias = a.a_bias[c], span = expf(-0.5f);
+    const float w0 = a.w0[c], bias = a.a_bias[c];
     const int head = threadIdx.x / a.dim;
 #pragma unroll
     for (int r = 0; r < ROWS; ++r) {
         if (r0 + r >= a.rows) break;
         const int64_t at = (int64_t)(r0 + r) * channels + c;
-        a.decay[at] = expf(-span * sigmoid_f(acc[r] + w0));
+        a.decay[at] = channel_decay_f(acc[r] + w0);
         a.removal[at] = sigmoid_f(gate[r] + bias) * k[r] * inv[r * tile_heads + head];
     }
 }

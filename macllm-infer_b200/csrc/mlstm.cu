@@ -41,27 +41,6 @@ struct Step {
     static constexpr int COLS = MS_WARPS * WARP_COLS;    // columns of a CTA
 };
 
-// N values per lane summed over LPC lanes (a power of two): lane l ends with value(s) first .. first + returned - 1 in v[0 ..].
-template <int N, int LPC>
-__device__ __forceinline__ int fold_lanes(float (&v)[N], int lane, int& first) {
-    int n = N;
-    first = 0;
-#pragma unroll
-    for (int x = 1; x < LPC; x <<= 1) {
-        if (n > 1) {
-            n >>= 1;
-            const bool up = (lane & x) != 0;
-#pragma unroll
-            for (int i = 0; i < N / 2; ++i)
-                if (i < n) v[i] = (up ? v[i + n] : v[i]) + __shfl_xor_sync(0xffffffffu, up ? v[i] : v[i + n], x);
-            first += up ? n : 0;
-        } else {
-            v[0] += __shfl_xor_sync(0xffffffffu, v[0], x);
-        }
-    }
-    return n;
-}
-
 template <int KD>
 __global__ void __launch_bounds__(MS_WARPS * 32, 4) mlstm_step_kernel(const __grid_constant__ MlstmScanArgs a, int vec) {
     using P = Step<KD>;

@@ -125,8 +125,8 @@ def zeros(name):
     return lambda w: w.update({name: np.zeros_like(w[name])})
 
 
-def without_first_key(w):
-    """The removal term alone: rates of zero."""
+def without_removal(w):
+    """Removal rates of zero."""
     w["l0.mix.right.a.b"] = np.full_like(w["l0.mix.right.a.b"], -1e4)
 
 
@@ -137,7 +137,7 @@ PARTS = {
     "a left constant": (PAR, None, lambda l: l["mixer"].update(left_scale=1.0), {}),
     "a right constant": (PAR, None, lambda l: l["mixer"].update(right_scale=1.0), {}),
     "a scale": (PAR, None, lambda l: l["mixer"]["left"].update(scale=0.6), {}),
-    "a removal": (PAR, without_first_key, None, {}),
+    "a removal": (PAR, without_removal, None, {}),
     "a removal's bias": (PAR, zeros("l0.mix.right.a.b"), None, {"right.a.b": 6.0, "right.a": 0.3, "right.o": 2.0}),
     "a decay's bias": (PAR, zeros("l0.mix.right.w0"), None, {}),
     "a decay that reads its input": (PAR, zeros("l0.mix.right.w2"), None, {"right.w2": 20.0, "right.w1": 3.0, "right.o": 2.0}),
