@@ -97,9 +97,15 @@ void launch_channel_delta_scan(const ChannelDeltaArgs& a, cudaStream_t s);
 // One-token lanes, from the projections; finishes (common.image is set).
 bool channel_delta_can_step(int dim, int rank);
 void launch_channel_delta_step(const ChannelDeltaArgs& a, cudaStream_t s);
+// Prompts in chunks on tensor cores, from the projections (w2h is set), lanes in packed order, the longest of `longest` rows; leaves
+// the raw rows in common.out.  `scratch`: channel_delta_chunk_bytes for all tokens and lanes of a tick.  Two kernels.
+bool channel_delta_can_chunk(int dim);
+size_t channel_delta_chunk_bytes(int dim, int heads, int tokens, int lanes);
+void launch_channel_delta_chunks(const ChannelDeltaArgs& a, int longest, void* scratch, cudaStream_t s);
 #ifdef __CUDACC__
-// The decay of a channel from the logit of its low-rank projection: exp(-exp(-1/2) sigmoid(z)).
-__device__ __forceinline__ float channel_decay_f(float z) { return expf(-0.60653066f * sigmoid_f(z)); }
+// The decay of a channel from the logit of its low-rank projection, exp(-exp(-1/2) sigmoid(z)), and its logarithm.
+__device__ __forceinline__ float channel_log_decay_f(float z) { return -0.60653066f * sigmoid_f(z); }
+__device__ __forceinline__ float channel_decay_f(float z) { return expf(channel_log_decay_f(z)); }
 
 // N values per lane summed over LPC lanes (a power of two): lane l ends with value(s) first .. first + returned - 1 in v[0 ..].
 template <int N, int LPC>

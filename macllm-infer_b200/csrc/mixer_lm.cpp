@@ -24,8 +24,6 @@ const RegisterModelFormat register_mixer_format(ModelFormat{
     "folder with config.json and model.safetensors", is_mixer_checkpoint,
     [](const std::string& path, const ModelConfig& cfg) -> std::unique_ptr<PagedLm> { return std::make_unique<MixerLm>(path, cfg); }});
 
-constexpr int kShortLane = 4;  // lanes up to this many tokens: the recurrence kernels finish the head rows themselves
-
 }  // namespace
 
 MixerLm::MixerLm(const std::string& dir, const ModelConfig& cfg) : DeviceLm(cfg, class_names) {
@@ -361,6 +359,7 @@ void MixerLm::alloc_activations() {
     int lat_ctas = 1;
     int64_t lat_part = 0;
     int64_t mlstm_heads = 0, qkv = 0, removal = 0;
+    size_t delta_scratch = 0;
     int64_t pairs = 0, experts = 0, expert_ff = 0, expert_gu = 0;  // routed rows, experts, widths of an expert's activations
     for (size_t l = 0; l < lw_.size(); ++l) {
         const MixerLayerSpec& s = ms_.layers[l];
@@ -422,6 +421,7 @@ void MixerLm::alloc_activations() {
             attn = std::max(attn, (int64_t)s.attn.heads * w.row_width);
             const int64_t n = (int64_t)s.channel_delta.heads * s.channel_delta.dim;
             removal = std::max(removal, n);
+            if (!f32_) delta_scratch = std::max(delta_scratch, channel_delta_chunk_bytes(s.channel_delta.dim, s.channel_delta.heads, (int)T, B));
             hd = std::max(hd, n);
             raw = std::max(raw, n);
         }
@@ -460,6 +460,7 @@ void MixerLm::alloc_activations() {
     }
     decay_.alloc((size_t)(T * hd) * 4);
     removal_.alloc((size_t)(T * removal) * 4);
+    delta_scratch_.alloc(delta_scratch);
     raw_.alloc((size_t)(T * raw) * 4);
     q_rot_.alloc((size_t)(T * attn) * 4);
     img_q_.alloc((size_t)(T * q_lat) * esz_);
@@ -484,6 +485,7 @@ void MixerLm::alloc_activations() {
     if (!f32_)
         for (DevBuf& p : partial_) p.alloc(kSplitScratchBytes);
     size_t extra = (size_t)B * sizeof(StateLane) + 16;
+    if (ms_.conv_taps > 0) extra += (size_t)B * sizeof(StateLane) + 48;
     size_t part_o = 0, part_ml = 0, counters = 0;
     for (const Geometry& g : geo_) {
         if (g.tc) {
@@ -886,6 +888,7 @@ void MixerLm::run_forward(const std::vector<LmLane>& lanes, KvReservation& r, ui
     longest_ = longest;
     short_lanes_ = longest <= kShortLane;
     const size_t off_halves = stage_bytes(t, halves.data(), halves.size() * sizeof(StateLane));
+    if (ms_.conv_taps > 0) split_delta_lanes(t, halves);
     std::vector<int32_t> sp((size_t)B), nt((size_t)B), nb((size_t)B);
     for (int i = 0; i < B; ++i) {
         sp[(size_t)i] = lanes[(size_t)i].start_pos;
@@ -916,6 +919,7 @@ void MixerLm::run_forward(const std::vector<LmLane>& lanes, KvReservation& r, ui
     upload_tick(t, 64, KC_BATCH);
     state_lanes_.lane = reinterpret_cast<const StateLane*>(t.dp + off_halves);
     state_lanes_.lanes = B;
+    for (LaneSet* s : {&delta_one_, &delta_rows_, &delta_chunks_}) s->lanes.lane = reinterpret_cast<const StateLane*>(t.dp + s->off);
     // copy-on-write page copies of shared partial tails
     for (const KvCowCopy& c : r.cow_copies())
         for (size_t i = 0; i < rs_.size(); ++i) {

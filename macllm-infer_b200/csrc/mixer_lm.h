@@ -17,6 +17,8 @@ namespace mk {
 
 inline int pad_to(int64_t n, int m) { return (int)((n + m - 1) / m * m); }
 
+constexpr int kShortLane = 4;  // lanes up to this many tokens: the recurrence kernels finish the head rows themselves
+
 class MixerLm : public DeviceLm {
 public:
     // `dir` holds config.json and model.safetensors.
@@ -186,6 +188,7 @@ private:
     void load_conv_input(const SafetensorsFile& f, int l);
     void run_conv_input(const Tick& t, int run, Pending& p, const std::vector<LmLane>& lanes);
     void run_channel_delta(const Tick& t, int run, const Shares& y, const RowImage& out);
+    void split_delta_lanes(Tick& t, const std::vector<StateLane>& lanes);
     void upload_low_rank(const SafetensorsFile& f, const std::string& prefix, int channels, int rank, Layer& w);
     // layers whose mixer and feed-forward read one norm
     void begin_pass(const Tick& t, int pass, Pending& p);
@@ -231,6 +234,15 @@ private:
     int attn_max_entries_ = 0;
     int cur_ = 0;             // which of x_ holds the residual stream
     StateLanes state_lanes_;  // of the running tick
+    // its lanes by the form the delta rule with channel gates takes
+    struct LaneSet {
+        StateLanes lanes;
+        int longest = 0;
+        int64_t rows = 0;
+        size_t off = 0;
+    };
+    LaneSet delta_one_, delta_rows_, delta_chunks_;   // one token; row by row; chunks
+    DevBuf delta_scratch_;
     bool short_lanes_ = false;
     int longest_ = 0;         // tokens of the longest lane
 

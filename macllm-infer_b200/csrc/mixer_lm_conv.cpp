@@ -2,8 +2,16 @@
 // shared keys and values beside the delta rule with channel gates, and windowed latent attention with a rotated part.  Both branches
 // of the former share one output matmul over their columns, to which each comes times its constant.  See mixer_lm.h.
 #include "mixer_lm.h"
+#include <algorithm>
 
 namespace mk {
+
+namespace {
+
+// Lanes with at least this many tokens in a tick run the delta rule in chunks of rows.
+constexpr int kChunkFrom = 48;
+
+}  // namespace
 
 // ---------------------------------------------------------------------------- load
 
@@ -125,7 +133,6 @@ void MixerLm::run_channel_delta(const Tick& t, int run, const Shares& y, const R
     Layer& w = lw_[(size_t)l];
     const double n = (double)d.heads * d.dim;
     ChannelDeltaArgs a;
-    a.common.lanes = state_lanes_;
     a.common.state = rs_[(size_t)run].state.as<float>();
     a.common.heads = d.heads;
     a.common.dim = a.common.vdim = d.dim;
@@ -148,46 +155,80 @@ void MixerLm::run_channel_delta(const Tick& t, int run, const Shares& y, const R
     a.w2h = w.w2h.as<__nv_bfloat16>();
     a.w0 = w.w0.as<float>();
     a.a_bias = w.a_b.as<float>();
-    const double state_io = 8.0 * t.B * n * d.dim;
-    if (longest_ <= 1 && channel_delta_can_step(d.dim, d.rank)) {
-        a.common.image = out;
-        prof_begin(KC_DELTA_SCAN, 4.0 * T * 5.0 * n + T * n * esz_ + n * d.rank * (f32_ ? 4.0 : 2.0) + state_io, T * n * (10.0 * d.dim + 2.0 * d.rank));
-        launch_channel_delta_step(a, stream_);
+    // Sets of lanes whose form this head size does not have go row by row.
+    const bool step = channel_delta_can_step(d.dim, d.rank), chunk = !f32_ && channel_delta_can_chunk(d.dim);
+    std::vector<const LaneSet*> by_row;
+    if (delta_rows_.rows > 0) by_row.push_back(&delta_rows_);
+    if (delta_one_.rows > 0 && !step) by_row.push_back(&delta_one_);
+    if (delta_chunks_.rows > 0 && !chunk) by_row.push_back(&delta_chunks_);
+    const bool chunks_run = chunk && delta_chunks_.rows > 0;
+    auto state_io = [&](const LaneSet& l) { return 8.0 * l.lanes.lanes * n * d.dim; };
+    bool unfinished = chunks_run;
+    for (const LaneSet* l : by_row) unfinished |= l->longest > kShortLane || !linear_state_can_finish(d.dim, d.dim);
+    for (const LaneSet* l : by_row) {
+        ChannelGatesArgs g;
+        g.y = y;
+        g.k_col = w.d_k;
+        g.a_col = w.d_a;
+        g.low_col = w.c_low;
+        g.lanes = a.common.lanes = l->lanes;
+        g.longest = l->longest;
+        g.heads = d.heads;
+        g.dim = d.dim;
+        g.rank = d.rank;
+        g.w2t = a.w2t;
+        g.w0 = a.w0;
+        g.a_bias = a.a_bias;
+        a.decay = g.decay = decay_.as<float>();
+        a.removal = g.removal = removal_.as<float>();
+        prof_begin(KC_CHANNEL_GATES, l->rows * (4.0 * n + d.rank) * 4.0 + n * d.rank * 4.0, 2.0 * l->rows * n * d.rank);
+        launch_channel_gates(g, stream_);
         prof_end();
-        ++launches_;
-        return;
+        a.common.image = unfinished ? RowImage{} : out;
+        prof_begin(KC_DELTA_SCAN, 4.0 * l->rows * 6.0 * n + state_io(*l), 10.0 * l->rows * n * d.dim);
+        launch_channel_delta_scan(a, stream_);
+        prof_end();
+        launches_ += 2;
     }
-    ChannelGatesArgs g;
-    g.y = y;
-    g.k_col = w.d_k;
-    g.a_col = w.d_a;
-    g.low_col = w.c_low;
-    g.rows = T;
-    g.heads = d.heads;
-    g.dim = d.dim;
-    g.rank = d.rank;
-    g.w2t = a.w2t;
-    g.w0 = a.w0;
-    g.a_bias = a.a_bias;
-    g.decay = decay_.as<float>();
-    g.removal = removal_.as<float>();
-    prof_begin(KC_CHANNEL_GATES, T * (4.0 * n + d.rank) * 4.0 + n * d.rank * 4.0, 2.0 * T * n * d.rank);
-    launch_channel_gates(g, stream_);
-    prof_end();
-    a.decay = g.decay;
-    a.removal = g.removal;
-    const bool finish = short_lanes_ && linear_state_can_finish(d.dim, d.dim);
-    if (finish) a.common.image = out;
-    prof_begin(KC_DELTA_SCAN, 4.0 * T * 6.0 * n + state_io, 10.0 * T * n * d.dim);
-    launch_channel_delta_scan(a, stream_);
-    prof_end();
-    launches_ += 2;
-    if (!finish) {
+    if (chunks_run) {
+        a.common.lanes = delta_chunks_.lanes;
+        a.common.image = RowImage{};
+        prof_begin(KC_DELTA_SCAN, 4.0 * delta_chunks_.rows * (5.0 * n + d.rank) + n * d.rank * 2.0 + state_io(delta_chunks_), delta_chunks_.rows * n * (10.0 * d.dim + 2.0 * d.rank));
+        launch_channel_delta_chunks(a, delta_chunks_.longest, delta_scratch_.ptr(), stream_);
+        prof_end();
+        launches_ += 2;
+    }
+    if (unfinished) {  // all rows of the tick; the one-token lanes' are written over
         a.common.image = out;
         prof_begin(KC_GATES, T * n * (8.0 + esz_), 0);
         launch_head_norm_gate(a.common, T, stream_);
         prof_end();
         ++launches_;
+    }
+    if (delta_one_.rows > 0 && step) {
+        a.common.lanes = delta_one_.lanes;
+        a.common.image = out;
+        prof_begin(KC_DELTA_SCAN, delta_one_.rows * n * (20.0 + esz_) + n * d.rank * (f32_ ? 4.0 : 2.0) + state_io(delta_one_), delta_one_.rows * n * (10.0 * d.dim + 2.0 * d.rank));
+        launch_channel_delta_step(a, stream_);
+        prof_end();
+        ++launches_;
+    }
+}
+
+// One-token lanes, lanes of a few tokens and prompts take different forms of the delta rule with channel gates.
+void MixerLm::split_delta_lanes(Tick& t, const std::vector<StateLane>& lanes) {
+    LaneSet* sets[] = {&delta_one_, &delta_rows_, &delta_chunks_};
+    std::vector<StateLane> of[3];
+    for (const StateLane& l : lanes) of[l.n <= 1 ? 0 : (l.n < kChunkFrom ? 1 : 2)].push_back(l);
+    for (int i = 0; i < 3; ++i) {
+        LaneSet& s = *sets[i];
+        s = LaneSet{};
+        s.lanes.lanes = (int)of[i].size();
+        for (const StateLane& l : of[i]) {
+            s.longest = std::max(s.longest, (int)l.n);
+            s.rows += l.n;
+        }
+        s.off = stage_bytes(t, of[i].data(), of[i].size() * sizeof(StateLane));
     }
 }
 

@@ -407,19 +407,21 @@ __global__ void __launch_bounds__(CG_COLS) channel_gates_kernel(ChannelGatesArgs
     float* z = cg_smem;                       // [rank][ROWS]
     float* ks = z + a.rank * ROWS;            // [ROWS][cols]
     float* inv = ks + ROWS * cols;            // [ROWS][tile_heads]
-    const int r0 = blockIdx.y * ROWS, c = blockIdx.x * cols + threadIdx.x;
+    const StateLane sl = a.lanes.at(blockIdx.z);
+    const int r0 = sl.first + blockIdx.y * ROWS, end = sl.first + sl.n, c = blockIdx.x * cols + threadIdx.x;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
+    if (r0 >= end) return;
     const bool live = (int)threadIdx.x < cols && c < channels;
     pdl_trigger();
     pdl_wait();
     for (int i = threadIdx.x; i < a.rank * ROWS; i += blockDim.x) {
         const int r = i / a.rank, j = i - r * a.rank;
-        z[j * ROWS + r] = r0 + r < a.rows ? tanhf(a.y.at(r0 + r, a.low_col + j)) : 0.f;
+        z[j * ROWS + r] = r0 + r < end ? tanhf(a.y.at(r0 + r, a.low_col + j)) : 0.f;
     }
     float k[ROWS], gate[ROWS];
 #pragma unroll
     for (int r = 0; r < ROWS; ++r) {
-        const bool there = live && r0 + r < a.rows;
+        const bool there = live && r0 + r < end;
         k[r] = there ? a.y.at(r0 + r, a.k_col + c) : 0.f;
         gate[r] = there ? a.y.at(r0 + r, a.a_col + c) : 0.f;
         if ((int)threadIdx.x < cols) ks[r * cols + threadIdx.x] = k[r];
@@ -455,7 +457,7 @@ __global__ void __launch_bounds__(CG_COLS) channel_gates_kernel(ChannelGatesArgs
     const int head = threadIdx.x / a.dim;
 #pragma unroll
     for (int r = 0; r < ROWS; ++r) {
-        if (r0 + r >= a.rows) break;
+        if (r0 + r >= end) break;
         const int64_t at = (int64_t)(r0 + r) * channels + c;
         a.decay[at] = channel_decay_f(acc[r] + w0);
         a.removal[at] = sigmoid_f(gate[r] + bias) * k[r] * inv[r * tile_heads + head];
@@ -468,7 +470,7 @@ void launch_channel_rows(const ChannelGatesArgs& a, cudaStream_t s) {
     const size_t smem = ((size_t)a.rank * ROWS + (size_t)ROWS * (cols + tile_heads)) * 4;
     if (smem > (size_t)220 * 1024) throw std::runtime_error("launch_channel_gates: the low rank is too large");
     ensure_dynamic_smem(reinterpret_cast<const void*>(&channel_gates_kernel<ROWS>), smem);
-    const dim3 grid((unsigned)((a.heads + tile_heads - 1) / tile_heads), (unsigned)((a.rows + ROWS - 1) / ROWS));
+    const dim3 grid((unsigned)((a.heads + tile_heads - 1) / tile_heads), (unsigned)((a.longest + ROWS - 1) / ROWS), (unsigned)a.lanes.lanes);
     launch_pdl(channel_gates_kernel<ROWS>, grid, dim3((unsigned)((cols + 31) / 32 * 32)), smem, s, a, tile_heads);
     MK_LAUNCH_CHECK();
 }
@@ -879,9 +881,10 @@ void launch_wkv_decay(const Shares& low, int low_col, int rows, int rank, int ch
 }
 
 void launch_channel_gates(const ChannelGatesArgs& a, cudaStream_t s) {
-    if (a.rows <= 0) return;
+    if (a.lanes.lanes <= 0 || a.longest <= 0) return;
     if (a.dim > CG_COLS) throw std::runtime_error("launch_channel_gates: head dimensions above 256 are not supported");
-    if (a.rows > 256) launch_channel_rows<16>(a, s);
+    if (a.lanes.lanes > 65535 || a.longest > 65535 * 4) throw std::runtime_error("launch_channel_gates: too many lanes or rows");
+    if (a.longest > 256) launch_channel_rows<16>(a, s);
     else launch_channel_rows<4>(a, s);
 }
 

@@ -55,13 +55,15 @@ void launch_row_update(const RowUpdateArgs& a, cudaStream_t s);
 // decay[t][c] = exp(-exp(sum_j tanh(low[t][j]) w2[c][j] + w0[c])), everything in f32.  w2t is w2 transposed, [rank][channels].
 void launch_wkv_decay(const Shares& low, int low_col, int rows, int rank, int channels, const float* w2t, const float* w0, float* decay, cudaStream_t s);
 
-// What the delta rule with channel gates needs beside its projections, everything in f32, per row and key channel c of a head:
+// What the delta rule with channel gates needs beside its projections, everything in f32, per row of the lanes and key channel c of a head:
 //   decay   = exp(-exp(-1/2) sigmoid(sum_j tanh(y[low_col + j]) w2[c][j] + w0[c]))
 //   removal = sigmoid(y[a_col + c] + a_bias[c]) k[c] / (sum of the head's k^2 + 1e-6),  k = y[k_col + c]
 struct ChannelGatesArgs {
     Shares y;
     int k_col = 0, a_col = 0, low_col = 0;
-    int rows = 0, heads = 0, dim = 0, rank = 0;
+    StateLanes lanes;
+    int longest = 0;                // rows of the longest lane
+    int heads = 0, dim = 0, rank = 0;
     const float* w2t = nullptr;     // w2 transposed, [rank][heads * dim]
     const float* w0 = nullptr;      // [heads * dim]
     const float* a_bias = nullptr;  // [heads * dim]

@@ -12,6 +12,7 @@
 // state - enters a product as the sum of two bfloat16 numbers (16 bits and more), and the state itself stays in f32 registers.
 #include "linear_state.h"
 #include "device_util.h"
+#include "mma_bf16.cuh"
 #include "recurrent_core.cuh"
 #include <algorithm>
 
@@ -184,30 +185,6 @@ constexpr int MC_THREADS = MC_WARPS * 32;           // that compute; one more wa
 
 // All warps of the CTA, the gates' one included.
 __device__ __forceinline__ void mc_sync() { asm volatile("bar.sync 1, %0;" ::"n"(MC_THREADS + 32) : "memory"); }
-
-__device__ __forceinline__ uint32_t mc_smem(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
-__device__ __forceinline__ void mc_ldmatrix(uint32_t (&r)[4], const __nv_bfloat16* p) {
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(mc_smem(p)));
-}
-__device__ __forceinline__ void mc_ldmatrix_t(uint32_t (&r)[4], const __nv_bfloat16* p) {
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(mc_smem(p)));
-}
-__device__ __forceinline__ void mc_mma(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
-                 : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
-                 : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-__device__ __forceinline__ void mc_cp_async16(void* dst, const void* src, bool valid) {
-    const int bytes = valid ? 16 : 0;  // 0: the 16 bytes become zeros
-    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(mc_smem(dst)), "l"(src), "r"(bytes) : "memory");
-}
-// x and y as bfloat16 numbers, and what that left of them.
-__device__ __forceinline__ void mc_split(float x, float y, uint32_t& hi, uint32_t& lo) {
-    const __nv_bfloat162 h = __floats2bfloat162_rn(x, y);
-    const __nv_bfloat162 l = __floats2bfloat162_rn(x - __low2float(h), y - __high2float(h));
-    hi = *reinterpret_cast<const uint32_t*>(&h);
-    lo = *reinterpret_cast<const uint32_t*>(&l);
-}
 
 // acc[N] (16 rows x 8 N columns) += A B over 16 STEPS inner indices, B in one or two parts.
 //   a_at(step): fragment of A.  b_at(step, tile): where the tile's 16 inner indices begin, its columns (or, TRANS, its inner indices)
