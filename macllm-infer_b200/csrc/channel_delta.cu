@@ -91,14 +91,33 @@ __global__ void __launch_bounds__(CS_THREADS, 2) channel_delta_step_kernel(const
     pdl_wait();
 
     const int64_t row = sl.first;
-    // r, k, v, the removal rate and the gate, then the low-rank input
-    for (int i = tid; i < 5 * KD; i += CS_THREADS) {
-        const int what = i / KD, d = i - what * KD;
-        const int col = what == 0 ? a.r_col : (what == 1 ? a.k_col : (what == 2 ? a.v_col : (what == 3 ? a.a_col : c.gate_col)));
-        float* dst = what == 0 ? s_r : (what == 1 ? s_k : (what == 2 ? s_v : (what == 3 ? s_b : s_g)));
-        dst[d] = d < dim ? a.y.at(row, col + h0 + d) : 0.f;
+    // r, k, v, the removal rate and the gate, and the low-rank input: all of a thread's numbers share by share, so that their loads overlap
+    constexpr int NV = (5 * KD + CS_THREADS - 1) / CS_THREADS;
+    {
+        const float* y = a.y.p + row * a.y.ld;
+        int col[NV + 1];
+        float val[NV + 1];
+#pragma unroll
+        for (int q = 0; q < NV; ++q) {
+            const int i = q * CS_THREADS + tid, what = i / KD, d = i - what * KD;
+            const int from = what == 0 ? a.r_col : (what == 1 ? a.k_col : (what == 2 ? a.v_col : (what == 3 ? a.a_col : c.gate_col)));
+            col[q] = what < 5 && d < dim ? from + h0 + d : -1;
+        }
+        col[NV] = tid < a.rank ? a.low_col + tid : -1;
+#pragma unroll
+        for (int q = 0; q <= NV; ++q) val[q] = col[q] >= 0 ? y[col[q]] : 0.f;
+#pragma unroll 4
+        for (int s = 1; s < a.y.n; ++s)
+#pragma unroll
+            for (int q = 0; q <= NV; ++q)
+                if (col[q] >= 0) val[q] += y[s * a.y.stride + col[q]];
+#pragma unroll
+        for (int q = 0; q < NV; ++q) {
+            const int i = q * CS_THREADS + tid, what = i / KD, d = i - what * KD;
+            if (what < 5) (what == 0 ? s_r : (what == 1 ? s_k : (what == 2 ? s_v : (what == 3 ? s_b : s_g))))[d] = val[q];
+        }
+        if (tid < a.rank) s_z[tid] = tanhf(val[NV]);
     }
-    for (int j = tid; j < a.rank; j += CS_THREADS) s_z[j] = tanhf(a.y.at(row, a.low_col + j));
     asm volatile("cp.async.wait_group 0;" ::: "memory");
     __syncthreads();
     {
@@ -229,7 +248,7 @@ struct ChunkSmem {
     static constexpr int OPERAND = CC_ROWS * KP;       // bfloat16 numbers of one part
     static constexpr int TRI = CC_ROWS * CC_AP;
     static constexpr size_t HALVES = (size_t)5 * 2 * OPERAND + 2 * 2 * TRI + 2 * 4 * 16 * 24;
-    static constexpr size_t FLOATS = 4 * 16 * 17 + 7 * KD;
+    static constexpr size_t FLOATS = 4 * 16 * 20 + 3 * KD + CC_THREADS;
     static constexpr size_t BYTES = HALVES * 2 + FLOATS * 4;
     static_assert(BYTES <= 227 * 1024, "shared memory");
     static_assert((size_t)CC_ROWS * (KD + 4) * 4 <= (size_t)2 * OPERAND * 2, "the log decays fit in an operand's place");
@@ -251,8 +270,8 @@ __global__ void __launch_bounds__(CC_THREADS, 1) channel_delta_chunk_kernel(cons
     __nv_bfloat16* tri = base + 10 * P::OPERAND;
     const Split A1{tri, AP, P::TRI}, A2{tri + 2 * P::TRI, AP, P::TRI};
     const Split Ti{tri + 4 * P::TRI, 24, 4 * 16 * 24};
-    float* s_diag = reinterpret_cast<float*>(tri + 4 * P::TRI + 2 * 4 * 16 * 24);   // [4][16][17]
-    float *s_mid = s_diag + 4 * 16 * 17, *s_em = s_mid + KD, *s_elm = s_em + KD, *s_sum = s_elm + KD;   // s_sum: [4][KD]
+    float* s_diag = reinterpret_cast<float*>(tri + 4 * P::TRI + 2 * 4 * 16 * 24);   // [4][16][20]
+    float *s_start = s_diag + 4 * 16 * 20, *s_em = s_start + KD, *s_elm = s_em + KD, *s_sum = s_elm + KD;   // s_sum: [CC_THREADS]
     float* s_l = reinterpret_cast<float*>(V.p);                                     // [C][KD + 4]
     constexpr int LP = KD + 4;
 
@@ -266,37 +285,100 @@ __global__ void __launch_bounds__(CC_THREADS, 1) channel_delta_chunk_kernel(cons
     const int m = min(C, sl.n - chunk * C);
     const int64_t row0 = (int64_t)sl.first + (int64_t)chunk * C, channels = (int64_t)cm.heads * dim;
     uint8_t* out = results + ((int64_t)chunk_slot(sl, blockIdx.z, chunk) * cm.heads + head) * R::BYTES;
-    pdl_wait();
-
-    const int r16 = (warp & 3) * 16, quarter = warp >> 2;
-    // ---- log decays: tanh of the low-rank input (three parts: f32) times w2
-    {
-        float acc[XT][4] = {};
-        const int c0 = quarter * (KD / 4);
-        __nv_bfloat16* zs = base;                 // [3][C][AP]
-        __nv_bfloat16* w2 = zs + 3 * P::TRI;      // [C][KP]
-        for (int j0 = 0; j0 < a.rank; j0 += C) {
-            const int nj = min(C, a.rank - j0);
-            if (j0 > 0) __syncthreads();
-            for (int i = tid; i < C * C; i += CC_THREADS) {
-                const int t = i / C, j = i % C;
-                float z = t < m && j < nj ? tanhf(a.y.at(row0 + t, a.low_col + j0 + j)) : 0.f;
-#pragma unroll
-                for (int p = 0; p < 3; ++p) {
-                    const __nv_bfloat16 h = __float2bfloat16_rn(z);
-                    zs[p * P::TRI + t * AP + j] = h;
-                    z -= __bfloat162float(h);
-                }
+    __nv_bfloat16* zs = base;                 // [3][C][AP]
+    __nv_bfloat16* w2 = zs + 3 * P::TRI;      // [C][KP]
+    // 64 rows of the low-rank matrix; columns past the head and rows past the rank are zeros
+    auto request_w2 = [&](int j0) {
+        const int nj = min(C, a.rank - j0);
+        if (vec && dim % 8 == 0) {
+            for (int i = tid; i < C * (KD / 8); i += CC_THREADS) {
+                const int j = i / (KD / 8), c = i % (KD / 8) * 8;
+                const bool live = j < nj && c < dim;
+                mc_cp_async16(w2 + j * KP + c, a.w2h + (live ? (int64_t)(j0 + j) * channels + h0 + c : 0), live);
             }
+        } else {
             for (int i = tid; i < C * KD; i += CC_THREADS) {
                 const int j = i / KD, c = i % KD;
                 w2[j * KP + c] = j < nj && c < dim ? a.w2h[(int64_t)(j0 + j) * channels + h0 + c] : __float2bfloat16_rn(0.f);
             }
+        }
+        asm volatile("cp.async.commit_group;" ::: "memory");
+    };
+    request_w2(0);
+    const int quarter = warp >> 2, z16 = (warp & 3) * 16;
+    constexpr int ROWS = C / CC_WARPS, EL = KD / 32;   // rows of a warp, channels of a lane
+    float w0[XT][2], bias[EL];
+#pragma unroll
+    for (int j = 0; j < XT; ++j)
+#pragma unroll
+        for (int x = 0; x < 2; ++x) {
+            const int c = quarter * (KD / 4) + j * 8 + 2 * tq + x;
+            w0[j][x] = c < dim ? a.w0[h0 + c] : 0.f;
+        }
+#pragma unroll
+    for (int e = 0; e < EL; ++e) bias[e] = lane * EL + e < dim ? a.a_bias[h0 + lane * EL + e] : 0.f;
+    pdl_wait();
+
+    // raw projections on their way while the decays are made: keys and queries in the places of operands, rates in the triangles'
+    const bool plain = vec && a.y.n == 1;
+    float *raw_k = reinterpret_cast<float*>(Kw.p), *raw_r = reinterpret_cast<float*>(Rq.p), *raw_g = reinterpret_cast<float*>(tri);   // [C][KD]
+    auto request_raw = [&](float* dst, int col) {
+        for (int i = tid; i < C * (KD / 4); i += CC_THREADS) {
+            const int t = i / (KD / 4), c = i % (KD / 4) * 4;
+            if (plain) {
+                const bool live = t < m && c < dim;
+                mc_cp_async16(dst + t * KD + c, a.y.p + (live ? (row0 + t) * a.y.ld + col + h0 + c : 0), live);
+            } else {
+#pragma unroll
+                for (int e = 0; e < 4; ++e) dst[t * KD + c + e] = t < m && c + e < dim ? a.y.at(row0 + t, col + h0 + c + e) : 0.f;
+            }
+        }
+    };
+    request_raw(raw_k, a.k_col);
+    request_raw(raw_r, a.r_col);
+    request_raw(raw_g, a.a_col);
+    asm volatile("cp.async.commit_group;" ::: "memory");
+    // ---- log decays: tanh of the low-rank input (three parts: f32) times w2
+    {
+        float acc[XT][4] = {};
+        const int c0 = quarter * (KD / 4);
+        for (int j0 = 0; j0 < a.rank; j0 += C) {
+            const int nj = min(C, a.rank - j0);
+            if (j0 > 0) {
+                __syncthreads();
+                request_w2(j0);
+            }
+            float z[C * C / CC_THREADS];
+#pragma unroll
+            for (int q = 0; q < C * C / CC_THREADS; ++q) {
+                const int i = q * CC_THREADS + tid, t = i / C, j = i % C;
+                const int64_t at = (row0 + t) * a.y.ld + a.low_col + j0 + j;
+                z[q] = t < m && j < nj ? a.y.p[at] : 0.f;
+            }
+            for (int p = 1; p < a.y.n; ++p)
+#pragma unroll
+                for (int q = 0; q < C * C / CC_THREADS; ++q) {
+                    const int i = q * CC_THREADS + tid, t = i / C, j = i % C;
+                    if (t < m && j < nj) z[q] += a.y.p[p * a.y.stride + (row0 + t) * a.y.ld + a.low_col + j0 + j];
+                }
+#pragma unroll
+            for (int q = 0; q < C * C / CC_THREADS; ++q) {
+                const int i = q * CC_THREADS + tid;
+                float x = 1.0f - __fdividef(2.0f, 1.0f + __expf(2.0f * z[q]));  // tanh, to a few 1e-7 of 1
+#pragma unroll
+                for (int p = 0; p < 3; ++p) {
+                    const __nv_bfloat16 h = __float2bfloat16_rn(x);
+                    zs[p * P::TRI + i / C * AP + i % C] = h;
+                    x -= __bfloat162float(h);
+                }
+            }
+            if (j0 == 0) asm volatile("cp.async.wait_group 1;" ::: "memory");
+            else asm volatile("cp.async.wait_group 0;" ::: "memory");
             __syncthreads();
             for (int k = 0; k < (nj + 15) / 16; ++k) {
                 uint32_t af[3][4], bf[4];
 #pragma unroll
-                for (int p = 0; p < 3; ++p) mma_a(af[p], zs + p * P::TRI + r16 * AP + k * 16, AP, lane);
+                for (int p = 0; p < 3; ++p) mma_a(af[p], zs + p * P::TRI + z16 * AP + k * 16, AP, lane);
 #pragma unroll
                 for (int j = 0; j < XT; j += 2) {
                     mma_b_t(bf, w2 + k * 16 * KP + c0 + j * 8, KP, lane);
@@ -312,109 +394,104 @@ __global__ void __launch_bounds__(CC_THREADS, 1) channel_delta_chunk_kernel(cons
         for (int j = 0; j < XT; ++j)
 #pragma unroll
             for (int x = 0; x < 4; ++x) {
-                const int t = r16 + gid + (x >> 1) * 8, c = c0 + j * 8 + 2 * tq + (x & 1);
-                s_l[t * LP + c] = t < m && c < dim ? channel_log_decay_f(acc[j][x] + a.w0[h0 + c]) : 0.f;
+                const int t = z16 + gid + (x >> 1) * 8, c = c0 + j * 8 + 2 * tq + (x & 1);
+                s_l[t * LP + c] = t < m && c < dim ? -0.60653066f * __fdividef(1.0f, 1.0f + __expf(-acc[j][x] - w0[j][x & 1])) : 0.f;
             }
     }
     __syncthreads();
-    // ---- running sums over the rows, a quarter of the rows per thread
-    if (tid < 4 * KD) {
+    // ---- running sums over the rows, a part of them per thread, against the middle row; then their exponentials
+    constexpr int PARTS = CC_THREADS / KD, PART = C / PARTS;
+    {
         const int c = tid % KD, part = tid / KD;
-        float sum = 0.f;
+        float l[PART], sum = 0.f;
 #pragma unroll
-        for (int t = 0; t < C / 4; ++t) {
-            float* p = s_l + (part * (C / 4) + t) * LP + c;
-            sum += *p;
-            *p = sum;
-        }
+        for (int t = 0; t < PART; ++t) l[t] = sum += s_l[(part * PART + t) * LP + c];
         s_sum[part * KD + c] = sum;
-    }
-    __syncthreads();
-    if (tid < KD) {
-        const float s0 = s_sum[tid], s1 = s0 + s_sum[KD + tid], s2 = s1 + s_sum[2 * KD + tid], s3 = s2 + s_sum[3 * KD + tid];
-        s_sum[tid] = 0.f;
-        s_sum[KD + tid] = s0;
-        s_sum[2 * KD + tid] = s1;
-        s_sum[3 * KD + tid] = s2;
-        s_mid[tid] = s1;
-        s_em[tid] = expf(s1);
-        s_elm[tid] = expf(s3 - s1);
-        reinterpret_cast<float*>(out + R::DECAY)[tid] = expf(s3);
-    }
-    __syncthreads();
-    // ---- operands: a warp per row, four channels per lane and pass; values on their way to registers
-    constexpr int PASSES = (KD + 127) / 128;
-    float4 v_reg[C / CC_WARPS][PASSES];
+        __syncthreads();
+        float before = 0.f, mid = 0.f, all = 0.f;
 #pragma unroll
-    for (int i = 0; i < C / CC_WARPS; ++i) {
-        const int t = i * CC_WARPS + warp;
-        auto row4 = [&](int col, int c) {
-            float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
-            if (t >= m || c >= dim) return x;
-            if (vec) return a.y.at4(row0 + t, col + h0 + c);
-            x.x = a.y.at(row0 + t, col + h0 + c);
-            if (c + 1 < dim) x.y = a.y.at(row0 + t, col + h0 + c + 1);
-            if (c + 2 < dim) x.z = a.y.at(row0 + t, col + h0 + c + 2);
-            if (c + 3 < dim) x.w = a.y.at(row0 + t, col + h0 + c + 3);
-            return x;
-        };
-        float4 k[PASSES], r[PASSES], g[PASSES];
+        for (int p = 0; p < PARTS; ++p) {
+            const float x = s_sum[p * KD + c];
+            if (p < part) before += x;
+            if (p < PARTS / 2) mid += x;
+            all += x;
+        }
+#pragma unroll
+        for (int t = 0; t < PART; ++t) s_l[(part * PART + t) * LP + c] = expf(l[t] + (before - mid));
+        if (part == 0) {
+            s_em[c] = expf(mid);
+            s_start[c] = expf(-mid);
+            s_elm[c] = expf(all - mid);
+            reinterpret_cast<float*>(out + R::DECAY)[c] = expf(all);
+        }
+    }
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    __syncthreads();
+    // ---- operands: a warp per row; the values on their way meanwhile
+    float kr[ROWS][EL], rr[ROWS][EL], gr[ROWS][EL], vr[ROWS][EL];
+#pragma unroll
+    for (int i = 0; i < ROWS; ++i) {
+        const int t = i * CC_WARPS + warp, c = lane * EL;
+        if (plain) {
+            const float* src = a.y.p + (t < m && c < dim ? (row0 + t) * a.y.ld + a.v_col + h0 + c : 0);
+#pragma unroll
+            for (int e = 0; e < EL; e += 2) {
+                const float2 v = *reinterpret_cast<const float2*>(src + e);
+                vr[i][e] = v.x;
+                vr[i][e + 1] = v.y;
+            }
+        } else {
+#pragma unroll
+            for (int e = 0; e < EL; ++e) vr[i][e] = t < m && c + e < dim ? a.y.at(row0 + t, a.v_col + h0 + c + e) : 0.f;
+        }
+#pragma unroll
+        for (int e = 0; e < EL; ++e) {
+            kr[i][e] = raw_k[t * KD + c + e];
+            rr[i][e] = raw_r[t * KD + c + e];
+            gr[i][e] = raw_g[t * KD + c + e];
+        }
+    }
+    __syncthreads();
+#pragma unroll
+    for (int i = 0; i < ROWS; ++i) {
+        const int t = i * CC_WARPS + warp, c = lane * EL;
         float kk = 0.f;
 #pragma unroll
-        for (int p = 0; p < PASSES; ++p) {
-            const int c = p * 128 + lane * 4;
-            const bool mine = c < KD;
-            k[p] = r[p] = g[p] = v_reg[i][p] = make_float4(0.f, 0.f, 0.f, 0.f);
-            if (mine) {
-                k[p] = row4(a.k_col, c);
-                r[p] = row4(a.r_col, c);
-                g[p] = row4(a.a_col, c);
-                v_reg[i][p] = row4(a.v_col, c);
-            }
-            kk = fmaf(k[p].x, k[p].x, fmaf(k[p].y, k[p].y, fmaf(k[p].z, k[p].z, fmaf(k[p].w, k[p].w, kk))));
-        }
+        for (int e = 0; e < EL; ++e) kk = fmaf(kr[i][e], kr[i][e], kk);
         kk = warp_sum(kk);
         const float unit = 1.0f / sqrtf(kk + 1e-6f);
+        const float* now = s_l + t * LP + c;
+        const float* prev = t == 0 ? s_start + c : now - LP;
+        float q[EL], b[EL], w[EL], o[EL];
 #pragma unroll
-        for (int p = 0; p < PASSES; ++p) {
-            const int c = p * 128 + lane * 4;
-            if (c >= KD) continue;
-            const float kx[4] = {k[p].x, k[p].y, k[p].z, k[p].w}, rx[4] = {r[p].x, r[p].y, r[p].z, r[p].w}, gx[4] = {g[p].x, g[p].y, g[p].z, g[p].w};
-            float q[4], b[4], w[4], o[4];
+        for (int e = 0; e < EL; ++e) {
+            const float l = now[e], later = __fdividef(1.0f, l), u = kr[i][e] * unit;
+            q[e] = u * prev[e];
+            b[e] = __fdividef(u * later, 1.0f + __expf(-(gr[i][e] + bias[e])));
+            w[e] = kr[i][e] * later;
+            o[e] = rr[i][e] * l;
+        }
 #pragma unroll
-            for (int e = 0; e < 4; ++e) {
-                const float mid = s_mid[c + e], l = s_l[t * LP + c + e] + s_sum[t / (C / 4) * KD + c + e] - mid;
-                const float before = t == 0 ? -mid : s_l[(t - 1) * LP + c + e] + s_sum[(t - 1) / (C / 4) * KD + c + e] - mid;
-                const float later = expf(-l), u = kx[e] * unit;
-                const float rate = c + e < dim ? sigmoid_f(gx[e] + a.a_bias[h0 + c + e]) : 0.f;
-                q[e] = u * expf(before);
-                b[e] = rate * u * later;
-                w[e] = kx[e] * later;
-                o[e] = rx[e] * expf(l);
-            }
-#pragma unroll
-            for (int e = 0; e < 4; e += 2) {
-                Kq.put2(t, c + e, q[e], q[e + 1]);
-                Br.put2(t, c + e, b[e], b[e + 1]);
-                Kw.put2(t, c + e, w[e], w[e + 1]);
-                Rq.put2(t, c + e, o[e], o[e + 1]);
-            }
+        for (int e = 0; e < EL; e += 2) {
+            Kq.put2(t, c + e, q[e], q[e + 1]);
+            Br.put2(t, c + e, b[e], b[e + 1]);
+            Kw.put2(t, c + e, w[e], w[e + 1]);
+            Rq.put2(t, c + e, o[e], o[e + 1]);
         }
     }
     __syncthreads();
 #pragma unroll
-    for (int i = 0; i < C / CC_WARPS; ++i)
+    for (int i = 0; i < ROWS; ++i)
 #pragma unroll
-        for (int p = 0; p < PASSES; ++p) {
-            const int t = i * CC_WARPS + warp, c = p * 128 + lane * 4;
-            if (c >= KD) continue;
-            V.put2(t, c, v_reg[i][p].x, v_reg[i][p].y);
-            V.put2(t, c + 2, v_reg[i][p].z, v_reg[i][p].w);
+        for (int e = 0; e < EL; e += 2) {
+            const bool live = i * CC_WARPS + warp < m && lane * EL < dim;  // a pack that was not there was read from elsewhere
+            V.put2(i * CC_WARPS + warp, lane * EL + e, live ? vr[i][e] : 0.f, live ? vr[i][e + 1] : 0.f);
         }
     // ---- products of the chunk's rows among themselves, 16 x 16 per warp; what lies behind a row is zero
-    const int s16 = quarter * 16;
+    const int s16 = quarter * 16, r16 = ((warp + (quarter < 2 ? 0 : quarter)) & 3) * 16;  // the tiles that count: two or three per scheduler
     float a_kb[2][4] = {}, a_kk[2][4] = {}, a_rk[2][4] = {}, a_rb[2][4] = {};
     if (s16 <= r16) {
+#pragma unroll 2
         for (int k = 0; k < KD / 16; ++k) {
             uint32_t qh[4], ql[4], rh[4], rl[4], bh[4], bl[4], wh[4], wl[4];
             mma_a(qh, Kq.at(r16, k * 16), KP, lane);
@@ -438,7 +515,7 @@ __global__ void __launch_bounds__(CC_THREADS, 1) channel_delta_chunk_kernel(cons
             const int t = r16 + gid + (x >> 1) * 8, s = s16 + j * 8 + 2 * tq + (x & 1);
             if (s >= t) a_kb[j][x] = a_kk[j][x] = 0.f;
             if (s > t) a_rk[j][x] = a_rb[j][x] = 0.f;
-            if (s16 == r16) s_diag[(r16 / 16 * 16 + t - r16) * 17 + s - s16] = a_kb[j][x];
+            if (s16 == r16) s_diag[t * 20 + s - s16] = a_kb[j][x];
         }
     auto put_tile = [&](const Split& to, const float (&v)[2][4]) {
 #pragma unroll
@@ -451,17 +528,20 @@ __global__ void __launch_bounds__(CC_THREADS, 1) channel_delta_chunk_kernel(cons
     __syncthreads();
     // ---- inverses of the diagonal blocks, a column per lane; meanwhile what the writes alone give
     if (warp < 4 && lane < 16) {
-        const float* d = s_diag + warp * 16 * 17;
+        const float4* d = reinterpret_cast<const float4*>(s_diag + warp * 16 * 20);
         float x[16];
+        float4 next[4] = {};
 #pragma unroll
         for (int i = 0; i < 16; ++i) {
-            float v = i == lane ? 1.f : 0.f;
+            const float row[16] = {next[0].x, next[0].y, next[0].z, next[0].w, next[1].x, next[1].y, next[1].z, next[1].w,
+                                   next[2].x, next[2].y, next[2].z, next[2].w, next[3].x, next[3].y, next[3].z, next[3].w};
 #pragma unroll
-            for (int k = 0; k < i; ++k) v = fmaf(-d[i * 17 + k], x[k], v);
-            x[i] = v;
-        }
+            for (int k = 0; k < 4; ++k)
+                if (i + 1 < 16 && 4 * k < i + 1) next[k] = d[(i + 1) * 5 + k];
+            float v[4] = {i == lane ? 1.f : 0.f, 0.f, 0.f, 0.f};
 #pragma unroll
-        for (int i = 0; i < 16; ++i) {
+            for (int k = 0; k < i; ++k) v[k & 3] = fmaf(-row[k], x[k], v[k & 3]);
+            x[i] = (v[0] + v[1]) + (v[2] + v[3]);
             const __nv_bfloat16 h = __float2bfloat16_rn(x[i]);
             *Ti.at(warp * 16 + i, lane) = h;
             *(Ti.at(warp * 16 + i, lane) + Ti.rest) = __float2bfloat16_rn(x[i] - __bfloat162float(h));
@@ -475,7 +555,7 @@ __global__ void __launch_bounds__(CC_THREADS, 1) channel_delta_chunk_kernel(cons
         mma_a_t(l, A.at(k * 16, vt) + A.rest, KP, lane);
     };
     float y[YT][4] = {}, n[NT][4] = {};
-#pragma unroll
+#pragma unroll 1
     for (int k = 0; k < C / 16; ++k) {
         uint32_t ah[4], al[4], bh[4], bl[4];
         values_times(V, k, ah, al);
@@ -501,12 +581,12 @@ __global__ void __launch_bounds__(CC_THREADS, 1) channel_delta_chunk_kernel(cons
         const bool values = warp >= VT;
         const Split to = values ? Kw : Kq;
         const int c16 = (values ? warp - VT : warp) * 16;
-#pragma unroll
+#pragma unroll 1
         for (int i = 0; i < C / 16; ++i) {
             float rhs[2][4] = {}, taken[2][4] = {}, x[2][4] = {};
             uint32_t ah[4], al[4], bh[4], bl[4];
             if (values) {
-#pragma unroll
+#pragma unroll 1
                 for (int k = 0; k <= i; ++k) {
                     mma_a(ah, A2.at(i * 16, k * 16), AP, lane);
                     mma_a(al, A2.at(i * 16, k * 16) + A2.rest, AP, lane);
@@ -524,7 +604,7 @@ __global__ void __launch_bounds__(CC_THREADS, 1) channel_delta_chunk_kernel(cons
                         rhs[j][2 * h + 1] = v.y;
                     }
             }
-#pragma unroll
+#pragma unroll 1
             for (int k = 0; k < i; ++k) {
                 mma_a(ah, A1.at(i * 16, k * 16), AP, lane);
                 mma_a(al, A1.at(i * 16, k * 16) + A1.rest, AP, lane);
@@ -567,7 +647,7 @@ __global__ void __launch_bounds__(CC_THREADS, 1) channel_delta_chunk_kernel(cons
         *reinterpret_cast<uint4*>(out + at + 512 + lane * 16) = lo;
     };
     // ---- values' side: Y and N
-#pragma unroll
+#pragma unroll 1
     for (int k = 0; k < C / 16; ++k) {
         uint32_t ah[4], al[4], bh[4], bl[4];
         values_times(G, k, ah, al);
@@ -602,7 +682,7 @@ __global__ void __launch_bounds__(CC_THREADS, 1) channel_delta_chunk_kernel(cons
     // ---- state's side: M, 16 keys x NT tiles per warp, and X, 16 rows x XT tiles
     {
         float mm[NT][4] = {};
-#pragma unroll
+#pragma unroll 1
         for (int k = 0; k < C / 16; ++k) {
             uint32_t ah[4], al[4], bh[4], bl[4];
             values_times(Br, k, ah, al);
@@ -627,13 +707,13 @@ __global__ void __launch_bounds__(CC_THREADS, 1) channel_delta_chunk_kernel(cons
     }
     {
         float xx[XT][4] = {};
-        const int c0 = quarter * (KD / 4);
-#pragma unroll
+        const int c0 = quarter * (KD / 4), t16 = ((warp + quarter) & 3) * 16;  // as many rows before them for every scheduler
+#pragma unroll 1
         for (int k = 0; k < C / 16; ++k) {
-            if (k * 16 > r16) continue;
+            if (k * 16 > t16) continue;
             uint32_t ah[4], al[4], bh[4], bl[4];
-            mma_a(ah, A2.at(r16, k * 16), AP, lane);
-            mma_a(al, A2.at(r16, k * 16) + A2.rest, AP, lane);
+            mma_a(ah, A2.at(t16, k * 16), AP, lane);
+            mma_a(al, A2.at(t16, k * 16) + A2.rest, AP, lane);
 #pragma unroll
             for (int j = 0; j < XT; j += 2) {
                 mma_b_t(bh, W.at(k * 16, c0 + j * 8), KP, lane);
@@ -646,13 +726,13 @@ __global__ void __launch_bounds__(CC_THREADS, 1) channel_delta_chunk_kernel(cons
             const float2 e = *reinterpret_cast<const float2*>(s_em + c0 + j * 8 + 2 * tq);
 #pragma unroll
             for (int h = 0; h < 2; ++h) {
-                const float2 r = Rq.get2(r16 + gid + 8 * h, c0 + j * 8 + 2 * tq);
+                const float2 r = Rq.get2(t16 + gid + 8 * h, c0 + j * 8 + 2 * tq);
                 xx[j][2 * h] = (r.x - xx[j][2 * h]) * e.x;
                 xx[j][2 * h + 1] = (r.y - xx[j][2 * h + 1]) * e.y;
             }
         }
 #pragma unroll
-        for (int j = 0; j < XT; j += 2) store_pair(R::X + (r16 / 16) * R::TILE + (c0 / 8 + j) / 2 * 1024, xx[j], xx[j + 1]);
+        for (int j = 0; j < XT; j += 2) store_pair(R::X + (t16 / 16) * R::TILE + (c0 / 8 + j) / 2 * 1024, xx[j], xx[j + 1]);
     }
 }
 

@@ -226,15 +226,16 @@ __global__ void __launch_bounds__(RU_THREADS) row_update_kernel(RowUpdateArgs a)
 }
 
 // Rows of a short convolution: a CTA takes ROWS consecutive rows and the taps - 1 before them (of the first one's lane), updates them
-// all into shared memory behind one barrier for their sums of squares, and then walks its columns.  A thread reads the staged columns
-// it has written itself.
-template <int VEC, int ROWS>
+// all into shared memory behind one barrier for their sums of squares, and then walks its columns down the rows with the last taps - 1
+// normed rows in registers (TAPS > 0) or in the staged rows (any number of taps).  A thread reads the columns it has staged itself.
+template <int VEC, int ROWS, int TAPS>
 __global__ void __launch_bounds__(RU_THREADS) conv_update_kernel(RowUpdateArgs a) {
     extern __shared__ __align__(16) float cu_smem[];   // [ROWS + taps - 1][width], then [ROWS + taps - 1] sums per warp and inverse roots
     constexpr int BATCH = ROWS >= 4 ? 4 : ROWS;
     constexpr int WARPS = RU_THREADS / 32;
-    const int hist = a.taps - 1, staged = ROWS + hist, W = a.width;
+    const int taps = TAPS > 0 ? TAPS : a.taps, hist = taps - 1, staged = ROWS + hist, W = a.width;
     float* red = cu_smem + (int64_t)staged * W;
+    float* inv = red + staged * WARPS;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, step = RU_THREADS * VEC;
     pdl_trigger();
     pdl_wait();
@@ -278,62 +279,88 @@ __global__ void __launch_bounds__(RU_THREADS) conv_update_kernel(RowUpdateArgs a
         }
     }
     __syncthreads();
-    // every thread needs every row's root: each of the first threads adds one up
-    float* root = red + staged * WARPS;
+    // every thread needs every row's root: the first threads add one up each
     for (int i = threadIdx.x; i < n; i += RU_THREADS) {
         float s = 0.f;
 #pragma unroll
         for (int w = 0; w < WARPS; ++w) s += red[i * WARPS + w];
-        root[i] = sqrtf(s / (float)W + a.norm_eps);
+        inv[i] = 1.0f / sqrtf(s / (float)W + a.norm_eps);
     }
     __syncthreads();
-    for (int r = r0; r < r1; ++r) {
-        if (r >= sl.first + sl.n) sl = a.lanes.at(a.token_lane[r]);
-        const bool last = r == sl.first + sl.n - 1;
-        for (int c = threadIdx.x * VEC; c < W; c += step) {
-            const Pack<VEC> w = load_pack<VEC>(a.norm_w + c);
-            auto normed = [&](int row) {  // h of a row of the lane, or of one before this tick
-                Pack<VEC> h;
-                if (row >= sl.first) {
-                    h = load_pack<VEC>(cu_smem + (int64_t)(row - lo) * W + c);
-                    const float d = root[row - lo];
+    const StateLane first_lane = sl;
+    for (int c = threadIdx.x * VEC; c < W; c += step) {
+        const Pack<VEC> w = load_pack<VEC>(a.norm_w + c);
+        sl = first_lane;
+        auto normed = [&](int row) {  // h of a row of the lane, or of one before this tick
+            Pack<VEC> h;
+            if (row >= sl.first) {
+                h = load_pack<VEC>(cu_smem + (int64_t)(row - lo) * W + c);
+                const float d = inv[row - lo];
 #pragma unroll
-                    for (int i = 0; i < VEC; ++i) h.v[i] = h.v[i] / d * w.v[i];
-                } else if (sl.in >= 0) {
-                    h = load_pack<VEC>(a.kept + ((int64_t)sl.in * hist + hist + row - sl.first) * W + c);
-                } else {
+                for (int i = 0; i < VEC; ++i) h.v[i] = h.v[i] * d * w.v[i];
+            } else if (sl.in >= 0) {
+                h = load_pack<VEC>(a.kept + ((int64_t)sl.in * hist + hist + row - sl.first) * W + c);
+            } else {
 #pragma unroll
-                    for (int i = 0; i < VEC; ++i) h.v[i] = 0.f;
-                }
-                return h;
-            };
-            Pack<VEC> sum;
-            const Pack<VEC> own = normed(r);
-#pragma unroll
-            for (int i = 0; i < VEC; ++i) sum.v[i] = 0.f;
-#pragma unroll 4
-            for (int j = 0; j < a.taps; ++j) {
-                const Pack<VEC> k = load_pack<VEC>(a.conv + (int64_t)j * W + c);
-                const Pack<VEC> h = j == hist ? own : normed(r - hist + j);
-#pragma unroll
-                for (int i = 0; i < VEC; ++i) sum.v[i] = fmaf(k.v[i], h.v[i], sum.v[i]);
+                for (int i = 0; i < VEC; ++i) h.v[i] = 0.f;
             }
+            return h;
+        };
+        if constexpr (TAPS > 0) {
+            Pack<VEC> k[TAPS], win[TAPS];  // win[j]: h of the row TAPS - 1 - j before
 #pragma unroll
-            for (int i = 0; i < VEC; ++i) sum.v[i] += own.v[i];
-            put_pack<VEC>(a.normed, r, c, sum);
-            if (last)
-                for (int t = 0; t < hist; ++t) store_pack<VEC>(a.kept + ((int64_t)sl.out * hist + t) * W + c, normed(r - hist + 1 + t));
+            for (int j = 0; j < TAPS; ++j) k[j] = load_pack<VEC>(a.conv + (int64_t)j * W + c);
+#pragma unroll
+            for (int j = 0; j < hist; ++j) win[j + 1] = normed(r0 - hist + j);
+            for (int r = r0; r < r1; ++r) {
+                if (r >= sl.first + sl.n) {
+                    sl = a.lanes.at(a.token_lane[r]);
+#pragma unroll
+                    for (int j = 0; j < hist; ++j) win[j + 1] = normed(r - hist + j);
+                }
+#pragma unroll
+                for (int j = 0; j < hist; ++j) win[j] = win[j + 1];
+                win[hist] = normed(r);
+                Pack<VEC> sum = win[hist];
+#pragma unroll
+                for (int j = 0; j < TAPS; ++j)
+#pragma unroll
+                    for (int i = 0; i < VEC; ++i) sum.v[i] = fmaf(k[j].v[i], win[j].v[i], sum.v[i]);
+                put_pack<VEC>(a.normed, r, c, sum);
+                if (r == sl.first + sl.n - 1)
+#pragma unroll
+                    for (int t = 0; t < hist; ++t) store_pack<VEC>(a.kept + ((int64_t)sl.out * hist + t) * W + c, win[t + 1]);
+            }
+        } else {
+            for (int r = r0; r < r1; ++r) {
+                if (r >= sl.first + sl.n) sl = a.lanes.at(a.token_lane[r]);
+                Pack<VEC> sum = normed(r);
+                for (int j = 0; j < taps; ++j) {
+                    const Pack<VEC> k = load_pack<VEC>(a.conv + (int64_t)j * W + c), h = normed(r - hist + j);
+#pragma unroll
+                    for (int i = 0; i < VEC; ++i) sum.v[i] = fmaf(k.v[i], h.v[i], sum.v[i]);
+                }
+                put_pack<VEC>(a.normed, r, c, sum);
+                if (r == sl.first + sl.n - 1)
+                    for (int t = 0; t < hist; ++t) store_pack<VEC>(a.kept + ((int64_t)sl.out * hist + t) * W + c, normed(r - hist + 1 + t));
+            }
         }
-        zero_tail(a.normed, r, W);
     }
+    for (int r = r0; r < r1; ++r) zero_tail(a.normed, r, W);
+}
+
+template <int VEC, int ROWS, int TAPS>
+void launch_conv_taps(const RowUpdateArgs& a, cudaStream_t s) {
+    const size_t staged = (size_t)ROWS + a.taps - 1, smem = (staged * a.width + staged * (RU_THREADS / 32 + 1)) * 4;
+    if (smem > (size_t)220 * 1024) throw std::runtime_error("launch_row_update: the model is too wide for its short convolution");
+    ensure_dynamic_smem(reinterpret_cast<const void*>(&conv_update_kernel<VEC, ROWS, TAPS>), smem);
+    launch_pdl(conv_update_kernel<VEC, ROWS, TAPS>, dim3((unsigned)((a.rows + ROWS - 1) / ROWS)), dim3(RU_THREADS), smem, s, a);
 }
 
 template <int VEC, int ROWS>
 void launch_conv_rows(const RowUpdateArgs& a, cudaStream_t s) {
-    const size_t staged = (size_t)ROWS + a.taps - 1, smem = (staged * a.width + staged * (RU_THREADS / 32 + 1)) * 4;
-    if (smem > (size_t)220 * 1024) throw std::runtime_error("launch_row_update: the model is too wide for its short convolution");
-    ensure_dynamic_smem(reinterpret_cast<const void*>(&conv_update_kernel<VEC, ROWS>), smem);
-    launch_pdl(conv_update_kernel<VEC, ROWS>, dim3((unsigned)((a.rows + ROWS - 1) / ROWS)), dim3(RU_THREADS), smem, s, a);
+    if (a.taps == 4) launch_conv_taps<VEC, ROWS, 4>(a, s);
+    else launch_conv_taps<VEC, ROWS, 0>(a, s);
 }
 
 // ------------------------------------------------------------------------------------------------ WKV decay
