@@ -196,9 +196,11 @@ def test_the_oldest_tap_crosses_every_cut(mk, tmp_path, taps, compute):
 
 
 @pytest.mark.parametrize("compute", DTYPES)
-def test_wide_ticks_convolve_like_narrow_ones(mk, tmp_path, compute):
-    """Ticks of more rows than the kernels' small forms take, made of several lanes whose borders fall anywhere."""
-    cfg = mc.mamivik([mc.scaled_parallel((4, 2, 32, 16), (3, 40), 50, ff=64), mc.rotated_latent(4, 24, 32, 40, 64, 16, 70, ff=40)], width=72, vocab=90, taps=4)
+@pytest.mark.parametrize("heads", [(3, 40), (2, 128), (2, 30), (1, 136)])
+def test_wide_ticks_are_like_narrow_ones(mk, tmp_path, heads, compute):
+    """Ticks of more rows than the kernels' small forms take, made of several lanes whose borders fall anywhere: prompts, a few tokens
+    and single ones side by side, which take different forms of the delta rule."""
+    cfg = mc.mamivik([mc.scaled_parallel((4, 2, 32, 16), heads, 50, ff=64), mc.rotated_latent(4, 24, 32, 40, 64, 16, 70, ff=40)], width=72, vocab=90, taps=4)
     folder, oracle, _ = checkpoint(tmp_path, cfg, seed=3)
     seqs = [tokens_of(n, 90, seed=n) for n in (611, 2, 437, 53)]
     want = [oracle.logits(s) for s in seqs]
@@ -223,6 +225,37 @@ def test_wide_ticks_convolve_like_narrow_ones(mk, tmp_path, compute):
 
 
 # ------------------------------------------------------------------------------------------------ the delta rule's state
+
+@pytest.mark.parametrize("heads", [(2, 64), (3, 128), (2, 100), (3, 48)])
+@pytest.mark.parametrize("decay", [None, -12.0, 12.0])
+def test_forms_of_the_delta_rule_agree(mk, tmp_path, heads, decay):
+    """In bfloat16 models the forms differ by what a rounding of their finished rows may flip: prompts in chunks, portions that go row
+    by row, single tokens, and prompts cut at and beside a chunk's edge - with random, no and the fastest decay."""
+    cfg = mc.mamivik([mc.scaled_parallel((2, 1, 16, 8), heads, 4, scales=(0.0, 1.0))], width=96, vocab=50, taps=2)
+
+    def change(w):
+        if decay is not None:
+            w["l0.mix.right.w0"][:] = decay
+
+    folder, oracle, _ = checkpoint(tmp_path, cfg, seed=3, rank=16, change=change)
+    model = mc.load(folder, "bfloat16")
+    toks = tokens_of(330, 50, seed=1)
+    base = oracle.embedding_output(toks)
+    size = np.sqrt(np.mean((oracle.residuals(toks)[0] - base) ** 2))
+    model.capture_residuals(True)
+    out = []
+    for portions in (mc.cut(330, [1]), [330], mc.cut(330, [40]), [64, 266], [63, 65, 202], mc.cut(330, [128, 2, 49])):
+        s, at, got = model.new_session(), 0, []
+        for k in portions:
+            model.forward_batch([(s, toks[at:at + k], at)], want_logits=False, want_tokens=False, rows=[[]])
+            got.append(model.residuals(k)[0])
+            at += k
+        s.close()
+        out.append(np.concatenate(got))
+    for other in out[1:]:
+        assert np.sqrt(np.mean((other - out[0]) ** 2)) / size < 6e-4
+        assert np.sqrt(np.mean((other - out[0]) ** 2, axis=1)).max() / size < 5e-3
+    model.close()
 
 @pytest.mark.parametrize("compute", DTYPES)
 @pytest.mark.parametrize("heads", [(2, 32), (3, 64), (1, 150)])
