@@ -753,7 +753,7 @@ __device__ __forceinline__ void poly_row(const LatentPrepArgs& a, int64_t row, f
     zero_tail(a.ff_image, row, a.ff);
 }
 
-// Shared memory: max(ff, q_rank + kv_rank) floats.
+// Shared memory: max(ff, q_rank + kv_rank + rot_width) floats.
 template <int VEC>
 __global__ void __launch_bounds__(LP_THREADS) latent_prep_kernel(LatentPrepArgs a) {
     extern __shared__ __align__(16) float lp_row[];
@@ -765,36 +765,112 @@ __global__ void __launch_bounds__(LP_THREADS) latent_prep_kernel(LatentPrepArgs 
         poly_row<VEC>(a, row, lp_row, red);
         return;
     }
-    float* kv = lp_row + a.q_rank;
+    float *kv = lp_row + a.q_rank, *rot = kv + a.kv_rank;
+    const int64_t at = a.slots[row] * a.kv_width, turn0 = a.rot_dims > 0 ? (int64_t)a.positions[row] * (a.rot_dims / 2) : 0;
     float3 ss = make_float3(0.f, 0.f, 0.f);
-    for (int c = threadIdx.x; c < a.q_rank; c += LP_THREADS) {
-        const float v = a.y.at(row, a.q_col + c);
-        lp_row[c] = v;
-        ss.x = fmaf(v, v, ss.x);
-    }
-    for (int c = threadIdx.x; c < a.kv_rank; c += LP_THREADS) {
-        const float v = a.y.at(row, a.kv_col + c);
-        kv[c] = v;
-        ss.y = fmaf(v, v, ss.y);
-    }
-    ss = block_sum3(ss, red);
-    const float rq = sqrtf(ss.x / (float)a.q_rank + a.eps), rk = sqrtf(ss.y / (float)a.kv_rank + a.eps);
-    for (int c = threadIdx.x; c < a.q_rank; c += LP_THREADS) a.q_image.put(row, c, lp_row[c] / rq * a.q_norm[c]);
-    zero_tail(a.q_image, row, a.q_rank);
-    const int64_t at = a.slots[row] * a.kv_width;
-    for (int c = threadIdx.x; c < a.kv_width; c += LP_THREADS) {
-        float v = c < a.kv_rank ? kv[c] / rk * a.kv_norm[c] : 0.f;
-        const int i = c - a.rot0;
-        if (a.rot_width > 0 && i >= 0 && i < a.rot_width) {
-            v = a.y.at(row, a.rot_col + i);
-            if (i < a.rot_dims) {
-                const int64_t turn = (int64_t)a.positions[row] * (a.rot_dims / 2) + (i >> 1);
-                const float other = a.y.at(row, a.rot_col + (i ^ 1)), cs = a.cos_t[turn], sn = a.sin_t[turn];
-                v = (i & 1) == 0 ? v * cs - other * sn : v * cs + other * sn;
+    // a latent's raw values into shared memory; returns the thread's sum of squares
+    auto stage = [&](float* dst, int n, int col) {
+        float s = 0.f;
+        if (a.lat_vec) {
+            for (int c = threadIdx.x * 4; c < n; c += LP_THREADS * 4) {
+                const float4 v = a.y.at4(row, col + c);
+                *reinterpret_cast<float4*>(dst + c) = v;
+                s = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, s))));
+            }
+        } else {
+            for (int c = threadIdx.x; c < n; c += LP_THREADS) {
+                const float v = a.y.at(row, col + c);
+                dst[c] = v;
+                s = fmaf(v, v, s);
             }
         }
-        if (a.pool_f16) static_cast<__half*>(a.pool)[at + c] = __float2half_rn(v);
-        else static_cast<float*>(a.pool)[at + c] = v;
+        return s;
+    };
+    ss.x = stage(lp_row, a.q_rank, a.q_col);
+    ss.y = stage(kv, a.kv_rank, a.kv_col);
+    for (int c = threadIdx.x; c < a.rot_width; c += LP_THREADS) rot[c] = a.y.at(row, a.rot_col + c);
+    ss = block_sum3(ss, red);
+    const float rq = sqrtf(ss.x / (float)a.q_rank + a.eps), rk = sqrtf(ss.y / (float)a.kv_rank + a.eps);
+    if (a.lat_vec) {
+        for (int c = threadIdx.x * 4; c < a.q_rank; c += LP_THREADS * 4) {
+            const float4 v = *reinterpret_cast<const float4*>(lp_row + c), w = *reinterpret_cast<const float4*>(a.q_norm + c);
+            a.q_image.put4(row, c, make_float4(v.x / rq * w.x, v.y / rq * w.y, v.z / rq * w.z, v.w / rq * w.w));
+        }
+    } else {
+        for (int c = threadIdx.x; c < a.q_rank; c += LP_THREADS) a.q_image.put(row, c, lp_row[c] / rq * a.q_norm[c]);
+    }
+    zero_tail(a.q_image, row, a.q_rank);
+    auto value = [&](int c) {  // column c of the page row
+        if (c < a.kv_rank) return kv[c] / rk * a.kv_norm[c];
+        const int i = c - a.rot0;
+        if (i < 0 || i >= a.rot_width) return 0.f;
+        if (i >= a.rot_dims) return rot[i];
+        const float cs = a.cos_t[turn0 + (i >> 1)], sn = a.sin_t[turn0 + (i >> 1)];
+        return (i & 1) == 0 ? rot[i] * cs - rot[i ^ 1] * sn : rot[i] * cs + rot[i ^ 1] * sn;
+    };
+    for (int c = threadIdx.x * 2; c < a.kv_width; c += LP_THREADS * 2) {  // a row is a multiple of 64 wide
+        const float x = value(c), y = value(c + 1);
+        if (a.pool_f16) *reinterpret_cast<__half2*>(static_cast<__half*>(a.pool) + at + c) = __floats2half2_rn(x, y);
+        else *reinterpret_cast<float2*>(static_cast<float*>(a.pool) + at + c) = make_float2(x, y);
+    }
+}
+
+// The latents of wide ticks, a warp per row: in whole packs of a finished matmul, read twice (the second time out of the cache).
+__global__ void __launch_bounds__(LP_THREADS) latent_rows_kernel(LatentPrepArgs a) {
+    pdl_trigger();
+    pdl_wait();
+    const int lane = threadIdx.x & 31;
+    const int64_t row = (int64_t)blockIdx.x * (LP_THREADS / 32) + (threadIdx.x >> 5);
+    if (row >= a.rows) return;
+    const float* y = a.y.p + row * a.y.ld;
+    const int64_t at = a.slots[row] * a.kv_width, turn0 = a.rot_dims > 0 ? (int64_t)a.positions[row] * (a.rot_dims / 2) : 0;
+    auto squares = [&](int n, int col) {
+        float s = 0.f;
+#pragma unroll 8
+        for (int c = lane * 4; c < n; c += 128) {
+            const float4 v = *reinterpret_cast<const float4*>(y + col + c);
+            s = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, s))));
+        }
+        return s;
+    };
+    float sq = squares(a.q_rank, a.q_col), sk = squares(a.kv_rank, a.kv_col);
+    sq = warp_sum(sq);
+    sk = warp_sum(sk);
+    const float rq = sqrtf(sq / (float)a.q_rank + a.eps), rk = sqrtf(sk / (float)a.kv_rank + a.eps);
+#pragma unroll 4
+    for (int c = lane * 4; c < a.q_image.end(); c += 128) {
+        float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (c < a.q_rank) {
+            const float4 x = *reinterpret_cast<const float4*>(y + a.q_col + c), w = *reinterpret_cast<const float4*>(a.q_norm + c);
+            v = make_float4(x.x / rq * w.x, x.y / rq * w.y, x.z / rq * w.z, x.w / rq * w.w);
+        }
+        a.q_image.put4(row, c, v);
+    }
+    auto rotated = [&](int i) {
+        const float v = y[a.rot_col + i];
+        if (i >= a.rot_dims) return v;
+        const float other = y[a.rot_col + (i ^ 1)], cs = a.cos_t[turn0 + (i >> 1)], sn = a.sin_t[turn0 + (i >> 1)];
+        return (i & 1) == 0 ? v * cs - other * sn : v * cs + other * sn;
+    };
+#pragma unroll 4
+    for (int c = lane * 4; c < a.kv_width; c += 128) {
+        float v[4] = {};
+        if (c < a.kv_rank) {
+            const float4 x = *reinterpret_cast<const float4*>(y + a.kv_col + c), w = *reinterpret_cast<const float4*>(a.kv_norm + c);
+            v[0] = x.x / rk * w.x; v[1] = x.y / rk * w.y; v[2] = x.z / rk * w.z; v[3] = x.w / rk * w.w;
+        } else {
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                const int i = c + e - a.rot0;
+                if (i >= 0 && i < a.rot_width) v[e] = rotated(i);
+            }
+        }
+        if (a.pool_f16) {
+            const __half2 lo = __floats2half2_rn(v[0], v[1]), hi = __floats2half2_rn(v[2], v[3]);
+            *reinterpret_cast<uint2*>(static_cast<__half*>(a.pool) + at + c) = make_uint2(*reinterpret_cast<const uint32_t*>(&lo), *reinterpret_cast<const uint32_t*>(&hi));
+        } else {
+            *reinterpret_cast<float4*>(static_cast<float*>(a.pool) + at + c) = make_float4(v[0], v[1], v[2], v[3]);
+        }
     }
 }
 
@@ -957,9 +1033,17 @@ void launch_embed_norm(const EmbedNormArgs& a, cudaStream_t s) {
     MK_LAUNCH_CHECK();
 }
 
-void launch_latent_prep(const LatentPrepArgs& a, cudaStream_t s) {
+void launch_latent_prep(const LatentPrepArgs& in, cudaStream_t s) {
+    LatentPrepArgs a = in;
     if (a.rows <= 0 || (a.q_rank == 0 && a.ff == 0)) return;
-    const size_t smem = (size_t)std::max(a.ff, a.q_rank + a.kv_rank) * 4;
+    a.lat_vec = a.q_rank % 4 == 0 && a.kv_rank % 4 == 0 && a.q_col % 4 == 0 && a.kv_col % 4 == 0 && a.y.ld % 4 == 0 && a.y.stride % 4 == 0 &&
+                (reinterpret_cast<uintptr_t>(a.y.p) & 15) == 0 ? 1 : 0;
+    if (a.ff == 0 && a.lat_vec && a.y.n == 1 && a.rows > 256) {
+        launch_pdl(latent_rows_kernel, dim3((unsigned)((a.rows + LP_THREADS / 32 - 1) / (LP_THREADS / 32))), dim3(LP_THREADS), 0, s, a);
+        MK_LAUNCH_CHECK();
+        return;
+    }
+    const size_t smem = (size_t)std::max(a.ff, a.q_rank + a.kv_rank + a.rot_width) * 4;
     if (smem > (size_t)220 * 1024) throw std::runtime_error("launch_latent_prep: the feed-forward or the latents are too wide");
     const bool vec = a.ff % 4 == 0 && a.ff_col % 4 == 0 && a.y.ld % 4 == 0 && a.y.stride % 4 == 0 && (reinterpret_cast<uintptr_t>(a.y.p) & 15) == 0;
     const dim3 grid((unsigned)a.rows, a.q_rank > 0 && a.ff > 0 ? 2u : 1u);

@@ -148,6 +148,7 @@ struct LatentPrepArgs {
     int rot_col = 0, rot0 = 0, rot_width = 0, rot_dims = 0;
     const float *cos_t = nullptr, *sin_t = nullptr;  // [positions][rot_dims / 2]
     const int32_t* positions = nullptr;
+    int lat_vec = 0;                            // the latents lie in whole 16-byte packs (filled in by the launcher)
     int ff_col = 0, ff = 0;
     const float* ff_bias = nullptr;
     const float* poly = nullptr;                // [4]
