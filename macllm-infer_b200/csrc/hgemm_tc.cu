@@ -260,7 +260,8 @@ __device__ __forceinline__ float hg_gelu_tanh(float x) {
     return 0.5f * x * (1.0f + tanhf(0.7978845608028654f * x * (1.0f + 0.044715f * x * x)));
 }
 
-template <int BN, int STAGES>
+// GATED: scattered results are multiplied by a gate (MatmulScatter::gate).
+template <int BN, int STAGES, bool GATED>
 __global__ void __launch_bounds__(HG_THREADS, 1)
 hgemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__ CUtensorMap tm_x, const __grid_constant__ CUtensorMap tm_w1,
                 const __grid_constant__ CUtensorMap tm_x1, const __grid_constant__ HgParams p) {
@@ -475,7 +476,7 @@ hgemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant_
         const int quad = warp & 3, odd_group = (warp - 2) >> 2;
         const int etid = (int)threadIdx.x - 64;  // among the epilogue threads
         const bool plain = p.out_scale == 1.0f && p.softcap == 0.f;
-        if (p.part[0].act_post != nullptr || (p.scattered != 0 && p.scatter.gate != nullptr)) pdl_wait();   // the factors of the rows come from a predecessor
+        if (GATED || p.part[0].act_post != nullptr) pdl_wait();   // the factors of the rows, or the gates, come from a predecessor
         uint32_t tile_it = 0;
         for (int item = blockIdx.x; item < total_items; item += gridDim.x, ++tile_it) {
             HgTile tile;
@@ -517,16 +518,6 @@ hgemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant_
                 uint32_t r[32];
                 tmem_ld32(tmem_base + ((uint32_t)(quad * 32) << 16) + acc * BN + (uint32_t)cb, r);
                 asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
-                if (p.scattered != 0 && p.scatter.gate != nullptr && row < tile.rows && p.scatter.column(row) >= 0) {
-                    float z[8];
-#pragma unroll
-                    for (int i0 = 0; i0 < 32; i0 += 8) {
-#pragma unroll
-                        for (int i = 0; i < 8; ++i) z[i] = tok0 + cb + i0 + i < tile.tok_end ? p.scatter.gate_sum(tok0 + cb + i0 + i, row) : 0.f;
-#pragma unroll
-                        for (int i = 0; i < 8; ++i) r[i0 + i] = __float_as_uint(__uint_as_float(r[i0 + i]) * hg_sigmoid(z[i]));
-                    }
-                }
                 if (p.gated != 0) {
                     // lanes 2i / 2i+1 hold gate / up of one feature: the even lane finishes the even token columns,
                     // the odd lane the odd ones, after one exchange per pair of columns
@@ -563,13 +554,29 @@ hgemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant_
                         for (int i = 0; i < 32; ++i, out += p.scatter.ld_rest)
                             if (tok0 + cb + i < tile.tok_end) *out = __uint_as_float(r[i]);
                     }
-                } else if (p.scattered != 0 && p.scatter.type == MatmulScatter::BF16 && p.scatter.row_map == nullptr && p.scatter.block_shift == 31) {
+                } else if (p.scattered != 0 && p.scatter.type == MatmulScatter::BF16 && p.scatter.row_map == nullptr && p.scatter.block_shift == 31 && !GATED) {
                     const int64_t col = row < tile.rows ? p.scatter.column(row) : -1;
                     if (col >= 0) {
                         __nv_bfloat16* out = static_cast<__nv_bfloat16*>(p.scatter.out) + (int64_t)(tok0 + cb) * p.scatter.ld_row + col;
 #pragma unroll
                         for (int i = 0; i < 32; ++i, out += p.scatter.ld_row)
                             if (tok0 + cb + i < tile.tok_end) *out = __float2bfloat16_rn(__uint_as_float(r[i]));
+                    }
+                } else if (GATED && p.scattered != 0) {
+                    const int64_t col = row < tile.rows ? p.scatter.column(row) : -1;
+                    if (col >= 0) {
+#pragma unroll 1
+                        for (int i0 = 0; i0 < 32; i0 += 8) {  // the gates of eight tokens on their way together
+                            float z[8];
+#pragma unroll
+                            for (int i = 0; i < 8; ++i) z[i] = tok0 + cb + i0 + i < tile.tok_end ? p.scatter.gate_sum(tok0 + cb + i0 + i, row) : 0.f;
+#pragma unroll
+                            for (int i = 0; i < 8; ++i) {
+                                const int tok = tok0 + cb + i0 + i;
+                                const float v = __uint_as_float(i0 == 0 ? r[i] : (i0 == 8 ? r[8 + i] : (i0 == 16 ? r[16 + i] : r[24 + i])));
+                                if (tok < tile.tok_end) p.scatter.put(p.scatter.row(tok) + col, v * hg_sigmoid(z[i]));
+                            }
+                        }
                     }
                 } else if (p.scattered != 0) {
                     const int64_t col = row < tile.rows ? p.scatter.column(row) : -1;
@@ -644,8 +651,9 @@ void encode_half_matrix(CUtensorMap* out, const void* base, int64_t n_rows, int6
 template <int BN, int STAGES>
 void launch_hg(const CUtensorMap& tw, const CUtensorMap& tx, const CUtensorMap& tw1, const CUtensorMap& tx1, const HgParams& p, int grid, cudaStream_t s) {
     constexpr size_t smem = HgSmem<BN, STAGES>::TOTAL;
-    ensure_dynamic_smem(reinterpret_cast<const void*>(&hgemm_tc_kernel<BN, STAGES>), smem);
-    launch_pdl(hgemm_tc_kernel<BN, STAGES>, dim3(grid), dim3(HG_THREADS), smem, s, tw, tx, tw1, tx1, p);
+    auto* kernel = p.scattered != 0 && p.scatter.gate != nullptr ? hgemm_tc_kernel<BN, STAGES, true> : hgemm_tc_kernel<BN, STAGES, false>;
+    ensure_dynamic_smem(reinterpret_cast<const void*>(kernel), smem);
+    launch_pdl(kernel, dim3(grid), dim3(HG_THREADS), smem, s, tw, tx, tw1, tx1, p);
     MK_LAUNCH_CHECK();
 }
 
